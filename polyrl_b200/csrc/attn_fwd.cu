@@ -14,7 +14,7 @@
 //                          two passes over its 64 scores in TMEM (max — exchanged with the other group through shared
 //                          memory and one 256-thread named barrier — then exp2 / sum), P_j written as bf16 into the
 //                          128B-swizzled K-major layout the MMA reads, running output half kept in 64 fp32 registers:
-//                          O = O * alpha + PV_j  (PV_j read back from TMEM).  exp2 is a single MUFU.EX2.
+//                          O = O * alpha + PV_j  (PV_j read back from TMEM).  exp2 is ex2.approx.
 // Epilogue: O / l -> bf16 (16-byte stores), log-sum-exp per (head, token) for the backward pass.
 #include "common.cuh"
 

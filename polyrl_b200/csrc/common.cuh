@@ -326,7 +326,7 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
-// single MUFU.EX2 (no range-reduction branches): 2^-inf = 0, fine for softmax weights
+// ex2.approx (no range-reduction branches): 2^-inf = 0, fine for softmax weights
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

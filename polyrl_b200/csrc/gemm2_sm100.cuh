@@ -25,7 +25,7 @@
 //
 // Epilogues: (a) functor mode — same `Epi` interface as gemm_sm100.cuh (SwiGLU, linear-CE, ...);
 // (b) TMA-store mode — accumulators -> bf16 -> 128B-swizzled shared staging -> `cp.async.bulk.tensor`
-// store (UTMASTG), optional fused residual add; each epilogue warp double-buffers its own 32 x 64
+// store, optional fused residual add; each epilogue warp double-buffers its own 32 x 64
 // box so no cross-warp barrier is needed.
 #pragma once
 #include "gemm_sm100.cuh"
