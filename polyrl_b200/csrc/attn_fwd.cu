@@ -1,4 +1,4 @@
-// polyrl_b200 — varlen causal flash-attention FORWARD on tcgen05 / TMEM / TMA (head_dim 128, GQA).
+// polyrl_b200 — varlen causal flash-attention FORWARD on tcgen05 / TMEM / TMA (query / key width 128 or 192, value width 128, GQA).
 //
 // Replaces the flash-attn 2 library call (mma.sync) the reference reaches through
 // 3rdparty/verl/verl/models/transformers/monkey_patch.py:49-117 (`_flash_attention_forward`) for training,
@@ -15,6 +15,9 @@
 //                          memory and one 256-thread named barrier — then exp2 / sum), P_j written as bf16 into the
 //                          128B-swizzled K-major layout the MMA reads, running output half kept in 64 fp32 registers:
 //                          O = O * alpha + PV_j  (PV_j read back from TMEM).  exp2 is ex2.approx.
+// DK = 192 (latent attention expanded to heads: 128 + 64 rotary) keeps both K stages and drops to one V stage, which is
+// reloaded while the next scores and their softmax run.  An optional per-head sink adds exp(sink_h) to the softmax
+// denominator in the epilogue.
 // Epilogue: O / l -> bf16 (16-byte stores), log-sum-exp per (head, token) for the backward pass.
 #include "common.cuh"
 
@@ -23,7 +26,12 @@ namespace prl {
 constexpr int kAfThreads = 320;          // warp0 TMA, warp1 MMA, warps 2-5 + 6-9: two softmax warpgroups
 constexpr int kAfBM = 128, kAfBN = 128, kAfD = 128;
 constexpr int kAfTile = 128 * 128 * 2;              // 32 KB: one 128 x 128 bf16 operand tile (2 chunks of 64 columns)
-constexpr int kAfSmem = kAfTile /*Q*/ + 2 * 2 * kAfTile /*K,V x 2 stages*/ + kAfTile /*P*/ + 1024 + 256;
+template <int DK>
+struct AfCfg {
+  static constexpr int QKT = 128 * DK * 2;            // Q or K tile: DK / 64 chunks of 128 rows x 64 columns
+  static constexpr int VST = DK == 128 ? 2 : 1;       // V stages
+  static constexpr int SMEM = 3 * QKT /*Q, K x 2*/ + VST * kAfTile /*V*/ + kAfTile /*P*/ + 1024 + 256;
+};
 
 struct AttnFwdParams {
   __nv_bfloat16* o;            // [Tq, ldo]
@@ -35,29 +43,33 @@ struct AttnFwdParams {
   float scale_log2;            // sm_scale * log2(e)
   float sm_scale;
   int causal;
+  const float* sink;           // [nq] or null: natural-log sink of the softmax denominator
   long long* dbg;              // optional timeline buffer (kernel experiments)
 };
 
+template <int DK>
 __global__ void __launch_bounds__(kAfThreads, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, AttnFwdParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
-  uint8_t* sK = smem + kAfTile;                       // [2 stages]
-  uint8_t* sV = smem + 3 * kAfTile;                   // [2 stages]
-  uint8_t* sP = smem + 5 * kAfTile;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 6 * kAfTile);
+  constexpr int QKT = AfCfg<DK>::QKT, VST = AfCfg<DK>::VST;
+  uint8_t* sK = smem + QKT;                           // [2 stages]
+  uint8_t* sV = smem + 3 * QKT;                       // [VST stages]
+  uint8_t* sP = sV + VST * kAfTile;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + kAfTile);
   uint64_t* q_full = bars;            // 1
   uint64_t* k_full = bars + 1;        // [2]
   uint64_t* v_full = bars + 3;        // [2]
-  uint64_t* kv_empty = bars + 5;      // [2]
+  uint64_t* k_empty = bars + 5;       // [2]
   uint64_t* s_full = bars + 7;        // [2]
   uint64_t* s_empty = bars + 9;       // [2]  (128 arrivals)
   uint64_t* p_full = bars + 11;       // 128 arrivals
   uint64_t* o_full = bars + 12;       // 1
   uint64_t* o_empty = bars + 13;      // 128 arrivals
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
+  uint64_t* v_empty = bars + 14;      // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
   __shared__ int s_seq, s_q0;
   __shared__ float s_mx[2][2][128];             // [tile parity][warpgroup][row]: half-row maxima / sums
 
@@ -91,7 +103,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
     mbar_init(q_full, 1);
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&kv_empty[i], 1);
+      mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&k_empty[i], 1); mbar_init(&v_empty[i], 1);
       mbar_init(&s_full[i], 1); mbar_init(&s_empty[i], 256);
     }
     mbar_init(p_full, 256); mbar_init(o_full, 1); mbar_init(o_empty, 256);
@@ -106,19 +118,21 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 
   if (warp == 0) {
     if (lane == 0) {
-      mbar_expect_tx(q_full, kAfTile);
-      tma_load_2d(&tmQ, q_full, sQ, h * kAfD, qs + q0);
-      tma_load_2d(&tmQ, q_full, sQ + 16384, h * kAfD + 64, qs + q0);
+      mbar_expect_tx(q_full, QKT);
+#pragma unroll
+      for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmQ, q_full, sQ + c * 16384, h * DK + c * 64, qs + q0);
       for (int j = 0; j < nt; ++j) {
         const int s = j & 1;
         const uint32_t ph = (j >> 1) & 1;
-        mbar_wait(&kv_empty[s], ph ^ 1);
-        mbar_expect_tx(&k_full[s], kAfTile);
-        tma_load_2d(&tmK, &k_full[s], sK + s * kAfTile, hk * kAfD, ks + j * kAfBN);
-        tma_load_2d(&tmK, &k_full[s], sK + s * kAfTile + 16384, hk * kAfD + 64, ks + j * kAfBN);
-        mbar_expect_tx(&v_full[s], kAfTile);
-        tma_load_2d(&tmV, &v_full[s], sV + s * kAfTile, hk * kAfD, ks + j * kAfBN);
-        tma_load_2d(&tmV, &v_full[s], sV + s * kAfTile + 16384, hk * kAfD + 64, ks + j * kAfBN);
+        const int sv = j % VST;
+        mbar_wait(&k_empty[s], ph ^ 1);
+        mbar_expect_tx(&k_full[s], QKT);
+#pragma unroll
+        for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmK, &k_full[s], sK + s * QKT + c * 16384, hk * DK + c * 64, ks + j * kAfBN);
+        mbar_wait(&v_empty[sv], ((j / VST) & 1) ^ 1);
+        mbar_expect_tx(&v_full[sv], kAfTile);
+        tma_load_2d(&tmV, &v_full[sv], sV + sv * kAfTile, hk * kAfD, ks + j * kAfBN);
+        tma_load_2d(&tmV, &v_full[sv], sV + sv * kAfTile + 16384, hk * kAfD + 64, ks + j * kAfBN);
       }
     }
   } else if (warp == 1) {
@@ -131,9 +145,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         mbar_wait(&s_empty[s], ((j >> 1) & 1) ^ 1);
         tc_fence_after();
 #pragma unroll
-        for (int kk = 0; kk < 8; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
           const uint64_t da = umma_desc_sw128_kmajor(sQ + (kk >> 2) * 16384) + 2 * (kk & 3);
-          const uint64_t db = umma_desc_sw128_kmajor(sK + s * kAfTile + (kk >> 2) * 16384) + 2 * (kk & 3);
+          const uint64_t db = umma_desc_sw128_kmajor(sK + s * QKT + (kk >> 2) * 16384) + 2 * (kk & 3);
           umma_bf16_ss(tS0 + s * 128, da, db, idS, kk != 0);
         }
         umma_commit(&s_full[s]);
@@ -144,17 +158,19 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         const int s = j & 1;
         if (j + 1 < nt) issue_s(j + 1);
         mbar_wait(p_full, j & 1);
-        mbar_wait(&v_full[s], (j >> 1) & 1);
+        const int sv = j % VST;
+        mbar_wait(&v_full[sv], (j / VST) & 1);
         mbar_wait(o_empty, (j & 1) ^ 1);
         tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk) {
           const uint64_t da = umma_desc_sw128_kmajor(sP + (kk >> 2) * 16384) + 2 * (kk & 3);
-          const uint64_t db = umma_desc_sw128_mnmajor(sV + s * kAfTile, 16384) + kk * 128;
+          const uint64_t db = umma_desc_sw128_mnmajor(sV + sv * kAfTile, 16384) + kk * 128;
           umma_bf16_ss(tO, da, db, idO, kk != 0);
         }
         umma_commit(o_full);
-        umma_commit(&kv_empty[s]);
+        umma_commit(&k_empty[s]);
+        umma_commit(&v_empty[sv]);
       }
     }
   } else {
@@ -268,7 +284,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     // total row sum = the two groups' partial sums (same running max on both sides)
     s_mx[0][g][r] = l_run;
     asm volatile("bar.sync 1, 256;" ::: "memory");
-    const float l_tot = l_run + s_mx[0][g ^ 1][r];
+    float l_tot = l_run + s_mx[0][g ^ 1][r];
+    if (p.sink != nullptr && m_run != -INFINITY) l_tot += fast_exp2(p.sink[h] * 1.4426950408889634f - m_run * p.scale_log2);
     if (qrow < lq) {
       const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
       __nv_bfloat16* dst = p.o + static_cast<int64_t>(qs + qrow) * p.ldo + h * kAfD + g * 64;
@@ -320,17 +337,31 @@ int af_tmap(CUtensorMap* m, const void* ptr, uint64_t rows, uint64_t cols, uint6
 
 using namespace prl;
 
-// q:[Tq, nq*128] (pitch ldq), k/v:[Tk, nkv*128] (pitches ldk/ldv), o:[Tq, nq*128] (pitch ldo); pitches in ELEMENTS.
-// cu_q / cu_k: int32 [B+1] device arrays.  max_tiles: upper bound on sum_b ceil(lq_b / 128) (e.g. Tq/128 + B).
+template <int DK>
+static int run_attn_fwd(const void* q, const void* k, const void* v, const AttnFwdParams& p, int Tk, int64_t ldq, int64_t ldk, int64_t ldv,
+                        int max_tiles, cudaStream_t stream) {
+  CUtensorMap tmQ, tmK, tmV;
+  if (af_tmap(&tmQ, q, p.Tq, static_cast<uint64_t>(p.nq) * DK, ldq * 2, kAfBM)) return -111;
+  if (af_tmap(&tmK, k, Tk, static_cast<uint64_t>(p.nkv) * DK, ldk * 2, kAfBN)) return -112;
+  if (af_tmap(&tmV, v, Tk, static_cast<uint64_t>(p.nkv) * kAfD, ldv * 2, kAfBN)) return -113;
+  static bool attr = false;
+  if (!attr) {
+    PRL_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, AfCfg<DK>::SMEM));
+    attr = true;
+  }
+  attn_fwd_kernel<DK><<<dim3(max_tiles, p.nq), kAfThreads, AfCfg<DK>::SMEM, stream>>>(tmQ, tmK, tmV, p);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// q:[Tq, nq*dk] (pitch ldq), k:[Tk, nkv*dk], v:[Tk, nkv*128] (pitches ldk/ldv), o:[Tq, nq*128] (pitch ldo); pitches in ELEMENTS;
+// dk = 128 or 192.  cu_q / cu_k: int32 [B+1] device arrays.  max_tiles: upper bound on sum_b ceil(lq_b / 128) (e.g. Tq/128 + B).
+// sink: fp32 [nq] or null.
 extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o, float* lse, const int32_t* cu_q,
-                            const int32_t* cu_k, int B, int Tq, int Tk, int nq, int nkv, int64_t ldq, int64_t ldk, int64_t ldv,
-                            int64_t ldo, float sm_scale, int causal, int max_tiles, long long* dbg, cudaStream_t stream) {
+                            const int32_t* cu_k, int B, int Tq, int Tk, int nq, int nkv, int dk, int64_t ldq, int64_t ldk, int64_t ldv,
+                            int64_t ldo, float sm_scale, int causal, int max_tiles, const float* sink, long long* dbg, cudaStream_t stream) {
   if (Tq <= 0 || B <= 0) return 0;
   if (nq % nkv != 0) return -110;
-  CUtensorMap tmQ, tmK, tmV;
-  if (af_tmap(&tmQ, q, Tq, static_cast<uint64_t>(nq) * kAfD, ldq * 2, kAfBM)) return -111;
-  if (af_tmap(&tmK, k, Tk, static_cast<uint64_t>(nkv) * kAfD, ldk * 2, kAfBN)) return -112;
-  if (af_tmap(&tmV, v, Tk, static_cast<uint64_t>(nkv) * kAfD, ldv * 2, kAfBN)) return -113;
   AttnFwdParams p;
   p.o = static_cast<__nv_bfloat16*>(o);
   p.lse = lse;
@@ -339,14 +370,9 @@ extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o
   p.sm_scale = sm_scale;
   p.scale_log2 = sm_scale * 1.4426950408889634f;
   p.causal = causal;
+  p.sink = sink;
   p.dbg = dbg;
-  static bool attr = false;
-  if (!attr) {
-    PRL_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kAfSmem));
-    attr = true;
-  }
-  dim3 grid(max_tiles, nq);
-  attn_fwd_kernel<<<grid, kAfThreads, kAfSmem, stream>>>(tmQ, tmK, tmV, p);
-  PRL_CUDA_CHECK(cudaGetLastError());
-  return 0;
+  if (dk == 128) return run_attn_fwd<128>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 192) return run_attn_fwd<192>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  return -114;
 }

@@ -1,18 +1,13 @@
 // polyrl_b200 — Python bindings (pybind11 through torch) for the sm_100a kernels in csrc/*.cu.
 // Kernel translation units are torch-free (raw pointers + cudaStream_t) so they compile in seconds;
-// this file is the only one that sees torch headers.
-#include <ATen/cuda/CUDAContext.h>
-#include "kv_manager.hpp"
-#include "scheduler.hpp"
-#include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+// only the bindings*.cpp files see torch headers (bindings_serve.cpp: what serving needs).
+#include "bindings_common.hpp"
 
 #include <cstdint>
 #include <string>
 #include <vector>
 
 extern "C" {
-int prl_gemm_bf16(const void*, const void*, void*, const void*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
 int prl_gemm2_bf16(const void*, const void*, void*, const void*, int, int, int, int64_t, int64_t, int64_t, int, int, int, cudaStream_t);
 int prl_gemm2_bf16_accum_f32(const void*, const void*, float*, float, int, int, int, int64_t, int64_t, int64_t, int, int, cudaStream_t);
 int prl_gemm_fp8(const void*, const void*, void*, const float*, const float*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
@@ -31,9 +26,6 @@ int prl_sumsq(const float*, int64_t, float*, cudaStream_t);
 int prl_adamw(float*, float*, float*, float*, void*, int64_t, float, float, float, float, float, int, float, const float*, int*, int, cudaStream_t);
 int prl_paged_decode_workspace_floats(int, int, int, int);
 int prl_paged_decode(const void*, int64_t, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, float, int, float*, void*, int64_t, cudaStream_t);
-int prl_sample(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int64_t*, float*, cudaStream_t);
-int prl_sample_topk_topp(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int, float, int64_t*, float*, cudaStream_t);
-int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int32_t*, const int32_t*, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, float, int, int, long long*, cudaStream_t);
 int prl_attn_bwd(const void*, const void*, const void*, const void*, const void*, const float*, float*, float*, void*, void*, const int32_t*, const int32_t*, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, int64_t, float, int, int, cudaStream_t);
 int prl_ipc_get_handle(void*, void*);
 int prl_ipc_open_handle(const void*, void**);
@@ -78,37 +70,8 @@ int prl_ag_gemm_bf16(const void*, void* const*, void*, void*, uint32_t*, uint32_
 
 namespace {
 
-inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
 std::vector<void*> to_ptrs(const std::vector<int64_t>& v);
 
-inline void check(int rc, const char* what) {
-  TORCH_CHECK(rc == 0, "polyrl_b200 kernel '", what, "' failed with code ", rc);
-}
-#define CHECK_BF16(t) TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kBFloat16, #t " must be a CUDA bf16 tensor")
-#define CHECK_F32(t) TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kFloat, #t " must be a CUDA fp32 tensor")
-#define CHECK_LASTDIM(t) TORCH_CHECK((t).stride(-1) == 1, #t " must be contiguous in the last dim")
-
-at::Tensor gemm_bf16(const at::Tensor& a, const at::Tensor& b, const c10::optional<at::Tensor>& residual,
-                     c10::optional<at::Tensor> out, int64_t force_bn) {
-  CHECK_BF16(a); CHECK_BF16(b);
-  TORCH_CHECK(a.dim() == 2 && b.dim() == 2 && a.size(1) == b.size(1), "gemm_bf16: A[M,K] B[N,K]");
-  CHECK_LASTDIM(a); CHECK_LASTDIM(b);
-  const int M = a.size(0), K = a.size(1), N = b.size(0);
-  TORCH_CHECK(K % 8 == 0 && N % 8 == 0, "K and N must be multiples of 8");
-  TORCH_CHECK(a.stride(0) % 8 == 0 && b.stride(0) % 8 == 0, "row pitch must be a multiple of 8 elements");
-  c10::cuda::CUDAGuard g(a.device());
-  at::Tensor d = out.has_value() ? *out : at::empty({M, N}, a.options());
-  CHECK_BF16(d); CHECK_LASTDIM(d);
-  const void* r = nullptr;
-  if (residual.has_value()) {
-    CHECK_BF16(*residual);
-    TORCH_CHECK(residual->sizes() == d.sizes() && residual->stride(0) == d.stride(0) && residual->stride(1) == 1);
-    r = residual->data_ptr();
-  }
-  check(prl_gemm_bf16(a.data_ptr(), b.data_ptr(), d.data_ptr(), r, M, N, K, a.stride(0), b.stride(0), d.stride(0),
-                      static_cast<int>(force_bn), cur_stream()), "gemm_bf16");
-  return d;
-}
 
 // CTA-pair (cta_group::2) GEMM family.  D[M,N] = sum_k A(m,k) B(n,k) (+residual).
 //   a_mn=false: a is [M,K];  a_mn=true: a is [K,M] (consumed MN-major, never transposed in memory)
@@ -348,68 +311,7 @@ at::Tensor paged_decode(const at::Tensor& q, const at::Tensor& k_cache, const at
   return o;
 }
 
-std::vector<at::Tensor> sample(const at::Tensor& logits, const c10::optional<at::Tensor>& inv_temp,
-                               const c10::optional<at::Tensor>& seeds, bool greedy) {
-  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1);
-  const int dt = logits.scalar_type() == at::kFloat ? 0 : 1;
-  TORCH_CHECK(dt == 0 || logits.scalar_type() == at::kBFloat16);
-  const int B = logits.size(0), V = logits.size(1);
-  c10::cuda::CUDAGuard g(logits.device());
-  at::Tensor tok = at::empty({B}, logits.options().dtype(at::kLong));
-  at::Tensor lp = at::empty({B}, logits.options().dtype(at::kFloat));
-  const uint64_t* sd = nullptr;
-  if (seeds.has_value()) { TORCH_CHECK(seeds->scalar_type() == at::kLong); sd = reinterpret_cast<const uint64_t*>(seeds->data_ptr<int64_t>()); }
-  check(prl_sample(logits.data_ptr(), dt, logits.stride(0), B, V,
-                   inv_temp.has_value() ? inv_temp->data_ptr<float>() : nullptr, sd, greedy ? 1 : 0,
-                   tok.data_ptr<int64_t>(), lp.data_ptr<float>(), cur_stream()), "sample");
-  return {tok, lp};
-}
-
-std::vector<at::Tensor> sample_topk_topp(const at::Tensor& logits, const c10::optional<at::Tensor>& inv_temp,
-                                         const c10::optional<at::Tensor>& seeds, bool greedy, int64_t top_k, double top_p) {
-  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1);
-  const int dt = logits.scalar_type() == at::kFloat ? 0 : 1;
-  TORCH_CHECK(dt == 0 || logits.scalar_type() == at::kBFloat16);
-  const int B = logits.size(0), V = logits.size(1);
-  c10::cuda::CUDAGuard g(logits.device());
-  at::Tensor tok = at::empty({B}, logits.options().dtype(at::kLong));
-  at::Tensor lp = at::empty({B}, logits.options().dtype(at::kFloat));
-  const uint64_t* sd = nullptr;
-  if (seeds.has_value()) { TORCH_CHECK(seeds->scalar_type() == at::kLong); sd = reinterpret_cast<const uint64_t*>(seeds->data_ptr<int64_t>()); }
-  check(prl_sample_topk_topp(logits.data_ptr(), dt, logits.stride(0), B, V,
-                             inv_temp.has_value() ? inv_temp->data_ptr<float>() : nullptr, sd, greedy ? 1 : 0,
-                             static_cast<int>(top_k), static_cast<float>(top_p), tok.data_ptr<int64_t>(), lp.data_ptr<float>(),
-                             cur_stream()), "sample_topk_topp");
-  return {tok, lp};
-}
-
 // varlen causal flash-attention forward on tcgen05 (csrc/attn_fwd.cu).  q:[Tq,nq,128] k,v:[Tk,nkv,128] (row-strided views allowed)
-std::vector<at::Tensor> attn_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& cu_q,
-                                 const at::Tensor& cu_k, double sm_scale, bool causal, bool want_lse,
-                                 const c10::optional<at::Tensor>& dbg) {
-  CHECK_BF16(q); CHECK_BF16(k); CHECK_BF16(v);
-  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.size(2) == 128 && k.size(2) == 128 && v.size(2) == 128,
-              "attn_fwd: head_dim must be 128");
-  TORCH_CHECK(q.stride(2) == 1 && q.stride(1) == 128 && k.stride(2) == 1 && k.stride(1) == 128 && v.stride(2) == 1 && v.stride(1) == 128,
-              "attn_fwd: heads must be contiguous inside a token row");
-  TORCH_CHECK(q.stride(0) % 8 == 0 && k.stride(0) % 8 == 0 && v.stride(0) % 8 == 0);
-  TORCH_CHECK((reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0 && (reinterpret_cast<uintptr_t>(k.data_ptr()) & 15) == 0 &&
-              (reinterpret_cast<uintptr_t>(v.data_ptr()) & 15) == 0, "attn_fwd: 16-byte aligned operands");
-  TORCH_CHECK(cu_q.is_cuda() && cu_q.scalar_type() == at::kInt && cu_q.is_contiguous() && cu_k.is_cuda() &&
-              cu_k.scalar_type() == at::kInt && cu_k.is_contiguous() && cu_q.numel() == cu_k.numel());
-  const int Tq = q.size(0), Tk = k.size(0), nq = q.size(1), nkv = k.size(1), B = cu_q.numel() - 1;
-  c10::cuda::CUDAGuard g(q.device());
-  at::Tensor o = at::empty({Tq, nq, 128}, q.options());
-  at::Tensor lse = want_lse ? at::empty({nq, Tq}, q.options().dtype(at::kFloat)) : at::Tensor();
-  check(prl_attn_fwd(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), want_lse ? lse.data_ptr<float>() : nullptr,
-                     cu_q.data_ptr<int>(), cu_k.data_ptr<int>(), B, Tq, Tk, nq, nkv, q.stride(0), k.stride(0), v.stride(0),
-                     static_cast<int64_t>(nq) * 128, static_cast<float>(sm_scale), causal ? 1 : 0, Tq / 128 + B,
-                     dbg.has_value() ? reinterpret_cast<long long*>(dbg->data_ptr<int64_t>()) : nullptr, cur_stream()),
-        "attn_fwd");
-  if (want_lse) return {o, lse};
-  return {o};
-}
-
 // flash-attention backward (csrc/attn_bwd.cu): returns (dq, dk, dv) in bf16, shapes of q / k / v (contiguous)
 std::vector<at::Tensor> attn_bwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& o,
                                  const at::Tensor& d_o, const at::Tensor& lse, const at::Tensor& cu_q, const at::Tensor& cu_k,
@@ -672,54 +574,7 @@ void nvls_bcast_store(const at::Tensor& src, int64_t mc_dst, int64_t ctas) {
                              cur_stream()), "nvls_bcast_store");
 }
 
-static at::Tensor vec_i64(const std::vector<int64_t>& v) {
-  return at::tensor(c10::ArrayRef<int64_t>(v.data(), v.size()), at::TensorOptions().dtype(at::kLong));
-}
-
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
-  py::class_<prl::EngineScheduler>(m, "EngineScheduler")
-      .def(py::init<prl::KvPageManager*, int64_t, int64_t, bool>(), py::arg("kv"), py::arg("max_num_seqs"), py::arg("page_size"),
-           py::arg("prefix_cache"), py::keep_alive<1, 2>())
-      .def("add", &prl::EngineScheduler::add, py::arg("prompt"), py::arg("max_new"), py::arg("group"), py::arg("cacheable"))
-      .def("remove_waiting", &prl::EngineScheduler::remove_waiting)
-      .def("num_waiting", &prl::EngineScheduler::num_waiting)
-      .def("num_free_slots", &prl::EngineScheduler::num_free_slots)
-      .def("num_live", &prl::EngineScheduler::num_live)
-      .def("admit", &prl::EngineScheduler::admit)
-      .def("info", [](const prl::EngineScheduler& s, int64_t h) {        // (slot, blocks, shared_prefix_blocks, cached_tokens, donor)
-        const prl::SchedRequest& r = s.get(h);
-        return py::make_tuple(r.slot, r.blocks, r.shared_prefix_blocks, r.cached_tokens, r.donor);
-      })
-      .def("prefill_arrays", [](const prl::EngineScheduler& s, const std::vector<std::tuple<int64_t, int64_t, int64_t>>& spans, bool gather) {
-        const prl::PrefillArrays a = s.prefill_arrays(spans, gather);
-        return py::make_tuple(vec_i64(a.ids), vec_i64(a.pos), vec_i64(a.slots), vec_i64(a.lens), vec_i64(a.g_blk), vec_i64(a.g_off), vec_i64(a.klens));
-      })
-      .def("block_rows", [](const prl::EngineScheduler& s, const std::vector<int64_t>& handles, int64_t width) {
-        const std::vector<int32_t> rows = s.block_rows(handles, width);
-        return at::tensor(c10::ArrayRef<int32_t>(rows.data(), rows.size()), at::TensorOptions().dtype(at::kInt))
-            .reshape({static_cast<int64_t>(handles.size()), width});
-      })
-      .def("move_slots", &prl::EngineScheduler::move_slots)
-      .def("free_slots", &prl::EngineScheduler::free_slots)
-      .def("finish", &prl::EngineScheduler::finish, py::arg("handle"), py::arg("tokens"), py::arg("to_cache"));
-  py::class_<prl::KvPageManager>(m, "KvPageManager")
-      .def(py::init<int64_t, int64_t>(), py::arg("num_blocks"), py::arg("page_size"))
-      .def_property_readonly("num_blocks", &prl::KvPageManager::num_blocks)
-      .def("available", &prl::KvPageManager::available)
-      .def("ref", &prl::KvPageManager::ref)
-      .def("alloc", &prl::KvPageManager::alloc)
-      .def("share", &prl::KvPageManager::share)
-      .def("release", &prl::KvPageManager::release)
-      .def("page_keys", &prl::KvPageManager::page_keys)
-      .def("match", &prl::KvPageManager::match)
-      .def("insert", &prl::KvPageManager::insert)
-      .def("evict", &prl::KvPageManager::evict)
-      .def("flush", &prl::KvPageManager::flush)
-      .def("cached_pages", &prl::KvPageManager::cached_pages)
-      .def_property_readonly("hits", &prl::KvPageManager::hits)
-      .def_property_readonly("misses", &prl::KvPageManager::misses);
-  m.def("gemm_bf16", &gemm_bf16, py::arg("a"), py::arg("b"), py::arg("residual") = py::none(),
-        py::arg("out") = py::none(), py::arg("force_bn") = 0);
   m.def("gemm2_bf16", &gemm2_bf16, py::arg("a"), py::arg("b"), py::arg("a_mn") = false, py::arg("b_mn") = false,
         py::arg("residual") = py::none(), py::arg("out") = py::none(), py::arg("force_bn") = 0);
   m.def("gemm2_accum_f32_", &gemm2_accum_f32_);
@@ -745,11 +600,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("paged_decode", &paged_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
         py::arg("seq_lens"), py::arg("nq"), py::arg("nkv"), py::arg("d"), py::arg("sm_scale"), py::arg("splits") = 1,
         py::arg("out") = py::none());
-  m.def("attn_fwd", &attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu_q"), py::arg("cu_k"), py::arg("sm_scale"),
-        py::arg("causal") = true, py::arg("want_lse") = true, py::arg("dbg") = py::none());
   m.def("attn_bwd", &attn_bwd);
-  m.def("sample", &sample);
-  m.def("sample_topk_topp", &sample_topk_topp);
   m.def("sym_malloc", &sym_malloc);
   m.def("sym_free", &sym_free);
   m.def("ipc_get_handle", &ipc_get_handle);

@@ -1,0 +1,397 @@
+// polyrl_b200 — bindings of the serving core (module ``_serve``): native scheduler and page manager, dense GEMMs, packed
+// attention, sampling and the sequence-mixer kernels.  Everything a rollout engine of a mixer stack needs is in this one
+// module, so a serving host builds it without the training and multi-GPU kernels of ``_C``.
+#include "bindings_common.hpp"
+#include "kv_manager.hpp"
+#include "scheduler.hpp"
+
+extern "C" {
+int prl_gemm_bf16(const void*, const void*, void*, const void*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
+int prl_sample(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int64_t*, float*, cudaStream_t);
+int prl_sample_topk_topp(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int, float, int64_t*, float*, cudaStream_t);
+int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int32_t*, const int32_t*, int, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, float, int, int, const float*, long long*, cudaStream_t);
+int prl_gemm_gelu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, cudaStream_t);
+int prl_mix_embed(const int64_t*, const void*, float*, void*, int, int, int, cudaStream_t);
+int prl_mix_norm_add(const void*, int64_t, float*, const float*, const float*, void*, int, int, float, int, cudaStream_t);
+int prl_mix_rms(const float*, const float*, void*, int, int, float, int, cudaStream_t);
+int prl_mix_gated_norm(const void*, int64_t, const void*, int64_t, const float*, void*, int64_t, int, int, int, float, int, int, cudaStream_t);
+int prl_mix_conv(const void*, int64_t, const float*, const float*, void*, const int32_t*, const int32_t*, const int64_t*, const int32_t*, void*, int64_t, int, int, int, int, int, cudaStream_t);
+int prl_mix_latent_prep(const void*, int64_t, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, int, float, int, cudaStream_t);
+int prl_mix_rope(void*, int64_t, int, int, int, int, const double*, const int64_t*, int, int, cudaStream_t);
+int prl_mix_gelu(void*, int64_t, int, cudaStream_t);
+int prl_mix_chunk_supported(int);
+int prl_mix_latent_tc_ok(int, int);
+}
+#include "mix_params.hpp"
+extern "C" {
+int prl_mix_scan(const prl::ScanParams*, int, int, cudaStream_t);
+int prl_mix_chunk(const prl::ScanParams*, int, cudaStream_t);
+int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
+}
+
+namespace {
+
+at::Tensor gemm_bf16(const at::Tensor& a, const at::Tensor& b, const c10::optional<at::Tensor>& residual,
+                     c10::optional<at::Tensor> out, int64_t force_bn) {
+  CHECK_BF16(a); CHECK_BF16(b);
+  TORCH_CHECK(a.dim() == 2 && b.dim() == 2 && a.size(1) == b.size(1), "gemm_bf16: A[M,K] B[N,K]");
+  CHECK_LASTDIM(a); CHECK_LASTDIM(b);
+  const int M = a.size(0), K = a.size(1), N = b.size(0);
+  TORCH_CHECK(K % 8 == 0 && N % 8 == 0, "K and N must be multiples of 8");
+  TORCH_CHECK(a.stride(0) % 8 == 0 && b.stride(0) % 8 == 0, "row pitch must be a multiple of 8 elements");
+  c10::cuda::CUDAGuard g(a.device());
+  at::Tensor d = out.has_value() ? *out : at::empty({M, N}, a.options());
+  CHECK_BF16(d); CHECK_LASTDIM(d);
+  const void* r = nullptr;
+  if (residual.has_value()) {
+    CHECK_BF16(*residual);
+    TORCH_CHECK(residual->sizes() == d.sizes() && residual->stride(0) == d.stride(0) && residual->stride(1) == 1);
+    r = residual->data_ptr();
+  }
+  check(prl_gemm_bf16(a.data_ptr(), b.data_ptr(), d.data_ptr(), r, M, N, K, a.stride(0), b.stride(0), d.stride(0),
+                      static_cast<int>(force_bn), cur_stream()), "gemm_bf16");
+  return d;
+}
+
+std::vector<at::Tensor> sample(const at::Tensor& logits, const c10::optional<at::Tensor>& inv_temp,
+                               const c10::optional<at::Tensor>& seeds, bool greedy) {
+  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1);
+  const int dt = logits.scalar_type() == at::kFloat ? 0 : 1;
+  TORCH_CHECK(dt == 0 || logits.scalar_type() == at::kBFloat16);
+  const int B = logits.size(0), V = logits.size(1);
+  c10::cuda::CUDAGuard g(logits.device());
+  at::Tensor tok = at::empty({B}, logits.options().dtype(at::kLong));
+  at::Tensor lp = at::empty({B}, logits.options().dtype(at::kFloat));
+  const uint64_t* sd = nullptr;
+  if (seeds.has_value()) { TORCH_CHECK(seeds->scalar_type() == at::kLong); sd = reinterpret_cast<const uint64_t*>(seeds->data_ptr<int64_t>()); }
+  check(prl_sample(logits.data_ptr(), dt, logits.stride(0), B, V,
+                   inv_temp.has_value() ? inv_temp->data_ptr<float>() : nullptr, sd, greedy ? 1 : 0,
+                   tok.data_ptr<int64_t>(), lp.data_ptr<float>(), cur_stream()), "sample");
+  return {tok, lp};
+}
+
+std::vector<at::Tensor> sample_topk_topp(const at::Tensor& logits, const c10::optional<at::Tensor>& inv_temp,
+                                         const c10::optional<at::Tensor>& seeds, bool greedy, int64_t top_k, double top_p) {
+  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1);
+  const int dt = logits.scalar_type() == at::kFloat ? 0 : 1;
+  TORCH_CHECK(dt == 0 || logits.scalar_type() == at::kBFloat16);
+  const int B = logits.size(0), V = logits.size(1);
+  c10::cuda::CUDAGuard g(logits.device());
+  at::Tensor tok = at::empty({B}, logits.options().dtype(at::kLong));
+  at::Tensor lp = at::empty({B}, logits.options().dtype(at::kFloat));
+  const uint64_t* sd = nullptr;
+  if (seeds.has_value()) { TORCH_CHECK(seeds->scalar_type() == at::kLong); sd = reinterpret_cast<const uint64_t*>(seeds->data_ptr<int64_t>()); }
+  check(prl_sample_topk_topp(logits.data_ptr(), dt, logits.stride(0), B, V,
+                             inv_temp.has_value() ? inv_temp->data_ptr<float>() : nullptr, sd, greedy ? 1 : 0,
+                             static_cast<int>(top_k), static_cast<float>(top_p), tok.data_ptr<int64_t>(), lp.data_ptr<float>(),
+                             cur_stream()), "sample_topk_topp");
+  return {tok, lp};
+}
+
+std::vector<at::Tensor> attn_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& cu_q,
+                                 const at::Tensor& cu_k, double sm_scale, bool causal, bool want_lse,
+                                 const c10::optional<at::Tensor>& dbg, const c10::optional<at::Tensor>& sink) {
+  CHECK_BF16(q); CHECK_BF16(k); CHECK_BF16(v);
+  const int64_t dk = q.size(-1);
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && (dk == 128 || dk == 192) && k.size(2) == dk && v.size(2) == 128 &&
+              v.size(1) == k.size(1) && v.size(0) == k.size(0), "attn_fwd: query / key width 128 or 192, value width 128");
+  TORCH_CHECK(q.stride(2) == 1 && q.stride(1) == dk && k.stride(2) == 1 && k.stride(1) == dk && v.stride(2) == 1 && v.stride(1) == 128,
+              "attn_fwd: heads must be contiguous inside a token row");
+  TORCH_CHECK(q.stride(0) % 8 == 0 && k.stride(0) % 8 == 0 && v.stride(0) % 8 == 0);
+  TORCH_CHECK((reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0 && (reinterpret_cast<uintptr_t>(k.data_ptr()) & 15) == 0 &&
+              (reinterpret_cast<uintptr_t>(v.data_ptr()) & 15) == 0, "attn_fwd: 16-byte aligned operands");
+  TORCH_CHECK(cu_q.is_cuda() && cu_q.scalar_type() == at::kInt && cu_q.is_contiguous() && cu_k.is_cuda() &&
+              cu_k.scalar_type() == at::kInt && cu_k.is_contiguous() && cu_q.numel() == cu_k.numel());
+  const int Tq = q.size(0), Tk = k.size(0), nq = q.size(1), nkv = k.size(1), B = cu_q.numel() - 1;
+  if (sink.has_value()) { CHECK_F32(*sink); TORCH_CHECK(sink->is_contiguous() && sink->numel() == nq); }
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor o = at::empty({Tq, nq, 128}, q.options());
+  at::Tensor lse = want_lse ? at::empty({nq, Tq}, q.options().dtype(at::kFloat)) : at::Tensor();
+  check(prl_attn_fwd(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), want_lse ? lse.data_ptr<float>() : nullptr,
+                     cu_q.data_ptr<int>(), cu_k.data_ptr<int>(), B, Tq, Tk, nq, nkv, static_cast<int>(dk), q.stride(0), k.stride(0), v.stride(0),
+                     static_cast<int64_t>(nq) * 128, static_cast<float>(sm_scale), causal ? 1 : 0, Tq / 128 + B,
+                     sink.has_value() ? sink->data_ptr<float>() : nullptr,
+                     dbg.has_value() ? reinterpret_cast<long long*>(dbg->data_ptr<int64_t>()) : nullptr, cur_stream()),
+        "attn_fwd");
+  if (want_lse) return {o, lse};
+  return {o};
+}
+
+static at::Tensor vec_i64(const std::vector<int64_t>& v) {
+  return at::tensor(c10::ArrayRef<int64_t>(v.data(), v.size()), at::TensorOptions().dtype(at::kLong));
+}
+
+// ---------------------------------------------------------------------------------------------- sequence mixers
+int dt_of(const at::Tensor& t, const char* what) {
+  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kFloat), what, ": CUDA bf16 or fp32 tensor expected");
+  return t.scalar_type() == at::kBFloat16 ? 0 : 1;
+}
+// rows with unit inner stride
+void rows2(const at::Tensor& t, const char* what) { TORCH_CHECK(t.dim() == 2 && t.stride(1) == 1, what, ": [rows, cols] with unit inner stride expected"); }
+const float* vecf(const at::Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() == n, what, ": contiguous fp32 vector of ", n, " expected");
+  return t.data_ptr<float>();
+}
+const float* vecf(const c10::optional<at::Tensor>& t, int64_t n, const char* what) { return t.has_value() ? vecf(*t, n, what) : nullptr; }
+template <class I>
+const I* veci(const at::Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == c10::CppTypeToScalarType<I>::value && t.is_contiguous() && t.numel() >= n, what, ": contiguous index vector of at least ",
+              n, " expected");
+  return t.data_ptr<I>();
+}
+
+std::vector<at::Tensor> mix_embed(const at::Tensor& ids, const at::Tensor& emb) {
+  const int dt = dt_of(emb, "mix_embed");
+  TORCH_CHECK(emb.is_contiguous() && emb.dim() == 2);
+  const int64_t rows = ids.numel(), W = emb.size(1);
+  const int64_t* ip = veci<int64_t>(ids, rows, "mix_embed ids");
+  c10::cuda::CUDAGuard g(emb.device());
+  at::Tensor x = at::empty({rows, W}, emb.options().dtype(at::kFloat));
+  at::Tensor h = dt == 0 ? at::empty({rows, W}, emb.options()) : x;
+  check(prl_mix_embed(ip, emb.data_ptr(), x.data_ptr<float>(), dt == 0 ? h.data_ptr() : nullptr, rows, W, dt, cur_stream()), "mix_embed");
+  return {x, h};
+}
+
+// x += rms(y) * w in place; returns x in y's dtype (x itself when fp32), or the next norm of x when w_next is given
+at::Tensor mix_norm_add_(const at::Tensor& y, at::Tensor x, const at::Tensor& w, double eps, const c10::optional<at::Tensor>& w_next) {
+  const int dt = dt_of(y, "mix_norm_add");
+  rows2(y, "mix_norm_add y");
+  CHECK_F32(x);
+  TORCH_CHECK(x.is_contiguous() && x.sizes() == y.sizes());
+  const int64_t rows = x.size(0), W = x.size(1);
+  c10::cuda::CUDAGuard g(y.device());
+  const bool own = dt == 0 || w_next.has_value();
+  at::Tensor h = own ? at::empty({rows, W}, y.options()) : x;
+  check(prl_mix_norm_add(y.data_ptr(), y.stride(0), x.data_ptr<float>(), vecf(w, W, "mix_norm_add w"), vecf(w_next, W, "mix_norm_add w_next"),
+                         own ? h.data_ptr() : nullptr, rows, W, static_cast<float>(eps), dt, cur_stream()), "mix_norm_add");
+  return h;
+}
+
+at::Tensor mix_rms(const at::Tensor& x, const at::Tensor& w, double eps, bool bf16) {
+  CHECK_F32(x);
+  TORCH_CHECK(x.is_contiguous() && x.dim() == 2);
+  c10::cuda::CUDAGuard g(x.device());
+  at::Tensor h = at::empty(x.sizes(), x.options().dtype(bf16 ? at::kBFloat16 : at::kFloat));
+  check(prl_mix_rms(x.data_ptr<float>(), vecf(w, x.size(1), "mix_rms w"), h.data_ptr(), x.size(0), x.size(1), static_cast<float>(eps), bf16 ? 0 : 1,
+                    cur_stream()), "mix_rms");
+  return h;
+}
+
+at::Tensor mix_gated_norm(const at::Tensor& y, const at::Tensor& z, const at::Tensor& w, int64_t groups, double eps, bool gate_first) {
+  const int dt = dt_of(y, "mix_gated_norm");
+  rows2(y, "mix_gated_norm y"); rows2(z, "mix_gated_norm z");
+  TORCH_CHECK(z.scalar_type() == y.scalar_type() && z.sizes() == y.sizes() && groups > 0 && y.size(1) % groups == 0);
+  c10::cuda::CUDAGuard g(y.device());
+  at::Tensor out = at::empty(y.sizes(), y.options());
+  check(prl_mix_gated_norm(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), vecf(w, y.size(1), "mix_gated_norm w"), out.data_ptr(), out.stride(0),
+                           y.size(0), groups, y.size(1) / groups, static_cast<float>(eps), gate_first ? 1 : 0, dt, cur_stream()), "mix_gated_norm");
+  return out;
+}
+
+// x [T, ch] -> silu(conv(x)); state [slots, taps - 1, ch] is read for what lies before a span and left holding its last inputs
+at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const at::Tensor& bias, at::Tensor state, const at::Tensor& cu, const at::Tensor& start,
+                    const at::Tensor& slot, const c10::optional<at::Tensor>& seq_of) {
+  const int dt = dt_of(x, "mix_conv");
+  rows2(x, "mix_conv x");
+  const int64_t T = x.size(0), ch = x.size(1), taps = w.size(0), spans = start.numel();
+  TORCH_CHECK(w.dim() == 2 && w.size(1) == ch && state.scalar_type() == x.scalar_type() && state.is_cuda() && state.is_contiguous() && state.dim() == 3 &&
+              state.size(1) == taps - 1 && state.size(2) == ch, "mix_conv: shapes");
+  TORCH_CHECK(seq_of.has_value() || spans == T, "mix_conv: one token per span without seq_of");
+  c10::cuda::CUDAGuard g(x.device());
+  at::Tensor out = at::empty({T, ch}, x.options());
+  check(prl_mix_conv(x.data_ptr(), x.stride(0), vecf(w, taps * ch, "mix_conv w"), vecf(bias, ch, "mix_conv bias"), state.data_ptr(),
+                     veci<int32_t>(cu, spans + 1, "cu"), veci<int32_t>(start, spans, "start"), veci<int64_t>(slot, spans, "slot"),
+                     seq_of.has_value() ? veci<int32_t>(*seq_of, T, "seq_of") : nullptr, out.data_ptr(), out.stride(0), ch, taps, T, spans, dt,
+                     cur_stream()), "mix_conv");
+  return out;
+}
+
+// gated linear recurrence over packed spans; mode 0 = state-space duality, 1 = matrix memory (csrc/mixers.cuh)
+void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
+                     const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log,
+                     const c10::optional<at::Tensor>& d_skip, double qscale, double cap, at::Tensor S, const c10::optional<at::Tensor>& nst,
+                     const c10::optional<at::Tensor>& mst, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, at::Tensor counter,
+                     bool chunk, at::Tensor out) {
+  const int dt = dt_of(v, "mix_scan");
+  rows2(q, "mix_scan q"); rows2(k, "mix_scan k"); rows2(v, "mix_scan v"); rows2(g0, "mix_scan g0");
+  CHECK_F32(S); CHECK_F32(g0);
+  TORCH_CHECK(mode == 0 || mode == 1);
+  TORCH_CHECK(S.dim() == 4 && S.is_contiguous());
+  const int64_t H = S.size(1), N = S.size(2), V = S.size(3), T = v.size(0), spans = start.numel();
+  TORCH_CHECK(q.scalar_type() == v.scalar_type() && k.scalar_type() == v.scalar_type() && q.size(0) == T && k.size(0) == T && v.size(1) == H * V &&
+              q.sizes() == k.sizes() && q.size(1) % N == 0 && q.size(1) > 0 && H % (q.size(1) / N) == 0, "mix_scan: shapes");
+  TORCH_CHECK(g0.size(0) == T && g0.size(1) == H);
+  TORCH_CHECK(N <= 512, "mix_scan: state rows per head <= 512");
+  prl::ScanParams p{};
+  p.q = q.data_ptr(); p.k = k.data_ptr(); p.v = v.data_ptr();
+  p.ldq = q.stride(0); p.ldk = k.stride(0); p.ldv = v.stride(0);
+  p.rep = H / (q.size(1) / N);
+  p.g0 = g0.data_ptr<float>(); p.ldg = g0.stride(0);
+  p.b0 = vecf(b0, H, "b0"); p.b1 = vecf(b1, H, "b1"); p.a_log = vecf(a_log, H, "a_log"); p.d_skip = vecf(d_skip, H, "d_skip");
+  if (mode == 1) {
+    TORCH_CHECK(g1.has_value() && nst.has_value() && mst.has_value());
+    CHECK_F32(*g1); CHECK_F32(*nst); CHECK_F32(*mst);
+    TORCH_CHECK(g1->dim() == 2 && g1->size(0) == T && g1->size(1) == H && g1->stride(1) == 1 && g1->stride(0) == g0.stride(0));
+    TORCH_CHECK(nst->is_contiguous() && nst->numel() == S.size(0) * H * N && mst->is_contiguous() && mst->numel() == S.size(0) * H && cap > 0);
+    p.g1 = g1->data_ptr<float>(); p.nst = nst->data_ptr<float>(); p.mst = mst->data_ptr<float>();
+  } else {
+    TORCH_CHECK(a_log.has_value());
+  }
+  p.qscale = static_cast<float>(qscale); p.cap = static_cast<float>(cap);
+  c10::cuda::CUDAGuard g(v.device());
+  TORCH_CHECK(out.is_cuda() && out.scalar_type() == v.scalar_type() && out.is_contiguous() && out.dim() == 2 && out.size(0) == T && out.size(1) == H * V);
+  p.out = out.data_ptr(); p.ldo = H * V;
+  p.S = S.data_ptr<float>();
+  p.cu = veci<int32_t>(cu, spans + 1, "cu"); p.start = veci<int32_t>(start, spans, "start"); p.slot = veci<int64_t>(slot, spans, "slot");
+  veci<int32_t>(counter, spans * H, "counter");
+  p.counter = counter.data_ptr<int32_t>();
+  p.H = H; p.N = N; p.V = V; p.spans = spans;
+  if (chunk) {
+    TORCH_CHECK(dt == 0 && prl_mix_chunk_supported(N), "mix_scan: the chunked kernel takes bf16 and N <= 256");
+    check(prl_mix_chunk(&p, static_cast<int>(mode), cur_stream()), "mix_chunk");
+  } else {
+    check(prl_mix_scan(&p, static_cast<int>(mode), dt, cur_stream()), "mix_scan");
+  }
+}
+
+// a [T, qr + r + rd] -> (normed query latent [T, qr], packed cache rows [T, r + rd] or empty); cache rows also go to pool[kvslot]
+std::vector<at::Tensor> mix_latent_prep(const at::Tensor& a, const at::Tensor& wq, const at::Tensor& wkv, const at::Tensor& freq, const at::Tensor& pos,
+                                        const at::Tensor& kvslot, at::Tensor pool, double eps, bool want_entry) {
+  const int dt = dt_of(a, "mix_latent_prep");
+  rows2(a, "mix_latent_prep a");
+  const int64_t T = a.size(0), qr = wq.numel(), r = wkv.numel(), rd = 2 * freq.numel();
+  TORCH_CHECK(a.size(1) >= qr + r + rd && pool.scalar_type() == a.scalar_type() && pool.is_cuda() && pool.is_contiguous() && pool.size(-1) == r + rd);
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == at::kDouble && freq.is_contiguous());
+  c10::cuda::CUDAGuard g(a.device());
+  at::Tensor cq = at::empty({T, qr}, a.options()), en = at::empty({want_entry ? T : 0, r + rd}, a.options());
+  check(prl_mix_latent_prep(a.data_ptr(), a.stride(0), qr, r, rd, vecf(wq, qr, "wq"), vecf(wkv, r, "wkv"), freq.data_ptr<double>(),
+                            veci<int64_t>(pos, T, "pos"), veci<int64_t>(kvslot, T, "kvslot"), cq.data_ptr(), want_entry ? en.data_ptr() : nullptr,
+                            pool.data_ptr(), T, static_cast<float>(eps), dt, cur_stream()), "mix_latent_prep");
+  return {cq, en};
+}
+
+// q [T, H, dq]: rotate columns [d, d + 2 * freq.numel()) of every head in place
+void mix_rope_(at::Tensor q, int64_t d, const at::Tensor& freq, const at::Tensor& pos) {
+  const int dt = dt_of(q, "mix_rope");
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && d + 2 * freq.numel() <= q.size(2));
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == at::kDouble && freq.is_contiguous());
+  c10::cuda::CUDAGuard g(q.device());
+  check(prl_mix_rope(q.data_ptr(), q.stride(0), q.size(1), q.size(2), d, 2 * freq.numel(), freq.data_ptr<double>(), veci<int64_t>(pos, q.size(0), "pos"),
+                     q.size(0), dt, cur_stream()), "mix_rope");
+}
+
+// absorbed latent attention: q_lat [H, R, r], q [R, H, dq] (rotated part at column d) over pool rows -> [H, R, r]
+at::Tensor mix_latent(const at::Tensor& q_lat, const at::Tensor& q, int64_t d, const at::Tensor& pool, const at::Tensor& table,
+                      const c10::optional<at::Tensor>& seq_of, const at::Tensor& kv_len, const c10::optional<at::Tensor>& sink, double scale, int64_t splits,
+                      bool tc) {
+  const int dt = dt_of(q, "mix_latent");
+  TORCH_CHECK(q_lat.dim() == 3 && q_lat.is_contiguous() && q_lat.scalar_type() == q.scalar_type() && q.dim() == 3 && q.stride(2) == 1 &&
+              q.stride(1) == q.size(2));
+  const int64_t H = q_lat.size(0), R = q_lat.size(1), r = q_lat.size(2), rd = pool.size(-1) - r;
+  TORCH_CHECK(q.size(0) == R && q.size(1) == H && rd >= 0 && d + rd <= q.size(2));
+  TORCH_CHECK(pool.is_cuda() && pool.is_contiguous() && pool.scalar_type() == q.scalar_type() && (reinterpret_cast<uintptr_t>(pool.data_ptr()) & 15) == 0);
+  TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.dim() == 2 && table.stride(1) == 1);
+  TORCH_CHECK(seq_of.has_value() || table.size(0) >= R);
+  TORCH_CHECK(splits >= 1);
+  prl::LatentParams p{};
+  p.q_lat = q_lat.data_ptr(); p.q = q.data_ptr(); p.ldq = q.stride(0); p.dq = q.size(2); p.d = d;
+  p.pool = pool.data_ptr(); p.table = table.data_ptr<int32_t>(); p.ld_table = table.stride(0);
+  p.seq_of = seq_of.has_value() ? veci<int32_t>(*seq_of, R, "seq_of") : nullptr;
+  p.kv_len = veci<int32_t>(kv_len, R, "kv_len");
+  p.sink = vecf(sink, H, "sink");
+  p.H = H; p.R = R; p.r = r; p.rd = rd; p.scale = static_cast<float>(scale);
+  p.splits = tc ? splits : 1;
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty({H, R, r}, q.options()), part;
+  p.out = out.data_ptr();
+  if (p.splits > 1) {
+    part = at::empty({H * R * p.splits * (r + 2)}, q.options().dtype(at::kFloat));
+    p.part = part.data_ptr<float>();
+  }
+  check(prl_mix_latent(&p, tc ? 1 : 0, dt, cur_stream()), "mix_latent");
+  return out;
+}
+
+at::Tensor gemm_gelu(const at::Tensor& a, const at::Tensor& w) {
+  CHECK_BF16(a); CHECK_BF16(w); CHECK_LASTDIM(a); CHECK_LASTDIM(w);
+  TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && a.size(1) == w.size(1) && w.size(0) % 8 == 0 && a.size(1) % 8 == 0 && a.stride(0) % 8 == 0 &&
+              w.stride(0) % 8 == 0);
+  c10::cuda::CUDAGuard g(a.device());
+  at::Tensor h = at::empty({a.size(0), w.size(0)}, a.options());
+  check(prl_gemm_gelu_bf16(a.data_ptr(), w.data_ptr(), h.data_ptr(), a.size(0), w.size(0), a.size(1), a.stride(0), w.stride(0), h.stride(0), cur_stream()),
+        "gemm_gelu");
+  return h;
+}
+void mix_gelu_(at::Tensor x) {
+  const int dt = dt_of(x, "mix_gelu");
+  TORCH_CHECK(x.is_contiguous());
+  c10::cuda::CUDAGuard g(x.device());
+  check(prl_mix_gelu(x.data_ptr(), x.numel(), dt, cur_stream()), "mix_gelu");
+}
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+  py::class_<prl::EngineScheduler>(m, "EngineScheduler")
+      .def(py::init<prl::KvPageManager*, int64_t, int64_t, bool>(), py::arg("kv"), py::arg("max_num_seqs"), py::arg("page_size"),
+           py::arg("prefix_cache"), py::keep_alive<1, 2>())
+      .def("add", &prl::EngineScheduler::add, py::arg("prompt"), py::arg("max_new"), py::arg("group"), py::arg("cacheable"))
+      .def("remove_waiting", &prl::EngineScheduler::remove_waiting)
+      .def("num_waiting", &prl::EngineScheduler::num_waiting)
+      .def("num_free_slots", &prl::EngineScheduler::num_free_slots)
+      .def("num_live", &prl::EngineScheduler::num_live)
+      .def("admit", &prl::EngineScheduler::admit)
+      .def("info", [](const prl::EngineScheduler& s, int64_t h) {        // (slot, blocks, shared_prefix_blocks, cached_tokens, donor)
+        const prl::SchedRequest& r = s.get(h);
+        return py::make_tuple(r.slot, r.blocks, r.shared_prefix_blocks, r.cached_tokens, r.donor);
+      })
+      .def("prefill_arrays", [](const prl::EngineScheduler& s, const std::vector<std::tuple<int64_t, int64_t, int64_t>>& spans, bool gather) {
+        const prl::PrefillArrays a = s.prefill_arrays(spans, gather);
+        return py::make_tuple(vec_i64(a.ids), vec_i64(a.pos), vec_i64(a.slots), vec_i64(a.lens), vec_i64(a.g_blk), vec_i64(a.g_off), vec_i64(a.klens));
+      })
+      .def("block_rows", [](const prl::EngineScheduler& s, const std::vector<int64_t>& handles, int64_t width) {
+        const std::vector<int32_t> rows = s.block_rows(handles, width);
+        return at::tensor(c10::ArrayRef<int32_t>(rows.data(), rows.size()), at::TensorOptions().dtype(at::kInt))
+            .reshape({static_cast<int64_t>(handles.size()), width});
+      })
+      .def("open", &prl::EngineScheduler::open, py::arg("tokens"))
+      .def("feed", &prl::EngineScheduler::feed, py::arg("handle"), py::arg("tokens"))
+      .def("move_slots", &prl::EngineScheduler::move_slots)
+      .def("free_slots", &prl::EngineScheduler::free_slots)
+      .def("finish", &prl::EngineScheduler::finish, py::arg("handle"), py::arg("tokens"), py::arg("to_cache"));
+  py::class_<prl::KvPageManager>(m, "KvPageManager")
+      .def(py::init<int64_t, int64_t>(), py::arg("num_blocks"), py::arg("page_size"))
+      .def_property_readonly("num_blocks", &prl::KvPageManager::num_blocks)
+      .def("available", &prl::KvPageManager::available)
+      .def("ref", &prl::KvPageManager::ref)
+      .def("alloc", &prl::KvPageManager::alloc)
+      .def("share", &prl::KvPageManager::share)
+      .def("release", &prl::KvPageManager::release)
+      .def("page_keys", &prl::KvPageManager::page_keys)
+      .def("match", &prl::KvPageManager::match)
+      .def("insert", &prl::KvPageManager::insert)
+      .def("evict", &prl::KvPageManager::evict)
+      .def("flush", &prl::KvPageManager::flush)
+      .def("cached_pages", &prl::KvPageManager::cached_pages)
+      .def_property_readonly("hits", &prl::KvPageManager::hits)
+      .def_property_readonly("misses", &prl::KvPageManager::misses);
+  m.def("gemm_bf16", &gemm_bf16, py::arg("a"), py::arg("b"), py::arg("residual") = py::none(),
+        py::arg("out") = py::none(), py::arg("force_bn") = 0);
+  m.def("attn_fwd", &attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu_q"), py::arg("cu_k"), py::arg("sm_scale"),
+        py::arg("causal") = true, py::arg("want_lse") = true, py::arg("dbg") = py::none(), py::arg("sink") = py::none());
+  m.def("sample", &sample);
+  m.def("sample_topk_topp", &sample_topk_topp);
+  m.def("mix_embed", &mix_embed);
+  m.def("mix_norm_add_", &mix_norm_add_);
+  m.def("mix_rms", &mix_rms);
+  m.def("mix_gated_norm", &mix_gated_norm);
+  m.def("mix_conv", &mix_conv);
+  m.def("mix_scan_", &mix_scan_);
+  m.def("mix_latent_prep", &mix_latent_prep);
+  m.def("mix_rope_", &mix_rope_);
+  m.def("mix_latent", &mix_latent);
+  m.def("gemm_gelu", &gemm_gelu);
+  m.def("mix_gelu_", &mix_gelu_);
+  m.def("mix_chunk_supported", [](int64_t n) { return prl_mix_chunk_supported(static_cast<int>(n)) != 0; });
+  m.def("mix_latent_tc_ok", [](int64_t r, int64_t rd) { return prl_mix_latent_tc_ok(static_cast<int>(r), static_cast<int>(rd)) != 0; });
+}

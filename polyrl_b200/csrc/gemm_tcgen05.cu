@@ -111,6 +111,33 @@ struct EpiSwiglu {
   }
 };
 
+// H[M, N] = gelu(acc), tanh form, in the exactly equivalent shape z * sigmoid(2 u)
+struct GeluParams {
+  __nv_bfloat16* H;
+  int64_t ldh;
+};
+struct EpiGelu {
+  using Params = GeluParams;
+  __device__ __forceinline__ void begin(const Params&, int, int, const WorkInfo&) {}
+  __device__ __forceinline__ void end(const Params&, int, int, const WorkInfo&) {}
+  template <int BN>
+  __device__ __forceinline__ void tile(const Params& p, const AccReader& acc, int row, int M, int n0, int N) {
+#pragma unroll 1
+    for (int c = 0; c < BN; c += 32) {
+      float v[32];
+      acc.load(c, v);
+      const int valid = min(32, N - (n0 + c));
+      if (row >= M || valid <= 0) continue;
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const float z = v[i];
+        v[i] = z / (1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+      }
+      store_row_chunk(p.H + static_cast<int64_t>(row) * p.ldh + n0 + c, v, valid);
+    }
+  }
+};
+
 template <int BN, bool FP8>
 static int run_store(const void* A, const void* B, const StoreParams& sp, int M, int N, int K, int64_t lda, int64_t ldb,
                      cudaStream_t s) {
@@ -175,4 +202,16 @@ extern "C" int prl_gemm_swiglu_bf16(const void* A, const void* Wgu, void* H, voi
   using Cfg = GemmCfg<256, 2>;
   return launch_gemm<Cfg, EpiSwiglu, NoGate, false>(A, Wgu, M, N2, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0,
                                                     stream);
+}
+
+// H = gelu_tanh(A·W^T)
+extern "C" int prl_gemm_gelu_bf16(const void* A, const void* W, void* H, int M, int N, int K, int64_t lda, int64_t ldw, int64_t ldh,
+                                  cudaStream_t stream) {
+  GeluParams sp{static_cast<__nv_bfloat16*>(H), ldh};
+  if (M > kBlockM && N > 128) {
+    using Cfg2 = Gemm2Cfg<256, false, false, false>;
+    return launch_gemm2<Cfg2, EpiGelu>(A, W, nullptr, M, N, K, lda * 2, ldw * 2, 0, sp, 0, stream);
+  }
+  using Cfg = GemmCfg<64, 2>;
+  return launch_gemm<Cfg, EpiGelu, NoGate, false>(A, W, M, N, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);
 }

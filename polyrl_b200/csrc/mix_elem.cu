@@ -1,0 +1,399 @@
+// polyrl_b200 — row-wise kernels of the mixer stacks: embedding, output-norm + residual add, gated group norm, causal
+// convolution with carried taps, latent-attention row preparation, GELU.  The residual stream is fp32.
+#include "mixers.cuh"
+
+namespace prl {
+
+// ---- x = embed[id] (fp32), h = the same in T (h may be null when T is fp32 and x is used directly)
+template <class T, int VEC>
+__global__ void mix_embed_kernel(const int64_t* __restrict__ ids, const T* __restrict__ emb, float* __restrict__ x, T* __restrict__ h, int W) {
+  const int64_t row = blockIdx.x;
+  const T* src = emb + ids[row] * W;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float v[VEC];
+    ld_vec<T, VEC>(src + c, v);
+    st_vec<float, VEC>(x + row * W + c, v);
+    if (h) st_vec<T, VEC>(h + row * W + c, v);
+  }
+}
+
+// ---- x += rms(y) * w;  h = T(x), or T(rms(x) * w_next) when w_next is given (the model's final norm)
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) mix_norm_add_kernel(const T* __restrict__ y, int64_t ldy, float* __restrict__ x, const float* __restrict__ w,
+                                                           const float* __restrict__ w_next, T* __restrict__ h, int W, float eps) {
+  __shared__ float red[8];
+  const int64_t row = blockIdx.x;
+  const T* yr = y + row * ldy;
+  float* xr = x + row * W;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+    float v[VEC];
+    ld_vec<T, VEC>(yr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
+  }
+  const float r = rsqrtf(block_sum<8>(ss, red) / W + eps);
+  float s2 = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+    float v[VEC], g[VEC], xx[VEC];
+    ld_vec<T, VEC>(yr + c, v);
+    ld_vec<float, VEC>(w + c, g);
+    ld_vec<float, VEC>(xr + c, xx);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { xx[i] += v[i] * r * g[i]; s2 += xx[i] * xx[i]; }
+    st_vec<float, VEC>(xr + c, xx);
+    if (h && !w_next) st_vec<T, VEC>(h + row * W + c, xx);
+  }
+  if (!w_next) return;
+  const float r2 = rsqrtf(block_sum<8>(s2, red) / W + eps);
+  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+    float g[VEC], xx[VEC];
+    ld_vec<float, VEC>(xr + c, xx);
+    ld_vec<float, VEC>(w_next + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) xx[i] *= r2 * g[i];
+    st_vec<T, VEC>(h + row * W + c, xx);
+  }
+}
+
+// ---- h = T(rms(x) * w) of fp32 rows
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) mix_rms_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, float eps) {
+  __shared__ float red[8];
+  const int64_t row = blockIdx.x;
+  const float* xr = x + row * W;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+    float v[VEC];
+    ld_vec<float, VEC>(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
+  }
+  const float r = rsqrtf(block_sum<8>(ss, red) / W + eps);
+  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+    float v[VEC], g[VEC];
+    ld_vec<float, VEC>(xr + c, v);
+    ld_vec<float, VEC>(w + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] *= r * g[i];
+    st_vec<T, VEC>(h + row * W + c, v);
+  }
+}
+
+// ---- group norm of mixer outputs with a gate: GATE_FIRST  rms(y silu(z)) w   else   rms(y) w sigmoid(z)
+// WPG warps share one (row, group); 8 / WPG groups per CTA
+template <class T, int VEC, bool GATE_FIRST, int WPG>
+__global__ void __launch_bounds__(256) mix_gated_norm_kernel(const T* __restrict__ y, int64_t ldy, const T* __restrict__ z, int64_t ldz,
+                                                             const float* __restrict__ w, T* __restrict__ out, int64_t ldo, int64_t items, int groups,
+                                                             int gs, float eps) {
+  __shared__ float red[8];
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * (8 / WPG) + (threadIdx.x >> 5) / WPG;
+  if (WPG == 1 && item >= items) return;                // (WPG == 8: one item per CTA, the grid is exact)
+  const int64_t row = item / groups;
+  const int c0 = static_cast<int>(item % groups) * gs;
+  const int t = threadIdx.x % (32 * WPG);
+  const T* yr = y + row * ldy + c0;
+  const T* zr = z + row * ldz + c0;
+  T* orow = out + row * ldo + c0;
+  float ss = 0.f;
+  for (int c = t * VEC; c < gs; c += 32 * WPG * VEC) {
+    float v[VEC], g[VEC];
+    ld_vec<T, VEC>(yr + c, v);
+    if constexpr (GATE_FIRST) ld_vec<T, VEC>(zr + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      const float u = GATE_FIRST ? v[i] * silu_f(g[i]) : v[i];
+      ss += u * u;
+    }
+  }
+  const float r = rsqrtf(block_sum<WPG>(ss, red) / gs + eps);
+  for (int c = t * VEC; c < gs; c += 32 * WPG * VEC) {
+    float v[VEC], g[VEC], ww[VEC];
+    ld_vec<T, VEC>(yr + c, v);
+    ld_vec<T, VEC>(zr + c, g);
+    ld_vec<float, VEC>(w + c0 + c, ww);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * (GATE_FIRST ? silu_f(g[i]) : sigmoid_f(g[i])) * r * ww[i];
+    st_vec<T, VEC>(orow + c, v);
+  }
+}
+
+// ---- causal convolution per channel + silu; w [taps, ch] (row taps - 1 = current token), state [slots, taps - 1, ch]
+template <class T, int VEC, int TT>
+__global__ void __launch_bounds__(128) mix_conv_kernel(const T* __restrict__ x, int64_t ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                                                       const T* __restrict__ state, const int32_t* __restrict__ cu, const int32_t* __restrict__ start,
+                                                       const int64_t* __restrict__ slot, const int32_t* __restrict__ seq_of, T* __restrict__ out,
+                                                       int64_t ldo, int ch, int taps, int total) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * VEC;
+  if (c >= ch) return;
+  const int tb = blockIdx.y * TT, te = min(total, tb + TT);
+  for (int t = tb; t < te; ++t) {
+    const int s = seq_of[t];
+    const int t0 = cu[s];
+    const bool fresh = start[s] == 0;
+    float acc[VEC];
+    ld_vec<float, VEC>(bias + c, acc);
+    for (int j = 0; j < taps; ++j) {
+      const int u = t - (taps - 1) + j;
+      float v[VEC], g[VEC];
+      if (u >= t0) {
+        ld_vec<T, VEC>(x + static_cast<int64_t>(u) * ldx + c, v);
+      } else {
+        if (fresh) continue;
+        ld_vec<T, VEC>(state + (slot[s] * (taps - 1) + (u - t0 + taps - 1)) * ch + c, v);
+      }
+      ld_vec<float, VEC>(w + static_cast<int64_t>(j) * ch + c, g);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) acc[i] += g[i] * v[i];
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = silu_f(acc[i]);
+    st_vec<T, VEC>(out + static_cast<int64_t>(t) * ldo + c, acc);
+  }
+}
+// the last taps - 1 inputs of every span become its slot's state (row j of the new state is input len - (taps - 1) + j)
+template <class T>
+__global__ void mix_conv_state_kernel(const T* __restrict__ x, int64_t ldx, T* __restrict__ state, const int32_t* __restrict__ cu,
+                                      const int32_t* __restrict__ start, const int64_t* __restrict__ slot, int ch, int taps) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y;
+  if (c >= ch) return;
+  const int t0 = cu[s], len = cu[s + 1] - t0;
+  if (len <= 0) return;
+  const bool fresh = start[s] == 0;
+  T* st = state + slot[s] * static_cast<int64_t>(taps - 1) * ch + c;
+  for (int j = 0; j < taps - 1; ++j) {                  // reads row j + len > j: in place in increasing order
+    const int u = len - (taps - 1) + j;
+    T v = from_f<T>(0.f);
+    if (u >= 0) v = x[static_cast<int64_t>(t0 + u) * ldx + c];
+    else if (!fresh) v = st[static_cast<int64_t>(j + len) * ch];
+    st[static_cast<int64_t>(j) * ch] = v;
+  }
+}
+// one token per span: convolution and state shift in one pass
+template <class T, int VEC>
+__global__ void __launch_bounds__(128) mix_conv_step_kernel(const T* __restrict__ x, int64_t ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                                                            T* __restrict__ state, const int32_t* __restrict__ start, const int64_t* __restrict__ slot,
+                                                            T* __restrict__ out, int64_t ldo, int ch, int taps) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * VEC, s = blockIdx.y;
+  if (c >= ch) return;
+  const bool fresh = start[s] == 0;
+  T* st = state + slot[s] * static_cast<int64_t>(taps - 1) * ch + c;
+  float acc[VEC], g[VEC], cur[VEC];
+  ld_vec<float, VEC>(bias + c, acc);
+  ld_vec<T, VEC>(x + static_cast<int64_t>(s) * ldx + c, cur);
+  for (int j = 0; j < taps - 1; ++j) {
+    float v[VEC];
+    if (fresh) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+    } else {
+      ld_vec<T, VEC>(st + static_cast<int64_t>(j) * ch, v);
+    }
+    ld_vec<float, VEC>(w + static_cast<int64_t>(j) * ch + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] += g[i] * v[i];
+    if (j > 0) st_vec<T, VEC>(st + static_cast<int64_t>(j - 1) * ch, v);
+  }
+  ld_vec<float, VEC>(w + static_cast<int64_t>(taps - 1) * ch + c, g);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) acc[i] = silu_f(acc[i] + g[i] * cur[i]);
+  if (taps > 1) st_vec<T, VEC>(st + static_cast<int64_t>(taps - 2) * ch, cur);
+  st_vec<T, VEC>(out + static_cast<int64_t>(s) * ldo + c, acc);
+}
+
+// ---- latent attention, per token: a = [query latent qr | key-value latent r | shared rotary key rd]
+//   cq = rms(a_q) wq;   entry = [rms(a_kv) wkv | rotate(a_rot)] -> pool row kvslot[t] (and a packed copy when asked for)
+__device__ __forceinline__ void rope_cs(int64_t pos, double f, float& c, float& s) {
+  double a = static_cast<double>(pos) * f;
+  a -= 6.283185307179586 * rint(a * 0.15915494309189535);
+  sincosf(static_cast<float>(a), &s, &c);
+}
+template <class T>
+__global__ void __launch_bounds__(128) mix_latent_prep_kernel(const T* __restrict__ a, int64_t lda, int qr, int r, int rd, const float* __restrict__ wq,
+                                                              const float* __restrict__ wkv, const double* __restrict__ freq,
+                                                              const int64_t* __restrict__ pos, const int64_t* __restrict__ kvslot, T* __restrict__ cq,
+                                                              T* __restrict__ entry, T* __restrict__ pool, float eps) {
+  __shared__ float red[4];
+  const int64_t t = blockIdx.x;
+  const T* row = a + t * lda;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < qr; c += 128) { const float v = to_f<T>(row[c]); ss += v * v; }
+  float g = rsqrtf(block_sum<4>(ss, red) / qr + eps);
+  for (int c = threadIdx.x; c < qr; c += 128) cq[t * qr + c] = from_f<T>(to_f<T>(row[c]) * g * wq[c]);
+  row += qr;
+  ss = 0.f;
+  for (int c = threadIdx.x; c < r; c += 128) { const float v = to_f<T>(row[c]); ss += v * v; }
+  g = rsqrtf(block_sum<4>(ss, red) / r + eps);
+  T* pe = pool + kvslot[t] * (r + rd);
+  T* en = entry ? entry + t * (r + rd) : nullptr;
+  for (int c = threadIdx.x; c < r; c += 128) {
+    const T v = from_f<T>(to_f<T>(row[c]) * g * wkv[c]);
+    pe[c] = v;
+    if (en) en[c] = v;
+  }
+  const int half = rd / 2;
+  for (int i = threadIdx.x; i < half; i += 128) {
+    float cs, sn;
+    rope_cs(pos[t], freq[i], cs, sn);
+    const float u = to_f<T>(row[r + i]), v = to_f<T>(row[r + half + i]);
+    const T x0 = from_f<T>(u * cs - v * sn), x1 = from_f<T>(v * cs + u * sn);
+    pe[r + i] = x0; pe[r + half + i] = x1;
+    if (en) { en[r + i] = x0; en[r + half + i] = x1; }
+  }
+}
+// rotate columns [d, d + rd) of every head of q [T, H, dq] in place
+template <class T>
+__global__ void __launch_bounds__(128) mix_rope_kernel(T* __restrict__ q, int64_t ldq, int H, int dq, int d, int rd, const double* __restrict__ freq,
+                                                       const int64_t* __restrict__ pos) {
+  const int64_t t = blockIdx.x;
+  const int half = rd / 2;
+  __shared__ float sc[256], ss[256];
+  for (int i = threadIdx.x; i < half; i += 128) rope_cs(pos[t], freq[i], sc[i], ss[i]);
+  __syncthreads();
+  for (int e = threadIdx.x; e < H * half; e += 128) {
+    const int h = e / half, i = e % half;
+    T* p = q + t * ldq + static_cast<int64_t>(h) * dq + d;
+    const float u = to_f<T>(p[i]), v = to_f<T>(p[half + i]);
+    p[i] = from_f<T>(u * sc[i] - v * ss[i]);
+    p[half + i] = from_f<T>(v * sc[i] + u * ss[i]);
+  }
+}
+
+template <class T, int VEC>
+__global__ void mix_gelu_kernel(T* __restrict__ x, int64_t n) {
+  for (int64_t i = (static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x) * VEC; i < n; i += static_cast<int64_t>(gridDim.x) * blockDim.x * VEC) {
+    float v[VEC];
+    ld_vec<T, VEC>(x + i, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = gelu_tanh_f(v[j]);
+    st_vec<T, VEC>(x + i, v);
+  }
+}
+
+static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace prl
+
+using namespace prl;
+
+// dtype: 0 = bf16, 1 = fp32.  VEC = 8 when every row of every operand starts on a 16-byte boundary.
+#define MIX_DISPATCH(vec_, ...)                                                                      \
+  do {                                                                                               \
+    if (dtype == 0) {                                                                                \
+      using T = __nv_bfloat16;                                                                       \
+      if (vec_) { constexpr int VEC = 8; __VA_ARGS__; } else { constexpr int VEC = 1; __VA_ARGS__; } \
+    } else {                                                                                         \
+      using T = float;                                                                               \
+      if (vec_) { constexpr int VEC = 8; __VA_ARGS__; } else { constexpr int VEC = 1; __VA_ARGS__; } \
+    }                                                                                                \
+  } while (0)
+
+extern "C" int prl_mix_embed(const int64_t* ids, const void* emb, float* x, void* h, int rows, int W, int dtype, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const bool vec = W % 8 == 0 && al16(emb) && al16(x) && al16(h);
+  MIX_DISPATCH(vec, (mix_embed_kernel<T, VEC><<<rows, 128, 0, st>>>(ids, static_cast<const T*>(emb), x, static_cast<T*>(h), W)));
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_norm_add(const void* y, int64_t ldy, float* x, const float* w, const float* w_next, void* h, int rows, int W, float eps,
+                                int dtype, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const bool vec = W % 8 == 0 && ldy % 8 == 0 && al16(y) && al16(x) && al16(w) && al16(w_next) && al16(h);
+  MIX_DISPATCH(vec, (mix_norm_add_kernel<T, VEC><<<rows, 256, 0, st>>>(static_cast<const T*>(y), ldy, x, w, w_next, static_cast<T*>(h), W, eps)));
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_rms(const float* x, const float* w, void* h, int rows, int W, float eps, int dtype, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const bool vec = W % 8 == 0 && al16(x) && al16(w) && al16(h);
+  MIX_DISPATCH(vec, (mix_rms_kernel<T, VEC><<<rows, 256, 0, st>>>(x, w, static_cast<T*>(h), W, eps)));
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_gated_norm(const void* y, int64_t ldy, const void* z, int64_t ldz, const float* w, void* out, int64_t ldo, int rows, int groups,
+                                  int gs, float eps, int gate_first, int dtype, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const int64_t items = static_cast<int64_t>(rows) * groups;
+  const bool vec = gs % 8 == 0 && ldy % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && al16(y) && al16(z) && al16(w) && al16(out);
+  const bool wide = gs > 1024;
+  const int64_t grid = wide ? items : (items + 7) / 8;
+#define MIX_GN(GF, WPG)                                                                                                                   \
+  MIX_DISPATCH(vec, (mix_gated_norm_kernel<T, VEC, GF, WPG><<<static_cast<unsigned>(grid), 256, 0, st>>>(                                 \
+                        static_cast<const T*>(y), ldy, static_cast<const T*>(z), ldz, w, static_cast<T*>(out), ldo, items, groups, gs, eps)))
+  if (gate_first) {
+    if (wide) MIX_GN(true, 8); else MIX_GN(true, 1);
+  } else {
+    if (wide) MIX_GN(false, 8); else MIX_GN(false, 1);
+  }
+#undef MIX_GN
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+// x [total, ldx] -> out [total, ldo] and the carried taps of every span.  seq_of == nullptr: one token per span.
+extern "C" int prl_mix_conv(const void* x, int64_t ldx, const float* w, const float* bias, void* state, const int32_t* cu, const int32_t* start,
+                            const int64_t* slot, const int32_t* seq_of, void* out, int64_t ldo, int ch, int taps, int total, int spans, int dtype,
+                            cudaStream_t st) {
+  if (total <= 0 || spans <= 0) return 0;
+  if (spans > 65535 || taps < 1) return -220;
+  const bool vec = ch % 8 == 0 && ldx % 8 == 0 && ldo % 8 == 0 && al16(x) && al16(w) && al16(bias) && al16(state) && al16(out);
+  const int per = 128 * (vec ? 8 : 1);
+  const unsigned gx = (ch + per - 1) / per;
+  if (seq_of == nullptr) {
+    MIX_DISPATCH(vec, (mix_conv_step_kernel<T, VEC><<<dim3(gx, spans), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<T*>(state), start,
+                                                                                    slot, static_cast<T*>(out), ldo, ch, taps)));
+    PRL_CUDA_CHECK(cudaGetLastError());
+    return 0;
+  }
+  const int TT = total > 65535 * 4 ? 32 : 4;
+  const unsigned gy = (total + TT - 1) / TT;
+  if (gy > 65535) return -221;
+  if (TT == 4)
+    MIX_DISPATCH(vec, (mix_conv_kernel<T, VEC, 4><<<dim3(gx, gy), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,
+                                                                               start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
+  else
+    MIX_DISPATCH(vec, (mix_conv_kernel<T, VEC, 32><<<dim3(gx, gy), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,
+                                                                                start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
+  PRL_CUDA_CHECK(cudaGetLastError());
+  if (taps > 1) {
+    dim3 g2((ch + 127) / 128, spans);
+    if (dtype == 0)
+      mix_conv_state_kernel<__nv_bfloat16><<<g2, 128, 0, st>>>(static_cast<const __nv_bfloat16*>(x), ldx, static_cast<__nv_bfloat16*>(state), cu, start,
+                                                               slot, ch, taps);
+    else
+      mix_conv_state_kernel<float><<<g2, 128, 0, st>>>(static_cast<const float*>(x), ldx, static_cast<float*>(state), cu, start, slot, ch, taps);
+    PRL_CUDA_CHECK(cudaGetLastError());
+  }
+  return 0;
+}
+extern "C" int prl_mix_latent_prep(const void* a, int64_t lda, int qr, int r, int rd, const float* wq, const float* wkv, const double* freq,
+                                   const int64_t* pos, const int64_t* kvslot, void* cq, void* entry, void* pool, int rows, float eps, int dtype,
+                                   cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (dtype == 0)
+    mix_latent_prep_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>(static_cast<const __nv_bfloat16*>(a), lda, qr, r, rd, wq, wkv, freq, pos, kvslot,
+                                                                static_cast<__nv_bfloat16*>(cq), static_cast<__nv_bfloat16*>(entry),
+                                                                static_cast<__nv_bfloat16*>(pool), eps);
+  else
+    mix_latent_prep_kernel<float><<<rows, 128, 0, st>>>(static_cast<const float*>(a), lda, qr, r, rd, wq, wkv, freq, pos, kvslot,
+                                                        static_cast<float*>(cq), static_cast<float*>(entry), static_cast<float*>(pool), eps);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_rope(void* q, int64_t ldq, int H, int dq, int d, int rd, const double* freq, const int64_t* pos, int rows, int dtype,
+                            cudaStream_t st) {
+  if (rows <= 0 || rd <= 0) return 0;
+  if (rd > 512) return -222;
+  if (dtype == 0) mix_rope_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>(static_cast<__nv_bfloat16*>(q), ldq, H, dq, d, rd, freq, pos);
+  else mix_rope_kernel<float><<<rows, 128, 0, st>>>(static_cast<float*>(q), ldq, H, dq, d, rd, freq, pos);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_gelu(void* x, int64_t n, int dtype, cudaStream_t st) {
+  if (n <= 0) return 0;
+  const bool vec = n % 8 == 0 && al16(x);
+  const int64_t blocks = (n / (vec ? 8 : 1) + 255) / 256;
+  const unsigned grid = static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16);
+  MIX_DISPATCH(vec, (mix_gelu_kernel<T, VEC><<<grid > 0 ? grid : 1, 256, 0, st>>>(static_cast<T*>(x), n)));
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}

@@ -1,0 +1,146 @@
+// polyrl_b200 — gated linear recurrences, token by token: decode steps, short spans, fp32 runs and any head size.
+//
+//   kSsd   (Mamba-2 / state-space duality)   S = exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x
+//   kMlstm (xLSTM matrix memory)             m' = max(f + m, i),  S = e^(f+m-m') S + e^(i-m') k v^T,  n likewise with k alone,
+//                                            y = S^T q / (max(|n . q|, e^(-m')) + 1e-6);  m starts at 0
+//
+// One CTA = one (span, head, 32 value columns): lane = value column, warp w owns the state rows w, w + 8, ... in registers,
+// so a state row of 32 columns is one 128-byte line and a decode step reads and writes every state byte exactly once.
+#include "mixers.cuh"
+
+namespace prl {
+
+constexpr int kScanWarps = 8;
+constexpr int kScanVT = 32;
+
+template <class T, int MODE, int RN>
+__global__ void __launch_bounds__(kScanWarps * 32)
+mix_scan_kernel(ScanParams p) {
+  constexpr int NMAX = RN * kScanWarps;
+  __shared__ float s_q[2][NMAX], s_k[2][NMAX], s_n[NMAX];
+  __shared__ float s_red[2][kScanWarps][33], s_dot[2][kScanWarps];
+  const int vt = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
+  const int w = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+  const int t0 = p.cu[s], t1 = p.cu[s + 1];
+  if (t1 <= t0) return;
+  const bool fresh = p.start[s] == 0;
+  const int64_t slot = p.slot[s];
+  const int col = vt * kScanVT + lane;
+  const bool col_ok = col < p.V;
+  float* Sg = p.S + (slot * p.H + h) * static_cast<int64_t>(p.N) * p.V + col;
+  const T* q = static_cast<const T*>(p.q) + static_cast<int64_t>(h / p.rep) * p.N;
+  const T* k = static_cast<const T*>(p.k) + static_cast<int64_t>(h / p.rep) * p.N;
+  const T* v = static_cast<const T*>(p.v) + static_cast<int64_t>(h) * p.V;
+  T* out = static_cast<T*>(p.out) + static_cast<int64_t>(h) * p.V;
+
+  float S[RN];
+#pragma unroll
+  for (int i = 0; i < RN; ++i) {
+    const int n = i * kScanWarps + w;
+    S[i] = (!fresh && col_ok && n < p.N) ? Sg[static_cast<int64_t>(n) * p.V] : 0.f;
+  }
+  float m = 0.f;
+  if constexpr (MODE == kMlstm) {
+    const int64_t hb = slot * p.H + h;
+    if (!fresh) m = p.mst[hb];
+    for (int n = tid; n < NMAX; n += kScanWarps * 32) s_n[n] = (!fresh && n < p.N) ? p.nst[hb * p.N + n] : 0.f;
+  }
+  const float b0 = p.b0 ? p.b0[h] : 0.f, b1 = p.b1 ? p.b1[h] : 0.f;
+  const float a_neg = MODE == kSsd ? -expf(p.a_log[h]) : 0.f;
+  const float skip = (MODE == kSsd && p.d_skip) ? p.d_skip[h] : 0.f;
+
+  for (int t = t0; t < t1; ++t) {
+    const int b = t & 1;
+    for (int n = tid; n < NMAX; n += kScanWarps * 32) {
+      s_q[b][n] = n < p.N ? to_f<T>(q[static_cast<int64_t>(t) * p.ldq + n]) * p.qscale : 0.f;
+      s_k[b][n] = n < p.N ? to_f<T>(k[static_cast<int64_t>(t) * p.ldk + n]) : 0.f;
+    }
+    const float vv = col_ok ? to_f<T>(v[static_cast<int64_t>(t) * p.ldv + col]) : 0.f;
+    float keep, add, floor_ = 0.f;
+    if constexpr (MODE == kSsd) {
+      add = softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0);
+      keep = expf(a_neg * add);
+    } else {
+      const float gi = softcap_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0, p.cap);
+      const float gf = logsigmoid_f(softcap_f(p.g1[static_cast<int64_t>(t) * p.ldg + h] + b1, p.cap));
+      const float m2 = fmaxf(gf + m, gi);
+      keep = expf(gf + m - m2);
+      add = expf(gi - m2);
+      m = m2;
+      floor_ = expf(-m2);
+    }
+    __syncthreads();
+    const float av = add * vv;
+    float acc = 0.f;
+#pragma unroll
+    for (int i = 0; i < RN; ++i) {
+      const int n = i * kScanWarps + w;
+      S[i] = keep * S[i] + av * s_k[b][n];
+      acc += s_q[b][n] * S[i];
+    }
+    s_red[b][w][lane] = acc;
+    if constexpr (MODE == kMlstm) {
+      float d = 0.f;
+      for (int n = tid; n < NMAX; n += kScanWarps * 32) {        // the same thread owns s_n[n] for every token
+        const float nn = keep * s_n[n] + add * s_k[b][n];
+        s_n[n] = nn;
+        d += nn * s_q[b][n];
+      }
+      d = warp_sum(d);
+      if (lane == 0) s_dot[b][w] = d;
+    }
+    __syncthreads();
+    if (w == 0 && col_ok) {
+      float y = 0.f;
+#pragma unroll
+      for (int i = 0; i < kScanWarps; ++i) y += s_red[b][i][lane];
+      if constexpr (MODE == kSsd) {
+        y += skip * vv;
+      } else {
+        float d = 0.f;
+#pragma unroll
+        for (int i = 0; i < kScanWarps; ++i) d += s_dot[b][i];
+        y /= fmaxf(fabsf(d), floor_) + 1e-6f;
+      }
+      out[static_cast<int64_t>(t) * p.ldo + col] = from_f<T>(y);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RN; ++i) {
+    const int n = i * kScanWarps + w;
+    if (col_ok && n < p.N) Sg[static_cast<int64_t>(n) * p.V] = S[i];
+  }
+  if constexpr (MODE == kMlstm) {
+    if (last_tile(p.counter + s * p.H + h, gridDim.x)) {
+      const int64_t hb = slot * p.H + h;
+      for (int n = tid; n < p.N; n += kScanWarps * 32) p.nst[hb * p.N + n] = s_n[n];
+      if (tid == 0) p.mst[hb] = m;
+    }
+  }
+}
+
+template <class T, int MODE>
+static int launch_scan(const ScanParams& p, cudaStream_t st) {
+  dim3 grid((p.V + kScanVT - 1) / kScanVT, p.H, p.spans);
+  const int threads = kScanWarps * 32;
+  if (p.N <= 32) mix_scan_kernel<T, MODE, 4><<<grid, threads, 0, st>>>(p);
+  else if (p.N <= 64) mix_scan_kernel<T, MODE, 8><<<grid, threads, 0, st>>>(p);
+  else if (p.N <= 128) mix_scan_kernel<T, MODE, 16><<<grid, threads, 0, st>>>(p);
+  else if (p.N <= 256) mix_scan_kernel<T, MODE, 32><<<grid, threads, 0, st>>>(p);
+  else if (p.N <= 512) mix_scan_kernel<T, MODE, 64><<<grid, threads, 0, st>>>(p);
+  else return -201;
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
+}  // namespace prl
+
+using namespace prl;
+
+// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm
+extern "C" int prl_mix_scan(const ScanParams* p, int mode, int dtype, cudaStream_t st) {
+  if (p->spans <= 0) return 0;
+  if (p->spans > 65535 || p->H > 65535) return -202;
+  if (dtype == 0) return mode == kSsd ? launch_scan<__nv_bfloat16, kSsd>(*p, st) : launch_scan<__nv_bfloat16, kMlstm>(*p, st);
+  return mode == kSsd ? launch_scan<float, kSsd>(*p, st) : launch_scan<float, kMlstm>(*p, st);
+}

@@ -135,6 +135,34 @@ class EngineScheduler {
     return admitted;
   }
 
+  // A request whose tokens arrive over time (the caller supplies them step by step): admitted at once with the pages of its
+  // first tokens, grown by feed().  Throws when no slot or not enough pages are free; nothing is changed then.
+  int64_t open(std::vector<int64_t> tokens) {
+    if (free_slots_.empty()) throw std::runtime_error("no free batch slot");
+    const int64_t need = (static_cast<int64_t>(tokens.size()) + page_ - 1) / page_;
+    SchedRequest r;
+    r.blocks = kv_->alloc(need);
+    r.prompt = std::move(tokens);
+    r.cacheable = false;
+    r.slot = free_slots_.back();
+    free_slots_.pop_back();
+    r.live = true;
+    const int64_t h = next_++;
+    reqs_.emplace(h, std::move(r));
+    return h;
+  }
+  // append tokens to an open request and reserve the pages they need
+  void feed(int64_t h, const std::vector<int64_t>& tokens) {
+    SchedRequest& r = reqs_.at(h);
+    const int64_t total = static_cast<int64_t>(r.prompt.size() + tokens.size());
+    const int64_t more = (total + page_ - 1) / page_ - static_cast<int64_t>(r.blocks.size());
+    if (more > 0) {
+      const std::vector<int64_t> got = kv_->alloc(more);
+      r.blocks.insert(r.blocks.end(), got.begin(), got.end());
+    }
+    r.prompt.insert(r.prompt.end(), tokens.begin(), tokens.end());
+  }
+
   const SchedRequest& get(int64_t h) const { return reqs_.at(h); }
 
   // Flat arrays of one prefill chunk: request spans[i] = (handle, c, e) contributes prompt tokens [c, e).

@@ -1,7 +1,8 @@
 """Model architecture configs (decoder-only transformers) and named presets.
 
 Families: ``llama`` (Llama-2/3, Qwen2/2.5/3 — RMSNorm, RoPE, SwiGLU, GQA, optional qkv bias / qk-norm) and
-``gpt2`` (LayerNorm, learned positions, GELU MLP, biases).  Shapes for the presets follow the public
+``gpt2`` (LayerNorm, learned positions, GELU MLP, biases); ``hybrid`` (stacks whose layers each pick a sequence mixer,
+models/hybrid.py: Ludesun).  Shapes for the presets follow the public
 HF configs (the reference loads the same families through HF AutoModel:
 3rdparty/verl/verl/workers/fsdp_workers.py:269-577).
 """
@@ -14,7 +15,7 @@ from pathlib import Path
 
 @dataclass
 class ModelConfig:
-    family: str = "llama"            # "llama" | "gpt2"
+    family: str = "llama"            # "llama" | "gpt2" | "hybrid"
     vocab_size: int = 32000
     hidden_size: int = 4096
     intermediate_size: int = 11008
@@ -91,8 +92,11 @@ class ModelConfig:
     video_token_id: int = -1
     vision_start_token_id: int = -1
     vision_end_token_id: int = -1
+    # mixer stacks (family "hybrid", models/hybrid.py): one dict per layer, {"kind", "sizes", "ff", "weights_of"}
+    layers: tuple = ()
 
     def __post_init__(self):
+        self.layers = tuple(self.layers or ())
         self.extra_eos_token_ids = tuple(self.extra_eos_token_ids or ())        # json round trip gives a list
         self.mrope_section = tuple(self.mrope_section or ())
         self.dense_layers = tuple(int(i) for i in (self.dense_layers or ()))
@@ -111,8 +115,12 @@ class ModelConfig:
             self.head_dim = self.hidden_size // self.num_heads
         if self.num_heads % self.num_kv_heads != 0:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
-        if self.family not in ("llama", "gpt2"):
+        if self.family not in ("llama", "gpt2", "hybrid"):
             raise ValueError(f"unknown model family {self.family!r}")
+        if self.family == "hybrid":
+            from .hybrid import validate
+
+            validate(self)
         if self.num_experts:
             if self.family != "llama" or not (0 < self.num_experts_per_tok <= self.num_experts) or self.moe_intermediate_size <= 0:
                 raise ValueError("MoE needs the llama family, 0 < num_experts_per_tok <= num_experts and moe_intermediate_size > 0")
@@ -159,6 +167,10 @@ class ModelConfig:
         return h * (self.q_size + 2 * self.kv_size) + self.q_size * h
 
     def num_params(self) -> int:
+        if self.family == "hybrid":
+            from .hybrid import num_params
+
+            return num_params(self)
         h, f, v = self.hidden_size, self.intermediate_size, self.vocab_size
         if self.family == "llama":
             mlp = 3 * h * f if self.mlp_act == "swiglu" else 2 * h * f + 2
@@ -208,6 +220,8 @@ class ModelConfig:
     @classmethod
     def from_hf_config(cls, hf: dict) -> "ModelConfig":
         """Translate a HuggingFace ``config.json`` dict (Llama / Mistral / Qwen2 / Qwen3 / Qwen3-MoE / Qwen2-VL / GPT-2)."""
+        if hf.get("architecture") in ARCHITECTURES:
+            return ARCHITECTURES[hf["architecture"]](hf)
         mt = hf.get("model_type", "llama")
         if mt == "gpt2":
             return cls(family="gpt2", vocab_size=hf["vocab_size"], hidden_size=hf["n_embd"],
@@ -361,6 +375,16 @@ class ModelConfig:
                    sliding_window=(hf.get("sliding_window") if (mt in ("mistral", "mixtral") or hf.get("use_sliding_window")) else None),
                    hf_model_type=("glm4v" if hf.get("_glm4v") else mt) if mt in ("mistral", "mixtral", "glm", "glm4", "qwen2_moe", "glm4_moe", "deepseek_v2", "deepseek_v3", "apertus") else "",
                    name=hf.get("_name_or_path", mt), **vis_kw, **{**moe_kw, **vl_moe_kw}, **{**glm_kw, **mla_kw, **act_kw})
+
+
+def _ludesun(hf: dict) -> ModelConfig:
+    from .hybrid import ludesun_config
+
+    return ludesun_config(hf)
+
+
+# designs whose config.json names an ``architecture`` instead of a ``model_type``
+ARCHITECTURES = {"Ludesun": _ludesun}
 
 
 def _qwen_dense_layers(hf: dict) -> tuple:
@@ -563,6 +587,22 @@ PRESETS: dict[str, dict] = {
     "tiny-llama-128": dict(family="llama", vocab_size=1024, hidden_size=512, intermediate_size=1024, num_layers=2,
                            num_heads=4, num_kv_heads=2, head_dim=128, max_position_embeddings=1024,
                            rope_theta=10000.0, eos_token_id=1, bos_token_id=2, pad_token_id=0),
+    # Ludesun stacks (models/hybrid.py): a small test size and one with the layer sizes of a model of a few billion parameters
+    "tiny-ludesun": dict(family="hybrid", vocab_size=512, hidden_size=256, intermediate_size=384, num_layers=4, num_heads=1, num_kv_heads=1,
+                         rms_norm_eps=1e-5, eos_token_id=-1, bos_token_id=-1, hf_model_type="ludesun", layers=(
+                             dict(kind="ssd", sizes=dict(heads=8, vdim=32, state=64, groups=2, conv=4, norm_groups=4), ff=384, weights_of=0),
+                             dict(kind="latent", sizes=dict(heads=4, dim=48, rot_dim=16, vdim=40, kv_rank=96, q_rank=64, scale=0.125, rot_base=10000.0),
+                                  ff=384, weights_of=1),
+                             dict(kind="mlstm", sizes=dict(heads=2, dim=64, vdim=96, gate_cap=15.0), ff=0, weights_of=2),
+                             dict(kind="ssd", sizes=dict(heads=8, vdim=32, state=64, groups=2, conv=4, norm_groups=4), ff=384, weights_of=0))),
+    "ludesun-4b": dict(family="hybrid", vocab_size=128256, hidden_size=4096, intermediate_size=14336, num_layers=16, num_heads=1, num_kv_heads=1,
+                       rms_norm_eps=1e-5, eos_token_id=-1, bos_token_id=-1, hf_model_type="ludesun", layers=tuple(
+                           dict(ff=14336, weights_of=i, **([
+                               dict(kind="mlstm", sizes=dict(heads=8, dim=256, vdim=512, gate_cap=15.0)),
+                               dict(kind="ssd", sizes=dict(heads=128, vdim=64, state=128, groups=8, conv=4, norm_groups=8)),
+                               dict(kind="latent", sizes=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536,
+                                                              scale=192 ** -0.5, rot_base=500000.0)),
+                               dict(kind="ssd", sizes=dict(heads=128, vdim=64, state=128, groups=8, conv=4, norm_groups=8))][i % 4])) for i in range(16))),
     "tiny-gpt2": dict(family="gpt2", vocab_size=512, hidden_size=128, intermediate_size=512, num_layers=2,
                       num_heads=4, num_kv_heads=4, max_position_embeddings=256, rms_norm_eps=1e-5,
                       tie_word_embeddings=True, eos_token_id=1, bos_token_id=2, pad_token_id=0),

@@ -176,6 +176,10 @@ def _vision_tensors(cfg: ModelConfig, ck: HFCheckpoint) -> dict[str, torch.Tenso
 
 def load_state_dict(cfg: ModelConfig, path: str | Path) -> dict[str, torch.Tensor]:
     ck = HFCheckpoint(path)
+    if cfg.family == "hybrid":
+        from .hybrid import ludesun_state_dict
+
+        return ludesun_state_dict(cfg, ck.get)
     embed, head = _embed_head(cfg, ck)
     out = {**embed, **head}
     if cfg.vision is not None:
@@ -190,6 +194,8 @@ def load_into_engine(engine, path: str | Path) -> int:
     """Fill every ZeRO unit of ``engine`` from the checkpoint; returns the number of tensors loaded.  Value-head engines keep
     their freshly initialised head projection (an LM checkpoint has none)."""
     cfg = engine.cfg
+    if cfg.family == "hybrid":
+        raise NotImplementedError("mixer stacks are served by the rollout engine only; training them is not implemented")
     ck = HFCheckpoint(path)
     embed, head = _embed_head(cfg, ck)
     n = 0
@@ -230,6 +236,10 @@ def hf_config_dict(cfg: ModelConfig) -> dict:
 
 
 def _lm_config_dict(cfg: ModelConfig) -> dict:
+    if cfg.family == "hybrid":
+        from .hybrid import ludesun_config_dict
+
+        return ludesun_config_dict(cfg)
     if cfg.family == "gpt2":
         return {"model_type": "gpt2", "architectures": ["GPT2LMHeadModel"], "vocab_size": cfg.vocab_size, "n_embd": cfg.hidden_size,
                 "n_inner": cfg.intermediate_size, "n_layer": cfg.num_layers, "n_head": cfg.num_heads, "n_positions": cfg.max_position_embeddings,

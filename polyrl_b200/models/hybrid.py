@@ -1,0 +1,412 @@
+"""Mixer stacks: decoder-only models whose layers each choose their own sequence mixer, served by the rollout engine.
+
+A layer is  x <- x + norm1(mixer(x)),  x <- x + norm2(ff(x))  — RMS norms on the sublayer outputs only, fp32 residual stream.
+Mixers (``LAYER_KINDS``): ``ssd`` (Mamba-2 state-space duality: causal convolution, scalar-decay recurrence, gate before a grouped
+norm), ``mlstm`` (xLSTM matrix memory with exponential gates) and ``latent`` (multi-head latent attention with query bottleneck,
+rotary key part and a softmax sink).  A layer may reuse the weights of an earlier one (``weights_of``) while keeping a cache or
+state of its own.
+
+``ModelConfig.layers`` holds one plain dict per layer: {"kind", "sizes", "ff" (0: no feed-forward), "weights_of" (own index when the
+layer owns its weights)}.  ``ludesun_config`` reads the Ludesun ``config.json``; another design built from the same mixers needs only
+another reader and name map.
+
+Everything is one function of a packed step (ops/mixers.py ``SpanBatch``): prompts, portions of prompts and decoded tokens take the
+same path, and the kernels pick chunked or token-by-token work by span length.
+"""
+from __future__ import annotations
+
+import torch
+import torch.nn.functional as F
+
+from .. import ops
+from ..ops import mixers as M
+from .config import ModelConfig
+
+LAYER_KINDS = ("ssd", "mlstm", "latent")
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def owner(cfg: ModelConfig, i: int) -> int:
+    """Index of the layer whose weights layer ``i`` uses."""
+    seen = set()
+    while cfg.layers[i]["weights_of"] != i:
+        if i in seen:
+            raise ValueError("weights_of forms a cycle")
+        seen.add(i)
+        i = cfg.layers[i]["weights_of"]
+    return i
+
+
+def validate(cfg: ModelConfig) -> None:
+    if len(cfg.layers) != cfg.num_layers or not cfg.layers:
+        raise ValueError("a mixer stack needs one entry of ``layers`` per layer")
+    for i, lay in enumerate(cfg.layers):
+        kind, m = lay["kind"], lay["sizes"]
+        if kind not in LAYER_KINDS:
+            raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+        if not 0 <= lay["weights_of"] < cfg.num_layers:
+            raise ValueError(f"layer {i}: weights_of is not a layer")
+        j = owner(cfg, i)
+        if {k: v for k, v in cfg.layers[j].items() if k != "weights_of"} != {k: v for k, v in lay.items() if k != "weights_of"}:
+            raise ValueError(f"layer {i} differs from layer {j} whose weights it uses")
+        if kind == "ssd" and (m["heads"] % m["groups"] or (m["heads"] * m["vdim"]) % m["norm_groups"] or m["conv"] < 1 or m["state"] > 512):
+            raise ValueError(f"layer {i}: ssd sizes")
+        if kind == "mlstm" and (m["dim"] > 512 or m["gate_cap"] <= 0):
+            raise ValueError(f"layer {i}: mlstm sizes")
+        if kind == "latent" and (m["rot_dim"] % 2 or m["rot_dim"] > 512 or m["kv_rank"] > 1024):
+            raise ValueError(f"layer {i}: latent sizes")
+
+
+# --------------------------------------------------------------------------------------------
+# parameters (our names; weights of a layer that reuses another's exist once)
+# --------------------------------------------------------------------------------------------
+def layer_param_specs(cfg: ModelConfig, i: int) -> list[tuple[str, tuple[int, ...]]]:
+    lay, w = cfg.layers[i], cfg.hidden_size
+    m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
+    out: list[tuple[str, tuple[int, ...]]] = [("norm1", (w,))]
+    if lay["kind"] == "ssd":            # one projection [gate | x | B | C]; the step sizes keep their own fp32-accumulated one
+        ch = h * v + 2 * m["groups"] * m["state"]
+        out += [("w_in", (h * v + ch, w)), ("w_dt", (h, w)), ("conv_w", (ch, m["conv"])), ("conv_b", (ch,)), ("dt_bias", (h,)), ("a_log", (h,)),
+                ("d_skip", (h,)), ("gn", (h * v,)), ("wo", (w, h * v))]
+    elif lay["kind"] == "mlstm":        # [q | k | v | output gate] and [input gate | forget gate]
+        out += [("w_in", (2 * h * m["dim"] + 2 * h * v, w)), ("w_if", (2 * h, w)), ("b_if", (2 * h,)), ("gn", (h * v,)), ("wo", (w, h * v))]
+    else:                               # [query latent | key-value latent | shared rotary key]
+        r, qr, d, rd = m["kv_rank"], m["q_rank"], m["dim"], m["rot_dim"]
+        out += [("wa", (qr + r + rd, w)), ("q_ln", (qr,)), ("kv_ln", (r,)), ("wq_up", (h * (d + rd), qr)), ("wk_up", (h * d, r)), ("wv_up", (h * v, r)),
+                ("sink", (h,)), ("wo", (w, h * v))]
+    if lay["ff"]:
+        out += [("norm2", (w,)), ("wup", (lay["ff"], w)), ("wdown", (w, lay["ff"]))]
+    return out
+
+
+def num_params(cfg: ModelConfig) -> int:
+    n = 2 * cfg.vocab_size * cfg.hidden_size + cfg.hidden_size
+    for i in range(cfg.num_layers):
+        if owner(cfg, i) == i:
+            for _, shp in layer_param_specs(cfg, i):
+                k = 1
+                for s in shp:
+                    k *= s
+                n += k
+    return n
+
+
+def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) -> bool:
+    """Random init of the tensors the generic rules do not cover; False when they do."""
+    base = name.split(".")[-1]
+    if base in ("norm1", "norm2", "gn", "q_ln", "kv_ln", "d_skip"):
+        t.fill_(1.0)
+    elif base in ("conv_b", "sink"):
+        t.zero_()
+    elif base == "a_log":
+        t.copy_(torch.linspace(-2.0, 1.0, t.numel(), device=t.device))
+    elif base == "dt_bias":
+        t.fill_(-2.0)
+    elif base == "b_if":
+        t.zero_()
+        t[t.numel() // 2:] = 3.0
+    elif base == "conv_w":
+        t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
+    elif base in ("w_in", "w_dt", "w_if", "wa", "wq_up", "wk_up", "wv_up", "wo", "wup", "wdown"):
+        t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
+    else:
+        return False
+    return True
+
+
+# --------------------------------------------------------------------------------------------
+# run-time weights
+# --------------------------------------------------------------------------------------------
+_VECTORS = ("norm1", "norm2", "gn", "q_ln", "kv_ln", "conv_b", "dt_bias", "a_log", "d_skip", "b_if", "sink")
+
+
+def query_width(m: dict, dtype: torch.dtype, is_cuda: bool) -> int:
+    """Per-head query width at run time: padded to what the packed attention kernel takes (128 or 192), or exact when that kernel cannot
+    serve the sizes (fp32, wider heads)."""
+    d = m["dim"] + m["rot_dim"]
+    return d if not expands(m, dtype, is_cuda) else (128 if d <= 128 else 192)
+
+
+def expands(m: dict, dtype: torch.dtype, is_cuda: bool) -> bool:
+    """Long spans of this layer run on expanded keys and values (packed tcgen05 attention) instead of the absorbed form."""
+    return is_cuda and dtype == torch.bfloat16 and m["vdim"] <= 128 and m["dim"] + m["rot_dim"] <= 192 and (m["kv_rank"] + m["rot_dim"]) % 8 == 0
+
+
+def _pad_heads(w: torch.Tensor, heads: int, rows: int) -> torch.Tensor:
+    """[heads * n, in] -> [heads * rows, in], zero rows behind every head's own."""
+    t = w.reshape(heads, -1, w.shape[-1])
+    return F.pad(t, (0, 0, 0, rows - t.shape[1])).reshape(heads * rows, -1)
+
+
+def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: dict | None = None) -> dict:
+    """Weights of layer ``i`` in run-time form: vectors in fp32, matrices in ``dtype`` with the layouts the kernels want.  ``old`` (the
+    previous result) is overwritten in place where shapes agree, so captured graphs stay valid across weight updates."""
+    lay = cfg.layers[i]
+    m, h = lay["sizes"], lay["sizes"]["heads"]
+    is_cuda = w["norm1"].is_cuda
+    out: dict[str, torch.Tensor] = {}
+    for k, t in w.items():
+        if k in _VECTORS:
+            out[k] = t.float().contiguous()
+        elif k == "conv_w":
+            out[k] = t.float().t().contiguous()                     # [taps, channels]
+        elif k not in ("wq_up", "wk_up", "wv_up"):
+            t = t if t.dtype == dtype else t.to(dtype)
+            if k == "w_in" and is_cuda and t.shape[0] % 8:
+                t = F.pad(t, (0, 0, 0, _pad8(t.shape[0]) - t.shape[0]))
+            out[k] = t.contiguous()
+    if lay["kind"] == "latent":
+        d, rd, v, r = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        dq = query_width(m, dtype, is_cuda)
+        up = {k: w[k].to(dtype) for k in ("wq_up", "wk_up", "wv_up")}
+        out["wq"] = _pad_heads(up["wq_up"], h, dq).contiguous()
+        out["wk_abs"] = up["wk_up"].reshape(h, d, r).contiguous()                       # folds the key up-projection into a query
+        out["wv_abs"] = up["wv_up"].reshape(h, v, r).transpose(1, 2).contiguous()       # folds the value up-projection into an output
+        out["freq"] = M.rope_frequencies(rd, m["rot_base"], w["norm1"].device)
+        if expands(m, dtype, is_cuda):
+            # cache row -> every head's [key | rotary key | 0] and [value | 0]: the rotary part is copied by identity rows
+            wk = torch.zeros(h, dq, r + rd, dtype=dtype, device=w["norm1"].device)
+            wk[:, :d, :r] = up["wk_up"].reshape(h, d, r)
+            wk[:, d:d + rd, r:] = torch.eye(rd, dtype=dtype, device=wk.device)
+            wv = torch.zeros(h, 128, r + rd, dtype=dtype, device=wk.device)
+            wv[:, :v, :r] = up["wv_up"].reshape(h, v, r)
+            out["w_expand"] = torch.cat([wk.reshape(h * dq, -1), wv.reshape(h * 128, -1)]).contiguous()
+    if old is not None:
+        for k, t in out.items():
+            o = old.get(k)
+            derived = k not in w or t.data_ptr() != w[k].data_ptr()
+            if derived and o is not None and o.shape == t.shape and o.dtype == t.dtype:
+                out[k] = o.copy_(t)
+    return out
+
+
+def prepare(cfg: ModelConfig, layer_w: list[dict], dtype: torch.dtype, old: list[dict] | None = None) -> list[dict]:
+    done: dict[int, dict] = {}
+    for i in range(cfg.num_layers):
+        j = owner(cfg, i)
+        if j not in done:
+            done[j] = prepare_layer(cfg, j, layer_w[j], dtype, old[j] if old else None)
+    return [done[owner(cfg, i)] for i in range(cfg.num_layers)]
+
+
+def prepare_head(head_w: dict, dtype: torch.dtype, old: dict | None = None) -> dict:
+    norm = head_w["norm_w"].float().contiguous()
+    if old is not None and norm.data_ptr() != head_w["norm_w"].data_ptr():
+        norm = old["norm_w"].copy_(norm)
+    return {"norm_w": norm, "lm_head": head_w["lm_head"].to(dtype)}
+
+
+# --------------------------------------------------------------------------------------------
+# caches and states
+# --------------------------------------------------------------------------------------------
+def cache_bytes(cfg: ModelConfig, dtype: torch.dtype) -> tuple[int, int]:
+    """(paged-cache bytes per token, state bytes per slot) of the whole stack."""
+    es = torch.empty(0, dtype=dtype).element_size()
+    tok = slot = 0
+    for lay in cfg.layers:
+        m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
+        if lay["kind"] == "latent":
+            tok += (m["kv_rank"] + m["rot_dim"]) * es
+        elif lay["kind"] == "ssd":
+            slot += 4 * h * v * m["state"] + es * (m["conv"] - 1) * (h * v + 2 * m["groups"] * m["state"])
+        else:
+            slot += 4 * h * (m["dim"] * v + m["dim"] + 1)
+    return tok, slot
+
+
+def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device, dtype: torch.dtype) -> dict[str, torch.Tensor]:
+    """Cache of layer ``i``: a page pool (attention) or state pools (recurrences; slot 0 belongs to idle batch rows)."""
+    lay = cfg.layers[i]
+    m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
+    if lay["kind"] == "latent":
+        return {"pool": torch.zeros(num_blocks, 1, M.PAGE, m["kv_rank"] + m["rot_dim"], device=device, dtype=dtype)}
+    f32 = dict(device=device, dtype=torch.float32)
+    if lay["kind"] == "ssd":
+        ch = h * v + 2 * m["groups"] * m["state"]
+        return {"S": torch.zeros(num_slots, h, m["state"], v, **f32), "conv": torch.zeros(num_slots, m["conv"] - 1, ch, device=device, dtype=dtype)}
+    return {"S": torch.zeros(num_slots, h, m["dim"], v, **f32), "n": torch.zeros(num_slots, h, m["dim"], **f32), "m": torch.zeros(num_slots, h, **f32)}
+
+
+def copy_cache(cache: dict, src_pages: torch.Tensor, dst_pages: torch.Tensor, src_slots: torch.Tensor, dst_slots: torch.Tensor) -> None:
+    """Duplicate pages / state slots of one layer (the members of an n-sample group continue from their donor's prompt)."""
+    for k, t in cache.items():
+        src, dst = (src_pages, dst_pages) if k == "pool" else (src_slots, dst_slots)
+        if src.numel():
+            t.index_copy_(0, dst, t.index_select(0, src))
+
+
+# --------------------------------------------------------------------------------------------
+# forward
+# --------------------------------------------------------------------------------------------
+def _ssd(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
+    inner, gn = m["heads"] * m["vdim"], m["groups"] * m["state"]
+    p = ops.linear(h, w["w_in"])
+    dt = M.linear_f32(h, w["w_dt"])
+    z, xbc = p[:, :inner], p[:, inner:2 * inner + 2 * gn]
+    xbc = M.conv_silu(xbc, w["conv_w"], w["conv_b"], cache["conv"], b)
+    y = M.scan(M.SSD, xbc[:, inner + gn:], xbc[:, inner:inner + gn], xbc[:, :inner],
+               M.Gates(dt, b0=w["dt_bias"], a_log=w["a_log"], d_skip=w["d_skip"]), 1.0, cache, b)
+    return M.gated_norm(y, z, w["gn"], m["norm_groups"], cfg.rms_norm_eps, True)
+
+
+def _mlstm(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
+    nh = m["heads"]
+    hd, hv = nh * m["dim"], nh * m["vdim"]
+    p = ops.linear(h, w["w_in"])
+    g = M.linear_f32(h, w["w_if"])
+    o = M.scan(M.MLSTM, p[:, :hd], p[:, hd:2 * hd], p[:, 2 * hd:2 * hd + hv],
+               M.Gates(g[:, :nh], g[:, nh:], w["b_if"][:nh], w["b_if"][nh:], cap=float(m["gate_cap"])), m["dim"] ** -0.5, cache, b)
+    return M.gated_norm(o, p[:, 2 * hd + hv:2 * hd + 2 * hv], w["gn"], nh, cfg.rms_norm_eps, False)
+
+
+def _latent(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
+    nh, d, rd, v, r = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    t, pool, scale = b.tokens, cache["pool"], float(m["scale"])
+    tl = b.t_long if expands(m, h.dtype, h.is_cuda) else 0          # tokens served on expanded keys
+    cq, entry = M.latent_prep(ops.linear(h, w["wa"]), w["q_ln"], w["kv_ln"], w["freq"], pool, b, cfg.rms_norm_eps, tl > 0 and b.gather is None)
+    q = ops.linear(cq, w["wq"]).view(t, nh, -1)
+    M.rope_(q, d, w["freq"], b.pos)
+    out = []
+    if tl:
+        if b.gather is None:
+            src, cu_k = entry[:tl], b.cu[:b.n_long + 1]
+        else:
+            src, cu_k = pool.view(-1, r + rd).index_select(0, b.gather[0]), b.gather[1]
+        kv = ops.linear(src, w["w_expand"])
+        dq = q.shape[-1]
+        k, vv = kv[:, :nh * dq].view(-1, nh, dq), kv[:, nh * dq:].view(-1, nh, 128)
+        a = M.sink_attention_varlen(q[:tl], k, vv, b.cu[:b.n_long + 1], cu_k, scale, w["sink"])
+        out.append(a[..., :v].reshape(tl, nh * v))
+    if tl < t:
+        qs = q[tl:]
+        q_lat = torch.bmm(qs[..., :d].transpose(0, 1), w["wk_abs"])
+        lo = b.n_long if tl else 0
+        seq_of = None if b.seq_of is None or tl else b.seq_of[tl:]
+        o_lat = M.latent_attention(q_lat, qs, d, pool, b.table[lo:], seq_of, b.kv_len[tl:], w["sink"], scale, b.max_len)
+        out.append(torch.bmm(o_lat, w["wv_abs"]).transpose(0, 1).reshape(t - tl, nh * v))
+    return out[0] if len(out) == 1 else torch.cat(out)
+
+
+_MIXERS = {"ssd": _ssd, "mlstm": _mlstm, "latent": _latent}
+
+
+def embed_forward(cfg: ModelConfig, w: dict, ids: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    return M.embed(ids, w["embed"])
+
+
+def layer_step(cfg: ModelConfig, i: int, w: dict, x: torch.Tensor, h: torch.Tensor, cache: dict, b: M.SpanBatch,
+               w_next: torch.Tensor | None = None) -> torch.Tensor:
+    """Layer ``i`` on one packed step.  x: fp32 residual stream, updated in place; h: x in the activation dtype (the sublayers read x
+    itself).  Returns the next h — or the final norm of x when its weight is given as ``w_next``."""
+    lay, eps = cfg.layers[i], cfg.rms_norm_eps
+    y = ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h, cache, b), w["wo"])
+    if not lay["ff"]:
+        return M.norm_add_(y, x, w["norm1"], eps, w_next)
+    h = M.norm_add_(y, x, w["norm1"], eps)
+    y = ops.linear(M.linear_gelu(h, w["wup"]), w["wdown"])
+    return M.norm_add_(y, x, w["norm2"], eps, w_next)
+
+
+# --------------------------------------------------------------------------------------------
+# Ludesun: configuration and checkpoint names
+# --------------------------------------------------------------------------------------------
+_LUDESUN_KIND = {"mamba2": "ssd", "mlstm": "mlstm", "latent_attention": "latent"}
+_LUDESUN_SIZES = {"ssd": ("heads", "vdim", "state", "groups", "conv", "norm_groups"), "mlstm": ("heads", "dim", "vdim", "gate_cap"),
+                  "latent": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "scale")}
+
+
+def ludesun_config(hf: dict) -> ModelConfig:
+    """``config.json`` of a Ludesun model: vocab, width, norm.eps and one entry of ``layers`` per layer."""
+    layers = []
+    for i, e in enumerate(hf["layers"]):
+        if e["type"] not in _LUDESUN_KIND:
+            raise ValueError(f"Ludesun layer {i}: unknown mixer type {e['type']!r}")
+        kind = _LUDESUN_KIND[e["type"]]
+        sizes = {k: e["mixer"][k] for k in _LUDESUN_SIZES[kind]}
+        if kind == "latent":
+            if e["mixer"]["rot"]["dims"] != sizes["rot_dim"]:
+                raise ValueError(f"Ludesun layer {i}: rot.dims and rot_dim differ")
+            sizes["rot_base"] = float(e["mixer"]["rot"]["base"])
+        mlp = e.get("mlp")
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"Ludesun layer {i}: feed-forward kind {mlp['kind']!r}")
+        layers.append({"kind": kind, "sizes": sizes, "ff": int(mlp["ff"]) if mlp else 0, "weights_of": int(e.get("weights_of", i))})
+    return ModelConfig(family="hybrid", vocab_size=hf["vocab"], hidden_size=hf["width"], num_layers=len(layers), layers=tuple(layers),
+                       intermediate_size=max([x["ff"] for x in layers] + [1]), num_heads=1, num_kv_heads=1, rms_norm_eps=float(hf["norm"]["eps"]),
+                       eos_token_id=-1, bos_token_id=-1, pad_token_id=0, hf_model_type="ludesun", name="ludesun")
+
+
+def ludesun_config_dict(cfg: ModelConfig) -> dict:
+    """Inverse of ``ludesun_config``."""
+    back = {v: k for k, v in _LUDESUN_KIND.items()}
+    layers = []
+    for i, lay in enumerate(cfg.layers):
+        mx = {k: lay["sizes"][k] for k in _LUDESUN_SIZES[lay["kind"]]}
+        if lay["kind"] == "latent":
+            mx["rot"] = {"dims": mx["rot_dim"], "base": lay["sizes"]["rot_base"]}
+        e = {"type": back[lay["kind"]], "mixer": mx, "mlp": {"kind": "dense", "ff": lay["ff"]} if lay["ff"] else None}
+        if lay["weights_of"] != i:
+            e["weights_of"] = lay["weights_of"]
+        layers.append(e)
+    return {"architecture": "Ludesun", "vocab": cfg.vocab_size, "width": cfg.hidden_size, "norm": {"eps": cfg.rms_norm_eps}, "layers": layers}
+
+
+def _ludesun_parts(kind: str, ff: int) -> list[tuple[str, list[str]]]:
+    """(our name, checkpoint names whose rows it stacks) of one layer; the SSD input projection is split separately."""
+    mix = {"ssd": [("conv_w", ["conv"]), ("conv_b", ["conv.b"]), ("dt_bias", ["dt_bias"]), ("a_log", ["A_log"]), ("d_skip", ["D"])],
+           "mlstm": [("w_in", ["q", "k", "v", "g"]), ("w_if", ["i", "f"]), ("b_if", ["i.b", "f.b"])],
+           "latent": [("wa", ["dq", "dkv"]), ("q_ln", ["dq.norm"]), ("kv_ln", ["dkv.norm"]), ("wq_up", ["uq"]), ("wk_up", ["uk"]), ("wv_up", ["uv"]),
+                      ("sink", ["sink"])]}[kind]
+    if kind != "latent":
+        mix = mix + [("gn", ["norm"])]
+    out = [(n, ["mix." + s for s in src]) for n, src in mix + [("wo", ["o"])]]
+    out.append(("norm1", ["norm1"]))
+    if ff:
+        out += [("norm2", ["norm2"]), ("wup", ["mlp.up"]), ("wdown", ["mlp.down"])]
+    return out
+
+
+def ludesun_layer(cfg: ModelConfig, i: int, get) -> dict[str, torch.Tensor]:
+    """Tensors of layer ``i`` (which owns its weights) in our names; ``get`` reads a checkpoint tensor by name."""
+    lay, p = cfg.layers[i], f"l{i}."
+    out = {n: (torch.cat([get(p + s) for s in src]) if len(src) > 1 else get(p + src[0])) for n, src in _ludesun_parts(lay["kind"], lay["ff"])}
+    if lay["kind"] == "ssd":
+        w, nh = get(p + "mix.in"), lay["sizes"]["heads"]
+        out["w_in"], out["w_dt"] = w[:-nh], w[-nh:]
+    return out
+
+
+def ludesun_state_dict(cfg: ModelConfig, get) -> dict[str, torch.Tensor]:
+    out = {"embed": get("embed"), "norm_w": get("final.norm"), "lm_head": get("head")}
+    for i in range(cfg.num_layers):
+        if owner(cfg, i) == i:
+            out.update({f"layers.{i}.{k}": t for k, t in ludesun_layer(cfg, i, get).items()})
+    return out
+
+
+def ludesun_export(cfg: ModelConfig, sd: dict) -> dict[str, torch.Tensor]:
+    """Our names -> checkpoint names (inverse of ``ludesun_state_dict``)."""
+    out = {"embed": sd["embed"], "final.norm": sd["norm_w"], "head": sd["lm_head"]}
+    for i, lay in enumerate(cfg.layers):
+        if owner(cfg, i) != i:
+            continue
+        p, q, m = f"l{i}.", f"layers.{i}.", lay["sizes"]
+        rows = {}
+        if lay["kind"] == "mlstm":
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            rows = {"mix.q": hd, "mix.k": hd, "mix.v": hv, "mix.g": hv, "mix.i": m["heads"], "mix.f": m["heads"], "mix.i.b": m["heads"], "mix.f.b": m["heads"]}
+        elif lay["kind"] == "latent":
+            rows = {"mix.dq": m["q_rank"], "mix.dkv": m["kv_rank"] + m["rot_dim"]}
+        for n, src in _ludesun_parts(lay["kind"], lay["ff"]):
+            t = sd[q + n]
+            if len(src) == 1:
+                out[p + src[0]] = t
+            else:
+                for s, piece in zip(src, t.split([rows[s] for s in src])):
+                    out[p + s] = piece.clone()
+        if lay["kind"] == "ssd":
+            out[p + "mix.in"] = torch.cat([sd[q + "w_in"], sd[q + "w_dt"]])
+    return out

@@ -36,6 +36,10 @@ def is_sparse_layer(cfg: ModelConfig, i: int | None) -> bool:
 
 def layer_param_specs(cfg: ModelConfig, i: int | None = None) -> ParamSpec:
     """Parameters of decoder block ``i`` (MoE stacks may mix sparse and dense blocks: ``cfg.dense_layers``)."""
+    if cfg.family == "hybrid":
+        from . import hybrid
+
+        return hybrid.layer_param_specs(cfg, i or 0)
     h, f = cfg.hidden_size, cfg.intermediate_size
     qkv = cfg.q_size + 2 * cfg.kv_size
     if cfg.family == "llama":
@@ -94,6 +98,11 @@ def head_param_specs(cfg: ModelConfig) -> ParamSpec:
 def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator: torch.Generator | None = None) -> None:
     """Random init (weights ~ N(0, 0.02), norm gains 1, biases 0), in place, any dtype/device."""
     base = name.split(".")[-1]
+    if cfg.family == "hybrid":
+        from . import hybrid
+
+        if hybrid.init_param_(name, t, cfg, generator):
+            return
     if base.startswith("lora_"):                    # peft default: A ~ U(-1/sqrt(in), 1/sqrt(in)), B = 0
         if base.endswith("_B"):
             t.zero_()
@@ -422,6 +431,8 @@ def _mlp_forward(cfg: ModelConfig, w: dict, x: torch.Tensor, aux_out: list | Non
 def layer_forward(cfg: ModelConfig, w: dict, x: torch.Tensor, inp: PackedInput, kv_sink=None, aux_out: list | None = None) -> torch.Tensor:
     """One decoder block on packed activations x:[T,H].  ``kv_sink`` = (k_cache, v_cache, slot_mapping)
     makes this a prefill step that also fills the paged KV cache (rollout engine)."""
+    if cfg.family == "hybrid":
+        raise NotImplementedError("mixer stacks are served by the rollout engine only (models/hybrid.py); training them is not implemented")
     nq, nkv, d = cfg.num_heads, cfg.num_kv_heads, cfg.head_dim
     t = x.shape[0]
     if cfg.sliding_window and inp.max_seqlen > cfg.sliding_window:
@@ -637,13 +648,25 @@ class TransformerWeights:
             return out
 
         self.embed = make(embed_param_specs(cfg))
-        self.layers = [make(layer_param_specs(cfg, i)) for i in range(cfg.num_layers)]
+        own = [self._owner(i) for i in range(cfg.num_layers)]
+        made = {i: make(layer_param_specs(cfg, i)) for i in range(cfg.num_layers) if own[i] == i}
+        self.layers = [made[j] for j in own]
         self.head = make(head_param_specs(cfg))
+
+    def _owner(self, i: int) -> int:
+        """Layer whose weights layer ``i`` uses (itself, except in stacks that reuse layers)."""
+        if self.cfg.family != "hybrid":
+            return i
+        from .hybrid import owner
+
+        return owner(self.cfg, i)
 
     def named_tensors(self):
         for n, t in self.embed.items():
             yield n, t
         for i, l in enumerate(self.layers):
+            if self._owner(i) != i:
+                continue
             for n, t in l.items():
                 yield f"layers.{i}.{n}", t
         for n, t in self.head.items():
@@ -840,6 +863,10 @@ def _export_mlp(cfg: ModelConfig, sd: dict, out: dict, i: int, p: str, fused_gu:
 
 
 def export_hf_state_dict(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict[str, torch.Tensor]:
+    if cfg.family == "hybrid":
+        from .hybrid import ludesun_export
+
+        return ludesun_export(cfg, sd)
     if cfg.family == "gpt2":
         out = {"transformer.wte.weight": sd["embed"], "transformer.wpe.weight": sd["pos_embed"], "transformer.ln_f.weight": sd["norm_w"],
                "transformer.ln_f.bias": sd["norm_b"], "lm_head.weight": sd["embed"]}

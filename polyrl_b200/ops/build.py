@@ -1,7 +1,7 @@
-"""In-tree build of the sm_100a extension ``polyrl_b200/_C.so``.
+"""In-tree build of the sm_100a extension modules ``polyrl_b200/_serve.so`` and ``polyrl_b200/_C.so``.
 
 Kernel ``.cu`` files are torch-free and compiled directly with ``nvcc -gencode arch=compute_100a,
-code=sm_100a -lineinfo``; only ``bindings.cpp`` sees torch headers.  The resulting ``.so`` lives in the
+code=sm_100a -lineinfo``; only the ``bindings*.cpp`` files see torch headers.  The resulting ``.so`` files live in the
 package directory (git-ignored, but shipped to the GPU box by ``gpurun``), never in a JIT cache.
 
 Usage:  python -m polyrl_b200.ops.build [--force] [--verbose]
@@ -19,27 +19,19 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent.parent
 CSRC = PKG / "csrc"
 BUILD = CSRC / "build"
-OUT = PKG / "_C.so"
 
-CU_SOURCES = [
-    "gemm_tcgen05.cu",
-    "gemm2.cu",
-    "skinny_gemm.cu",
-    "decode_gemm.cu",
-    "vmm.cu",
-    "linear_ce.cu",
-    "ag_gemm.cu",
-    "elementwise.cu",
-    "optim.cu",
-    "decode_attn.cu",
-    "attn_fwd.cu",
-    "attn_bwd.cu",
-    "sampling.cu",
-    "p2p.cu",
-    "nvls.cu",
-]
-HEADERS = ["common.cuh", "gemm_sm100.cuh", "gemm2_sm100.cuh"]
-HOST_HEADERS = ["kv_manager.hpp", "scheduler.hpp"]          # included by bindings.cpp only
+# One shared object per module.  ``_serve`` holds what a rollout engine of a mixer stack needs (scheduler, dense GEMMs, packed
+# attention, sampling, sequence mixers); ``_C`` the rest (training, decode kernels of the llama family, multi-GPU).  A kernel
+# object may be linked into both.
+MODULES: dict[str, dict] = {
+    "_serve": {"bindings": "bindings_serve.cpp",
+               "cu": ["gemm_tcgen05.cu", "gemm2.cu", "attn_fwd.cu", "sampling.cu", "mix_elem.cu", "mix_scan.cu", "mix_chunk.cu", "mix_latent.cu"]},
+    "_C": {"bindings": "bindings.cpp",
+           "cu": ["gemm_tcgen05.cu", "gemm2.cu", "skinny_gemm.cu", "decode_gemm.cu", "vmm.cu", "linear_ce.cu", "ag_gemm.cu", "elementwise.cu",
+                  "optim.cu", "decode_attn.cu", "attn_bwd.cu", "attn_fwd.cu", "p2p.cu", "nvls.cu"]},
+}
+HEADERS = ["common.cuh", "gemm_sm100.cuh", "gemm2_sm100.cuh", "mixers.cuh", "mix_params.hpp"]
+HOST_HEADERS = ["kv_manager.hpp", "scheduler.hpp", "bindings_common.hpp", "mix_params.hpp"]          # included by the bindings only
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-lineinfo", "-O3", "-std=c++17",
@@ -75,60 +67,81 @@ def _run(cmd: list[str], verbose: bool) -> None:
         print(r.stdout + r.stderr)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def module_path(module: str) -> Path:
+    return PKG / f"{module}.so"
+
+
+def build(force: bool = False, verbose: bool = False, modules: tuple[str, ...] = ("_serve", "_C")) -> Path:
+    """Compile what is out of date and link the requested modules; returns the path of the last one."""
     import torch  # noqa: F401  (headers + libs)
     from torch.utils import cpp_extension as ce
 
     BUILD.mkdir(parents=True, exist_ok=True)
     hdrs = [CSRC / h for h in HEADERS]
     jobs: list[list[str]] = []
-    objs: list[Path] = []
-    for name in CU_SOURCES:
-        src = CSRC / name
-        obj = BUILD / (src.stem + ".o")
-        objs.append(obj)
-        if force or _newer(src, obj, hdrs):
-            jobs.append([_nvcc(), *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
-    bsrc = CSRC / "bindings.cpp"
-    bobj = BUILD / "bindings.o"
-    objs.append(bobj)
-    if force or _newer(bsrc, bobj, [CSRC / h for h in HOST_HEADERS]):
-        inc = []
-        for p in ce.include_paths("cuda") if "device_type" in ce.include_paths.__code__.co_varnames else ce.include_paths(True):
-            inc += ["-isystem", p]
-        inc += ["-isystem", sysconfig.get_paths()["include"]]
-        jobs.append([
-            "g++", "-O2", "-std=c++17", "-fPIC", "-DTORCH_EXTENSION_NAME=_C", "-DTORCH_API_INCLUDE_EXTENSION_H",
-            f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}", *inc, "-c", str(bsrc), "-o", str(bobj),
-        ])
+    objs: dict[str, list[Path]] = {}
+    stale: dict[str, bool] = {}
+    queued: set[Path] = set()
+    for mod in modules:
+        objs[mod], stale[mod] = [], force or not module_path(mod).exists()
+        for name in MODULES[mod]["cu"]:
+            src = CSRC / name
+            obj = BUILD / (src.stem + ".o")
+            objs[mod].append(obj)
+            if obj in queued:
+                stale[mod] = True
+            elif force or _newer(src, obj, hdrs):
+                jobs.append([_nvcc(), *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
+                queued.add(obj)
+                stale[mod] = True
+        bsrc = CSRC / MODULES[mod]["bindings"]
+        bobj = BUILD / (bsrc.stem + ".o")
+        objs[mod].append(bobj)
+        if force or _newer(bsrc, bobj, [CSRC / h for h in HOST_HEADERS]):
+            inc = []
+            for p in ce.include_paths("cuda") if "device_type" in ce.include_paths.__code__.co_varnames else ce.include_paths(True):
+                inc += ["-isystem", p]
+            inc += ["-isystem", sysconfig.get_paths()["include"]]
+            jobs.insert(0, [
+                "g++", "-O2", "-std=c++17", "-fPIC", f"-DTORCH_EXTENSION_NAME={mod}", "-DTORCH_API_INCLUDE_EXTENSION_H",
+                f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}", *inc, "-c", str(bsrc), "-o", str(bobj),
+            ])
+            stale[mod] = True
+        so = module_path(mod)
+        stale[mod] = stale[mod] or any(o.exists() and so.exists() and o.stat().st_mtime > so.stat().st_mtime for o in objs[mod])
     import time
 
     t0 = time.time()
     if jobs:
-        with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
+        with cf.ThreadPoolExecutor(max_workers=min(max(2, os.cpu_count() or 2), 16, len(jobs))) as ex:
             list(ex.map(lambda c: _run(c, verbose), jobs))
     global LAST_BUILD
-    LAST_BUILD = {"build_mode": "clean" if len(jobs) == len(objs) else ("incremental" if jobs else "up-to-date"),
-                  "objects_compiled": len(jobs), "objects_total": len(objs), "compile_s": round(time.time() - t0, 1),
+    total = len({o for v in objs.values() for o in v})
+    LAST_BUILD = {"build_mode": "clean" if len(jobs) == total else ("incremental" if jobs else "up-to-date"), "modules": list(modules),
+                  "objects_compiled": len(jobs), "objects_total": total, "compile_s": round(time.time() - t0, 1),
                   "arch": "compute_100a/sm_100a", "nvcc_flags": NVCC_FLAGS}
-    if jobs or force or not OUT.exists():
+    for mod in modules:
+        if not stale[mod]:
+            continue
+        out = module_path(mod)
         lib_dirs = ce.library_paths("cuda") if "device_type" in ce.library_paths.__code__.co_varnames else ce.library_paths(True)
-        tmp_out = OUT.with_suffix(".so.tmp")           # link next to the target, then rename: readers never see a half-written .so
-        link = ["g++", "-shared", "-o", str(tmp_out), *map(str, objs)]
+        tmp_out = out.with_suffix(f".so.tmp{os.getpid()}")     # link next to the target, then rename: readers never see a half-written .so
+        link = ["g++", "-shared", "-o", str(tmp_out), *map(str, objs[mod])]
         for d in lib_dirs:
             link += [f"-L{d}", f"-Wl,-rpath,{d}"]
         link += ["-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-ltorch_python", "-lcudart"]
         _run(link, verbose)
-        tmp_out.replace(OUT)
-    return OUT
+        tmp_out.replace(out)
+    return module_path(modules[-1])
 
 
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true")
+    ap.add_argument("--modules", default="_serve,_C", help="comma-separated subset of the modules to build")
     a = ap.parse_args()
-    print(build(a.force, a.verbose))
+    print(build(a.force, a.verbose, tuple(a.modules.split(","))))
     import json
 
     print(json.dumps(LAST_BUILD))

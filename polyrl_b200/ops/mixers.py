@@ -1,0 +1,303 @@
+"""Sequence-mixer ops over packed spans: sm_100a kernels on CUDA tensors (bf16 or fp32), plain PyTorch on CPU tensors.
+
+A ``SpanBatch`` describes one engine step: span ``s`` is the tokens ``[cu[s], cu[s + 1])`` of one sequence whose first
+``start[s]`` tokens were processed earlier.  A decoded token is a span of one.  Recurrent state lives in pools indexed by
+``slot``, keys in a paged pool indexed by ``kv_slot`` / ``table``; a span with ``start == 0`` begins from the zero state.
+Spans are ordered: the ``n_long`` spans of several tokens first, then the single tokens.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+import torch.nn.functional as F
+
+PAGE = 16
+
+
+@dataclass
+class SpanBatch:
+    cu: torch.Tensor                    # [n + 1] int32
+    start: torch.Tensor                 # [n] int32
+    slot: torch.Tensor                  # [n] int64 state slot
+    pos: torch.Tensor                   # [T] int64
+    kv_slot: torch.Tensor               # [T] int64 flat cache row (page * PAGE + offset)
+    kv_len: torch.Tensor                # [T] int32 keys a token sees, its own included (0: idle row)
+    table: torch.Tensor                 # [n, width] int32 page numbers
+    seq_of: torch.Tensor | None = None  # [T] int32 span of a token; None: every span is one token
+    n_long: int = 0
+    t_long: int = 0
+    max_long: int = 0                   # longest span
+    max_len: int = 0                    # bound on kv_len
+    # keys of the long spans: (flat cache rows [Tk] int64, cu_k [n_long + 1] int32); None: no span has earlier tokens
+    gather: tuple | None = None
+
+    @property
+    def spans(self) -> int:
+        return self.start.numel()
+
+    @property
+    def tokens(self) -> int:
+        return self.pos.numel()
+
+
+def _C():
+    from . import ext
+
+    return ext()
+
+
+_COUNTERS: dict = {}
+_RETIRED: list = []     # outgrown counters stay alive: captured graphs hold their address
+
+
+def _counter(device: torch.device, n: int) -> torch.Tensor:
+    """Zeroed arrival counters of the recurrence kernels (each launch leaves them zero again)."""
+    key = (device.type, device.index)
+    if key not in _COUNTERS or _COUNTERS[key].numel() < n:
+        _RETIRED.append(_COUNTERS.get(key))
+        _COUNTERS[key] = torch.zeros(max(n, 1 << 17), device=device, dtype=torch.int32)
+    return _COUNTERS[key]
+
+
+# --------------------------------------------------------------------------------------------
+# rows
+# --------------------------------------------------------------------------------------------
+def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def embed(ids: torch.Tensor, w: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """(fp32 residual stream, the same in the activation dtype — one tensor when that is fp32)."""
+    if w.is_cuda:
+        return tuple(_C().mix_embed(ids, w))
+    x = F.embedding(ids, w).float()
+    return x, (x if w.dtype == torch.float32 else x.to(w.dtype))
+
+
+def norm_add_(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, eps: float, w_next: torch.Tensor | None = None) -> torch.Tensor:
+    """x += rms(y) * w (fp32, in place); returns x in y's dtype, or rms(x) * w_next in y's dtype."""
+    if y.is_cuda:
+        return _C().mix_norm_add_(y, x, w, eps, w_next)
+    x.add_(_rms(y.float(), eps) * w)
+    if w_next is not None:
+        return (_rms(x, eps) * w_next).to(y.dtype)
+    return x if y.dtype == torch.float32 else x.to(y.dtype)
+
+
+def rms(x: torch.Tensor, w: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """rms(x) * w of fp32 rows in ``dtype``."""
+    if x.is_cuda:
+        return _C().mix_rms(x.contiguous(), w, eps, dtype == torch.bfloat16)
+    return (_rms(x, eps) * w).to(dtype)
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate_first: bool) -> torch.Tensor:
+    """Group RMS norm with a gate: rms(y * silu(z)) * w (``gate_first``) or rms(y) * w * sigmoid(z)."""
+    if y.is_cuda:
+        return _C().mix_gated_norm(y, z, w, groups, eps, gate_first)
+    yf, zf = y.float(), z.float()
+    if gate_first:
+        yf = yf * F.silu(zf)
+    n = _rms(yf.reshape(y.shape[0], groups, -1), eps).reshape(y.shape) * w
+    return (n if gate_first else n * torch.sigmoid(zf)).to(y.dtype)
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x @ w.T with the fp32 accumulator as the result (gates and step sizes of a recurrence)."""
+    if x.is_cuda and x.dtype == torch.bfloat16:
+        return torch.mm(x, w.t(), out_dtype=torch.float32)
+    return F.linear(x.float(), w.float())
+
+
+def linear_gelu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(x @ w.T); fused into the GEMM epilogue for bf16 rows."""
+    if x.is_cuda:
+        if x.dtype == torch.bfloat16 and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0:
+            return _C().gemm_gelu(x, w)
+        y = F.linear(x, w)
+        _C().mix_gelu_(y)
+        return y
+    return F.gelu(F.linear(x, w.to(x.dtype)), approximate="tanh")
+
+
+# --------------------------------------------------------------------------------------------
+# causal convolution with carried taps
+# --------------------------------------------------------------------------------------------
+def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, b: SpanBatch) -> torch.Tensor:
+    """silu(causal conv) per channel; w [taps, ch] (last row: the current token), state [slots, taps - 1, ch]."""
+    if x.is_cuda:
+        return _C().mix_conv(x, w, bias, state, b.cu, b.start, b.slot, b.seq_of)
+    taps = w.shape[0]
+    out = torch.empty_like(x)
+    cu = b.cu.tolist()
+    for s in range(b.spans):
+        lo, hi = cu[s], cu[s + 1]
+        old = state[b.slot[s]] if int(b.start[s]) else torch.zeros_like(state[0])
+        full = torch.cat([old, x[lo:hi]]).float()
+        y = bias + sum(w[j] * full[j:j + hi - lo] for j in range(taps))
+        out[lo:hi] = F.silu(y).to(x.dtype)
+        state[b.slot[s]] = full[full.shape[0] - (taps - 1):].to(state.dtype)
+    return out
+
+
+# --------------------------------------------------------------------------------------------
+# gated linear recurrences
+# --------------------------------------------------------------------------------------------
+SSD, MLSTM = 0, 1
+
+
+@dataclass
+class Gates:
+    """Raw gate projections (fp32 [T, H]) and per-head constants of a recurrence."""
+    g0: torch.Tensor
+    g1: torch.Tensor | None = None
+    b0: torch.Tensor | None = None
+    b1: torch.Tensor | None = None
+    a_log: torch.Tensor | None = None
+    d_skip: torch.Tensor | None = None
+    cap: float = 1.0
+
+
+CHUNK_MIN = 8           # spans shorter than this go through the token-by-token kernel
+
+
+def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Gates, qscale: float, cache: dict, b: SpanBatch) -> torch.Tensor:
+    """S_t = keep_t S_(t-1) + add_t k_t v_t^T,  y_t = S_t^T (qscale q_t), over the spans of ``b``.
+
+    ``SSD``: add = softplus(g0 + b0), keep = exp(-exp(a_log) add), y += d_skip v.  ``MLSTM``: capped log gates with a running
+    maximum and a normaliser.  q / k [T, groups * N] (consecutive heads share a group), v [T, H * V], cache["S"] [slots, H, N, V]
+    (+ "n" [slots, H, N], "m" [slots, H])."""
+    if not v.is_cuda:
+        return _scan_cpu(mode, q, k, v, gates, qscale, cache, b)
+    S, H, N = cache["S"], cache["S"].shape[1], cache["S"].shape[2]
+    ctr = _counter(v.device, b.spans * H)
+    out = torch.empty(v.shape, device=v.device, dtype=v.dtype)
+
+    def run(lo: int, hi: int, chunk: bool) -> None:
+        _C().mix_scan_(mode, q, k, v, gates.g0, gates.g1, gates.b0, gates.b1, gates.a_log, gates.d_skip, qscale, gates.cap, S, cache.get("n"),
+                       cache.get("m"), b.cu[lo:hi + 1], b.start[lo:hi], b.slot[lo:hi], ctr, chunk, out)
+
+    chunk = v.dtype == torch.bfloat16 and b.max_long >= CHUNK_MIN and _C().mix_chunk_supported(N)
+    if chunk and b.n_long:
+        run(0, b.n_long, True)
+        if b.n_long < b.spans:
+            run(b.n_long, b.spans, False)
+    else:
+        run(0, b.spans, False)
+    return out
+
+
+def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
+    S_pool = cache["S"]
+    H, N, V = S_pool.shape[1:]
+    rep = H // (q.shape[1] // N)
+    out = torch.empty_like(v)
+    cu = b.cu.tolist()
+    for s in range(b.spans):
+        sl, fresh = int(b.slot[s]), int(b.start[s]) == 0
+        S = torch.zeros_like(S_pool[0]) if fresh else S_pool[sl].clone()
+        if mode == MLSTM:
+            n = torch.zeros_like(cache["n"][0]) if fresh else cache["n"][sl].clone()
+            m = torch.zeros_like(cache["m"][0]) if fresh else cache["m"][sl].clone()
+        for t in range(cu[s], cu[s + 1]):
+            qt = q[t].float().reshape(-1, N).repeat_interleave(rep, 0) * qscale
+            kt = k[t].float().reshape(-1, N).repeat_interleave(rep, 0)
+            vt = v[t].float().reshape(H, V)
+            if mode == SSD:
+                add = F.softplus(g.g0[t] + g.b0, threshold=1e9)
+                keep = torch.exp(-torch.exp(g.a_log) * add)
+            else:
+                gi = g.cap * torch.tanh((g.g0[t] + g.b0) / g.cap)
+                gf = F.logsigmoid(g.cap * torch.tanh((g.g1[t] + g.b1) / g.cap))
+                m2 = torch.maximum(gf + m, gi)
+                keep, add, m = torch.exp(gf + m - m2), torch.exp(gi - m2), m2
+                n = keep[:, None] * n + add[:, None] * kt
+            S = keep[:, None, None] * S + (add[:, None] * kt)[:, :, None] * vt[:, None, :]
+            y = torch.einsum("hnv,hn->hv", S, qt)
+            if mode == SSD:
+                y = y + g.d_skip[:, None] * vt
+            else:
+                y = y / (torch.maximum((n * qt).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None]
+            out[t] = y.reshape(-1).to(v.dtype)
+        S_pool[sl] = S
+        if mode == MLSTM:
+            cache["n"][sl], cache["m"][sl] = n, m
+    return out
+
+
+# --------------------------------------------------------------------------------------------
+# latent attention
+# --------------------------------------------------------------------------------------------
+def rope_frequencies(dims: int, base: float, device) -> torch.Tensor:
+    """base^(-2 i / dims), i < dims / 2, double precision (angles are reduced before the fp32 sine / cosine)."""
+    return torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=device)
+
+
+def _rotate(x: torch.Tensor, freq: torch.Tensor, pos: torch.Tensor) -> torch.Tensor:
+    a = torch.outer(pos.double(), freq)
+    c, s = a.cos().float(), a.sin().float()
+    if x.dim() == 3:
+        c, s = c[:, None], s[:, None]
+    u, v = x.float().chunk(2, -1)
+    return torch.cat([u * c - v * s, v * c + u * s], -1).to(x.dtype)
+
+
+def latent_prep(a: torch.Tensor, wq: torch.Tensor, wkv: torch.Tensor, freq: torch.Tensor, pool: torch.Tensor, b: SpanBatch, eps: float,
+                want_entry: bool) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """Rows [query latent | key-value latent | shared rotary key] -> normed query latent; the cache row [normed latent | rotated key] of
+    every token is written to ``pool`` and also returned when asked for."""
+    if a.is_cuda:
+        cq, en = _C().mix_latent_prep(a, wq, wkv, freq, b.pos, b.kv_slot, pool, eps, want_entry)
+        return cq, en if want_entry else None
+    qr, r, rd = wq.numel(), wkv.numel(), 2 * freq.numel()
+    cq = (_rms(a[:, :qr].float(), eps) * wq).to(a.dtype)
+    c = (_rms(a[:, qr:qr + r].float(), eps) * wkv).to(a.dtype)
+    en = torch.cat([c, _rotate(a[:, qr + r:qr + r + rd], freq, b.pos)], -1)
+    pool.view(-1, r + rd)[b.kv_slot] = en
+    return cq, en
+
+
+def rope_(q: torch.Tensor, d: int, freq: torch.Tensor, pos: torch.Tensor) -> None:
+    """Rotate columns [d, d + 2 * freq.numel()) of every head of q [T, H, *] in place."""
+    if q.is_cuda:
+        _C().mix_rope_(q, d, freq, pos)
+        return
+    rd = 2 * freq.numel()
+    q[..., d:d + rd] = _rotate(q[..., d:d + rd], freq, pos)
+
+
+def _splits(rows: int, heads: int, max_len: int) -> int:
+    ctas = rows * ((heads + 15) // 16)
+    return max(1, min((2 * 148 + ctas - 1) // ctas, max(1, max_len // 256), 32))
+
+
+def latent_attention(q_lat: torch.Tensor, q: torch.Tensor, d: int, pool: torch.Tensor, table: torch.Tensor, seq_of: torch.Tensor | None,
+                     kv_len: torch.Tensor, sink: torch.Tensor | None, scale: float, max_len: int) -> torch.Tensor:
+    """Absorbed form over the paged pool: q_lat [H, R, r], q [R, H, *] (rotated part at column d) -> softmax-weighted latents [H, R, r];
+    ``sink`` [H] adds exp(sink) to the denominator."""
+    h, rows, r = q_lat.shape
+    if q.is_cuda:
+        tc = q.dtype == torch.bfloat16 and _C().mix_latent_tc_ok(r, pool.shape[-1] - r)
+        return _C().mix_latent(q_lat, q, d, pool, table, seq_of, kv_len, sink, scale, _splits(rows, h, max_len), tc)
+    rd = pool.shape[-1] - r
+    out = torch.zeros_like(q_lat)
+    for i in range(rows):
+        n = int(kv_len[i])
+        if n == 0:
+            continue
+        pages = table[int(seq_of[i]) if seq_of is not None else i, : (n + PAGE - 1) // PAGE].long()
+        kv = pool.view(-1, PAGE, r + rd)[pages].reshape(-1, r + rd)[:n].float()
+        s = (q_lat[:, i].float() @ kv[:, :r].T + q[i, :, d:d + rd].float() @ kv[:, r:].T) * scale
+        if sink is not None:
+            s = torch.cat([s, sink[:, None]], -1)
+        p = torch.softmax(s, -1)[:, :n]
+        out[:, i] = (p @ kv[:, :r]).to(out.dtype)
+    return out
+
+
+def sink_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.Tensor, cu_k: torch.Tensor, scale: float,
+                          sink: torch.Tensor | None) -> torch.Tensor:
+    """Causal (bottom-right aligned) attention of packed spans on expanded keys, with a sink: the tcgen05 kernel, query / key width
+    128 or 192, value width 128, bf16."""
+    return _C().attn_fwd(q, k, v, cu_q, cu_k, scale, True, False, None, sink)[0]

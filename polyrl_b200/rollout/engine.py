@@ -75,10 +75,12 @@ class Request:
     mrope_delta: int = 0
     image_embeds: object = None            # tower output, computed at the first prefill chunk and dropped after the last
     h: int = -1                            # handle inside the native scheduler (csrc/scheduler.hpp), -1 = not registered
+    state_slot: int = 0                    # recurrent-state slot (mixer stacks), 0 = none
+    fed: bool = False                      # tokens are supplied step by step (RolloutEngine.extend), nothing is sampled
 
     @property
     def decoding(self) -> bool:
-        return self.prefilled >= len(self.prompt_ids) and self.finish_reason is None
+        return self.prefilled >= len(self.prompt_ids) and self.finish_reason is None and not self.fed
 
     @property
     def finished(self) -> bool:
@@ -87,6 +89,23 @@ class Request:
     @property
     def num_tokens(self) -> int:
         return len(self.prompt_ids) + len(self.output_ids)
+
+
+class StateSlots:
+    """Free list of recurrent-state slots (mixer stacks, models/hybrid.py).  Slot 0 belongs to idle batch rows.  A slot needs no clearing
+    when it is handed on: the first span of a sequence starts from the zero state."""
+
+    def __init__(self, num_slots: int):
+        self.free = deque(range(1, num_slots))
+
+    def alloc(self) -> int:
+        if not self.free:
+            raise MemoryError("no free state slot")
+        return self.free.popleft()
+
+    def release(self, slot: int) -> None:
+        if slot > 0:
+            self.free.append(slot)
 
 
 class BlockAllocator:
@@ -283,6 +302,11 @@ class RolloutEngine:
         self.weight_dtype = weight_dtype               # fp8: projections re-quantised (e4m3, per-row scale) at every sync
         self._fp8_cache: list[dict] = []
         self.tp = tp                               # rollout.tp.TPContext for tensor-parallel engines
+        self.hybrid = cfg.family == "hybrid"
+        if self.hybrid and (tp is not None or weight_dtype == "fp8" or kv_vmm):
+            raise NotImplementedError("mixer stacks: tensor parallelism, fp8 weights and the VMM-backed cache are not implemented")
+        self.kv_vmm = self.kv_vmm and not self.hybrid
+        self.state: StateSlots | None = None           # recurrent-state slots, created with the cache pools
         self.full_cfg = cfg
         cfg = tp.local_cfg() if tp is not None else cfg   # per-rank view: local heads / kv heads / intermediate
         self.cfg = cfg
@@ -331,6 +355,13 @@ class RolloutEngine:
             layer_w = [self.tp.shard_layer(w) for w in layer_w]
         if self.weight_dtype == "fp8":
             layer_w = self._quantize_layers(layer_w)
+        if self.hybrid:                 # run-time form; what is derived is overwritten in place on later syncs
+            from ..models import hybrid
+
+            layer_w = hybrid.prepare(self.cfg, layer_w, self.dtype, self.layer_w)
+            head_w = hybrid.prepare_head(head_w, self.dtype, self.head_w)
+            if embed_w["embed"].dtype != self.dtype:
+                embed_w = {"embed": embed_w["embed"].to(self.dtype)}
         self.embed_w, self.layer_w, self.head_w = embed_w, layer_w, head_w
         if old != self._weight_ptrs():
             self._graphs.clear()
@@ -372,6 +403,10 @@ class RolloutEngine:
 
     def kv_bytes_per_token(self) -> int:
         c = self.cfg
+        if self.hybrid:
+            from ..models import hybrid
+
+            return hybrid.cache_bytes(c, self.dtype)[0]
         heads, width, two = c.kv_cache_layout()          # MLA: one shared latent entry per token, no separate value pool
         return (2 if two else 1) * c.num_layers * heads * width * torch.empty(0, dtype=self.dtype).element_size()
 
@@ -385,12 +420,26 @@ class RolloutEngine:
             tokens = self._kv_tokens_req
         elif self.is_cuda:
             free, total = torch.cuda.mem_get_info(self.device)
-            tokens = int(free * self.gpu_memory_utilization) // self.kv_bytes_per_token()
+            budget = int(free * self.gpu_memory_utilization)
+            if self.hybrid:
+                from ..models import hybrid
+
+                budget -= (self.max_num_seqs + 1) * hybrid.cache_bytes(self.cfg, self.dtype)[1]
+            tokens = max(budget, 0) // max(1, self.kv_bytes_per_token())
         else:
             tokens = self.max_num_seqs * self.max_model_len
         tokens = min(tokens, self.max_num_seqs * self.max_blocks_per_seq * PAGE + PAGE)
         num_blocks = max(2, tokens // PAGE)
         c = self.cfg
+        if self.hybrid:
+            from ..models import hybrid
+
+            self.state = StateSlots(self.max_num_seqs + 1)
+            self.k_cache = [hybrid.make_cache(c, i, num_blocks, self.max_num_seqs + 1, self.device, self.dtype) for i in range(c.num_layers)]
+            self.alloc, self.prefix_cache = make_kv_manager(num_blocks, False)
+            self._make_scheduler()
+            self._graphs.clear()
+            return
         kv_heads, kv_width, two_pools = c.kv_cache_layout()
         shape = (num_blocks, kv_heads, PAGE, kv_width)
         if not two_pools:
@@ -444,7 +493,7 @@ class RolloutEngine:
         if "kv_cache" in tags:
             if self.running or self.waiting:
                 raise RuntimeError("cannot release the KV cache with requests in flight")
-            self.k_cache, self.v_cache, self.alloc, self.prefix_cache, self.sched = [], [], None, None, None
+            self.k_cache, self.v_cache, self.alloc, self.prefix_cache, self.sched, self.state = [], [], None, None, None, None
             if self.kv_vmm and self._vmm is not None:
                 torch.cuda.synchronize(self.device)        # nothing may still read the pool
                 self._vmm.unmap()                          # graphs stay valid: same addresses after the next resume
@@ -472,6 +521,8 @@ class RolloutEngine:
         self.st_positions = torch.zeros(s, dtype=torch.long, device=dev)
         self.st_seq_lens = torch.zeros(s, dtype=torch.int32, device=dev)
         self.st_active = torch.zeros(s, dtype=torch.long, device=dev)
+        self.st_state = torch.zeros(s, dtype=torch.long, device=dev)           # recurrent-state slot of a batch slot
+        self.arange32 = torch.arange(s + 1, dtype=torch.int32, device=dev)
         self.st_block_table = torch.zeros(s, self.max_blocks_per_seq + 2, dtype=torch.int32, device=dev)   # + overshoot slack -> scratch page 0
         self.st_temp = torch.ones(s, dtype=torch.float32, device=dev)
         self.st_seeds = torch.zeros(s, dtype=torch.long, device=dev)
@@ -547,8 +598,13 @@ class RolloutEngine:
 
     def _admit(self) -> list[Request]:
         """Pop waiting requests that fit (slots, KV pages reserved up front, prefill token budget)."""
-        if self.sched is not None:
-            return self._admit_native()
+        admitted = self._admit_native() if self.sched is not None else self._admit_python()
+        if self.state is not None:                # as many state slots as batch slots: an admitted request always gets one
+            for r in admitted:
+                r.state_slot = self.state.alloc()
+        return admitted
+
+    def _admit_python(self) -> list[Request]:
         admitted, tokens = [], 0
         shared: dict = {}
         while self.waiting and self.free_slots:
@@ -622,6 +678,9 @@ class RolloutEngine:
             self.st_seq_lens[r.slot] = 0
             self.free_slots.append(r.slot)
             r.slot = -1
+        if self.state is not None:
+            self.state.release(r.state_slot)
+            r.state_slot = 0
         if r.h >= 0 and self.sched is not None:
             to_cache = self.prefix_cache is not None and reason != "abort" and r.mm is None
             self.sched.finish(r.h, (r.prompt_ids + r.output_ids) if to_cache else [], to_cache)
@@ -667,7 +726,83 @@ class RolloutEngine:
             budget -= e - c
         if not donors:
             return
+        if self.hybrid:                         # single tokens last (ops/mixers.py)
+            order = sorted(range(len(donors)), key=lambda i: spans[i][1] - spans[i][0] == 1)
+            donors, spans = [donors[i] for i in order], [spans[i] for i in order]
         d_index = {id(r): i for i, r in enumerate(donors)}
+        x, cu = self._forward_spans(donors, spans)
+        for r, (_, e) in zip(donors, spans):
+            r.prefilled = e
+        self.stats["prefill_tokens"] += sum(e - c for c, e in spans)
+        done_ids = {id(r) for r in donors if r.prefilled >= len(r.prompt_ids)}
+        reqs = [r for r in reqs if not r.finished and (id(r) in done_ids or (r.donor is not None and id(r.donor) in done_ids))]
+        self._prefill_queue = [r for r in self._prefill_queue if not r.finished and not any(r is q for q in reqs)]
+        if not reqs:
+            return
+        logits_d = self._span_logits(x, (cu[1:] - 1).long().to(dev))
+        src_blk, dst_blk = [], []
+        for r in reqs:
+            if r.donor is not None:
+                r.prefilled = len(r.prompt_ids)
+            if r.donor is not None and len(r.prompt_ids) % PAGE != 0:
+                fp = len(r.prompt_ids) // PAGE
+                src_blk.append(r.donor.blocks[fp])
+                dst_blk.append(r.blocks[fp])
+        if dst_blk:
+            s_t = torch.tensor(src_blk, dtype=torch.long, device=dev)
+            d_t = torch.tensor(dst_blk, dtype=torch.long, device=dev)
+            for i in range(len(self.layer_w) if not self.hybrid else 0):
+                self.k_cache[i].index_copy_(0, d_t, self.k_cache[i].index_select(0, s_t))
+                self.v_cache[i].index_copy_(0, d_t, self.v_cache[i].index_select(0, s_t))
+        if self.hybrid and any(r.donor is not None for r in reqs):
+            # followers continue from the donor's prompt: its partial last page and its recurrent state (still the prompt's — the donor
+            # has not decoded yet)
+            from ..models import hybrid
+
+            pairs = [(r.donor.state_slot, r.state_slot) for r in reqs if r.donor is not None]
+            idx = [torch.tensor(v, dtype=torch.long, device=dev) for v in (src_blk, dst_blk, [a for a, _ in pairs], [b for _, b in pairs])]
+            for c in self.k_cache:
+                hybrid.copy_cache(c, *idx)
+        row = torch.tensor([d_index[id(r.donor if r.donor is not None else r)] for r in reqs], dtype=torch.long, device=dev)
+        logits = logits_d.index_select(0, row)
+        temps = torch.tensor([r.params.temperature for r in reqs], dtype=torch.float32, device=dev)
+        seeds = torch.tensor([self._seed_for(r, 0) for r in reqs], dtype=torch.long, device=dev)
+        p0 = reqs[0].params
+        tok, lp = ops.sample_tokens(logits, temps, seeds, greedy=False, top_k=p0.top_k, top_p=p0.top_p)
+        tok_c, lp_c = tok.tolist(), lp.tolist()
+        for r in reqs:
+            r.donor = None            # release the reference; pages stay shared through the allocator's ref-counts
+        live, rows = [], []
+        for r, t, l in zip(reqs, tok_c, lp_c):
+            self._append_token(r, t, l)
+            if r.finished:
+                continue
+            n = r.num_tokens            # tokens so far; the new token sits at position n-1 (+ the M-RoPE offset of image prompts)
+            live.append((r.slot, t, n - 1 + r.mrope_delta, n, 1, r.params.temperature, self._seed_for(r, 1), r.state_slot))
+            rows.append(r)
+        if live:
+            cols = list(zip(*live))
+            sl = torch.tensor(cols[0], dtype=torch.long, device=dev)
+            self.st_input_ids[sl] = torch.tensor(cols[1], dtype=torch.long, device=dev)
+            self.st_positions[sl] = torch.tensor(cols[2], dtype=torch.long, device=dev)
+            self.st_seq_lens[sl] = torch.tensor(cols[3], dtype=torch.int32, device=dev)
+            self.st_active[sl] = torch.tensor(cols[4], dtype=torch.long, device=dev)
+            self.st_temp[sl] = torch.tensor(cols[5], dtype=torch.float32, device=dev)
+            self.st_seeds[sl] = torch.tensor(cols[6], dtype=torch.long, device=dev)
+            self.st_state[sl] = torch.tensor(cols[7], dtype=torch.long, device=dev)
+            width = self.st_block_table.shape[1]
+            if self.sched is not None and all(r.h >= 0 for r in rows):
+                table = self.sched.block_rows([r.h for r in rows], width)
+            else:
+                table = torch.tensor([r.blocks + [0] * (width - len(r.blocks)) for r in rows], dtype=torch.int32)
+            self.st_block_table[sl] = table.to(dev)
+
+    def _forward_spans(self, donors: list[Request], spans: list[tuple[int, int]]) -> tuple[torch.Tensor, torch.Tensor]:
+        """Run the tokens [c, e) of every request as ONE packed step over the cache and state that earlier steps left.  Returns the
+        last layer's rows (in span order) and cu_seqlens on the host."""
+        if self.hybrid:
+            return self._forward_spans_hybrid(donors, spans)
+        cfg, dev = self.cfg, self.device
         ids, pos, slots, lens = [], [], [], []
         any_cached = any(c > 0 for c, _ in spans)
         g_blk, g_off, klens = [], [], []
@@ -676,8 +811,6 @@ class RolloutEngine:
             ids_t, pos_t, slots_t, lens_t, g_blk, g_off, klens_t = self.sched.prefill_arrays(
                 [(r.h, c, e) for r, (c, e) in zip(donors, spans)], any_cached)
             lens, klens = lens_t.tolist(), klens_t.tolist()
-            for r, (c, e) in zip(donors, spans):
-                r.prefilled = e
         else:
             for r, (c, e) in zip(donors, spans):
                 ids += r.prompt_ids[c:e]
@@ -688,7 +821,6 @@ class RolloutEngine:
                     g_blk += [r.blocks[t // PAGE] for t in range(e)]
                     g_off += [t % PAGE for t in range(e)]
                     klens.append(e)
-                r.prefilled = e
             ids_t, pos_t, slots_t = (torch.tensor(v, dtype=torch.long) for v in (ids, pos, slots))
             if any_cached:
                 g_blk, g_off = torch.tensor(g_blk, dtype=torch.long), torch.tensor(g_off, dtype=torch.long)
@@ -714,61 +846,64 @@ class RolloutEngine:
                 from ..models.vision import deepstack_add
 
                 x = deepstack_add(self.full_cfg, x, inp.input_ids, inp.image_embeds, i)      # Qwen3-VL DeepStack (no-op otherwise)
-        self.stats["prefill_tokens"] += int(ids_t.numel())
-        done_ids = {id(r) for r in donors if r.prefilled >= len(r.prompt_ids)}
-        reqs = [r for r in reqs if not r.finished and (id(r) in done_ids or (r.donor is not None and id(r.donor) in done_ids))]
-        self._prefill_queue = [r for r in self._prefill_queue if not r.finished and not any(r is q for q in reqs)]
-        if not reqs:
-            return
-        last = (cu[1:] - 1).long().to(dev)
-        h = tf.final_norm(cfg, self.head_w, x.index_select(0, last))
-        logits_d = self._lm_logits(h)
-        src_blk, dst_blk = [], []
-        for r in reqs:
-            if r.donor is not None:
-                r.prefilled = len(r.prompt_ids)
-            if r.donor is not None and len(r.prompt_ids) % PAGE != 0:
-                fp = len(r.prompt_ids) // PAGE
-                src_blk.append(r.donor.blocks[fp])
-                dst_blk.append(r.blocks[fp])
-        if dst_blk:
-            s_t = torch.tensor(src_blk, dtype=torch.long, device=dev)
-            d_t = torch.tensor(dst_blk, dtype=torch.long, device=dev)
-            for i in range(len(self.layer_w)):
-                self.k_cache[i].index_copy_(0, d_t, self.k_cache[i].index_select(0, s_t))
-                self.v_cache[i].index_copy_(0, d_t, self.v_cache[i].index_select(0, s_t))
-        row = torch.tensor([d_index[id(r.donor if r.donor is not None else r)] for r in reqs], dtype=torch.long, device=dev)
-        logits = logits_d.index_select(0, row)
-        temps = torch.tensor([r.params.temperature for r in reqs], dtype=torch.float32, device=dev)
-        seeds = torch.tensor([self._seed_for(r, 0) for r in reqs], dtype=torch.long, device=dev)
-        p0 = reqs[0].params
-        tok, lp = ops.sample_tokens(logits, temps, seeds, greedy=False, top_k=p0.top_k, top_p=p0.top_p)
-        tok_c, lp_c = tok.tolist(), lp.tolist()
-        for r in reqs:
-            r.donor = None            # release the reference; pages stay shared through the allocator's ref-counts
-        live, rows = [], []
-        for r, t, l in zip(reqs, tok_c, lp_c):
-            self._append_token(r, t, l)
-            if r.finished:
-                continue
-            n = r.num_tokens            # tokens so far; the new token sits at position n-1 (+ the M-RoPE offset of image prompts)
-            live.append((r.slot, t, n - 1 + r.mrope_delta, n, 1, r.params.temperature, self._seed_for(r, 1)))
-            rows.append(r)
-        if live:
-            cols = list(zip(*live))
-            sl = torch.tensor(cols[0], dtype=torch.long, device=dev)
-            self.st_input_ids[sl] = torch.tensor(cols[1], dtype=torch.long, device=dev)
-            self.st_positions[sl] = torch.tensor(cols[2], dtype=torch.long, device=dev)
-            self.st_seq_lens[sl] = torch.tensor(cols[3], dtype=torch.int32, device=dev)
-            self.st_active[sl] = torch.tensor(cols[4], dtype=torch.long, device=dev)
-            self.st_temp[sl] = torch.tensor(cols[5], dtype=torch.float32, device=dev)
-            self.st_seeds[sl] = torch.tensor(cols[6], dtype=torch.long, device=dev)
-            width = self.st_block_table.shape[1]
-            if self.sched is not None and all(r.h >= 0 for r in rows):
-                table = self.sched.block_rows([r.h for r in rows], width)
-            else:
-                table = torch.tensor([r.blocks + [0] * (width - len(r.blocks)) for r in rows], dtype=torch.int32)
-            self.st_block_table[sl] = table.to(dev)
+        return x, cu
+
+    def _forward_spans_hybrid(self, reqs: list[Request], spans: list[tuple[int, int]]) -> tuple[torch.Tensor, torch.Tensor]:
+        """``_forward_spans`` of a mixer stack: spans of several tokens come first, single tokens last (ops/mixers.py)."""
+        from ..models import hybrid
+        from ..ops.mixers import SpanBatch
+
+        dev = self.device
+        lens = [e - c for c, e in spans]
+        n_long = sum(n > 1 for n in lens)
+        if any(n <= 1 for n in lens[:n_long]):
+            raise ValueError("spans of several tokens must precede single tokens")
+        t_long = sum(lens[:n_long])
+        ids, pos, kv_slot = self._span_arrays(reqs, spans)
+        cu = torch.zeros(len(spans) + 1, dtype=torch.int32)
+        cu[1:] = torch.tensor(lens, dtype=torch.int32).cumsum(0)
+        max_len = max(e for _, e in spans)
+        width = (max_len + PAGE - 1) // PAGE
+        table = torch.tensor([(r.blocks + [0] * width)[:width] for r in reqs], dtype=torch.int32)
+        gather = None
+        if any(c > 0 for c, _ in spans[:n_long]):       # keys of the long spans, earlier tokens included
+            at = torch.arange(PAGE)
+            rows = [(torch.tensor(r.blocks[: (e + PAGE - 1) // PAGE]).unsqueeze(1) * PAGE + at).reshape(-1)[:e]
+                    for r, (_, e) in zip(reqs[:n_long], spans[:n_long])]
+            cu_k = torch.zeros(n_long + 1, dtype=torch.int32)
+            cu_k[1:] = torch.tensor([e for _, e in spans[:n_long]], dtype=torch.int32).cumsum(0)
+            gather = (torch.cat(rows).to(dev), cu_k.to(dev))
+        seq_of = torch.repeat_interleave(torch.arange(len(spans), dtype=torch.int32), torch.tensor(lens))
+        pos = pos.to(dev)
+        b = SpanBatch(cu=cu.to(dev), start=torch.tensor([c for c, _ in spans], dtype=torch.int32, device=dev),
+                      slot=torch.tensor([r.state_slot for r in reqs], dtype=torch.long, device=dev), pos=pos, kv_slot=kv_slot.to(dev),
+                      kv_len=(pos + 1).to(torch.int32), table=table.to(dev), seq_of=seq_of.to(dev) if n_long else None, n_long=n_long, t_long=t_long,
+                      max_long=max(lens) if n_long else 0, max_len=max_len, gather=gather)
+        x, h = hybrid.embed_forward(self.cfg, self.embed_w, ids.to(dev))
+        for i, w in enumerate(self.layer_w):
+            h = hybrid.layer_step(self.cfg, i, w, x, h, self.k_cache[i], b)
+        return x, cu
+
+    def _span_arrays(self, reqs: list[Request], spans: list[tuple[int, int]]) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+        """(token ids, positions, flat cache rows) of the packed tokens, on the host."""
+        if self.sched is not None and all(r.h >= 0 for r in reqs):
+            return self.sched.prefill_arrays([(r.h, c, e) for r, (c, e) in zip(reqs, spans)], False)[:3]
+        ids, pos, slots = [], [], []
+        for r, (c, e) in zip(reqs, spans):
+            ids += r.prompt_ids[c:e]
+            pos += list(range(c, e))
+            slots += [r.blocks[t // PAGE] * PAGE + t % PAGE for t in range(c, e)]
+        return tuple(torch.tensor(v, dtype=torch.long) for v in (ids, pos, slots))
+
+    def _span_logits(self, x: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
+        """Logits of the given rows of ``_forward_spans``'s result."""
+        if self.hybrid:
+            from ..ops import mixers
+
+            h = mixers.rms(x.index_select(0, rows), self.head_w["norm_w"], self.cfg.rms_norm_eps, self.dtype)
+        else:
+            h = tf.final_norm(self.cfg, self.head_w, x.index_select(0, rows))
+        return self._lm_logits(h)
 
     def _mm_prefill_inputs(self, donors: list[Request], spans: list[tuple[int, int]]):
         """M-RoPE positions [3, T] and tower embeddings for the image-token rows of this prefill chunk.  The tower runs once per
@@ -817,8 +952,9 @@ class RolloutEngine:
         elif len(r.output_ids) >= p.max_new_tokens or r.num_tokens >= self.max_model_len:
             self._finish(r, "length")
 
-    def _decode_body(self, bs: int) -> None:
-        """One decode step over the first ``bs`` batch slots (captured into a CUDA graph)."""
+    def _decode_body(self, bs: int, sample: bool = True) -> torch.Tensor:
+        """One decode step over the first ``bs`` batch slots (captured into a CUDA graph); returns its logits.  ``sample=False`` stops
+        there: the caller supplies every next token (``extend``)."""
         cfg = self.cfg
         ids, pos = self.st_input_ids[:bs], self.st_positions[:bs]
         bt, sl, act = self.st_block_table[:bs], self.st_seq_lens[:bs], self.st_active[:bs]
@@ -828,6 +964,11 @@ class RolloutEngine:
         page_idx = torch.div(kvpos, PAGE, rounding_mode="floor").clamp_(max=self.max_blocks_per_seq)
         blk = bt.gather(1, page_idx.unsqueeze(1)).squeeze(1).long()
         slot = (blk * PAGE + kvpos % PAGE) * act          # idle slots write into scratch page 0
+        if self.hybrid:
+            logits = self._decode_hybrid(bs, kvpos, slot)
+            if sample:
+                self._decode_sample(bs, logits)
+            return logits
         inp = tf.DecodeInput(ids, pos, slot, bt, sl, self.max_model_len)
         x = torch.nn.functional.embedding(ids, self.embed_w["embed"]).to(self.dtype)
         if cfg.family == "gpt2":
@@ -849,6 +990,26 @@ class RolloutEngine:
         else:
             h = tf.final_norm(cfg, self.head_w, x)
         logits = self._lm_logits(h)
+        if sample:
+            self._decode_sample(bs, logits)
+        return logits
+
+    def _decode_hybrid(self, bs: int, kvpos: torch.Tensor, kv_slot: torch.Tensor) -> torch.Tensor:
+        """Decode step of a mixer stack: every batch slot is a span of one token; idle slots use page 0, state slot 0 and see no keys."""
+        from ..models import hybrid
+        from ..ops.mixers import SpanBatch
+
+        act = self.st_active[:bs]
+        b = SpanBatch(cu=self.arange32[:bs + 1], start=(kvpos * act).to(torch.int32), slot=self.st_state[:bs] * act, pos=kvpos, kv_slot=kv_slot,
+                      kv_len=self.st_seq_lens[:bs] * act.to(torch.int32), table=self.st_block_table[:bs], max_len=self.max_model_len)
+        x, h = hybrid.embed_forward(self.cfg, self.embed_w, self.st_input_ids[:bs])
+        last = len(self.layer_w) - 1
+        for i, w in enumerate(self.layer_w):
+            h = hybrid.layer_step(self.cfg, i, w, x, h, self.k_cache[i], b, self.head_w["norm_w"] if i == last else None)
+        return self._lm_logits(h)
+
+    def _decode_sample(self, bs: int, logits: torch.Tensor) -> None:
+        act = self.st_active[:bs]
         tok, lp = ops.sample_tokens(logits, self.st_temp[:bs], self.st_seeds[:bs], top_k=self._top_k, top_p=self._top_p)
         self.st_out_tok[:bs].copy_(tok)
         self.st_out_lp[:bs].copy_(lp)
@@ -864,34 +1025,39 @@ class RolloutEngine:
             b *= 2
         return min(b, self.max_num_seqs)
 
-    def _run_decode(self, bs: int) -> None:
-        if not self.use_cuda_graph or self._top_k > 0 or self._top_p < 1.0:
+    def _run_decode(self, bs: int, sample: bool = True) -> torch.Tensor:
+        """One decode step, through its CUDA graph where there is one; returns the step's logits (overwritten by the next step)."""
+        if not self.use_cuda_graph or (sample and (self._top_k > 0 or self._top_p < 1.0)):
             # top-k / top-p go through the sort-based library sampler (host-seeded RNG): not captured into a graph
-            self._decode_body(bs)
-            return
-        key = (bs, self._top_k, self._top_p)
+            return self._decode_body(bs, sample)
+        key = (bs, self._top_k, self._top_p) if sample else (bs, "logits")
         g = self._graphs.get(key)
         if g is None:
-            # warm-up on a side stream (also sets kernel attributes), then capture
-            snap = [t.clone() for t in (self.st_input_ids, self.st_positions, self.st_seq_lens, self.st_seeds)]
+            # warm-up on a side stream (also sets kernel attributes), then capture.  The warm-up step is real work: with every slot
+            # idle it leaves caches and recurrent states alone.
+            keep = (self.st_input_ids, self.st_positions, self.st_seq_lens, self.st_seeds, self.st_active)
+            snap = [t.clone() for t in keep]
+            if self.hybrid:
+                self.st_active.zero_()
             s = torch.cuda.Stream(device=self.device)
             s.wait_stream(torch.cuda.current_stream(self.device))
             with torch.cuda.stream(s):
-                self._decode_body(bs)
+                self._decode_body(bs, sample)
             torch.cuda.current_stream(self.device).wait_stream(s)
-            for dst, src in zip((self.st_input_ids, self.st_positions, self.st_seq_lens, self.st_seeds), snap):
+            for dst, src in zip(keep, snap):
                 dst.copy_(src)
             graph = torch.cuda.CUDAGraph()
             n0 = ops.total_launches()
             with torch.cuda.graph(graph):
-                self._decode_body(bs)
+                logits = self._decode_body(bs, sample)
             per_replay = ops.total_launches() - n0
-            for dst, src in zip((self.st_input_ids, self.st_positions, self.st_seq_lens, self.st_seeds), snap):
+            for dst, src in zip(keep, snap):
                 dst.copy_(src)
-            self._graphs[key] = (graph, per_replay)
+            self._graphs[key] = (graph, per_replay, logits)
             g = self._graphs[key]
         g[0].replay()
         ops.LAUNCHES["graph_replayed_kernels"] = ops.LAUNCHES.get("graph_replayed_kernels", 0) + g[1]
+        return g[2]
 
     def _compact_slots(self) -> None:
         """Keep running sequences in the lowest slots so a smaller graph bucket can be used."""
@@ -908,7 +1074,7 @@ class RolloutEngine:
         for src, dst in zip(high, low_free):
             r = self.running.pop(src)
             for t in (self.st_input_ids, self.st_positions, self.st_seq_lens, self.st_active, self.st_temp,
-                      self.st_seeds):
+                      self.st_seeds, self.st_state):
                 t[dst] = t[src]
             self.st_block_table[dst] = self.st_block_table[src]
             self.st_active[src] = 0
@@ -992,6 +1158,103 @@ class RolloutEngine:
         self._pending = new_pending
         self.stats["steps"] += 1
         return finished
+
+    # ------------------------------------------------------------------ given tokens
+    @torch.no_grad()
+    def extend(self, entries: list[tuple[Request, list[int], list[int]]]) -> torch.Tensor | None:
+        """One step over GIVEN tokens: every entry is (request, its next tokens, places among them whose logits are wanted).  All entries
+        are one batch — portions of prompts beside single tokens of others — run from the cache and state that earlier steps left; pages
+        are reserved as a request grows.  Requests come from ``open``; ``close`` gives back what they hold.  Sampling requests may not
+        be running at the same time.  Returns the wanted logits as fp32 rows in entry order, or None."""
+        if self.layer_w is None:
+            raise RuntimeError("RolloutEngine has no weights (call set_weights)")
+        if self.tp is not None or self.cfg.family == "gpt2" or self.full_cfg.vision is not None:
+            raise NotImplementedError("extend: single-GPU llama-family and mixer-stack text models")
+        self.init_kv_cache()
+        if any(not r.fed for r in self.running.values()) or self._pending is not None:
+            raise RuntimeError("extend while sampling requests are running")
+        spans = []
+        for r, tokens, _ in entries:
+            if not r.fed or r.finished:
+                raise ValueError("extend takes requests opened with open()")
+            c = len(r.prompt_ids)
+            if not tokens or c + len(tokens) > self.max_model_len:
+                raise ValueError(f"{r.rid}: {c} + {len(tokens)} tokens (at least one new token, at most {self.max_model_len} in all)")
+            self._grow(r, [int(t) for t in tokens])
+            spans.append((c, c + len(tokens)))
+        rows_of: list[list[int]] = [[] for _ in entries]       # row of the step's output for every token of an entry
+        if all(e - c == 1 and c > 0 for c, e in spans):
+            logits = self._extend_decode([r for r, _, _ in entries], spans)
+            rows_of = [[r.slot] for r, _, _ in entries]
+            x = None
+        else:
+            order = sorted(range(len(entries)), key=lambda i: spans[i][1] - spans[i][0] == 1)      # single tokens last
+            x, cu = self._forward_spans([entries[i][0] for i in order], [spans[i] for i in order])
+            for k, i in enumerate(order):
+                rows_of[i] = list(range(int(cu[k]), int(cu[k + 1])))
+        for (r, _, _), (_, e) in zip(entries, spans):
+            r.prefilled = e
+        self.stats["prefill_tokens"] += sum(e - c for c, e in spans)
+        self.stats["steps"] += 1
+        want = [rows_of[i][j] for i, (_, _, places) in enumerate(entries) for j in places]
+        if not want:
+            return None
+        rows = torch.tensor(want, dtype=torch.long, device=self.device)
+        return (logits.index_select(0, rows) if x is None else self._span_logits(x, rows)).float()
+
+    def open(self, rid: str | None = None) -> Request:
+        """A request whose tokens are supplied step by step (``extend``); it takes its slot and pages with its first tokens."""
+        return Request(rid or f"r{next(self._rid)}", [], SamplingParams(max_new_tokens=0), t_arrival=time.time(), fed=True)
+
+    def close(self, r: Request) -> None:
+        """Give back what an opened request holds."""
+        if r.slot >= 0:
+            self._finish(r, "stop")
+        r.finish_reason = "stop"
+
+    def _grow(self, r: Request, tokens: list[int]) -> None:
+        """Append given tokens to an open request: slot, state slot and pages at its first tokens, more pages as it grows."""
+        first = r.slot < 0
+        if self.sched is not None:
+            if first:
+                r.h = self.sched.open(tokens)
+                slot, r.blocks = self.sched.info(r.h)[:2]
+                if self.free_slots.pop() != slot:
+                    raise RuntimeError("native scheduler out of step with the engine's slots")
+                r.slot = slot
+            else:
+                self.sched.feed(r.h, tokens)
+                r.blocks = self.sched.info(r.h)[1]
+        else:
+            if first and not self.free_slots:
+                raise MemoryError("no free batch slot")
+            need = (len(r.prompt_ids) + len(tokens) + PAGE - 1) // PAGE - len(r.blocks)
+            r.blocks = r.blocks + self.alloc.alloc(max(0, need))
+            if first:
+                r.slot = self.free_slots.pop()
+        if first:
+            self.running[r.slot] = r
+            if self.state is not None:
+                r.state_slot = self.state.alloc()
+        r.prompt_ids += tokens
+
+    def _extend_decode(self, reqs: list[Request], spans: list[tuple[int, int]]) -> torch.Tensor:
+        """One given token for each request through the decode step (its CUDA graph where there is one); every other slot is idle."""
+        dev = self.device
+        bs = self._bucket(max(r.slot for r in reqs) + 1)
+        sl = torch.tensor([r.slot for r in reqs], dtype=torch.long, device=dev)
+        width = self.st_block_table.shape[1]
+        self.st_active.zero_()
+        self.st_active[sl] = 1
+        self.st_input_ids[sl] = torch.tensor([r.prompt_ids[c] for r, (c, _) in zip(reqs, spans)], dtype=torch.long, device=dev)
+        self.st_positions[sl] = torch.tensor([c for c, _ in spans], dtype=torch.long, device=dev)
+        self.st_seq_lens.zero_()
+        self.st_seq_lens[sl] = torch.tensor([e for _, e in spans], dtype=torch.int32, device=dev)
+        self.st_state[sl] = torch.tensor([r.state_slot for r in reqs], dtype=torch.long, device=dev)
+        self.st_block_table[sl] = torch.tensor([r.blocks + [0] * (width - len(r.blocks)) for r in reqs], dtype=torch.int32).to(dev)
+        logits = self._run_decode(bs, sample=False)
+        self.st_active.zero_()
+        return logits
 
     # ------------------------------------------------------------------ batch API
     @torch.no_grad()
