@@ -52,6 +52,11 @@ def parse():
     ap.add_argument("--mode", default="colocated", choices=["colocated", "disagg"],
                     help="colocated: every GPU rolls out and trains; disagg: N/2 rollout GPUs (TP engine servers behind the C++ "
                          "manager) stream to N/2 ZeRO trainers with a weight push every step (BASELINE config 3)")
+    ap.add_argument("--workload", default="ppo", choices=["ppo", "serving"],
+                    help="ppo: the flagship step (default); serving: prefill / decode throughput of a Ludesun stack beside the closest "
+                         "llama-family models of equal size (random weights, one GPU)")
+    ap.add_argument("--serving-layers", type=int, default=16)
+    ap.add_argument("--kernels", action="store_true", help="with --workload serving: time the single kernels against their rooflines instead")
     ap.add_argument("--comm", default=os.environ.get("BENCH_COMM", "p2p"), choices=["p2p", "nccl"])
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--rollout-weight-dtype", default="bf16", choices=["bf16", "fp8"],
@@ -287,6 +292,10 @@ def main() -> int:
     args = parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.workload == "serving":
+        from polyrl_b200.rollout.bench_serving import main as serving_main
+
+        return serving_main(args)
     if args.mode == "disagg":
         from polyrl_b200.trainer.bench_disagg import main as disagg_main
 

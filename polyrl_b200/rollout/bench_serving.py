@@ -1,0 +1,237 @@
+"""Serving throughput of mixer stacks beside the closest llama-family models of equal size: ``python bench.py --workload serving``.
+
+Random weights.  Prefill: packed prompts through ``RolloutEngine.extend`` (device time of the step); decode: the engine's CUDA-graph
+decode step; both timed with CUDA events after warm-up, weights (gigabytes) far larger than L2.  ``--kernels`` times the single kernels at
+the same layer sizes, with L2 flushed between iterations, against their roofline: the larger of bytes / measured copy bandwidth and
+FLOPs / measured bf16 GEMM rate.
+"""
+from __future__ import annotations
+
+import json
+import os
+from pathlib import Path
+
+import torch
+
+
+def _peaks() -> tuple[float, float, str]:
+    p = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
+    if p.exists():
+        d = json.loads(p.read_text())
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "measured"
+    return 6.65e12, 1.59e15, "fallback"
+
+
+def models(layers: int) -> dict:
+    """The mixer stack and, at the same width, feed-forward width and depth, the llama and the latent-attention (MLA) stack."""
+    from ..models import ModelConfig, get_model_config
+
+    hy = get_model_config("ludesun-4b")
+    lay = tuple(dict(hy.layers[i % 4], weights_of=i) for i in range(layers))
+    base = dict(family="llama", vocab_size=hy.vocab_size, hidden_size=hy.hidden_size, intermediate_size=hy.intermediate_size, num_layers=layers, num_heads=32,
+                max_position_embeddings=16384, rope_theta=500000.0, rms_norm_eps=1e-5, eos_token_id=-1)
+    return {"ludesun": ModelConfig(**{**hy.to_dict(), "num_layers": layers, "layers": lay}),
+            "llama": ModelConfig(**base, num_kv_heads=8),
+            "mla": ModelConfig(**base, num_kv_heads=32, attn_type="mla", q_lora_rank=1536, kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64,
+                               v_head_dim=128)}
+
+
+def _events(fn, iters: int, warmup: int, flush: torch.Tensor | None = None) -> float:
+    """Median device milliseconds of ``fn``."""
+    for _ in range(warmup):
+        fn()
+    ts = []
+    for _ in range(iters):
+        if flush is not None:
+            flush.zero_()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        ts.append(a.elapsed_time(b))
+    return sorted(ts)[len(ts) // 2]
+
+
+def run_models(args) -> list[dict]:
+    from ..models import TransformerWeights
+    from .engine import RolloutEngine
+
+    dev, rows = torch.device("cuda"), []
+    prefills = [(16, 1024), (2, 8192)]
+    decodes = [(64, 1024), (128, 2048)]
+    for name, cfg in models(args.serving_layers).items():
+        w = TransformerWeights(cfg, device=dev, dtype=torch.bfloat16, init=True)
+        n_params = cfg.num_params()
+        for nseq, length in prefills:
+            eng = RolloutEngine(cfg, dev, max_num_seqs=nseq, max_model_len=length + 64, kv_cache_tokens=nseq * (length + 64))
+            eng.set_weights(w.embed, w.layers, w.head)
+            g = torch.Generator().manual_seed(0)
+            toks = [torch.randint(3, cfg.vocab_size, (length,), generator=g).tolist() for _ in range(nseq)]
+
+            def step():
+                rs = [eng.open() for _ in toks]
+                eng.extend([(r, t, [length - 1]) for r, t in zip(rs, toks)])
+                for r in rs:
+                    eng.close(r)
+
+            ms = _events(step, args.steps_serving, 3)
+            rows.append({"model": name, "params": n_params, "phase": "prefill", "seqs": nseq, "len": length, "ms": round(ms, 3),
+                         "tokens_per_s": round(nseq * length / ms * 1e3)})
+            print(json.dumps(rows[-1]), flush=True)
+            del eng
+            torch.cuda.empty_cache()
+        for nseq, ctx in decodes:
+            eng = RolloutEngine(cfg, dev, max_num_seqs=nseq, max_model_len=ctx + 128, kv_cache_tokens=nseq * (ctx + 128) + 16)
+            eng.set_weights(w.embed, w.layers, w.head)
+            rs = [eng.open() for _ in range(nseq)]
+            g = torch.Generator().manual_seed(1)
+            for lo in range(0, nseq, 8):                      # prompts in, eight at a time
+                eng.extend([(r, torch.randint(3, cfg.vocab_size, (ctx,), generator=g).tolist(), []) for r in rs[lo:lo + 8]])
+            eng.extend([(r, [5], []) for r in rs])            # first decode step: captures the graph
+            eng.st_active.fill_(1)
+            ms = _events(lambda: eng._run_decode(nseq, sample=False), args.steps_serving, 3)
+            rows.append({"model": name, "params": n_params, "phase": "decode", "seqs": nseq, "len": ctx, "ms": round(ms, 3),
+                         "tokens_per_s": round(nseq / ms * 1e3)})
+            print(json.dumps(rows[-1]), flush=True)
+            for r in rs:
+                eng.close(r)
+            del eng
+            torch.cuda.empty_cache()
+        del w
+        torch.cuda.empty_cache()
+    return rows
+
+
+def run_kernels(args) -> list[dict]:
+    from .. import ops
+    from ..models import get_model_config, mla
+    from ..ops import mixers as M
+
+    C = ops.ext()
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    hbm, flops, kind = _peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows = []
+
+    def rnd(*s, dtype=bf, scale=1.0):
+        return (torch.randn(*s, device=dev) * scale).to(dtype)
+
+    def rec(name, like, shape, fn, nbytes, fl=0.0):
+        ms = _events(fn, args.steps_serving, 3, flush)
+        roof = max(nbytes / hbm, fl / flops) * 1e3
+        rows.append({"kernel": name, "like": like, "shape": shape, "us": round(ms * 1e3, 1), "roofline_us": round(roof * 1e3, 1),
+                     "of_" + kind: round(roof / ms, 3)})
+        print(json.dumps(rows[-1]), flush=True)
+
+    W, FF = 4096, 14336
+
+    def batch(lens, start, ctx=0):
+        n, t = len(lens), sum(lens)
+        cu = torch.tensor([0] + lens, dtype=torch.int32).cumsum(0).to(torch.int32)
+        seq_of = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), torch.tensor(lens)).to(dev)
+        long = lens[0] > 1
+        pos = torch.cat([torch.arange(start, start + x) for x in lens]).to(dev)
+        width = (start + max(lens) + 15) // 16
+        table = (torch.arange(n * width).reshape(n, width) + 1).int().to(dev)
+        kv = (table.long()[seq_of.long(), pos // 16] * 16 + pos % 16)
+        return M.SpanBatch(cu=cu.to(dev), start=torch.full((n,), start, dtype=torch.int32, device=dev), slot=torch.arange(1, n + 1, device=dev), pos=pos,
+                           kv_slot=kv, kv_len=(pos + 1).int(), table=table, seq_of=seq_of if long else None, n_long=n if long else 0,
+                           t_long=t if long else 0, max_long=max(lens) if long else 0, max_len=start + max(lens)), width * n + 1
+
+    for tag, lens, start in (("16 x 1024", [1024] * 16, 0), ("2 x 8192", [8192] * 2, 0), ("decode 128 @ 2048", [1] * 128, 2047)):
+        b, blocks = batch(lens, start)
+        t, n, dec = sum(lens), len(lens), lens[0] == 1
+        st_rw = 2 if dec else 1
+        # ---- recurrences
+        H, V, N, G = 128, 64, 128, 8
+        cache = {"S": torch.zeros(n + 1, H, N, V, device=dev)}
+        q, k, v = rnd(t, G * N), rnd(t, G * N, scale=N ** -0.5), rnd(t, H * V)
+        gates = M.Gates(rnd(t, H, dtype=torch.float32), None, torch.full((H,), -2.0, device=dev), None, torch.linspace(-2, 1, H, device=dev), torch.ones(H, device=dev))
+        rec("recurrence ssd", "attention", tag, lambda: M.scan(M.SSD, q, k, v, gates, 1.0, cache, b),
+            t * (2 * G * N * 2 + 2 * H * V * 2 + H * 4) + st_rw * n * H * N * V * 4, 0 if dec else t * H * (64 * (N + V) + 4 * N * V))
+        cw, cb = torch.randn(4, H * V + 2 * G * N, device=dev), torch.randn(H * V + 2 * G * N, device=dev)
+        cst, xc = torch.zeros(n + 1, 3, H * V + 2 * G * N, device=dev, dtype=bf), rnd(t, 2 * H * V + 2 * G * N)
+        ch = H * V + 2 * G * N
+        rec("conv + silu", "rope", tag, lambda: M.conv_silu(xc[:, H * V:], cw, cb, cst, b), t * ch * 4 + n * 6 * ch * 2)
+        y, z, gn = rnd(t, H * V), xc[:, :H * V], torch.ones(H * V, device=dev)
+        rec("gated norm (gate first)", "rmsnorm", tag, lambda: M.gated_norm(y, z, gn, 8, 1e-5, True), t * H * V * 6)
+        del cache, q, k, v, xc, y
+        H, V, N = 8, 512, 256
+        cache = {"S": torch.zeros(n + 1, H, N, V, device=dev), "n": torch.zeros(n + 1, H, N, device=dev), "m": torch.zeros(n + 1, H, device=dev)}
+        p = rnd(t, 2 * H * N + 2 * H * V)
+        g = rnd(t, 2 * H, dtype=torch.float32)
+        gates = M.Gates(g[:, :H], g[:, H:], torch.zeros(H, device=dev), torch.full((H,), 3.0, device=dev), cap=15.0)
+        rec("recurrence mlstm", "attention", tag, lambda: M.scan(M.MLSTM, p[:, :H * N], p[:, H * N:2 * H * N], p[:, 2 * H * N:2 * H * N + H * V], gates, N ** -0.5, cache, b),
+            t * (2 * H * N * 2 + 2 * H * V * 2 + 2 * H * 4) + st_rw * n * H * N * V * 4, 0 if dec else t * H * (64 * (N + V) + 4 * N * V))
+        y, gn = rnd(t, H * V), torch.ones(H * V, device=dev)
+        rec("gated norm (gate last)", "rmsnorm", tag, lambda: M.gated_norm(y, p[:, 2 * H * N + H * V:], gn, 8, 1e-5, False), t * H * V * 6)
+        del cache, p, y
+        # ---- latent attention
+        H, d, rd, V, r, qr = 32, 128, 64, 128, 512, 1536
+        pool = rnd(blocks, 1, 16, r + rd)
+        freq = M.rope_frequencies(rd, 1e4, dev)
+        a, q = rnd(t, qr + r + rd), rnd(t, H, d + rd)
+        wq, wkv, sink = torch.ones(qr, device=dev), torch.ones(r, device=dev), torch.zeros(H, device=dev)
+        rec("latent rows", "rmsnorm", tag, lambda: M.latent_prep(a, wq, wkv, freq, pool, b, 1e-5, not dec), t * ((qr + r + rd) * 4 + (0 if dec else (r + rd) * 2)))
+        rec("rope of queries", "rope", tag, lambda: M.rope_(q, d, freq, b.pos), t * H * rd * 4)
+        if dec:
+            q_lat = rnd(H, t, r)
+            rec("paged latent attention + sink", "paged attention", tag, lambda: M.latent_attention(q_lat, q, d, pool, b.table, None, b.kv_len, sink, 0.07, 2048),
+                t * 2048 * (r + rd) * 2, t * 2048 * H * 2 * (2 * r + rd))
+            qa = torch.cat([q_lat.transpose(0, 1), q[..., d:]], -1).contiguous()
+            rec("existing: mla.paged_latent_attention", "paged attention", tag, lambda: mla.paged_latent_attention(qa, pool, b.table, b.kv_len, r, 0.07),
+                t * 2048 * (r + rd) * 2, t * 2048 * H * 2 * (2 * r + rd))
+            kc, vc = rnd(blocks, 8, 16, 128), rnd(blocks, 8, 16, 128)
+            qq = rnd(t, 32 * 128)
+            rec("existing: paged_decode (GQA 32/8)", "paged attention", tag,
+                lambda: ops.paged_decode_attention(qq, kc, vc, b.table, b.kv_len, 32, 8, 128, 0.088, max_len=2048), t * 2048 * 8 * 128 * 4)
+            del kc, vc
+        else:
+            from ..ops.attention import attention_varlen
+
+            kk, vv = rnd(t, H, d + rd), rnd(t, H, V)
+            L = lens[0]
+            fl = n * L * L / 2 * H * 2 * (d + rd + V)
+            rec("packed attention 192 / 128 + sink", "attention", tag, lambda: M.sink_attention_varlen(q, kk, vv, b.cu, b.cu, 0.07, sink),
+                t * H * (2 * (d + rd) + 2 * V) * 2, fl)
+            vp = torch.nn.functional.pad(vv, (0, rd))
+            rec("existing: attention_varlen of the MLA stack", "attention", tag, lambda: attention_varlen(q, kk, vp, b.cu, L, True, 0.07),
+                t * H * (2 * (d + rd) + 2 * V) * 2, fl)
+            q8, k8, v8 = rnd(t, 32, 128), rnd(t, 8, 128), rnd(t, 8, 128)
+            rec("existing: attention_varlen (GQA 32/8)", "attention", tag, lambda: attention_varlen(q8, k8, v8, b.cu, L, True, 0.088),
+                t * 80 * 128 * 2, n * L * L / 2 * 32 * 2 * 256)
+            del kk, vv, vp, q8, k8, v8
+        del pool, a, q
+        # ---- rows and feed-forward
+        x32, yb, wn, hb = torch.randn(t, W, device=dev), rnd(t, W), torch.ones(W, device=dev), rnd(t, W)
+        rec("norm + residual add", "rmsnorm", tag, lambda: M.norm_add_(yb, x32, wn, 1e-5), t * W * 12)
+        wb = torch.ones(W, device=dev, dtype=bf)
+        rec("existing: add_rmsnorm", "rmsnorm", tag, lambda: C.add_rmsnorm_(hb, yb, wb, 1e-5), t * W * 8)
+        up, gu = rnd(FF, W, scale=W ** -0.5), rnd(2 * FF, W, scale=W ** -0.5)
+        rec("up projection + gelu", "gate/up + swiglu", tag, lambda: M.linear_gelu(hb, up), (t * W + FF * W + t * FF) * 2, 2.0 * t * W * FF)
+        rec("existing: gate/up + swiglu", "gate/up + swiglu", tag, lambda: ops.linear_swiglu(hb, gu), (t * W + 2 * FF * W + t * FF) * 2, 4.0 * t * W * FF)
+        qkv = rnd(t, 48 * 128)
+        ll = get_model_config("llama3-8b", max_position_embeddings=16384)
+        from ..models.transformer import rope_tables
+
+        cos, sin = rope_tables(ll, dev)
+        rec("existing: rope (GQA 32/8)", "rope", tag, lambda: ops.apply_rope(qkv, b.pos, cos, sin, 32, 8, 128), t * 40 * 128 * 4)
+        del x32, yb, hb, up, gu, qkv
+        torch.cuda.empty_cache()
+    return rows
+
+
+@torch.no_grad()
+def main(args) -> int:
+    if not torch.cuda.is_available():
+        print(json.dumps({"error": "the serving workload needs a CUDA device"}))
+        return 1
+    args.steps_serving = max(5, args.steps)
+    out = {"workload": "serving", "dtype": "bf16", "data": "random weights and tokens", "device": torch.cuda.get_device_name(), "peaks": _peaks()[2]}
+    out["kernels" if args.kernels else "models"] = run_kernels(args) if args.kernels else run_models(args)
+    if os.environ.get("BENCH_SERVING_OUT"):
+        Path(os.environ["BENCH_SERVING_OUT"]).write_text(json.dumps(out, indent=1))
+    print(json.dumps({k: v for k, v in out.items() if k not in ("kernels", "models")}), flush=True)
+    return 0
