@@ -24,7 +24,7 @@ int prl_mix_latent_tc_ok(int, int);
 }
 #include "mix_params.hpp"
 extern "C" {
-int prl_mix_scan(const prl::ScanParams*, int, int, cudaStream_t);
+int prl_mix_scan(const prl::ScanParams*, int, int, int, cudaStream_t);
 int prl_mix_chunk(const prl::ScanParams*, int, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
 }
@@ -206,12 +206,12 @@ at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const at::Tensor& 
   return out;
 }
 
-// gated linear recurrence over packed spans; mode 0 = state-space duality, 1 = matrix memory (csrc/mixers.cuh)
+// gated linear recurrence over packed spans; form 0 = token by token, 1 = every span is one token, 2 = chunked (bf16); mode 0 = state-space duality, 1 = matrix memory (csrc/mixers.cuh)
 void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
                      const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log,
                      const c10::optional<at::Tensor>& d_skip, double qscale, double cap, at::Tensor S, const c10::optional<at::Tensor>& nst,
                      const c10::optional<at::Tensor>& mst, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, at::Tensor counter,
-                     bool chunk, at::Tensor out) {
+                     int64_t form, at::Tensor out) {
   const int dt = dt_of(v, "mix_scan");
   rows2(q, "mix_scan q"); rows2(k, "mix_scan k"); rows2(v, "mix_scan v"); rows2(g0, "mix_scan g0");
   CHECK_F32(S); CHECK_F32(g0);
@@ -246,11 +246,11 @@ void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at:
   veci<int32_t>(counter, spans * H, "counter");
   p.counter = counter.data_ptr<int32_t>();
   p.H = H; p.N = N; p.V = V; p.spans = spans;
-  if (chunk) {
+  if (form == 2) {
     TORCH_CHECK(dt == 0 && prl_mix_chunk_supported(N), "mix_scan: the chunked kernel takes bf16 and N <= 256");
     check(prl_mix_chunk(&p, static_cast<int>(mode), cur_stream()), "mix_chunk");
   } else {
-    check(prl_mix_scan(&p, static_cast<int>(mode), dt, cur_stream()), "mix_scan");
+    check(prl_mix_scan(&p, static_cast<int>(mode), dt, form == 1, cur_stream()), "mix_scan");
   }
 }
 

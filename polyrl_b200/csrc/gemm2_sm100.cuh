@@ -61,7 +61,16 @@ struct TmaStoreParams {
 };
 struct EpiTmaStore {
   using Params = TmaStoreParams;
+  static constexpr bool kGelu = false;
 };
+// same with gelu (tanh form) on the accumulators, in the exactly equivalent shape z * sigmoid(2 u)
+struct EpiTmaStoreGelu {
+  using Params = TmaStoreParams;
+  static constexpr bool kGelu = true;
+};
+__device__ __forceinline__ float gelu_fast(float z) {
+  return __fdividef(z, 1.0f + __expf(fminf(-1.5957691216057308f * (z + 0.044715f * z * z * z), 80.f)));
+}
 
 template <class Cfg, class Epi>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kNumThreads, 1)
@@ -235,6 +244,10 @@ gemm2_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
                   r[8 * j + 7] = __float_as_uint(__uint_as_float(r[8 * j + 7]) + d.y);
                 }
               }
+            }
+            if constexpr (Epi::kGelu) {
+#pragma unroll
+              for (int j = 0; j < 64; ++j) r[j] = __float_as_uint(gelu_fast(__uint_as_float(r[j])));
             }
             // row `lane` of the 32 x 64 box: 8 x 16 B chunks, chunk j lands at (j ^ (lane & 7)) (128B swizzle)
             const uint32_t row_base = smem_u32(buf) + lane * 128;

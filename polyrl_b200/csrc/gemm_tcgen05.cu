@@ -111,7 +111,7 @@ struct EpiSwiglu {
   }
 };
 
-// H[M, N] = gelu(acc), tanh form, in the exactly equivalent shape z * sigmoid(2 u)
+// H[M, N] = gelu(acc)
 struct GeluParams {
   __nv_bfloat16* H;
   int64_t ldh;
@@ -130,8 +130,7 @@ struct EpiGelu {
       if (row >= M || valid <= 0) continue;
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        const float z = v[i];
-        v[i] = z / (1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+        v[i] = gelu_fast(v[i]);
       }
       store_row_chunk(p.H + static_cast<int64_t>(row) * p.ldh + n0 + c, v, valid);
     }
@@ -209,8 +208,8 @@ extern "C" int prl_gemm_gelu_bf16(const void* A, const void* W, void* H, int M, 
                                   cudaStream_t stream) {
   GeluParams sp{static_cast<__nv_bfloat16*>(H), ldh};
   if (M > kBlockM && N > 128) {
-    using Cfg2 = Gemm2Cfg<256, false, false, false>;
-    return launch_gemm2<Cfg2, EpiGelu>(A, W, nullptr, M, N, K, lda * 2, ldw * 2, 0, sp, 0, stream);
+    using Cfg2 = Gemm2Cfg<256, false, false, true>;
+    return launch_gemm2<Cfg2, EpiTmaStoreGelu>(A, W, H, M, N, K, lda * 2, ldw * 2, ldh * 2, TmaStoreParams{nullptr, 0}, 0, stream);
   }
   using Cfg = GemmCfg<64, 2>;
   return launch_gemm<Cfg, EpiGelu, NoGate, false>(A, W, M, N, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);

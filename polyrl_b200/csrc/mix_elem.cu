@@ -96,6 +96,41 @@ __global__ void __launch_bounds__(256) mix_gated_norm_kernel(const T* __restrict
   const T* zr = z + row * ldz + c0;
   T* orow = out + row * ldo + c0;
   float ss = 0.f;
+  if constexpr (VEC == 8) {
+    constexpr int HOLD = 4;                              // groups of up to 32 * WPG * 8 * HOLD elements stay in registers
+    if (gs <= 32 * WPG * VEC * HOLD) {
+      float u[HOLD][VEC];
+#pragma unroll
+      for (int k = 0; k < HOLD; ++k) {
+        const int c = (k * 32 * WPG + t) * VEC;
+        if (c < gs) {
+          float g[VEC];
+          ld_vec<T, VEC>(yr + c, u[k]);
+          ld_vec<T, VEC>(zr + c, g);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) {
+            const float f = GATE_FIRST ? silu_t<T>(g[i]) : sigmoid_t<T>(g[i]);
+            if (!GATE_FIRST) ss += u[k][i] * u[k][i];
+            u[k][i] *= f;
+            if (GATE_FIRST) ss += u[k][i] * u[k][i];
+          }
+        }
+      }
+      const float r = rsqrtf(block_sum<WPG>(ss, red) / gs + eps);
+#pragma unroll
+      for (int k = 0; k < HOLD; ++k) {
+        const int c = (k * 32 * WPG + t) * VEC;
+        if (c < gs) {
+          float ww[VEC];
+          ld_vec<float, VEC>(w + c0 + c, ww);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) u[k][i] *= r * ww[i];
+          st_vec<T, VEC>(orow + c, u[k]);
+        }
+      }
+      return;
+    }
+  }
   for (int c = t * VEC; c < gs; c += 32 * WPG * VEC) {
     float v[VEC], g[VEC];
     ld_vec<T, VEC>(yr + c, v);
@@ -149,6 +184,57 @@ __global__ void __launch_bounds__(128) mix_conv_kernel(const T* __restrict__ x, 
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc[i] = silu_f(acc[i]);
     st_vec<T, VEC>(out + static_cast<int64_t>(t) * ldo + c, acc);
+  }
+}
+// the same for a fixed small tap count: 8 channels per thread, TT tokens with the window and the taps in registers
+template <class T, int TAPS, int TT>
+__global__ void __launch_bounds__(128) mix_conv_window_kernel(const T* __restrict__ x, int64_t ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                                                              const T* __restrict__ state, const int32_t* __restrict__ cu, const int32_t* __restrict__ start,
+                                                              const int64_t* __restrict__ slot, const int32_t* __restrict__ seq_of, T* __restrict__ out,
+                                                              int64_t ldo, int ch, int total) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (c >= ch) return;
+  const int tb = blockIdx.y * TT, te = min(total, tb + TT);
+  float wt[TAPS][8], bs[8], win[TAPS][8];               // win[j]: input of token t - (TAPS - 1) + j
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) ld_vec<float, 8>(w + static_cast<int64_t>(j) * ch + c, wt[j]);
+  ld_vec<float, 8>(bias + c, bs);
+  int cur = -1;
+#pragma unroll 4
+  for (int t = tb; t < te; ++t) {
+    const int s = seq_of[t];
+    if (s != cur) {                                      // (re)fill the window at a span's start or at the tile's first token
+      cur = s;
+      const int t0 = cu[s];
+      const bool fresh = start[s] == 0;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int u = t - (TAPS - 1) + j;
+        if (u >= t0) {
+          ld_vec<T, 8>(x + static_cast<int64_t>(u) * ldx + c, win[j]);
+        } else if (!fresh) {
+          ld_vec<T, 8>(state + (slot[s] * (TAPS - 1) + (u - t0 + TAPS - 1)) * ch + c, win[j]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) win[j][i] = 0.f;
+        }
+      }
+    }
+    ld_vec<T, 8>(x + static_cast<int64_t>(t) * ldx + c, win[TAPS - 1]);
+    float acc[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = bs[i];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[i] += wt[j][i] * win[j][i];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = silu_t<T>(acc[i]);
+    st_vec<T, 8>(out + static_cast<int64_t>(t) * ldo + c, acc);
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
   }
 }
 // the last taps - 1 inputs of every span become its slot's state (row j of the new state is input len - (taps - 1) + j)
@@ -344,16 +430,37 @@ extern "C" int prl_mix_conv(const void* x, int64_t ldx, const float* w, const fl
     PRL_CUDA_CHECK(cudaGetLastError());
     return 0;
   }
-  const int TT = total > 65535 * 4 ? 32 : 4;
-  const unsigned gy = (total + TT - 1) / TT;
-  if (gy > 65535) return -221;
-  if (TT == 4)
-    MIX_DISPATCH(vec, (mix_conv_kernel<T, VEC, 4><<<dim3(gx, gy), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,
-                                                                               start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
-  else
-    MIX_DISPATCH(vec, (mix_conv_kernel<T, VEC, 32><<<dim3(gx, gy), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,
-                                                                                start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
-  PRL_CUDA_CHECK(cudaGetLastError());
+  if (vec && taps >= 2 && taps <= 4 && total <= 65535 * 16) {
+    dim3 gw(gx, (total + 15) / 16);
+#define MIX_CW(TAPS)                                                                                                                     \
+  do {                                                                                                                                   \
+    if (dtype == 0) {                                                                                                                    \
+      using T = __nv_bfloat16;                                                                                                           \
+      mix_conv_window_kernel<T, TAPS, 16><<<gw, 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,   \
+                                                              start, slot, seq_of, static_cast<T*>(out), ldo, ch, total);                \
+    } else {                                                                                                                             \
+      using T = float;                                                                                                                   \
+      mix_conv_window_kernel<T, TAPS, 16><<<gw, 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,   \
+                                                              start, slot, seq_of, static_cast<T*>(out), ldo, ch, total);                \
+    }                                                                                                                                    \
+  } while (0)
+    if (taps == 2) MIX_CW(2);
+    else if (taps == 3) MIX_CW(3);
+    else MIX_CW(4);
+#undef MIX_CW
+    PRL_CUDA_CHECK(cudaGetLastError());
+  } else {
+    const int TT = total > 65535 * 4 ? 32 : 4;
+    const unsigned gy = (total + TT - 1) / TT;
+    if (gy > 65535) return -221;
+    if (TT == 4)
+      MIX_DISPATCH(vec, (mix_conv_kernel<T, VEC, 4><<<dim3(gx, gy), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,
+                                                                                 start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
+    else
+      MIX_DISPATCH(vec, (mix_conv_kernel<T, VEC, 32><<<dim3(gx, gy), 128, 0, st>>>(static_cast<const T*>(x), ldx, w, bias, static_cast<const T*>(state), cu,
+                                                                                  start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
+    PRL_CUDA_CHECK(cudaGetLastError());
+  }
   if (taps > 1) {
     dim3 g2((ch + 127) / 128, spans);
     if (dtype == 0)

@@ -3,8 +3,8 @@
 // The cache holds ONE row per token and layer: [latent r | rotated shared key rd].  Query row (t, head) is
 // [q_lat r | q_rot rd] (key up-projection folded into q_lat), so   score = q . row * scale,   out = softmax . row[:r],
 // where the sink adds exp(sink_h) to the softmax denominator and nothing else.
-//   * mix_latent_tc_kernel   decode: 16 heads x 32 keys per step on the tensor cores, cp.async double buffering over
-//                            pages, split over the keys with a merge kernel — every cache byte is read once per 16 heads
+//   * mix_latent_tc_kernel   decode: 16 or 32 heads x 32 keys per step on the tensor cores, cp.async double buffering
+//                            over pages, split over the keys with a merge kernel
 //   * mix_latent_row_kernel  any size, bf16 or fp32: one CTA per (row, head), fp32 throughout
 #include "mixers.cuh"
 
@@ -91,66 +91,92 @@ __device__ __forceinline__ void lt_ldsm_t(uint32_t (&r)[4], const __nv_bfloat16*
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
 }
 
-// NTW: output column tiles (8 wide) per warp; r <= 32 * NTW, r a multiple of 16, r + rd a multiple of 8
-template <int NTW>
-__global__ void __launch_bounds__(kLtWarps * 32) mix_latent_tc_kernel(LatentParams p) {
+// MT row tiles of 16 heads per CTA, 4 * MT warps: warp w scores keys [8 (w % 4), +8) for row tile w / 4 and owns NTW output column
+// tiles (8 wide) of every row tile.  r <= 32 * MT * NTW, r a multiple of 16, r + rd a multiple of 8.
+template <int NTW, int MT>
+__global__ void __launch_bounds__(128 * MT) mix_latent_tc_kernel(LatentParams p) {
+  constexpr int NW = 4 * MT, HT = 16 * MT;
   extern __shared__ __align__(128) uint8_t raw[];
   const int D = p.r + p.rd, Dp = (D + 31) / 32 * 32, LD = Dp + 8;
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(raw);       // [16][LD]
-  __nv_bfloat16* sK = sQ + 16 * LD;                                // [2][32][LD]
-  __nv_bfloat16* sP = sK + 2 * kLtKeys * LD;                       // [16][40]
-  __shared__ float s_m[kLtWarps][16], s_l[kLtWarps][16];
-  const int h0 = blockIdx.x * 16, row = blockIdx.y, split = blockIdx.z;
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(raw);       // [HT][LD]
+  __nv_bfloat16* sK = sQ + HT * LD;                                // [2][32][LD]
+  __nv_bfloat16* sP = sK + 2 * kLtKeys * LD;                       // [HT][40]
+  __shared__ float s_m[4][HT], s_l[4][HT];
+  const int h0 = blockIdx.x * HT, row = blockIdx.y, split = blockIdx.z;
   const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, gq = lane >> 2, qd = lane & 3;
-  const int hn = min(16, p.H - h0);
+  const int wn = w & 3, wm = w >> 2;
+  const int hn = min(HT, p.H - h0);
   const int len = p.kv_len[row];
   const int tiles = (len + kLtKeys - 1) / kLtKeys, per = (tiles + p.splits - 1) / p.splits;
   const int tb = split * per, te = min(tiles, tb + per);
   const int32_t* bt = p.table + static_cast<int64_t>(p.seq_of ? p.seq_of[row] : row) * p.ld_table;
   const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(p.pool);
 
-  for (int i = tid; i < 16 * Dp; i += kLtWarps * 32) {
-    const int h = i / Dp, c = i % Dp;
-    __nv_bfloat16 v = __float2bfloat16(0.f);
-    if (h < hn && c < D)
-      v = c < p.r ? static_cast<const __nv_bfloat16*>(p.q_lat)[(static_cast<int64_t>(h0 + h) * p.R + row) * p.r + c]
-                  : static_cast<const __nv_bfloat16*>(p.q)[row * p.ldq + static_cast<int64_t>(h0 + h) * p.dq + p.d + c - p.r];
-    sQ[h * LD + c] = v;
-  }
-  auto load = [&](int tile, int buf) {
-    for (int i = tid; i < kLtKeys * (Dp / 8); i += kLtWarps * 32) {
-      const int j = i / (Dp / 8), c = (i % (Dp / 8)) * 8, key = tile * kLtKeys + j;
-      const bool ok = key < len && c < D;
-      const __nv_bfloat16* g = pool + (ok ? (static_cast<int64_t>(bt[key / kLtPage]) * kLtPage + key % kLtPage) * D + c : 0);
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(sK + (buf * kLtKeys + j) * LD + c)), "l"(g), "r"(ok ? 16 : 0) : "memory");
+  // rows w, w + NW, ... of a tile per warp: one page number for each, neighbouring lanes on neighbouring 16-byte pieces
+  int64_t src[kLtKeys / NW];
+  auto pages = [&](int tile) {
+#pragma unroll
+    for (int i = 0; i < kLtKeys / NW; ++i) {
+      const int key = tile * kLtKeys + w + i * NW;
+      src[i] = key < len ? (static_cast<int64_t>(bt[key / kLtPage]) * kLtPage + key % kLtPage) * D : -1;
+    }
+  };
+  auto load = [&](int buf) {
+#pragma unroll
+    for (int i = 0; i < kLtKeys / NW; ++i) {
+      __nv_bfloat16* dst = sK + (buf * kLtKeys + w + i * NW) * LD;
+      for (int c = lane * 8; c < Dp; c += 256) {
+        const bool ok = src[i] >= 0 && c < D;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + c)), "l"(pool + (ok ? src[i] + c : 0)), "r"(ok ? 16 : 0) : "memory");
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float o[NTW][4];
+  if (tb < te) {
+    pages(tb);
+    load(0);
+    if (tb + 1 < te) pages(tb + 1);
+  }
+  for (int h = w; h < HT; h += NW) {
+    for (int c = lane; c < Dp; c += 32) {
+      __nv_bfloat16 v = __float2bfloat16(0.f);
+      if (h < hn && c < D)
+        v = c < p.r ? static_cast<const __nv_bfloat16*>(p.q_lat)[(static_cast<int64_t>(h0 + h) * p.R + row) * p.r + c]
+                    : static_cast<const __nv_bfloat16*>(p.q)[row * p.ldq + static_cast<int64_t>(h0 + h) * p.dq + p.d + c - p.r];
+      sQ[h * LD + c] = v;
+    }
+  }
+  float o[MT][NTW][4];
 #pragma unroll
-  for (int i = 0; i < NTW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;        // rows gq, gq + 8
-  if (tb < te) load(tb, 0);
+  for (int a = 0; a < MT; ++a)
+#pragma unroll
+    for (int i = 0; i < NTW; ++i) o[a][i][0] = o[a][i][1] = o[a][i][2] = o[a][i][3] = 0.f;
+  float m[MT][2], l0 = 0.f, l1 = 0.f;                              // maxima of every row pair; sums of this warp's own row tile and keys
+#pragma unroll
+  for (int a = 0; a < MT; ++a) m[a][0] = m[a][1] = -INFINITY;
   for (int t = tb; t < te; ++t) {
     const int buf = (t - tb) & 1;
     asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();                                               // tile t is in; everyone is done with the other buffer
-    if (t + 1 < te) load(t + 1, buf ^ 1);
+    if (t + 1 < te) {
+      load(buf ^ 1);
+      if (t + 2 < te) pages(t + 2);
+    }
     const __nv_bfloat16* kt = sK + buf * kLtKeys * LD;
     float sa[4] = {0.f, 0.f, 0.f, 0.f}, sb[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 2
+#pragma unroll 3
     for (int k = 0; k < Dp; k += 32) {
       uint32_t a[4], b[4];
-      lt_ldsm(b, &kt[(w * 8 + (lane & 7)) * LD + k + (lane >> 3) * 8]);
-      lt_ldsm(a, &sQ[(lane & 15) * LD + k + (lane >> 4) * 8]);
+      lt_ldsm(b, &kt[(wn * 8 + (lane & 7)) * LD + k + (lane >> 3) * 8]);
+      lt_ldsm(a, &sQ[(wm * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8]);
       lt_mma(sa, a, b[0], b[1]);
-      lt_ldsm(a, &sQ[(lane & 15) * LD + k + 16 + (lane >> 4) * 8]);
+      lt_ldsm(a, &sQ[(wm * 16 + (lane & 15)) * LD + k + 16 + (lane >> 4) * 8]);
       lt_mma(sb, a, b[2], b[3]);
     }
     float x[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int key = t * kLtKeys + w * 8 + 2 * qd + (e & 1);
+      const int key = t * kLtKeys + wn * 8 + 2 * qd + (e & 1);
       x[e] = key < len ? (sa[e] + sb[e]) * p.scale : -INFINITY;
     }
     float c0 = fmaxf(x[0], x[1]), c1 = fmaxf(x[2], x[3]);
@@ -158,32 +184,41 @@ __global__ void __launch_bounds__(kLtWarps * 32) mix_latent_tc_kernel(LatentPara
     c0 = fmaxf(c0, __shfl_xor_sync(0xffffffffu, c0, 2));
     c1 = fmaxf(c1, __shfl_xor_sync(0xffffffffu, c1, 1));
     c1 = fmaxf(c1, __shfl_xor_sync(0xffffffffu, c1, 2));
-    if (qd == 0) { s_m[w][gq] = c0; s_m[w][gq + 8] = c1; }
+    if (qd == 0) { s_m[wn][wm * 16 + gq] = c0; s_m[wn][wm * 16 + gq + 8] = c1; }
     __syncthreads();
-    float n0 = m0, n1 = m1;
+    float own0 = 0.f, own1 = 0.f, al0 = 1.f, al1 = 1.f;            // this warp's row tile
 #pragma unroll
-    for (int i = 0; i < kLtWarps; ++i) { n0 = fmaxf(n0, s_m[i][gq]); n1 = fmaxf(n1, s_m[i][gq + 8]); }
-    const float a0 = expf(m0 - n0), a1 = expf(m1 - n1);            // n is finite: a tile holds at least one key
-    m0 = n0; m1 = n1;
-    const float p0 = expf(x[0] - n0), p1 = expf(x[1] - n0), p2 = expf(x[2] - n1), p3 = expf(x[3] - n1);
-    l0 = l0 * a0 + p0 + p1;
-    l1 = l1 * a1 + p2 + p3;
-    *reinterpret_cast<uint32_t*>(&sP[gq * 40 + w * 8 + 2 * qd]) = pack_bf16(p0, p1);
-    *reinterpret_cast<uint32_t*>(&sP[(gq + 8) * 40 + w * 8 + 2 * qd]) = pack_bf16(p2, p3);
+    for (int a = 0; a < MT; ++a) {
+      float n0 = m[a][0], n1 = m[a][1];
 #pragma unroll
-    for (int i = 0; i < NTW; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+      for (int i = 0; i < 4; ++i) { n0 = fmaxf(n0, s_m[i][a * 16 + gq]); n1 = fmaxf(n1, s_m[i][a * 16 + gq + 8]); }
+      const float a0 = __expf(m[a][0] - n0), a1 = __expf(m[a][1] - n1);        // n is finite: a tile holds at least one key
+      m[a][0] = n0; m[a][1] = n1;
+      if (a == wm) { own0 = n0; own1 = n1; al0 = a0; al1 = a1; }
+#pragma unroll
+      for (int i = 0; i < NTW; ++i) { o[a][i][0] *= a0; o[a][i][1] *= a0; o[a][i][2] *= a1; o[a][i][3] *= a1; }
+    }
+    const float p0 = __expf(x[0] - own0), p1 = __expf(x[1] - own0), p2 = __expf(x[2] - own1), p3 = __expf(x[3] - own1);
+    l0 = l0 * al0 + p0 + p1;
+    l1 = l1 * al1 + p2 + p3;
+    *reinterpret_cast<uint32_t*>(&sP[(wm * 16 + gq) * 40 + wn * 8 + 2 * qd]) = pack_bf16(p0, p1);
+    *reinterpret_cast<uint32_t*>(&sP[(wm * 16 + gq + 8) * 40 + wn * 8 + 2 * qd]) = pack_bf16(p2, p3);
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < kLtKeys; k += 16) {
-      uint32_t a[4], b[4];
-      lt_ldsm(a, &sP[(lane & 15) * 40 + k + (lane >> 4) * 8]);
+      uint32_t a[MT][4], b[4];
+#pragma unroll
+      for (int i = 0; i < MT; ++i) lt_ldsm(a[i], &sP[(i * 16 + (lane & 15)) * 40 + k + (lane >> 4) * 8]);
 #pragma unroll
       for (int i = 0; i < NTW; i += 2) {
         const int col = (w * NTW + i) * 8;
         if (col < p.r) {
           lt_ldsm_t(b, &kt[(k + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + col + (lane >> 4) * 8]);
-          lt_mma(o[i], a, b[0], b[1]);
-          lt_mma(o[i + 1], a, b[2], b[3]);
+#pragma unroll
+          for (int j = 0; j < MT; ++j) {
+            lt_mma(o[j][i], a[j], b[0], b[1]);
+            lt_mma(o[j][i + 1], a[j], b[2], b[3]);
+          }
         }
       }
     }
@@ -192,34 +227,34 @@ __global__ void __launch_bounds__(kLtWarps * 32) mix_latent_tc_kernel(LatentPara
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  if (qd == 0) { s_l[w][gq] = l0; s_l[w][gq + 8] = l1; }
+  if (qd == 0) { s_l[wn][wm * 16 + gq] = l0; s_l[wn][wm * 16 + gq + 8] = l1; }
   __syncthreads();
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
+  for (int e = 0; e < 2 * MT; ++e) {
     const int hr = gq + 8 * e, h = h0 + hr;
     if (hr >= hn) continue;
-    const float l = s_l[0][hr] + s_l[1][hr] + s_l[2][hr] + s_l[3][hr], m = e ? m1 : m0;
+    const float l = s_l[0][hr] + s_l[1][hr] + s_l[2][hr] + s_l[3][hr], mx = m[e >> 1][e & 1];
     const int64_t base = static_cast<int64_t>(h) * p.R + row;
     if (p.splits == 1) {
-      const float snk = p.sink ? p.sink[h] : -INFINITY, mm = fmaxf(m, snk);
-      const float f = m == -INFINITY ? 0.f : expf(m - mm);
+      const float snk = p.sink ? p.sink[h] : -INFINITY, mm = fmaxf(mx, snk);
+      const float f = mx == -INFINITY ? 0.f : expf(mx - mm);
       const float den = l * f + (p.sink ? expf(snk - mm) : 0.f), g = den > 0.f ? f / den : 0.f;
       __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + base * p.r;
 #pragma unroll
       for (int i = 0; i < NTW; ++i) {
         const int c = (w * NTW + i) * 8 + 2 * qd;
-        if (c < p.r) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[i][2 * e] * g, o[i][2 * e + 1] * g);
+        if (c < p.r) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[e >> 1][i][2 * (e & 1)] * g, o[e >> 1][i][2 * (e & 1) + 1] * g);
       }
     } else {
       float* dst = p.part + (base * p.splits + split) * p.r;
 #pragma unroll
       for (int i = 0; i < NTW; ++i) {
         const int c = (w * NTW + i) * 8 + 2 * qd;
-        if (c < p.r) *reinterpret_cast<float2*>(dst + c) = make_float2(o[i][2 * e], o[i][2 * e + 1]);
+        if (c < p.r) *reinterpret_cast<float2*>(dst + c) = make_float2(o[e >> 1][i][2 * (e & 1)], o[e >> 1][i][2 * (e & 1) + 1]);
       }
       if (w == 0 && qd == 0) {
         float* ml = p.part + static_cast<int64_t>(p.H) * p.R * p.splits * p.r + (base * p.splits + split) * 2;
-        ml[0] = m;
+        ml[0] = mx;
         ml[1] = l;
       }
     }
@@ -244,17 +279,17 @@ __global__ void __launch_bounds__(128) mix_latent_merge_kernel(LatentParams p) {
   }
 }
 
-template <int NTW>
+template <int NTW, int MT>
 static int run_tc(const LatentParams& p, cudaStream_t st) {
   const int LD = (p.r + p.rd + 31) / 32 * 32 + 8;
-  const int smem = (16 + 2 * kLtKeys) * LD * 2 + 16 * 40 * 2;
+  const int smem = (16 * MT + 2 * kLtKeys) * LD * 2 + 16 * MT * 40 * 2;
   static bool attr = false;
   if (!attr) {
-    PRL_CUDA_CHECK(cudaFuncSetAttribute(mix_latent_tc_kernel<NTW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    PRL_CUDA_CHECK(cudaFuncSetAttribute(mix_latent_tc_kernel<NTW, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
     attr = true;
   }
   if (smem > 160 * 1024) return -232;
-  mix_latent_tc_kernel<NTW><<<dim3((p.H + 15) / 16, p.R, p.splits), kLtWarps * 32, smem, st>>>(p);
+  mix_latent_tc_kernel<NTW, MT><<<dim3((p.H + 16 * MT - 1) / (16 * MT), p.R, p.splits), 128 * MT, smem, st>>>(p);
   PRL_CUDA_CHECK(cudaGetLastError());
   if (p.splits > 1) {
     mix_latent_merge_kernel<<<dim3(p.H, p.R), 128, 0, st>>>(p);
@@ -292,8 +327,13 @@ extern "C" int prl_mix_latent(const LatentParams* p, int tc, int dtype, cudaStre
   if (p->R > 65535 || p->splits < 1 || p->splits > 65535) return -230;
   if (!tc) return dtype == 0 ? pick_row<__nv_bfloat16>(*p, st) : pick_row<float>(*p, st);
   if (dtype != 0 || !prl_mix_latent_tc_ok(p->r, p->rd)) return -231;
-  if (p->r <= 64) return run_tc<2>(*p, st);
-  if (p->r <= 128) return run_tc<4>(*p, st);
-  if (p->r <= 256) return run_tc<8>(*p, st);
-  return run_tc<16>(*p, st);
+  if (p->H > 16) {                  // two row tiles share every key load
+    if (p->r <= 128) return run_tc<2, 2>(*p, st);
+    if (p->r <= 256) return run_tc<4, 2>(*p, st);
+    return run_tc<8, 2>(*p, st);
+  }
+  if (p->r <= 64) return run_tc<2, 1>(*p, st);
+  if (p->r <= 128) return run_tc<4, 1>(*p, st);
+  if (p->r <= 256) return run_tc<8, 1>(*p, st);
+  return run_tc<16, 1>(*p, st);
 }

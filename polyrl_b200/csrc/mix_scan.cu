@@ -4,8 +4,9 @@
 //   kMlstm (xLSTM matrix memory)             m' = max(f + m, i),  S = e^(f+m-m') S + e^(i-m') k v^T,  n likewise with k alone,
 //                                            y = S^T q / (max(|n . q|, e^(-m')) + 1e-6);  m starts at 0
 //
-// One CTA = one (span, head, 32 value columns): lane = value column, warp w owns the state rows w, w + 8, ... in registers,
-// so a state row of 32 columns is one 128-byte line and a decode step reads and writes every state byte exactly once.
+// mix_step_kernel serves spans of one token (decode): every state byte is read and written once, streaming.
+// mix_scan_kernel: one CTA = one (span, head, 32 value columns): lane = value column, warp w owns the state rows w, w + 8, ... in registers
+// from the first token to the last.
 #include "mixers.cuh"
 
 namespace prl {
@@ -119,6 +120,141 @@ mix_scan_kernel(ScanParams p) {
   }
 }
 
+// ---- one token per span: the state streams through registers, CPL neighbouring value columns per lane
+template <int CPL>
+__device__ __forceinline__ void ld_cols(const float* p, float (&v)[CPL]) {
+  if constexpr (CPL == 4) { const float4 q = __ldcs(reinterpret_cast<const float4*>(p)); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+  else if constexpr (CPL == 2) { const float2 q = __ldcs(reinterpret_cast<const float2*>(p)); v[0] = q.x; v[1] = q.y; }
+  else v[0] = __ldcs(p);
+}
+template <int CPL>
+__device__ __forceinline__ void st_cols(float* p, const float (&v)[CPL]) {
+  if constexpr (CPL == 4) __stcs(reinterpret_cast<float4*>(p), make_float4(v[0], v[1], v[2], v[3]));
+  else if constexpr (CPL == 2) __stcs(reinterpret_cast<float2*>(p), make_float2(v[0], v[1]));
+  else __stcs(p, v[0]);
+}
+
+template <class T, int MODE, int CPL>
+__global__ void __launch_bounds__(kScanWarps * 32)
+mix_step_kernel(ScanParams p) {
+  constexpr int U = 8;                                   // state rows in flight per warp
+  __shared__ float s_q[512], s_k[512], s_n[512];
+  __shared__ float s_red[kScanWarps][32 * CPL + 1], s_dot[kScanWarps];
+  const int vt = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
+  const int w = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+  const int t = p.cu[s];
+  if (p.cu[s + 1] <= t) return;
+  const bool fresh = p.start[s] == 0;
+  const int64_t slot = p.slot[s], hb = slot * p.H + h;
+  const int col = vt * 32 * CPL + lane * CPL;
+  const bool ok = col < p.V;                             // V is a multiple of CPL
+  float* Sg = p.S + hb * static_cast<int64_t>(p.N) * p.V + col;
+  float st[U][CPL];
+  auto load = [&](int n0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int n = n0 + u * kScanWarps + w;
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) st[u][c] = 0.f;
+      if (!fresh && ok && n < p.N) ld_cols<CPL>(Sg + static_cast<int64_t>(n) * p.V, st[u]);
+    }
+  };
+  load(0);
+  const T* q = static_cast<const T*>(p.q) + static_cast<int64_t>(t) * p.ldq + static_cast<int64_t>(h / p.rep) * p.N;
+  const T* k = static_cast<const T*>(p.k) + static_cast<int64_t>(t) * p.ldk + static_cast<int64_t>(h / p.rep) * p.N;
+  const T* v = static_cast<const T*>(p.v) + static_cast<int64_t>(t) * p.ldv + static_cast<int64_t>(h) * p.V;
+  float vv[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) vv[c] = ok ? to_f<T>(v[col + c]) : 0.f;
+  float keep, add, floor_ = 0.f, m2 = 0.f;
+  const float b0 = p.b0 ? p.b0[h] : 0.f;
+  if constexpr (MODE == kSsd) {
+    add = softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0);
+    keep = expf(-expf(p.a_log[h]) * add);
+  } else {
+    const float m = fresh ? 0.f : p.mst[hb];
+    const float gi = softcap_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0, p.cap);
+    const float gf = logsigmoid_f(softcap_f(p.g1[static_cast<int64_t>(t) * p.ldg + h] + (p.b1 ? p.b1[h] : 0.f), p.cap));
+    m2 = fmaxf(gf + m, gi);
+    keep = expf(gf + m - m2);
+    add = expf(gi - m2);
+    floor_ = expf(-m2);
+  }
+  float dot = 0.f;
+  for (int n = tid; n < p.N; n += kScanWarps * 32) {
+    const float qn = to_f<T>(q[n]) * p.qscale, kn = to_f<T>(k[n]);
+    s_q[n] = qn;
+    s_k[n] = kn;
+    if constexpr (MODE == kMlstm) {
+      const float nn = keep * (fresh ? 0.f : p.nst[hb * p.N + n]) + add * kn;
+      s_n[n] = nn;
+      dot += nn * qn;
+    }
+  }
+  if constexpr (MODE == kMlstm) {
+    dot = warp_sum(dot);
+    if (lane == 0) s_dot[w] = dot;
+  }
+  __syncthreads();
+  float acc[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) acc[c] = 0.f;
+  for (int n0 = 0; n0 < p.N; n0 += U * kScanWarps) {
+    if (n0) load(n0);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int n = n0 + u * kScanWarps + w;
+      if (n < p.N) {
+        const float ak = add * s_k[n], qn = s_q[n];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          st[u][c] = keep * st[u][c] + ak * vv[c];
+          acc[c] += qn * st[u][c];
+        }
+        if (ok) st_cols<CPL>(Sg + static_cast<int64_t>(n) * p.V, st[u]);
+      }
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) s_red[w][lane * CPL + c] = acc[c];
+  __syncthreads();
+  for (int c = tid; c < 32 * CPL; c += kScanWarps * 32) {
+    const int gc = vt * 32 * CPL + c;
+    if (gc < p.V) {
+      float y = 0.f;
+#pragma unroll
+      for (int i = 0; i < kScanWarps; ++i) y += s_red[i][c];
+      if constexpr (MODE == kSsd) {
+        if (p.d_skip) y += p.d_skip[h] * to_f<T>(v[gc]);
+      } else {
+        float d = 0.f;
+#pragma unroll
+        for (int i = 0; i < kScanWarps; ++i) d += s_dot[i];
+        y /= fmaxf(fabsf(d), floor_) + 1e-6f;
+      }
+      static_cast<T*>(p.out)[static_cast<int64_t>(t) * p.ldo + static_cast<int64_t>(h) * p.V + gc] = from_f<T>(y);
+    }
+  }
+  if constexpr (MODE == kMlstm) {
+    if (last_tile(p.counter + s * p.H + h, gridDim.x)) {
+      for (int n = tid; n < p.N; n += kScanWarps * 32) p.nst[hb * p.N + n] = s_n[n];
+      if (tid == 0) p.mst[hb] = m2;
+    }
+  }
+}
+
+template <class T, int MODE>
+static int launch_step(const ScanParams& p, cudaStream_t st) {
+  const bool al = (reinterpret_cast<uintptr_t>(p.S) & 15) == 0;
+  const int threads = kScanWarps * 32;
+  if (p.N > 512) return -203;
+  if (al && p.V % 4 == 0 && p.V > 64) mix_step_kernel<T, MODE, 4><<<dim3((p.V + 127) / 128, p.H, p.spans), threads, 0, st>>>(p);
+  else if (al && p.V % 2 == 0 && p.V > 32) mix_step_kernel<T, MODE, 2><<<dim3((p.V + 63) / 64, p.H, p.spans), threads, 0, st>>>(p);
+  else mix_step_kernel<T, MODE, 1><<<dim3((p.V + 31) / 32, p.H, p.spans), threads, 0, st>>>(p);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
 template <class T, int MODE>
 static int launch_scan(const ScanParams& p, cudaStream_t st) {
   dim3 grid((p.V + kScanVT - 1) / kScanVT, p.H, p.spans);
@@ -137,10 +273,14 @@ static int launch_scan(const ScanParams& p, cudaStream_t st) {
 
 using namespace prl;
 
-// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm
-extern "C" int prl_mix_scan(const ScanParams* p, int mode, int dtype, cudaStream_t st) {
+// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm; single: every span is one token
+extern "C" int prl_mix_scan(const ScanParams* p, int mode, int dtype, int single, cudaStream_t st) {
   if (p->spans <= 0) return 0;
   if (p->spans > 65535 || p->H > 65535) return -202;
+  if (single) {
+    if (dtype == 0) return mode == kSsd ? launch_step<__nv_bfloat16, kSsd>(*p, st) : launch_step<__nv_bfloat16, kMlstm>(*p, st);
+    return mode == kSsd ? launch_step<float, kSsd>(*p, st) : launch_step<float, kMlstm>(*p, st);
+  }
   if (dtype == 0) return mode == kSsd ? launch_scan<__nv_bfloat16, kSsd>(*p, st) : launch_scan<__nv_bfloat16, kMlstm>(*p, st);
   return mode == kSsd ? launch_scan<float, kSsd>(*p, st) : launch_scan<float, kMlstm>(*p, st);
 }

@@ -56,6 +56,13 @@ __device__ __forceinline__ void st_vec(T* p, const float (&v)[VEC]) {
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// bf16 outputs: the fast exponential and division (relative error about 2^-21) are far below the output's rounding
+template <class T>
+__device__ __forceinline__ float sigmoid_t(float z) {
+  return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(fminf(-z, 80.f))) : sigmoid_f(z);
+}
+template <class T>
+__device__ __forceinline__ float silu_t(float z) { return z * sigmoid_t<T>(z); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float logsigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float softcap_f(float z, float cap) { return cap * tanhf(z / cap); }

@@ -174,17 +174,15 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
     ctr = _counter(v.device, b.spans * H)
     out = torch.empty(v.shape, device=v.device, dtype=v.dtype)
 
-    def run(lo: int, hi: int, chunk: bool) -> None:
+    def run(lo: int, hi: int, form: int) -> None:       # 0: token by token, 1: one token per span, 2: chunked
         _C().mix_scan_(mode, q, k, v, gates.g0, gates.g1, gates.b0, gates.b1, gates.a_log, gates.d_skip, qscale, gates.cap, S, cache.get("n"),
-                       cache.get("m"), b.cu[lo:hi + 1], b.start[lo:hi], b.slot[lo:hi], ctr, chunk, out)
+                       cache.get("m"), b.cu[lo:hi + 1], b.start[lo:hi], b.slot[lo:hi], ctr, form, out)
 
     chunk = v.dtype == torch.bfloat16 and b.max_long >= CHUNK_MIN and _C().mix_chunk_supported(N)
-    if chunk and b.n_long:
-        run(0, b.n_long, True)
-        if b.n_long < b.spans:
-            run(b.n_long, b.spans, False)
-    else:
-        run(0, b.spans, False)
+    if b.n_long:
+        run(0, b.n_long, 2 if chunk else 0)
+    if b.n_long < b.spans:
+        run(b.n_long, b.spans, 1)
     return out
 
 
@@ -268,7 +266,7 @@ def rope_(q: torch.Tensor, d: int, freq: torch.Tensor, pos: torch.Tensor) -> Non
 
 
 def _splits(rows: int, heads: int, max_len: int) -> int:
-    ctas = rows * ((heads + 15) // 16)
+    ctas = rows * ((heads + 31) // 32)
     return max(1, min((2 * 148 + ctas - 1) // ctas, max(1, max_len // 256), 32))
 
 
