@@ -26,6 +26,8 @@ int prl_mix_latent_tc_ok(int, int);
 extern "C" {
 int prl_mix_scan(const prl::ScanParams*, int, int, int, cudaStream_t);
 int prl_mix_chunk(const prl::ScanParams*, int, cudaStream_t);
+int prl_mix_chunk_tc_ok(const prl::ScanParams*);
+int prl_mix_chunk_tc(const prl::ScanParams*, int, int32_t*, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
 }
 
@@ -206,7 +208,8 @@ at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const at::Tensor& 
   return out;
 }
 
-// gated linear recurrence over packed spans; form 0 = token by token, 1 = every span is one token, 2 = chunked (bf16); mode 0 = state-space duality, 1 = matrix memory (csrc/mixers.cuh)
+// gated linear recurrence over packed spans; form 0 = token by token, 1 = every span is one token, 2 = chunked (bf16), 3 = chunked on
+// tcgen05 where the layout allows, else 2; the last counter element is the error flag; mode 0 = state-space duality, 1 = matrix memory (csrc/mixers.cuh)
 void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
                      const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log,
                      const c10::optional<at::Tensor>& d_skip, double qscale, double cap, at::Tensor S, const c10::optional<at::Tensor>& nst,
@@ -243,10 +246,12 @@ void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at:
   p.out = out.data_ptr(); p.ldo = H * V;
   p.S = S.data_ptr<float>();
   p.cu = veci<int32_t>(cu, spans + 1, "cu"); p.start = veci<int32_t>(start, spans, "start"); p.slot = veci<int64_t>(slot, spans, "slot");
-  veci<int32_t>(counter, spans * H, "counter");
+  veci<int32_t>(counter, spans * H + 1, "counter");
   p.counter = counter.data_ptr<int32_t>();
   p.H = H; p.N = N; p.V = V; p.spans = spans;
-  if (form == 2) {
+  if (form == 3 && dt == 0 && prl_mix_chunk_tc_ok(&p)) {
+    check(prl_mix_chunk_tc(&p, static_cast<int>(mode), p.counter + counter.numel() - 1, cur_stream()), "mix_chunk_tc");
+  } else if (form >= 2) {
     TORCH_CHECK(dt == 0 && prl_mix_chunk_supported(N), "mix_scan: the chunked kernel takes bf16 and N <= 256");
     check(prl_mix_chunk(&p, static_cast<int>(mode), cur_stream()), "mix_chunk");
   } else {

@@ -52,12 +52,19 @@ _RETIRED: list = []     # outgrown counters stay alive: captured graphs hold the
 
 
 def _counter(device: torch.device, n: int) -> torch.Tensor:
-    """Zeroed arrival counters of the recurrence kernels (each launch leaves them zero again)."""
+    """Zeroed arrival counters of the recurrence kernels (each launch leaves them zero again); the last element is an error flag."""
     key = (device.type, device.index)
-    if key not in _COUNTERS or _COUNTERS[key].numel() < n:
+    if key not in _COUNTERS or _COUNTERS[key].numel() <= n:
         _RETIRED.append(_COUNTERS.get(key))
-        _COUNTERS[key] = torch.zeros(max(n, 1 << 17), device=device, dtype=torch.int32)
+        _COUNTERS[key] = torch.zeros(max(n, 1 << 17) + 1, device=device, dtype=torch.int32)
     return _COUNTERS[key]
+
+
+def check_errors(device: torch.device) -> None:
+    """Raise if a bounded wait inside a kernel ran out (reads one flag back: call it where the host synchronises anyway)."""
+    c = _COUNTERS.get((device.type, device.index))
+    if c is not None and int(c[-1]):
+        raise RuntimeError("a wait inside a chunked recurrence kernel timed out")
 
 
 # --------------------------------------------------------------------------------------------
@@ -160,6 +167,7 @@ class Gates:
 
 
 CHUNK_MIN = 8           # spans shorter than this go through the token-by-token kernel
+TC_MIN = 65             # from here on the 128-token tcgen05 chunks pay
 
 
 def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Gates, qscale: float, cache: dict, b: SpanBatch) -> torch.Tensor:
@@ -174,13 +182,13 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
     ctr = _counter(v.device, b.spans * H)
     out = torch.empty(v.shape, device=v.device, dtype=v.dtype)
 
-    def run(lo: int, hi: int, form: int) -> None:       # 0: token by token, 1: one token per span, 2: chunked
+    def run(lo: int, hi: int, form: int) -> None:       # 0: token by token, 1: one token per span, 2 / 3: chunked
         _C().mix_scan_(mode, q, k, v, gates.g0, gates.g1, gates.b0, gates.b1, gates.a_log, gates.d_skip, qscale, gates.cap, S, cache.get("n"),
                        cache.get("m"), b.cu[lo:hi + 1], b.start[lo:hi], b.slot[lo:hi], ctr, form, out)
 
     chunk = v.dtype == torch.bfloat16 and b.max_long >= CHUNK_MIN and _C().mix_chunk_supported(N)
     if b.n_long:
-        run(0, b.n_long, 2 if chunk else 0)
+        run(0, b.n_long, (3 if b.max_long >= TC_MIN else 2) if chunk else 0)
     if b.n_long < b.spans:
         run(b.n_long, b.spans, 1)
     return out

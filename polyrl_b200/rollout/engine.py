@@ -770,6 +770,10 @@ class RolloutEngine:
         p0 = reqs[0].params
         tok, lp = ops.sample_tokens(logits, temps, seeds, greedy=False, top_k=p0.top_k, top_p=p0.top_p)
         tok_c, lp_c = tok.tolist(), lp.tolist()
+        if self.hybrid and self.is_cuda:
+            from ..ops import mixers
+
+            mixers.check_errors(tok.device)
         for r in reqs:
             r.donor = None            # release the reference; pages stay shared through the allocator's ref-counts
         live, rows = [], []
@@ -1200,6 +1204,10 @@ class RolloutEngine:
         if not want:
             return None
         rows = torch.tensor(want, dtype=torch.long, device=self.device)
+        if self.hybrid and self.is_cuda and x is not None:
+            from ..ops import mixers
+
+            mixers.check_errors(x.device)
         return (logits.index_select(0, rows) if x is None else self._span_logits(x, rows)).float()
 
     def open(self, rid: str | None = None) -> Request:

@@ -45,16 +45,17 @@ SIZES = [(1, 1, 1, 1), (3, 1, 7, 10), (2, 2, 24, 40), (4, 2, 64, 64), (2, 1, 128
 
 
 @pytest.mark.parametrize("mode", ["ssd", "mlstm"])
-@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+@pytest.mark.parametrize("dtype,tc_min", [(torch.bfloat16, 2), (torch.bfloat16, 1 << 30), (torch.float32, 0)])
 @pytest.mark.parametrize("H,G,N,V", SIZES)
-def test_scan(mode, dtype, H, G, N, V):
-    """Fresh spans, then a second call that continues some of them in other places of the batch: outputs and final states."""
+def test_scan(mode, dtype, tc_min, H, G, N, V, monkeypatch):
+    """Every form of the recurrence kernels (tcgen05 chunks, mma chunks, token by token, single step).  Fresh spans, then a second call that continues some of them in other places of the batch: outputs and final states."""
     from polyrl_b200.ops import mixers as M
 
+    monkeypatch.setattr(M, "TC_MIN", tc_min)
     if mode == "mlstm":
         G = H
-    lens = {"a": 150, "b": 64, "c": 9, "d": 2, "e": 1, "f": 65}
-    cuts = {"a": 77, "b": 63, "c": 1, "d": 1, "e": 1, "f": 64}
+    lens = {"a": 300, "b": 128, "c": 9, "d": 2, "e": 1, "f": 129}
+    cuts = {"a": 140, "b": 127, "c": 1, "d": 1, "e": 1, "f": 128}
     g = gen(N + V)
     data = {k: dict(q=torch.randn(n, G * N, generator=g).to(dtype), k=(torch.randn(n, G * N, generator=g) * N ** -0.5).to(dtype),
                     v=torch.randn(n, H * V, generator=g).to(dtype), g0=torch.randn(n, H, generator=g) * 2, g1=torch.randn(n, H, generator=g) + 1)
@@ -97,7 +98,8 @@ def test_scan(mode, dtype, H, G, N, V):
         y = torch.cat(got[k])
         assert rel(y, want[k]) < tol, k
         assert rel(y[-1:], want[k][-1:]) < 3 * tol, k
-    # the state itself: one more fp32 step with q = e_j reads it out through the token-by-token kernel
+    M.check_errors(cache["S"].device)
+    # the state itself
     fin = {k: cache["S"][slot[k]].cpu().double() for k in lens}
     for k in ("a", "f"):
         x = {n: t.double() for n, t in data[k].items()}
