@@ -32,13 +32,19 @@ struct ChunkTc {
   static constexpr int OFF_V = OFF_K + KBUF * QB;
   static constexpr int OFF_S = OFF_V + kTcTile;                       // hi: MB tiles, lo: MB tiles
   static constexpr int OFF_F = OFF_S + 2 * MB * kTcTile;
-  static constexpr int SMEM = OFF_F + 8192 + 1024;
+  static constexpr int SMEM = OFF_F + 11264 + 1024;
 };
 
+struct alignas(16) TcGates {                       // weights of one chunk
+  float row[kTcC], col[kTcC], mul[kTcC], carry[kTcC], wgt[kTcC], flo[kTcC];
+  float keep;
+};
+static_assert(sizeof(TcGates) % 16 == 0, "both copies are read as float4");
 struct TcShared {                        // behind the tiles
-  float row[kTcC], col[kTcC], mul[kTcC], carry[kTcC], wgt[kTcC], flo[kTcC], den[2][kTcC], deni[2][kTcC];
+  TcGates gate[2];
+  float den[2][kTcC], deni[2][kTcC], half[2][kTcC];
   float n[256];
-  float keep, m;
+  float m;
   uint64_t bar[4];
   uint32_t tmem;
 };
@@ -88,7 +94,7 @@ __device__ __forceinline__ void tc_raw(TcRaw& g, const ScanParams& p, int64_t t0
 // one warp: weights of the chunk.  weight(t, s) = 2^(row_t + col_s) mul_s (qscale folded into row), carry: carried-in factor with
 // qscale, wgt: weight of a token in the chunk's final state
 template <int MODE>
-__device__ __forceinline__ void tc_gates(TcShared& sm, const TcRaw& g, const ScanParams& p, int nv, float b0, float b1, float a_neg, int lane) {
+__device__ __forceinline__ void tc_gates(TcGates& sm, float& m_run, const TcRaw& g, const ScanParams& p, int nv, float b0, float b1, float a_neg, int lane) {
   constexpr float kL2e = 1.4426950408889634f;
   const float lq = log2f(p.qscale);
   float la[4], ad[4];
@@ -138,7 +144,7 @@ __device__ __forceinline__ void tc_gates(TcShared& sm, const TcRaw& g, const Sca
       const float x = __shfl_up_sync(0xffffffffu, rm, o);
       if (lane >= o) rm = fmaxf(rm, x);
     }
-    const float m0 = sm.m;
+    const float m0 = m_run;
     const float pm = __shfl_up_sync(0xffffffffu, rm, 1);
     const float base = lane ? fmaxf(pm, m0) : m0;
     const float m_end = fmaxf(__shfl_sync(0xffffffffu, rm, 31), m0);
@@ -154,7 +160,7 @@ __device__ __forceinline__ void tc_gates(TcShared& sm, const TcRaw& g, const Sca
       sm.flo[t] = expf(-(la[e] + M));
     }
     __syncwarp();
-    if (lane == 0) { sm.keep = expf(m0 - m_end); sm.m = end + m_end; }
+    if (lane == 0) { sm.keep = expf(m0 - m_end); m_run = end + m_end; }
   }
 }
 
@@ -198,7 +204,7 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
   load_k(0, 0);
   load_v(0);
   TcRaw raw;
-  if (w == 1) tc_raw<MODE>(raw, p, t0, min(kTcC, len), h, lane);
+  if (w == 4) tc_raw<MODE>(raw, p, t0, min(kTcC, len), h, lane);
   if (tid == 0) {
     for (int i = 0; i < 4; ++i) mbar_init(&sm.bar[i], 1);
     fence_barrier_init();
@@ -234,7 +240,12 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
   if (MODE == kMlstm) {
     const int64_t hb = slot * p.H + h;
     sm.n[tid] = (!fresh && tid < N) ? p.nst[hb * N + tid] : 0.f;
-    if (tid == 0) sm.m = fresh ? 0.f : p.mst[hb];
+  }
+  if (w == 4) {          // rows 0..31, columns 64..127 of the scores: the warp whose share lies above the diagonal runs the gates, a chunk ahead
+    if (MODE == kMlstm && lane == 0) sm.m = fresh ? 0.f : p.mst[slot * p.H + h];
+    __syncwarp();
+    tc_gates<MODE>(sm.gate[0], sm.m, raw, p, min(kTcC, len), b0, b1, a_neg, lane);
+    if (len > kTcC) tc_raw<MODE>(raw, p, t0 + kTcC, min(kTcC, len - kTcC), h, lane);
   }
   tc_fence_before();
   __syncthreads();
@@ -251,6 +262,7 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
     const int c0 = ci * kTcC, nv = min(kTcC, len - c0);
     const uint32_t ph = ci & 1;
     const bool more = ci + 1 < chunks;
+    const TcGates& gt = sm.gate[ci & 1];
     const uint8_t* sK = smem + Cfg::OFF_K + (Cfg::KBUF == 2 ? (ci & 1) : 0) * QB;
     asm volatile("cp.async.wait_all;" ::: "memory");
     fence_proxy_async();
@@ -274,10 +286,6 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
     }
     __syncwarp();          // the issuing lane first: its warp must not sit in a wait for products that are not issued yet
     if (Cfg::KBUF == 2 && more) load_k(c0 + kTcC, (ci + 1) & 1);                 // (its last reader finished with the previous chunk)
-    if (w == 1) {
-      tc_gates<MODE>(sm, raw, p, nv, b0, b1, a_neg, lane);
-      if (more) tc_raw<MODE>(raw, p, t0 + c0 + kTcC, min(kTcC, len - c0 - kTcC), h, lane);
-    }
     if (MODE == kMlstm) {                                                        // n_0 . q_t, half of the columns per thread
       float d0 = 0.f, d1 = 0.f;
       if (have_state) {
@@ -293,13 +301,18 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
       }
       sm.deni[g][r] = d0 + d1;
     }
-    __syncthreads();                                                             // gates
+    if (MODE == kMlstm) __syncthreads();                                         // (the scores may overlay the Q that was just read)
     ok = tc_wait(&sm.bar[0], ph) && ok;
     if (NB == 4) ok = tc_wait(&sm.bar[1], ph) && ok;                             // the scores overlay Q
     tc_fence_after();
+    if (w == 4 && more) {
+      const int c1 = c0 + kTcC;
+      tc_gates<MODE>(sm.gate[(ci + 1) & 1], sm.m, raw, p, min(kTcC, len - c1), b0, b1, a_neg, lane);
+      if (len > c1 + kTcC) tc_raw<MODE>(raw, p, t0 + c1 + kTcC, min(kTcC, len - c1 - kTcC), h, lane);
+    }
     // ---- weighted scores of row r, columns [64 g, +64)
     {
-      const float row = sm.row[r];
+      const float row = gt.row[r];
       float den = 0.f;
 #pragma unroll
       for (int c = 0; c < 64; c += 32) {
@@ -312,11 +325,11 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
           tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 32; i += 4) {
-            const float4 cc = *reinterpret_cast<const float4*>(&sm.col[cb + i]);
+            const float4 cc = *reinterpret_cast<const float4*>(&gt.col[cb + i]);
             float x[4] = {__uint_as_float(v[i]) * fast_exp2(row + cc.x), __uint_as_float(v[i + 1]) * fast_exp2(row + cc.y),
                           __uint_as_float(v[i + 2]) * fast_exp2(row + cc.z), __uint_as_float(v[i + 3]) * fast_exp2(row + cc.w)};
             if (MODE == kSsd) {
-              const float4 mm = *reinterpret_cast<const float4*>(&sm.mul[cb + i]);
+              const float4 mm = *reinterpret_cast<const float4*>(&gt.mul[cb + i]);
               x[0] *= mm.x; x[1] *= mm.y; x[2] *= mm.z; x[3] *= mm.w;
             }
             if (cb + 31 > quad * 32) {                                           // block on the diagonal
@@ -354,7 +367,7 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
       umma_commit(&sm.bar[2]);
     }
     __syncwarp();
-    const float keep = sm.keep, wgt = sm.wgt[r];
+    const float keep = gt.keep, wgt = gt.wgt[r];
     if (MODE == kMlstm) {                                                        // n = keep n + sum_s w_s k_s: two state rows, half of the tokens
       float a0 = 0.f, a1 = 0.f;
       const int np = tid & 127, half = tid >> 7, n = 2 * np;
@@ -364,16 +377,15 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
 #pragma unroll 8
         for (int t = half * 64; t < half * 64 + 64; ++t) {
           const float2 x = unpack_bf16(*reinterpret_cast<const uint32_t*>(kt + t * 128 + ((u ^ (t & 7)) << 4) + off));
-          a0 += sm.wgt[t] * x.x;
-          a1 += sm.wgt[t] * x.y;
+          a0 += gt.wgt[t] * x.x;
+          a1 += gt.wgt[t] * x.y;
         }
       }
-      // the second half's sums travel through `row` / `col`, whose readers are past the barrier above
-      if (half == 1) { sm.row[np] = a0; sm.col[np] = a1; }
+      if (half == 1) { sm.half[0][np] = a0; sm.half[1][np] = a1; }
       __syncthreads();
       if (half == 0) {
-        sm.n[n] = keep * sm.n[n] + a0 + sm.row[np];
-        sm.n[n + 1] = keep * sm.n[n + 1] + a1 + sm.col[np];
+        sm.n[n] = keep * sm.n[n] + a0 + sm.half[0][np];
+        sm.n[n + 1] = keep * sm.n[n + 1] + a1 + sm.half[1][np];
       }
     }
     if (NB == 2) {
@@ -424,11 +436,11 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
       tmem_ld_32x32(tP + lane_base + g * 32, a);
       if (have_state) tmem_ld_32x32(tI + lane_base + g * 32, b);
       tmem_ld_wait();
-      const float carry = have_state ? sm.carry[r] : 0.f;
+      const float carry = have_state ? gt.carry[r] : 0.f;
       float inv = 1.f;
       if (MODE == kMlstm) {
         const float den = sm.den[0][r] + sm.den[1][r] + carry * (sm.deni[0][r] + sm.deni[1][r]);
-        inv = 1.f / (fmaxf(fabsf(den), sm.flo[r]) + 1e-6f);
+        inv = 1.f / (fmaxf(fabsf(den), gt.flo[r]) + 1e-6f);
       }
       if (r < nv) {
         __nv_bfloat16* dst = gO + static_cast<int64_t>(c0 + r) * p.ldo + g * 32;
@@ -509,7 +521,7 @@ template <int MODE, int NB>
 static int run_tc(const ScanParams& p, int32_t* err, cudaStream_t st) {
   auto kern = mix_chunk_tc_kernel<MODE, NB>;
   constexpr int smem = ChunkTc<NB>::SMEM;
-  static_assert(smem <= 232448 && sizeof(TcShared) <= 8192, "shared memory");
+  static_assert(smem <= 232448 && sizeof(TcShared) <= 11264, "shared memory");
   static bool attr = false;
   if (!attr) {
     PRL_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
