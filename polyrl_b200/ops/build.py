@@ -36,7 +36,9 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-lineinfo", "-O3", "-std=c++17",
     "--use_fast_math" if False else "-DPRL_NO_FAST_MATH",
-    "-Xcompiler", "-fPIC",
+    # a function-local static of a kernel launcher (e.g. "attributes are set") belongs to ONE module: launchers linked into both
+    # modules must not share it, as GNU unique symbols would across shared objects
+    "-Xcompiler", "-fPIC,-fvisibility=hidden,-fno-gnu-unique",
     "--expt-relaxed-constexpr",
 ]
 
@@ -103,7 +105,7 @@ def build(force: bool = False, verbose: bool = False, modules: tuple[str, ...] =
                 inc += ["-isystem", p]
             inc += ["-isystem", sysconfig.get_paths()["include"]]
             jobs.insert(0, [
-                "g++", "-O2", "-std=c++17", "-fPIC", f"-DTORCH_EXTENSION_NAME={mod}", "-DTORCH_API_INCLUDE_EXTENSION_H",
+                "g++", "-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-fno-gnu-unique", f"-DTORCH_EXTENSION_NAME={mod}", "-DTORCH_API_INCLUDE_EXTENSION_H",
                 f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}", *inc, "-c", str(bsrc), "-o", str(bobj),
             ])
             stale[mod] = True
