@@ -52,7 +52,8 @@ def generate(model: str, rows: list[dict], n_samples: int = 1, temperature: floa
     cfg = get_model_config(model)
     tok = None
     is_dir = Path(model).is_dir()
-    if tokenizer_path or is_dir:
+    has_tok = is_dir and any((Path(model) / f).exists() for f in ("tokenizer.json", "tokenizer_config.json", "tokenizer.model", "vocab.json"))
+    if tokenizer_path or has_tok:            # (a folder without one serves token-id prompts)
         tok = load_tokenizer(tokenizer_path or model)
     dtype = torch.bfloat16 if dev.type == "cuda" else torch.float32
     eng = RolloutEngine(cfg, dev, max_num_seqs=min(256, max(8, batch_size)), max_model_len=prompt_length + response_length,

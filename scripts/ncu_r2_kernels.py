@@ -1,5 +1,5 @@
 """One launch each of the round-2 flagship kernels (CTA-pair GEMM forward, flash attention forward / backward) for an
-`ncu --set full` capture:  ncu --set full --clock-control none --import-source on -k regex:'gemm2_sm100|attn_fwd_kernel|attn_bwd_kernel'
+`ncu --set full` capture:  ncu --set full --clock-control none -k regex:'gemm2_sm100|attn_fwd_kernel|attn_bwd_kernel'
 -c 3 -o gpurun_out/r2_kernels python scripts/ncu_r2_kernels.py"""
 import torch
 

@@ -191,6 +191,15 @@ def test_greedy_generation_through_the_scheduler(folders, chunk, native, monkeyp
     assert len(eng.state.free) == 3 and not eng.running
 
 
+def test_offline_generation_entry_point(folders):
+    from polyrl_b200.trainer.main_generation import generate
+
+    cfg, sd, d = folders["even"]
+    rows = [{"prompt": seq(n, cfg["vocab"], n)} for n in (4, 19)]
+    out = generate(str(d), rows, temperature=0.0, response_length=6, prompt_length=32, device="cpu")
+    assert [r["response_ids"][0] for r in out] == [greedy_oracle(cfg, sd, r["prompt"], 6) for r in rows]
+
+
 def test_sample_groups_share_the_prompt(folders):
     cfg, sd, d = folders["even"]
     prompt = seq(21, cfg["vocab"], 2)
