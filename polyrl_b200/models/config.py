@@ -36,6 +36,7 @@ class ModelConfig:
     partial_rotary_factor: float = 1.0
     rope_interleaved: bool = False
     sandwich_norm: bool = False      # GLM-4: extra RMSNorm on the attention output and on the MLP output, before the residual adds
+    norm_offset: float = 0.0         # mixer stacks: added to the stored weights of the residual stream's norms
     qkv_bias: bool = False           # Qwen2
     qk_norm: bool = False            # Qwen3: per-head RMSNorm on q and k (weights [head_dim]) before RoPE
     tie_word_embeddings: bool = False
@@ -377,14 +378,14 @@ class ModelConfig:
                    name=hf.get("_name_or_path", mt), **vis_kw, **{**moe_kw, **vl_moe_kw}, **{**glm_kw, **mla_kw, **act_kw})
 
 
-def _ludesun(hf: dict) -> ModelConfig:
-    from .hybrid import ludesun_config
+def _stack(hf: dict) -> ModelConfig:
+    from .stacks import DESIGNS, stack_config
 
-    return ludesun_config(hf)
+    return stack_config(DESIGNS[hf["architecture"].lower()], hf)
 
 
 # designs whose config.json names an ``architecture`` instead of a ``model_type``
-ARCHITECTURES = {"Ludesun": _ludesun}
+ARCHITECTURES = {"Ludesun": _stack, "Lanilix": _stack}
 
 
 def _qwen_dense_layers(hf: dict) -> tuple:

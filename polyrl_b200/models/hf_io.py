@@ -177,9 +177,9 @@ def _vision_tensors(cfg: ModelConfig, ck: HFCheckpoint) -> dict[str, torch.Tenso
 def load_state_dict(cfg: ModelConfig, path: str | Path) -> dict[str, torch.Tensor]:
     ck = HFCheckpoint(path)
     if cfg.family == "hybrid":
-        from .hybrid import ludesun_state_dict
+        from .stacks import stack_state_dict
 
-        return ludesun_state_dict(cfg, ck.get)
+        return stack_state_dict(cfg, ck.get)
     embed, head = _embed_head(cfg, ck)
     out = {**embed, **head}
     if cfg.vision is not None:
@@ -237,9 +237,9 @@ def hf_config_dict(cfg: ModelConfig) -> dict:
 
 def _lm_config_dict(cfg: ModelConfig) -> dict:
     if cfg.family == "hybrid":
-        from .hybrid import ludesun_config_dict
+        from .stacks import stack_config_dict
 
-        return ludesun_config_dict(cfg)
+        return stack_config_dict(cfg)
     if cfg.family == "gpt2":
         return {"model_type": "gpt2", "architectures": ["GPT2LMHeadModel"], "vocab_size": cfg.vocab_size, "n_embd": cfg.hidden_size,
                 "n_inner": cfg.intermediate_size, "n_layer": cfg.num_layers, "n_head": cfg.num_heads, "n_positions": cfg.max_position_embeddings,

@@ -1,14 +1,20 @@
 """Mixer stacks: decoder-only models whose layers each choose their own sequence mixer, served by the rollout engine.
 
-A layer is  x <- x + norm1(mixer(x)),  x <- x + norm2(ff(x))  — RMS norms on the sublayer outputs only, fp32 residual stream.
-Mixers (``LAYER_KINDS``): ``ssd`` (Mamba-2 state-space duality: causal convolution, scalar-decay recurrence, gate before a grouped
-norm), ``mlstm`` (xLSTM matrix memory with exponential gates) and ``latent`` (multi-head latent attention with query bottleneck,
-rotary key part and a softmax sink).  A layer may reuse the weights of an earlier one (``weights_of``) while keeping a cache or
-state of its own.
+A layer is  x <- x + norm1(mixer(pre1(x))),  x <- x + norm2(ff(pre2(x)))  over an fp32 residual stream: RMS norms on the sublayer outputs
+and, with ``ModelConfig.sandwich_norm``, on their inputs too; ``norm_offset`` is added to the stored weights of these norms and of the
+final one.  Mixers (``LAYER_KINDS``):
+  ``ssd``     Mamba-2 state-space duality: causal convolution, scalar-decay recurrence, gate before a grouped norm
+  ``mlstm``   xLSTM matrix memory with exponential gates
+  ``delta``   gated delta rule: short convolutions, unit queries and keys, one decay per head, gated norm per head
+  ``latent``  multi-head latent attention with query bottleneck, rotary key part and a softmax sink
+  ``window``  grouped-query attention in a sliding window with kept first tokens; queries and keys are normed over the whole projection
+              and partly rotated in neighbouring pairs, the values are the keys as projected
+Feed-forwards (``act``): ``gelu`` or ``clamped_glu``.  A layer may reuse the weights of an earlier one (``weights_of``) while keeping a
+cache or state of its own.
 
 ``ModelConfig.layers`` holds one plain dict per layer: {"kind", "sizes", "ff" (0: no feed-forward), "weights_of" (own index when the
-layer owns its weights)}.  ``ludesun_config`` reads the Ludesun ``config.json``; another design built from the same mixers needs only
-another reader and name map.
+layer owns its weights)} and what its feed-forward needs ("act", "limit", "alpha").  ``stacks.py`` reads the designs' config.json and
+checkpoint names; another design built from the same mixers needs only another reader and name map.
 
 Everything is one function of a packed step (ops/mixers.py ``SpanBatch``): prompts, portions of prompts and decoded tokens take the
 same path, and the kernels pick chunked or token-by-token work by span length.
@@ -20,9 +26,10 @@ import torch.nn.functional as F
 
 from .. import ops
 from ..ops import mixers as M
+from ..ops import reference as ref
 from .config import ModelConfig
 
-LAYER_KINDS = ("ssd", "mlstm", "latent")
+LAYER_KINDS = ("ssd", "mlstm", "delta", "latent", "window")
 
 
 def _pad8(n: int) -> int:
@@ -58,6 +65,15 @@ def validate(cfg: ModelConfig) -> None:
             raise ValueError(f"layer {i}: mlstm sizes")
         if kind == "latent" and (m["rot_dim"] % 2 or m["rot_dim"] > 512 or m["kv_rank"] > 1024):
             raise ValueError(f"layer {i}: latent sizes")
+        if kind in ("delta", "window") and m["heads"] % m["kv_heads"]:
+            raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
+        if kind == "delta" and (m["dim"] > 512 or m["conv"] < 1):
+            raise ValueError(f"layer {i}: delta sizes")
+        if kind == "window" and (m["vdim"] != m["dim"] or m["rot_dim"] % 2 or not 0 <= m["rot_dim"] <= min(512, m["dim"]) or m["dim"] > 1024 or m["window"] < 1
+                                 or m["keep_first"] < 0):
+            raise ValueError(f"layer {i}: window sizes (values are keys: vdim equals dim)")
+        if lay["ff"] and lay.get("act", "gelu") not in ("gelu", "clamped_glu"):
+            raise ValueError(f"layer {i}: unknown feed-forward {lay['act']!r}")
 
 
 # --------------------------------------------------------------------------------------------
@@ -66,19 +82,29 @@ def validate(cfg: ModelConfig) -> None:
 def layer_param_specs(cfg: ModelConfig, i: int) -> list[tuple[str, tuple[int, ...]]]:
     lay, w = cfg.layers[i], cfg.hidden_size
     m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
-    out: list[tuple[str, tuple[int, ...]]] = [("norm1", (w,))]
+    out: list[tuple[str, tuple[int, ...]]] = ([("pre1", (w,))] if cfg.sandwich_norm else []) + [("norm1", (w,))]
     if lay["kind"] == "ssd":            # one projection [gate | x | B | C]; the step sizes keep their own fp32-accumulated one
         ch = h * v + 2 * m["groups"] * m["state"]
         out += [("w_in", (h * v + ch, w)), ("w_dt", (h, w)), ("conv_w", (ch, m["conv"])), ("conv_b", (ch,)), ("dt_bias", (h,)), ("a_log", (h,)),
                 ("d_skip", (h,)), ("gn", (h * v,)), ("wo", (w, h * v))]
     elif lay["kind"] == "mlstm":        # [q | k | v | output gate] and [input gate | forget gate]
         out += [("w_in", (2 * h * m["dim"] + 2 * h * v, w)), ("w_if", (2 * h, w)), ("b_if", (2 * h,)), ("gn", (h * v,)), ("wo", (w, h * v))]
+    elif lay["kind"] == "delta":        # [q | k | v | output gate], [decay | write strength]; the convolution runs over [q | k | v]
+        qk = m["kv_heads"] * m["dim"]
+        out += [("w_in", (2 * qk + 2 * h * v, w)), ("w_ab", (2 * h, w)), ("conv_w", (2 * qk + h * v, m["conv"])), ("dt_bias", (h,)), ("a_log", (h,)),
+                ("gn", (v,)), ("wo", (w, h * v))]
+    elif lay["kind"] == "window":       # [q | k]
+        hd, gd = h * m["dim"], m["kv_heads"] * m["dim"]
+        out += [("wqk", (hd + gd, w)), ("q_norm", (hd,)), ("k_norm", (gd,)), ("wo", (w, hd))]
     else:                               # [query latent | key-value latent | shared rotary key]
         r, qr, d, rd = m["kv_rank"], m["q_rank"], m["dim"], m["rot_dim"]
         out += [("wa", (qr + r + rd, w)), ("q_ln", (qr,)), ("kv_ln", (r,)), ("wq_up", (h * (d + rd), qr)), ("wk_up", (h * d, r)), ("wv_up", (h * v, r)),
                 ("sink", (h,)), ("wo", (w, h * v))]
     if lay["ff"]:
-        out += [("norm2", (w,)), ("wup", (lay["ff"], w)), ("wdown", (w, lay["ff"]))]
+        f = lay["ff"]
+        out += ([("pre2", (w,))] if cfg.sandwich_norm else []) + [("norm2", (w,))]
+        # gate and up rows: interleaved in blocks of 128 (as the llama family's) where ff allows it, else one after the other
+        out += [("wgu", (2 * f, w)) if lay.get("act") == "clamped_glu" else ("wup", (f, w)), ("wdown", (w, f))]
     return out
 
 
@@ -97,7 +123,9 @@ def num_params(cfg: ModelConfig) -> int:
 def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) -> bool:
     """Random init of the tensors the generic rules do not cover; False when they do."""
     base = name.split(".")[-1]
-    if base in ("norm1", "norm2", "gn", "q_ln", "kv_ln", "d_skip"):
+    if base in ("pre1", "norm1", "pre2", "norm2", "norm_w"):
+        t.fill_(1.0 - cfg.norm_offset)
+    elif base in ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "d_skip"):
         t.fill_(1.0)
     elif base in ("conv_b", "sink"):
         t.zero_()
@@ -110,7 +138,7 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
         t[t.numel() // 2:] = 3.0
     elif base == "conv_w":
         t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
-    elif base in ("w_in", "w_dt", "w_if", "wa", "wq_up", "wk_up", "wv_up", "wo", "wup", "wdown"):
+    elif base in ("w_in", "w_dt", "w_if", "wa", "wq_up", "wk_up", "wv_up", "wo", "wup", "wdown", "w_ab", "wqk", "wgu"):
         t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
     else:
         return False
@@ -120,7 +148,18 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
 # --------------------------------------------------------------------------------------------
 # run-time weights
 # --------------------------------------------------------------------------------------------
-_VECTORS = ("norm1", "norm2", "gn", "q_ln", "kv_ln", "conv_b", "dt_bias", "a_log", "d_skip", "b_if", "sink")
+_STREAM_NORMS = ("pre1", "norm1", "pre2", "norm2")               # of the residual stream: ``norm_offset`` applies
+_VECTORS = ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "conv_b", "dt_bias", "a_log", "d_skip", "b_if", "sink")
+
+
+def packs(m: dict, dtype: torch.dtype, is_cuda: bool) -> bool:
+    """Long spans of this ``window`` layer run on the packed tcgen05 attention."""
+    return is_cuda and dtype == torch.bfloat16 and m["dim"] <= 128
+
+
+def cache_width(m: dict, dtype: torch.dtype) -> int:
+    """Width of a cached key of a ``window`` layer: what the bf16 kernels take (64 or 128, zeros behind the key), else its own."""
+    return m["dim"] if dtype != torch.bfloat16 or m["dim"] > 128 else (64 if m["dim"] <= 64 else 128)
 
 
 def query_width(m: dict, dtype: torch.dtype, is_cuda: bool) -> int:
@@ -149,15 +188,26 @@ def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: di
     is_cuda = w["norm1"].is_cuda
     out: dict[str, torch.Tensor] = {}
     for k, t in w.items():
-        if k in _VECTORS:
+        if k in _STREAM_NORMS:
+            out[k] = (t.float() + cfg.norm_offset).contiguous() if cfg.norm_offset else t.float().contiguous()
+        elif k == "gn" and t.numel() < h * m["vdim"]:             # one weight for all heads
+            out[k] = t.float().repeat(h)
+        elif k in _VECTORS:
             out[k] = t.float().contiguous()
         elif k == "conv_w":
             out[k] = t.float().t().contiguous()                     # [taps, channels]
         elif k not in ("wq_up", "wk_up", "wv_up"):
             t = t if t.dtype == dtype else t.to(dtype)
-            if k == "w_in" and is_cuda and t.shape[0] % 8:
+            if k in ("w_in", "wqk") and is_cuda and t.shape[0] % 8:
                 t = F.pad(t, (0, 0, 0, _pad8(t.shape[0]) - t.shape[0]))
             out[k] = t.contiguous()
+    if lay["kind"] == "window":
+        out["freq"] = M.rope_frequencies(m["rot_dim"], m["rot_base"], w["norm1"].device)
+    if "wgu" in out and is_cuda and dtype == torch.bfloat16 and lay["ff"] % 128:
+        # the fused gate / up kernel wants 128-row blocks: zero rows behind the last ones
+        f, pad = lay["ff"], -lay["ff"] % 128
+        out["wgu"] = ref.interleave_gate_up(*(F.pad(t, (0, 0, 0, pad)) for t in (out["wgu"][:f], out["wgu"][f:])))
+        out["wdown"] = F.pad(out["wdown"], (0, pad))
     if lay["kind"] == "latent":
         d, rd, v, r = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
         dq = query_width(m, dtype, is_cuda)
@@ -192,8 +242,10 @@ def prepare(cfg: ModelConfig, layer_w: list[dict], dtype: torch.dtype, old: list
     return [done[owner(cfg, i)] for i in range(cfg.num_layers)]
 
 
-def prepare_head(head_w: dict, dtype: torch.dtype, old: dict | None = None) -> dict:
+def prepare_head(cfg: ModelConfig, head_w: dict, dtype: torch.dtype, old: dict | None = None) -> dict:
     norm = head_w["norm_w"].float().contiguous()
+    if cfg.norm_offset:
+        norm = norm + cfg.norm_offset
     if old is not None and norm.data_ptr() != head_w["norm_w"].data_ptr():
         norm = old["norm_w"].copy_(norm)
     return {"norm_w": norm, "lm_head": head_w["lm_head"].to(dtype)}
@@ -210,11 +262,20 @@ def cache_bytes(cfg: ModelConfig, dtype: torch.dtype) -> tuple[int, int]:
         m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
         if lay["kind"] == "latent":
             tok += (m["kv_rank"] + m["rot_dim"]) * es
+        elif lay["kind"] == "window":
+            tok += 2 * m["kv_heads"] * cache_width(m, dtype) * es
+        elif lay["kind"] == "delta":
+            slot += 4 * h * v * m["dim"] + es * (m["conv"] - 1) * (h * v + 2 * m["kv_heads"] * m["dim"])
         elif lay["kind"] == "ssd":
             slot += 4 * h * v * m["state"] + es * (m["conv"] - 1) * (h * v + 2 * m["groups"] * m["state"])
         else:
             slot += 4 * h * (m["dim"] * v + m["dim"] + 1)
     return tok, slot
+
+
+def key_views(cfg: ModelConfig) -> list[tuple[int, int]]:
+    """The distinct (window, kept first tokens) of the stack's attention layers; (0, 0) sees every key."""
+    return sorted({(lay["sizes"].get("window", 0), lay["sizes"].get("keep_first", 0)) for lay in cfg.layers if lay["kind"] in ("latent", "window")})
 
 
 def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device, dtype: torch.dtype) -> dict[str, torch.Tensor]:
@@ -223,7 +284,13 @@ def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device
     m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
     if lay["kind"] == "latent":
         return {"pool": torch.zeros(num_blocks, 1, M.PAGE, m["kv_rank"] + m["rot_dim"], device=device, dtype=dtype)}
+    if lay["kind"] == "window":
+        shape = (num_blocks, m["kv_heads"], M.PAGE, cache_width(m, dtype))
+        return {n: torch.zeros(shape, device=device, dtype=dtype) for n in ("k_pool", "v_pool")}
     f32 = dict(device=device, dtype=torch.float32)
+    if lay["kind"] == "delta":
+        ch = 2 * m["kv_heads"] * m["dim"] + h * v
+        return {"S": torch.zeros(num_slots, h, m["dim"], v, **f32), "conv": torch.zeros(num_slots, m["conv"] - 1, ch, device=device, dtype=dtype)}
     if lay["kind"] == "ssd":
         ch = h * v + 2 * m["groups"] * m["state"]
         return {"S": torch.zeros(num_slots, h, m["state"], v, **f32), "conv": torch.zeros(num_slots, m["conv"] - 1, ch, device=device, dtype=dtype)}
@@ -233,7 +300,7 @@ def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device
 def copy_cache(cache: dict, src_pages: torch.Tensor, dst_pages: torch.Tensor, src_slots: torch.Tensor, dst_slots: torch.Tensor) -> None:
     """Duplicate pages / state slots of one layer (the members of an n-sample group continue from their donor's prompt)."""
     for k, t in cache.items():
-        src, dst = (src_pages, dst_pages) if k == "pool" else (src_slots, dst_slots)
+        src, dst = (src_pages, dst_pages) if k.endswith("pool") else (src_slots, dst_slots)
         if src.numel():
             t.index_copy_(0, dst, t.index_select(0, src))
 
@@ -249,7 +316,7 @@ def _ssd(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.
     xbc = M.conv_silu(xbc, w["conv_w"], w["conv_b"], cache["conv"], b)
     y = M.scan(M.SSD, xbc[:, inner + gn:], xbc[:, inner:inner + gn], xbc[:, :inner],
                M.Gates(dt, b0=w["dt_bias"], a_log=w["a_log"], d_skip=w["d_skip"]), 1.0, cache, b)
-    return M.gated_norm(y, z, w["gn"], m["norm_groups"], cfg.rms_norm_eps, True)
+    return M.gated_norm(y, z, w["gn"], m["norm_groups"], cfg.rms_norm_eps, M.SILU_FIRST)
 
 
 def _mlstm(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
@@ -259,7 +326,7 @@ def _mlstm(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: 
     g = M.linear_f32(h, w["w_if"])
     o = M.scan(M.MLSTM, p[:, :hd], p[:, hd:2 * hd], p[:, 2 * hd:2 * hd + hv],
                M.Gates(g[:, :nh], g[:, nh:], w["b_if"][:nh], w["b_if"][nh:], cap=float(m["gate_cap"])), m["dim"] ** -0.5, cache, b)
-    return M.gated_norm(o, p[:, 2 * hd + hv:2 * hd + 2 * hv], w["gn"], nh, cfg.rms_norm_eps, False)
+    return M.gated_norm(o, p[:, 2 * hd + hv:2 * hd + 2 * hv], w["gn"], nh, cfg.rms_norm_eps, M.SIGMOID_LAST)
 
 
 def _latent(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
@@ -274,7 +341,8 @@ def _latent(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b:
         if b.gather is None:
             src, cu_k = entry[:tl], b.cu[:b.n_long + 1]
         else:
-            src, cu_k = pool.view(-1, r + rd).index_select(0, b.gather[0]), b.gather[1]
+            rows, cu_k = b.gather[0, 0]
+            src = pool.view(-1, r + rd).index_select(0, rows)
         kv = ops.linear(src, w["w_expand"])
         dq = q.shape[-1]
         k, vv = kv[:, :nh * dq].view(-1, nh, dq), kv[:, nh * dq:].view(-1, nh, 128)
@@ -290,123 +358,61 @@ def _latent(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b:
     return out[0] if len(out) == 1 else torch.cat(out)
 
 
-_MIXERS = {"ssd": _ssd, "mlstm": _mlstm, "latent": _latent}
+def _delta(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
+    nh, qk = m["heads"], m["kv_heads"] * m["dim"]
+    hv = nh * m["vdim"]
+    p = ops.linear(h, w["w_in"])
+    ab = M.linear_f32(h, w["w_ab"])
+    c = M.conv_silu(p[:, :2 * qk + hv], w["conv_w"], None, cache["conv"], b)
+    o = M.scan(M.DELTA, c[:, :qk], c[:, qk:2 * qk], c[:, 2 * qk:], M.Gates(ab[:, :nh], ab[:, nh:], b0=w["dt_bias"], a_log=w["a_log"]), m["dim"] ** -0.5,
+               cache, b)
+    return M.gated_norm(o, p[:, 2 * qk + hv:2 * qk + 2 * hv], w["gn"], nh, cfg.rms_norm_eps, M.SILU_LAST)
 
 
-def embed_forward(cfg: ModelConfig, w: dict, ids: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
-    return M.embed(ids, w["embed"])
+def _window(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
+    nh, d, t = m["heads"], m["dim"], b.tokens
+    view = (m["window"], m["keep_first"])
+    scale, kp, vp = float(m["scale"]), cache["k_pool"], cache["v_pool"]
+    tl = b.t_long if packs(m, h.dtype, h.is_cuda) else 0            # tokens served by the packed kernel
+    q, kv = M.qk_prep(ops.linear(h, w["wqk"]), nh, d, w["q_norm"], w["k_norm"], w["freq"], kp, vp, b, cfg.rms_norm_eps, tl > 0 and b.gather is None)
+    out = []
+    if tl:
+        if b.gather is None:
+            k, v, cu_k = kv[0][:tl], kv[1][:tl], b.cu[:b.n_long + 1]
+        else:
+            rows, cu_k = b.gather[view]
+            k, v = M.gather_keys(kp, vp, rows)
+        out.append(M.window_attention_varlen(q[:tl], k, v, b.cu[:b.n_long + 1], cu_k, scale, *view))
+    if tl < t:
+        lo = b.n_long if tl else 0
+        seq_of = None if b.seq_of is None or tl else b.seq_of[tl:]
+        out.append(M.window_attention(q[tl:], kp, vp, b.table[lo:], seq_of, b.kv_len[tl:], scale, *view, b.max_len))
+    o = out[0] if len(out) == 1 else torch.cat(out)
+    return o[..., :d].reshape(t, nh * d)
+
+
+_MIXERS = {"ssd": _ssd, "mlstm": _mlstm, "delta": _delta, "latent": _latent, "window": _window}
 
 
 def layer_step(cfg: ModelConfig, i: int, w: dict, x: torch.Tensor, h: torch.Tensor, cache: dict, b: M.SpanBatch,
                w_next: torch.Tensor | None = None) -> torch.Tensor:
-    """Layer ``i`` on one packed step.  x: fp32 residual stream, updated in place; h: x in the activation dtype (the sublayers read x
-    itself).  Returns the next h — or the final norm of x when its weight is given as ``w_next``."""
+    """Layer ``i`` on one packed step.  x: fp32 residual stream, updated in place; h: what its mixer reads, in the activation dtype (x
+    itself, or its norm ``pre1``).  Returns x in that dtype — or the norm of x with the weight ``w_next``, which is the next layer's
+    ``pre1`` or the model's final norm."""
     lay, eps = cfg.layers[i], cfg.rms_norm_eps
     y = ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h, cache, b), w["wo"])
     if not lay["ff"]:
         return M.norm_add_(y, x, w["norm1"], eps, w_next)
-    h = M.norm_add_(y, x, w["norm1"], eps)
-    y = ops.linear(M.linear_gelu(h, w["wup"]), w["wdown"])
-    return M.norm_add_(y, x, w["norm2"], eps, w_next)
+    h = M.norm_add_(y, x, w["norm1"], eps, w.get("pre2"))
+    a = M.linear_clamped_glu(h, w["wgu"], lay["limit"], lay["alpha"]) if lay.get("act") == "clamped_glu" else M.linear_gelu(h, w["wup"])
+    return M.norm_add_(ops.linear(a, w["wdown"]), x, w["norm2"], eps, w_next)
 
 
-# --------------------------------------------------------------------------------------------
-# Ludesun: configuration and checkpoint names
-# --------------------------------------------------------------------------------------------
-_LUDESUN_KIND = {"mamba2": "ssd", "mlstm": "mlstm", "latent_attention": "latent"}
-_LUDESUN_SIZES = {"ssd": ("heads", "vdim", "state", "groups", "conv", "norm_groups"), "mlstm": ("heads", "dim", "vdim", "gate_cap"),
-                  "latent": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "scale")}
-
-
-def ludesun_config(hf: dict) -> ModelConfig:
-    """``config.json`` of a Ludesun model: vocab, width, norm.eps and one entry of ``layers`` per layer."""
-    layers = []
-    for i, e in enumerate(hf["layers"]):
-        if e["type"] not in _LUDESUN_KIND:
-            raise ValueError(f"Ludesun layer {i}: unknown mixer type {e['type']!r}")
-        kind = _LUDESUN_KIND[e["type"]]
-        sizes = {k: e["mixer"][k] for k in _LUDESUN_SIZES[kind]}
-        if kind == "latent":
-            if e["mixer"]["rot"]["dims"] != sizes["rot_dim"]:
-                raise ValueError(f"Ludesun layer {i}: rot.dims and rot_dim differ")
-            sizes["rot_base"] = float(e["mixer"]["rot"]["base"])
-        mlp = e.get("mlp")
-        if mlp and mlp.get("kind", "dense") != "dense":
-            raise ValueError(f"Ludesun layer {i}: feed-forward kind {mlp['kind']!r}")
-        layers.append({"kind": kind, "sizes": sizes, "ff": int(mlp["ff"]) if mlp else 0, "weights_of": int(e.get("weights_of", i))})
-    return ModelConfig(family="hybrid", vocab_size=hf["vocab"], hidden_size=hf["width"], num_layers=len(layers), layers=tuple(layers),
-                       intermediate_size=max([x["ff"] for x in layers] + [1]), num_heads=1, num_kv_heads=1, rms_norm_eps=float(hf["norm"]["eps"]),
-                       eos_token_id=-1, bos_token_id=-1, pad_token_id=0, hf_model_type="ludesun", name="ludesun")
-
-
-def ludesun_config_dict(cfg: ModelConfig) -> dict:
-    """Inverse of ``ludesun_config``."""
-    back = {v: k for k, v in _LUDESUN_KIND.items()}
-    layers = []
-    for i, lay in enumerate(cfg.layers):
-        mx = {k: lay["sizes"][k] for k in _LUDESUN_SIZES[lay["kind"]]}
-        if lay["kind"] == "latent":
-            mx["rot"] = {"dims": mx["rot_dim"], "base": lay["sizes"]["rot_base"]}
-        e = {"type": back[lay["kind"]], "mixer": mx, "mlp": {"kind": "dense", "ff": lay["ff"]} if lay["ff"] else None}
-        if lay["weights_of"] != i:
-            e["weights_of"] = lay["weights_of"]
-        layers.append(e)
-    return {"architecture": "Ludesun", "vocab": cfg.vocab_size, "width": cfg.hidden_size, "norm": {"eps": cfg.rms_norm_eps}, "layers": layers}
-
-
-def _ludesun_parts(kind: str, ff: int) -> list[tuple[str, list[str]]]:
-    """(our name, checkpoint names whose rows it stacks) of one layer; the SSD input projection is split separately."""
-    mix = {"ssd": [("conv_w", ["conv"]), ("conv_b", ["conv.b"]), ("dt_bias", ["dt_bias"]), ("a_log", ["A_log"]), ("d_skip", ["D"])],
-           "mlstm": [("w_in", ["q", "k", "v", "g"]), ("w_if", ["i", "f"]), ("b_if", ["i.b", "f.b"])],
-           "latent": [("wa", ["dq", "dkv"]), ("q_ln", ["dq.norm"]), ("kv_ln", ["dkv.norm"]), ("wq_up", ["uq"]), ("wk_up", ["uk"]), ("wv_up", ["uv"]),
-                      ("sink", ["sink"])]}[kind]
-    if kind != "latent":
-        mix = mix + [("gn", ["norm"])]
-    out = [(n, ["mix." + s for s in src]) for n, src in mix + [("wo", ["o"])]]
-    out.append(("norm1", ["norm1"]))
-    if ff:
-        out += [("norm2", ["norm2"]), ("wup", ["mlp.up"]), ("wdown", ["mlp.down"])]
-    return out
-
-
-def ludesun_layer(cfg: ModelConfig, i: int, get) -> dict[str, torch.Tensor]:
-    """Tensors of layer ``i`` (which owns its weights) in our names; ``get`` reads a checkpoint tensor by name."""
-    lay, p = cfg.layers[i], f"l{i}."
-    out = {n: (torch.cat([get(p + s) for s in src]) if len(src) > 1 else get(p + src[0])) for n, src in _ludesun_parts(lay["kind"], lay["ff"])}
-    if lay["kind"] == "ssd":
-        w, nh = get(p + "mix.in"), lay["sizes"]["heads"]
-        out["w_in"], out["w_dt"] = w[:-nh], w[-nh:]
-    return out
-
-
-def ludesun_state_dict(cfg: ModelConfig, get) -> dict[str, torch.Tensor]:
-    out = {"embed": get("embed"), "norm_w": get("final.norm"), "lm_head": get("head")}
-    for i in range(cfg.num_layers):
-        if owner(cfg, i) == i:
-            out.update({f"layers.{i}.{k}": t for k, t in ludesun_layer(cfg, i, get).items()})
-    return out
-
-
-def ludesun_export(cfg: ModelConfig, sd: dict) -> dict[str, torch.Tensor]:
-    """Our names -> checkpoint names (inverse of ``ludesun_state_dict``)."""
-    out = {"embed": sd["embed"], "final.norm": sd["norm_w"], "head": sd["lm_head"]}
-    for i, lay in enumerate(cfg.layers):
-        if owner(cfg, i) != i:
-            continue
-        p, q, m = f"l{i}.", f"layers.{i}.", lay["sizes"]
-        rows = {}
-        if lay["kind"] == "mlstm":
-            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
-            rows = {"mix.q": hd, "mix.k": hd, "mix.v": hv, "mix.g": hv, "mix.i": m["heads"], "mix.f": m["heads"], "mix.i.b": m["heads"], "mix.f.b": m["heads"]}
-        elif lay["kind"] == "latent":
-            rows = {"mix.dq": m["q_rank"], "mix.dkv": m["kv_rank"] + m["rot_dim"]}
-        for n, src in _ludesun_parts(lay["kind"], lay["ff"]):
-            t = sd[q + n]
-            if len(src) == 1:
-                out[p + src[0]] = t
-            else:
-                for s, piece in zip(src, t.split([rows[s] for s in src])):
-                    out[p + s] = piece.clone()
-        if lay["kind"] == "ssd":
-            out[p + "mix.in"] = torch.cat([sd[q + "w_in"], sd[q + "w_dt"]])
-    return out
+def forward(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids: torch.Tensor, caches: list[dict], b: M.SpanBatch,
+            final_norm: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """The stack on one packed step: (fp32 residual stream after the last layer, the same in the activation dtype — normed with
+    ``final_norm`` when that is given)."""
+    x, h = M.embed(ids, embed_w["embed"], layer_w[0].get("pre1"), cfg.rms_norm_eps)
+    for i, w in enumerate(layer_w):
+        h = layer_step(cfg, i, w, x, h, caches[i], b, layer_w[i + 1].get("pre1") if i + 1 < len(layer_w) else final_norm)
+    return x, h

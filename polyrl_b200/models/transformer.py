@@ -864,9 +864,9 @@ def _export_mlp(cfg: ModelConfig, sd: dict, out: dict, i: int, p: str, fused_gu:
 
 def export_hf_state_dict(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict[str, torch.Tensor]:
     if cfg.family == "hybrid":
-        from .hybrid import ludesun_export
+        from .stacks import stack_export
 
-        return ludesun_export(cfg, sd)
+        return stack_export(cfg, sd)
     if cfg.family == "gpt2":
         out = {"transformer.wte.weight": sd["embed"], "transformer.wpe.weight": sd["pos_embed"], "transformer.ln_f.weight": sd["norm_w"],
                "transformer.ln_f.bias": sd["norm_b"], "lm_head.weight": sd["embed"]}

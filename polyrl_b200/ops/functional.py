@@ -529,11 +529,14 @@ def _auto_splits(num_seqs: int, nkv: int, max_len: int) -> int:
 
 @torch.no_grad()
 def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, nq, nkv, d, sm_scale, splits: int = 0,
-                           max_len: int = 0, out=None):
+                           max_len: int = 0, out=None, window: int = 0, keep_first: int = 0):
+    """``window`` > 0: a sequence sees its last ``window`` keys and its first ``keep_first``; ``max_len`` bounds the keys seen."""
     if _is_kernel_tensor(q):
         if splits <= 0:
             splits = _auto_splits(q.shape[0], nkv, max_len if max_len > 0 else 1024)
-        return _C().paged_decode(q, k_cache, v_cache, block_table, seq_lens, nq, nkv, d, sm_scale, splits, out)
+        return _C().paged_decode(q, k_cache, v_cache, block_table, seq_lens, nq, nkv, d, sm_scale, splits, out, window, keep_first)
+    if window:
+        raise NotImplementedError("windowed paged attention on CPU: ops.mixers.window_attention")
     return ref.paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, nq, nkv, d, sm_scale)
 
 

@@ -12,6 +12,8 @@ from dataclasses import dataclass
 import torch
 import torch.nn.functional as F
 
+from .reference import split_gate_up
+
 PAGE = 16
 
 
@@ -29,8 +31,9 @@ class SpanBatch:
     t_long: int = 0
     max_long: int = 0                   # longest span
     max_len: int = 0                    # bound on kv_len
-    # keys of the long spans: (flat cache rows [Tk] int64, cu_k [n_long + 1] int32); None: no span has earlier tokens
-    gather: tuple | None = None
+    # keys of the long spans, per (window, kept first tokens) — (0, 0): all of them: (flat cache rows [Tk] int64, cu_k [n_long + 1]
+    # int32), kept first tokens ahead of the window's; None: no span has earlier tokens
+    gather: dict | None = None
 
     @property
     def spans(self) -> int:
@@ -74,11 +77,14 @@ def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
-def embed(ids: torch.Tensor, w: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
-    """(fp32 residual stream, the same in the activation dtype — one tensor when that is fp32)."""
+def embed(ids: torch.Tensor, w: torch.Tensor, w_norm: torch.Tensor | None = None, eps: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """(fp32 residual stream, the same in the activation dtype — one tensor when that is fp32); with ``w_norm`` the second is
+    rms(x) * w_norm."""
     if w.is_cuda:
-        return tuple(_C().mix_embed(ids, w))
+        return tuple(_C().mix_embed(ids, w, w_norm, eps))
     x = F.embedding(ids, w).float()
+    if w_norm is not None:
+        return x, (_rms(x, eps) * w_norm).to(w.dtype)
     return x, (x if w.dtype == torch.float32 else x.to(w.dtype))
 
 
@@ -99,15 +105,18 @@ def rms(x: torch.Tensor, w: torch.Tensor, eps: float, dtype: torch.dtype) -> tor
     return (_rms(x, eps) * w).to(dtype)
 
 
-def gated_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate_first: bool) -> torch.Tensor:
-    """Group RMS norm with a gate: rms(y * silu(z)) * w (``gate_first``) or rms(y) * w * sigmoid(z)."""
+SIGMOID_LAST, SILU_FIRST, SILU_LAST = 0, 1, 2
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate: int) -> torch.Tensor:
+    """Group RMS norm with a gate: rms(y) * w * sigmoid(z), rms(y * silu(z)) * w or rms(y) * w * silu(z)."""
     if y.is_cuda:
-        return _C().mix_gated_norm(y, z, w, groups, eps, gate_first)
+        return _C().mix_gated_norm(y, z, w, groups, eps, gate)
     yf, zf = y.float(), z.float()
-    if gate_first:
+    if gate == SILU_FIRST:
         yf = yf * F.silu(zf)
     n = _rms(yf.reshape(y.shape[0], groups, -1), eps).reshape(y.shape) * w
-    return (n if gate_first else n * torch.sigmoid(zf)).to(y.dtype)
+    return (n if gate == SILU_FIRST else n * (torch.sigmoid(zf) if gate == SIGMOID_LAST else F.silu(zf))).to(y.dtype)
 
 
 def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -128,10 +137,24 @@ def linear_gelu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return F.gelu(F.linear(x, w.to(x.dtype)), approximate="tanh")
 
 
+def linear_clamped_glu(x: torch.Tensor, wgu: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    """g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); ``wgu`` holds gate and up rows interleaved in
+    blocks of 128 when there are whole blocks, else one after the other.  Fused into the GEMM epilogue for bf16 rows."""
+    f = wgu.shape[0] // 2
+    if x.is_cuda and x.dtype == torch.bfloat16 and f % 128 == 0 and x.shape[1] % 8 == 0:
+        return _C().gemm_clamped_glu(x, wgu, limit, alpha)
+    gu = F.linear(x, wgu.to(x.dtype))
+    if x.is_cuda:
+        return _C().mix_clamped_glu(gu, 128 if f % 128 == 0 else f, limit, alpha)
+    g, u = split_gate_up(gu.float()) if f % 128 == 0 else gu.float().split(f, -1)
+    g = g.clamp(max=limit)
+    return (g * torch.sigmoid(alpha * g) * (u.clamp(-limit, limit) + 1)).to(x.dtype)
+
+
 # --------------------------------------------------------------------------------------------
 # causal convolution with carried taps
 # --------------------------------------------------------------------------------------------
-def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, b: SpanBatch) -> torch.Tensor:
+def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor, b: SpanBatch) -> torch.Tensor:
     """silu(causal conv) per channel; w [taps, ch] (last row: the current token), state [slots, taps - 1, ch]."""
     if x.is_cuda:
         return _C().mix_conv(x, w, bias, state, b.cu, b.start, b.slot, b.seq_of)
@@ -142,7 +165,7 @@ def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, state: torch
         lo, hi = cu[s], cu[s + 1]
         old = state[b.slot[s]] if int(b.start[s]) else torch.zeros_like(state[0])
         full = torch.cat([old, x[lo:hi]]).float()
-        y = bias + sum(w[j] * full[j:j + hi - lo] for j in range(taps))
+        y = (0 if bias is None else bias) + sum(w[j] * full[j:j + hi - lo] for j in range(taps))
         out[lo:hi] = F.silu(y).to(x.dtype)
         state[b.slot[s]] = full[full.shape[0] - (taps - 1):].to(state.dtype)
     return out
@@ -151,7 +174,7 @@ def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, state: torch
 # --------------------------------------------------------------------------------------------
 # gated linear recurrences
 # --------------------------------------------------------------------------------------------
-SSD, MLSTM = 0, 1
+SSD, MLSTM, DELTA = 0, 1, 2
 
 
 @dataclass
@@ -174,7 +197,8 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
     """S_t = keep_t S_(t-1) + add_t k_t v_t^T,  y_t = S_t^T (qscale q_t), over the spans of ``b``.
 
     ``SSD``: add = softplus(g0 + b0), keep = exp(-exp(a_log) add), y += d_skip v.  ``MLSTM``: capped log gates with a running
-    maximum and a normaliser.  q / k [T, groups * N] (consecutive heads share a group), v [T, H * V], cache["S"] [slots, H, N, V]
+    maximum and a normaliser.  ``DELTA``: the gated delta rule on unit vectors k' = k / |k|, q' = q / |q| (1e-6 under the root): keep =
+    exp(-exp(a_log) softplus(g0 + b0)) and the write is k' u^T with u = sigmoid(g1) (v - keep S^T k').  q / k [T, groups * N] (consecutive heads share a group), v [T, H * V], cache["S"] [slots, H, N, V]
     (+ "n" [slots, H, N], "m" [slots, H])."""
     if not v.is_cuda:
         return _scan_cpu(mode, q, k, v, gates, qscale, cache, b)
@@ -186,8 +210,12 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
         _C().mix_scan_(mode, q, k, v, gates.g0, gates.g1, gates.b0, gates.b1, gates.a_log, gates.d_skip, qscale, gates.cap, S, cache.get("n"),
                        cache.get("m"), b.cu[lo:hi + 1], b.start[lo:hi], b.slot[lo:hi], ctr, form, out)
 
-    chunk = v.dtype == torch.bfloat16 and b.max_long >= CHUNK_MIN and _C().mix_chunk_supported(N)
-    if b.n_long:
+    chunk = v.dtype == torch.bfloat16 and b.max_long >= CHUNK_MIN
+    if b.n_long and mode == DELTA and chunk and _C().mix_delta_chunk_ok(q, k, v, S):
+        _C().mix_delta_chunk_(q, k, v, gates.g0, gates.g1, gates.b0, gates.a_log, qscale, S, b.cu[:b.n_long + 1], b.start[:b.n_long],
+                              b.slot[:b.n_long], ctr, out)
+    elif b.n_long:
+        chunk = chunk and mode != DELTA and _C().mix_chunk_supported(N)
         run(0, b.n_long, (3 if b.max_long >= TC_MIN else 2) if chunk else 0)
     if b.n_long < b.spans:
         run(b.n_long, b.spans, 1)
@@ -207,10 +235,13 @@ def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
             n = torch.zeros_like(cache["n"][0]) if fresh else cache["n"][sl].clone()
             m = torch.zeros_like(cache["m"][0]) if fresh else cache["m"][sl].clone()
         for t in range(cu[s], cu[s + 1]):
-            qt = q[t].float().reshape(-1, N).repeat_interleave(rep, 0) * qscale
+            qt = q[t].float().reshape(-1, N).repeat_interleave(rep, 0)
             kt = k[t].float().reshape(-1, N).repeat_interleave(rep, 0)
+            if mode == DELTA:
+                qt, kt = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6) for x in (qt, kt))
+            qt = qt * qscale
             vt = v[t].float().reshape(H, V)
-            if mode == SSD:
+            if mode in (SSD, DELTA):
                 add = F.softplus(g.g0[t] + g.b0, threshold=1e9)
                 keep = torch.exp(-torch.exp(g.a_log) * add)
             else:
@@ -219,11 +250,16 @@ def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
                 m2 = torch.maximum(gf + m, gi)
                 keep, add, m = torch.exp(gf + m - m2), torch.exp(gi - m2), m2
                 n = keep[:, None] * n + add[:, None] * kt
-            S = keep[:, None, None] * S + (add[:, None] * kt)[:, :, None] * vt[:, None, :]
+            if mode == DELTA:
+                S = keep[:, None, None] * S
+                u = torch.sigmoid(g.g1[t])[:, None] * (vt - torch.einsum("hnv,hn->hv", S, kt))
+                S = S + kt[:, :, None] * u[:, None, :]
+            else:
+                S = keep[:, None, None] * S + (add[:, None] * kt)[:, :, None] * vt[:, None, :]
             y = torch.einsum("hnv,hn->hv", S, qt)
             if mode == SSD:
                 y = y + g.d_skip[:, None] * vt
-            else:
+            elif mode == MLSTM:
                 y = y / (torch.maximum((n * qt).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None]
             out[t] = y.reshape(-1).to(v.dtype)
         S_pool[sl] = S
@@ -307,3 +343,75 @@ def sink_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_
     """Causal (bottom-right aligned) attention of packed spans on expanded keys, with a sink: the tcgen05 kernel, query / key width
     128 or 192, value width 128, bf16."""
     return _C().attn_fwd(q, k, v, cu_q, cu_k, scale, True, False, None, sink)[0]
+
+
+# --------------------------------------------------------------------------------------------
+# grouped-query attention in a sliding window with kept first tokens
+# --------------------------------------------------------------------------------------------
+def _rotate_pairs(x: torch.Tensor, freq: torch.Tensor, pos: torch.Tensor) -> torch.Tensor:
+    """x [T, heads, d]: neighbours (2 i, 2 i + 1) of the first entries turned by pos * freq[i]."""
+    a = torch.outer(pos.double(), freq)
+    c, s = a.cos().float()[:, None], a.sin().float()[:, None]
+    y, n = x.clone(), 2 * freq.numel()
+    u, v = x[..., 0:n:2], x[..., 1:n:2]
+    y[..., 0:n:2], y[..., 1:n:2] = u * c - v * s, v * c + u * s
+    return y
+
+
+def qk_prep(p: torch.Tensor, heads: int, dim: int, wq: torch.Tensor, wk: torch.Tensor, freq: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
+            b: SpanBatch, eps: float, want_kv: bool) -> tuple[torch.Tensor, tuple | None]:
+    """Rows [queries | keys] as projected -> queries [T, heads, width], RMS-normed over the whole row and rotated; the keys treated alike go to
+    ``k_pool`` and, as projected, to ``v_pool`` ([pages, key heads, PAGE, width], zeros beyond ``dim``).  Packed keys and values [T, key heads,
+    width] are returned too when asked for."""
+    g, width = k_pool.shape[1], k_pool.shape[3]
+    if p.is_cuda:
+        q, k, v = _C().mix_qk_prep(p, heads, dim, wq, wk, freq, b.pos, b.kv_slot, k_pool, v_pool, eps, want_kv)
+        return q, ((k, v) if want_kv else None)
+    t = p.shape[0]
+    raw = p[:, heads * dim:(heads + g) * dim]
+    q = _rotate_pairs((_rms(p[:, :heads * dim].float(), eps) * wq).reshape(t, heads, dim), freq, b.pos)
+    k = _rotate_pairs((_rms(raw.float(), eps) * wk).reshape(t, g, dim), freq, b.pos)
+    q, k, v = (F.pad(x.to(p.dtype), (0, width - dim)) for x in (q, k, raw.reshape(t, g, dim)))
+    page, off = b.kv_slot // PAGE, b.kv_slot % PAGE
+    k_pool[page, :, off], v_pool[page, :, off] = k, v
+    return q, ((k, v) if want_kv else None)
+
+
+def gather_keys(k_pool: torch.Tensor, v_pool: torch.Tensor, rows: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """Keys and values of flat cache rows, [rows, key heads, width] each."""
+    if k_pool.is_cuda:
+        return tuple(_C().mix_gather_keys(k_pool, v_pool, rows))
+    return k_pool[rows // PAGE, :, rows % PAGE], v_pool[rows // PAGE, :, rows % PAGE]
+
+
+def window_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, table: torch.Tensor, seq_of: torch.Tensor | None, kv_len: torch.Tensor,
+                     scale: float, window: int, keep_first: int, max_len: int) -> torch.Tensor:
+    """Paged form, one query row [heads, width] per entry of ``kv_len``: the row's own token is its last key; it sees the last ``window``
+    keys and the first ``keep_first``."""
+    rows, h, width = q.shape
+    g = k_pool.shape[1]
+    if q.is_cuda:
+        if q.dtype == torch.bfloat16 and width in (64, 128) and h // g <= 16 and seq_of is None:
+            from .functional import paged_decode_attention
+
+            return paged_decode_attention(q.reshape(rows, h * width), k_pool, v_pool, table, kv_len, h, g, width, scale,
+                                          max_len=min(max_len, window + keep_first + 2 * PAGE), window=window, keep_first=keep_first).view(rows, h, width)
+        return _C().mix_window_attention(q, k_pool, v_pool, table, seq_of, kv_len, scale, window, keep_first)
+    out = torch.zeros_like(q)
+    for i in range(rows):
+        n = int(kv_len[i])
+        if n == 0:
+            continue
+        pages = table[int(seq_of[i]) if seq_of is not None else i, : (n + PAGE - 1) // PAGE].long()
+        j = torch.arange(n)
+        j = j[(j >= n - window) | (j < keep_first)]
+        k, v = (x[pages[j // PAGE], :, j % PAGE].float().repeat_interleave(h // g, 1) for x in (k_pool, v_pool))
+        s = torch.softmax(torch.einsum("hd,jhd->hj", q[i].float(), k) * scale, -1)
+        out[i] = torch.einsum("hj,jhd->hd", s, v).to(q.dtype)
+    return out
+
+
+def window_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.Tensor, cu_k: torch.Tensor, scale: float, window: int,
+                            keep_first: int) -> torch.Tensor:
+    """Packed spans, bottom-right aligned: the tcgen05 kernel, width 64 or 128, bf16."""
+    return _C().attn_fwd(q, k, v, cu_q, cu_k, scale, True, False, None, None, window, keep_first)[0]

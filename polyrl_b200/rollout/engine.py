@@ -359,7 +359,7 @@ class RolloutEngine:
             from ..models import hybrid
 
             layer_w = hybrid.prepare(self.cfg, layer_w, self.dtype, self.layer_w)
-            head_w = hybrid.prepare_head(head_w, self.dtype, self.head_w)
+            head_w = hybrid.prepare_head(self.cfg, head_w, self.dtype, self.head_w)
             if embed_w["embed"].dtype != self.dtype:
                 embed_w = {"embed": embed_w["embed"].to(self.dtype)}
         self.embed_w, self.layer_w, self.head_w = embed_w, layer_w, head_w
@@ -874,19 +874,20 @@ class RolloutEngine:
             at = torch.arange(PAGE)
             rows = [(torch.tensor(r.blocks[: (e + PAGE - 1) // PAGE]).unsqueeze(1) * PAGE + at).reshape(-1)[:e]
                     for r, (_, e) in zip(reqs[:n_long], spans[:n_long])]
-            cu_k = torch.zeros(n_long + 1, dtype=torch.int32)
-            cu_k[1:] = torch.tensor([e for _, e in spans[:n_long]], dtype=torch.int32).cumsum(0)
-            gather = (torch.cat(rows).to(dev), cu_k.to(dev))
+            gather = {}
+            for window, keep in hybrid.key_views(self.cfg):             # only keys that some token of the span sees
+                cut = [(min(keep, c), max(min(keep, c), c - window + 1) if window else 0) for c, _ in spans[:n_long]]
+                seen = [torch.cat([x[:k], x[lo:]]) if lo > k else x for x, (k, lo) in zip(rows, cut)]
+                cu_k = torch.zeros(n_long + 1, dtype=torch.int32)
+                cu_k[1:] = torch.tensor([x.numel() for x in seen], dtype=torch.int32).cumsum(0)
+                gather[window, keep] = (torch.cat(seen).to(dev), cu_k.to(dev))
         seq_of = torch.repeat_interleave(torch.arange(len(spans), dtype=torch.int32), torch.tensor(lens))
         pos = pos.to(dev)
         b = SpanBatch(cu=cu.to(dev), start=torch.tensor([c for c, _ in spans], dtype=torch.int32, device=dev),
                       slot=torch.tensor([r.state_slot for r in reqs], dtype=torch.long, device=dev), pos=pos, kv_slot=kv_slot.to(dev),
                       kv_len=(pos + 1).to(torch.int32), table=table.to(dev), seq_of=seq_of.to(dev) if n_long else None, n_long=n_long, t_long=t_long,
                       max_long=max(lens) if n_long else 0, max_len=max_len, gather=gather)
-        x, h = hybrid.embed_forward(self.cfg, self.embed_w, ids.to(dev))
-        for i, w in enumerate(self.layer_w):
-            h = hybrid.layer_step(self.cfg, i, w, x, h, self.k_cache[i], b)
-        return x, cu
+        return hybrid.forward(self.cfg, self.embed_w, self.layer_w, ids.to(dev), self.k_cache, b)[0], cu
 
     def _span_arrays(self, reqs: list[Request], spans: list[tuple[int, int]]) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
         """(token ids, positions, flat cache rows) of the packed tokens, on the host."""
@@ -1006,10 +1007,7 @@ class RolloutEngine:
         act = self.st_active[:bs]
         b = SpanBatch(cu=self.arange32[:bs + 1], start=(kvpos * act).to(torch.int32), slot=self.st_state[:bs] * act, pos=kvpos, kv_slot=kv_slot,
                       kv_len=self.st_seq_lens[:bs] * act.to(torch.int32), table=self.st_block_table[:bs], max_len=self.max_model_len)
-        x, h = hybrid.embed_forward(self.cfg, self.embed_w, self.st_input_ids[:bs])
-        last = len(self.layer_w) - 1
-        for i, w in enumerate(self.layer_w):
-            h = hybrid.layer_step(self.cfg, i, w, x, h, self.k_cache[i], b, self.head_w["norm_w"] if i == last else None)
+        _, h = hybrid.forward(self.cfg, self.embed_w, self.layer_w, self.st_input_ids[:bs], self.k_cache, b, self.head_w["norm_w"])
         return self._lm_logits(h)
 
     def _decode_sample(self, bs: int, logits: torch.Tensor) -> None:
