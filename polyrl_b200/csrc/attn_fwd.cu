@@ -1,4 +1,4 @@
-// polyrl_b200 — varlen causal flash-attention FORWARD on tcgen05 / TMEM / TMA (query / key width 128 or 192, value width 128, GQA).
+// polyrl_b200 — varlen causal flash-attention FORWARD on tcgen05 / TMEM / TMA (query / key width 64, 128 or 192, value width 64 or 128, GQA).
 //
 // Replaces the flash-attn 2 library call (mma.sync) the reference reaches through
 // 3rdparty/verl/verl/models/transformers/monkey_patch.py:49-117 (`_flash_attention_forward`) for training,
@@ -18,19 +18,23 @@
 // DK = 192 (latent attention expanded to heads: 128 + 64 rotary) keeps both K stages and drops to one V stage, which is
 // reloaded while the next scores and their softmax run.  An optional per-head sink adds exp(sink_h) to the softmax
 // denominator in the epilogue.
+// A sliding window with kept first tokens (query i sees key j if i - j < window or j < keep_first) skips the key tiles between the
+// kept ones and the window of the tile's first query.
 // Epilogue: O / l -> bf16 (16-byte stores), log-sum-exp per (head, token) for the backward pass.
 #include "common.cuh"
 
 namespace prl {
 
 constexpr int kAfThreads = 320;          // warp0 TMA, warp1 MMA, warps 2-5 + 6-9: two softmax warpgroups
-constexpr int kAfBM = 128, kAfBN = 128, kAfD = 128;
+constexpr int kAfBM = 128, kAfBN = 128;
 constexpr int kAfTile = 128 * 128 * 2;              // 32 KB: one 128 x 128 bf16 operand tile (2 chunks of 64 columns)
 template <int DK>
 struct AfCfg {
   static constexpr int QKT = 128 * DK * 2;            // Q or K tile: DK / 64 chunks of 128 rows x 64 columns
-  static constexpr int VST = DK == 128 ? 2 : 1;       // V stages
-  static constexpr int SMEM = 3 * QKT /*Q, K x 2*/ + VST * kAfTile /*V*/ + kAfTile /*P*/ + 1024 + 256;
+  static constexpr int DV = DK == 64 ? 64 : 128;      // value width
+  static constexpr int VT = 128 * DV * 2;             // V tile
+  static constexpr int VST = DK <= 128 ? 2 : 1;       // V stages
+  static constexpr int SMEM = 3 * QKT /*Q, K x 2*/ + VST * VT /*V*/ + kAfTile /*P*/ + 1024 + 256;
 };
 
 struct AttnFwdParams {
@@ -43,6 +47,7 @@ struct AttnFwdParams {
   float scale_log2;            // sm_scale * log2(e)
   float sm_scale;
   int causal;
+  int window, keep_first;      // window: 0x7fffffff when every earlier key is seen
   const float* sink;           // [nq] or null: natural-log sink of the softmax denominator
   long long* dbg;              // optional timeline buffer (kernel experiments)
 };
@@ -54,10 +59,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
-  constexpr int QKT = AfCfg<DK>::QKT, VST = AfCfg<DK>::VST;
+  constexpr int QKT = AfCfg<DK>::QKT, VST = AfCfg<DK>::VST, VT = AfCfg<DK>::VT, kAfD = AfCfg<DK>::DV, OW = kAfD / 2;
   uint8_t* sK = smem + QKT;                           // [2 stages]
   uint8_t* sV = smem + 3 * QKT;                       // [VST stages]
-  uint8_t* sP = sV + VST * kAfTile;
+  uint8_t* sP = sV + VST * VT;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + kAfTile);
   uint64_t* q_full = bars;            // 1
   uint64_t* k_full = bars + 1;        // [2]
@@ -97,7 +102,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   const int off = lk - lq;                             // bottom-right aligned causal mask (prefix-cached prefill: lk > lq)
   int kv_end = lk;
   if (p.causal) kv_end = min(lk, q0 + kAfBM + off);    // keys beyond the last row's diagonal are never needed
-  const int nt = max(1, (kv_end + kAfBN - 1) / kAfBN);
+  // key tiles in use: those of the kept first keys, then those from the window of this tile's first query on
+  const int w_tile = max(0, q0 + off - p.window + 1) / kAfBN;
+  const int kept_tiles = min((p.keep_first + kAfBN - 1) / kAfBN, w_tile), gap = w_tile - kept_tiles;
+  const int nt = max(1, (kv_end + kAfBN - 1) / kAfBN - gap);
+  auto tile_of = [&](int j) { return j < kept_tiles ? j : j + gap; };
 
   if (warp == 0 && lane == 0) {
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
@@ -128,17 +137,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         mbar_wait(&k_empty[s], ph ^ 1);
         mbar_expect_tx(&k_full[s], QKT);
 #pragma unroll
-        for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmK, &k_full[s], sK + s * QKT + c * 16384, hk * DK + c * 64, ks + j * kAfBN);
+        for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmK, &k_full[s], sK + s * QKT + c * 16384, hk * DK + c * 64, ks + tile_of(j) * kAfBN);
         mbar_wait(&v_empty[sv], ((j / VST) & 1) ^ 1);
-        mbar_expect_tx(&v_full[sv], kAfTile);
-        tma_load_2d(&tmV, &v_full[sv], sV + sv * kAfTile, hk * kAfD, ks + j * kAfBN);
-        tma_load_2d(&tmV, &v_full[sv], sV + sv * kAfTile + 16384, hk * kAfD + 64, ks + j * kAfBN);
+        mbar_expect_tx(&v_full[sv], VT);
+#pragma unroll
+        for (int c = 0; c < kAfD / 64; ++c) tma_load_2d(&tmV, &v_full[sv], sV + sv * VT + c * 16384, hk * kAfD + c * 64, ks + tile_of(j) * kAfBN);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr uint32_t idS = umma_idesc(128, 128, 1, 1);
-      constexpr uint32_t idO = umma_idesc_major(128, 128, 1, 1, 0, 1);      // B = V consumed MN-major
+      constexpr uint32_t idO = umma_idesc_major(128, kAfD, 1, 1, 0, 1);     // B = V consumed MN-major
       auto issue_s = [&](int j) {
         const int s = j & 1;
         mbar_wait(&k_full[s], (j >> 1) & 1);
@@ -165,7 +174,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk) {
           const uint64_t da = umma_desc_sw128_kmajor(sP + (kk >> 2) * 16384) + 2 * (kk & 3);
-          const uint64_t db = umma_desc_sw128_mnmajor(sV + sv * kAfTile, 16384) + kk * 128;
+          const uint64_t db = umma_desc_sw128_mnmajor(sV + sv * VT, 16384) + kk * 128;
           umma_bf16_ss(tO, da, db, idO, kk != 0);
         }
         umma_commit(o_full);
@@ -174,7 +183,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       }
     }
   } else {
-    // two softmax warpgroups: group g owns score / output columns [64g, 64g+64) of every row
+    // two softmax warpgroups: group g owns score columns [64g, 64g+64) and its half of the output columns of every row
     const int g = (warp - 2) >> 2;
     const int quad = warp & 3;
     const int r = quad * 32 + lane;                       // query row inside the tile == TMEM lane
@@ -182,9 +191,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const int qrow = q0 + r;                              // position inside the sequence's queries
     const int kmax = p.causal ? qrow + off : lk - 1;      // last key this row may attend to
     float m_run = -INFINITY, l_run = 0.f;
-    float O[64];
+    const int klo = qrow + off - p.window;                // keys up to here are behind the window (unless kept)
+    float O[OW];
 #pragma unroll
-    for (int i = 0; i < 64; ++i) O[i] = 0.f;
+    for (int i = 0; i < OW; ++i) O[i] = 0.f;
     const uint32_t sP_u32 = smem_u32(sP) + g * 16384 + r * 128;
     const bool rec = p.dbg != nullptr && blockIdx.x == gridDim.x / 2 && blockIdx.y == 0 && threadIdx.x == 64;
     long long* dbg = p.dbg;
@@ -195,8 +205,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       tc_fence_after();
       if (rec && j < 30) dbg[1 + 5 * j] = clock64();
       const uint32_t tS = tS0 + s * 128 + lane_base + g * 64;
-      const int col0 = j * kAfBN + g * 64;
-      const bool need_mask = (j * kAfBN + kAfBN - 1 > kmax) || (j * kAfBN + kAfBN > lk);
+      const int base = tile_of(j) * kAfBN, col0 = base + g * 64;
+      const bool need_mask = (base + kAfBN - 1 > kmax) || (base + kAfBN > lk) || base <= klo;
+      auto seen = [&](int col) { return col <= kmax && col < lk && (col > klo || col < p.keep_first); };
       // pass 1: max over this thread's 64 scores, then exchange with the other warpgroup's half of the row
       float mx = -INFINITY;
 #pragma unroll
@@ -209,7 +220,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int col = col0 + c + i;
-            mx = fmaxf(mx, (col <= kmax && col < lk) ? __uint_as_float(v[i]) : -INFINITY);
+            mx = fmaxf(mx, seen(col) ? __uint_as_float(v[i]) : -INFINITY);
           }
         } else {
 #pragma unroll
@@ -237,7 +248,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int col = col0 + c + i;
-            pv[i] = fast_exp2((col <= kmax && col < lk) ? __uint_as_float(v[i]) * p.scale_log2 - mb : -INFINITY);
+            pv[i] = fast_exp2(seen(col) ? __uint_as_float(v[i]) * p.scale_log2 - mb : -INFINITY);
           }
         } else {
 #pragma unroll
@@ -264,15 +275,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       mbar_arrive(&s_empty[s]);
       l_run = l_run * alpha + lsum;
       m_run = m_new;
-      // O[:, 64g:64g+64] = O * alpha + (P V)[:, 64g:64g+64]
+      // own half of O = O * alpha + P V
       mbar_wait(o_full, j & 1);
       tc_fence_after();
       if (rec && j < 30) dbg[4 + 5 * j] = clock64();
 #pragma unroll
-      for (int c = 0; c < 64; c += 32) {
+      for (int c = 0; c < OW; c += 32) {
         uint32_t v[32];
         __syncwarp();
-        tmem_ld_32x32(tO + lane_base + g * 64 + c, v);
+        tmem_ld_32x32(tO + lane_base + g * OW + c, v);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i) O[c + i] = O[c + i] * alpha + __uint_as_float(v[i]);
@@ -288,9 +299,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     if (p.sink != nullptr && m_run != -INFINITY) l_tot += fast_exp2(p.sink[h] * 1.4426950408889634f - m_run * p.scale_log2);
     if (qrow < lq) {
       const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
-      __nv_bfloat16* dst = p.o + static_cast<int64_t>(qs + qrow) * p.ldo + h * kAfD + g * 64;
+      __nv_bfloat16* dst = p.o + static_cast<int64_t>(qs + qrow) * p.ldo + h * kAfD + g * OW;
 #pragma unroll
-      for (int c = 0; c < 64; c += 8) {
+      for (int c = 0; c < OW; c += 8) {
         int4 ov;
         ov.x = pack_bf16(O[c] * inv, O[c + 1] * inv); ov.y = pack_bf16(O[c + 2] * inv, O[c + 3] * inv);
         ov.z = pack_bf16(O[c + 4] * inv, O[c + 5] * inv); ov.w = pack_bf16(O[c + 6] * inv, O[c + 7] * inv);
@@ -343,7 +354,7 @@ static int run_attn_fwd(const void* q, const void* k, const void* v, const AttnF
   CUtensorMap tmQ, tmK, tmV;
   if (af_tmap(&tmQ, q, p.Tq, static_cast<uint64_t>(p.nq) * DK, ldq * 2, kAfBM)) return -111;
   if (af_tmap(&tmK, k, Tk, static_cast<uint64_t>(p.nkv) * DK, ldk * 2, kAfBN)) return -112;
-  if (af_tmap(&tmV, v, Tk, static_cast<uint64_t>(p.nkv) * kAfD, ldv * 2, kAfBN)) return -113;
+  if (af_tmap(&tmV, v, Tk, static_cast<uint64_t>(p.nkv) * AfCfg<DK>::DV, ldv * 2, kAfBN)) return -113;
   static bool attr = false;
   if (!attr) {
     PRL_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, AfCfg<DK>::SMEM));
@@ -354,12 +365,13 @@ static int run_attn_fwd(const void* q, const void* k, const void* v, const AttnF
   return 0;
 }
 
-// q:[Tq, nq*dk] (pitch ldq), k:[Tk, nkv*dk], v:[Tk, nkv*128] (pitches ldk/ldv), o:[Tq, nq*128] (pitch ldo); pitches in ELEMENTS;
-// dk = 128 or 192.  cu_q / cu_k: int32 [B+1] device arrays.  max_tiles: upper bound on sum_b ceil(lq_b / 128) (e.g. Tq/128 + B).
+// q:[Tq, nq*dk] (pitch ldq), k:[Tk, nkv*dk], v:[Tk, nkv*dv] (pitches ldk/ldv), o:[Tq, nq*dv] (pitch ldo); pitches in ELEMENTS;
+// dk = 64 (dv = 64), 128 or 192 (dv = 128).  window > 0 (causal only): query i sees keys j <= i with i - j < window or j < keep_first.  cu_q / cu_k: int32 [B+1] device arrays.  max_tiles: upper bound on sum_b ceil(lq_b / 128) (e.g. Tq/128 + B).
 // sink: fp32 [nq] or null.
 extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o, float* lse, const int32_t* cu_q,
                             const int32_t* cu_k, int B, int Tq, int Tk, int nq, int nkv, int dk, int64_t ldq, int64_t ldk, int64_t ldv,
-                            int64_t ldo, float sm_scale, int causal, int max_tiles, const float* sink, long long* dbg, cudaStream_t stream) {
+                            int64_t ldo, float sm_scale, int causal, int max_tiles, const float* sink, int window, int keep_first, long long* dbg,
+                            cudaStream_t stream) {
   if (Tq <= 0 || B <= 0) return 0;
   if (nq % nkv != 0) return -110;
   AttnFwdParams p;
@@ -370,8 +382,12 @@ extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o
   p.sm_scale = sm_scale;
   p.scale_log2 = sm_scale * 1.4426950408889634f;
   p.causal = causal;
+  if (window > 0 && !causal) return -115;
+  p.window = window > 0 ? window : 0x7fffffff;
+  p.keep_first = window > 0 ? keep_first : 0;
   p.sink = sink;
   p.dbg = dbg;
+  if (dk == 64) return run_attn_fwd<64>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
   if (dk == 128) return run_attn_fwd<128>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
   if (dk == 192) return run_attn_fwd<192>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
   return -114;

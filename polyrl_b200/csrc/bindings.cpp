@@ -24,8 +24,6 @@ int prl_quant_fp8_rowwise(const void*, void*, float*, int, int, cudaStream_t);
 int prl_grad_accum(float*, const void*, int, float, int64_t, float*, cudaStream_t);
 int prl_sumsq(const float*, int64_t, float*, cudaStream_t);
 int prl_adamw(float*, float*, float*, float*, void*, int64_t, float, float, float, float, float, int, float, const float*, int*, int, cudaStream_t);
-int prl_paged_decode_workspace_floats(int, int, int, int);
-int prl_paged_decode(const void*, int64_t, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, float, int, float*, void*, int64_t, cudaStream_t);
 int prl_attn_bwd(const void*, const void*, const void*, const void*, const void*, const float*, float*, float*, void*, void*, const int32_t*, const int32_t*, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, int64_t, float, int, int, cudaStream_t);
 int prl_ipc_get_handle(void*, void*);
 int prl_ipc_open_handle(const void*, void**);
@@ -290,25 +288,6 @@ void adamw_(at::Tensor master, at::Tensor m, at::Tensor v, at::Tensor grad, cons
                   master.numel(), lr, beta1, beta2, eps, wd, static_cast<int>(step), max_norm,
                   total_sumsq.has_value() ? total_sumsq->data_ptr<float>() : nullptr,
                   status.has_value() ? status->data_ptr<int>() : nullptr, zero_grad ? 1 : 0, cur_stream()), "adamw");
-}
-
-at::Tensor paged_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache,
-                        const at::Tensor& block_table, const at::Tensor& seq_lens, int64_t nq, int64_t nkv, int64_t d,
-                        double sm_scale, int64_t splits, c10::optional<at::Tensor> out) {
-  CHECK_BF16(q); CHECK_BF16(k_cache); CHECK_BF16(v_cache);
-  TORCH_CHECK(block_table.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt);
-  TORCH_CHECK(q.dim() == 2 && q.stride(1) == 1 && k_cache.is_contiguous() && v_cache.is_contiguous());
-  TORCH_CHECK(k_cache.size(2) == 16, "KV page size must be 16 tokens");
-  const int B = q.size(0);
-  c10::cuda::CUDAGuard g(q.device());
-  at::Tensor o = out.has_value() ? *out : at::empty({B, nq * d}, q.options());
-  const int64_t ws = prl_paged_decode_workspace_floats(B, nq, d, splits);
-  at::Tensor workspace = at::empty({ws}, q.options().dtype(at::kFloat));
-  check(prl_paged_decode(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
-                         block_table.data_ptr<int32_t>(), block_table.stride(0), seq_lens.data_ptr<int32_t>(), B, nq,
-                         nkv, d, static_cast<float>(sm_scale), splits, workspace.data_ptr<float>(), o.data_ptr(),
-                         o.stride(0), cur_stream()), "paged_decode");
-  return o;
 }
 
 // varlen causal flash-attention forward on tcgen05 (csrc/attn_fwd.cu).  q:[Tq,nq,128] k,v:[Tk,nkv,128] (row-strided views allowed)
@@ -597,9 +576,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("grad_accum_", &grad_accum_);
   m.def("sumsq_", &sumsq_);
   m.def("adamw_", &adamw_);
-  m.def("paged_decode", &paged_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
-        py::arg("seq_lens"), py::arg("nq"), py::arg("nkv"), py::arg("d"), py::arg("sm_scale"), py::arg("splits") = 1,
-        py::arg("out") = py::none());
   m.def("attn_bwd", &attn_bwd);
   m.def("sym_malloc", &sym_malloc);
   m.def("sym_free", &sym_free);

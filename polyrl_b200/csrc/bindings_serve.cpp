@@ -9,9 +9,12 @@ extern "C" {
 int prl_gemm_bf16(const void*, const void*, void*, const void*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
 int prl_sample(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int64_t*, float*, cudaStream_t);
 int prl_sample_topk_topp(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int, float, int64_t*, float*, cudaStream_t);
-int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int32_t*, const int32_t*, int, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, float, int, int, const float*, long long*, cudaStream_t);
+int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int32_t*, const int32_t*, int, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, float, int, int, const float*, int, int, long long*, cudaStream_t);
+int prl_paged_decode_workspace_floats(int, int, int, int);
+int prl_paged_decode(const void*, int64_t, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, float, int, int, int, float*, void*, int64_t, cudaStream_t);
+int prl_gemm_clamped_glu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, float, float, cudaStream_t);
 int prl_gemm_gelu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, cudaStream_t);
-int prl_mix_embed(const int64_t*, const void*, float*, void*, int, int, int, cudaStream_t);
+int prl_mix_embed(const int64_t*, const void*, const float*, float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_norm_add(const void*, int64_t, float*, const float*, const float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_rms(const float*, const float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_gated_norm(const void*, int64_t, const void*, int64_t, const float*, void*, int64_t, int, int, int, float, int, int, cudaStream_t);
@@ -19,6 +22,13 @@ int prl_mix_conv(const void*, int64_t, const float*, const float*, void*, const 
 int prl_mix_latent_prep(const void*, int64_t, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, int, float, int, cudaStream_t);
 int prl_mix_rope(void*, int64_t, int, int, int, int, const double*, const int64_t*, int, int, cudaStream_t);
 int prl_mix_gelu(void*, int64_t, int, cudaStream_t);
+int prl_mix_qk_prep(const void*, int64_t, int, int, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, void*, void*, int, float, int, cudaStream_t);
+int prl_mix_gather_keys(const void*, const void*, const int64_t*, void*, void*, int64_t, int, int, cudaStream_t);
+int prl_mix_clamped_glu(const void*, void*, int64_t, int, int, float, float, int, cudaStream_t);
+int prl_mix_delta_ok(const void*, int64_t, const void*, int64_t, const void*, int64_t, int, int);
+int64_t prl_mix_delta_chunks(int64_t, int64_t);
+int prl_mix_delta_work_bytes();
+int prl_mix_delta_gate_floats();
 int prl_mix_chunk_supported(int);
 int prl_mix_latent_tc_ok(int, int);
 }
@@ -29,6 +39,8 @@ int prl_mix_chunk(const prl::ScanParams*, int, cudaStream_t);
 int prl_mix_chunk_tc_ok(const prl::ScanParams*);
 int prl_mix_chunk_tc(const prl::ScanParams*, int, int32_t*, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
+int prl_mix_window(const prl::WindowParams*, int, cudaStream_t);
+int prl_mix_delta(const prl::ScanParams*, int64_t, void*, float*, int32_t*, cudaStream_t);
 }
 
 namespace {
@@ -92,12 +104,13 @@ std::vector<at::Tensor> sample_topk_topp(const at::Tensor& logits, const c10::op
 
 std::vector<at::Tensor> attn_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& cu_q,
                                  const at::Tensor& cu_k, double sm_scale, bool causal, bool want_lse,
-                                 const c10::optional<at::Tensor>& dbg, const c10::optional<at::Tensor>& sink) {
+                                 const c10::optional<at::Tensor>& dbg, const c10::optional<at::Tensor>& sink, int64_t window, int64_t keep_first) {
   CHECK_BF16(q); CHECK_BF16(k); CHECK_BF16(v);
-  const int64_t dk = q.size(-1);
-  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && (dk == 128 || dk == 192) && k.size(2) == dk && v.size(2) == 128 &&
-              v.size(1) == k.size(1) && v.size(0) == k.size(0), "attn_fwd: query / key width 128 or 192, value width 128");
-  TORCH_CHECK(q.stride(2) == 1 && q.stride(1) == dk && k.stride(2) == 1 && k.stride(1) == dk && v.stride(2) == 1 && v.stride(1) == 128,
+  const int64_t dk = q.size(-1), dv = dk == 64 ? 64 : 128;
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && (dk == 64 || dk == 128 || dk == 192) && k.size(2) == dk && v.size(2) == dv &&
+              v.size(1) == k.size(1) && v.size(0) == k.size(0), "attn_fwd: query / key width 64, 128 or 192, value width 64 or 128");
+  TORCH_CHECK(window >= 0 && window <= 0x7fffffff && keep_first >= 0 && keep_first <= 0x7fffff00 && (window == 0 || causal), "attn_fwd: window");
+  TORCH_CHECK(q.stride(2) == 1 && q.stride(1) == dk && k.stride(2) == 1 && k.stride(1) == dk && v.stride(2) == 1 && v.stride(1) == dv,
               "attn_fwd: heads must be contiguous inside a token row");
   TORCH_CHECK(q.stride(0) % 8 == 0 && k.stride(0) % 8 == 0 && v.stride(0) % 8 == 0);
   TORCH_CHECK((reinterpret_cast<uintptr_t>(q.data_ptr()) & 15) == 0 && (reinterpret_cast<uintptr_t>(k.data_ptr()) & 15) == 0 &&
@@ -107,16 +120,36 @@ std::vector<at::Tensor> attn_fwd(const at::Tensor& q, const at::Tensor& k, const
   const int Tq = q.size(0), Tk = k.size(0), nq = q.size(1), nkv = k.size(1), B = cu_q.numel() - 1;
   if (sink.has_value()) { CHECK_F32(*sink); TORCH_CHECK(sink->is_contiguous() && sink->numel() == nq); }
   c10::cuda::CUDAGuard g(q.device());
-  at::Tensor o = at::empty({Tq, nq, 128}, q.options());
+  at::Tensor o = at::empty({Tq, nq, dv}, q.options());
   at::Tensor lse = want_lse ? at::empty({nq, Tq}, q.options().dtype(at::kFloat)) : at::Tensor();
   check(prl_attn_fwd(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), want_lse ? lse.data_ptr<float>() : nullptr,
                      cu_q.data_ptr<int>(), cu_k.data_ptr<int>(), B, Tq, Tk, nq, nkv, static_cast<int>(dk), q.stride(0), k.stride(0), v.stride(0),
-                     static_cast<int64_t>(nq) * 128, static_cast<float>(sm_scale), causal ? 1 : 0, Tq / 128 + B,
-                     sink.has_value() ? sink->data_ptr<float>() : nullptr,
+                     static_cast<int64_t>(nq) * dv, static_cast<float>(sm_scale), causal ? 1 : 0, Tq / 128 + B,
+                     sink.has_value() ? sink->data_ptr<float>() : nullptr, static_cast<int>(window), static_cast<int>(keep_first),
                      dbg.has_value() ? reinterpret_cast<long long*>(dbg->data_ptr<int64_t>()) : nullptr, cur_stream()),
         "attn_fwd");
   if (want_lse) return {o, lse};
   return {o};
+}
+
+at::Tensor paged_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache,
+                        const at::Tensor& block_table, const at::Tensor& seq_lens, int64_t nq, int64_t nkv, int64_t d,
+                        double sm_scale, int64_t splits, c10::optional<at::Tensor> out, int64_t window, int64_t keep_first) {
+  CHECK_BF16(q); CHECK_BF16(k_cache); CHECK_BF16(v_cache);
+  TORCH_CHECK(block_table.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt);
+  TORCH_CHECK(q.dim() == 2 && q.stride(1) == 1 && k_cache.is_contiguous() && v_cache.is_contiguous());
+  TORCH_CHECK(k_cache.size(2) == 16, "KV page size must be 16 tokens");
+  TORCH_CHECK(window >= 0 && window <= 0x7fffffff && keep_first >= 0 && keep_first <= 0x7fffff00, "paged_decode: window");
+  const int B = q.size(0);
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor o = out.has_value() ? *out : at::empty({B, nq * d}, q.options());
+  const int64_t ws = prl_paged_decode_workspace_floats(B, nq, d, splits);
+  at::Tensor workspace = at::empty({ws}, q.options().dtype(at::kFloat));
+  check(prl_paged_decode(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
+                         block_table.data_ptr<int32_t>(), block_table.stride(0), seq_lens.data_ptr<int32_t>(), B, nq,
+                         nkv, d, static_cast<float>(sm_scale), splits, static_cast<int>(window), static_cast<int>(keep_first),
+                         workspace.data_ptr<float>(), o.data_ptr(), o.stride(0), cur_stream()), "paged_decode");
+  return o;
 }
 
 static at::Tensor vec_i64(const std::vector<int64_t>& v) {
@@ -142,15 +175,17 @@ const I* veci(const at::Tensor& t, int64_t n, const char* what) {
   return t.data_ptr<I>();
 }
 
-std::vector<at::Tensor> mix_embed(const at::Tensor& ids, const at::Tensor& emb) {
+std::vector<at::Tensor> mix_embed(const at::Tensor& ids, const at::Tensor& emb, const c10::optional<at::Tensor>& w, double eps) {
   const int dt = dt_of(emb, "mix_embed");
   TORCH_CHECK(emb.is_contiguous() && emb.dim() == 2);
   const int64_t rows = ids.numel(), W = emb.size(1);
   const int64_t* ip = veci<int64_t>(ids, rows, "mix_embed ids");
   c10::cuda::CUDAGuard g(emb.device());
   at::Tensor x = at::empty({rows, W}, emb.options().dtype(at::kFloat));
-  at::Tensor h = dt == 0 ? at::empty({rows, W}, emb.options()) : x;
-  check(prl_mix_embed(ip, emb.data_ptr(), x.data_ptr<float>(), dt == 0 ? h.data_ptr() : nullptr, rows, W, dt, cur_stream()), "mix_embed");
+  const bool own = dt == 0 || w.has_value();
+  at::Tensor h = own ? at::empty({rows, W}, emb.options()) : x;
+  check(prl_mix_embed(ip, emb.data_ptr(), vecf(w, W, "mix_embed w"), x.data_ptr<float>(), own ? h.data_ptr() : nullptr, rows, W, static_cast<float>(eps), dt,
+                      cur_stream()), "mix_embed");
   return {x, h};
 }
 
@@ -179,19 +214,19 @@ at::Tensor mix_rms(const at::Tensor& x, const at::Tensor& w, double eps, bool bf
   return h;
 }
 
-at::Tensor mix_gated_norm(const at::Tensor& y, const at::Tensor& z, const at::Tensor& w, int64_t groups, double eps, bool gate_first) {
+at::Tensor mix_gated_norm(const at::Tensor& y, const at::Tensor& z, const at::Tensor& w, int64_t groups, double eps, int64_t gate) {
   const int dt = dt_of(y, "mix_gated_norm");
   rows2(y, "mix_gated_norm y"); rows2(z, "mix_gated_norm z");
   TORCH_CHECK(z.scalar_type() == y.scalar_type() && z.sizes() == y.sizes() && groups > 0 && y.size(1) % groups == 0);
   c10::cuda::CUDAGuard g(y.device());
   at::Tensor out = at::empty(y.sizes(), y.options());
   check(prl_mix_gated_norm(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), vecf(w, y.size(1), "mix_gated_norm w"), out.data_ptr(), out.stride(0),
-                           y.size(0), groups, y.size(1) / groups, static_cast<float>(eps), gate_first ? 1 : 0, dt, cur_stream()), "mix_gated_norm");
+                           y.size(0), groups, y.size(1) / groups, static_cast<float>(eps), static_cast<int>(gate), dt, cur_stream()), "mix_gated_norm");
   return out;
 }
 
 // x [T, ch] -> silu(conv(x)); state [slots, taps - 1, ch] is read for what lies before a span and left holding its last inputs
-at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const at::Tensor& bias, at::Tensor state, const at::Tensor& cu, const at::Tensor& start,
+at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const c10::optional<at::Tensor>& bias, at::Tensor state, const at::Tensor& cu, const at::Tensor& start,
                     const at::Tensor& slot, const c10::optional<at::Tensor>& seq_of) {
   const int dt = dt_of(x, "mix_conv");
   rows2(x, "mix_conv x");
@@ -208,17 +243,15 @@ at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const at::Tensor& 
   return out;
 }
 
-// gated linear recurrence over packed spans; form 0 = token by token, 1 = every span is one token, 2 = chunked (bf16), 3 = chunked on
-// tcgen05 where the layout allows, else 2; the last counter element is the error flag; mode 0 = state-space duality, 1 = matrix memory (csrc/mixers.cuh)
-void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
-                     const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log,
-                     const c10::optional<at::Tensor>& d_skip, double qscale, double cap, at::Tensor S, const c10::optional<at::Tensor>& nst,
-                     const c10::optional<at::Tensor>& mst, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, at::Tensor counter,
-                     int64_t form, at::Tensor out) {
-  const int dt = dt_of(v, "mix_scan");
+// gated linear recurrences over packed spans (mix_scan_): form 0 = token by token, 1 = every span is one token, 2 = chunked (bf16), 3 = chunked on
+// tcgen05 where the layout allows, else 2; the last counter element is the error flag; mode 0 = state-space duality, 1 = matrix memory, 2 = gated delta rule (csrc/mixers.cuh)
+prl::ScanParams scan_params(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
+                            const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log, double qscale,
+                            const at::Tensor& S, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, const at::Tensor& counter,
+                            const at::Tensor& out) {
   rows2(q, "mix_scan q"); rows2(k, "mix_scan k"); rows2(v, "mix_scan v"); rows2(g0, "mix_scan g0");
   CHECK_F32(S); CHECK_F32(g0);
-  TORCH_CHECK(mode == 0 || mode == 1);
+  TORCH_CHECK(mode >= 0 && mode <= 2);
   TORCH_CHECK(S.dim() == 4 && S.is_contiguous());
   const int64_t H = S.size(1), N = S.size(2), V = S.size(3), T = v.size(0), spans = start.numel();
   TORCH_CHECK(q.scalar_type() == v.scalar_type() && k.scalar_type() == v.scalar_type() && q.size(0) == T && k.size(0) == T && v.size(1) == H * V &&
@@ -230,18 +263,15 @@ void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at:
   p.ldq = q.stride(0); p.ldk = k.stride(0); p.ldv = v.stride(0);
   p.rep = H / (q.size(1) / N);
   p.g0 = g0.data_ptr<float>(); p.ldg = g0.stride(0);
-  p.b0 = vecf(b0, H, "b0"); p.b1 = vecf(b1, H, "b1"); p.a_log = vecf(a_log, H, "a_log"); p.d_skip = vecf(d_skip, H, "d_skip");
-  if (mode == 1) {
-    TORCH_CHECK(g1.has_value() && nst.has_value() && mst.has_value());
-    CHECK_F32(*g1); CHECK_F32(*nst); CHECK_F32(*mst);
+  p.b0 = vecf(b0, H, "b0"); p.b1 = vecf(b1, H, "b1"); p.a_log = vecf(a_log, H, "a_log");
+  if (mode != 0) {
+    TORCH_CHECK(g1.has_value());
+    CHECK_F32(*g1);
     TORCH_CHECK(g1->dim() == 2 && g1->size(0) == T && g1->size(1) == H && g1->stride(1) == 1 && g1->stride(0) == g0.stride(0));
-    TORCH_CHECK(nst->is_contiguous() && nst->numel() == S.size(0) * H * N && mst->is_contiguous() && mst->numel() == S.size(0) * H && cap > 0);
-    p.g1 = g1->data_ptr<float>(); p.nst = nst->data_ptr<float>(); p.mst = mst->data_ptr<float>();
-  } else {
-    TORCH_CHECK(a_log.has_value());
+    p.g1 = g1->data_ptr<float>();
   }
-  p.qscale = static_cast<float>(qscale); p.cap = static_cast<float>(cap);
-  c10::cuda::CUDAGuard g(v.device());
+  TORCH_CHECK(mode == 1 || a_log.has_value());
+  p.qscale = static_cast<float>(qscale);
   TORCH_CHECK(out.is_cuda() && out.scalar_type() == v.scalar_type() && out.is_contiguous() && out.dim() == 2 && out.size(0) == T && out.size(1) == H * V);
   p.out = out.data_ptr(); p.ldo = H * V;
   p.S = S.data_ptr<float>();
@@ -249,14 +279,50 @@ void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at:
   veci<int32_t>(counter, spans * H + 1, "counter");
   p.counter = counter.data_ptr<int32_t>();
   p.H = H; p.N = N; p.V = V; p.spans = spans;
+  return p;
+}
+
+void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
+                     const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log,
+                     const c10::optional<at::Tensor>& d_skip, double qscale, double cap, at::Tensor S, const c10::optional<at::Tensor>& nst,
+                     const c10::optional<at::Tensor>& mst, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, at::Tensor counter,
+                     int64_t form, at::Tensor out) {
+  const int dt = dt_of(v, "mix_scan");
+  prl::ScanParams p = scan_params(mode, q, k, v, g0, g1, b0, b1, a_log, qscale, S, cu, start, slot, counter, out);
+  p.d_skip = vecf(d_skip, p.H, "d_skip");
+  p.cap = static_cast<float>(cap);
+  if (mode == 1) {
+    TORCH_CHECK(nst.has_value() && mst.has_value());
+    CHECK_F32(*nst); CHECK_F32(*mst);
+    TORCH_CHECK(nst->is_contiguous() && nst->numel() == S.size(0) * p.H * p.N && mst->is_contiguous() && mst->numel() == S.size(0) * p.H && cap > 0);
+    p.nst = nst->data_ptr<float>(); p.mst = mst->data_ptr<float>();
+  }
+  c10::cuda::CUDAGuard g(v.device());
+  TORCH_CHECK(form < 2 || mode < 2, "mix_scan: the delta rule has its own chunked kernel");
   if (form == 3 && dt == 0 && prl_mix_chunk_tc_ok(&p)) {
     check(prl_mix_chunk_tc(&p, static_cast<int>(mode), p.counter + counter.numel() - 1, cur_stream()), "mix_chunk_tc");
   } else if (form >= 2) {
-    TORCH_CHECK(dt == 0 && prl_mix_chunk_supported(N), "mix_scan: the chunked kernel takes bf16 and N <= 256");
+    TORCH_CHECK(dt == 0 && prl_mix_chunk_supported(p.N), "mix_scan: the chunked kernel takes bf16 and N <= 256");
     check(prl_mix_chunk(&p, static_cast<int>(mode), cur_stream()), "mix_chunk");
   } else {
     check(prl_mix_scan(&p, static_cast<int>(mode), dt, form == 1, cur_stream()), "mix_scan");
   }
+}
+
+bool mix_delta_chunk_ok(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& S) {
+  return v.scalar_type() == at::kBFloat16 && prl_mix_delta_ok(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), S.size(2), S.size(3));
+}
+// gated delta rule in chunks of 64 tokens (bf16); the last counter element is the error flag
+void mix_delta_chunk_(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const at::Tensor& g1, const c10::optional<at::Tensor>& b0,
+                      const at::Tensor& a_log, double qscale, at::Tensor S, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot,
+                      at::Tensor counter, at::Tensor out) {
+  TORCH_CHECK(dt_of(v, "mix_delta_chunk") == 0 && mix_delta_chunk_ok(q, k, v, S), "mix_delta_chunk: layout");
+  const prl::ScanParams p = scan_params(2, q, k, v, g0, g1, b0, c10::nullopt, a_log, qscale, S, cu, start, slot, counter, out);
+  c10::cuda::CUDAGuard g(v.device());
+  const int64_t chunks = prl_mix_delta_chunks(v.size(0), p.spans);
+  at::Tensor work = at::empty({chunks * p.H * prl_mix_delta_work_bytes()}, v.options().dtype(at::kByte));
+  at::Tensor gates = at::empty({chunks * p.H * prl_mix_delta_gate_floats()}, v.options().dtype(at::kFloat));
+  check(prl_mix_delta(&p, chunks, work.data_ptr(), gates.data_ptr<float>(), p.counter + counter.numel() - 1, cur_stream()), "mix_delta_chunk");
 }
 
 // a [T, qr + r + rd] -> (normed query latent [T, qr], packed cache rows [T, r + rd] or empty); cache rows also go to pool[kvslot]
@@ -314,6 +380,81 @@ at::Tensor mix_latent(const at::Tensor& q_lat, const at::Tensor& q, int64_t d, c
     p.part = part.data_ptr<float>();
   }
   check(prl_mix_latent(&p, tc ? 1 : 0, dt, cur_stream()), "mix_latent");
+  return out;
+}
+
+// rows [queries H x dim | keys G x dim] -> q [T, H, width] (normed, rotated), the same of the keys and the raw keys to the pools
+// [pages, G, 16, width] and, when asked for, packed [T, G, width]
+std::vector<at::Tensor> mix_qk_prep(const at::Tensor& p, int64_t heads, int64_t dim, const at::Tensor& wq, const at::Tensor& wk, const at::Tensor& freq,
+                                    const at::Tensor& pos, const at::Tensor& kvslot, at::Tensor k_pool, at::Tensor v_pool, double eps, bool want_kv) {
+  const int dt = dt_of(p, "mix_qk_prep");
+  rows2(p, "mix_qk_prep p");
+  TORCH_CHECK(k_pool.dim() == 4 && k_pool.size(2) == 16 && k_pool.sizes() == v_pool.sizes());
+  for (const at::Tensor& t : {k_pool, v_pool}) TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.scalar_type() == p.scalar_type(), "mix_qk_prep: pools");
+  const int64_t T = p.size(0), G = k_pool.size(1), width = k_pool.size(3), rd = 2 * freq.numel();
+  TORCH_CHECK(p.size(1) >= (heads + G) * dim && rd <= dim && width >= dim && (width == dim || width % 8 == 0));
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == at::kDouble && freq.is_contiguous());
+  c10::cuda::CUDAGuard g(p.device());
+  at::Tensor q = at::empty({T, heads, width}, p.options()), k = at::empty({want_kv ? T : 0, G, width}, p.options()), v = at::empty_like(k);
+  check(prl_mix_qk_prep(p.data_ptr(), p.stride(0), heads, G, dim, width, rd, vecf(wq, heads * dim, "wq"), vecf(wk, G * dim, "wk"), freq.data_ptr<double>(),
+                        veci<int64_t>(pos, T, "pos"), veci<int64_t>(kvslot, T, "kvslot"), q.data_ptr(), want_kv ? k.data_ptr() : nullptr,
+                        want_kv ? v.data_ptr() : nullptr, k_pool.data_ptr(), v_pool.data_ptr(), T, static_cast<float>(eps), dt, cur_stream()), "mix_qk_prep");
+  return {q, k, v};
+}
+
+std::vector<at::Tensor> mix_gather_keys(const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& rows) {
+  TORCH_CHECK(k_pool.is_cuda() && k_pool.dim() == 4 && k_pool.size(2) == 16 && k_pool.is_contiguous() && v_pool.is_contiguous() && v_pool.is_cuda() &&
+              v_pool.sizes() == k_pool.sizes() && v_pool.scalar_type() == k_pool.scalar_type());
+  const int64_t n = rows.numel(), G = k_pool.size(1), width = k_pool.size(3);
+  c10::cuda::CUDAGuard g(k_pool.device());
+  at::Tensor k = at::empty({n, G, width}, k_pool.options()), v = at::empty_like(k);
+  check(prl_mix_gather_keys(k_pool.data_ptr(), v_pool.data_ptr(), veci<int64_t>(rows, n, "rows"), k.data_ptr(), v.data_ptr(), n, G,
+                            width * k_pool.element_size(), cur_stream()), "mix_gather_keys");
+  return {k, v};
+}
+
+// paged windowed attention, any width: q [R, H, D] -> [R, H, D]
+at::Tensor mix_window_attention(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table,
+                                const c10::optional<at::Tensor>& seq_of, const at::Tensor& kv_len, double scale, int64_t window, int64_t keep_first) {
+  const int dt = dt_of(q, "mix_window_attention");
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && k_pool.dim() == 4 && k_pool.size(2) == 16 && k_pool.sizes() == v_pool.sizes() && k_pool.size(3) == q.size(2));
+  for (const at::Tensor& t : {k_pool, v_pool}) TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.scalar_type() == q.scalar_type(), "mix_window_attention: pools");
+  TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.dim() == 2 && table.stride(1) == 1);
+  const int64_t R = q.size(0);
+  TORCH_CHECK(seq_of.has_value() || table.size(0) >= R);
+  TORCH_CHECK(window >= 1 && window <= 0x7fffffff && keep_first >= 0 && keep_first <= 0x7fffffff);
+  prl::WindowParams p{};
+  p.q = q.data_ptr(); p.k_pool = k_pool.data_ptr(); p.v_pool = v_pool.data_ptr();
+  p.table = table.data_ptr<int32_t>(); p.ld_table = table.stride(0);
+  p.seq_of = seq_of.has_value() ? veci<int32_t>(*seq_of, R, "seq_of") : nullptr;
+  p.kv_len = veci<int32_t>(kv_len, R, "kv_len");
+  p.R = R; p.H = q.size(1); p.G = k_pool.size(1); p.D = q.size(2);
+  p.window = window; p.keep_first = keep_first; p.scale = static_cast<float>(scale);
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty_like(q);
+  p.out = out.data_ptr();
+  check(prl_mix_window(&p, dt, cur_stream()), "mix_window_attention");
+  return out;
+}
+
+at::Tensor gemm_clamped_glu(const at::Tensor& a, const at::Tensor& wgu, double limit, double alpha) {
+  CHECK_BF16(a); CHECK_BF16(wgu); CHECK_LASTDIM(a); CHECK_LASTDIM(wgu);
+  TORCH_CHECK(a.dim() == 2 && wgu.dim() == 2 && a.size(1) == wgu.size(1) && wgu.size(0) % 256 == 0 && a.size(1) % 8 == 0 && a.stride(0) % 8 == 0 &&
+              wgu.stride(0) % 8 == 0, "gemm_clamped_glu: gate / up rows in blocks of 128");
+  c10::cuda::CUDAGuard g(a.device());
+  at::Tensor h = at::empty({a.size(0), wgu.size(0) / 2}, a.options());
+  check(prl_gemm_clamped_glu_bf16(a.data_ptr(), wgu.data_ptr(), h.data_ptr(), a.size(0), wgu.size(0), a.size(1), a.stride(0), wgu.stride(0), h.stride(0),
+                                  static_cast<float>(limit), static_cast<float>(alpha), cur_stream()), "gemm_clamped_glu");
+  return h;
+}
+// gu [T, 2 F], gate and up columns in alternating blocks of blk -> [T, F]
+at::Tensor mix_clamped_glu(const at::Tensor& gu, int64_t blk, double limit, double alpha) {
+  const int dt = dt_of(gu, "mix_clamped_glu");
+  TORCH_CHECK(gu.dim() == 2 && gu.is_contiguous() && blk > 0 && gu.size(1) % (2 * blk) == 0);
+  c10::cuda::CUDAGuard g(gu.device());
+  at::Tensor out = at::empty({gu.size(0), gu.size(1) / 2}, gu.options());
+  check(prl_mix_clamped_glu(gu.data_ptr(), out.data_ptr(), gu.size(0), gu.size(1) / 2, blk, static_cast<float>(limit), static_cast<float>(alpha), dt,
+                            cur_stream()), "mix_clamped_glu");
   return out;
 }
 
@@ -383,7 +524,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_bf16", &gemm_bf16, py::arg("a"), py::arg("b"), py::arg("residual") = py::none(),
         py::arg("out") = py::none(), py::arg("force_bn") = 0);
   m.def("attn_fwd", &attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu_q"), py::arg("cu_k"), py::arg("sm_scale"),
-        py::arg("causal") = true, py::arg("want_lse") = true, py::arg("dbg") = py::none(), py::arg("sink") = py::none());
+        py::arg("causal") = true, py::arg("want_lse") = true, py::arg("dbg") = py::none(), py::arg("sink") = py::none(), py::arg("window") = 0,
+        py::arg("keep_first") = 0);
+  m.def("paged_decode", &paged_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
+        py::arg("seq_lens"), py::arg("nq"), py::arg("nkv"), py::arg("d"), py::arg("sm_scale"), py::arg("splits") = 1,
+        py::arg("out") = py::none(), py::arg("window") = 0, py::arg("keep_first") = 0);
   m.def("sample", &sample);
   m.def("sample_topk_topp", &sample_topk_topp);
   m.def("mix_embed", &mix_embed);
@@ -395,6 +540,13 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mix_latent_prep", &mix_latent_prep);
   m.def("mix_rope_", &mix_rope_);
   m.def("mix_latent", &mix_latent);
+  m.def("mix_delta_chunk_ok", &mix_delta_chunk_ok);
+  m.def("mix_delta_chunk_", &mix_delta_chunk_);
+  m.def("mix_qk_prep", &mix_qk_prep);
+  m.def("mix_gather_keys", &mix_gather_keys);
+  m.def("mix_window_attention", &mix_window_attention);
+  m.def("gemm_clamped_glu", &gemm_clamped_glu);
+  m.def("mix_clamped_glu", &mix_clamped_glu);
   m.def("gemm_gelu", &gemm_gelu);
   m.def("mix_gelu_", &mix_gelu_);
   m.def("mix_chunk_supported", [](int64_t n) { return prl_mix_chunk_supported(static_cast<int>(n)) != 0; });

@@ -39,7 +39,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32, MINB)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [num_seqs, nq*D] (row pitch ldq)
                     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                     const int32_t* __restrict__ block_table, int64_t ld_bt, const int32_t* __restrict__ seq_lens,
-                    int nq, int nkv, int splits, float scale_log2, float* __restrict__ o_part,
+                    int nq, int nkv, int splits, float scale_log2, int window, int keep_first, float* __restrict__ o_part,
                     float* __restrict__ ml_part, __nv_bfloat16* __restrict__ out_direct, int64_t ldo) {
   static_assert(D % 64 == 0, "head dim must be a multiple of 64");
   constexpr int KC = D / 32;     // 32-wide d chunks for QK (two MMAs each)
@@ -52,7 +52,11 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
   const int gq = lane >> 2, qd = lane & 3;    // fragment row / quad index
 
   const int len = seq_lens[seq];
-  const int num_pages = (len + kPage - 1) / kPage;
+  // visible keys: the last `window` and the first `keep_first`; their pages are numbered 0, 1, ... across the gap between the two
+  const int first = max(0, len - window);
+  const int kept_pages = min((min(keep_first, len) + kPage - 1) / kPage, first / kPage);
+  const int gap = first / kPage - kept_pages;
+  const int num_pages = (len + kPage - 1) / kPage - gap;
   const int pages_per_split = (num_pages + splits - 1) / splits;
   const int p_begin = split * pages_per_split;
   const int p_end = min(num_pages, p_begin + pages_per_split);
@@ -79,7 +83,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
 
   const int32_t* bt = block_table + static_cast<int64_t>(seq) * ld_bt;
   constexpr int kLinesPerPage = kPage * D * 2 / 128;          // 128-byte lines in one K (or V) page of one kv head
-  int64_t blk_next = (p_begin + warp < p_end) ? bt[p_begin + warp] : 0;
+  auto page_of = [&](int p) { return p < kept_pages ? p : p + gap; };
+  int64_t blk_next = (p_begin + warp < p_end) ? bt[page_of(p_begin + warp)] : 0;
   for (int p = p_begin + warp; p < p_end; p += kAttnWarps) {
     const int64_t blk = blk_next;
     const __nv_bfloat16* kp = k_cache + ((blk * nkv + kvh) * kPage) * D;
@@ -87,7 +92,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
     // ---- software prefetch: look up this warp's NEXT page now (breaks the block-table -> KV dependent-load chain) and pull
     // its K and V lines into L2 while the current page is being consumed (zero register cost, doubles bytes in flight)
     if (p + kAttnWarps < p_end) {
-      blk_next = bt[p + kAttnWarps];
+      blk_next = bt[page_of(p + kAttnWarps)];
       if (lane < kLinesPerPage) {
         const int64_t off = ((blk_next * nkv + kvh) * kPage) * D + lane * 64;
         asm volatile("prefetch.global.L2 [%0];" ::"l"(k_cache + off));
@@ -121,13 +126,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
       }
     }
     // ---- mask + online softmax (base-2 domain)
-    const int tok0 = p * kPage;
+    const int tok0 = page_of(p) * kPage;
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const bool ok = tok0 + 8 * j + 2 * qd + e < len;
+        const int tok = tok0 + 8 * j + 2 * qd + e;
+        const bool ok = tok < len && (tok >= first || tok < keep_first);
         s[j][e] = ok ? s[j][e] * scale_log2 : -INFINITY;
         s[j][2 + e] = ok ? s[j][2 + e] * scale_log2 : -INFINITY;
         mx_lo = fmaxf(mx_lo, s[j][e]);
@@ -260,14 +266,16 @@ extern "C" int prl_paged_decode_workspace_floats(int num_seqs, int nq, int d, in
 }
 
 // q:[num_seqs, nq*d] bf16; k/v cache [num_blocks, nkv, 16, d] bf16; block_table int32 [num_seqs, ld_bt];
-// seq_lens int32 (INCLUDING the current token, already appended to the cache).
+// seq_lens int32 (INCLUDING the current token, already appended to the cache).  window > 0: a sequence sees its last `window` keys
+// and its first `keep_first`.
 extern "C" int prl_paged_decode(const void* q, int64_t ldq, const void* k_cache, const void* v_cache,
                                 const int32_t* block_table, int64_t ld_bt, const int32_t* seq_lens, int num_seqs,
-                                int nq, int nkv, int d, float sm_scale, int splits, float* workspace, void* out,
+                                int nq, int nkv, int d, float sm_scale, int splits, int window, int keep_first, float* workspace, void* out,
                                 int64_t ldo, cudaStream_t s) {
   if (num_seqs <= 0) return 0;
   if (nq % nkv != 0 || nq / nkv > 16) return -30;
   if (splits < 1) splits = 1;
+  if (window <= 0) window = 0x7fffffff, keep_first = 0;
   float* o_part = workspace;
   float* ml_part = workspace + static_cast<int64_t>(num_seqs) * nq * splits * d;
   const float scale_log2 = sm_scale * 1.4426950408889634f;
@@ -277,14 +285,14 @@ extern "C" int prl_paged_decode(const void* q, int64_t ldq, const void* k_cache,
     auto kern = minb >= 4 ? paged_decode_kernel<128, 4> : paged_decode_kernel<128, 3>;
     kern<<<grid, kAttnWarps * 32, 0, s>>>(
         static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(k_cache),
-        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, o_part,
+        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, o_part,
         ml_part, splits == 1 ? static_cast<__nv_bfloat16*>(out) : nullptr, ldo);
     if (splits > 1)
       decode_merge_kernel<128><<<num_seqs * nq, 128, 0, s>>>(o_part, ml_part, splits, static_cast<__nv_bfloat16*>(out), ldo, nq);
   } else if (d == 64) {
     paged_decode_kernel<64, 3><<<grid, kAttnWarps * 32, 0, s>>>(
         static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(k_cache),
-        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, o_part,
+        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, o_part,
         ml_part, splits == 1 ? static_cast<__nv_bfloat16*>(out) : nullptr, ldo);
     if (splits > 1)
       decode_merge_kernel<64><<<num_seqs * nq, 64, 0, s>>>(o_part, ml_part, splits, static_cast<__nv_bfloat16*>(out), ldo, nq);

@@ -111,6 +111,35 @@ struct EpiSwiglu {
   }
 };
 
+// the same weight layout with a clamped gate: H = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+struct ClampedGluParams {
+  __nv_bfloat16* H;      // [M, ldh]   N/2 columns
+  int64_t ldh;
+  float limit, alpha;
+};
+struct EpiClampedGlu {
+  using Params = ClampedGluParams;
+  __device__ __forceinline__ void begin(const Params&, int, int, const WorkInfo&) {}
+  __device__ __forceinline__ void end(const Params&, int, int, const WorkInfo&) {}
+  template <int BN>
+  __device__ __forceinline__ void tile(const Params& p, const AccReader& acc, int row, int M, int n0, int N) {
+    static_assert(BN == 256, "gate / up epilogues expect 256-wide interleaved n-blocks");
+#pragma unroll 1
+    for (int c = 0; c < 128; c += 32) {
+      float g[32], u[32];
+      acc.load(c, g);
+      acc.load(128 + c, u);
+      if (row >= M || n0 + 128 + c >= N) continue;
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const float x = fminf(g[i], p.limit), y = fminf(fmaxf(u[i], -p.limit), p.limit);
+        g[i] = __fdividef(x, 1.0f + __expf(fminf(-p.alpha * x, 80.f))) * (y + 1.f);
+      }
+      store_row_chunk(p.H + static_cast<int64_t>(row) * p.ldh + (n0 >> 1) + c, g, 32);
+    }
+  }
+};
+
 // H[M, N] = gelu(acc)
 struct GeluParams {
   __nv_bfloat16* H;
@@ -201,6 +230,18 @@ extern "C" int prl_gemm_swiglu_bf16(const void* A, const void* Wgu, void* H, voi
   using Cfg = GemmCfg<256, 2>;
   return launch_gemm<Cfg, EpiSwiglu, NoGate, false>(A, Wgu, M, N2, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0,
                                                     stream);
+}
+
+extern "C" int prl_gemm_clamped_glu_bf16(const void* A, const void* Wgu, void* H, int M, int N2, int K, int64_t lda, int64_t ldw, int64_t ldh, float limit,
+                                         float alpha, cudaStream_t stream) {
+  if (N2 % 256 != 0) return -11;
+  ClampedGluParams sp{static_cast<__nv_bfloat16*>(H), ldh, limit, alpha};
+  if (M > kBlockM) {
+    using Cfg2 = Gemm2Cfg<256, false, false, false>;
+    return launch_gemm2<Cfg2, EpiClampedGlu>(A, Wgu, nullptr, M, N2, K, lda * 2, ldw * 2, 0, sp, 0, stream);
+  }
+  using Cfg = GemmCfg<256, 2>;
+  return launch_gemm<Cfg, EpiClampedGlu, NoGate, false>(A, Wgu, M, N2, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);
 }
 
 // H = gelu_tanh(A·W^T)

@@ -13,7 +13,7 @@
 // Shared memory: NB chunks of 64 state columns.  NB = 2 (N <= 128) keeps Q, the scores and two K tiles side by side, so every
 // load of the next chunk is in flight during this one; NB = 4 (N <= 256) overlays the scores on Q.
 // Every wait is bounded: on a timeout the CTA raises *err, stops computing, frees its TMEM and returns.
-#include "mixers.cuh"
+#include "mix_tc.cuh"
 
 namespace prl {
 
@@ -49,34 +49,9 @@ struct TcShared {                        // behind the tiles
   uint32_t tmem;
 };
 
-__device__ __forceinline__ bool tc_wait(uint64_t* bar, uint32_t parity) {
-  if (mbar_try_wait(bar, parity)) return true;
-  const long long t0 = clock64();
-  while (!mbar_try_wait(bar, parity)) {
-    if (clock64() - t0 > 4000000000ll) return false;                  // about two seconds
-  }
-  return true;
-}
 // one 128 x 64 chunk: rows [0, nv) x columns [c0, c0 + 64) of src (columns below n), zero elsewhere
 __device__ __forceinline__ void tc_load(uint8_t* dst, const __nv_bfloat16* src, int64_t ld, int nv, int c0, int n) {
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int idx = threadIdx.x + i * kTcThreads, r = idx >> 3, u = idx & 7, c = c0 + u * 8;
-    const bool ok = r < nv && c < n;
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst) + r * 128 + ((u ^ (r & 7)) << 4)),
-                 "l"(src + (ok ? static_cast<int64_t>(r) * ld + c : 0)), "r"(ok ? 16 : 0) : "memory");
-  }
-}
-__device__ __forceinline__ uint4 tc_ld16(const uint8_t* tile, int r, int u) {
-  return *reinterpret_cast<const uint4*>(tile + r * 128 + ((u ^ (r & 7)) << 4));
-}
-__device__ __forceinline__ void tc_st16(uint8_t* tile, int r, int u, const uint32_t (&q)[4]) {
-  *reinterpret_cast<uint4*>(tile + r * 128 + ((u ^ (r & 7)) << 4)) = make_uint4(q[0], q[1], q[2], q[3]);
-}
-__device__ __forceinline__ void tc_split(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(a, b);
-  const float2 h = unpack_bf16(hi);
-  lo = pack_bf16(a - h.x, b - h.y);
+  tc_load_rows<128, kTcThreads>(dst, src, ld, nv, c0, n);
 }
 
 // raw gate values of the lane's four tokens (4 lane, ...) of a chunk

@@ -4,16 +4,31 @@
 
 namespace prl {
 
-// ---- x = embed[id] (fp32), h = the same in T (h may be null when T is fp32 and x is used directly)
+// ---- x = embed[id] (fp32), h = the same in T (h may be null when T is fp32 and x is used directly), or T(rms(x) * w) when w is given
 template <class T, int VEC>
-__global__ void mix_embed_kernel(const int64_t* __restrict__ ids, const T* __restrict__ emb, float* __restrict__ x, T* __restrict__ h, int W) {
+__global__ void __launch_bounds__(128) mix_embed_kernel(const int64_t* __restrict__ ids, const T* __restrict__ emb, const float* __restrict__ w,
+                                                        float* __restrict__ x, T* __restrict__ h, int W, float eps) {
+  __shared__ float red[4];
   const int64_t row = blockIdx.x;
   const T* src = emb + ids[row] * W;
-  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += 128 * VEC) {
     float v[VEC];
     ld_vec<T, VEC>(src + c, v);
     st_vec<float, VEC>(x + row * W + c, v);
-    if (h) st_vec<T, VEC>(h + row * W + c, v);
+    if (h && !w) st_vec<T, VEC>(h + row * W + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
+  }
+  if (!w) return;
+  const float r = rsqrtf(block_sum<4>(ss, red) / W + eps);
+  for (int c = threadIdx.x * VEC; c < W; c += 128 * VEC) {
+    float v[VEC], g[VEC];
+    ld_vec<T, VEC>(src + c, v);
+    ld_vec<float, VEC>(w + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] *= r * g[i];
+    st_vec<T, VEC>(h + row * W + c, v);
   }
 }
 
@@ -80,12 +95,14 @@ __global__ void __launch_bounds__(256) mix_rms_kernel(const float* __restrict__ 
   }
 }
 
-// ---- group norm of mixer outputs with a gate: GATE_FIRST  rms(y silu(z)) w   else   rms(y) w sigmoid(z)
+// ---- group norm of mixer outputs with a gate: kSiluFirst  rms(y silu(z)) w,   else  rms(y) w sigmoid(z)  or  rms(y) w silu(z)
 // WPG warps share one (row, group); 8 / WPG groups per CTA
-template <class T, int VEC, bool GATE_FIRST, int WPG>
+enum : int { kSigmoidLast = 0, kSiluFirst = 1, kSiluLast = 2 };
+template <class T, int VEC, int GATE, int WPG>
 __global__ void __launch_bounds__(256) mix_gated_norm_kernel(const T* __restrict__ y, int64_t ldy, const T* __restrict__ z, int64_t ldz,
                                                              const float* __restrict__ w, T* __restrict__ out, int64_t ldo, int64_t items, int groups,
                                                              int gs, float eps) {
+  constexpr bool GATE_FIRST = GATE == kSiluFirst;
   __shared__ float red[8];
   const int64_t item = static_cast<int64_t>(blockIdx.x) * (8 / WPG) + (threadIdx.x >> 5) / WPG;
   if (WPG == 1 && item >= items) return;                // (WPG == 8: one item per CTA, the grid is exact)
@@ -109,7 +126,7 @@ __global__ void __launch_bounds__(256) mix_gated_norm_kernel(const T* __restrict
           ld_vec<T, VEC>(zr + c, g);
 #pragma unroll
           for (int i = 0; i < VEC; ++i) {
-            const float f = GATE_FIRST ? silu_t<T>(g[i]) : sigmoid_t<T>(g[i]);
+            const float f = GATE == kSigmoidLast ? sigmoid_t<T>(g[i]) : silu_t<T>(g[i]);
             if (!GATE_FIRST) ss += u[k][i] * u[k][i];
             u[k][i] *= f;
             if (GATE_FIRST) ss += u[k][i] * u[k][i];
@@ -148,12 +165,21 @@ __global__ void __launch_bounds__(256) mix_gated_norm_kernel(const T* __restrict
     ld_vec<T, VEC>(zr + c, g);
     ld_vec<float, VEC>(w + c0 + c, ww);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[i] = v[i] * (GATE_FIRST ? silu_f(g[i]) : sigmoid_f(g[i])) * r * ww[i];
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * (GATE == kSigmoidLast ? sigmoid_f(g[i]) : silu_f(g[i])) * r * ww[i];
     st_vec<T, VEC>(orow + c, v);
   }
 }
 
-// ---- causal convolution per channel + silu; w [taps, ch] (row taps - 1 = current token), state [slots, taps - 1, ch]
+template <int VEC>
+__device__ __forceinline__ void ld_bias(const float* bias, int c, float (&v)[VEC]) {
+  if (bias) {
+    ld_vec<float, VEC>(bias + c, v);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+  }
+}
+// ---- causal convolution per channel + silu (bias may be null); w [taps, ch] (row taps - 1 = current token), state [slots, taps - 1, ch]
 template <class T, int VEC, int TT>
 __global__ void __launch_bounds__(128) mix_conv_kernel(const T* __restrict__ x, int64_t ldx, const float* __restrict__ w, const float* __restrict__ bias,
                                                        const T* __restrict__ state, const int32_t* __restrict__ cu, const int32_t* __restrict__ start,
@@ -167,7 +193,7 @@ __global__ void __launch_bounds__(128) mix_conv_kernel(const T* __restrict__ x, 
     const int t0 = cu[s];
     const bool fresh = start[s] == 0;
     float acc[VEC];
-    ld_vec<float, VEC>(bias + c, acc);
+    ld_bias<VEC>(bias, c, acc);
     for (int j = 0; j < taps; ++j) {
       const int u = t - (taps - 1) + j;
       float v[VEC], g[VEC];
@@ -198,7 +224,7 @@ __global__ void __launch_bounds__(128) mix_conv_window_kernel(const T* __restric
   float wt[TAPS][8], bs[8], win[TAPS][8];               // win[j]: input of token t - (TAPS - 1) + j
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) ld_vec<float, 8>(w + static_cast<int64_t>(j) * ch + c, wt[j]);
-  ld_vec<float, 8>(bias + c, bs);
+  ld_bias<8>(bias, c, bs);
   int cur = -1;
 #pragma unroll 4
   for (int t = tb; t < te; ++t) {
@@ -265,7 +291,7 @@ __global__ void __launch_bounds__(128) mix_conv_step_kernel(const T* __restrict_
   const bool fresh = start[s] == 0;
   T* st = state + slot[s] * static_cast<int64_t>(taps - 1) * ch + c;
   float acc[VEC], g[VEC], cur[VEC];
-  ld_vec<float, VEC>(bias + c, acc);
+  ld_bias<VEC>(bias, c, acc);
   ld_vec<T, VEC>(x + static_cast<int64_t>(s) * ldx + c, cur);
   for (int j = 0; j < taps - 1; ++j) {
     float v[VEC];
@@ -345,6 +371,134 @@ __global__ void __launch_bounds__(128) mix_rope_kernel(T* __restrict__ q, int64_
   }
 }
 
+// ---- windowed attention, per token: p = [queries heads x dim | keys kheads x dim].  Queries and keys are RMS-normed over the whole row
+// and rotated in neighbouring pairs; q, k [T, heads, width] and the cached rows are zero beyond dim, values are the keys as projected.
+// Pools are [pages, kheads, 16, width]; kp / vp (packed keys and values) may be null.
+template <class T>
+__global__ void __launch_bounds__(256) mix_qk_prep_kernel(const T* __restrict__ p, int64_t ldp, int heads, int kheads, int dim, int width, int rd,
+                                                          const float* __restrict__ wq, const float* __restrict__ wk, const double* __restrict__ freq,
+                                                          const int64_t* __restrict__ pos, const int64_t* __restrict__ kvslot, T* __restrict__ q,
+                                                          T* __restrict__ kp, T* __restrict__ vp, T* __restrict__ k_pool, T* __restrict__ v_pool, float eps) {
+  __shared__ float sc[256], sn[256], red[8];
+  const int64_t t = blockIdx.x;
+  const T* row = p + t * ldp;
+  const int nq = heads * dim, nk = kheads * dim;
+  for (int i = threadIdx.x; i < rd / 2; i += 256) rope_cs(pos[t], freq[i], sc[i], sn[i]);
+  const bool vec = sizeof(T) == 2 && dim % 8 == 0 && ldp % 8 == 0 && rd % 8 == 0 && (reinterpret_cast<uintptr_t>(p) & 15) == 0;
+  float sq = 0.f, sk = 0.f;
+  if (vec) {
+    for (int c = threadIdx.x * 8; c < nq + nk; c += 2048) {
+      float v[8];
+      ld_vec<T, 8>(row + c, v);
+      float a = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a += v[i] * v[i];
+      if (c < nq) sq += a; else sk += a;
+    }
+  } else {
+    for (int c = threadIdx.x; c < nq + nk; c += 256) {
+      const float v = to_f<T>(row[c]);
+      if (c < nq) sq += v * v; else sk += v * v;
+    }
+  }
+  const float rq = rsqrtf(block_sum<8>(sq, red) / nq + eps);
+  const float rk = rsqrtf(block_sum<8>(sk, red) / nk + eps);           // (both sums end in a barrier: the angles are in place)
+  const int64_t slot = kvslot[t], page = slot / 16, off = slot % 16;
+  auto dst = [&](int g) { return ((page * kheads + g) * 16 + off) * width; };
+  if (vec) {
+    const int wu = width / 8;                                          // 16-byte units of a head
+    for (int u = threadIdx.x; u < (heads + kheads) * wu; u += 256) {
+      const int hd = u / wu, c = (u % wu) * 8;
+      const bool key = hd >= heads;
+      float x[8], y[8];
+      if (c < dim) {
+        float w[8];
+        ld_vec<T, 8>(row + hd * dim + c, x);
+        ld_vec<float, 8>(key ? wk + (hd - heads) * dim + c : wq + hd * dim + c, w);
+        const float r = key ? rk : rq;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = x[i] * r * w[i];
+        if (c < rd) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float cs = sc[c / 2 + i], s = sn[c / 2 + i], a = y[2 * i], b = y[2 * i + 1];
+            y[2 * i] = a * cs - b * s;
+            y[2 * i + 1] = b * cs + a * s;
+          }
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] = y[i] = 0.f;
+      }
+      if (!key) {
+        st_vec<T, 8>(q + (t * heads + hd) * width + c, y);
+      } else {
+        const int g = hd - heads;
+        st_vec<T, 8>(k_pool + dst(g) + c, y);
+        st_vec<T, 8>(v_pool + dst(g) + c, x);
+        if (kp) {
+          st_vec<T, 8>(kp + (t * kheads + g) * width + c, y);
+          st_vec<T, 8>(vp + (t * kheads + g) * width + c, x);
+        }
+      }
+    }
+    return;
+  }
+  for (int e = threadIdx.x; e < (heads + kheads) * width; e += 256) {
+    const int hd = e / width, c = e % width;
+    const bool key = hd >= heads;
+    float x = 0.f, y = 0.f;
+    if (c < dim) {
+      const T* src = row + hd * dim;
+      const float* w = key ? wk + (hd - heads) * dim : wq + hd * dim;
+      const float r = key ? rk : rq;
+      x = to_f<T>(src[c]);
+      y = x * r * w[c];
+      if (c < rd) {
+        const int o = c ^ 1;
+        const float z = to_f<T>(src[o]) * r * w[o], cs = sc[c / 2], s = sn[c / 2];
+        y = (c & 1) ? y * cs + z * s : y * cs - z * s;
+      }
+    }
+    if (!key) {
+      q[(t * heads + hd) * width + c] = from_f<T>(y);
+    } else {
+      const int g = hd - heads;
+      k_pool[dst(g) + c] = from_f<T>(y);
+      v_pool[dst(g) + c] = from_f<T>(x);
+      if (kp) {
+        kp[(t * kheads + g) * width + c] = from_f<T>(y);
+        vp[(t * kheads + g) * width + c] = from_f<T>(x);
+      }
+    }
+  }
+}
+// packed keys and values of flat cache rows; 16-byte units
+__global__ void __launch_bounds__(256) mix_gather_keys_kernel(const uint4* __restrict__ k_pool, const uint4* __restrict__ v_pool,
+                                                              const int64_t* __restrict__ rows, uint4* __restrict__ k, uint4* __restrict__ v, int64_t n,
+                                                              int kheads, int units) {
+  const int64_t per = static_cast<int64_t>(kheads) * units;
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x; i < n * per; i += static_cast<int64_t>(gridDim.x) * 256) {
+    const int64_t r = rows[i / per];
+    const int rest = static_cast<int>(i % per), g = rest / units, u = rest % units;
+    const int64_t src = ((r / 16 * kheads + g) * 16 + r % 16) * units + u;
+    k[i] = k_pool[src];
+    v[i] = v_pool[src];
+  }
+}
+
+// gate and up columns interleaved in blocks of blk: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+template <class T>
+__global__ void mix_clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, int64_t rows, int F, int blk, float limit, float alpha) {
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < rows * F; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t r = i / F;
+    const int c = static_cast<int>(i % F);
+    const T* src = gu + r * 2 * F + (c / blk) * 2 * blk + c % blk;
+    const float g = fminf(to_f<T>(src[0]), limit), u = fminf(fmaxf(to_f<T>(src[blk]), -limit), limit);
+    out[i] = from_f<T>(g * sigmoid_f(alpha * g) * (u + 1.f));
+  }
+}
+
 template <class T, int VEC>
 __global__ void mix_gelu_kernel(T* __restrict__ x, int64_t n) {
   for (int64_t i = (static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x) * VEC; i < n; i += static_cast<int64_t>(gridDim.x) * blockDim.x * VEC) {
@@ -374,10 +528,11 @@ using namespace prl;
     }                                                                                                \
   } while (0)
 
-extern "C" int prl_mix_embed(const int64_t* ids, const void* emb, float* x, void* h, int rows, int W, int dtype, cudaStream_t st) {
+extern "C" int prl_mix_embed(const int64_t* ids, const void* emb, const float* w, float* x, void* h, int rows, int W, float eps, int dtype,
+                             cudaStream_t st) {
   if (rows <= 0) return 0;
-  const bool vec = W % 8 == 0 && al16(emb) && al16(x) && al16(h);
-  MIX_DISPATCH(vec, (mix_embed_kernel<T, VEC><<<rows, 128, 0, st>>>(ids, static_cast<const T*>(emb), x, static_cast<T*>(h), W)));
+  const bool vec = W % 8 == 0 && al16(emb) && al16(x) && al16(h) && al16(w);
+  MIX_DISPATCH(vec, (mix_embed_kernel<T, VEC><<<rows, 128, 0, st>>>(ids, static_cast<const T*>(emb), w, x, static_cast<T*>(h), W, eps)));
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
@@ -397,7 +552,7 @@ extern "C" int prl_mix_rms(const float* x, const float* w, void* h, int rows, in
   return 0;
 }
 extern "C" int prl_mix_gated_norm(const void* y, int64_t ldy, const void* z, int64_t ldz, const float* w, void* out, int64_t ldo, int rows, int groups,
-                                  int gs, float eps, int gate_first, int dtype, cudaStream_t st) {
+                                  int gs, float eps, int gate, int dtype, cudaStream_t st) {
   if (rows <= 0) return 0;
   const int64_t items = static_cast<int64_t>(rows) * groups;
   const bool vec = gs % 8 == 0 && ldy % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && al16(y) && al16(z) && al16(w) && al16(out);
@@ -406,10 +561,14 @@ extern "C" int prl_mix_gated_norm(const void* y, int64_t ldy, const void* z, int
 #define MIX_GN(GF, WPG)                                                                                                                   \
   MIX_DISPATCH(vec, (mix_gated_norm_kernel<T, VEC, GF, WPG><<<static_cast<unsigned>(grid), 256, 0, st>>>(                                 \
                         static_cast<const T*>(y), ldy, static_cast<const T*>(z), ldz, w, static_cast<T*>(out), ldo, items, groups, gs, eps)))
-  if (gate_first) {
-    if (wide) MIX_GN(true, 8); else MIX_GN(true, 1);
+  if (gate == kSiluFirst) {
+    if (wide) MIX_GN(kSiluFirst, 8); else MIX_GN(kSiluFirst, 1);
+  } else if (gate == kSiluLast) {
+    if (wide) MIX_GN(kSiluLast, 8); else MIX_GN(kSiluLast, 1);
+  } else if (gate == kSigmoidLast) {
+    if (wide) MIX_GN(kSigmoidLast, 8); else MIX_GN(kSigmoidLast, 1);
   } else {
-    if (wide) MIX_GN(false, 8); else MIX_GN(false, 1);
+    return -223;
   }
 #undef MIX_GN
   PRL_CUDA_CHECK(cudaGetLastError());
@@ -492,6 +651,46 @@ extern "C" int prl_mix_rope(void* q, int64_t ldq, int H, int dq, int d, int rd, 
   if (rd > 512) return -222;
   if (dtype == 0) mix_rope_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>(static_cast<__nv_bfloat16*>(q), ldq, H, dq, d, rd, freq, pos);
   else mix_rope_kernel<float><<<rows, 128, 0, st>>>(static_cast<float*>(q), ldq, H, dq, d, rd, freq, pos);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_qk_prep(const void* p, int64_t ldp, int heads, int kheads, int dim, int width, int rd, const float* wq, const float* wk,
+                               const double* freq, const int64_t* pos, const int64_t* kvslot, void* q, void* kp, void* vp, void* k_pool, void* v_pool, int rows,
+                               float eps, int dtype, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (rd > 512 || rd > dim || width < dim) return -224;
+  if (dtype == 0) {
+    using T = __nv_bfloat16;
+    mix_qk_prep_kernel<T><<<rows, 256, 0, st>>>(static_cast<const T*>(p), ldp, heads, kheads, dim, width, rd, wq, wk, freq, pos, kvslot, static_cast<T*>(q),
+                                                static_cast<T*>(kp), static_cast<T*>(vp), static_cast<T*>(k_pool), static_cast<T*>(v_pool), eps);
+  } else {
+    using T = float;
+    mix_qk_prep_kernel<T><<<rows, 256, 0, st>>>(static_cast<const T*>(p), ldp, heads, kheads, dim, width, rd, wq, wk, freq, pos, kvslot, static_cast<T*>(q),
+                                                static_cast<T*>(kp), static_cast<T*>(vp), static_cast<T*>(k_pool), static_cast<T*>(v_pool), eps);
+  }
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+// row_bytes: bytes of one head's key, a multiple of 16
+extern "C" int prl_mix_gather_keys(const void* k_pool, const void* v_pool, const int64_t* rows, void* k, void* v, int64_t n, int kheads, int row_bytes,
+                                   cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (row_bytes % 16 || !al16(k_pool) || !al16(v_pool) || !al16(k) || !al16(v)) return -225;
+  const int64_t blocks = (n * kheads * (row_bytes / 16) + 255) / 256;
+  mix_gather_keys_kernel<<<static_cast<unsigned>(blocks < 148 * 32 ? blocks : 148 * 32), 256, 0, st>>>(
+      static_cast<const uint4*>(k_pool), static_cast<const uint4*>(v_pool), rows, static_cast<uint4*>(k), static_cast<uint4*>(v), n, kheads, row_bytes / 16);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+extern "C" int prl_mix_clamped_glu(const void* gu, void* out, int64_t rows, int F, int blk, float limit, float alpha, int dtype, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (F <= 0 || blk <= 0 || F % blk) return -226;
+  const int64_t blocks = (rows * F + 255) / 256;
+  const unsigned grid = static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16);
+  if (dtype == 0)
+    mix_clamped_glu_kernel<<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(out), rows, F, blk, limit, alpha);
+  else
+    mix_clamped_glu_kernel<<<grid, 256, 0, st>>>(static_cast<const float*>(gu), static_cast<float*>(out), rows, F, blk, limit, alpha);
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

@@ -11,7 +11,7 @@ struct ScanParams {
   const float *g0, *g1;         // raw gate projections [tokens, ldg], one column per head
   int64_t ldg;
   const float *b0, *b1;         // their biases [H]
-  const float *a_log, *d_skip;  // kSsd [H]
+  const float *a_log, *d_skip;  // kSsd, kDelta (a_log only) [H]
   float qscale, cap;            // q is multiplied by qscale; cap bounds the kMlstm gates
   void* out;                    // T [tokens, ldo], head h at h * V
   int64_t ldo;
@@ -23,6 +23,18 @@ struct ScanParams {
   const int64_t* slot;          // [spans]
   int32_t* counter;             // [>= spans * H], zero between launches
   int H, N, V, spans;
+};
+
+struct WindowParams {
+  const void* q;                // T [R, H, D]
+  const void *k_pool, *v_pool;  // T [blocks, G, 16, D]
+  const int32_t* table;         // [spans, ld_table] page numbers
+  int64_t ld_table;
+  const int32_t* seq_of;        // [R] span of a row (null: row r is span r)
+  const int32_t* kv_len;        // [R] keys up to the row's own; 0 = idle row
+  void* out;                    // T [R, H, D]
+  int R, H, G, D, window, keep_first;
+  float scale;
 };
 
 struct LatentParams {

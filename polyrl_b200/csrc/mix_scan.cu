@@ -3,8 +3,11 @@
 //   kSsd   (Mamba-2 / state-space duality)   S = exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x
 //   kMlstm (xLSTM matrix memory)             m' = max(f + m, i),  S = e^(f+m-m') S + e^(i-m') k v^T,  n likewise with k alone,
 //                                            y = S^T q / (max(|n . q|, e^(-m')) + 1e-6);  m starts at 0
+//   kDelta (gated delta rule)                k' = k / |k|, q' = scale q / |q|,  S = keep S + k' u^T,  u = beta (v - keep S^T k'),  y = S^T q'
+//                                            with keep = exp(-exp(A_log) softplus(a + bias)), beta = sigmoid(b).  With S the state before the
+//                                            token, y = keep S^T q' + (k' . q') u, so one pass over S gives both products.
 //
-// mix_step_kernel serves spans of one token (decode): every state byte is read and written once, streaming.
+// mix_step_kernel (mix_delta_step_kernel for kDelta) serves spans of one token (decode): every state byte is read and written once, streaming.
 // mix_scan_kernel: one CTA = one (span, head, 32 value columns): lane = value column, warp w owns the state rows w, w + 8, ... in registers
 // from the first token to the last.
 #include "mixers.cuh"
@@ -19,7 +22,8 @@ __global__ void __launch_bounds__(kScanWarps * 32)
 mix_scan_kernel(ScanParams p) {
   constexpr int NMAX = RN * kScanWarps;
   __shared__ float s_q[2][NMAX], s_k[2][NMAX], s_n[NMAX];
-  __shared__ float s_red[2][kScanWarps][33], s_dot[2][kScanWarps];
+  constexpr int ND = MODE == kDelta ? 3 : 1;
+  __shared__ float s_red[2][kScanWarps][33], s_dot[2][ND][kScanWarps], s_red2[MODE == kDelta ? 2 : 1][kScanWarps][33];
   const int vt = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
   const int w = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
   const int t0 = p.cu[s], t1 = p.cu[s + 1];
@@ -47,11 +51,49 @@ mix_scan_kernel(ScanParams p) {
     for (int n = tid; n < NMAX; n += kScanWarps * 32) s_n[n] = (!fresh && n < p.N) ? p.nst[hb * p.N + n] : 0.f;
   }
   const float b0 = p.b0 ? p.b0[h] : 0.f, b1 = p.b1 ? p.b1[h] : 0.f;
-  const float a_neg = MODE == kSsd ? -expf(p.a_log[h]) : 0.f;
+  const float a_neg = MODE != kMlstm ? -expf(p.a_log[h]) : 0.f;
   const float skip = (MODE == kSsd && p.d_skip) ? p.d_skip[h] : 0.f;
 
   for (int t = t0; t < t1; ++t) {
     const int b = t & 1;
+    if constexpr (MODE == kDelta) {
+      float kk = 0.f, qq = 0.f, kq = 0.f;
+      for (int n = tid; n < NMAX; n += kScanWarps * 32) {
+        const float qn = n < p.N ? to_f<T>(q[static_cast<int64_t>(t) * p.ldq + n]) : 0.f;
+        const float kn = n < p.N ? to_f<T>(k[static_cast<int64_t>(t) * p.ldk + n]) : 0.f;
+        s_q[b][n] = qn;
+        s_k[b][n] = kn;
+        kk += kn * kn; qq += qn * qn; kq += kn * qn;
+      }
+      kk = warp_sum(kk); qq = warp_sum(qq); kq = warp_sum(kq);
+      if (lane == 0) { s_dot[b][0][w] = kk; s_dot[b][1][w] = qq; s_dot[b][2][w] = kq; }
+      const float vv = col_ok ? to_f<T>(v[static_cast<int64_t>(t) * p.ldv + col]) : 0.f;
+      const float keep = expf(a_neg * softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0));
+      const float beta = sigmoid_f(p.g1[static_cast<int64_t>(t) * p.ldg + h] + b1);
+      __syncthreads();
+      float ak = 0.f, aq = 0.f;
+#pragma unroll
+      for (int i = 0; i < RN; ++i) {
+        const int n = i * kScanWarps + w;
+        ak += s_k[b][n] * S[i];
+        aq += s_q[b][n] * S[i];
+      }
+      s_red[b][w][lane] = ak;
+      s_red2[b][w][lane] = aq;
+      __syncthreads();
+      ak = aq = kk = qq = kq = 0.f;
+#pragma unroll
+      for (int i = 0; i < kScanWarps; ++i) {
+        ak += s_red[b][i][lane]; aq += s_red2[b][i][lane];
+        kk += s_dot[b][0][i]; qq += s_dot[b][1][i]; kq += s_dot[b][2][i];
+      }
+      const float rk = rsqrtf(kk + kUnitEps), rq = rsqrtf(qq + kUnitEps) * p.qscale;
+      const float u = beta * (vv - keep * rk * ak), uk = u * rk;
+#pragma unroll
+      for (int i = 0; i < RN; ++i) S[i] = keep * S[i] + uk * s_k[b][i * kScanWarps + w];
+      if (w == 0 && col_ok) out[static_cast<int64_t>(t) * p.ldo + col] = from_f<T>(rq * (keep * aq + uk * kq));
+      continue;
+    }
     for (int n = tid; n < NMAX; n += kScanWarps * 32) {
       s_q[b][n] = n < p.N ? to_f<T>(q[static_cast<int64_t>(t) * p.ldq + n]) * p.qscale : 0.f;
       s_k[b][n] = n < p.N ? to_f<T>(k[static_cast<int64_t>(t) * p.ldk + n]) : 0.f;
@@ -88,7 +130,7 @@ mix_scan_kernel(ScanParams p) {
         d += nn * s_q[b][n];
       }
       d = warp_sum(d);
-      if (lane == 0) s_dot[b][w] = d;
+      if (lane == 0) s_dot[b][0][w] = d;
     }
     __syncthreads();
     if (w == 0 && col_ok) {
@@ -100,7 +142,7 @@ mix_scan_kernel(ScanParams p) {
       } else {
         float d = 0.f;
 #pragma unroll
-        for (int i = 0; i < kScanWarps; ++i) d += s_dot[b][i];
+        for (int i = 0; i < kScanWarps; ++i) d += s_dot[b][0][i];
         y /= fmaxf(fabsf(d), floor_) + 1e-6f;
       }
       out[static_cast<int64_t>(t) * p.ldo + col] = from_f<T>(y);
@@ -243,6 +285,104 @@ mix_step_kernel(ScanParams p) {
   }
 }
 
+// ---- kDelta, one token per span: the state tile waits in registers for its two products, then is updated and written back
+template <class T, int RN, int CPL>
+__global__ void __launch_bounds__(kScanWarps * 32)
+mix_delta_step_kernel(ScanParams p) {
+  __shared__ float s_q[RN * kScanWarps], s_k[RN * kScanWarps], s_dot[3][kScanWarps];
+  __shared__ alignas(16) float s_red[2][kScanWarps][32 * CPL];
+  const int vt = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
+  const int w = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+  const int t = p.cu[s];
+  if (p.cu[s + 1] <= t) return;
+  const bool fresh = p.start[s] == 0;
+  const int64_t hb = p.slot[s] * p.H + h;
+  const int col = vt * 32 * CPL + lane * CPL;
+  const bool ok = col < p.V;                             // V is a multiple of CPL
+  float* Sg = p.S + hb * static_cast<int64_t>(p.N) * p.V + col;
+  float st[RN][CPL];
+#pragma unroll
+  for (int i = 0; i < RN; ++i) {
+    const int n = i * kScanWarps + w;
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) st[i][c] = 0.f;
+    if (!fresh && ok && n < p.N) ld_cols<CPL>(Sg + static_cast<int64_t>(n) * p.V, st[i]);
+  }
+  const T* q = static_cast<const T*>(p.q) + static_cast<int64_t>(t) * p.ldq + static_cast<int64_t>(h / p.rep) * p.N;
+  const T* k = static_cast<const T*>(p.k) + static_cast<int64_t>(t) * p.ldk + static_cast<int64_t>(h / p.rep) * p.N;
+  const T* v = static_cast<const T*>(p.v) + static_cast<int64_t>(t) * p.ldv + static_cast<int64_t>(h) * p.V;
+  float kk = 0.f, qq = 0.f, kq = 0.f;
+  for (int n = tid; n < RN * kScanWarps; n += kScanWarps * 32) {
+    const float qn = n < p.N ? to_f<T>(q[n]) : 0.f, kn = n < p.N ? to_f<T>(k[n]) : 0.f;
+    s_q[n] = qn;
+    s_k[n] = kn;
+    kk += kn * kn; qq += qn * qn; kq += kn * qn;
+  }
+  kk = warp_sum(kk); qq = warp_sum(qq); kq = warp_sum(kq);
+  if (lane == 0) { s_dot[0][w] = kk; s_dot[1][w] = qq; s_dot[2][w] = kq; }
+  float vv[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) vv[c] = ok ? to_f<T>(v[col + c]) : 0.f;
+  const float keep = expf(-expf(p.a_log[h]) * softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + (p.b0 ? p.b0[h] : 0.f)));
+  const float beta = sigmoid_f(p.g1[static_cast<int64_t>(t) * p.ldg + h] + (p.b1 ? p.b1[h] : 0.f));
+  __syncthreads();
+  float ak[CPL], aq[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) ak[c] = aq[c] = 0.f;
+#pragma unroll
+  for (int i = 0; i < RN; ++i) {
+    const float kn = s_k[i * kScanWarps + w], qn = s_q[i * kScanWarps + w];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) { ak[c] += kn * st[i][c]; aq[c] += qn * st[i][c]; }
+  }
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) { s_red[0][w][lane * CPL + c] = ak[c]; s_red[1][w][lane * CPL + c] = aq[c]; ak[c] = aq[c] = 0.f; }
+  __syncthreads();
+  kk = qq = kq = 0.f;
+#pragma unroll
+  for (int i = 0; i < kScanWarps; ++i) {
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) { ak[c] += s_red[0][i][lane * CPL + c]; aq[c] += s_red[1][i][lane * CPL + c]; }
+    kk += s_dot[0][i]; qq += s_dot[1][i]; kq += s_dot[2][i];
+  }
+  const float rk = rsqrtf(kk + kUnitEps), rq = rsqrtf(qq + kUnitEps) * p.qscale;
+  float uk[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) uk[c] = beta * (vv[c] - keep * rk * ak[c]) * rk;
+#pragma unroll
+  for (int i = 0; i < RN; ++i) {
+    const int n = i * kScanWarps + w;
+    const float kn = s_k[n];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) st[i][c] = keep * st[i][c] + uk[c] * kn;
+    if (ok && n < p.N) st_cols<CPL>(Sg + static_cast<int64_t>(n) * p.V, st[i]);
+  }
+  if (w == 0 && ok) {
+    T* o = static_cast<T*>(p.out) + static_cast<int64_t>(t) * p.ldo + static_cast<int64_t>(h) * p.V + col;
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) o[c] = from_f<T>(rq * (keep * aq[c] + uk[c] * kq));
+  }
+}
+template <class T, int RN>
+static int launch_delta_step(const ScanParams& p, cudaStream_t st) {
+  constexpr int C4 = RN <= 16 ? 4 : 1, C2 = RN <= 32 ? 2 : 1;          // (at most 64 state entries per thread)
+  const bool al = (reinterpret_cast<uintptr_t>(p.S) & 15) == 0;
+  const int threads = kScanWarps * 32;
+  if (al && C4 == 4 && p.V % 4 == 0 && p.V > 64) mix_delta_step_kernel<T, RN, C4><<<dim3((p.V + 127) / 128, p.H, p.spans), threads, 0, st>>>(p);
+  else if (al && C2 == 2 && p.V % 2 == 0 && p.V > 32) mix_delta_step_kernel<T, RN, C2><<<dim3((p.V + 63) / 64, p.H, p.spans), threads, 0, st>>>(p);
+  else mix_delta_step_kernel<T, RN, 1><<<dim3((p.V + 31) / 32, p.H, p.spans), threads, 0, st>>>(p);
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+template <class T>
+static int launch_delta_step(const ScanParams& p, cudaStream_t st) {
+  if (p.N <= 64) return launch_delta_step<T, 8>(p, st);
+  if (p.N <= 128) return launch_delta_step<T, 16>(p, st);
+  if (p.N <= 256) return launch_delta_step<T, 32>(p, st);
+  if (p.N <= 512) return launch_delta_step<T, 64>(p, st);
+  return -203;
+}
+
 template <class T, int MODE>
 static int launch_step(const ScanParams& p, cudaStream_t st) {
   const bool al = (reinterpret_cast<uintptr_t>(p.S) & 15) == 0;
@@ -273,14 +413,15 @@ static int launch_scan(const ScanParams& p, cudaStream_t st) {
 
 using namespace prl;
 
-// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm; single: every span is one token
+template <class T>
+static int run_scan(const ScanParams& p, int mode, int single, cudaStream_t st) {
+  if (mode == kDelta) return single ? launch_delta_step<T>(p, st) : launch_scan<T, kDelta>(p, st);
+  if (single) return mode == kSsd ? launch_step<T, kSsd>(p, st) : launch_step<T, kMlstm>(p, st);
+  return mode == kSsd ? launch_scan<T, kSsd>(p, st) : launch_scan<T, kMlstm>(p, st);
+}
+// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm / kDelta; single: every span is one token
 extern "C" int prl_mix_scan(const ScanParams* p, int mode, int dtype, int single, cudaStream_t st) {
   if (p->spans <= 0) return 0;
   if (p->spans > 65535 || p->H > 65535) return -202;
-  if (single) {
-    if (dtype == 0) return mode == kSsd ? launch_step<__nv_bfloat16, kSsd>(*p, st) : launch_step<__nv_bfloat16, kMlstm>(*p, st);
-    return mode == kSsd ? launch_step<float, kSsd>(*p, st) : launch_step<float, kMlstm>(*p, st);
-  }
-  if (dtype == 0) return mode == kSsd ? launch_scan<__nv_bfloat16, kSsd>(*p, st) : launch_scan<__nv_bfloat16, kMlstm>(*p, st);
-  return mode == kSsd ? launch_scan<float, kSsd>(*p, st) : launch_scan<float, kMlstm>(*p, st);
+  return dtype == 0 ? run_scan<__nv_bfloat16>(*p, mode, single, st) : run_scan<float>(*p, mode, single, st);
 }

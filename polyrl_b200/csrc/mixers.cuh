@@ -84,11 +84,13 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return s;
 }
 
-// The two gated linear recurrences served by mix_scan.cu / mix_chunk.cu:
+// The gated linear recurrences served by mix_scan.cu / mix_chunk.cu / mix_delta.cu:
 //   S_t = keep_t S_(t-1) + add_t k_t v_t^T,     y_t = S_t^T q_t
 //   kSsd    state-space duality: dt = softplus(g0 + b0), keep = exp(-exp(A_log) dt), add = dt;   y += D v
 //   kMlstm  matrix memory with a running maximum m and normaliser n (csrc/mix_scan.cu)
-enum : int { kSsd = 0, kMlstm = 1 };
+//   kDelta  gated delta rule: unit k and q, the write corrects what the decayed state already answers for k (csrc/mix_scan.cu)
+enum : int { kSsd = 0, kMlstm = 1, kDelta = 2 };
+constexpr float kUnitEps = 1e-6f;        // under the root of a unit vector's norm
 
 // n and m are read by every value tile of a head and may be overwritten only after the last tile has read them: the last
 // CTA of a (span, head) to finish writes them (all tiles compute the same values).  Returns true for that CTA.

@@ -604,6 +604,20 @@ PRESETS: dict[str, dict] = {
                                dict(kind="latent", sizes=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536,
                                                               scale=192 ** -0.5, rot_base=500000.0)),
                                dict(kind="ssd", sizes=dict(heads=128, vdim=64, state=128, groups=8, conv=4, norm_groups=8))][i % 4])) for i in range(16))),
+    # Lanilix stacks (models/hybrid.py)
+    "tiny-lanilix": dict(family="hybrid", vocab_size=512, hidden_size=256, intermediate_size=384, num_layers=4, num_heads=1, num_kv_heads=1,
+                         rms_norm_eps=1e-6, eos_token_id=-1, bos_token_id=-1, hf_model_type="lanilix", sandwich_norm=True, norm_offset=1.0, layers=tuple(
+                             dict(kind=k, sizes=s, ff=384, weights_of=w, act="clamped_glu", limit=7.0, alpha=1.702) for k, s, w in (
+                                 ("delta", dict(heads=4, kv_heads=2, dim=48, vdim=64, conv=4), 0),
+                                 ("window", dict(heads=6, kv_heads=2, dim=48, vdim=48, scale=48 ** -0.5, window=96, keep_first=4, rot_dim=24, rot_base=10000.0), 1),
+                                 ("delta", dict(heads=4, kv_heads=2, dim=48, vdim=64, conv=4), 2),
+                                 ("delta", dict(heads=4, kv_heads=2, dim=48, vdim=64, conv=4), 0)))),
+    "lanilix-4b": dict(family="hybrid", vocab_size=128256, hidden_size=4096, intermediate_size=14336, num_layers=16, num_heads=1, num_kv_heads=1,
+                       rms_norm_eps=1e-6, eos_token_id=-1, bos_token_id=-1, hf_model_type="lanilix", sandwich_norm=True, norm_offset=1.0, layers=tuple(
+                           dict(ff=14336, weights_of=i, act="clamped_glu", limit=7.0, alpha=1.702, **(
+                               dict(kind="window", sizes=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, window=4096, keep_first=4, rot_dim=64,
+                                                              rot_base=500000.0)) if i % 4 == 3 else
+                               dict(kind="delta", sizes=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4)))) for i in range(16))),
     "tiny-gpt2": dict(family="gpt2", vocab_size=512, hidden_size=128, intermediate_size=512, num_layers=2,
                       num_heads=4, num_kv_heads=4, max_position_embeddings=256, rms_norm_eps=1e-5,
                       tie_word_embeddings=True, eos_token_id=1, bos_token_id=2, pad_token_id=0),

@@ -21,16 +21,17 @@ CSRC = PKG / "csrc"
 BUILD = CSRC / "build"
 
 # One shared object per module.  ``_serve`` holds what a rollout engine of a mixer stack needs (scheduler, dense GEMMs, packed
-# attention, sampling, sequence mixers); ``_C`` the rest (training, decode kernels of the llama family, multi-GPU).  A kernel
+# attention, paged decode attention, sampling, sequence mixers); ``_C`` the rest (training, decode GEMMs, multi-GPU).  A kernel
 # object may be linked into both.
 MODULES: dict[str, dict] = {
     "_serve": {"bindings": "bindings_serve.cpp",
-               "cu": ["gemm_tcgen05.cu", "gemm2.cu", "attn_fwd.cu", "sampling.cu", "mix_elem.cu", "mix_scan.cu", "mix_chunk.cu", "mix_chunk_tc.cu", "mix_latent.cu"]},
+               "cu": ["gemm_tcgen05.cu", "gemm2.cu", "attn_fwd.cu", "decode_attn.cu", "sampling.cu", "mix_elem.cu", "mix_scan.cu", "mix_chunk.cu", "mix_chunk_tc.cu", "mix_delta.cu", "mix_latent.cu",
+                      "mix_window.cu"]},
     "_C": {"bindings": "bindings.cpp",
            "cu": ["gemm_tcgen05.cu", "gemm2.cu", "skinny_gemm.cu", "decode_gemm.cu", "vmm.cu", "linear_ce.cu", "ag_gemm.cu", "elementwise.cu",
-                  "optim.cu", "decode_attn.cu", "attn_bwd.cu", "attn_fwd.cu", "p2p.cu", "nvls.cu"]},
+                  "optim.cu", "attn_bwd.cu", "attn_fwd.cu", "p2p.cu", "nvls.cu"]},
 }
-HEADERS = ["common.cuh", "gemm_sm100.cuh", "gemm2_sm100.cuh", "mixers.cuh", "mix_params.hpp"]
+HEADERS = ["common.cuh", "gemm_sm100.cuh", "gemm2_sm100.cuh", "mixers.cuh", "mix_tc.cuh", "mix_params.hpp"]
 HOST_HEADERS = ["kv_manager.hpp", "scheduler.hpp", "bindings_common.hpp", "mix_params.hpp"]          # included by the bindings only
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
