@@ -68,7 +68,7 @@ mix_scan_kernel(ScanParams p) {
       kk = warp_sum(kk); qq = warp_sum(qq); kq = warp_sum(kq);
       if (lane == 0) { s_dot[b][0][w] = kk; s_dot[b][1][w] = qq; s_dot[b][2][w] = kq; }
       const float vv = col_ok ? to_f<T>(v[static_cast<int64_t>(t) * p.ldv + col]) : 0.f;
-      const float keep = expf(a_neg * softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0));
+      const float keep = decay_f(a_neg * softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0));
       const float beta = sigmoid_f(p.g1[static_cast<int64_t>(t) * p.ldg + h] + b1);
       __syncthreads();
       float ak = 0.f, aq = 0.f;
@@ -323,7 +323,7 @@ mix_delta_step_kernel(ScanParams p) {
   float vv[CPL];
 #pragma unroll
   for (int c = 0; c < CPL; ++c) vv[c] = ok ? to_f<T>(v[col + c]) : 0.f;
-  const float keep = expf(-expf(p.a_log[h]) * softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + (p.b0 ? p.b0[h] : 0.f)));
+  const float keep = decay_f(-expf(p.a_log[h]) * softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + (p.b0 ? p.b0[h] : 0.f)));
   const float beta = sigmoid_f(p.g1[static_cast<int64_t>(t) * p.ldg + h] + (p.b1 ? p.b1[h] : 0.f));
   __syncthreads();
   float ak[CPL], aq[CPL];

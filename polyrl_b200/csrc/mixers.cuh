@@ -65,6 +65,8 @@ template <class T>
 __device__ __forceinline__ float silu_t(float z) { return z * sigmoid_t<T>(z); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float logsigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// exp of x <= 0, to the last bit near 1: a slow decay is the distance from 1, and its rounding adds up over a sequence
+__device__ __forceinline__ float decay_f(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
 __device__ __forceinline__ float softcap_f(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));

@@ -3,7 +3,7 @@
 Random weights.  Prefill: packed prompts through ``RolloutEngine.extend`` (device time of the step); decode: the engine's CUDA-graph
 decode step; both timed with CUDA events after warm-up, weights (gigabytes) far larger than L2.  ``--kernels`` times the single kernels at
 the same layer sizes, with L2 flushed between iterations, against their roofline: the larger of bytes / measured copy bandwidth and
-FLOPs / measured bf16 GEMM rate.
+FLOPs / measured bf16 GEMM rate.  ``--serving-design`` picks the mixer stack.
 """
 from __future__ import annotations
 
@@ -22,15 +22,21 @@ def _peaks() -> tuple[float, float, str]:
     return 6.65e12, 1.59e15, "fallback"
 
 
-def models(layers: int) -> dict:
-    """The mixer stack and, at the same width, feed-forward width and depth, the llama and the latent-attention (MLA) stack."""
+def models(layers: int, design: str) -> dict:
+    """The mixer stack and its closest stacks at the same width, feed-forward width and depth: llama with latent attention (MLA) beside
+    ludesun, ludesun beside lanilix, llama beside both."""
     from ..models import ModelConfig, get_model_config
 
-    hy = get_model_config("ludesun-4b")
-    lay = tuple(dict(hy.layers[i % 4], weights_of=i) for i in range(layers))
+    def stack(name):
+        c = get_model_config(name)
+        return ModelConfig(**{**c.to_dict(), "num_layers": layers, "layers": tuple(dict(c.layers[i % 4], weights_of=i) for i in range(layers))})
+
+    hy = stack("ludesun-4b")
     base = dict(family="llama", vocab_size=hy.vocab_size, hidden_size=hy.hidden_size, intermediate_size=hy.intermediate_size, num_layers=layers, num_heads=32,
                 max_position_embeddings=16384, rope_theta=500000.0, rms_norm_eps=1e-5, eos_token_id=-1)
-    return {"ludesun": ModelConfig(**{**hy.to_dict(), "num_layers": layers, "layers": lay}),
+    if design == "lanilix":
+        return {"lanilix": stack("lanilix-4b"), "ludesun": hy, "llama": ModelConfig(**base, num_kv_heads=8)}
+    return {"ludesun": hy,
             "llama": ModelConfig(**base, num_kv_heads=8),
             "mla": ModelConfig(**base, num_kv_heads=32, attn_type="mla", q_lora_rank=1536, kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64,
                                v_head_dim=128)}
@@ -61,7 +67,7 @@ def run_models(args) -> list[dict]:
     dev, rows = torch.device("cuda"), []
     prefills = [(16, 1024), (2, 8192)]
     decodes = [(64, 1024), (128, 2048)]
-    for name, cfg in models(args.serving_layers).items():
+    for name, cfg in models(args.serving_layers, args.serving_design).items():
         w = TransformerWeights(cfg, device=dev, dtype=torch.bfloat16, init=True)
         n_params = cfg.num_params()
         for nseq, length in prefills:
@@ -104,36 +110,35 @@ def run_models(args) -> list[dict]:
     return rows
 
 
-def run_kernels(args) -> list[dict]:
-    from .. import ops
-    from ..models import get_model_config, mla
-    from ..ops import mixers as M
+class _Kernels:
+    """Times single kernels against their roofline and collects the rows."""
 
-    C = ops.ext()
-    dev, bf = torch.device("cuda"), torch.bfloat16
-    hbm, flops, kind = _peaks()
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    rows = []
+    def __init__(self, args):
+        self.dev, self.args, self.rows = torch.device("cuda"), args, []
+        self.hbm, self.flops, self.kind = _peaks()
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=self.dev)
 
-    def rnd(*s, dtype=bf, scale=1.0):
-        return (torch.randn(*s, device=dev) * scale).to(dtype)
+    def rnd(self, *s, dtype=torch.bfloat16, scale=1.0):
+        return (torch.randn(*s, device=self.dev) * scale).to(dtype)
 
-    def rec(name, like, shape, fn, nbytes, fl=0.0):
+    def rec(self, name, like, shape, fn, nbytes, fl=0.0):
         fn()                                                  # (sets kernel attributes, sizes workspaces)
         torch.cuda.synchronize()
         graph = torch.cuda.CUDAGraph()                        # launch latency of the Python wrappers stays out of the device time
         with torch.cuda.graph(graph):
             fn()
-        ms = _events(graph.replay, args.steps_serving, 3, flush)
+        ms = _events(graph.replay, self.args.steps_serving, 3, self.flush)
         del graph
-        roof = max(nbytes / hbm, fl / flops) * 1e3
-        rows.append({"kernel": name, "like": like, "shape": shape, "us": round(ms * 1e3, 1), "roofline_us": round(roof * 1e3, 1),
-                     "of_" + kind: round(roof / ms, 3)})
-        print(json.dumps(rows[-1]), flush=True)
+        roof = max(nbytes / self.hbm, fl / self.flops) * 1e3
+        self.rows.append({"kernel": name, "like": like, "shape": shape, "us": round(ms * 1e3, 1), "roofline_us": round(roof * 1e3, 1),
+                          "of_" + self.kind: round(roof / ms, 3)})
+        print(json.dumps(self.rows[-1]), flush=True)
 
-    W, FF = 4096, 14336
+    def batch(self, lens, start):
+        """(SpanBatch of equal spans behind ``start`` earlier tokens, pages of the pool)."""
+        from ..ops import mixers as M
 
-    def batch(lens, start, ctx=0):
+        dev = self.dev
         n, t = len(lens), sum(lens)
         cu = torch.tensor([0] + lens, dtype=torch.int32).cumsum(0).to(torch.int32)
         seq_of = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), torch.tensor(lens)).to(dev)
@@ -146,8 +151,103 @@ def run_kernels(args) -> list[dict]:
                            kv_slot=kv, kv_len=(pos + 1).int(), table=table, seq_of=seq_of if long else None, n_long=n if long else 0,
                            t_long=t if long else 0, max_long=max(lens) if long else 0, max_len=start + max(lens)), width * n + 1
 
-    for tag, lens, start in (("16 x 1024", [1024] * 16, 0), ("2 x 8192", [8192] * 2, 0), ("decode 128 @ 2048", [1] * 128, 2047)):
-        b, blocks = batch(lens, start)
+
+_SHAPES = (("16 x 1024", [1024] * 16, 0), ("2 x 8192", [8192] * 2, 0), ("decode 128 @ 2048", [1] * 128, 2047))
+
+
+def run_kernels_lanilix(args) -> list[dict]:
+    """Layer sizes of ``lanilix-4b``; ``like`` names the kernel of the same kind, ``existing:`` rows are those kernels."""
+    from .. import ops
+    from ..ops import mixers as M
+    from ..ops.attention import attention_varlen
+
+    C, K = ops.ext(), _Kernels(args)
+    dev, rnd, rec = K.dev, K.rnd, K.rec
+    W, FF = 4096, 14336
+    f32 = dict(device=dev, dtype=torch.float32)
+    for tag, lens, start in _SHAPES:
+        b, blocks = K.batch(lens, start)
+        t, n, L, dec = sum(lens), len(lens), lens[0], lens[0] == 1
+        # ---- recurrences
+        H, G, N, V = 32, 16, 128, 128
+        ch = 2 * G * N + H * V
+        cache = {"S": torch.zeros(n + 1, H, N, V, **f32)}
+        c = rnd(t, ch)
+        gates = M.Gates(rnd(t, H, dtype=torch.float32), rnd(t, H, dtype=torch.float32), torch.full((H,), -2.0, **f32), None, torch.linspace(-4, 1, H, **f32))
+        # per token and head: three products with the state, and half a chunk of 64 earlier tokens for each of K K', Q K', the solve and P U
+        rec("recurrence delta", "recurrence ssd", tag, lambda: M.scan(M.DELTA, c[:, :G * N], c[:, G * N:2 * G * N], c[:, 2 * G * N:], gates, N ** -0.5, cache, b),
+            t * (2 * G * N * 2 + 2 * H * V * 2 + 2 * H * 4) + (2 if dec else 1) * n * H * N * V * 4, 0 if dec else t * H * (6 * N * V + 64 * (2 * N + 2 * V)))
+        H2, V2, N2, G2 = 128, 64, 128, 8
+        cache2 = {"S": torch.zeros(n + 1, H2, N2, V2, **f32)}
+        q2, k2, v2 = rnd(t, G2 * N2), rnd(t, G2 * N2, scale=N2 ** -0.5), rnd(t, H2 * V2)
+        gates2 = M.Gates(rnd(t, H2, dtype=torch.float32), None, torch.full((H2,), -2.0, **f32), None, torch.linspace(-2, 1, H2, **f32), torch.ones(H2, **f32))
+        rec("existing: recurrence ssd", "recurrence ssd", tag, lambda: M.scan(M.SSD, q2, k2, v2, gates2, 1.0, cache2, b),
+            t * (2 * G2 * N2 * 2 + 2 * H2 * V2 * 2 + H2 * 4) + (2 if dec else 1) * n * H2 * N2 * V2 * 4, 0 if dec else t * H2 * (64 * (N2 + V2) + 4 * N2 * V2))
+        del cache2, q2, k2, v2, c
+        p = rnd(t, ch + H * V)
+        cw, cb, cst = torch.randn(4, ch, device=dev), torch.randn(ch, device=dev), torch.zeros(n + 1, 3, ch, device=dev, dtype=torch.bfloat16)
+        rec("conv + silu, no bias", "conv + silu", tag, lambda: M.conv_silu(p[:, :ch], cw, None, cst, b), t * ch * 4 + n * 6 * ch * 2)
+        rec("existing: conv + silu", "conv + silu", tag, lambda: M.conv_silu(p[:, :ch], cw, cb, cst, b), t * ch * 4 + n * 6 * ch * 2)
+        y, gn = rnd(t, H * V), torch.ones(H * V, device=dev)
+        rec("gated norm (silu last)", "gated norm", tag, lambda: M.gated_norm(y, p[:, ch:], gn, H, 1e-6, M.SILU_LAST), t * H * V * 6)
+        rec("existing: gated norm (gate first)", "gated norm", tag, lambda: M.gated_norm(y, p[:, ch:], gn, 8, 1e-6, M.SILU_FIRST), t * H * V * 6)
+        del cache, p, y
+        # ---- attention
+        H, G, D, rd = 32, 8, 128, 64
+        qk = rnd(t, (H + G) * D)
+        kp, vp = rnd(blocks, G, 16, D), rnd(blocks, G, 16, D)
+        wq, wk, freq = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev), M.rope_frequencies(rd, 5e5, dev)
+        rec("query / key norm, rotation, cache write", "latent rows", tag, lambda: M.qk_prep(qk, H, D, wq, wk, freq, kp, vp, b, 1e-6, not dec),
+            t * ((H + G) * D * 2 + (H + (2 if dec else 4) * G) * D * 2))
+        r, lr, qr = 512, 64, 1536
+        pool, a = rnd(blocks, 1, 16, r + lr), rnd(t, qr + r + lr)
+        w1, w2, fr = torch.ones(qr, device=dev), torch.ones(r, device=dev), M.rope_frequencies(lr, 1e4, dev)
+        rec("existing: latent rows", "latent rows", tag, lambda: M.latent_prep(a, w1, w2, fr, pool, b, 1e-5, not dec), t * ((qr + r + lr) * 4 + (0 if dec else (r + lr) * 2)))
+        del pool, a, qk
+        q = rnd(t, H, D)
+        k, v = (None, None) if dec else (rnd(t, G, D), rnd(t, G, D))
+        for window, keep in ((4096, 4), (512, 4)):
+            if dec:
+                seen = min(2048, window + keep)
+                rec(f"paged windowed attention, window {window}", "paged decode", tag,
+                    lambda: M.window_attention(q, kp, vp, b.table, None, b.kv_len, 0.088, window, keep, b.max_len), t * seen * G * D * 4)
+            else:
+                pairs = sum(min(i + 1, window + min(keep, max(0, i + 1 - window))) for i in range(L))
+                rec(f"packed windowed attention, window {window}", "packed attention", tag,
+                    lambda: M.window_attention_varlen(q, k, v, b.cu, b.cu, 0.088, window, keep), t * (2 * H + 2 * G) * D * 2, n * pairs * H * 4 * D)
+        if dec:
+            rec("existing: paged decode (GQA 32/8)", "paged decode", tag,
+                lambda: ops.paged_decode_attention(q.view(t, H * D), kp, vp, b.table, b.kv_len, H, G, D, 0.088, max_len=2048), t * 2048 * G * D * 4)
+        else:
+            rec("existing: attention_varlen (GQA 32/8)", "packed attention", tag, lambda: attention_varlen(q, k, v, b.cu, L, True, 0.088),
+                t * (2 * H + 2 * G) * D * 2, n * L * L / 2 * H * 4 * D)
+        del kp, vp, q, k, v
+        # ---- rows and feed-forward
+        x32, yb, wn, hb = torch.randn(t, W, device=dev), rnd(t, W), torch.ones(W, device=dev), rnd(t, W)
+        rec("norm + residual add + next norm", "norm + residual add", tag, lambda: M.norm_add_(yb, x32, wn, 1e-6, wn), t * W * 12)
+        rec("existing: norm + residual add", "norm + residual add", tag, lambda: M.norm_add_(yb, x32, wn, 1e-6), t * W * 12)
+        wb = torch.ones(W, device=dev, dtype=torch.bfloat16)
+        rec("existing: add_rmsnorm", "norm + residual add", tag, lambda: C.add_rmsnorm_(hb, yb, wb, 1e-5), t * W * 8)
+        gu = rnd(2 * FF, W, scale=W ** -0.5)
+        rec("gate / up + clamped glu", "gate / up + swiglu", tag, lambda: M.linear_clamped_glu(hb, gu, 7.0, 1.702), (t * W + 2 * FF * W + t * FF) * 2, 4.0 * t * W * FF)
+        rec("existing: gate / up + swiglu", "gate / up + swiglu", tag, lambda: ops.linear_swiglu(hb, gu), (t * W + 2 * FF * W + t * FF) * 2, 4.0 * t * W * FF)
+        emb, ids = rnd(128256, W), torch.randint(0, 128256, (t,), device=dev)
+        rec("embedding + norm", "norm + residual add", tag, lambda: M.embed(ids, emb, wn, 1e-6), t * W * 8)
+        del x32, yb, hb, gu, emb
+        torch.cuda.empty_cache()
+    return K.rows
+
+
+def run_kernels(args) -> list[dict]:
+    from .. import ops
+    from ..models import get_model_config, mla
+    from ..ops import mixers as M
+
+    C, K = ops.ext(), _Kernels(args)
+    dev, rnd, rec, bf = K.dev, K.rnd, K.rec, torch.bfloat16
+    W, FF = 4096, 14336
+    for tag, lens, start in _SHAPES:
+        b, blocks = K.batch(lens, start)
         t, n, dec = sum(lens), len(lens), lens[0] == 1
         st_rw = 2 if dec else 1
         # ---- recurrences
@@ -162,7 +262,7 @@ def run_kernels(args) -> list[dict]:
         ch = H * V + 2 * G * N
         rec("conv + silu", "rope", tag, lambda: M.conv_silu(xc[:, H * V:], cw, cb, cst, b), t * ch * 4 + n * 6 * ch * 2)
         y, z, gn = rnd(t, H * V), xc[:, :H * V], torch.ones(H * V, device=dev)
-        rec("gated norm (gate first)", "rmsnorm", tag, lambda: M.gated_norm(y, z, gn, 8, 1e-5, True), t * H * V * 6)
+        rec("gated norm (gate first)", "rmsnorm", tag, lambda: M.gated_norm(y, z, gn, 8, 1e-5, M.SILU_FIRST), t * H * V * 6)
         del cache, q, k, v, xc, y
         H, V, N = 8, 512, 256
         cache = {"S": torch.zeros(n + 1, H, N, V, device=dev), "n": torch.zeros(n + 1, H, N, device=dev), "m": torch.zeros(n + 1, H, device=dev)}
@@ -172,7 +272,7 @@ def run_kernels(args) -> list[dict]:
         rec("recurrence mlstm", "attention", tag, lambda: M.scan(M.MLSTM, p[:, :H * N], p[:, H * N:2 * H * N], p[:, 2 * H * N:2 * H * N + H * V], gates, N ** -0.5, cache, b),
             t * (2 * H * N * 2 + 2 * H * V * 2 + 2 * H * 4) + st_rw * n * H * N * V * 4, 0 if dec else t * H * (64 * (N + V) + 4 * N * V))
         y, gn = rnd(t, H * V), torch.ones(H * V, device=dev)
-        rec("gated norm (gate last)", "rmsnorm", tag, lambda: M.gated_norm(y, p[:, 2 * H * N + H * V:], gn, 8, 1e-5, False), t * H * V * 6)
+        rec("gated norm (gate last)", "rmsnorm", tag, lambda: M.gated_norm(y, p[:, 2 * H * N + H * V:], gn, 8, 1e-5, M.SIGMOID_LAST), t * H * V * 6)
         del cache, p, y
         # ---- latent attention
         H, d, rd, V, r, qr = 32, 128, 64, 128, 512, 1536
@@ -226,7 +326,7 @@ def run_kernels(args) -> list[dict]:
         rec("existing: rope (GQA 32/8)", "rope", tag, lambda: ops.apply_rope(qkv, b.pos, cos, sin, 32, 8, 128), t * 40 * 128 * 4)
         del x32, yb, hb, up, gu, qkv
         torch.cuda.empty_cache()
-    return rows
+    return K.rows
 
 
 @torch.no_grad()
@@ -236,7 +336,8 @@ def main(args) -> int:
         return 1
     args.steps_serving = max(5, args.steps)
     out = {"workload": "serving", "dtype": "bf16", "data": "random weights and tokens", "device": torch.cuda.get_device_name(), "peaks": _peaks()[2]}
-    out["kernels" if args.kernels else "models"] = run_kernels(args) if args.kernels else run_models(args)
+    kernels = {"ludesun": run_kernels, "lanilix": run_kernels_lanilix}[args.serving_design]
+    out["kernels" if args.kernels else "models"] = kernels(args) if args.kernels else run_models(args)
     if os.environ.get("BENCH_SERVING_OUT"):
         Path(os.environ["BENCH_SERVING_OUT"]).write_text(json.dumps(out, indent=1))
     print(json.dumps({k: v for k, v in out.items() if k not in ("kernels", "models")}), flush=True)
