@@ -40,7 +40,7 @@ int prl_mix_chunk_tc_ok(const prl::ScanParams*);
 int prl_mix_chunk_tc(const prl::ScanParams*, int, int32_t*, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
 int prl_mix_window(const prl::WindowParams*, int, cudaStream_t);
-int prl_mix_delta(const prl::ScanParams*, int64_t, void*, float*, int32_t*, cudaStream_t);
+int prl_mix_delta(const prl::ScanParams*, int64_t, int64_t, void*, float*, int32_t*, cudaStream_t);
 }
 
 namespace {
@@ -322,7 +322,7 @@ void mix_delta_chunk_(const at::Tensor& q, const at::Tensor& k, const at::Tensor
   const int64_t chunks = prl_mix_delta_chunks(v.size(0), p.spans);
   at::Tensor work = at::empty({chunks * p.H * prl_mix_delta_work_bytes()}, v.options().dtype(at::kByte));
   at::Tensor gates = at::empty({chunks * p.H * prl_mix_delta_gate_floats()}, v.options().dtype(at::kFloat));
-  check(prl_mix_delta(&p, chunks, work.data_ptr(), gates.data_ptr<float>(), p.counter + counter.numel() - 1, cur_stream()), "mix_delta_chunk");
+  check(prl_mix_delta(&p, v.size(0), chunks, work.data_ptr(), gates.data_ptr<float>(), p.counter + counter.numel() - 1, cur_stream()), "mix_delta_chunk");
 }
 
 // a [T, qr + r + rd] -> (normed query latent [T, qr], packed cache rows [T, r + rd] or empty); cache rows also go to pool[kvslot]

@@ -13,10 +13,12 @@
 // mix_delta_chunk_kernel  one CTA per (span, head, 128 value columns) marching over its chunks, all products transposed so that the value
 //                         columns are the 128 rows (TMEM lane = value column) and the tokens or state rows the columns:
 //                             carried = S_0^T [K | Q]^T     U^T = R^T T^T     own = U^T P^T     delta = (weighted U)^T K
-//                         The fp32 state lives in registers, thread (value column, half) owning half of the state rows, and is restaged as the
-//                         hi + lo operand once per chunk.  A chunk's outputs are written while the next chunk's first product runs.
+//                         The left operands (state, R, U) are staged from registers into TMEM, the right ones lie in shared memory.  The fp32
+//                         state lives in registers, thread (value column, half) owning half of the state rows, and is restaged once per chunk.
+//                         Warps 0-7 do that arithmetic; warp 8 issues the products of the chain and the loads (a chunk ahead), warp 9 the own part
+//                         and the stores.  A chunk's outputs are written while the next chunk's first products run.
 // Operands that are not bf16 by nature (S, R, U, T, P) enter the products as bf16 pairs hi + lo.
-// Every wait is bounded: on a timeout the CTA raises *err, stops computing, frees its TMEM and returns.
+// Every wait is bounded: on a timeout the CTA raises *err, runs out its chunks without waiting, loading or multiplying, frees its TMEM and returns.
 #include "mix_tc.cuh"
 
 namespace prl {
@@ -25,7 +27,7 @@ constexpr int kDc = 64;                        // tokens per chunk
 constexpr int kDcTile = 64 * 128;              // bytes of a 64 x 64 bf16 tile
 constexpr int kDcWork = 4 * kDcTile;           // workspace of one (chunk, head): T hi, T lo, P hi, P lo
 constexpr int kDcGates = 3 * kDc + 4;          // floats: carry of a key row, weight in the final state, carry of a query row, keep
-constexpr int kDpThreads = 128, kDcThreads = 256;
+constexpr int kDpThreads = 128, kDcThreads = 384;
 constexpr int kDpLd = 68;                      // row pitch of A in floats
 
 __device__ __forceinline__ int delta_chunk_base(const int32_t* cu, int s) { return cu[s] / kDc + s; }     // workspace rows of a span start here
@@ -52,8 +54,8 @@ __device__ __forceinline__ void delta_solve(const float* A, int c, float (&x)[kD
 template <int NB>
 __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p, uint8_t* work, float* gates, int32_t* err) {
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* tile = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));   // NB chunks of [64 Q rows; 64 K rows]
-  float* sA = reinterpret_cast<float*>(tile + NB * 2 * kDcTile);       // [2][64][kDpLd]
+  uint8_t* tile = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));   // NB chunks of [64 Q rows; 64 K rows],
+  float* sA = reinterpret_cast<float*>(tile + 4 * kDcTile);            // later P of two heads; [2][64][kDpLd], later T of two heads
   __shared__ float s_L[2][kDc], s_beta[2][kDc], s_rq[kDc], s_rk[kDc];
   __shared__ int s_span;
   __shared__ uint64_t bar;
@@ -156,10 +158,11 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
     }
     __syncthreads();
     const int t = r & 63;
+    const int64_t item = static_cast<int64_t>(b) * p.H + kh * p.rep + h0;
     for (int j = 0; j < pair; ++j) {
       const float Lt = s_L[j][t];
       if (r < kDc) {                                                   // P, row t
-        uint8_t* dst = work + (static_cast<int64_t>(b) * p.H + kh * p.rep + h0 + j) * kDcWork + 2 * kDcTile;
+        uint8_t* dst = tile + j * 2 * kDcTile;
         const float rq = s_rq[t];
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
@@ -188,18 +191,20 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
     }
     __syncthreads();
     const int j = r >> 6;
+    float x[kDc];
     if (j < pair) {
-      const int64_t item = static_cast<int64_t>(b) * p.H + kh * p.rep + h0 + j;
       const float Lt = s_L[j][t], end = s_L[j][kDc - 1], et = fast_exp2(Lt), rk = s_rk[t];
-      float* gt = gates + item * kDcGates;
+      float* gt = gates + (item + j) * kDcGates;
       gt[t] = et * rk;
       gt[kDc + t] = fast_exp2(end - Lt) * rk;
       gt[2 * kDc + t] = et * s_rq[t];
       if (t < 4) gt[3 * kDc + t] = fast_exp2(end);
-      float x[kDc];
       if (t < 32) delta_solve<0>(sA + j * kDc * kDpLd, t, x); else delta_solve<32>(sA + j * kDc * kDpLd, t, x);
+    }
+    __syncthreads();
+    if (j < pair) {                                                    // T over A, column t
       const float be = s_beta[j][t];
-      uint8_t* dst = work + item * kDcWork;
+      uint8_t* dst = reinterpret_cast<uint8_t*>(sA + j * kDc * kDpLd);
       const int unit = t >> 3, sub = (t & 7) * 2;
 #pragma unroll
       for (int i = 0; i < kDc; ++i) {
@@ -210,6 +215,16 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
         *reinterpret_cast<__nv_bfloat16*>(dst + kDcTile + at) = lo;
       }
     }
+    fence_proxy_async();
+    __syncthreads();
+    if (r == 0) {
+      for (int i = 0; i < pair; ++i) {
+        bulk_store(work + (item + i) * kDcWork, sA + i * kDc * kDpLd, 2 * kDcTile);
+        bulk_store(work + (item + i) * kDcWork + 2 * kDcTile, tile + i * 2 * kDcTile, 2 * kDcTile);
+      }
+      tma_store_commit();
+      if (h0 + 2 < p.rep) tma_store_wait_read<0>(); else tma_store_wait<0>();
+    }
     __syncthreads();
   }
 }
@@ -217,315 +232,396 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
 template <int NB>
 struct DeltaTc {
   static constexpr int NT = NB * kDcTile;                    // 64 tokens x N
-  static constexpr int ST = NB * 2 * kDcTile;                // 128 value columns x N
-  static constexpr int OFF_K = 2 * ST;                       // two buffers (S: hi, lo ahead of it)
-  static constexpr int OFF_Q = OFF_K + 2 * NT;
-  static constexpr int OFF_V = OFF_Q + NT;                   // 64 tokens x 128 value columns, plain rows
-  static constexpr int OFF_T = OFF_V + 2 * kDcTile;          // hi, lo
-  static constexpr int OFF_P = OFF_T + 2 * kDcTile;
-  static constexpr int OFF_R = OFF_P + 2 * kDcTile;          // R, then U: 128 x 64 hi, lo
-  static constexpr int OFF_W = OFF_R + 4 * kDcTile;          // weighted U: hi, lo
-  static constexpr int OFF_F = OFF_W + 4 * kDcTile;
+  static constexpr int VT = 2 * kDcTile;                     // 64 tokens x 128 value columns, plain rows
+  static constexpr int OFF_Q = 2 * NT;                       // everything but the outputs in two buffers
+  static constexpr int OFF_V = 4 * NT;
+  static constexpr int OFF_W = OFF_V + 2 * VT;               // T hi, T lo, P hi, P lo
+  static constexpr int OFF_O = OFF_W + 2 * kDcWork;
+  static constexpr int OFF_F = OFF_O + VT;
+  static constexpr uint32_t LOAD = 2 * NT + VT + kDcWork + kDcGates * 4;        // bytes of a chunk
 };
 struct DeltaShared {                                         // behind the tiles
-  float ck[2][kDc], wgt[2][kDc], cq[3][kDc];                 // (a chunk's query carries are read while the chunk after the next one loads)
-  float keep[2][4];
-  uint64_t bar[5];
+  float gates[3][kDcGates];                                  // (a chunk's query carries are read while the chunk after the next one loads)
+  uint64_t carried, writes, delta, own, full[2];             // products done: S_0^T K, U, the state's increment, U P; a chunk has arrived
   uint32_t tmem;
+  int fail;
 };
+static_assert(kDcGates * 4 % 16 == 0, "copied in 16-byte units");
+// warps 0-7 hand over to warp 8 (state, R, weighted U) and warp 9 (U, outputs); at state and outputs they wait too, which keeps all in one chunk
+enum : int { kBarState = 1, kBarR, kBarW, kBarU, kBarOut };
+constexpr int kDcHandoff = 288;
+// 12 warps x 168 registers at launch = 8 x 216 + 4 x 72
+constexpr int kDcRegsMath = 216, kDcRegsIo = 72;
+static_assert(8 * kDcRegsMath + 4 * kDcRegsIo <= 12 * 168, "register split");
+
+__device__ __forceinline__ void delta_arrive(int id) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "n"(kDcHandoff) : "memory"); }
+__device__ __forceinline__ void delta_sync(int id) { asm volatile("bar.sync %0, %1;" ::"r"(id), "n"(kDcHandoff) : "memory"); }
+__device__ __forceinline__ void delta_wait(DeltaShared& sm, uint64_t* bar, uint32_t parity) {
+  if (*reinterpret_cast<volatile int*>(&sm.fail)) return;
+  if (!tc_wait(bar, parity)) *reinterpret_cast<volatile int*>(&sm.fail) = 1;
+}
+// C values of a row as bf16 pairs: hi + lo
+template <int C>
+__device__ __forceinline__ void delta_stage(uint32_t hi_at, uint32_t lo_at, const float* x) {
+#pragma unroll
+  for (int c = 0; c < C; c += 32) {
+    uint32_t hi[16], lo[16];
+#pragma unroll
+    for (int e = 0; e < 16; ++e) tc_split(x[c + 2 * e], x[c + 2 * e + 1], hi[e], lo[e]);
+    tmem_st_32x16(hi_at + c / 2, hi);
+    tmem_st_32x16(lo_at + c / 2, lo);
+  }
+}
 
 template <int NB>
 __global__ void __launch_bounds__(kDcThreads, 1)
-mix_delta_chunk_kernel(ScanParams p, const uint8_t* work, const float* gates, int32_t* err) {
+mix_delta_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmO,
+                       ScanParams p, const uint8_t* work, const float* gates, int32_t* err) {
   using Cfg = DeltaTc<NB>;
   constexpr int OWN = NB * 32;                               // state rows per thread
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t *sS = smem, *sQ = smem + Cfg::OFF_Q, *sV = smem + Cfg::OFF_V, *sT = smem + Cfg::OFF_T, *sP = smem + Cfg::OFF_P, *sR = smem + Cfg::OFF_R,
-          *sW = smem + Cfg::OFF_W;
+  uint8_t* sO = smem + Cfg::OFF_O;
   DeltaShared& sm = *reinterpret_cast<DeltaShared*>(smem + Cfg::OFF_F);
   const int h = blockIdx.y, s = blockIdx.z, v0 = blockIdx.x * 128;
-  const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, quad = w & 3, g = w >> 2, r = quad * 32 + lane;
+  const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
   const int t0 = p.cu[s], len = p.cu[s + 1] - t0;
   if (len <= 0) return;
   const bool fresh = p.start[s] == 0;
   const int N = p.N, V = p.V, vn = min(128, V - v0);
-  const __nv_bfloat16* gQ = static_cast<const __nv_bfloat16*>(p.q) + static_cast<int64_t>(t0) * p.ldq + static_cast<int64_t>(h / p.rep) * N;
-  const __nv_bfloat16* gK = static_cast<const __nv_bfloat16*>(p.k) + static_cast<int64_t>(t0) * p.ldk + static_cast<int64_t>(h / p.rep) * N;
-  const __nv_bfloat16* gV = static_cast<const __nv_bfloat16*>(p.v) + static_cast<int64_t>(t0) * p.ldv + static_cast<int64_t>(h) * V + v0;
-  __nv_bfloat16* gO = static_cast<__nv_bfloat16*>(p.out) + static_cast<int64_t>(t0) * p.ldo + static_cast<int64_t>(h) * V + v0 + r;
-  float* gS = p.S + (p.slot[s] * p.H + h) * static_cast<int64_t>(N) * V + v0 + r;
-  const int64_t item0 = static_cast<int64_t>(delta_chunk_base(p.cu, s)) * p.H + h;
   const int chunks = (len + kDc - 1) / kDc;
-
-  auto load_k = [&](int ci) {                                // keys and gates of a chunk
-    const int nv = min(kDc, len - ci * kDc);
-#pragma unroll
-    for (int i = 0; i < NB; ++i)
-      tc_load_rows<kDc, kDcThreads>(smem + Cfg::OFF_K + (ci & 1) * Cfg::NT + i * kDcTile, gK + static_cast<int64_t>(ci) * kDc * p.ldk, p.ldk, nv, i * 64, N);
-    const float* gt = gates + (item0 + static_cast<int64_t>(ci) * p.H) * kDcGates;
-    if (tid < 16) tc_cp16(&sm.ck[ci & 1][tid * 4], gt + tid * 4, true);
-    else if (tid < 32) tc_cp16(&sm.wgt[ci & 1][(tid - 16) * 4], gt + kDc + (tid - 16) * 4, true);
-    else if (tid < 48) tc_cp16(&sm.cq[ci % 3][(tid - 32) * 4], gt + 2 * kDc + (tid - 32) * 4, true);
-    else if (tid == 48) tc_cp16(sm.keep[ci & 1], gt + 3 * kDc, true);
-  };
-  auto load_q = [&](int ci) {
-    const int nv = min(kDc, len - ci * kDc);
-#pragma unroll
-    for (int i = 0; i < NB; ++i) tc_load_rows<kDc, kDcThreads>(sQ + i * kDcTile, gQ + static_cast<int64_t>(ci) * kDc * p.ldq, p.ldq, nv, i * 64, N);
-  };
-  auto load_v = [&](int ci) {
-    const int nv = min(kDc, len - ci * kDc);
-    const __nv_bfloat16* src = gV + static_cast<int64_t>(ci) * kDc * p.ldv;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int idx = tid + i * kDcThreads, t = idx >> 4, c = (idx & 15) * 8;
-      const bool ok = t < nv && c < vn;
-      tc_cp16(sV + t * 256 + c * 2, src + (ok ? static_cast<int64_t>(t) * p.ldv + c : 0), ok);
-    }
-  };
-  auto load_pair = [&](uint8_t* dst, int ci, int which) {    // 0: T, 1: P
-    const uint8_t* src = work + (item0 + static_cast<int64_t>(ci) * p.H) * kDcWork + which * 2 * kDcTile;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) tc_cp16(dst + (tid + i * kDcThreads) * 16, src + (tid + i * kDcThreads) * 16, true);
-  };
-
-  load_k(0);
-  load_q(0);
-  load_v(0);
-  tc_cp_commit();
-  load_pair(sT, 0, 0);
-  tc_cp_commit();
   if (tid == 0) {
-    for (int i = 0; i < 5; ++i) mbar_init(&sm.bar[i], 1);
+    mbar_init(&sm.carried, 1);
+    mbar_init(&sm.writes, 1);
+    mbar_init(&sm.delta, 1);
+    mbar_init(&sm.own, 1);
+    mbar_init(&sm.full[0], 1);
+    mbar_init(&sm.full[1], 1);
+    sm.fail = 0;
     fence_barrier_init();
   }
-  if (w == 0) { tmem_alloc(&sm.tmem, 512); tmem_relinquish(); }
-
-  float S[OWN];                                              // state rows g * OWN + i of value column r
-#pragma unroll
-  for (int i = 0; i < OWN; ++i) {
-    const int n = g * OWN + i;
-    S[i] = (!fresh && n < N && r < vn) ? gS[static_cast<int64_t>(n) * V] : 0.f;
-  }
-  auto stage_state = [&]() {
-#pragma unroll
-    for (int u = 0; u < OWN / 8; ++u) {
-      uint32_t hi[4], lo[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) tc_split(S[u * 8 + 2 * e], S[u * 8 + 2 * e + 1], hi[e], lo[e]);
-      const int n = g * OWN + u * 8;
-      tc_st16(sS + (n >> 6) * 2 * kDcTile, r, (n & 63) >> 3, hi);
-      tc_st16(sS + Cfg::ST + (n >> 6) * 2 * kDcTile, r, (n & 63) >> 3, lo);
-    }
-  };
-  bool have_state = !fresh, ok = true;
-  if (have_state) stage_state();
+  if (w == 8) { tmem_alloc(&sm.tmem, 512); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = sm.tmem, tK = tmem, tQ = tmem + 64, tU = tmem + 192, tO = tmem + 256, tD = tmem + 320;
-  const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
-  constexpr uint32_t idKK = umma_idesc(128, kDc, 1, 1);
-  constexpr uint32_t idKM = umma_idesc_major(128, NB * 64, 1, 1, 0, 1);
+  // TMEM columns.  State operand of half g: hi at tS + g * OWN, lo behind it; the state's increment uses the same columns once the operand is
+  // spent, row by row where the thread that reads it stages its next operand.  U overwrites R, and its accumulator that of the carried keys.
+  const uint32_t tS = sm.tmem, tR = tS + 128, tW = tS + 192, tK = tS + 256, tQ = tS + 320, tO = tS + 448;
 
-  // y of chunk ci: columns are its tokens, this thread's half
-  auto write_out = [&](int ci, bool carried) {
-    uint32_t a[32], b[32];
-    __syncwarp();
-    tmem_ld_32x32(tO + lanes + g * 32, a);
-    if (carried) tmem_ld_32x32(tQ + (ci & 1) * 64 + lanes + g * 32, b);
-    tmem_ld_wait();
-    const int nv = min(kDc, len - ci * kDc) - g * 32;
-    const float* cq = sm.cq[ci % 3] + g * 32;
-    __nv_bfloat16* dst = gO + (static_cast<int64_t>(ci) * kDc + g * 32) * p.ldo;
-    if (r < vn) {
+  if (w >= 8) {
+    // ================================ products, loads, stores ================================
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kDcRegsIo));
+    constexpr uint32_t idKK = umma_idesc(128, kDc, 1, 1);
+    // D [128 x 64] = (A hi + A lo) (B hi + B lo)^T over the chunk's tokens, without lo lo
+    auto mma_pairs = [&](uint32_t d, const uint8_t* b) {
+      const uint64_t desc = umma_desc_sw128_kmajor(b);
 #pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const float y = __uint_as_float(a[i]) + (carried ? cq[i] * __uint_as_float(b[i]) : 0.f);
-        if (i < nv) dst[i * p.ldo] = __float2bfloat16(y);
+      for (int kk = 0; kk < 4; ++kk) {
+        umma_bf16_ts(d, tR + kk * 8, desc + 2 * kk, idKK, kk != 0);
+        umma_bf16_ts(d, tR + 32 + kk * 8, desc + 2 * kk, idKK, 1);
+        umma_bf16_ts(d, tR + kk * 8, desc + (kDcTile >> 4) + 2 * kk, idKK, 1);
       }
+    };
+    if (w == 9) {
+      __nv_bfloat16* gO = static_cast<__nv_bfloat16*>(p.out) + static_cast<int64_t>(t0) * p.ldo + static_cast<int64_t>(h) * V + v0;
+      auto store = [&](int ci) {
+        if (*reinterpret_cast<volatile int*>(&sm.fail)) return;
+        const int nv = len - ci * kDc;
+        if (nv >= kDc) {
+          if (lane == 0) tma_store_3d(&tmO, sO, v0, h, t0 + ci * kDc);
+        } else {                                             // a row at a time: the next rows are another span's
+          for (int t = lane; t < nv; t += 32) bulk_store(gO + (static_cast<int64_t>(ci) * kDc + t) * p.ldo, sO + t * 256, vn * 2);
+        }
+        tma_store_commit();
+      };
+      for (int ci = 0; ci < chunks; ++ci) {
+        if (ci > 0) {
+          delta_sync(kBarOut);
+          store(ci - 1);
+        }
+        delta_sync(kBarU);
+        tma_store_wait_read<0>();                            // (`own` also tells that sO is free)
+        __syncwarp();
+        if (lane == 0 && !*reinterpret_cast<volatile int*>(&sm.fail)) {
+          tc_fence_after();
+          mma_pairs(tO, smem + Cfg::OFF_W + (ci & 1) * kDcWork + 2 * kDcTile);
+          umma_commit(&sm.own);
+        }
+        __syncwarp();
+      }
+      delta_sync(kBarOut);
+      store(chunks - 1);
+      tma_store_wait<0>();
+    } else if (w == 8) {
+    constexpr uint32_t idKM = umma_idesc_major(128, NB * 64, 1, 1, 0, 1);
+    const int64_t item0 = static_cast<int64_t>(delta_chunk_base(p.cu, s)) * p.H + h;
+    auto load = [&](int ci) {
+      const int bf = ci & 1, t = t0 + ci * kDc;
+      const int64_t item = item0 + static_cast<int64_t>(ci) * p.H;
+      uint64_t* bar = &sm.full[bf];
+      mbar_expect_tx(bar, Cfg::LOAD);
+#pragma unroll
+      for (int c = 0; c < NB; ++c) tma_load_3d(&tmK, bar, smem + bf * Cfg::NT + c * kDcTile, c * 64, h / p.rep, t);
+#pragma unroll
+      for (int c = 0; c < NB; ++c) tma_load_3d(&tmQ, bar, smem + Cfg::OFF_Q + bf * Cfg::NT + c * kDcTile, c * 64, h / p.rep, t);
+      tma_load_3d(&tmV, bar, smem + Cfg::OFF_V + bf * Cfg::VT, v0, h, t);
+      bulk_load(bar, smem + Cfg::OFF_W + bf * kDcWork, work + item * kDcWork, kDcWork);
+      bulk_load(bar, sm.gates[ci % 3], gates + item * kDcGates, kDcGates * 4);
+    };
+    // D [128 x 64] = S_0^T X^T, X = keys or queries of the chunk
+    auto mma_state = [&](uint32_t d, const uint8_t* x) {
+      const uint64_t desc = umma_desc_sw128_kmajor(x);
+#pragma unroll
+      for (int kk = 0; kk < NB * 4; ++kk) {
+        const uint32_t a = tS + (kk * 16 / OWN) * OWN + (kk * 16 % OWN) / 2;
+        const uint64_t b = desc + (kk >> 2) * (kDcTile >> 4) + 2 * (kk & 3);
+        umma_bf16_ts(d, a, b, idKK, kk != 0);
+        umma_bf16_ts(d, a + OWN / 2, b, idKK, 1);
+      }
+    };
+    int loaded = 0;
+    if (lane == 0) {
+      tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
+      load(0);
+      loaded = 1;
     }
-  };
-  // 32 values of row r as hi + lo, columns g * 32 ...
-  auto stage_half = [&](uint8_t* tile, const float (&x)[32]) {
+    for (int ci = 0; ci < chunks; ++ci) {
+      const uint32_t ph = ci & 1, fph = (ci >> 1) & 1;
+      uint8_t *sK = smem + ph * Cfg::NT, *sT = smem + Cfg::OFF_W + ph * kDcWork;
+      if (lane == 0) delta_wait(sm, &sm.full[ph], fph);
+      __syncwarp();
+      const int nv = len - ci * kDc;
+      if (nv < kDc) {                                        // the tile's last rows are another span's tokens
+        for (int i = lane; i < (kDc - nv) * 8 * NB; i += 32) {
+          const int row = nv + i / (8 * NB), at = (i % (8 * NB) / 8) * kDcTile + row * 128 + (i % 8) * 16;
+          *reinterpret_cast<uint4*>(sK + at) = make_uint4(0, 0, 0, 0);
+          *reinterpret_cast<uint4*>(sK + Cfg::OFF_Q + at) = make_uint4(0, 0, 0, 0);
+        }
+        fence_proxy_async();
+      }
+      __syncwarp();
+      delta_sync(kBarState);
+      const bool run = !*reinterpret_cast<volatile int*>(&sm.fail);
+      if (lane == 0 && run) {
+        tc_fence_after();
+        const bool have_state = ci > 0 || !fresh;
+        if (have_state) mma_state(tK, sK);
+        umma_commit(&sm.carried);
+        if (have_state) mma_state(tQ + ph * 64, sK + Cfg::OFF_Q);
+        if (ci > 0) delta_wait(sm, &sm.own, ph ^ 1);        // the last reader of the buffers that fill next
+        if (ci + 1 < chunks) { load(ci + 1); ++loaded; }
+      }
+      __syncwarp();
+      delta_sync(kBarR);
+      if (lane == 0 && run) {
+        tc_fence_after();
+        mma_pairs(tK, sT);
+        umma_commit(&sm.writes);
+      }
+      __syncwarp();
+      delta_sync(kBarW);
+      if (lane == 0 && run) {
+        tc_fence_after();
+        const uint64_t desc = umma_desc_sw128_mnmajor(sK, kDcTile);
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      uint32_t hi[4], lo[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) tc_split(x[u * 8 + 2 * e], x[u * 8 + 2 * e + 1], hi[e], lo[e]);
-      tc_st16(tile, r, g * 4 + u, hi);
-      tc_st16(tile + 2 * kDcTile, r, g * 4 + u, lo);
+        for (int kk = 0; kk < 4; ++kk) {
+          umma_bf16_ts(tS, tW + kk * 8, desc + kk * 128, idKM, kk != 0);
+          umma_bf16_ts(tS, tW + 32 + kk * 8, desc + kk * 128, idKM, 1);
+        }
+        umma_commit(&sm.delta);
+      }
+      __syncwarp();
     }
-  };
-  // D[128 x 64] = (A hi + A lo) (B hi + B lo)^T over 64, without lo lo; both K-major
-  auto mma_pairs = [&](uint32_t d, const uint8_t* a, const uint8_t* b) {
+    delta_sync(kBarState);                                   // (after the last chunk: every wait of the others is over)
+    if (*reinterpret_cast<volatile int*>(&sm.fail) && lane == 0) {
+      atomicExch(err, 1);                                    // copies in flight end before the shared memory is given up
+      if (loaded > 0) tc_wait(&sm.full[0], ((loaded + 1) / 2 - 1) & 1);
+      if (loaded > 1) tc_wait(&sm.full[1], (loaded / 2 - 1) & 1);
+    }
+    __syncwarp();
+    }
+  } else {
+    // ================================ warps 0-7: state, R, U and outputs ================================
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kDcRegsMath));
+    const int quad = w & 3, g = w >> 2, r = quad * 32 + lane;          // value column, half of the state rows or tokens
+    const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
+    float* gS = p.S + (p.slot[s] * p.H + h) * static_cast<int64_t>(N) * V + v0 + r;
+    float S[OWN];                                            // state rows g * OWN + i
 #pragma unroll
-    for (int c = 0; c < 3; ++c)
+    for (int i = 0; i < OWN; ++i) {
+      const int n = g * OWN + i;
+      S[i] = (!fresh && n < N && r < vn) ? gS[static_cast<int64_t>(n) * V] : 0.f;
+    }
+    auto stage_state = [&]() { delta_stage<OWN>(tS + lanes + g * OWN, tS + lanes + g * OWN + OWN / 2, S); };
+    bool have_state = !fresh, carried_prev = false;
+    if (have_state) stage_state();
+    auto stage_out = [&](int ci, bool carried) {             // y of chunk ci, this thread's half of its tokens
+      uint32_t a[32], b[32];
+      __syncwarp();
+      tmem_ld_32x32(tO + lanes + g * 32, a);
+      if (carried) tmem_ld_32x32(tQ + (ci & 1) * 64 + lanes + g * 32, b);
+      tmem_ld_wait();
+      const float* cq = sm.gates[ci % 3] + 2 * kDc + g * 32;
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(sO) + g * 32 * 128 + r;
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk)
-        umma_bf16_ss(d, umma_desc_sw128_kmajor(a + (c == 1 ? 2 * kDcTile : 0)) + 2 * kk, umma_desc_sw128_kmajor(b + (c == 2 ? kDcTile : 0)) + 2 * kk, idKK,
-                     (c | kk) != 0);
-  };
-  bool carried_prev = false;
+      for (int i = 0; i < 32; i += 4) {
+        const float4 c = *reinterpret_cast<const float4*>(cq + i);
+        const float cc[4] = {c.x, c.y, c.z, c.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          dst[(i + e) * 128] = __float2bfloat16(__uint_as_float(a[i + e]) + (carried ? cc[e] * __uint_as_float(b[i + e]) : 0.f));
+      }
+    };
 
-  for (int ci = 0; ci < chunks; ++ci) {
-    const uint32_t ph = ci & 1;
-    const bool more = ci + 1 < chunks;
-    const uint8_t* sK = smem + Cfg::OFF_K + (ci & 1) * Cfg::NT;
-    tc_cp_wait<1>();                                         // keys, gates, queries and values; T may still be on its way
-    fence_proxy_async();
-    tc_fence_before();
-    if (__syncthreads_or(!ok)) {
-      if (tid == 0) atomicExch(err, 1);
-      ok = false;
-      break;
-    }
-    if (tid == 0) {
-      tc_fence_after();
-      if (have_state) {
-#pragma unroll
-        for (int hl = 0; hl < 2; ++hl)
-#pragma unroll
-          for (int kk = 0; kk < NB * 4; ++kk)
-            umma_bf16_ss(tK, umma_desc_sw128_kmajor(sS + hl * Cfg::ST + (kk >> 2) * 2 * kDcTile) + 2 * (kk & 3),
-                         umma_desc_sw128_kmajor(sK + (kk >> 2) * kDcTile) + 2 * (kk & 3), idKK, (hl | kk) != 0);
+    for (int ci = 0; ci < chunks; ++ci) {
+      const uint32_t ph = ci & 1, fph = (ci >> 1) & 1;
+      const float* gt = sm.gates[ci % 3];
+      tmem_st_wait();
+      tc_fence_before();
+      delta_sync(kBarState);
+      if (ci > 0) {
+        delta_wait(sm, &sm.own, ph ^ 1);
+        tc_fence_after();
+        stage_out(ci - 1, carried_prev);
+        fence_proxy_async();
+        delta_sync(kBarOut);
       }
-      umma_commit(&sm.bar[0]);
-      if (have_state) {
-#pragma unroll
-        for (int hl = 0; hl < 2; ++hl)
-#pragma unroll
-          for (int kk = 0; kk < NB * 4; ++kk)
-            umma_bf16_ss(tQ + (ci & 1) * 64, umma_desc_sw128_kmajor(sS + hl * Cfg::ST + (kk >> 2) * 2 * kDcTile) + 2 * (kk & 3),
-                         umma_desc_sw128_kmajor(sQ + (kk >> 2) * kDcTile) + 2 * (kk & 3), idKK, (hl | kk) != 0);
-      }
-      umma_commit(&sm.bar[1]);
-    }
-    __syncwarp();
-    if (more) load_k(ci + 1);
-    tc_cp_commit();
-    if (ci > 0) {
-      ok = tc_wait(&sm.bar[4], ph ^ 1) && ok;
+      carried_prev = have_state;
+      delta_wait(sm, &sm.full[ph], fph);
+      delta_wait(sm, &sm.carried, ph);
       tc_fence_after();
-      write_out(ci - 1, carried_prev);
-    }
-    load_pair(sP, ci, 1);                                    // (its reader, the own part of the previous chunk, is done)
-    tc_cp_commit();
-    carried_prev = have_state;
-    ok = tc_wait(&sm.bar[0], ph) && ok;
-    tc_fence_after();
-    {                                                        // R = v - carry_t S_0^T k_t  (T holds beta)
-      float x[32];
-      uint32_t d[32];
-      if (have_state) {
+      {                                                      // R = v - carry_t S_0^T k_t  (T holds beta)
+        float x[32];
+        uint32_t d[32];
+        if (have_state) {
+          __syncwarp();
+          tmem_ld_32x32(tK + lanes + g * 32, d);
+          tmem_ld_wait();
+        }
+        const float* ck = gt + g * 32;
+        const uint8_t* vv = smem + Cfg::OFF_V + ph * Cfg::VT + g * 32 * 256 + r * 2;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4) {
+          const float4 c = *reinterpret_cast<const float4*>(ck + i);
+          const float cc[4] = {c.x, c.y, c.z, c.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float v = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(vv + (i + e) * 256));
+            x[i + e] = have_state ? v - cc[e] * __uint_as_float(d[i + e]) : v;
+          }
+        }
+        const int nv = len - ci * kDc - g * 32;
+        if (nv < 32) {                                       // rows of another span
+#pragma unroll
+          for (int i = 0; i < 32; ++i) x[i] = i < nv ? x[i] : 0.f;
+        }
+        __syncwarp();
+        delta_stage<32>(tR + lanes + g * 16, tR + lanes + 32 + g * 16, x);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      delta_arrive(kBarR);
+      delta_wait(sm, &sm.writes, ph);
+      tc_fence_after();
+      {                                                      // U, weighted by its part in the final state and as it is
+        uint32_t d[32];
         __syncwarp();
         tmem_ld_32x32(tK + lanes + g * 32, d);
         tmem_ld_wait();
+        float x[32];
+        const float* wg = gt + kDc + g * 32;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4) {
+          const float4 c = *reinterpret_cast<const float4*>(wg + i);
+          x[i] = __uint_as_float(d[i]) * c.x; x[i + 1] = __uint_as_float(d[i + 1]) * c.y;
+          x[i + 2] = __uint_as_float(d[i + 2]) * c.z; x[i + 3] = __uint_as_float(d[i + 3]) * c.w;
+        }
+        delta_stage<32>(tW + lanes + g * 16, tW + lanes + 32 + g * 16, x);
+        tmem_st_wait();
+        tc_fence_before();
+        delta_arrive(kBarW);
+#pragma unroll
+        for (int i = 0; i < 32; ++i) x[i] = __uint_as_float(d[i]);
+        delta_stage<32>(tR + lanes + g * 16, tR + lanes + 32 + g * 16, x);
       }
-      const float* ck = sm.ck[ci & 1] + g * 32;
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const float v = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sV + (g * 32 + i) * 256 + r * 2));
-        x[i] = have_state ? v - ck[i] * __uint_as_float(d[i]) : v;
-      }
-      stage_half(sR, x);
-    }
-    tc_cp_wait<2>();                                         // T
-    fence_proxy_async();
-    tc_fence_before();
-    __syncthreads();
-    if (tid == 0) {
-      tc_fence_after();
-      mma_pairs(tU, sR, sT);
-      umma_commit(&sm.bar[2]);
-    }
-    __syncwarp();
-    ok = tc_wait(&sm.bar[1], ph) && ok;
-    if (more) load_q(ci + 1);
-    tc_cp_commit();
-    if (more) load_v(ci + 1);
-    tc_cp_commit();
-    ok = tc_wait(&sm.bar[2], ph) && ok;
-    tc_fence_after();
-    {                                                        // U, and U weighted by its part in the final state
-      uint32_t d[32];
-      __syncwarp();
-      tmem_ld_32x32(tU + lanes + g * 32, d);
-      tmem_ld_wait();
-      float x[32];
-#pragma unroll
-      for (int i = 0; i < 32; ++i) x[i] = __uint_as_float(d[i]);
-      stage_half(sR, x);
-      const float* wg = sm.wgt[ci & 1] + g * 32;
-#pragma unroll
-      for (int i = 0; i < 32; ++i) x[i] *= wg[i];
-      stage_half(sW, x);
-    }
-    tc_cp_wait<2>();                                         // P
-    fence_proxy_async();
-    tc_fence_before();
-    __syncthreads();
-    if (tid == 0) {
+      tmem_st_wait();
+      tc_fence_before();
+      delta_arrive(kBarU);
+      const float keep = gt[3 * kDc];
+      delta_wait(sm, &sm.delta, ph);
       tc_fence_after();
 #pragma unroll
-      for (int hl = 0; hl < 2; ++hl)
+      for (int c = 0; c < OWN; c += 32) {
+        uint32_t d[32];
+        __syncwarp();
+        tmem_ld_32x32(tS + lanes + g * OWN + c, d);
+        tmem_ld_wait();
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk)
-          umma_bf16_ss(tD, umma_desc_sw128_kmajor(sW + hl * 2 * kDcTile) + 2 * kk, umma_desc_sw128_mnmajor(sK, kDcTile) + kk * 128, idKM, (hl | kk) != 0);
-      umma_commit(&sm.bar[3]);
-      mma_pairs(tO, sR, sP);
-      umma_commit(&sm.bar[4]);
+        for (int i = 0; i < 32; ++i) S[c + i] = keep * S[c + i] + __uint_as_float(d[i]);
+      }
+      have_state = true;
+      if (ci + 1 < chunks) stage_state();
     }
-    __syncwarp();
-    if (more) load_pair(sT, ci + 1, 0);
-    tc_cp_commit();
-    const float keep = sm.keep[ci & 1][0];
-    ok = tc_wait(&sm.bar[3], ph) && ok;
+    tmem_st_wait();
+    delta_wait(sm, &sm.own, (chunks - 1) & 1);
     tc_fence_after();
+    stage_out(chunks - 1, carried_prev);
+    fence_proxy_async();
+    delta_sync(kBarOut);
+    delta_sync(kBarState);
+    if (!*reinterpret_cast<volatile int*>(&sm.fail) && r < vn) {
+      int64_t ld = V;
+      asm volatile("" : "+l"(gS), "+l"(ld));                 // (addresses are computed again, not kept across the loop)
+      float* dst = gS + g * OWN * ld;
 #pragma unroll
-    for (int c = 0; c < OWN; c += 32) {
-      uint32_t d[32];
-      __syncwarp();
-      tmem_ld_32x32(tD + lanes + g * OWN + c, d);
-      tmem_ld_wait();
-#pragma unroll
-      for (int i = 0; i < 32; ++i) S[c + i] = keep * S[c + i] + __uint_as_float(d[i]);
-    }
-    have_state = true;
-    if (more) stage_state();
-  }
-  tc_cp_wait<0>();
-  ok = ok && tc_wait(&sm.bar[4], (chunks - 1) & 1);
-  if (__syncthreads_or(!ok)) {
-    if (tid == 0) atomicExch(err, 1);
-  } else {
-    tc_fence_after();
-    write_out(chunks - 1, carried_prev);
-    if (r < vn) {
-#pragma unroll
-      for (int i = 0; i < OWN; ++i)
-        if (g * OWN + i < N) gS[static_cast<int64_t>(g * OWN + i) * V] = S[i];
+      for (int i = 0; i < OWN; ++i, dst += ld)
+        if (g * OWN + i < N) *dst = S[i];
     }
   }
   tc_fence_before();
   __syncthreads();
-  if (w == 0) { tc_fence_after(); tmem_dealloc(sm.tmem, 512); }
+  if (w == 8) { tc_fence_after(); tmem_dealloc(sm.tmem, 512); }
+}
+
+using DeltaEncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                   const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// rows [tokens, heads * width] of pitch ld -> boxes of 64 tokens x 1 head x box columns, zeros beyond the head's width
+static int delta_tmap(CUtensorMap* m, const void* ptr, int64_t tokens, int heads, int width, int64_t ld, int box, bool swizzle) {
+  ensure_thread_ctx();
+  static DeltaEncodeFn fn = nullptr;
+  if (!fn) {
+    void* q = nullptr;
+    cudaDriverEntryPointQueryResult qr;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &q, cudaEnableDefault, &qr) != cudaSuccess || !q) return -1;
+    fn = reinterpret_cast<DeltaEncodeFn>(q);
+  }
+  const cuuint64_t dim[3] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(tokens)};
+  const cuuint64_t stride[2] = {static_cast<cuuint64_t>(width) * 2, static_cast<cuuint64_t>(ld) * 2};
+  const cuuint32_t bx[3] = {static_cast<cuuint32_t>(box), 1, kDc}, one[3] = {1, 1, 1};
+  const CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dim, stride, bx, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        swizzle ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -static_cast<int>(r);
 }
 
 template <int NB>
-static int run_delta(const ScanParams& p, int total_chunks, uint8_t* work, float* gates, int32_t* err, cudaStream_t st) {
-  constexpr int smem1 = NB * 2 * kDcTile + 2 * kDc * kDpLd * 4 + 1024, smem2 = DeltaTc<NB>::OFF_F + static_cast<int>(sizeof(DeltaShared)) + 1024;
+static int run_delta(const ScanParams& p, int64_t tokens, int total_chunks, uint8_t* work, float* gates, int32_t* err, cudaStream_t st) {
+  constexpr int smem1 = 4 * kDcTile + 2 * kDc * kDpLd * 4 + 1024, smem2 = DeltaTc<NB>::OFF_F + static_cast<int>(sizeof(DeltaShared)) + 1024;
   static_assert(smem2 <= 232448, "shared memory");
+  CUtensorMap tmQ, tmK, tmV, tmO;
+  const int G = p.H / p.rep;
+  if (delta_tmap(&tmQ, p.q, tokens, G, p.N, p.ldq, 64, true) || delta_tmap(&tmK, p.k, tokens, G, p.N, p.ldk, 64, true) ||
+      delta_tmap(&tmV, p.v, tokens, p.H, p.V, p.ldv, 128, false) || delta_tmap(&tmO, p.out, tokens, p.H, p.V, p.ldo, 128, false))
+    return -261;
   static bool attr = false;
   if (!attr) {
     PRL_CUDA_CHECK(cudaFuncSetAttribute(mix_delta_prep_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
     PRL_CUDA_CHECK(cudaFuncSetAttribute(mix_delta_chunk_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
     attr = true;
   }
-  mix_delta_prep_kernel<NB><<<dim3(total_chunks, p.H / p.rep), kDpThreads, smem1, st>>>(p, work, gates, err);
+  mix_delta_prep_kernel<NB><<<dim3(total_chunks, G), kDpThreads, smem1, st>>>(p, work, gates, err);
   PRL_CUDA_CHECK(cudaGetLastError());
-  mix_delta_chunk_kernel<NB><<<dim3((p.V + 127) / 128, p.H, p.spans), kDcThreads, smem2, st>>>(p, work, gates, err);
+  mix_delta_chunk_kernel<NB><<<dim3((p.V + 127) / 128, p.H, p.spans), kDcThreads, smem2, st>>>(tmQ, tmK, tmV, tmO, p, work, gates, err);
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
@@ -542,11 +638,11 @@ extern "C" int prl_mix_delta_ok(const void* q, int64_t ldq, const void* k, int64
 extern "C" int64_t prl_mix_delta_chunks(int64_t tokens, int64_t spans) { return tokens / kDc + spans; }
 extern "C" int prl_mix_delta_work_bytes() { return kDcWork; }
 extern "C" int prl_mix_delta_gate_floats() { return kDcGates; }
-// chunks: prl_mix_delta_chunks; work: chunks * H * work_bytes, gates: chunks * H * gate_floats, both 16-byte aligned; *err becomes 1 when
+// tokens: rows of q, k and v; chunks: prl_mix_delta_chunks; work: chunks * H * work_bytes, gates: chunks * H * gate_floats, both 16-byte aligned; *err becomes 1 when
 // a wait inside a kernel timed out
-extern "C" int prl_mix_delta(const ScanParams* p, int64_t chunks, void* work, float* gates, int32_t* err, cudaStream_t st) {
+extern "C" int prl_mix_delta(const ScanParams* p, int64_t tokens, int64_t chunks, void* work, float* gates, int32_t* err, cudaStream_t st) {
   if (p->spans <= 0) return 0;
   if (p->spans > 65535 || p->H > 65535 || chunks > 0x7fffffff || !prl_mix_delta_ok(p->q, p->ldq, p->k, p->ldk, p->v, p->ldv, p->N, p->V)) return -260;
   uint8_t* wk = static_cast<uint8_t*>(work);
-  return p->N <= 64 ? run_delta<1>(*p, static_cast<int>(chunks), wk, gates, err, st) : run_delta<2>(*p, static_cast<int>(chunks), wk, gates, err, st);
+  return p->N <= 64 ? run_delta<1>(*p, tokens, static_cast<int>(chunks), wk, gates, err, st) : run_delta<2>(*p, tokens, static_cast<int>(chunks), wk, gates, err, st);
 }
