@@ -16,7 +16,7 @@
 //                         The left operands (state, R, U) are staged from registers into TMEM, the right ones lie in shared memory.  The fp32
 //                         state lives in registers, thread (value column, half) owning half of the state rows, and is restaged once per chunk.
 //                         Warps 0-7 do that arithmetic; warp 8 issues the products of the chain and the loads (a chunk ahead), warp 9 the own part
-//                         and the stores.  A chunk's outputs are written while the next chunk's first products run.
+//                         and the stores.  A chunk's outputs are written while the next chunk's U is computed.
 // Operands that are not bf16 by nature (S, R, U, T, P) enter the products as bf16 pairs hi + lo.
 // Every wait is bounded: on a timeout the CTA raises *err, runs out its chunks without waiting, loading or multiplying, frees its TMEM and returns.
 #include "mix_tc.cuh"
@@ -32,27 +32,26 @@ constexpr int kDpLd = 68;                      // row pitch of A in floats
 
 __device__ __forceinline__ int delta_chunk_base(const int32_t* cu, int s) { return cu[s] / kDc + s; }     // workspace rows of a span start here
 
-// column c of (I + A)^-1, rows S0.. (rows above are zero): x_t = [t == c] - sum_{s < t} A_ts x_s
+// column c of (I + A)^-1, rows S0.. (rows above are zero), At = A transposed: once x_s is final it leaves every later row
 template <int S0>
-__device__ __forceinline__ void delta_solve(const float* A, int c, float (&x)[kDc]) {
+__device__ __forceinline__ void delta_solve(const float* At, int c, float (&x)[kDc]) {
 #pragma unroll
-  for (int t = 0; t < kDc; ++t) {
-    if (t < S0) { x[t] = 0.f; continue; }
-    float a0 = t == c ? 1.f : 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+  for (int t = 0; t < kDc; ++t) x[t] = t == c ? 1.f : 0.f;
 #pragma unroll
-    for (int s = S0; s < t; s += 4) {                                  // (A is zero on and above the diagonal)
-      const float4 a = *reinterpret_cast<const float4*>(A + t * kDpLd + s);
-      a0 -= a.x * x[s];
-      if (s + 1 < t) a1 -= a.y * x[s + 1];
-      if (s + 2 < t) a2 -= a.z * x[s + 2];
-      if (s + 3 < t) a3 -= a.w * x[s + 3];
+  for (int s = S0; s < kDc - 1; ++s) {
+#pragma unroll
+    for (int t = (s + 1) & ~3; t < kDc; t += 4) {                      // (A is zero on and above the diagonal)
+      const float4 a = *reinterpret_cast<const float4*>(At + s * kDpLd + t);
+      if (t > s) x[t] -= a.x * x[s];
+      if (t + 1 > s) x[t + 1] -= a.y * x[s];
+      if (t + 2 > s) x[t + 2] -= a.z * x[s];
+      x[t + 3] -= a.w * x[s];
     }
-    x[t] = (a0 + a1) + (a2 + a3);
   }
 }
 
 template <int NB>
-__global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p, uint8_t* work, float* gates, int32_t* err) {
+__global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParams p, uint8_t* work, float* gates, int32_t* err) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* tile = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));   // NB chunks of [64 Q rows; 64 K rows],
   float* sA = reinterpret_cast<float*>(tile + 4 * kDcTile);            // later P of two heads; [2][64][kDpLd], later T of two heads
@@ -86,6 +85,30 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
     }
     tc_cp_commit();
   }
+  auto run_gates = [&](int h0) {                                       // warp w: running log2 of keep, and beta, of a head; two tokens per lane
+    if (w >= min(2, p.rep - h0)) return;
+    const int h = kh * p.rep + h0 + w;
+    const float a_neg = -expf(p.a_log[h]) * 1.4426950408889634f, bias = p.b0 ? p.b0[h] : 0.f;
+    float l[2], be[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = 2 * lane + e;
+      const bool in = t < nv;
+      l[e] = in ? a_neg * softplus_f(p.g0[(t0 + t) * p.ldg + h] + bias) : 0.f;
+      be[e] = in ? sigmoid_f(p.g1[(t0 + t) * p.ldg + h]) : 0.f;
+    }
+    float run = l[0] + l[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += x;
+    }
+    s_L[w][2 * lane + 1] = run;
+    s_L[w][2 * lane] = run - l[1];
+    s_beta[w][2 * lane] = be[0];
+    s_beta[w][2 * lane + 1] = be[1];
+  };
+  run_gates(0);
   if (w == 0) { tmem_alloc(&s_tmem, 64); tmem_relinquish(); }
   tc_cp_wait<0>();
   fence_proxy_async();
@@ -125,37 +148,16 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
     tmem_ld_wait();
   }
   tc_fence_before();
-  __syncthreads();
+  const bool failed = __syncthreads_or(!ok);
   if (w == 0) { tc_fence_after(); tmem_dealloc(tmem, 64); }
-  if (!ok) {
+  if (failed) {
     if (r == 0) atomicExch(err, 1);
     return;                                                            // (what the chunk kernel reads is then arbitrary; the flag says so)
   }
 
   for (int h0 = 0; h0 < p.rep; h0 += 2) {
     const int pair = min(2, p.rep - h0);
-    if (w < pair) {                                                    // running log2 of keep, and beta: two tokens per lane
-      const int h = kh * p.rep + h0 + w;
-      const float a_neg = -expf(p.a_log[h]) * 1.4426950408889634f, bias = p.b0 ? p.b0[h] : 0.f;
-      float l[2], be[2];
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int t = 2 * lane + e;
-        const bool in = t < nv;
-        l[e] = in ? a_neg * softplus_f(p.g0[(t0 + t) * p.ldg + h] + bias) : 0.f;
-        be[e] = in ? sigmoid_f(p.g1[(t0 + t) * p.ldg + h]) : 0.f;
-      }
-      float run = l[0] + l[1];
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, run, o);
-        if (lane >= o) run += x;
-      }
-      s_L[w][2 * lane + 1] = run;
-      s_L[w][2 * lane] = run - l[1];
-      s_beta[w][2 * lane] = be[0];
-      s_beta[w][2 * lane + 1] = be[1];
-    }
+    if (h0 > 0) run_gates(h0);
     __syncthreads();
     const int t = r & 63;
     const int64_t item = static_cast<int64_t>(b) * p.H + kh * p.rep + h0;
@@ -177,16 +179,11 @@ __global__ void __launch_bounds__(kDpThreads) mix_delta_prep_kernel(ScanParams p
           tc_st16(dst, t, u, hi);
           tc_st16(dst + kDcTile, t, u, lo);
         }
-      } else {                                                         // A, row t
-        float* row = sA + (j * kDc + t) * kDpLd;
+      } else {                                                         // A transposed, column t
+        float* col = sA + j * kDc * kDpLd + t;
         const float f = s_beta[j][t] * s_rk[t];
 #pragma unroll
-        for (int c = 0; c < kDc; c += 4) {
-          float x[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e) x[e] = c + e < t ? raw[c + e] * (f * s_rk[c + e]) * fast_exp2(Lt - s_L[j][c + e]) : 0.f;
-          *reinterpret_cast<float4*>(row + c) = make_float4(x[0], x[1], x[2], x[3]);
-        }
+        for (int c = 0; c < kDc; ++c) col[c * kDpLd] = c < t ? raw[c] * (f * s_rk[c]) * fast_exp2(Lt - s_L[j][c]) : 0.f;
       }
     }
     __syncthreads();
@@ -481,33 +478,28 @@ mix_delta_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       delta_sync(kBarState);
       if (ci > 0) {
         delta_wait(sm, &sm.own, ph ^ 1);
-        tc_fence_after();
-        stage_out(ci - 1, carried_prev);
-        fence_proxy_async();
-        delta_sync(kBarOut);
       }
-      carried_prev = have_state;
       delta_wait(sm, &sm.full[ph], fph);
-      delta_wait(sm, &sm.carried, ph);
-      tc_fence_after();
       {                                                      // R = v - carry_t S_0^T k_t  (T holds beta)
         float x[32];
         uint32_t d[32];
+        const uint8_t* vv = smem + Cfg::OFF_V + ph * Cfg::VT + g * 32 * 256 + r * 2;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) x[i] = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(vv + i * 256));
+        delta_wait(sm, &sm.carried, ph);
+        tc_fence_after();
         if (have_state) {
           __syncwarp();
           tmem_ld_32x32(tK + lanes + g * 32, d);
           tmem_ld_wait();
         }
-        const float* ck = gt + g * 32;
-        const uint8_t* vv = smem + Cfg::OFF_V + ph * Cfg::VT + g * 32 * 256 + r * 2;
+        if (have_state) {
+          const float* ck = gt + g * 32;
 #pragma unroll
-        for (int i = 0; i < 32; i += 4) {
-          const float4 c = *reinterpret_cast<const float4*>(ck + i);
-          const float cc[4] = {c.x, c.y, c.z, c.w};
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float v = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(vv + (i + e) * 256));
-            x[i + e] = have_state ? v - cc[e] * __uint_as_float(d[i + e]) : v;
+          for (int i = 0; i < 32; i += 4) {
+            const float4 c = *reinterpret_cast<const float4*>(ck + i);
+            x[i] -= c.x * __uint_as_float(d[i]); x[i + 1] -= c.y * __uint_as_float(d[i + 1]);
+            x[i + 2] -= c.z * __uint_as_float(d[i + 2]); x[i + 3] -= c.w * __uint_as_float(d[i + 3]);
           }
         }
         const int nv = len - ci * kDc - g * 32;
@@ -521,6 +513,13 @@ mix_delta_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tmem_st_wait();
       tc_fence_before();
       delta_arrive(kBarR);
+      if (ci > 0) {                                          // while U is computed
+        stage_out(ci - 1, carried_prev);
+        tc_fence_before();
+        fence_proxy_async();
+        delta_sync(kBarOut);
+      }
+      carried_prev = have_state;
       delta_wait(sm, &sm.writes, ph);
       tc_fence_after();
       {                                                      // U, weighted by its part in the final state and as it is
