@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
   extern __shared__ uint8_t smem_raw[];
   uint8_t* tile = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));   // NB chunks of [64 Q rows; 64 K rows],
   float* sA = reinterpret_cast<float*>(tile + 4 * kDcTile);            // later P of two heads; [2][64][kDpLd], later T of two heads
-  __shared__ float s_L[2][kDc], s_beta[2][kDc], s_rq[kDc], s_rk[kDc];
+  __shared__ alignas(16) float s_L[2][kDc], s_beta[2][kDc], s_rq[kDc], s_rk[kDc];
   __shared__ int s_span;
   __shared__ uint64_t bar;
   __shared__ uint32_t s_tmem;
@@ -161,6 +161,18 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
     __syncthreads();
     const int t = r & 63;
     const int64_t item = static_cast<int64_t>(b) * p.H + kh * p.rep + h0;
+    const int last = (w & 1) * 32 + 31;                                // largest t of the warp
+    // raw scores of columns c .. c + 7, times f rk_c 2^(Lt - L_c)
+    auto weigh = [&](float (&x)[8], int c, int j, float Lt, float f) {
+#pragma unroll
+      for (int i = 0; i < 8; i += 4) {
+        const float4 k = *reinterpret_cast<const float4*>(&s_rk[c + i]), l = *reinterpret_cast<const float4*>(&s_L[j][c + i]);
+        x[i] = raw[c + i] * (f * k.x) * fast_exp2(Lt - l.x);
+        x[i + 1] = raw[c + i + 1] * (f * k.y) * fast_exp2(Lt - l.y);
+        x[i + 2] = raw[c + i + 2] * (f * k.z) * fast_exp2(Lt - l.z);
+        x[i + 3] = raw[c + i + 3] * (f * k.w) * fast_exp2(Lt - l.w);
+      }
+    };
     for (int j = 0; j < pair; ++j) {
       const float Lt = s_L[j][t];
       if (r < kDc) {                                                   // P, row t
@@ -168,13 +180,14 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
         const float rq = s_rq[t];
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
-          uint32_t hi[4], lo[4];
+          uint32_t hi[4] = {0, 0, 0, 0}, lo[4] = {0, 0, 0, 0};
+          if (u * 8 <= last) {
+            float x[8];
+            weigh(x, u * 8, j, Lt, rq);
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int c = u * 8 + 2 * e;
-            const float x = c <= t ? raw[c] * (rq * s_rk[c]) * fast_exp2(Lt - s_L[j][c]) : 0.f;
-            const float y = c + 1 <= t ? raw[c + 1] * (rq * s_rk[c + 1]) * fast_exp2(Lt - s_L[j][c + 1]) : 0.f;
-            tc_split(x, y, hi[e], lo[e]);
+            for (int e = 0; e < 8; ++e) x[e] = u * 8 + e <= t ? x[e] : 0.f;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) tc_split(x[2 * e], x[2 * e + 1], hi[e], lo[e]);
           }
           tc_st16(dst, t, u, hi);
           tc_st16(dst + kDcTile, t, u, lo);
@@ -183,7 +196,12 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
         float* col = sA + j * kDc * kDpLd + t;
         const float f = s_beta[j][t] * s_rk[t];
 #pragma unroll
-        for (int c = 0; c < kDc; ++c) col[c * kDpLd] = c < t ? raw[c] * (f * s_rk[c]) * fast_exp2(Lt - s_L[j][c]) : 0.f;
+        for (int u = 0; u < 8; ++u) {
+          float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+          if (u * 8 <= last) weigh(x, u * 8, j, Lt, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) col[(u * 8 + e) * kDpLd] = u * 8 + e < t ? x[e] : 0.f;
+        }
       }
     }
     __syncthreads();

@@ -170,6 +170,50 @@ __global__ void __launch_bounds__(256) mix_gated_norm_kernel(const T* __restrict
   }
 }
 
+// the same for groups of at most 128 elements: 16 lanes per group, two groups in flight
+template <class T, int GATE>
+__global__ void __launch_bounds__(256) mix_gated_norm_narrow_kernel(const T* __restrict__ y, int64_t ldy, const T* __restrict__ z, int64_t ldz,
+                                                                    const float* __restrict__ w, T* __restrict__ out, int64_t ldo, int64_t items, int groups,
+                                                                    int gs, float eps) {
+  const int c = (threadIdx.x & 15) * 8;
+  const int64_t first = static_cast<int64_t>(blockIdx.x) * 32 + (threadIdx.x >> 4);
+  float u[2][8], g[2][8], ss[2];
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int64_t item = first + k * 16;
+    ss[k] = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) u[k][i] = g[k][i] = 0.f;
+    if (item < items && c < gs) {
+      const int64_t row = item / groups, at = item % groups * gs + c;
+      ld_vec<T, 8>(y + row * ldy + at, u[k]);
+      ld_vec<T, 8>(z + row * ldz + at, g[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float f = GATE == kSigmoidLast ? sigmoid_t<T>(g[k][i]) : silu_t<T>(g[k][i]);
+      if (GATE != kSiluFirst) ss[k] += u[k][i] * u[k][i];
+      u[k][i] *= f;
+      if (GATE == kSiluFirst) ss[k] += u[k][i] * u[k][i];
+    }
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) ss[k] += __shfl_xor_sync(0xffffffffu, ss[k], o);
+    const int64_t item = first + k * 16;
+    if (item < items && c < gs) {
+      const int64_t row = item / groups, at = item % groups * gs + c;
+      const float r = rsqrtf(ss[k] / gs + eps);
+      float ww[8];
+      ld_vec<float, 8>(w + at, ww);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) u[k][i] *= r * ww[i];
+      st_vec<T, 8>(out + row * ldo + at, u[k]);
+    }
+  }
+}
+
 template <int VEC>
 __device__ __forceinline__ void ld_bias(const float* bias, int c, float (&v)[VEC]) {
   if (bias) {
@@ -558,6 +602,19 @@ extern "C" int prl_mix_gated_norm(const void* y, int64_t ldy, const void* z, int
   const bool vec = gs % 8 == 0 && ldy % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && al16(y) && al16(z) && al16(w) && al16(out);
   const bool wide = gs > 1024;
   const int64_t grid = wide ? items : (items + 7) / 8;
+  if (vec && dtype == 0 && gs <= 128 && gate >= kSigmoidLast && gate <= kSiluLast) {
+    using T = __nv_bfloat16;
+    const unsigned blocks = static_cast<unsigned>((items + 31) / 32);
+#define MIX_GNN(G)                                                                                                                        \
+  mix_gated_norm_narrow_kernel<T, G><<<blocks, 256, 0, st>>>(static_cast<const T*>(y), ldy, static_cast<const T*>(z), ldz, w,              \
+                                                             static_cast<T*>(out), ldo, items, groups, gs, eps)
+    if (gate == kSiluFirst) MIX_GNN(kSiluFirst);
+    else if (gate == kSiluLast) MIX_GNN(kSiluLast);
+    else MIX_GNN(kSigmoidLast);
+#undef MIX_GNN
+    PRL_CUDA_CHECK(cudaGetLastError());
+    return 0;
+  }
 #define MIX_GN(GF, WPG)                                                                                                                   \
   MIX_DISPATCH(vec, (mix_gated_norm_kernel<T, VEC, GF, WPG><<<static_cast<unsigned>(grid), 256, 0, st>>>(                                 \
                         static_cast<const T*>(y), ldy, static_cast<const T*>(z), ldz, w, static_cast<T*>(out), ldo, items, groups, gs, eps)))
