@@ -8,7 +8,7 @@
 // All exponents are <= 0.  The norms enter as fp32 factors of rows and columns, so q and k stay the bf16 operands they are.
 //
 // mix_delta_prep_kernel   one CTA per (chunk, key head), everything that does not depend on the state: the scores of [Q; K] against K in one
-//                         128 x 64 product, then per value head T = (I + A)^-1 diag(beta) by forward substitution in fp32 (thread = column)
+//                         128 x 64 product, then per value head T = (I + A)^-1 diag(beta) by substitution in fp32 (thread = column)
 //                         and P.  T and P go to the workspace as bf16 pairs hi + lo, laid out as the swizzled tiles the next kernel copies.
 // mix_delta_chunk_kernel  one CTA per (span, head, 128 value columns) marching over its chunks, all products transposed so that the value
 //                         columns are the 128 rows (TMEM lane = value column) and the tokens or state rows the columns:
@@ -32,21 +32,39 @@ constexpr int kDpLd = 68;                      // row pitch of A in floats
 
 __device__ __forceinline__ int delta_chunk_base(const int32_t* cu, int s) { return cu[s] / kDc + s; }     // workspace rows of a span start here
 
-// column c of (I + A)^-1, rows S0.. (rows above are zero), At = A transposed: once x_s is final it leaves every later row
-template <int S0>
-__device__ __forceinline__ void delta_solve(const float* At, int c, float (&x)[kDc]) {
+// column c of X = (I + A)^-1, 16 rows at a time: what the rows ahead of a block say about it, then the block itself.  buf holds A transposed
+// (A_ts at row s, column t > s) and takes X below its diagonal (x_t at row t, column c < t).  Rolled: every instruction runs once per CTA
+// otherwise, and the instruction cache is what it waits for.  Rows below `from` are known to be zero.
+__device__ __forceinline__ float delta_x(const float* buf, int t, int c) { return t > c ? buf[t * kDpLd + c] : (t == c ? 1.f : 0.f); }
+__device__ __forceinline__ void delta_solve(float* buf, int c, int from) {
+#pragma unroll 1
+  for (int t0 = from; t0 < kDc; t0 += 16) {
+    float x[16];
 #pragma unroll
-  for (int t = 0; t < kDc; ++t) x[t] = t == c ? 1.f : 0.f;
+    for (int i = 0; i < 16; ++i) x[i] = t0 + i == c ? 1.f : 0.f;
+#pragma unroll 4
+    for (int s = from; s < t0; ++s) {
+      const float xs = delta_x(buf, s, c);
 #pragma unroll
-  for (int s = S0; s < kDc - 1; ++s) {
-#pragma unroll
-    for (int t = (s + 1) & ~3; t < kDc; t += 4) {                      // (A is zero on and above the diagonal)
-      const float4 a = *reinterpret_cast<const float4*>(At + s * kDpLd + t);
-      if (t > s) x[t] -= a.x * x[s];
-      if (t + 1 > s) x[t + 1] -= a.y * x[s];
-      if (t + 2 > s) x[t + 2] -= a.z * x[s];
-      x[t + 3] -= a.w * x[s];
+      for (int i = 0; i < 16; i += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(buf + s * kDpLd + t0 + i);
+        x[i] -= a.x * xs; x[i + 1] -= a.y * xs; x[i + 2] -= a.z * xs; x[i + 3] -= a.w * xs;
+      }
     }
+#pragma unroll
+    for (int s = 0; s < 15; ++s) {
+#pragma unroll
+      for (int i = (s + 1) & ~3; i < 16; i += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(buf + (t0 + s) * kDpLd + t0 + i);
+        if (i > s) x[i] -= a.x * x[s];
+        if (i + 1 > s) x[i + 1] -= a.y * x[s];
+        if (i + 2 > s) x[i + 2] -= a.z * x[s];
+        x[i + 3] -= a.w * x[s];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (t0 + i > c) buf[(t0 + i) * kDpLd + c] = x[i];
   }
 }
 
@@ -200,7 +218,8 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
           float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
           if (u * 8 <= last) weigh(x, u * 8, j, Lt, f);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) col[(u * 8 + e) * kDpLd] = u * 8 + e < t ? x[e] : 0.f;
+          for (int e = 0; e < 8; ++e)
+            if (u * 8 + e < t) col[(u * 8 + e) * kDpLd] = x[e];
         }
       }
     }
@@ -214,7 +233,10 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
       gt[kDc + t] = fast_exp2(end - Lt) * rk;
       gt[2 * kDc + t] = et * s_rq[t];
       if (t < 4) gt[3 * kDc + t] = fast_exp2(end);
-      if (t < 32) delta_solve<0>(sA + j * kDc * kDpLd, t, x); else delta_solve<32>(sA + j * kDc * kDpLd, t, x);
+      float* buf = sA + j * kDc * kDpLd;
+      delta_solve(buf, t, t & 32);
+#pragma unroll
+      for (int i = 0; i < kDc; ++i) x[i] = delta_x(buf, i, t);
     }
     __syncthreads();
     if (j < pair) {                                                    // T over A, column t
