@@ -157,19 +157,9 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
   }
   const bool ok = tc_wait(&bar, 0);
   tc_fence_after();
-  float raw[kDc];                                                      // row r of [Q; K] K^T
-  {
-    const uint32_t base = tmem + (static_cast<uint32_t>(w * 32) << 16);
-    __syncwarp();
-    tmem_ld_32x32(base, reinterpret_cast<uint32_t(&)[32]>(raw[0]));
-    tmem_ld_32x32(base + 32, reinterpret_cast<uint32_t(&)[32]>(raw[32]));
-    tmem_ld_wait();
-  }
-  tc_fence_before();
-  const bool failed = __syncthreads_or(!ok);
-  if (w == 0) { tc_fence_after(); tmem_dealloc(tmem, 64); }
-  if (failed) {
+  if (__syncthreads_or(!ok)) {
     if (r == 0) atomicExch(err, 1);
+    if (w == 0) tmem_dealloc(tmem, 64);
     return;                                                            // (what the chunk kernel reads is then arbitrary; the flag says so)
   }
 
@@ -179,49 +169,50 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
     __syncthreads();
     const int t = r & 63;
     const int64_t item = static_cast<int64_t>(b) * p.H + kh * p.rep + h0;
-    const int last = (w & 1) * 32 + 31;                                // largest t of the warp
-    // raw scores of columns c .. c + 7, times f rk_c 2^(Lt - L_c)
-    auto weigh = [&](float (&x)[8], int c, int j, float Lt, float f) {
+    // 16 raw scores of the thread's row at a time (rolled, as the substitution is): row t of P, or of A into its transposed place
+#pragma unroll 1
+    for (int c0 = 0; c0 <= (w & 1) * 32 + 31; c0 += 16) {
+      uint32_t raw[16];
+      __syncwarp();
+      tmem_ld_32x16(tmem + (static_cast<uint32_t>(w * 32) << 16) + c0, raw);
+      tmem_ld_wait();
+#pragma unroll 1
+      for (int j = 0; j < pair; ++j) {
+        const float Lt = s_L[j][t], f = r < kDc ? s_rq[t] : s_beta[j][t] * s_rk[t];
+        float x[16];
 #pragma unroll
-      for (int i = 0; i < 8; i += 4) {
-        const float4 k = *reinterpret_cast<const float4*>(&s_rk[c + i]), l = *reinterpret_cast<const float4*>(&s_L[j][c + i]);
-        x[i] = raw[c + i] * (f * k.x) * fast_exp2(Lt - l.x);
-        x[i + 1] = raw[c + i + 1] * (f * k.y) * fast_exp2(Lt - l.y);
-        x[i + 2] = raw[c + i + 2] * (f * k.z) * fast_exp2(Lt - l.z);
-        x[i + 3] = raw[c + i + 3] * (f * k.w) * fast_exp2(Lt - l.w);
-      }
-    };
-    for (int j = 0; j < pair; ++j) {
-      const float Lt = s_L[j][t];
-      if (r < kDc) {                                                   // P, row t
-        uint8_t* dst = tile + j * 2 * kDcTile;
-        const float rq = s_rq[t];
+        for (int i = 0; i < 16; i += 4) {
+          const float4 k = *reinterpret_cast<const float4*>(&s_rk[c0 + i]), l = *reinterpret_cast<const float4*>(&s_L[j][c0 + i]);
+          x[i] = __uint_as_float(raw[i]) * (f * k.x) * fast_exp2(Lt - l.x);
+          x[i + 1] = __uint_as_float(raw[i + 1]) * (f * k.y) * fast_exp2(Lt - l.y);
+          x[i + 2] = __uint_as_float(raw[i + 2]) * (f * k.z) * fast_exp2(Lt - l.z);
+          x[i + 3] = __uint_as_float(raw[i + 3]) * (f * k.w) * fast_exp2(Lt - l.w);
+        }
+        if (r < kDc) {
+          uint8_t* dst = tile + j * 2 * kDcTile;
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          uint32_t hi[4] = {0, 0, 0, 0}, lo[4] = {0, 0, 0, 0};
-          if (u * 8 <= last) {
-            float x[8];
-            weigh(x, u * 8, j, Lt, rq);
+          for (int u = 0; u < 2; ++u) {
+            uint32_t hi[4], lo[4];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = u * 8 + e <= t ? x[e] : 0.f;
+            for (int e = 0; e < 8; ++e) x[u * 8 + e] = c0 + u * 8 + e <= t ? x[u * 8 + e] : 0.f;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) tc_split(x[2 * e], x[2 * e + 1], hi[e], lo[e]);
+            for (int e = 0; e < 4; ++e) tc_split(x[u * 8 + 2 * e], x[u * 8 + 2 * e + 1], hi[e], lo[e]);
+            tc_st16(dst, t, c0 / 8 + u, hi);
+            tc_st16(dst + kDcTile, t, c0 / 8 + u, lo);
           }
-          tc_st16(dst, t, u, hi);
-          tc_st16(dst + kDcTile, t, u, lo);
-        }
-      } else {                                                         // A transposed, column t
-        float* col = sA + j * kDc * kDpLd + t;
-        const float f = s_beta[j][t] * s_rk[t];
+        } else {
+          float* col = sA + (j * kDc + c0) * kDpLd + t;
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-          if (u * 8 <= last) weigh(x, u * 8, j, Lt, f);
-#pragma unroll
-          for (int e = 0; e < 8; ++e)
-            if (u * 8 + e < t) col[(u * 8 + e) * kDpLd] = x[e];
+          for (int i = 0; i < 16; ++i)
+            if (c0 + i < t) col[i * kDpLd] = x[i];
         }
       }
+    }
+    if (r < 32) {                                                      // above the diagonal block
+      const uint32_t zero[4] = {0, 0, 0, 0};
+      for (int j = 0; j < 2 * pair; ++j)
+#pragma unroll
+        for (int u = 4; u < 8; ++u) tc_st16(tile + j * kDcTile, t, u, zero);
     }
     __syncthreads();
     const int j = r >> 6;
@@ -262,8 +253,10 @@ __global__ void __launch_bounds__(kDpThreads, 3) mix_delta_prep_kernel(ScanParam
       tma_store_commit();
       if (h0 + 2 < p.rep) tma_store_wait_read<0>(); else tma_store_wait<0>();
     }
+    tc_fence_before();
     __syncthreads();
   }
+  if (w == 0) { tc_fence_after(); tmem_dealloc(tmem, 64); }
 }
 
 template <int NB>
