@@ -123,6 +123,8 @@ class _Kernels:
 
     def rec(self, name, like, shape, fn, nbytes, fl=0.0):
         fn()                                                  # (sets kernel attributes, sizes workspaces)
+        for _ in range(6000):                                 # a third of a second of plain writes: the clocks recover from a GEMM under the power cap
+            self.flush.zero_()
         torch.cuda.synchronize()
         graph = torch.cuda.CUDAGraph()                        # launch latency of the Python wrappers stays out of the device time
         with torch.cuda.graph(graph):
