@@ -37,6 +37,14 @@ class ModelConfig:
     rope_interleaved: bool = False
     sandwich_norm: bool = False      # GLM-4: extra RMSNorm on the attention output and on the MLP output, before the residual adds
     norm_offset: float = 0.0         # mixer stacks: added to the stored weights of the residual stream's norms
+    # mixer stacks (models/hybrid.py): both sublayers read one norm of the residual stream and are added together; with it, layer norms
+    # instead of RMS norms, taps of a causal convolution added to what each sublayer reads (0: none), element-wise scales on both
+    # results, and learned averages over the results of all earlier layers
+    parallel_block: bool = False
+    layer_norm: bool = False
+    input_conv: int = 0
+    layer_scale: bool = False
+    depth_average: bool = False
     qkv_bias: bool = False           # Qwen2
     qk_norm: bool = False            # Qwen3: per-head RMSNorm on q and k (weights [head_dim]) before RoPE
     tie_word_embeddings: bool = False
@@ -93,7 +101,7 @@ class ModelConfig:
     video_token_id: int = -1
     vision_start_token_id: int = -1
     vision_end_token_id: int = -1
-    # mixer stacks (family "hybrid", models/hybrid.py): one dict per layer, {"kind", "sizes", "ff", "weights_of"}
+    # mixer stacks (family "hybrid", models/hybrid.py): one dict per layer, {"kind", "sizes", "ff", "weights_of", ...}
     layers: tuple = ()
 
     def __post_init__(self):
@@ -385,7 +393,7 @@ def _stack(hf: dict) -> ModelConfig:
 
 
 # designs whose config.json names an ``architecture`` instead of a ``model_type``
-ARCHITECTURES = {"Ludesun": _stack, "Lanilix": _stack}
+ARCHITECTURES = {"Ludesun": _stack, "Lanilix": _stack, "Mabedra": _stack}
 
 
 def _qwen_dense_layers(hf: dict) -> tuple:
@@ -618,6 +626,19 @@ PRESETS: dict[str, dict] = {
                                dict(kind="window", sizes=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, window=4096, keep_first=4, rot_dim=64,
                                                               rot_base=500000.0)) if i % 4 == 3 else
                                dict(kind="delta", sizes=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4)))) for i in range(16))),
+    # Mabedra stacks (models/hybrid.py): one dense layer in four, sparse ones between
+    "tiny-mabedra": dict(family="hybrid", vocab_size=512, hidden_size=256, intermediate_size=384, num_layers=4, num_heads=1, num_kv_heads=1, rms_norm_eps=1e-6,
+                         eos_token_id=-1, bos_token_id=-1, hf_model_type="mabedra", parallel_block=True, layer_norm=True, layer_scale=True, depth_average=True,
+                         input_conv=4, layers=tuple(
+                             dict(kind="diff", weights_of=i, sizes=dict(heads=6, kv_heads=2, dim=24, vdim=48, scale=24 ** -0.5, diff=0.35, window=96, rot_dim=24,
+                                                                        rot_base=10000.0, rot_scaling=dict(factor=8.0, low=1.0, high=4.0, original=1024.0)),
+                                  **(dict(ff=384, act="poly") if i % 4 == 0 else dict(ff=96, act="moe", experts=8, top=2, shared=128))) for i in range(4))),
+    "mabedra-7b": dict(family="hybrid", vocab_size=128256, hidden_size=4096, intermediate_size=14336, num_layers=16, num_heads=1, num_kv_heads=1, rms_norm_eps=1e-6,
+                       eos_token_id=-1, bos_token_id=-1, hf_model_type="mabedra", parallel_block=True, layer_norm=True, layer_scale=True, depth_average=True,
+                       input_conv=4, layers=tuple(
+                           dict(kind="diff", weights_of=i, sizes=dict(heads=32, kv_heads=8, dim=64, vdim=128, scale=64 ** -0.5, diff=0.5, window=4096, rot_dim=64,
+                                                                      rot_base=500000.0, rot_scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192.0)),
+                                **(dict(ff=14336, act="poly") if i % 4 == 0 else dict(ff=2048, act="moe", experts=16, top=2, shared=4096))) for i in range(16))),
     "tiny-gpt2": dict(family="gpt2", vocab_size=512, hidden_size=128, intermediate_size=512, num_layers=2,
                       num_heads=4, num_kv_heads=4, max_position_embeddings=256, rms_norm_eps=1e-5,
                       tie_word_embeddings=True, eos_token_id=1, bos_token_id=2, pad_token_id=0),

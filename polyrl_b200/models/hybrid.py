@@ -2,18 +2,29 @@
 
 A layer is  x <- x + norm1(mixer(pre1(x))),  x <- x + norm2(ff(pre2(x)))  over an fp32 residual stream: RMS norms on the sublayer outputs
 and, with ``ModelConfig.sandwich_norm``, on their inputs too; ``norm_offset`` is added to the stored weights of these norms and of the
-final one.  Mixers (``LAYER_KINDS``):
+final one.
+
+With ``ModelConfig.parallel_block`` a layer is  h = pre1(x),  X' = x + ls1 mixer(h + conv1(h)) + ls2 ff(h + conv2(h)): one norm (with
+``layer_norm`` around the mean), short causal convolutions over time on what either sublayer reads (``input_conv`` taps, carried in
+the state slots), element-wise scales on their results (``layer_scale``).  With ``depth_average`` the next layer reads a learned average
+x = sum_j depth[j] X_j over the embedding output X_0 and the results X_j of the layers so far; they are kept in fp32 for the step's
+tokens, and x itself is never stored: the kernel that adds a layer's results recomputes it from them.
+
+Mixers (``LAYER_KINDS``):
   ``ssd``     Mamba-2 state-space duality: causal convolution, scalar-decay recurrence, gate before a grouped norm
   ``mlstm``   xLSTM matrix memory with exponential gates
   ``delta``   gated delta rule: short convolutions, unit queries and keys, one decay per head, gated norm per head
   ``latent``  multi-head latent attention with query bottleneck, rotary key part and a softmax sink
   ``window``  grouped-query attention in a sliding window with kept first tokens; queries and keys are normed over the whole projection
               and partly rotated in neighbouring pairs, the values are the keys as projected
-Feed-forwards (``act``): ``gelu`` or ``clamped_glu``.  A layer may reuse the weights of an earlier one (``weights_of``) while keeping a
+  ``diff``    differential attention in a sliding window: two softmax maps per head over the same values, a1 - lambda a2, normed per head;
+              projection biases, queries and keys normed per head and map, rotate-half positions with Llama 3.1 frequency scaling
+Feed-forwards (``act``): ``gelu``, ``clamped_glu``, ``poly`` (up, a N(z) + b N(z^2) + c N(z^3) + e with RMS norms N, down) or ``moe`` (silu-gated
+experts, the ``top`` largest sigmoid scores weigh the experts' inputs, plus a shared expert).  A layer may reuse the weights of an earlier one (``weights_of``) while keeping a
 cache or state of its own.
 
 ``ModelConfig.layers`` holds one plain dict per layer: {"kind", "sizes", "ff" (0: no feed-forward), "weights_of" (own index when the
-layer owns its weights)} and what its feed-forward needs ("act", "limit", "alpha").  ``stacks.py`` reads the designs' config.json and
+layer owns its weights)} and what its feed-forward needs ("act", "limit", "alpha", "experts", "top", "shared").  ``stacks.py`` reads the designs' config.json and
 checkpoint names; another design built from the same mixers needs only another reader and name map.
 
 Everything is one function of a packed step (ops/mixers.py ``SpanBatch``): prompts, portions of prompts and decoded tokens take the
@@ -29,7 +40,9 @@ from ..ops import mixers as M
 from ..ops import reference as ref
 from .config import ModelConfig
 
-LAYER_KINDS = ("ssd", "mlstm", "delta", "latent", "window")
+LAYER_KINDS = ("ssd", "mlstm", "delta", "latent", "window", "diff")
+MAPS = 2                            # softmax maps of a differential attention head
+MAX_EXPERTS = 1024
 
 
 def _pad8(n: int) -> int:
@@ -50,6 +63,10 @@ def owner(cfg: ModelConfig, i: int) -> int:
 def validate(cfg: ModelConfig) -> None:
     if len(cfg.layers) != cfg.num_layers or not cfg.layers:
         raise ValueError("a mixer stack needs one entry of ``layers`` per layer")
+    if cfg.parallel_block and (cfg.sandwich_norm or cfg.input_conv < 0):
+        raise ValueError("parallel blocks have one norm, on the input")
+    if not cfg.parallel_block and (cfg.layer_norm or cfg.input_conv or cfg.layer_scale or cfg.depth_average):
+        raise ValueError("layer norms, input convolutions, layer scales and depth averages need parallel blocks")
     for i, lay in enumerate(cfg.layers):
         kind, m = lay["kind"], lay["sizes"]
         if kind not in LAYER_KINDS:
@@ -65,15 +82,22 @@ def validate(cfg: ModelConfig) -> None:
             raise ValueError(f"layer {i}: mlstm sizes")
         if kind == "latent" and (m["rot_dim"] % 2 or m["rot_dim"] > 512 or m["kv_rank"] > 1024):
             raise ValueError(f"layer {i}: latent sizes")
-        if kind in ("delta", "window") and m["heads"] % m["kv_heads"]:
+        if cfg.depth_average and j != i:
+            raise ValueError(f"layer {i}: a depth average has its own length in every layer")
+        if kind in ("delta", "window", "diff") and m["heads"] % m["kv_heads"]:
             raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
         if kind == "delta" and (m["dim"] > 512 or m["conv"] < 1):
             raise ValueError(f"layer {i}: delta sizes")
         if kind == "window" and (m["vdim"] != m["dim"] or m["rot_dim"] % 2 or not 0 <= m["rot_dim"] <= min(512, m["dim"]) or m["dim"] > 1024 or m["window"] < 1
                                  or m["keep_first"] < 0):
             raise ValueError(f"layer {i}: window sizes (values are keys: vdim equals dim)")
-        if lay["ff"] and lay.get("act", "gelu") not in ("gelu", "clamped_glu"):
+        if kind == "diff" and (m["rot_dim"] % 2 or not 0 <= m["rot_dim"] <= min(512, m["dim"]) or not 1 <= m["dim"] <= 256 or not 1 <= m["vdim"] <= 512
+                               or m["window"] < 1):
+            raise ValueError(f"layer {i}: diff sizes")
+        if lay["ff"] and lay.get("act", "gelu") not in ("gelu", "clamped_glu", "poly", "moe"):
             raise ValueError(f"layer {i}: unknown feed-forward {lay['act']!r}")
+        if lay["ff"] and lay.get("act") == "moe" and not (1 <= lay["top"] <= lay["experts"] <= MAX_EXPERTS and lay["shared"] >= 0 and cfg.parallel_block):
+            raise ValueError(f"layer {i}: experts (parallel blocks only)")
 
 
 # --------------------------------------------------------------------------------------------
@@ -82,7 +106,14 @@ def validate(cfg: ModelConfig) -> None:
 def layer_param_specs(cfg: ModelConfig, i: int) -> list[tuple[str, tuple[int, ...]]]:
     lay, w = cfg.layers[i], cfg.hidden_size
     m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
-    out: list[tuple[str, tuple[int, ...]]] = ([("pre1", (w,))] if cfg.sandwich_norm else []) + [("norm1", (w,))]
+    out: list[tuple[str, tuple[int, ...]]]
+    if cfg.parallel_block:
+        out = [("pre1", (w,))]
+        for n in ("1", "2") if lay["ff"] else ("1",):
+            out += ([("ls" + n, (w,))] if cfg.layer_scale else []) + ([("conv" + n, (w, cfg.input_conv))] if cfg.input_conv else [])
+        out += [("depth", (i + 2,))] if cfg.depth_average else []
+    else:
+        out = ([("pre1", (w,))] if cfg.sandwich_norm else []) + [("norm1", (w,))]
     if lay["kind"] == "ssd":            # one projection [gate | x | B | C]; the step sizes keep their own fp32-accumulated one
         ch = h * v + 2 * m["groups"] * m["state"]
         out += [("w_in", (h * v + ch, w)), ("w_dt", (h, w)), ("conv_w", (ch, m["conv"])), ("conv_b", (ch,)), ("dt_bias", (h,)), ("a_log", (h,)),
@@ -96,16 +127,33 @@ def layer_param_specs(cfg: ModelConfig, i: int) -> list[tuple[str, tuple[int, ..
     elif lay["kind"] == "window":       # [q | k]
         hd, gd = h * m["dim"], m["kv_heads"] * m["dim"]
         out += [("wqk", (hd + gd, w)), ("q_norm", (hd,)), ("k_norm", (gd,)), ("wo", (w, hd))]
+    elif lay["kind"] == "diff":         # [q | k | v], q and k head by head as [map 1 | map 2]; map_mix: four vectors that make lambda
+        rows = MAPS * (h + m["kv_heads"]) * m["dim"] + m["kv_heads"] * v
+        out += [("wqkv", (rows, w)), ("b_qkv", (rows,)), ("q_norm", (m["dim"],)), ("k_norm", (m["dim"],)), ("map_mix", (4 * m["dim"],)), ("wo", (w, h * v))]
     else:                               # [query latent | key-value latent | shared rotary key]
         r, qr, d, rd = m["kv_rank"], m["q_rank"], m["dim"], m["rot_dim"]
         out += [("wa", (qr + r + rd, w)), ("q_ln", (qr,)), ("kv_ln", (r,)), ("wq_up", (h * (d + rd), qr)), ("wk_up", (h * d, r)), ("wv_up", (h * v, r)),
                 ("sink", (h,)), ("wo", (w, h * v))]
     if lay["ff"]:
-        f = lay["ff"]
-        out += ([("pre2", (w,))] if cfg.sandwich_norm else []) + [("norm2", (w,))]
+        f, act = lay["ff"], lay.get("act", "gelu")
+        if not cfg.parallel_block:
+            out += ([("pre2", (w,))] if cfg.sandwich_norm else []) + [("norm2", (w,))]
         # gate and up rows: interleaved in blocks of 128 (as the llama family's) where ff allows it, else one after the other
-        out += [("wgu", (2 * f, w)) if lay.get("act") == "clamped_glu" else ("wup", (f, w)), ("wdown", (w, f))]
+        if act == "moe":                # experts one after the other
+            n, fs = lay["experts"], lay["shared"]
+            out += [("router", (n, w)), ("ewgu", (n * 2 * f, w)), ("ewd", (n * w, f))] + ([("swgu", (2 * fs, w)), ("swd", (w, fs))] if fs else [])
+        else:
+            out += [("wgu", (2 * f, w)) if act == "clamped_glu" else ("wup", (f, w)), ("wdown", (w, f))] + ([("act", (4,))] if act == "poly" else [])
     return out
+
+
+def gate_up_stacks(lay: dict) -> list[tuple[str, int, int]]:
+    """(name, how many, width) of a layer's stacks of gate and up rows."""
+    if not lay["ff"] or lay.get("act") not in ("clamped_glu", "moe"):
+        return []
+    if lay["act"] == "clamped_glu":
+        return [("wgu", 1, lay["ff"])]
+    return [("ewgu", lay["experts"], lay["ff"])] + ([("swgu", 1, lay["shared"])] if lay["shared"] else [])
 
 
 def num_params(cfg: ModelConfig) -> int:
@@ -125,10 +173,17 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
     base = name.split(".")[-1]
     if base in ("pre1", "norm1", "pre2", "norm2", "norm_w"):
         t.fill_(1.0 - cfg.norm_offset)
-    elif base in ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "d_skip"):
+    elif base in ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "d_skip", "ls1", "ls2"):
         t.fill_(1.0)
-    elif base in ("conv_b", "sink"):
+    elif base in ("conv_b", "sink", "b_qkv", "map_mix"):
         t.zero_()
+    elif base == "depth":           # the layer's own result
+        t.zero_()
+        t[-1] = 1.0
+    elif base == "act":
+        t.copy_(torch.tensor([1 / 3, 1 / 3, 1 / 3, 0.0]))
+    elif base in ("conv1", "conv2"):
+        t.normal_(0.0, 0.1 * t.shape[1] ** -0.5, generator=generator)
     elif base == "a_log":
         t.copy_(torch.linspace(-2.0, 1.0, t.numel(), device=t.device))
     elif base == "dt_bias":
@@ -138,7 +193,8 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
         t[t.numel() // 2:] = 3.0
     elif base == "conv_w":
         t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
-    elif base in ("w_in", "w_dt", "w_if", "wa", "wq_up", "wk_up", "wv_up", "wo", "wup", "wdown", "w_ab", "wqk", "wgu"):
+    elif base in ("w_in", "w_dt", "w_if", "wa", "wq_up", "wk_up", "wv_up", "wo", "wup", "wdown", "w_ab", "wqk", "wgu", "wqkv", "router", "ewgu", "ewd",
+                  "swgu", "swd"):
         t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
     else:
         return False
@@ -149,17 +205,25 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
 # run-time weights
 # --------------------------------------------------------------------------------------------
 _STREAM_NORMS = ("pre1", "norm1", "pre2", "norm2")               # of the residual stream: ``norm_offset`` applies
-_VECTORS = ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "conv_b", "dt_bias", "a_log", "d_skip", "b_if", "sink")
+_VECTORS = ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "conv_b", "dt_bias", "a_log", "d_skip", "b_if", "sink", "b_qkv", "ls1", "ls2", "depth", "act")
+_DERIVED_ONLY = ("wq_up", "wk_up", "wv_up", "map_mix")              # stored tensors that only enter others
 
 
 def packs(m: dict, dtype: torch.dtype, is_cuda: bool) -> bool:
-    """Long spans of this ``window`` layer run on the packed tcgen05 attention."""
-    return is_cuda and dtype == torch.bfloat16 and m["dim"] <= 128
+    """Long spans of this ``window`` or ``diff`` layer run on the packed tcgen05 attention."""
+    return is_cuda and dtype == torch.bfloat16 and max(m["dim"], m["vdim"]) <= 128
 
 
 def cache_width(m: dict, dtype: torch.dtype) -> int:
     """Width of a cached key of a ``window`` layer: what the bf16 kernels take (64 or 128, zeros behind the key), else its own."""
     return m["dim"] if dtype != torch.bfloat16 or m["dim"] > 128 else (64 if m["dim"] <= 64 else 128)
+
+
+def map_widths(m: dict, dtype: torch.dtype) -> tuple[int, int]:
+    """(key width of one map, value width) of a ``diff`` layer in the cache: what the bf16 kernels take (zeros behind the sizes), else exact."""
+    if dtype != torch.bfloat16 or max(m["dim"], m["vdim"]) > 128:
+        return m["dim"], m["vdim"]
+    return next(x for x in (32, 64, 128) if m["dim"] <= x), 64 if m["vdim"] <= 64 else 128
 
 
 def query_width(m: dict, dtype: torch.dtype, is_cuda: bool) -> int:
@@ -185,7 +249,8 @@ def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: di
     previous result) is overwritten in place where shapes agree, so captured graphs stay valid across weight updates."""
     lay = cfg.layers[i]
     m, h = lay["sizes"], lay["sizes"]["heads"]
-    is_cuda = w["norm1"].is_cuda
+    device = w["wo"].device
+    is_cuda = device.type == "cuda"
     out: dict[str, torch.Tensor] = {}
     for k, t in w.items():
         if k in _STREAM_NORMS:
@@ -194,20 +259,25 @@ def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: di
             out[k] = t.float().repeat(h)
         elif k in _VECTORS:
             out[k] = t.float().contiguous()
-        elif k == "conv_w":
+        elif k in ("conv_w", "conv1", "conv2"):
             out[k] = t.float().t().contiguous()                     # [taps, channels]
-        elif k not in ("wq_up", "wk_up", "wv_up"):
+        elif k not in _DERIVED_ONLY:
             t = t if t.dtype == dtype else t.to(dtype)
-            if k in ("w_in", "wqk") and is_cuda and t.shape[0] % 8:
+            if k in ("w_in", "wqk", "wqkv") and is_cuda and t.shape[0] % 8:
                 t = F.pad(t, (0, 0, 0, _pad8(t.shape[0]) - t.shape[0]))
             out[k] = t.contiguous()
     if lay["kind"] == "window":
-        out["freq"] = M.rope_frequencies(m["rot_dim"], m["rot_base"], w["norm1"].device)
-    if "wgu" in out and is_cuda and dtype == torch.bfloat16 and lay["ff"] % 128:
-        # the fused gate / up kernel wants 128-row blocks: zero rows behind the last ones
-        f, pad = lay["ff"], -lay["ff"] % 128
-        out["wgu"] = ref.interleave_gate_up(*(F.pad(t, (0, 0, 0, pad)) for t in (out["wgu"][:f], out["wgu"][f:])))
-        out["wdown"] = F.pad(out["wdown"], (0, pad))
+        out["freq"] = M.rope_frequencies(m["rot_dim"], m["rot_base"], device)
+    if lay["kind"] == "diff":
+        out["freq"] = M.scaled_frequencies(m["rot_dim"], m["rot_base"], m.get("rot_scaling"), device)
+        q1, k1, q2, k2 = w["map_mix"].float().chunk(4)
+        out["lam"] = ((q1 * k1).sum().exp() - (q2 * k2).sum().exp() + m["diff"]).reshape(1)
+    for name, count, f in gate_up_stacks(lay):
+        if is_cuda and dtype == torch.bfloat16 and f % 128:
+            # the fused gate / up kernels want 128-row blocks: zero rows behind the last ones
+            pad, down = -f % 128, {"wgu": "wdown", "ewgu": "ewd", "swgu": "swd"}[name]
+            out[name] = torch.cat([ref.interleave_gate_up(*(F.pad(t, (0, 0, 0, pad)) for t in x.chunk(2))) for x in out[name].chunk(count)])
+            out[down] = F.pad(out[down], (0, pad))
     if lay["kind"] == "latent":
         d, rd, v, r = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
         dq = query_width(m, dtype, is_cuda)
@@ -215,10 +285,10 @@ def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: di
         out["wq"] = _pad_heads(up["wq_up"], h, dq).contiguous()
         out["wk_abs"] = up["wk_up"].reshape(h, d, r).contiguous()                       # folds the key up-projection into a query
         out["wv_abs"] = up["wv_up"].reshape(h, v, r).transpose(1, 2).contiguous()       # folds the value up-projection into an output
-        out["freq"] = M.rope_frequencies(rd, m["rot_base"], w["norm1"].device)
+        out["freq"] = M.rope_frequencies(rd, m["rot_base"], device)
         if expands(m, dtype, is_cuda):
             # cache row -> every head's [key | rotary key | 0] and [value | 0]: the rotary part is copied by identity rows
-            wk = torch.zeros(h, dq, r + rd, dtype=dtype, device=w["norm1"].device)
+            wk = torch.zeros(h, dq, r + rd, dtype=dtype, device=device)
             wk[:, :d, :r] = up["wk_up"].reshape(h, d, r)
             wk[:, d:d + rd, r:] = torch.eye(rd, dtype=dtype, device=wk.device)
             wv = torch.zeros(h, 128, r + rd, dtype=dtype, device=wk.device)
@@ -264,22 +334,34 @@ def cache_bytes(cfg: ModelConfig, dtype: torch.dtype) -> tuple[int, int]:
             tok += (m["kv_rank"] + m["rot_dim"]) * es
         elif lay["kind"] == "window":
             tok += 2 * m["kv_heads"] * cache_width(m, dtype) * es
+        elif lay["kind"] == "diff":
+            kw, vw = map_widths(m, dtype)
+            tok += m["kv_heads"] * (MAPS * kw + vw) * es
         elif lay["kind"] == "delta":
             slot += 4 * h * v * m["dim"] + es * (m["conv"] - 1) * (h * v + 2 * m["kv_heads"] * m["dim"])
         elif lay["kind"] == "ssd":
             slot += 4 * h * v * m["state"] + es * (m["conv"] - 1) * (h * v + 2 * m["groups"] * m["state"])
         else:
             slot += 4 * h * (m["dim"] * v + m["dim"] + 1)
+        slot += es * max(0, cfg.input_conv - 1) * cfg.hidden_size
     return tok, slot
 
 
 def key_views(cfg: ModelConfig) -> list[tuple[int, int]]:
     """The distinct (window, kept first tokens) of the stack's attention layers; (0, 0) sees every key."""
-    return sorted({(lay["sizes"].get("window", 0), lay["sizes"].get("keep_first", 0)) for lay in cfg.layers if lay["kind"] in ("latent", "window")})
+    return sorted({(lay["sizes"].get("window", 0), lay["sizes"].get("keep_first", 0)) for lay in cfg.layers
+                   if lay["kind"] in ("latent", "window", "diff")})
 
 
 def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device, dtype: torch.dtype) -> dict[str, torch.Tensor]:
-    """Cache of layer ``i``: a page pool (attention) or state pools (recurrences; slot 0 belongs to idle batch rows)."""
+    """Cache of layer ``i``: page pools (attention), state pools (recurrences, convolutions; slot 0 belongs to idle batch rows)."""
+    out = _mixer_cache(cfg, i, num_blocks, num_slots, device, dtype)
+    if cfg.input_conv:              # the last inputs of both sublayers' convolutions, which are the same rows
+        out["input"] = torch.zeros(num_slots, cfg.input_conv - 1, cfg.hidden_size, device=device, dtype=dtype)
+    return out
+
+
+def _mixer_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device, dtype: torch.dtype) -> dict[str, torch.Tensor]:
     lay = cfg.layers[i]
     m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
     if lay["kind"] == "latent":
@@ -287,6 +369,9 @@ def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device
     if lay["kind"] == "window":
         shape = (num_blocks, m["kv_heads"], M.PAGE, cache_width(m, dtype))
         return {n: torch.zeros(shape, device=device, dtype=dtype) for n in ("k_pool", "v_pool")}
+    if lay["kind"] == "diff":           # keys [map 1 | map 2]
+        kw, vw = map_widths(m, dtype)
+        return {n: torch.zeros(num_blocks, m["kv_heads"], M.PAGE, x, device=device, dtype=dtype) for n, x in (("k_pool", MAPS * kw), ("v_pool", vw))}
     f32 = dict(device=device, dtype=torch.float32)
     if lay["kind"] == "delta":
         ch = 2 * m["kv_heads"] * m["dim"] + h * v
@@ -391,7 +476,29 @@ def _window(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b:
     return o[..., :d].reshape(t, nh * d)
 
 
-_MIXERS = {"ssd": _ssd, "mlstm": _mlstm, "delta": _delta, "latent": _latent, "window": _window}
+def _diff(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
+    nh, t, window = m["heads"], b.tokens, m["window"]
+    kp, vp, eps = cache["k_pool"], cache["v_pool"], cfg.rms_norm_eps
+    mix = M.MapMix(w["lam"], float(m["diff"]), eps, m["vdim"])
+    tl = b.t_long if packs(m, h.dtype, h.is_cuda) else 0            # tokens served by the packed kernel
+    q, kv = M.map_prep(ops.linear(h, w["wqkv"]), w["b_qkv"], nh, m["dim"], m["vdim"], w["q_norm"], w["k_norm"], w["freq"], kp, vp, b, eps,
+                       tl > 0 and b.gather is None)
+    out = []
+    if tl:
+        if b.gather is None:
+            k, v, cu_k = kv[0][:tl], kv[1][:tl], b.cu[:b.n_long + 1]
+        else:
+            rows, cu_k = b.gather[window, 0]
+            k, v = M.gather_keys(kp, vp, rows)
+        out.append(M.map_attention_varlen(q[:tl], k, v, b.cu[:b.n_long + 1], cu_k, float(m["scale"]), window, mix))
+    if tl < t:
+        lo = b.n_long if tl else 0
+        seq_of = None if b.seq_of is None or tl else b.seq_of[tl:]
+        out.append(M.map_attention(q[tl:], kp, vp, b.table[lo:], seq_of, b.kv_len[tl:], float(m["scale"]), window, mix, b.max_len))
+    return out[0] if len(out) == 1 else torch.cat(out)
+
+
+_MIXERS = {"ssd": _ssd, "mlstm": _mlstm, "delta": _delta, "latent": _latent, "window": _window, "diff": _diff}
 
 
 def layer_step(cfg: ModelConfig, i: int, w: dict, x: torch.Tensor, h: torch.Tensor, cache: dict, b: M.SpanBatch,
@@ -408,10 +515,45 @@ def layer_step(cfg: ModelConfig, i: int, w: dict, x: torch.Tensor, h: torch.Tens
     return M.norm_add_(ops.linear(a, w["wdown"]), x, w["norm2"], eps, w_next)
 
 
+def _feed_forward(cfg: ModelConfig, lay: dict, w: dict, h: torch.Tensor) -> tuple[torch.Tensor | None, M.Routed | None]:
+    """(rows, routed rows that are still to be gathered) of a parallel block's feed-forward."""
+    act = lay.get("act", "gelu")
+    if act == "moe":
+        y = ops.linear(M.linear_silu_glu(h, w["swgu"]), w["swd"]) if "swgu" in w else None
+        return y, M.experts(h, w["router"], w["ewgu"], w["ewd"], lay["top"])
+    if act == "poly":
+        a = M.poly_norm(ops.linear(h, w["wup"]), w["act"], cfg.rms_norm_eps)
+    else:
+        a = M.linear_clamped_glu(h, w["wgu"], lay["limit"], lay["alpha"]) if act == "clamped_glu" else M.linear_gelu(h, w["wup"])
+    return ops.linear(a, w["wdown"]), None
+
+
+def _conv_of(cfg: ModelConfig, w: dict, cache: dict) -> M.InputConv | None:
+    return M.InputConv(w["conv1"], w.get("conv2"), cache["input"]) if cfg.input_conv else None
+
+
+def _forward_parallel(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids: torch.Tensor, caches: list[dict], b: M.SpanBatch,
+                      final_norm: torch.Tensor | None) -> tuple[torch.Tensor, torch.Tensor]:
+    n = len(layer_w)
+    past, h = M.block_embed(ids, embed_w["embed"], n + 1 if cfg.depth_average else 1, layer_w[0]["pre1"], cfg.rms_norm_eps, cfg.layer_norm,
+                            _conv_of(cfg, layer_w[0], caches[0]), b)
+    x = None
+    for i, w in enumerate(layer_w):
+        lay, last = cfg.layers[i], i + 1 == n
+        y1 = ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h[0], caches[i], b), w["wo"])
+        y2, routed = _feed_forward(cfg, lay, w, h[1]) if lay["ff"] else (None, None)
+        x, h = M.block_add(past, i, y1, y2, routed, w.get("ls1"), w.get("ls2"), layer_w[i - 1].get("depth") if i else None, w.get("depth"),
+                           final_norm if last else layer_w[i + 1]["pre1"], cfg.rms_norm_eps, cfg.layer_norm,
+                           None if last else _conv_of(cfg, layer_w[i + 1], caches[i + 1]), b, want_x=last)
+    return x, h[0]
+
+
 def forward(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids: torch.Tensor, caches: list[dict], b: M.SpanBatch,
             final_norm: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """The stack on one packed step: (fp32 residual stream after the last layer, the same in the activation dtype — normed with
     ``final_norm`` when that is given)."""
+    if cfg.parallel_block:
+        return _forward_parallel(cfg, embed_w, layer_w, ids, caches, b, final_norm)
     x, h = M.embed(ids, embed_w["embed"], layer_w[0].get("pre1"), cfg.rms_norm_eps)
     for i, w in enumerate(layer_w):
         h = layer_step(cfg, i, w, x, h, caches[i], b, layer_w[i + 1].get("pre1") if i + 1 < len(layer_w) else final_norm)

@@ -12,7 +12,7 @@ import torch
 
 from ..ops import reference as ref
 from .config import ModelConfig
-from .hybrid import owner
+from .hybrid import gate_up_stacks, owner
 
 
 @dataclass(frozen=True)
@@ -22,8 +22,9 @@ class Design:
     read_layer: Callable                # (entry of config.json's layers, kind, index) -> {"sizes", "ff", ...}
     write_layer: Callable               # (layer of ModelConfig.layers) -> {"mixer", "mlp"}
     parts: Callable                     # (cfg, i) -> [(our name, [checkpoint names whose rows it stacks], [rows of each])]
-    glu: bool = False                   # feed-forward is gate / up / down
-    model_fields: dict = None           # further ModelConfig fields of the design
+    mlp_kinds: tuple = ("dense",)       # feed-forward kinds of config.json
+    read_model: Callable = lambda hf: {}            # config.json -> further ModelConfig fields of the design
+    write_model: Callable = lambda cfg: {}          # and back: further entries of config.json
 
 
 def stack_config(design: Design, hf: dict) -> ModelConfig:
@@ -32,14 +33,14 @@ def stack_config(design: Design, hf: dict) -> ModelConfig:
         if e["type"] not in design.kinds:
             raise ValueError(f"{design.architecture} layer {i}: unknown mixer type {e['type']!r}")
         mlp = e.get("mlp")
-        if mlp and mlp.get("kind", "dense") != "dense":
+        if mlp and mlp.get("kind", "dense") not in design.mlp_kinds:
             raise ValueError(f"{design.architecture} layer {i}: feed-forward kind {mlp['kind']!r}")
         kind = design.kinds[e["type"]]
-        layers.append({"kind": kind, "ff": int(mlp["ff"]) if mlp else 0, "weights_of": int(e.get("weights_of", i)), **design.read_layer(e, kind, i)})
+        layers.append({"kind": kind, "ff": int(mlp.get("ff", 0)) if mlp else 0, "weights_of": int(e.get("weights_of", i)), **design.read_layer(e, kind, i)})
     return ModelConfig(family="hybrid", vocab_size=hf["vocab"], hidden_size=hf["width"], num_layers=len(layers), layers=tuple(layers),
                        intermediate_size=max([x["ff"] for x in layers] + [1]), num_heads=1, num_kv_heads=1, rms_norm_eps=float(hf["norm"]["eps"]),
                        eos_token_id=-1, bos_token_id=-1, pad_token_id=0, hf_model_type=design.architecture.lower(), name=design.architecture.lower(),
-                       **(design.model_fields or {}))
+                       **design.read_model(hf))
 
 
 def stack_config_dict(cfg: ModelConfig) -> dict:
@@ -52,10 +53,19 @@ def stack_config_dict(cfg: ModelConfig) -> dict:
         if lay["weights_of"] != i:
             e["weights_of"] = lay["weights_of"]
         layers.append(e)
-    return {"architecture": design.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "norm": {"eps": cfg.rms_norm_eps}, "layers": layers}
+    return {"architecture": design.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "norm": {"eps": cfg.rms_norm_eps}, "layers": layers,
+            **design.write_model(cfg)}
 
 
 _MODEL_NAMES = {"embed": "embed", "norm_w": "final.norm", "lm_head": "head"}
+
+
+def _map_gate_up(cfg: ModelConfig, i: int, t: dict, fn: Callable) -> None:
+    """Replace every stack of gate and up rows of layer ``i`` by ``fn(rows)``, expert by expert, where the width has whole blocks of 128."""
+    for name, count, width in gate_up_stacks(cfg.layers[i]):
+        if width % 128 == 0:
+            key = f"layers.{i}.{name}"
+            t[key] = torch.cat([fn(x) for x in t[key].chunk(count)])
 
 
 def stack_state_dict(cfg: ModelConfig, get) -> dict[str, torch.Tensor]:
@@ -71,24 +81,22 @@ def stack_state_dict(cfg: ModelConfig, get) -> dict[str, torch.Tensor]:
         if design.kinds.get("mamba2") == lay["kind"]:            # one checkpoint tensor [in | step sizes] is two of ours
             w, nh = get(p + "mix.in"), lay["sizes"]["heads"]
             out[q + "w_in"], out[q + "w_dt"] = w[:-nh], w[-nh:]
-        if design.glu and lay["ff"] and lay["ff"] % 128 == 0:
-            f = lay["ff"]
-            out[q + "wgu"] = ref.interleave_gate_up(out[q + "wgu"][:f], out[q + "wgu"][f:])
+        _map_gate_up(cfg, i, out, lambda x: ref.interleave_gate_up(*x.chunk(2)))
     return out
 
 
 def stack_export(cfg: ModelConfig, sd: dict) -> dict[str, torch.Tensor]:
     """Our names -> checkpoint names (inverse of ``stack_state_dict``)."""
     design = DESIGNS[cfg.hf_model_type]
+    sd = dict(sd)
     out = {s: sd[n] for n, s in _MODEL_NAMES.items()}
     for i, lay in enumerate(cfg.layers):
         if owner(cfg, i) != i:
             continue
         p, q = f"l{i}.", f"layers.{i}."
+        _map_gate_up(cfg, i, sd, lambda x: torch.cat(ref.deinterleave_gate_up(x)))
         for n, names, rows in design.parts(cfg, i):
             t = sd[q + n]
-            if n == "wgu" and lay["ff"] % 128 == 0:
-                t = torch.cat(ref.deinterleave_gate_up(t))
             if len(names) == 1:
                 out[p + names[0]] = t
             else:
@@ -188,8 +196,71 @@ def _lanilix_parts(cfg: ModelConfig, i: int) -> list:
     return out
 
 
+# --------------------------------------------------------------------------------------------
+# Mabedra: differential attention in a sliding window; parallel blocks behind layer norms, with input convolutions, layer scales and
+# averages over depth; dense layers with a polynomial activation, sparse ones with a sigmoid router and a shared expert
+# --------------------------------------------------------------------------------------------
+_MABEDRA_SIZES = ("heads", "kv_heads", "dim", "vdim", "scale", "diff")
+_MABEDRA_MAPS = 2
+
+
+def _mabedra_read(e: dict, kind: str, i: int) -> dict:
+    m, mlp = e["mixer"], e.get("mlp")
+    rot = m["rot"]
+    sizes = {k: m[k] for k in _MABEDRA_SIZES}
+    sizes.update(window=int(m["mask"]["size"]), rot_dim=int(rot["dims"]), rot_base=float(rot["base"]))
+    if rot.get("scaling"):
+        sizes["rot_scaling"] = {k: float(rot["scaling"][k]) for k in ("factor", "low", "high", "original")}
+    out = {"sizes": sizes}
+    if mlp and mlp["kind"] == "moe":
+        out.update(act="moe", ff=int(mlp["expert"]["ff"]), experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]),
+                   shared=int(mlp["shared"]["ff"]) if mlp.get("shared") else 0)
+    elif mlp:
+        out["act"] = "poly"
+    return out
+
+
+def _mabedra_write(lay: dict) -> dict:
+    s, mlp = lay["sizes"], None
+    mx = {k: s[k] for k in _MABEDRA_SIZES}
+    mx.update(mask={"size": s["window"]}, rot={"dims": s["rot_dim"], "base": s["rot_base"]})
+    if "rot_scaling" in s:
+        mx["rot"]["scaling"] = dict(s["rot_scaling"])
+    if lay["ff"] and lay["act"] == "moe":
+        mlp = {"kind": "moe", "expert": {"ff": lay["ff"]}, "router": {"experts": lay["experts"], "top": lay["top"]}}
+        if lay["shared"]:
+            mlp["shared"] = {"ff": lay["shared"]}
+    elif lay["ff"]:
+        mlp = {"kind": "dense", "ff": lay["ff"]}
+    return {"mixer": mx, "mlp": mlp}
+
+
+def _mabedra_parts(cfg: ModelConfig, i: int) -> list:
+    lay = cfg.layers[i]
+    m, h, g, f = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["kv_heads"], lay["ff"]
+    rows = [_MABEDRA_MAPS * h * m["dim"], _MABEDRA_MAPS * g * m["dim"], g * m["vdim"]]
+    out = [("wqkv", ["mix.q", "mix.k", "mix.v"], rows), ("b_qkv", ["mix.q.b", "mix.k.b", "mix.v.b"], rows), _one("q_norm", "mix.q.norm"),
+           _one("k_norm", "mix.k.norm"), ("map_mix", ["mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"], [m["dim"]] * 4), _one("wo", "mix.o"),
+           _one("pre1", "norm1"), _one("ls1", "ls1"), _one("conv1", "canon1"), _one("depth", "dwa")]
+    if not f:
+        return out
+    out += [_one("ls2", "ls2"), _one("conv2", "canon2")]
+    if lay["act"] == "poly":
+        return out + [_one("wup", "mlp.up"), _one("wdown", "mlp.down"), _one("act", "mlp.act")]
+    n = lay["experts"]
+    out += [("ewgu", [f"mlp.e{j}.{k}" for j in range(n) for k in ("gate", "up")], [f] * (2 * n)),
+            ("ewd", [f"mlp.e{j}.down" for j in range(n)], [cfg.hidden_size] * n), _one("router", "mlp.router")]
+    if lay["shared"]:
+        out += [("swgu", ["mlp.shared.gate", "mlp.shared.up"], [lay["shared"]] * 2), _one("swd", "mlp.shared.down")]
+    return out
+
+
 DESIGNS = {
     "ludesun": Design("Ludesun", {"mamba2": "ssd", "mlstm": "mlstm", "latent_attention": "latent"}, _ludesun_read, _ludesun_write, _ludesun_parts),
-    "lanilix": Design("Lanilix", {"delta": "delta", "attention": "window"}, _lanilix_read, _lanilix_write, _lanilix_parts, glu=True,
-                      model_fields={"sandwich_norm": True, "norm_offset": 1.0}),
+    "lanilix": Design("Lanilix", {"delta": "delta", "attention": "window"}, _lanilix_read, _lanilix_write, _lanilix_parts,
+                      read_model=lambda hf: {"sandwich_norm": True, "norm_offset": 1.0}),
+    "mabedra": Design("Mabedra", {"attention": "diff"}, _mabedra_read, _mabedra_write, _mabedra_parts, mlp_kinds=("dense", "moe"),
+                      read_model=lambda hf: {"parallel_block": True, "layer_norm": True, "layer_scale": True, "depth_average": True,
+                                             "input_conv": int(hf["canon"]["taps"])},
+                      write_model=lambda cfg: {"canon": {"taps": cfg.input_conv}}),
 }

@@ -7,6 +7,7 @@ Spans are ordered: the ``n_long`` spans of several tokens first, then the single
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 
 import torch
@@ -98,11 +99,15 @@ def norm_add_(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, eps: float, w_n
     return x if y.dtype == torch.float32 else x.to(y.dtype)
 
 
-def rms(x: torch.Tensor, w: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
-    """rms(x) * w of fp32 rows in ``dtype``."""
+def _norm(x: torch.Tensor, eps: float, center: bool) -> torch.Tensor:
+    return _rms(x - x.mean(-1, keepdim=True) if center else x, eps)
+
+
+def rms(x: torch.Tensor, w: torch.Tensor, eps: float, dtype: torch.dtype, center: bool = False) -> torch.Tensor:
+    """rms(x) * w of fp32 rows in ``dtype``; ``center``: of x minus its mean (layer norm)."""
     if x.is_cuda:
-        return _C().mix_rms(x.contiguous(), w, eps, dtype == torch.bfloat16)
-    return (_rms(x, eps) * w).to(dtype)
+        return _C().mix_rms(x.contiguous(), w, eps, dtype == torch.bfloat16, center)
+    return (_norm(x, eps, center) * w).to(dtype)
 
 
 SIGMOID_LAST, SILU_FIRST, SILU_LAST = 0, 1, 2
@@ -149,6 +154,149 @@ def linear_clamped_glu(x: torch.Tensor, wgu: torch.Tensor, limit: float, alpha: 
     g, u = split_gate_up(gu.float()) if f % 128 == 0 else gu.float().split(f, -1)
     g = g.clamp(max=limit)
     return (g * torch.sigmoid(alpha * g) * (u.clamp(-limit, limit) + 1)).to(x.dtype)
+
+
+def linear_silu_glu(x: torch.Tensor, wgu: torch.Tensor) -> torch.Tensor:
+    """silu(gate) * up; ``wgu`` laid out as in ``linear_clamped_glu``.  Fused into the GEMM epilogue for bf16 rows."""
+    f = wgu.shape[0] // 2
+    if x.is_cuda and x.dtype == torch.bfloat16 and f % 128 == 0 and x.shape[1] % 8 == 0:
+        return _C().gemm_silu_glu(x, wgu)
+    return silu_glu(F.linear(x, wgu.to(x.dtype)), f)
+
+
+def silu_glu(gu: torch.Tensor, f: int) -> torch.Tensor:
+    if gu.is_cuda:
+        return _C().mix_silu_glu(gu, 128 if f % 128 == 0 else f)
+    g, u = split_gate_up(gu.float()) if f % 128 == 0 else gu.float().split(f, -1)
+    return (F.silu(g) * u).to(gu.dtype)
+
+
+def poly_norm(z: torch.Tensor, act: torch.Tensor, eps: float) -> torch.Tensor:
+    """a N(z) + b N(z^2) + c N(z^3) + e with N(u) = u / sqrt(mean(u^2) + eps) over a row and act = [a, b, c, e]."""
+    if z.is_cuda:
+        return _C().mix_poly_norm(z, act, eps)
+    x = z.float()
+    return (act[0] * _rms(x, eps) + act[1] * _rms(x * x, eps) + act[2] * _rms(x ** 3, eps) + act[3]).to(z.dtype)
+
+
+# --------------------------------------------------------------------------------------------
+# parallel blocks: results of the layers so far, input convolutions
+# --------------------------------------------------------------------------------------------
+@dataclass
+class InputConv:
+    """h -> h + conv(h) for one or two sublayers that read the same h: weights [taps, ch] (last row: the current token), and the state
+    [slots, taps - 1, ch] that both share."""
+    w1: torch.Tensor
+    w2: torch.Tensor | None
+    state: torch.Tensor
+
+
+@dataclass
+class Routed:
+    """Rows of ``experts`` in the experts' order; row ``pos[t, j]`` belongs to token t."""
+    rows: torch.Tensor
+    pos: torch.Tensor
+
+    def sum(self) -> torch.Tensor:
+        return self.rows.float()[self.pos.long()].sum(1)
+
+
+def input_conv(h: torch.Tensor, conv: InputConv | None, b: SpanBatch) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """What the two sublayers read (the second is None when there is no second weight)."""
+    if conv is None:
+        return h, h
+    if h.is_cuda:
+        out = _C().mix_input_conv(h, conv.w1, conv.w2, conv.state, b.cu, b.start, b.slot, b.seq_of)
+        return out[0], (out[1] if conv.w2 is not None else None)
+    taps = conv.w1.shape[0]
+    out = [None if w is None else torch.empty_like(h) for w in (conv.w1, conv.w2)]
+    cu = b.cu.tolist()
+    for s in range(b.spans):
+        lo, hi = cu[s], cu[s + 1]
+        old = conv.state[b.slot[s]] if int(b.start[s]) else torch.zeros_like(conv.state[0])
+        full = torch.cat([old, h[lo:hi]]).float()
+        for o, w in zip(out, (conv.w1, conv.w2)):
+            if o is not None:
+                o[lo:hi] = (full[taps - 1:] + sum(w[j] * full[j:j + hi - lo] for j in range(taps))).to(h.dtype)
+        conv.state[b.slot[s]] = full[full.shape[0] - (taps - 1):].to(h.dtype)
+    return out[0], out[1]
+
+
+def _fused_conv(conv: InputConv | None, b: SpanBatch) -> tuple:
+    """Arguments of the kernels that end in the convolution of single tokens, or nothing."""
+    return (None,) * 5 if conv is None or b.seq_of is not None else (conv.w1, conv.w2, conv.state, b.start, b.slot)
+
+
+def block_embed(ids: torch.Tensor, w: torch.Tensor, slots: int, w_norm: torch.Tensor, eps: float, center: bool, conv: InputConv | None,
+                b: SpanBatch) -> tuple[torch.Tensor, tuple]:
+    """(results of the layers [slots, T, W] in fp32 with the embedding in the first, what the first layer's sublayers read)."""
+    if w.is_cuda:
+        past, *h = _C().mix_block_embed(ids, w, slots, w_norm, eps, center, *_fused_conv(conv, b))
+        return past, _read(h, conv, b)
+    x = F.embedding(ids, w).float()
+    past = x.new_empty(slots, *x.shape)
+    past[0] = x
+    return past, input_conv((_norm(x, eps, center) * w_norm).to(w.dtype), conv, b)
+
+
+def _read(h: list, conv: InputConv | None, b: SpanBatch) -> tuple:
+    if conv is None:
+        return h[0], h[0]
+    return input_conv(h[0], conv, b) if b.seq_of is not None else (h[0], h[1] if conv.w2 is not None else None)
+
+
+def block_add(past: torch.Tensor, i: int, y1: torch.Tensor, y2: torch.Tensor | None, routed: Routed | None, s1: torch.Tensor | None,
+              s2: torch.Tensor | None, a_prev: torch.Tensor | None, a_cur: torch.Tensor | None, w_next: torch.Tensor | None, eps: float, center: bool,
+              conv: InputConv | None, b: SpanBatch, want_x: bool = False) -> tuple[torch.Tensor | None, tuple]:
+    """Layer ``i`` of a stack of parallel blocks:  X = x + s1 y1 + s2 (y2 + sum of its routed rows)  with x = sum_j a_prev[j] past[j] (past[0]
+    without ``a_prev``), then x' = sum_j a_cur[j] past[j] + a_cur[i + 1] X.  X goes to past[i + 1] (without averages: to past[0], and x' = X).
+    Returns (x' in fp32 if wanted, what the next layer's sublayers read: norm(x') * w_next through ``conv``)."""
+    if y1.is_cuda:
+        rows, pos = (routed.rows, routed.pos) if routed is not None else (None, None)
+        x, *h = _C().mix_block_add(past, i, y1, y2, rows, pos, s1, s2, a_prev, a_cur, w_next, eps, center, want_x, *_fused_conv(conv, b))
+        return (x if want_x else None), ((None, None) if w_next is None else _read(h, conv, b))
+    x = past[0].clone() if a_prev is None else torch.einsum("j,jtw->tw", a_prev, past[:i + 1])
+    y = y1.float() if s1 is None else y1.float() * s1
+    if y2 is not None or routed is not None:
+        f = (0 if y2 is None else y2.float()) + (0 if routed is None else routed.sum())
+        y = y + (f if s2 is None else f * s2)
+    x = x + y
+    past[0 if a_cur is None else i + 1] = x
+    if a_cur is not None:
+        x = torch.einsum("j,jtw->tw", a_cur, past[:i + 2])
+    return (x if want_x else None), ((None, None) if w_next is None else input_conv((_norm(x, eps, center) * w_next).to(y1.dtype), conv, b))
+
+
+# --------------------------------------------------------------------------------------------
+# experts
+# --------------------------------------------------------------------------------------------
+TILE = 128              # rows of the expert kernels' tiles: every expert's rows start on one
+
+
+def experts(h: torch.Tensor, router: torch.Tensor, wgu: torch.Tensor, wd: torch.Tensor, top: int) -> Routed:
+    """Silu-gated experts on weighted inputs: token t goes to the ``top`` experts with the largest s = sigmoid(router h), each reads s h.
+    wgu [E * 2 F, W] holds every expert's gate and up rows as in ``linear_silu_glu``, wd [E * W, F].  No host synchronisation."""
+    e, width = router.shape[0], h.shape[1]
+    f = wgu.shape[0] // (2 * e)
+    logits = linear_f32(h, router)
+    if h.is_cuda:
+        C = _C()
+        pick, score, rank, plan = C.mix_route(logits, top)
+        rows, pos = C.mix_expert_rows(h, pick, score, rank, plan)
+        if h.dtype == torch.bfloat16 and f % 128 == 0 and width % 8 == 0:
+            return Routed(C.gemm_experts(C.gemm_experts(rows, wgu, plan, True), wd, plan, False), pos)
+        gu = C.mix_expert_gemm(rows, wgu, plan)
+        return Routed(C.mix_expert_gemm(silu_glu(gu, f), wd, plan), pos)
+    score, pick = torch.topk(torch.sigmoid(logits), top, dim=-1)
+    rows = h.new_empty(h.shape[0] * top, width)
+    pos = torch.arange(rows.shape[0]).reshape(-1, top)
+    x = (h.float()[:, None] * score[..., None]).to(h.dtype)
+    for j in range(e):
+        t, k = (pick == j).nonzero(as_tuple=True)
+        if t.numel():
+            a = silu_glu(F.linear(x[t, k], wgu[j * 2 * f:(j + 1) * 2 * f]), f)
+            rows[pos[t, k]] = F.linear(a, wd[j * width:(j + 1) * width])
+    return Routed(rows, pos)
 
 
 # --------------------------------------------------------------------------------------------
@@ -274,6 +422,16 @@ def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
 def rope_frequencies(dims: int, base: float, device) -> torch.Tensor:
     """base^(-2 i / dims), i < dims / 2, double precision (angles are reduced before the fp32 sine / cosine)."""
     return torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=device)
+
+
+def scaled_frequencies(dims: int, base: float, scaling: dict | None, device) -> torch.Tensor:
+    """``rope_frequencies`` with Llama 3.1's scaling {"factor", "low", "high", "original"}: wavelengths above original / low are stretched by
+    ``factor``, those below original / high stay, the ones between are blended."""
+    f = rope_frequencies(dims, base, "cpu")
+    if scaling:
+        s = ((scaling["original"] * f / (2 * math.pi) - scaling["low"]) / (scaling["high"] - scaling["low"])).clamp(0, 1)
+        f = (1 - s) * f / scaling["factor"] + s * f
+    return f.to(device)
 
 
 def _rotate(x: torch.Tensor, freq: torch.Tensor, pos: torch.Tensor) -> torch.Tensor:
@@ -415,3 +573,92 @@ def window_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, c
                             keep_first: int) -> torch.Tensor:
     """Packed spans, bottom-right aligned: the tcgen05 kernel, width 64 or 128, bf16."""
     return _C().attn_fwd(q, k, v, cu_q, cu_k, scale, True, False, None, None, window, keep_first)[0]
+
+
+# --------------------------------------------------------------------------------------------
+# differential attention: two softmax maps per head over the same values
+# --------------------------------------------------------------------------------------------
+@dataclass
+class MapMix:
+    """o = a1 - lam a2,  o / sqrt(mean(o^2) + eps) * (1 - diff)  over the ``vdim`` values of a head."""
+    lam: torch.Tensor           # [1] fp32
+    diff: float
+    eps: float
+    vdim: int
+
+    def __call__(self, a1: torch.Tensor, a2: torch.Tensor) -> torch.Tensor:
+        return _rms((a1 - self.lam * a2)[..., :self.vdim], self.eps) * (1 - self.diff)
+
+
+def query_map_width(kw: int, dtype: torch.dtype) -> int:
+    """Width of a map's query at run time: the keys' — or 64 for bf16 keys of width 32, whose two maps share one 64-wide row: the query of map m
+    then lies at column 32 m, zeros beside it."""
+    return 64 if kw == 32 and dtype == torch.bfloat16 else kw
+
+
+def map_prep(p: torch.Tensor, bias: torch.Tensor, heads: int, dim: int, vdim: int, wq: torch.Tensor, wk: torch.Tensor, freq: torch.Tensor,
+             k_pool: torch.Tensor, v_pool: torch.Tensor, b: SpanBatch, eps: float, want_kv: bool) -> tuple[torch.Tensor, tuple | None]:
+    """Rows [queries: heads x 2 maps x dim | keys: groups x 2 maps x dim | values: groups x vdim] as projected, without their ``bias`` -> queries
+    [T, 2 heads, query_map_width], RMS-normed per map and rotated (entries i and i + freq.numel()); the keys treated alike go to ``k_pool``
+    ([pages, groups, PAGE, 2 key widths]) and the values to ``v_pool``.  Packed keys and values are returned too when asked for."""
+    g, kw, vw = k_pool.shape[1], k_pool.shape[3] // 2, v_pool.shape[3]
+    qw = query_map_width(kw, p.dtype)
+    if p.is_cuda:
+        q, k, v = _C().mix_map_prep(p, bias, heads, dim, vdim, wq, wk, freq, b.pos, b.kv_slot, k_pool, v_pool, eps, want_kv, qw)
+        return q, ((k, v) if want_kv else None)
+    t, nq = p.shape[0], 2 * heads * dim
+    x = p.float()[:, :nq + 2 * g * dim + g * vdim] + bias
+    a = torch.outer(b.pos.double(), freq)
+    c, s = a.cos().float()[:, None], a.sin().float()[:, None]
+
+    def turned(y, w):
+        y = _rms(y.reshape(t, -1, dim), eps) * w
+        n = freq.numel()
+        u, v, rest = y[..., :n], y[..., n:2 * n], y[..., 2 * n:]
+        return torch.cat([u * c - v * s, v * c + u * s, rest], -1).to(p.dtype)
+
+    q, k = turned(x[:, :nq], wq), F.pad(turned(x[:, nq:nq + 2 * g * dim], wk), (0, kw - dim)).reshape(t, g, 2 * kw)
+    v = F.pad(x[:, nq + 2 * g * dim:].reshape(t, g, vdim), (0, vw - vdim)).to(p.dtype)
+    if qw == kw:
+        q = F.pad(q, (0, qw - dim))
+    else:
+        q = torch.stack([F.pad(q[:, m::2], (m * kw, qw - m * kw - dim)) for m in range(2)], 2).reshape(t, 2 * heads, qw)
+    page, off = b.kv_slot // PAGE, b.kv_slot % PAGE
+    k_pool[page, :, off], v_pool[page, :, off] = k, v
+    return q, ((k, v) if want_kv else None)
+
+
+def map_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, table: torch.Tensor, seq_of: torch.Tensor | None, kv_len: torch.Tensor,
+                  scale: float, window: int, mix: MapMix, max_len: int) -> torch.Tensor:
+    """Paged form, one query row per entry of ``kv_len`` (its own token is its last key, it sees the last ``window``): [rows, heads * vdim]."""
+    rows, h, qw = q.shape[0], q.shape[1] // 2, q.shape[2]
+    g, kw = k_pool.shape[1], k_pool.shape[3] // 2
+    if q.is_cuda:
+        if q.dtype == torch.bfloat16 and _C().map_decode_ok(kw, v_pool.shape[3], h // g) and seq_of is None:
+            from .functional import _auto_splits
+
+            return _C().map_decode(q, k_pool, v_pool, table, kv_len, scale, _auto_splits(rows, g, min(max_len, window + 2 * PAGE)), window, mix.lam, mix.diff,
+                                   mix.eps, mix.vdim)
+        return _C().mix_map_attention(q, k_pool, v_pool, table, seq_of, kv_len, scale, window, mix.lam, mix.diff, mix.eps, mix.vdim)
+    out = q.new_zeros(rows, h, mix.vdim)
+    for i in range(rows):
+        n = int(kv_len[i])
+        if n == 0:
+            continue
+        pages = table[int(seq_of[i]) if seq_of is not None else i, : (n + PAGE - 1) // PAGE].long()
+        j = torch.arange(max(0, n - window), n)
+        k, v = (x[pages[j // PAGE], :, j % PAGE].float().repeat_interleave(h // g, 1) for x in (k_pool, v_pool))
+        a = []
+        for m in range(2):
+            km = k if qw != kw else k[..., m * kw:(m + 1) * kw]
+            p = torch.softmax(torch.einsum("hd,jhd->hj", q[i, m::2].float(), km) * scale, -1)
+            a.append(torch.einsum("hj,jhd->hd", p, v))
+        out[i] = mix(*a).to(q.dtype)
+    return out.reshape(rows, -1)
+
+
+def map_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.Tensor, cu_k: torch.Tensor, scale: float, window: int,
+                         mix: MapMix) -> torch.Tensor:
+    """Packed spans, bottom-right aligned, q [T, 2 heads, width], k [Tk, groups, 2 key widths], v [Tk, groups, value width]: the tcgen05 kernel
+    with both maps of a head in one CTA and their difference in its epilogue -> [T, heads * vdim] (bf16)."""
+    return _C().map_attn_fwd(q, k, v, cu_q, cu_k, scale, window, mix.lam, mix.diff, mix.eps, mix.vdim)

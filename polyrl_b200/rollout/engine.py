@@ -905,7 +905,7 @@ class RolloutEngine:
         if self.hybrid:
             from ..ops import mixers
 
-            h = mixers.rms(x.index_select(0, rows), self.head_w["norm_w"], self.cfg.rms_norm_eps, self.dtype)
+            h = mixers.rms(x.index_select(0, rows), self.head_w["norm_w"], self.cfg.rms_norm_eps, self.dtype, self.cfg.layer_norm)
         else:
             h = tf.final_norm(self.cfg, self.head_w, x.index_select(0, rows))
         return self._lm_logits(h)
