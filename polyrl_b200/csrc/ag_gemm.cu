@@ -18,7 +18,7 @@ namespace prl {
 
 constexpr int kAgMaxPeers = 16;
 
-struct AgComm {
+struct AgComm : NoComm {
   static constexpr int kCommWarps = 2;
   struct Params {
     const int4* shard[kAgMaxPeers];   // peer shard base pointers (index = rank)

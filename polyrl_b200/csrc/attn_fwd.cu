@@ -1,4 +1,5 @@
-// polyrl_b200 — varlen causal flash-attention FORWARD on tcgen05 / TMEM / TMA (query / key width 64, 128 or 192, value width 64 or 128, GQA).
+// polyrl_b200 — varlen causal flash-attention FORWARD on tcgen05 / TMEM / TMA (query / key width 64, 128 or 192, value width 64 or 128, GQA,
+// one or two softmax maps per head).
 //
 // Replaces the flash-attn 2 library call (mma.sync) the reference reaches through
 // 3rdparty/verl/verl/models/transformers/monkey_patch.py:49-117 (`_flash_attention_forward`) for training,
@@ -18,6 +19,9 @@
 // DK = 192 (latent attention expanded to heads: 128 + 64 rotary) keeps both K stages and drops to one V stage, which is
 // reloaded while the next scores and their softmax run.  An optional per-head sink adds exp(sink_h) to the softmax
 // denominator in the epilogue.
+// Two maps per head (differential attention): the CTA runs the loop twice over the same values, keeps the first map's output in
+// TMEM (fp32) and writes  (a1 - lambda a2) / sqrt(mean^2 + eps) * keep.  Keys of width 32 lie pairwise in rows of 64 (both maps read
+// the same row, the queries are zero outside their half).
 // A sliding window with kept first tokens (query i sees key j if i - j < window or j < keep_first) skips the key tiles between the
 // kept ones and the window of the tile's first query.
 // Epilogue: O / l -> bf16 (16-byte stores), log-sum-exp per (head, token) for the backward pass.
@@ -28,13 +32,12 @@ namespace prl {
 constexpr int kAfThreads = 320;          // warp0 TMA, warp1 MMA, warps 2-5 + 6-9: two softmax warpgroups
 constexpr int kAfBM = 128, kAfBN = 128;
 constexpr int kAfTile = 128 * 128 * 2;              // 32 KB: one 128 x 128 bf16 operand tile (2 chunks of 64 columns)
-template <int DK>
+template <int DK, int DV, int MAPS>
 struct AfCfg {
   static constexpr int QKT = 128 * DK * 2;            // Q or K tile: DK / 64 chunks of 128 rows x 64 columns
-  static constexpr int DV = DK == 64 ? 64 : 128;      // value width
   static constexpr int VT = 128 * DV * 2;             // V tile
-  static constexpr int VST = DK <= 128 ? 2 : 1;       // V stages
-  static constexpr int SMEM = 3 * QKT /*Q, K x 2*/ + VST * VT /*V*/ + kAfTile /*P*/ + 1024 + 256;
+  static constexpr int VST = DK * MAPS + DV <= 256 ? 2 : 1;       // V stages
+  static constexpr int SMEM = (MAPS + 2) * QKT /*Q, K x 2*/ + VST * VT /*V*/ + kAfTile /*P*/ + 1024 + 256;
 };
 
 struct AttnFwdParams {
@@ -43,25 +46,29 @@ struct AttnFwdParams {
   const int32_t* cu_q;         // [B+1]
   const int32_t* cu_k;         // [B+1]
   int64_t ldo;
-  int B, nq, nkv, Tq;
+  int B, nq, nkv, Tq;          // nq: output heads (q holds MAPS of each)
   float scale_log2;            // sm_scale * log2(e)
   float sm_scale;
   int causal;
   int window, keep_first;      // window: 0x7fffffff when every earlier key is seen
   const float* sink;           // [nq] or null: natural-log sink of the softmax denominator
+  const float* lam;            // two maps: [1] weight of the second
+  float keep, eps;             // two maps: factor behind the norm, and what is added under its root
+  int dv_out, shared_row;      // two maps: values of a head that are written (<= DV); both maps' keys in one row
   long long* dbg;              // optional timeline buffer (kernel experiments)
 };
 
-template <int DK>
+template <int DK, int kAfD, int MAPS>
 __global__ void __launch_bounds__(kAfThreads, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                 const __grid_constant__ CUtensorMap tmV, AttnFwdParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
-  constexpr int QKT = AfCfg<DK>::QKT, VST = AfCfg<DK>::VST, VT = AfCfg<DK>::VT, kAfD = AfCfg<DK>::DV, OW = kAfD / 2;
-  uint8_t* sK = smem + QKT;                           // [2 stages]
-  uint8_t* sV = smem + 3 * QKT;                       // [VST stages]
+  using Cfg = AfCfg<DK, kAfD, MAPS>;
+  constexpr int QKT = Cfg::QKT, VST = Cfg::VST, VT = Cfg::VT, OW = kAfD / 2;
+  uint8_t* sK = smem + MAPS * QKT;                    // [2 stages]
+  uint8_t* sV = smem + (MAPS + 2) * QKT;              // [VST stages]
   uint8_t* sP = sV + VST * VT;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + kAfTile);
   uint64_t* q_full = bars;            // 1
@@ -76,7 +83,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   uint64_t* v_empty = bars + 14;      // [2]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
   __shared__ int s_seq, s_q0;
-  __shared__ float s_mx[2][2][128];             // [tile parity][warpgroup][row]: half-row maxima / sums
+  __shared__ float s_mx[2][2][128];             // [tile parity][warpgroup][row]: half-row maxima
+  __shared__ float s_sum[MAPS][2][128];         // half-row sums
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y;
@@ -127,21 +135,22 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 
   if (warp == 0) {
     if (lane == 0) {
-      mbar_expect_tx(q_full, QKT);
+      mbar_expect_tx(q_full, MAPS * QKT);
 #pragma unroll
-      for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmQ, q_full, sQ + c * 16384, h * DK + c * 64, qs + q0);
-      for (int j = 0; j < nt; ++j) {
-        const int s = j & 1;
+      for (int c = 0; c < MAPS * DK / 64; ++c) tma_load_2d(&tmQ, q_full, sQ + c * 16384, h * MAPS * DK + c * 64, qs + q0);
+      for (int j = 0; j < MAPS * nt; ++j) {               // two maps: the key tiles of the first, then those of the second
+        const int s = j & 1, map = MAPS == 2 && j >= nt ? 1 : 0, key0 = ks + tile_of(j - map * nt) * kAfBN;
+        const int kcol = (MAPS == 1 || p.shared_row ? hk : hk * MAPS + map) * DK;
         const uint32_t ph = (j >> 1) & 1;
         const int sv = j % VST;
         mbar_wait(&k_empty[s], ph ^ 1);
         mbar_expect_tx(&k_full[s], QKT);
 #pragma unroll
-        for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmK, &k_full[s], sK + s * QKT + c * 16384, hk * DK + c * 64, ks + tile_of(j) * kAfBN);
+        for (int c = 0; c < DK / 64; ++c) tma_load_2d(&tmK, &k_full[s], sK + s * QKT + c * 16384, kcol + c * 64, key0);
         mbar_wait(&v_empty[sv], ((j / VST) & 1) ^ 1);
         mbar_expect_tx(&v_full[sv], VT);
 #pragma unroll
-        for (int c = 0; c < kAfD / 64; ++c) tma_load_2d(&tmV, &v_full[sv], sV + sv * VT + c * 16384, hk * kAfD + c * 64, ks + tile_of(j) * kAfBN);
+        for (int c = 0; c < kAfD / 64; ++c) tma_load_2d(&tmV, &v_full[sv], sV + sv * VT + c * 16384, hk * kAfD + c * 64, key0);
       }
     }
   } else if (warp == 1) {
@@ -153,9 +162,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         mbar_wait(&k_full[s], (j >> 1) & 1);
         mbar_wait(&s_empty[s], ((j >> 1) & 1) ^ 1);
         tc_fence_after();
+        const uint8_t* q = sQ + (MAPS == 2 && j >= nt ? QKT : 0);
 #pragma unroll
         for (int kk = 0; kk < DK / 16; ++kk) {
-          const uint64_t da = umma_desc_sw128_kmajor(sQ + (kk >> 2) * 16384) + 2 * (kk & 3);
+          const uint64_t da = umma_desc_sw128_kmajor(q + (kk >> 2) * 16384) + 2 * (kk & 3);
           const uint64_t db = umma_desc_sw128_kmajor(sK + s * QKT + (kk >> 2) * 16384) + 2 * (kk & 3);
           umma_bf16_ss(tS0 + s * 128, da, db, idS, kk != 0);
         }
@@ -163,9 +173,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       };
       mbar_wait(q_full, 0);
       issue_s(0);
-      for (int j = 0; j < nt; ++j) {
+      for (int j = 0; j < MAPS * nt; ++j) {
         const int s = j & 1;
-        if (j + 1 < nt) issue_s(j + 1);
+        if (j + 1 < MAPS * nt) issue_s(j + 1);
         mbar_wait(p_full, j & 1);
         const int sv = j % VST;
         mbar_wait(&v_full[sv], (j / VST) & 1);
@@ -199,13 +209,23 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     const bool rec = p.dbg != nullptr && blockIdx.x == gridDim.x / 2 && blockIdx.y == 0 && threadIdx.x == 64;
     long long* dbg = p.dbg;
     if (rec) dbg[0] = clock64();
-    for (int j = 0; j < nt; ++j) {
+    auto store = [&](__nv_bfloat16* dst, float f) {
+#pragma unroll
+      for (int c = 0; c < OW; c += 8) {
+        int4 ov;
+        ov.x = pack_bf16(O[c] * f, O[c + 1] * f); ov.y = pack_bf16(O[c + 2] * f, O[c + 3] * f);
+        ov.z = pack_bf16(O[c + 4] * f, O[c + 5] * f); ov.w = pack_bf16(O[c + 6] * f, O[c + 7] * f);
+        st_v4(dst + c, ov);
+      }
+    };
+    for (int map = 0; map < MAPS; ++map) {
+    for (int j = map * nt; j < (map + 1) * nt; ++j) {
       const int s = j & 1;
       mbar_wait(&s_full[s], (j >> 1) & 1);
       tc_fence_after();
       if (rec && j < 30) dbg[1 + 5 * j] = clock64();
       const uint32_t tS = tS0 + s * 128 + lane_base + g * 64;
-      const int base = tile_of(j) * kAfBN, col0 = base + g * 64;
+      const int base = tile_of(j - map * nt) * kAfBN, col0 = base + g * 64;
       const bool need_mask = (base + kAfBN - 1 > kmax) || (base + kAfBN > lk) || base <= klo;
       auto seen = [&](int col) { return col <= kmax && col < lk && (col > klo || col < p.keep_first); };
       // pass 1: max over this thread's 64 scores, then exchange with the other warpgroup's half of the row
@@ -293,22 +313,63 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (rec && j < 30) dbg[5 + 5 * j] = clock64();
     }
     // total row sum = the two groups' partial sums (same running max on both sides)
-    s_mx[0][g][r] = l_run;
+    s_sum[map][g][r] = l_run;
     asm volatile("bar.sync 1, 256;" ::: "memory");
-    float l_tot = l_run + s_mx[0][g ^ 1][r];
+    float l_tot = l_run + s_sum[map][g ^ 1][r];
     if (p.sink != nullptr && m_run != -INFINITY) l_tot += fast_exp2(p.sink[h] * 1.4426950408889634f - m_run * p.scale_log2);
-    if (qrow < lq) {
-      const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
-      __nv_bfloat16* dst = p.o + static_cast<int64_t>(qs + qrow) * p.ldo + h * kAfD + g * OW;
-#pragma unroll
-      for (int c = 0; c < OW; c += 8) {
-        int4 ov;
-        ov.x = pack_bf16(O[c] * inv, O[c + 1] * inv); ov.y = pack_bf16(O[c + 2] * inv, O[c + 3] * inv);
-        ov.z = pack_bf16(O[c + 4] * inv, O[c + 5] * inv); ov.w = pack_bf16(O[c + 6] * inv, O[c + 7] * inv);
-        st_v4(dst + c, ov);
+    const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
+    if constexpr (MAPS == 1) {
+      if (qrow < lq) {
+        store(p.o + static_cast<int64_t>(qs + qrow) * p.ldo + h * kAfD + g * OW, inv);
+        if (p.lse && g == 0)
+          p.lse[static_cast<int64_t>(h) * p.Tq + qs + qrow] = (m_run == -INFINITY) ? -INFINITY : m_run * p.sm_scale + __logf(l_tot);
       }
-      if (p.lse && g == 0)
-        p.lse[static_cast<int64_t>(h) * p.Tq + qs + qrow] = (m_run == -INFINITY) ? -INFINITY : m_run * p.sm_scale + __logf(l_tot);
+    } else {
+      const uint32_t t_first = tO + 128 + lane_base + g * OW;          // the first map's output
+      if (map == 0) {
+#pragma unroll
+        for (int c = 0; c < OW; c += 16) {
+          uint32_t v[16];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) { v[i] = __float_as_uint(O[c + i] * inv); O[c + i] = 0.f; }
+          __syncwarp();
+          tmem_st_32x16(t_first + c, v);
+        }
+        tmem_st_wait();
+        m_run = -INFINITY;
+        l_run = 0.f;
+      } else {
+        const float lam = p.lam[0];
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < OW; c += 32) {
+          uint32_t v[32];
+          __syncwarp();
+          tmem_ld_32x32(t_first + c, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            O[c + i] = __uint_as_float(v[i]) - lam * (O[c + i] * inv);
+            ss += O[c + i] * O[c + i];
+          }
+        }
+        s_sum[0][g][r] = ss;                     // (the first map's sums were read before this map's last barrier)
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        ss += s_sum[0][g ^ 1][r];
+        const float f = rsqrtf(ss / p.dv_out + p.eps) * p.keep;
+        if (qrow < lq) {
+          const int n = p.dv_out - g * OW;       // values of this half
+          __nv_bfloat16* dst = p.o + static_cast<int64_t>(qs + qrow) * p.ldo + h * p.dv_out + g * OW;
+          if (n >= OW && p.dv_out % 8 == 0 && p.ldo % 8 == 0) {
+            store(dst, f);
+          } else {
+#pragma unroll
+            for (int c = 0; c < OW; ++c)
+              if (c < n) dst[c] = __float2bfloat16(O[c] * f);
+          }
+        }
+      }
+    }
     }
   }
   tc_fence_before();
@@ -348,19 +409,20 @@ int af_tmap(CUtensorMap* m, const void* ptr, uint64_t rows, uint64_t cols, uint6
 
 using namespace prl;
 
-template <int DK>
+template <int DK, int DV, int MAPS>
 static int run_attn_fwd(const void* q, const void* k, const void* v, const AttnFwdParams& p, int Tk, int64_t ldq, int64_t ldk, int64_t ldv,
                         int max_tiles, cudaStream_t stream) {
+  using Cfg = AfCfg<DK, DV, MAPS>;
   CUtensorMap tmQ, tmK, tmV;
-  if (af_tmap(&tmQ, q, p.Tq, static_cast<uint64_t>(p.nq) * DK, ldq * 2, kAfBM)) return -111;
-  if (af_tmap(&tmK, k, Tk, static_cast<uint64_t>(p.nkv) * DK, ldk * 2, kAfBN)) return -112;
-  if (af_tmap(&tmV, v, Tk, static_cast<uint64_t>(p.nkv) * AfCfg<DK>::DV, ldv * 2, kAfBN)) return -113;
+  if (af_tmap(&tmQ, q, p.Tq, static_cast<uint64_t>(p.nq) * MAPS * DK, ldq * 2, kAfBM)) return -111;
+  if (af_tmap(&tmK, k, Tk, static_cast<uint64_t>(p.nkv) * (MAPS == 2 && !p.shared_row ? 2 : 1) * DK, ldk * 2, kAfBN)) return -112;
+  if (af_tmap(&tmV, v, Tk, static_cast<uint64_t>(p.nkv) * DV, ldv * 2, kAfBN)) return -113;
   static bool attr = false;
   if (!attr) {
-    PRL_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, AfCfg<DK>::SMEM));
+    PRL_CUDA_CHECK(cudaFuncSetAttribute(attn_fwd_kernel<DK, DV, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM));
     attr = true;
   }
-  attn_fwd_kernel<DK><<<dim3(max_tiles, p.nq), kAfThreads, AfCfg<DK>::SMEM, stream>>>(tmQ, tmK, tmV, p);
+  attn_fwd_kernel<DK, DV, MAPS><<<dim3(max_tiles, p.nq), kAfThreads, Cfg::SMEM, stream>>>(tmQ, tmK, tmV, p);
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
@@ -374,7 +436,7 @@ extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o
                             cudaStream_t stream) {
   if (Tq <= 0 || B <= 0) return 0;
   if (nq % nkv != 0) return -110;
-  AttnFwdParams p;
+  AttnFwdParams p{};
   p.o = static_cast<__nv_bfloat16*>(o);
   p.lse = lse;
   p.cu_q = cu_q; p.cu_k = cu_k;
@@ -387,8 +449,32 @@ extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o
   p.keep_first = window > 0 ? keep_first : 0;
   p.sink = sink;
   p.dbg = dbg;
-  if (dk == 64) return run_attn_fwd<64>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
-  if (dk == 128) return run_attn_fwd<128>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
-  if (dk == 192) return run_attn_fwd<192>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 64) return run_attn_fwd<64, 64, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 128) return run_attn_fwd<128, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 192) return run_attn_fwd<192, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  return -114;
+}
+
+// differential attention, causal: q:[Tq, nq*2*dk], k:[Tk, nkv*2*dk] — or [Tk, nkv*64] when shared_row (dk = 64: both maps' keys of width 32 in one row) —
+// v:[Tk, nkv*dv], o:[Tq, nq*dv_out], all contiguous; dk, dv = 64 or 128
+extern "C" int prl_map_attn_fwd(const void* q, const void* k, const void* v, void* o, const int32_t* cu_q, const int32_t* cu_k, int B, int Tq, int Tk, int nq,
+                                int nkv, int dk, int dv, int dv_out, int shared_row, float sm_scale, int window, const float* lam, float keep, float eps,
+                                int max_tiles, cudaStream_t stream) {
+  if (Tq <= 0 || B <= 0) return 0;
+  if (nq % nkv != 0 || dv_out < 1 || dv_out > dv || window < 1 || (shared_row && dk != 64)) return -110;
+  AttnFwdParams p{};
+  p.o = static_cast<__nv_bfloat16*>(o);
+  p.cu_q = cu_q; p.cu_k = cu_k;
+  p.ldo = static_cast<int64_t>(nq) * dv_out; p.B = B; p.nq = nq; p.nkv = nkv; p.Tq = Tq;
+  p.sm_scale = sm_scale;
+  p.scale_log2 = sm_scale * 1.4426950408889634f;
+  p.causal = 1;
+  p.window = window;
+  p.lam = lam; p.keep = keep; p.eps = eps; p.dv_out = dv_out; p.shared_row = shared_row;
+  const int64_t ldq = static_cast<int64_t>(nq) * 2 * dk, ldk = static_cast<int64_t>(nkv) * (shared_row ? 1 : 2) * dk, ldv = static_cast<int64_t>(nkv) * dv;
+  if (dk == 64 && dv == 64) return run_attn_fwd<64, 64, 2>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 64 && dv == 128) return run_attn_fwd<64, 128, 2>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 128 && dv == 64) return run_attn_fwd<128, 64, 2>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 128 && dv == 128) return run_attn_fwd<128, 128, 2>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
   return -114;
 }

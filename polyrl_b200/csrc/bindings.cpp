@@ -11,7 +11,6 @@ extern "C" {
 int prl_gemm2_bf16(const void*, const void*, void*, const void*, int, int, int, int64_t, int64_t, int64_t, int, int, int, cudaStream_t);
 int prl_gemm2_bf16_accum_f32(const void*, const void*, float*, float, int, int, int, int64_t, int64_t, int64_t, int, int, cudaStream_t);
 int prl_gemm_fp8(const void*, const void*, void*, const float*, const float*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
-int prl_gemm_swiglu_bf16(const void*, const void*, void*, void*, int, int, int, int64_t, int64_t, int64_t, int64_t, cudaStream_t);
 int prl_linear_ce_num_splits(int, int);
 int prl_linear_ce_fwd(const void*, const void*, const int64_t*, float, int, int, int, int64_t, int64_t, float*, int, float*, float*, float*, float*, cudaStream_t);
 int prl_linear_ce_dz(const void*, const void*, const int64_t*, const float*, const float*, const float*, const float*, float, int, int, int, int, int64_t, int64_t, void*, int64_t, cudaStream_t);
@@ -130,20 +129,6 @@ at::Tensor gemm_fp8(const at::Tensor& a, const at::Tensor& b, const at::Tensor& 
                      col_scale.data_ptr<float>(), M, N, K, a.stride(0), b.stride(0), d.stride(0),
                      static_cast<int>(force_bn), cur_stream()), "gemm_fp8");
   return d;
-}
-
-std::vector<at::Tensor> gemm_swiglu(const at::Tensor& a, const at::Tensor& wgu, bool save_gu) {
-  CHECK_BF16(a); CHECK_BF16(wgu); CHECK_LASTDIM(a); CHECK_LASTDIM(wgu);
-  const int M = a.size(0), K = a.size(1), N2 = wgu.size(0);
-  TORCH_CHECK(wgu.size(1) == K && N2 % 256 == 0 && K % 8 == 0);
-  c10::cuda::CUDAGuard g(a.device());
-  at::Tensor h = at::empty({M, N2 / 2}, a.options());
-  at::Tensor gu = save_gu ? at::empty({M, N2}, a.options()) : at::Tensor();
-  check(prl_gemm_swiglu_bf16(a.data_ptr(), wgu.data_ptr(), h.data_ptr(), save_gu ? gu.data_ptr() : nullptr, M, N2, K,
-                             a.stride(0), wgu.stride(0), h.stride(0), save_gu ? gu.stride(0) : 0, cur_stream()),
-        "gemm_swiglu");
-  if (save_gu) return {h, gu};
-  return {h};
 }
 
 std::vector<at::Tensor> linear_ce_fwd(const at::Tensor& hidden, const at::Tensor& w, const at::Tensor& labels,
@@ -559,7 +544,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm2_accum_f32_", &gemm2_accum_f32_);
   m.def("gemm_fp8", &gemm_fp8, py::arg("a"), py::arg("b"), py::arg("row_scale"), py::arg("col_scale"),
         py::arg("force_bn") = 0);
-  m.def("gemm_swiglu", &gemm_swiglu);
   m.def("skinny_gemm", &skinny_gemm);
   m.def("skinny_gemm_tp", &skinny_gemm_tp);
   m.def("stream_gemm", &stream_gemm, py::arg("x"), py::arg("w"), py::arg("residual") = py::none(), py::arg("bias") = py::none(),

@@ -13,17 +13,30 @@ int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int
 int prl_paged_decode_workspace_floats(int, int, int, int);
 int prl_paged_decode(const void*, int64_t, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, float, int, int, int, float*, void*, int64_t, cudaStream_t);
 int prl_gemm_clamped_glu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, float, float, cudaStream_t);
+int prl_gemm_swiglu_bf16(const void*, const void*, void*, void*, int, int, int, int64_t, int64_t, int64_t, int64_t, cudaStream_t);
+int prl_gemm_experts_bf16(const void*, const void*, void*, const int32_t*, int, int, int, int, int, cudaStream_t);
+int prl_map_attn_fwd(const void*, const void*, const void*, void*, const int32_t*, const int32_t*, int, int, int, int, int, int, int, int, int, float, int, const float*, float, float, int, cudaStream_t);
+int prl_map_decode_ok(int, int, int);
+int prl_map_decode(const void*, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, int, int, float, int, int, const float*, float, float, float*, void*, cudaStream_t);
 int prl_gemm_gelu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, cudaStream_t);
 int prl_mix_embed(const int64_t*, const void*, const float*, float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_norm_add(const void*, int64_t, float*, const float*, const float*, void*, int, int, float, int, cudaStream_t);
-int prl_mix_rms(const float*, const float*, void*, int, int, float, int, cudaStream_t);
+int prl_mix_rms(const float*, const float*, void*, int, int, float, int, int, cudaStream_t);
 int prl_mix_gated_norm(const void*, int64_t, const void*, int64_t, const float*, void*, int64_t, int, int, int, float, int, int, cudaStream_t);
 int prl_mix_conv(const void*, int64_t, const float*, const float*, void*, const int32_t*, const int32_t*, const int64_t*, const int32_t*, void*, int64_t, int, int, int, int, int, cudaStream_t);
 int prl_mix_latent_prep(const void*, int64_t, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, int, float, int, cudaStream_t);
 int prl_mix_rope(void*, int64_t, int, int, int, int, const double*, const int64_t*, int, int, cudaStream_t);
 int prl_mix_gelu(void*, int64_t, int, cudaStream_t);
 int prl_mix_qk_prep(const void*, int64_t, int, int, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, void*, void*, int, float, int, cudaStream_t);
-int prl_mix_gather_keys(const void*, const void*, const int64_t*, void*, void*, int64_t, int, int, cudaStream_t);
+int prl_mix_gather_keys(const void*, const void*, const int64_t*, void*, void*, int64_t, int, int, int, cudaStream_t);
+int prl_mix_map_rows(const void*, int64_t, const float*, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, void*, void*, int, int, int, int, int, int, int, int, int, float, int, cudaStream_t);
+int prl_mix_input_conv(const void*, int64_t, const float*, const float*, void*, const int32_t*, const int32_t*, const int64_t*, const int32_t*, void*, void*, int, int, int, int, int, cudaStream_t);
+int prl_mix_poly_norm(const void*, int64_t, const float*, void*, int, int, float, int, cudaStream_t);
+int prl_mix_silu_glu(const void*, void*, int64_t, int, int, int, cudaStream_t);
+int prl_mix_route_tiles(int64_t, int64_t);
+int prl_mix_route(const float*, int64_t, int, int, int, int32_t*, float*, int32_t*, int32_t*, int32_t*, cudaStream_t);
+int prl_mix_expert_rows(const void*, int64_t, const int32_t*, const float*, const int32_t*, const int32_t*, void*, int32_t*, int, int, int, int, cudaStream_t);
+int prl_mix_expert_gemm(const void*, const void*, const int32_t*, void*, int, int, int, int, int, cudaStream_t);
 int prl_mix_clamped_glu(const void*, void*, int64_t, int, int, float, float, int, cudaStream_t);
 int prl_mix_delta_ok(const void*, int64_t, const void*, int64_t, const void*, int64_t, int, int);
 int64_t prl_mix_delta_chunks(int64_t, int64_t);
@@ -40,6 +53,8 @@ int prl_mix_chunk_tc_ok(const prl::ScanParams*);
 int prl_mix_chunk_tc(const prl::ScanParams*, int, int32_t*, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
 int prl_mix_window(const prl::WindowParams*, int, cudaStream_t);
+int prl_mix_block(const prl::BlockParams*, int, cudaStream_t);
+int prl_mix_map_attention(const prl::MapParams*, int, cudaStream_t);
 int prl_mix_delta(const prl::ScanParams*, int64_t, int64_t, void*, float*, int32_t*, cudaStream_t);
 }
 
@@ -204,12 +219,12 @@ at::Tensor mix_norm_add_(const at::Tensor& y, at::Tensor x, const at::Tensor& w,
   return h;
 }
 
-at::Tensor mix_rms(const at::Tensor& x, const at::Tensor& w, double eps, bool bf16) {
+at::Tensor mix_rms(const at::Tensor& x, const at::Tensor& w, double eps, bool bf16, bool center) {
   CHECK_F32(x);
   TORCH_CHECK(x.is_contiguous() && x.dim() == 2);
   c10::cuda::CUDAGuard g(x.device());
   at::Tensor h = at::empty(x.sizes(), x.options().dtype(bf16 ? at::kBFloat16 : at::kFloat));
-  check(prl_mix_rms(x.data_ptr<float>(), vecf(w, x.size(1), "mix_rms w"), h.data_ptr(), x.size(0), x.size(1), static_cast<float>(eps), bf16 ? 0 : 1,
+  check(prl_mix_rms(x.data_ptr<float>(), vecf(w, x.size(1), "mix_rms w"), h.data_ptr(), x.size(0), x.size(1), static_cast<float>(eps), center, bf16 ? 0 : 1,
                     cur_stream()), "mix_rms");
   return h;
 }
@@ -403,13 +418,14 @@ std::vector<at::Tensor> mix_qk_prep(const at::Tensor& p, int64_t heads, int64_t 
 }
 
 std::vector<at::Tensor> mix_gather_keys(const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& rows) {
-  TORCH_CHECK(k_pool.is_cuda() && k_pool.dim() == 4 && k_pool.size(2) == 16 && k_pool.is_contiguous() && v_pool.is_contiguous() && v_pool.is_cuda() &&
-              v_pool.sizes() == k_pool.sizes() && v_pool.scalar_type() == k_pool.scalar_type());
-  const int64_t n = rows.numel(), G = k_pool.size(1), width = k_pool.size(3);
+  for (const at::Tensor& t : {k_pool, v_pool})
+    TORCH_CHECK(t.is_cuda() && t.dim() == 4 && t.size(2) == 16 && t.is_contiguous() && t.size(0) == k_pool.size(0) && t.size(1) == k_pool.size(1) &&
+                t.scalar_type() == k_pool.scalar_type(), "mix_gather_keys: pools");
+  const int64_t n = rows.numel(), G = k_pool.size(1), es = k_pool.element_size();
   c10::cuda::CUDAGuard g(k_pool.device());
-  at::Tensor k = at::empty({n, G, width}, k_pool.options()), v = at::empty_like(k);
-  check(prl_mix_gather_keys(k_pool.data_ptr(), v_pool.data_ptr(), veci<int64_t>(rows, n, "rows"), k.data_ptr(), v.data_ptr(), n, G,
-                            width * k_pool.element_size(), cur_stream()), "mix_gather_keys");
+  at::Tensor k = at::empty({n, G, k_pool.size(3)}, k_pool.options()), v = at::empty({n, G, v_pool.size(3)}, v_pool.options());
+  check(prl_mix_gather_keys(k_pool.data_ptr(), v_pool.data_ptr(), veci<int64_t>(rows, n, "rows"), k.data_ptr(), v.data_ptr(), n, G, k_pool.size(3) * es,
+                            v_pool.size(3) * es, cur_stream()), "mix_gather_keys");
   return {k, v};
 }
 
@@ -473,6 +489,275 @@ void mix_gelu_(at::Tensor x) {
   TORCH_CHECK(x.is_contiguous());
   c10::cuda::CUDAGuard g(x.device());
   check(prl_mix_gelu(x.data_ptr(), x.numel(), dt, cur_stream()), "mix_gelu");
+}
+
+std::vector<at::Tensor> gemm_swiglu(const at::Tensor& a, const at::Tensor& wgu, bool save_gu) {
+  CHECK_BF16(a); CHECK_BF16(wgu); CHECK_LASTDIM(a); CHECK_LASTDIM(wgu);
+  const int M = a.size(0), K = a.size(1), N2 = wgu.size(0);
+  TORCH_CHECK(wgu.size(1) == K && N2 % 256 == 0 && K % 8 == 0);
+  c10::cuda::CUDAGuard g(a.device());
+  at::Tensor h = at::empty({M, N2 / 2}, a.options());
+  at::Tensor gu = save_gu ? at::empty({M, N2}, a.options()) : at::Tensor();
+  check(prl_gemm_swiglu_bf16(a.data_ptr(), wgu.data_ptr(), h.data_ptr(), save_gu ? gu.data_ptr() : nullptr, M, N2, K,
+                             a.stride(0), wgu.stride(0), h.stride(0), save_gu ? gu.stride(0) : 0, cur_stream()),
+        "gemm_swiglu");
+  if (save_gu) return {h, gu};
+  return {h};
+}
+
+at::Tensor mix_silu_glu(const at::Tensor& gu, int64_t blk) {
+  const int dt = dt_of(gu, "mix_silu_glu");
+  TORCH_CHECK(gu.dim() == 2 && gu.is_contiguous() && blk > 0 && gu.size(1) % (2 * blk) == 0);
+  c10::cuda::CUDAGuard g(gu.device());
+  at::Tensor out = at::empty({gu.size(0), gu.size(1) / 2}, gu.options());
+  check(prl_mix_silu_glu(gu.data_ptr(), out.data_ptr(), gu.size(0), gu.size(1) / 2, blk, dt, cur_stream()), "mix_silu_glu");
+  return out;
+}
+
+at::Tensor mix_poly_norm(const at::Tensor& z, const at::Tensor& act, double eps) {
+  const int dt = dt_of(z, "mix_poly_norm");
+  rows2(z, "mix_poly_norm z");
+  c10::cuda::CUDAGuard g(z.device());
+  at::Tensor out = at::empty(z.sizes(), z.options());
+  check(prl_mix_poly_norm(z.data_ptr(), z.stride(0), vecf(act, 4, "act"), out.data_ptr(), z.size(0), z.size(1), static_cast<float>(eps), dt, cur_stream()),
+        "mix_poly_norm");
+  return out;
+}
+
+// ---------------------------------------------------------------------------------------------- parallel blocks
+// convolution of single-token rows at the end of a block kernel (all absent: none)
+void block_conv(prl::BlockParams& p, const at::Tensor& like, const c10::optional<at::Tensor>& c1, const c10::optional<at::Tensor>& c2,
+                const c10::optional<at::Tensor>& state, const c10::optional<at::Tensor>& start, const c10::optional<at::Tensor>& slot) {
+  if (!c1.has_value()) return;
+  TORCH_CHECK(state.has_value() && start.has_value() && slot.has_value() && c1->dim() == 2);
+  p.taps = c1->size(0);
+  p.c1 = vecf(c1, static_cast<int64_t>(p.taps) * p.W, "conv 1");
+  p.c2 = vecf(c2, static_cast<int64_t>(p.taps) * p.W, "conv 2");
+  TORCH_CHECK(state->is_cuda() && state->scalar_type() == like.scalar_type() && state->is_contiguous() && state->dim() == 3 && state->size(1) == p.taps - 1 &&
+              state->size(2) == p.W, "block: convolution state");
+  p.state = state->data_ptr();
+  p.start = veci<int32_t>(*start, p.R, "start"); p.slot = veci<int64_t>(*slot, p.R, "slot");
+}
+std::vector<at::Tensor> block_run(prl::BlockParams& p, const at::Tensor& first, const at::Tensor& like, int dt, const c10::optional<at::Tensor>& w_next) {
+  at::Tensor h, h2;
+  if (w_next.has_value()) {
+    p.w_next = vecf(w_next, p.W, "w_next");
+    h = at::empty({p.R, p.W}, like.options());
+    p.h = h.data_ptr();
+    if (p.c2) { h2 = at::empty({p.R, p.W}, like.options()); p.h2 = h2.data_ptr(); }
+  } else {
+    TORCH_CHECK(!p.c1, "block: a convolution without its norm");
+  }
+  check(prl_mix_block(&p, dt, cur_stream()), "mix_block");
+  return {first, h, h2};
+}
+// -> (results [slots, T, W] with the embedding in the first, h, h2)
+std::vector<at::Tensor> mix_block_embed(const at::Tensor& ids, const at::Tensor& emb, int64_t slots, const at::Tensor& w_norm, double eps, bool center,
+                                        const c10::optional<at::Tensor>& c1, const c10::optional<at::Tensor>& c2, const c10::optional<at::Tensor>& state,
+                                        const c10::optional<at::Tensor>& start, const c10::optional<at::Tensor>& slot) {
+  const int dt = dt_of(emb, "mix_block_embed");
+  TORCH_CHECK(emb.is_contiguous() && emb.dim() == 2 && slots >= 1);
+  c10::cuda::CUDAGuard g(emb.device());
+  prl::BlockParams p{};
+  p.R = ids.numel(); p.W = emb.size(1);
+  p.ids = veci<int64_t>(ids, p.R, "ids");
+  p.emb = emb.data_ptr();
+  at::Tensor past = at::empty({slots, p.R, p.W}, emb.options().dtype(at::kFloat));
+  p.past = past.data_ptr<float>(); p.stride = past.stride(0);
+  p.eps = static_cast<float>(eps); p.center = center;
+  block_conv(p, emb, c1, c2, state, start, slot);
+  return block_run(p, past, emb, dt, w_norm);
+}
+// layer i of a stack of parallel blocks -> (x' if wanted, h, h2)
+std::vector<at::Tensor> mix_block_add(at::Tensor past, int64_t i, const at::Tensor& y1, const c10::optional<at::Tensor>& y2, const c10::optional<at::Tensor>& rows,
+                                      const c10::optional<at::Tensor>& pos, const c10::optional<at::Tensor>& s1, const c10::optional<at::Tensor>& s2,
+                                      const c10::optional<at::Tensor>& a_prev, const c10::optional<at::Tensor>& a_cur, const c10::optional<at::Tensor>& w_next,
+                                      double eps, bool center, bool want_x, const c10::optional<at::Tensor>& c1, const c10::optional<at::Tensor>& c2,
+                                      const c10::optional<at::Tensor>& state, const c10::optional<at::Tensor>& start, const c10::optional<at::Tensor>& slot) {
+  const int dt = dt_of(y1, "mix_block_add");
+  rows2(y1, "mix_block_add y1");
+  CHECK_F32(past);
+  prl::BlockParams p{};
+  p.R = y1.size(0); p.W = y1.size(1); p.n = i;
+  TORCH_CHECK(past.dim() == 3 && past.is_contiguous() && past.size(1) == p.R && past.size(2) == p.W && i >= 0);
+  TORCH_CHECK(a_cur.has_value() ? past.size(0) >= i + 2 : !a_prev.has_value(), "mix_block_add: one slot per result");
+  c10::cuda::CUDAGuard g(y1.device());
+  p.past = past.data_ptr<float>(); p.stride = past.stride(0);
+  p.y1 = y1.data_ptr(); p.ld1 = y1.stride(0);
+  if (y2.has_value()) {
+    rows2(*y2, "mix_block_add y2");
+    TORCH_CHECK(y2->scalar_type() == y1.scalar_type() && y2->sizes() == y1.sizes());
+    p.y2 = y2->data_ptr(); p.ld2 = y2->stride(0);
+  }
+  if (rows.has_value()) {
+    TORCH_CHECK(pos.has_value() && rows->scalar_type() == y1.scalar_type() && rows->is_contiguous() && rows->dim() == 2 && rows->size(1) == p.W &&
+                pos->dim() == 2 && pos->size(0) == p.R);
+    p.rows = rows->data_ptr(); p.top = pos->size(1);
+    p.pos = veci<int32_t>(*pos, static_cast<int64_t>(p.R) * p.top, "pos");
+  }
+  p.s1 = vecf(s1, p.W, "s1"); p.s2 = vecf(s2, p.W, "s2");
+  p.a_prev = vecf(a_prev, i + 1, "a_prev"); p.a_cur = vecf(a_cur, i + 2, "a_cur");
+  p.eps = static_cast<float>(eps); p.center = center;
+  at::Tensor x;
+  if (want_x) { x = at::empty({p.R, p.W}, past.options()); p.x_out = x.data_ptr<float>(); }
+  block_conv(p, y1, c1, c2, state, start, slot);
+  return block_run(p, x, y1, dt, w_next);
+}
+
+std::vector<at::Tensor> mix_input_conv(const at::Tensor& h, const at::Tensor& w1, const c10::optional<at::Tensor>& w2, at::Tensor state, const at::Tensor& cu,
+                                       const at::Tensor& start, const at::Tensor& slot, const c10::optional<at::Tensor>& seq_of) {
+  const int dt = dt_of(h, "mix_input_conv");
+  rows2(h, "mix_input_conv h");
+  const int64_t T = h.size(0), ch = h.size(1), taps = w1.size(0), spans = start.numel();
+  TORCH_CHECK(w1.dim() == 2 && w1.size(1) == ch && state.scalar_type() == h.scalar_type() && state.is_cuda() && state.is_contiguous() && state.dim() == 3 &&
+              state.size(1) == taps - 1 && state.size(2) == ch, "mix_input_conv: shapes");
+  TORCH_CHECK(seq_of.has_value() || spans == T, "mix_input_conv: one token per span without seq_of");
+  c10::cuda::CUDAGuard g(h.device());
+  at::Tensor o1 = at::empty({T, ch}, h.options()), o2;
+  if (w2.has_value()) o2 = at::empty({T, ch}, h.options());
+  check(prl_mix_input_conv(h.data_ptr(), h.stride(0), vecf(w1, taps * ch, "w1"), vecf(w2, taps * ch, "w2"), state.data_ptr(), veci<int32_t>(cu, spans + 1, "cu"),
+                           veci<int32_t>(start, spans, "start"), veci<int64_t>(slot, spans, "slot"),
+                           seq_of.has_value() ? veci<int32_t>(*seq_of, T, "seq_of") : nullptr, o1.data_ptr(), w2.has_value() ? o2.data_ptr() : nullptr, ch, taps,
+                           T, spans, dt, cur_stream()), "mix_input_conv");
+  return {o1, o2};
+}
+
+// ---------------------------------------------------------------------------------------------- experts
+// logits [T, E] -> (experts [T, top], scores, ranks, plan); counter: >= E + 1 zeros, left zero
+std::vector<at::Tensor> mix_route(const at::Tensor& logits, int64_t top, at::Tensor counter) {
+  CHECK_F32(logits);
+  rows2(logits, "mix_route logits");
+  const int64_t T = logits.size(0), E = logits.size(1);
+  TORCH_CHECK(top >= 1 && top <= E && T * top < 0x7fffffff);
+  veci<int32_t>(counter, E + 1, "counter");
+  c10::cuda::CUDAGuard g(logits.device());
+  const auto i32 = logits.options().dtype(at::kInt);
+  at::Tensor pick = at::empty({T, top}, i32), score = at::empty({T, top}, logits.options()), rank = at::empty({T, top}, i32);
+  at::Tensor plan = at::empty({1 + E + prl_mix_route_tiles(T * top, E)}, i32);
+  check(prl_mix_route(logits.data_ptr<float>(), logits.stride(0), T, E, top, pick.data_ptr<int32_t>(), score.data_ptr<float>(), rank.data_ptr<int32_t>(),
+                      counter.data_ptr<int32_t>(), plan.data_ptr<int32_t>(), cur_stream()), "mix_route");
+  return {pick, score, rank, plan};
+}
+// -> (rows in the experts' order [tiles * 128, W], place of every (token, choice))
+std::vector<at::Tensor> mix_expert_rows(const at::Tensor& h, const at::Tensor& pick, const at::Tensor& score, const at::Tensor& rank, const at::Tensor& plan,
+                                        int64_t experts) {
+  const int dt = dt_of(h, "mix_expert_rows");
+  rows2(h, "mix_expert_rows h");
+  const int64_t T = h.size(0), W = h.size(1), top = pick.size(1), tiles = prl_mix_route_tiles(T * top, experts);
+  c10::cuda::CUDAGuard g(h.device());
+  at::Tensor rows = at::empty({tiles * 128, W}, h.options()), pos = at::empty({T, top}, pick.options());
+  check(prl_mix_expert_rows(h.data_ptr(), h.stride(0), veci<int32_t>(pick, T * top, "pick"), vecf(score, T * top, "score"), veci<int32_t>(rank, T * top, "rank"),
+                            veci<int32_t>(plan, 1 + experts + tiles, "plan"), rows.data_ptr(), pos.data_ptr<int32_t>(), T, top, W, dt, cur_stream()),
+        "mix_expert_rows");
+  return {rows, pos};
+}
+// rows [tiles * 128, K] x w [experts * N, K]
+at::Tensor mix_expert_gemm(const at::Tensor& x, const at::Tensor& w, const at::Tensor& plan, int64_t experts) {
+  const int dt = dt_of(x, "mix_expert_gemm");
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w.is_cuda() && w.dim() == 2 && w.is_contiguous() && w.scalar_type() == x.scalar_type() && w.size(1) == x.size(1) &&
+              x.size(0) % 128 == 0 && experts >= 1 && w.size(0) % experts == 0, "mix_expert_gemm: shapes");
+  const int64_t tiles = x.size(0) / 128, N = w.size(0) / experts;
+  c10::cuda::CUDAGuard g(x.device());
+  at::Tensor out = at::empty({x.size(0), N}, x.options());
+  check(prl_mix_expert_gemm(x.data_ptr(), w.data_ptr(), veci<int32_t>(plan, 1 + experts + tiles, "plan"), out.data_ptr(), tiles, experts, N, x.size(1), dt,
+                            cur_stream()), "mix_expert_gemm");
+  return out;
+}
+// the same on tcgen05 (bf16); glu: w holds gate and up rows in blocks of 128, the result is silu(gate) * up
+at::Tensor gemm_experts(const at::Tensor& x, const at::Tensor& w, const at::Tensor& plan, int64_t experts, bool glu) {
+  CHECK_BF16(x); CHECK_BF16(w);
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w.dim() == 2 && w.is_contiguous() && w.size(1) == x.size(1) && x.size(0) % 128 == 0 && experts >= 1 &&
+              w.size(0) % experts == 0 && x.size(1) % 8 == 0, "gemm_experts: shapes");
+  const int64_t tiles = x.size(0) / 128, N = w.size(0) / experts;
+  c10::cuda::CUDAGuard g(x.device());
+  at::Tensor out = at::empty({x.size(0), glu ? N / 2 : N}, x.options());
+  check(prl_gemm_experts_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), veci<int32_t>(plan, 1 + experts + tiles, "plan"), tiles, experts, N, x.size(1), glu,
+                              cur_stream()), "gemm_experts");
+  return out;
+}
+
+// ---------------------------------------------------------------------------------------------- differential attention
+// rows [queries H x 2 x D | keys G x 2 x D | values G x V] -> q [T, 2 H, qw], pools, and packed keys / values when asked for
+std::vector<at::Tensor> mix_map_prep(const at::Tensor& p, const at::Tensor& bias, int64_t heads, int64_t dim, int64_t vdim, const at::Tensor& wq,
+                                     const at::Tensor& wk, const at::Tensor& freq, const at::Tensor& pos, const at::Tensor& kvslot, at::Tensor k_pool,
+                                     at::Tensor v_pool, double eps, bool want_kv, int64_t qw) {
+  const int dt = dt_of(p, "mix_map_prep");
+  rows2(p, "mix_map_prep p");
+  for (const at::Tensor& t : {k_pool, v_pool})
+    TORCH_CHECK(t.is_cuda() && t.dim() == 4 && t.size(2) == 16 && t.is_contiguous() && t.scalar_type() == p.scalar_type() && t.size(0) == k_pool.size(0) &&
+                t.size(1) == k_pool.size(1), "mix_map_prep: pools");
+  const int64_t T = p.size(0), G = k_pool.size(1), kw = k_pool.size(3) / 2, vw = v_pool.size(3), rd = 2 * freq.numel(), cols = 2 * (heads + G) * dim + G * vdim;
+  TORCH_CHECK(p.size(1) >= cols && k_pool.size(3) == 2 * kw && G >= 1 && heads % G == 0);
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == at::kDouble && freq.is_contiguous());
+  c10::cuda::CUDAGuard g(p.device());
+  at::Tensor q = at::empty({T, 2 * heads, qw}, p.options()), k = at::empty({want_kv ? T : 0, G, 2 * kw}, p.options()),
+             v = at::empty({want_kv ? T : 0, G, vw}, p.options());
+  check(prl_mix_map_rows(p.data_ptr(), p.stride(0), vecf(bias, cols, "bias"), vecf(wq, dim, "wq"), vecf(wk, dim, "wk"), freq.data_ptr<double>(),
+                         veci<int64_t>(pos, T, "pos"), veci<int64_t>(kvslot, T, "kvslot"), q.data_ptr(), want_kv ? k.data_ptr() : nullptr,
+                         want_kv ? v.data_ptr() : nullptr, k_pool.data_ptr(), v_pool.data_ptr(), T, heads, G, dim, vdim, rd, qw, kw, vw, static_cast<float>(eps), dt,
+                         cur_stream()), "mix_map_prep");
+  return {q, k, v};
+}
+void map_pools(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table, int64_t window, const char* what) {
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && q.size(1) % 2 == 0, what, ": q [rows, 2 heads, width]");
+  for (const at::Tensor& t : {k_pool, v_pool})
+    TORCH_CHECK(t.is_cuda() && t.dim() == 4 && t.size(2) == 16 && t.is_contiguous() && t.scalar_type() == q.scalar_type() && t.size(0) == k_pool.size(0) &&
+                t.size(1) == k_pool.size(1), what, ": pools");
+  TORCH_CHECK(k_pool.size(3) % 2 == 0 && k_pool.size(1) >= 1 && (q.size(1) / 2) % k_pool.size(1) == 0, what, ": heads");
+  TORCH_CHECK(q.size(2) == k_pool.size(3) / 2 || q.size(2) == k_pool.size(3), what, ": query width");
+  TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.dim() == 2 && table.stride(1) == 1, what, ": table");
+  TORCH_CHECK(window >= 1 && window <= 0x7fffffff, what, ": window");
+}
+at::Tensor mix_map_attention(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table,
+                             const c10::optional<at::Tensor>& seq_of, const at::Tensor& kv_len, double scale, int64_t window, const at::Tensor& lam, double diff,
+                             double eps, int64_t vdim, int64_t dim) {
+  const int dt = dt_of(q, "mix_map_attention");
+  map_pools(q, k_pool, v_pool, table, window, "mix_map_attention");
+  prl::MapParams p{};
+  p.R = q.size(0); p.H = q.size(1) / 2; p.G = k_pool.size(1); p.qw = q.size(2); p.kw = k_pool.size(3) / 2; p.vw = v_pool.size(3); p.D = dim; p.V = vdim;
+  TORCH_CHECK(dim >= 1 && dim <= p.kw && vdim >= 1 && vdim <= p.vw && (seq_of.has_value() || table.size(0) >= p.R));
+  p.q = q.data_ptr(); p.k_pool = k_pool.data_ptr(); p.v_pool = v_pool.data_ptr();
+  p.table = table.data_ptr<int32_t>(); p.ld_table = table.stride(0);
+  p.seq_of = seq_of.has_value() ? veci<int32_t>(*seq_of, p.R, "seq_of") : nullptr;
+  p.kv_len = veci<int32_t>(kv_len, p.R, "kv_len");
+  p.lam = vecf(lam, 1, "lam");
+  p.window = window; p.scale = static_cast<float>(scale); p.keep = static_cast<float>(1.0 - diff); p.eps = static_cast<float>(eps);
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty({p.R, p.H * vdim}, q.options());
+  p.out = out.data_ptr();
+  check(prl_mix_map_attention(&p, dt, cur_stream()), "mix_map_attention");
+  return out;
+}
+at::Tensor map_decode(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table, const at::Tensor& kv_len, double scale,
+                      int64_t splits, int64_t window, const at::Tensor& lam, double diff, double eps, int64_t vdim) {
+  CHECK_BF16(q);
+  map_pools(q, k_pool, v_pool, table, window, "map_decode");
+  const int64_t R = q.size(0), H = q.size(1) / 2, G = k_pool.size(1), kw = k_pool.size(3) / 2, vw = v_pool.size(3);
+  TORCH_CHECK(prl_map_decode_ok(kw, vw, H / G) && q.size(2) == 64 && table.size(0) >= R && splits >= 1, "map_decode: sizes");
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty({R, H * vdim}, q.options());
+  at::Tensor work = at::empty({prl_paged_decode_workspace_floats(R, 2 * H, vw, splits)}, q.options().dtype(at::kFloat));
+  check(prl_map_decode(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), table.data_ptr<int32_t>(), table.stride(0), veci<int32_t>(kv_len, R, "kv_len"), R, H, G,
+                       kw, vw, vdim, static_cast<float>(scale), splits, window, vecf(lam, 1, "lam"), static_cast<float>(1.0 - diff), static_cast<float>(eps),
+                       work.data_ptr<float>(), out.data_ptr(), cur_stream()), "map_decode");
+  return out;
+}
+at::Tensor map_attn_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& cu_q, const at::Tensor& cu_k, double scale, int64_t window,
+                        const at::Tensor& lam, double diff, double eps, int64_t vdim) {
+  CHECK_BF16(q); CHECK_BF16(k); CHECK_BF16(v);
+  const int64_t dk = q.size(-1), G = k.size(1), dv = v.size(-1);
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous() && q.size(1) % 2 == 0 && G >= 1 &&
+              (q.size(1) / 2) % G == 0 && v.size(1) == G && v.size(0) == k.size(0) && (k.size(2) == 2 * dk || (k.size(2) == 64 && dk == 64)), "map_attn_fwd: shapes");
+  for (const at::Tensor& t : {q, k, v}) TORCH_CHECK((reinterpret_cast<uintptr_t>(t.data_ptr()) & 15) == 0, "map_attn_fwd: 16-byte aligned operands");
+  TORCH_CHECK(window >= 1 && window <= 0x7fffffff);
+  const int Tq = q.size(0), B = cu_q.numel() - 1;
+  veci<int32_t>(cu_q, B + 1, "cu_q"); veci<int32_t>(cu_k, B + 1, "cu_k");
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty({Tq, q.size(1) / 2 * vdim}, q.options());
+  check(prl_map_attn_fwd(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), cu_q.data_ptr<int32_t>(), cu_k.data_ptr<int32_t>(), B, Tq, k.size(0),
+                         q.size(1) / 2, G, dk, dv, vdim, k.size(2) == dk, static_cast<float>(scale), window, vecf(lam, 1, "lam"), static_cast<float>(1.0 - diff),
+                         static_cast<float>(eps), Tq / 128 + B, cur_stream()), "map_attn_fwd");
+  return out;
 }
 
 }  // namespace
@@ -549,6 +834,21 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mix_clamped_glu", &mix_clamped_glu);
   m.def("gemm_gelu", &gemm_gelu);
   m.def("mix_gelu_", &mix_gelu_);
+  m.def("gemm_swiglu", &gemm_swiglu);
+  m.def("mix_silu_glu", &mix_silu_glu);
+  m.def("mix_poly_norm", &mix_poly_norm);
+  m.def("mix_block_embed", &mix_block_embed);
+  m.def("mix_block_add", &mix_block_add);
+  m.def("mix_input_conv", &mix_input_conv);
+  m.def("mix_route", &mix_route);
+  m.def("mix_expert_rows", &mix_expert_rows);
+  m.def("mix_expert_gemm", &mix_expert_gemm);
+  m.def("gemm_experts", &gemm_experts);
+  m.def("mix_map_prep", &mix_map_prep);
+  m.def("mix_map_attention", &mix_map_attention);
+  m.def("map_attn_fwd", &map_attn_fwd);
+  m.def("map_decode", &map_decode);
+  m.def("map_decode_ok", [](int64_t kw, int64_t vw, int64_t rep) { return prl_map_decode_ok(static_cast<int>(kw), static_cast<int>(vw), static_cast<int>(rep)) != 0; });
   m.def("mix_chunk_supported", [](int64_t n) { return prl_mix_chunk_supported(static_cast<int>(n)) != 0; });
   m.def("mix_latent_tc_ok", [](int64_t r, int64_t rd) { return prl_mix_latent_tc_ok(static_cast<int>(r), static_cast<int>(rd)) != 0; });
 }

@@ -10,6 +10,8 @@
 //     the k-index of an MMA is a free permutation, so each lane's 16-byte load is wired to the
 //     k-slots it feeds; V fragments are built with two PRMTs per register pair)
 //   * fp32 online softmax in registers, split results merged by a second tiny kernel.
+// Differential attention (two maps per head over the same values): a cache row holds [map 1 | map 2] keys, the maps' queries are two
+// rows of the MMA that are zero in the other map's columns (QM = 2), and the merge kernel combines and norms the two outputs.
 #include <cstdlib>
 
 #include "common.cuh"
@@ -34,16 +36,18 @@ __device__ __forceinline__ uint32_t prmt(uint32_t a, uint32_t b, uint32_t sel) {
 // partial outputs: o_part [num_seqs, nq, splits, D] fp32, ml_part [num_seqs, nq, splits, 2] (max2, sum)
 // MINB = minimum resident CTAs per SM (register budget): 3 -> 168 regs, no spills; 4 -> 128 regs, ~76 B of spills but a third
 // more warps in flight to hide HBM latency.  Both are compiled; POLYRL_DECODE_MINB picks (default from the microbench).
-template <int D, int MINB>
+// DK / DV: width of a cached key / value row.  QM = 2: query row r has DK / 2 entries, for the columns of map r % 2.
+template <int DK, int DV, int QM, int MINB>
 __global__ void __launch_bounds__(kAttnWarps * 32, MINB)
-paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [num_seqs, nq*D] (row pitch ldq)
+paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [num_seqs, nq * DK / QM] (row pitch ldq)
                     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                     const int32_t* __restrict__ block_table, int64_t ld_bt, const int32_t* __restrict__ seq_lens,
                     int nq, int nkv, int splits, float scale_log2, int window, int keep_first, float* __restrict__ o_part,
                     float* __restrict__ ml_part, __nv_bfloat16* __restrict__ out_direct, int64_t ldo) {
-  static_assert(D % 64 == 0, "head dim must be a multiple of 64");
-  constexpr int KC = D / 32;     // 32-wide d chunks for QK (two MMAs each)
-  constexpr int DB = D / 64;     // 64-wide d blocks for PV (eight n-tiles each)
+  static_assert(DK % 64 == 0 && DV % 64 == 0, "row widths must be multiples of 64");
+  constexpr int KC = DK / 32;    // 32-wide d chunks for QK (two MMAs each)
+  constexpr int DB = DV / 64;    // 64-wide d blocks for PV (eight n-tiles each)
+  constexpr int QW = DK / QM;
   const int G = nq / nkv;        // query heads per kv head (<= 16)
   const int split = blockIdx.x % splits;
   const int kvh = (blockIdx.x / splits) % nkv;
@@ -64,13 +68,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
   // ---- Q fragments (A operand), rows = heads of the group, k-slots permuted to match 16 B K loads
   uint32_t qf[KC][2][4];
   {
-    const __nv_bfloat16* qbase = q + static_cast<int64_t>(seq) * ldq + static_cast<int64_t>(kvh) * G * D;
+    const __nv_bfloat16* qbase = q + static_cast<int64_t>(seq) * ldq + static_cast<int64_t>(kvh) * G * QW;
 #pragma unroll
     for (int kc = 0; kc < KC; ++kc) {
-      const int dcol = 32 * kc + 8 * qd;
+      const int map = 32 * kc / QW, dcol = 32 * kc - map * QW + 8 * qd;
+      const bool mine = QM == 1 || (gq & 1) == map;               // (rows gq and gq + 8 belong to the same map)
       uint4 lo = make_uint4(0, 0, 0, 0), hi = make_uint4(0, 0, 0, 0);
-      if (gq < G) lo = *reinterpret_cast<const uint4*>(qbase + gq * D + dcol);
-      if (gq + 8 < G) hi = *reinterpret_cast<const uint4*>(qbase + (gq + 8) * D + dcol);
+      if (gq < G && mine) lo = *reinterpret_cast<const uint4*>(qbase + gq * QW + dcol);
+      if (gq + 8 < G && mine) hi = *reinterpret_cast<const uint4*>(qbase + (gq + 8) * QW + dcol);
       qf[kc][0][0] = lo.x; qf[kc][0][1] = hi.x; qf[kc][0][2] = lo.y; qf[kc][0][3] = hi.y;
       qf[kc][1][0] = lo.z; qf[kc][1][1] = hi.z; qf[kc][1][2] = lo.w; qf[kc][1][3] = hi.w;
     }
@@ -82,22 +87,20 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;   // rows gq and gq+8
 
   const int32_t* bt = block_table + static_cast<int64_t>(seq) * ld_bt;
-  constexpr int kLinesPerPage = kPage * D * 2 / 128;          // 128-byte lines in one K (or V) page of one kv head
+  constexpr int kLinesK = kPage * DK * 2 / 128, kLinesV = kPage * DV * 2 / 128;          // 128-byte lines in one page of one kv head
   auto page_of = [&](int p) { return p < kept_pages ? p : p + gap; };
   int64_t blk_next = (p_begin + warp < p_end) ? bt[page_of(p_begin + warp)] : 0;
   for (int p = p_begin + warp; p < p_end; p += kAttnWarps) {
     const int64_t blk = blk_next;
-    const __nv_bfloat16* kp = k_cache + ((blk * nkv + kvh) * kPage) * D;
-    const __nv_bfloat16* vp = v_cache + ((blk * nkv + kvh) * kPage) * D;
+    const __nv_bfloat16* kp = k_cache + ((blk * nkv + kvh) * kPage) * DK;
+    const __nv_bfloat16* vp = v_cache + ((blk * nkv + kvh) * kPage) * DV;
     // ---- software prefetch: look up this warp's NEXT page now (breaks the block-table -> KV dependent-load chain) and pull
     // its K and V lines into L2 while the current page is being consumed (zero register cost, doubles bytes in flight)
     if (p + kAttnWarps < p_end) {
       blk_next = bt[page_of(p + kAttnWarps)];
-      if (lane < kLinesPerPage) {
-        const int64_t off = ((blk_next * nkv + kvh) * kPage) * D + lane * 64;
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(k_cache + off));
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(v_cache + off));
-      }
+      const int64_t next = (blk_next * nkv + kvh) * kPage;
+      if (lane < kLinesK) asm volatile("prefetch.global.L2 [%0];" ::"l"(k_cache + next * DK + lane * 64));
+      if (lane < kLinesV) asm volatile("prefetch.global.L2 [%0];" ::"l"(v_cache + next * DV + lane * 64));
     }
     // ---- issue every load of this page up front (16 x LDG.128 in flight per lane)
     uint4 kr[2][KC];
@@ -105,14 +108,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int kc = 0; kc < KC; ++kc)
-        kr[j][kc] = *reinterpret_cast<const uint4*>(kp + (8 * j + gq) * D + 32 * kc + 8 * qd);
+        kr[j][kc] = *reinterpret_cast<const uint4*>(kp + (8 * j + gq) * DK + 32 * kc + 8 * qd);
     uint4 vr[4][DB];
     const int vt[4] = {2 * qd, 2 * qd + 1, 8 + 2 * qd, 9 + 2 * qd};
 #pragma unroll
     for (int t = 0; t < 4; ++t)
 #pragma unroll
       for (int db = 0; db < DB; ++db)
-        vr[t][db] = *reinterpret_cast<const uint4*>(vp + vt[t] * D + 64 * db + 8 * gq);
+        vr[t][db] = *reinterpret_cast<const uint4*>(vp + vt[t] * DV + 64 * db + 8 * gq);
 
     // ---- S = Q K^T for 16 tokens (two n-tiles of 8)
     float s[2][4];
@@ -193,7 +196,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
 
   // ---- combine the 4 warps through shared memory
   __shared__ float sm_m[kAttnWarps][16], sm_l[kAttnWarps][16];
-  __shared__ float sm_o[kAttnWarps][16][D + 4];
+  __shared__ float sm_o[kAttnWarps][16][DV + 4];
   if (qd == 0) {
     sm_m[warp][gq] = m_lo; sm_m[warp][gq + 8] = m_hi;
     sm_l[warp][gq] = l_lo; sm_l[warp][gq + 8] = l_hi;
@@ -210,8 +213,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
       sm_o[warp][gq + 8][64 * db + 8 * (2 * qd + 1) + nt] = acc[3];
     }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < G * D; idx += kAttnWarps * 32) {
-    const int g = idx / D, dcol = idx - g * D;
+  for (int idx = threadIdx.x; idx < G * DV; idx += kAttnWarps * 32) {
+    const int g = idx / DV, dcol = idx - g * DV;
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kAttnWarps; ++w) mm = fmaxf(mm, sm_m[w][g]);
@@ -224,11 +227,11 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
     }
     const int head = kvh * G + g;
     if (out_direct) {        // single split: normalise and write the final bf16 output here (no merge kernel)
-      out_direct[static_cast<int64_t>(seq) * ldo + head * D + dcol] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+      out_direct[static_cast<int64_t>(seq) * ldo + head * DV + dcol] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
       continue;
     }
     const int64_t base = (static_cast<int64_t>(seq) * nq + head) * splits + split;
-    o_part[base * D + dcol] = acc;
+    o_part[base * DV + dcol] = acc;
     if (dcol == 0) { ml_part[base * 2] = mm; ml_part[base * 2 + 1] = ll; }
   }
 }
@@ -257,6 +260,42 @@ __global__ void decode_merge_kernel(const float* __restrict__ o_part, const floa
   }
 }
 
+// merge splits of both maps -> (a1 - lam a2) / sqrt(mean^2 + eps) * keep, bf16 [num_seqs, nh * dv_out]; one CTA of D threads per (sequence, head)
+template <int D>
+__global__ void __launch_bounds__(D) decode_merge_maps_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part, int splits,
+                                                              const float* __restrict__ lam, float keep, float eps, __nv_bfloat16* __restrict__ out, int nh,
+                                                              int dv_out) {
+  __shared__ float red[D / 32];
+  const int64_t row = blockIdx.x;                 // sequence * nh + head
+  const int c = threadIdx.x;
+  float a[2];
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const int64_t base = (row * 2 + m) * splits;
+    float mm = -INFINITY;
+    for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ml_part[(base + s) * 2]);
+    float ll = 0.f, acc = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float ms = ml_part[(base + s) * 2];
+      if (ms == -INFINITY) continue;
+      const float f = exp2f(ms - mm);
+      ll += ml_part[(base + s) * 2 + 1] * f;
+      acc += o_part[(base + s) * D + c] * f;
+    }
+    a[m] = ll > 0.f ? acc / ll : 0.f;
+  }
+  const float o = c < dv_out ? a[0] - lam[0] * a[1] : 0.f;
+  float ss = o * o;
+#pragma unroll
+  for (int k = 16; k; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+  if ((c & 31) == 0) red[c >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < D / 32; ++k) ss += red[k];
+  if (c < dv_out) out[row * dv_out + c] = __float2bfloat16(o * rsqrtf(ss / dv_out + eps) * keep);
+}
+
 }  // namespace prl
 
 using namespace prl;
@@ -282,7 +321,7 @@ extern "C" int prl_paged_decode(const void* q, int64_t ldq, const void* k_cache,
   const int grid = num_seqs * nkv * splits;
   static const int minb = [] { const char* e = getenv("POLYRL_DECODE_MINB"); return e ? atoi(e) : 3; }();
   if (d == 128) {
-    auto kern = minb >= 4 ? paged_decode_kernel<128, 4> : paged_decode_kernel<128, 3>;
+    auto kern = minb >= 4 ? paged_decode_kernel<128, 128, 1, 4> : paged_decode_kernel<128, 128, 1, 3>;
     kern<<<grid, kAttnWarps * 32, 0, s>>>(
         static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(k_cache),
         static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, o_part,
@@ -290,7 +329,7 @@ extern "C" int prl_paged_decode(const void* q, int64_t ldq, const void* k_cache,
     if (splits > 1)
       decode_merge_kernel<128><<<num_seqs * nq, 128, 0, s>>>(o_part, ml_part, splits, static_cast<__nv_bfloat16*>(out), ldo, nq);
   } else if (d == 64) {
-    paged_decode_kernel<64, 3><<<grid, kAttnWarps * 32, 0, s>>>(
+    paged_decode_kernel<64, 64, 1, 3><<<grid, kAttnWarps * 32, 0, s>>>(
         static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(k_cache),
         static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, o_part,
         ml_part, splits == 1 ? static_cast<__nv_bfloat16*>(out) : nullptr, ldo);
@@ -299,6 +338,36 @@ extern "C" int prl_paged_decode(const void* q, int64_t ldq, const void* k_cache,
   } else {
     return -31;
   }
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// differential attention: kw = width of a map's cached key (32 or 64; 32: q rows are 64 wide, zero outside their map's half), vw = 64 or 128
+extern "C" int prl_map_decode_ok(int kw, int vw, int rep) { return (kw == 32 || kw == 64) && (vw == 64 || vw == 128) && rep >= 1 && 2 * rep <= 16; }
+
+// q:[num_seqs, nh * 2, 64] contiguous, caches [blocks, nkv, 16, 2 kw] / [blocks, nkv, 16, vw], out [num_seqs, nh * dv_out]; workspace of
+// prl_paged_decode_workspace_floats(num_seqs, 2 * nh, vw, splits)
+extern "C" int prl_map_decode(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_table, int64_t ld_bt, const int32_t* seq_lens,
+                              int num_seqs, int nh, int nkv, int kw, int vw, int dv_out, float sm_scale, int splits, int window, const float* lam, float keep,
+                              float eps, float* workspace, void* out, cudaStream_t s) {
+  if (num_seqs <= 0) return 0;
+  if (nkv < 1 || nh % nkv || !prl_map_decode_ok(kw, vw, nh / nkv) || window < 1 || dv_out < 1 || dv_out > vw) return -32;
+  if (splits < 1) splits = 1;
+  const int nq = 2 * nh, grid = num_seqs * nkv * splits;
+  float* ml_part = workspace + static_cast<int64_t>(num_seqs) * nq * splits * vw;
+  const float scale_log2 = sm_scale * 1.4426950408889634f;
+#define PRL_MAP_DECODE(DK, DV, QM)                                                                                                                       \
+  paged_decode_kernel<DK, DV, QM, 3><<<grid, kAttnWarps * 32, 0, s>>>(                                                                                    \
+      static_cast<const __nv_bfloat16*>(q), nq * 64, static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache), block_table, \
+      ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, 0, workspace, ml_part, nullptr, 0)
+  if (kw == 32 && vw == 64) PRL_MAP_DECODE(64, 64, 1);
+  else if (kw == 32) PRL_MAP_DECODE(64, 128, 1);
+  else if (vw == 64) PRL_MAP_DECODE(128, 64, 2);
+  else PRL_MAP_DECODE(128, 128, 2);
+#undef PRL_MAP_DECODE
+  __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
+  if (vw == 64) decode_merge_maps_kernel<64><<<num_seqs * nh, 64, 0, s>>>(workspace, ml_part, splits, lam, keep, eps, o, nh, dv_out);
+  else decode_merge_maps_kernel<128><<<num_seqs * nh, 128, 0, s>>>(workspace, ml_part, splits, lam, keep, eps, o, nh, dv_out);
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

@@ -96,20 +96,25 @@ struct AccReader {
   }
 };
 
-// Communication policy.  kCommWarps extra warps per CTA run `Comm::run` (peer-memory copies) while
+// Communication and grouping policy.  `m_blocks` and `b_row` let a grouped product (one weight per group of m-blocks) read its plan
+// from device memory: the number of m-blocks in use, and the first row of B for an m-block.  kCommWarps extra warps per CTA run `Comm::run` (peer-memory copies) while
 // the TMA producer consults `Comm::wait_n_block` before touching the rows of B of an n-block.
 struct NoComm {
   struct Params {};
   static constexpr int kCommWarps = 0;
   __device__ __forceinline__ static void wait_n_block(const Params&, int /*n_blk*/) {}
   __device__ __forceinline__ static void run(const Params&, int /*tid*/) {}
+  template <class P>
+  __device__ __forceinline__ static int m_blocks(const P&, int launched) { return launched; }
+  template <class P>
+  __device__ __forceinline__ static int b_row(const P&, int /*m_blk*/, int /*N*/) { return 0; }
 };
 using NoGate = NoComm;
 
 template <class Cfg, class Epi, class Gate, bool IS_FP8>
 __global__ void __launch_bounds__(kNumThreads + 32 * Gate::kCommWarps, 1)
 gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
-                  typename Epi::Params ep, typename Gate::Params gp, int M, int N, int K, int num_m_blocks,
+                  typename Epi::Params ep, typename Gate::Params gp, int M, int N, int K, int launched_m_blocks,
                   int num_n_blocks, int n_splits, int nb_per_split, Sched sc) {
   constexpr int BN = Cfg::BLOCK_N;
   constexpr int kStages = Cfg::STAGES;
@@ -126,6 +131,7 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
+  const int num_m_blocks = Gate::m_blocks(gp, launched_m_blocks);
   const int total_work = num_m_blocks * n_splits;
   const int num_kb = (K + Cfg::BLOCK_K - 1) / Cfg::BLOCK_K;
 
@@ -158,6 +164,7 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
       uint32_t phase = 0;
       for (int w = blockIdx.x; w < total_work; w += gridDim.x) {
         const WorkInfo wi = decode_work(w, num_m_blocks, num_n_blocks, n_splits, nb_per_split, sc);
+        const int b0 = Gate::b_row(gp, wi.m_blk, N);
         for (int nbs = wi.n_begin; nbs < wi.n_end; ++nbs) {
           const int nb = rot_n(nbs, num_n_blocks, sc);
           Gate::wait_n_block(gp, nb);
@@ -166,7 +173,7 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
             mbar_expect_tx(&full_bar[stage], Cfg::STAGE_BYTES);
             tma_load_2d(&tmA, &full_bar[stage], smem_a + stage * Cfg::A_BYTES, kb * Cfg::BLOCK_K,
                         wi.m_blk * kBlockM);
-            tma_load_2d(&tmB, &full_bar[stage], smem_b + stage * Cfg::B_BYTES, kb * Cfg::BLOCK_K, nb * BN);
+            tma_load_2d(&tmB, &full_bar[stage], smem_b + stage * Cfg::B_BYTES, kb * Cfg::BLOCK_K, b0 + nb * BN);
             if (++stage == kStages) { stage = 0; phase ^= 1; }
           }
         }
@@ -294,12 +301,12 @@ inline int sm_count() {
 template <class Cfg, class Epi, class Gate, bool IS_FP8>
 int launch_gemm(const void* A, const void* B, int M, int N, int K, int64_t lda_bytes, int64_t ldb_bytes,
                 const typename Epi::Params& ep, const typename Gate::Params& gp, int n_splits, int max_ctas,
-                cudaStream_t stream, Sched sc = Sched{0, 1, 0}, bool full_grid = false) {
+                cudaStream_t stream, Sched sc = Sched{0, 1, 0}, bool full_grid = false, int groups = 1) {
   constexpr int EB = IS_FP8 ? 1 : 2;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   CUtensorMap tmA, tmB;
   if (make_tmap_kmajor(&tmA, A, M, K, lda_bytes, kBlockM, EB)) return -2;
-  if (make_tmap_kmajor(&tmB, B, N, K, ldb_bytes, Cfg::BLOCK_N, EB)) return -3;
+  if (make_tmap_kmajor(&tmB, B, static_cast<uint64_t>(N) * groups, K, ldb_bytes, Cfg::BLOCK_N, EB)) return -3;      // N rows per group
   const int num_m_blocks = (M + kBlockM - 1) / kBlockM;
   const int num_n_blocks = (N + Cfg::BLOCK_N - 1) / Cfg::BLOCK_N;
   if (n_splits <= 0 || n_splits > num_n_blocks) n_splits = num_n_blocks;

@@ -166,6 +166,18 @@ struct EpiGelu {
   }
 };
 
+// one weight [N, K] per group of 128-row tiles: plan[0] = tiles in use, plan[1 + groups + i] = group of tile i (mix_experts.cu)
+struct GroupedTiles : NoComm {
+  struct Params {
+    const int32_t* plan;
+    int groups;
+  };
+  __device__ __forceinline__ static void wait_n_block(const Params&, int) {}
+  __device__ __forceinline__ static void run(const Params&, int) {}
+  __device__ __forceinline__ static int m_blocks(const Params& p, int) { return p.plan[0]; }
+  __device__ __forceinline__ static int b_row(const Params& p, int m_blk, int N) { return p.plan[1 + p.groups + m_blk] * N; }
+};
+
 template <int BN, bool FP8>
 static int run_store(const void* A, const void* B, const StoreParams& sp, int M, int N, int K, int64_t lda, int64_t ldb,
                      cudaStream_t s) {
@@ -254,4 +266,27 @@ extern "C" int prl_gemm_gelu_bf16(const void* A, const void* W, void* H, int M, 
   }
   using Cfg = GemmCfg<64, 2>;
   return launch_gemm<Cfg, EpiGelu, NoGate, false>(A, W, M, N, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);
+}
+
+// rows of D = A · (weight of the rows' group)^T for 128-row tiles sorted by group.  A:[tiles * 128, K], W:[groups * N, K], contiguous.  glu: W holds gate
+// and up rows in blocks of 128, D:[., N / 2] = silu(gate) * up
+extern "C" int prl_gemm_experts_bf16(const void* A, const void* W, void* D, const int32_t* plan, int tiles, int groups, int N, int K, int glu,
+                                     cudaStream_t stream) {
+  if (tiles <= 0) return 0;
+  if (N <= 0 || K <= 0 || K % 8 || groups < 1 || static_cast<int64_t>(groups) * N > 0x7fffffff) return -12;
+  const int M = tiles * kBlockM;
+  const GroupedTiles::Params gp{plan, groups};
+  if (glu) {
+    if (N % 256) return -11;
+    SwigluParams sp{static_cast<__nv_bfloat16*>(D), nullptr, N / 2, 0};
+    return launch_gemm<GemmCfg<256, 2>, EpiSwiglu, GroupedTiles, false>(A, W, M, N, K, 2 * static_cast<int64_t>(K), 2 * static_cast<int64_t>(K), sp, gp, 0, 0,
+                                                                        stream, Sched{0, 1, 0}, false, groups);
+  }
+  if (N % 8) return -13;
+  StoreParams sp{static_cast<__nv_bfloat16*>(D), nullptr, N, nullptr, nullptr};
+  if (tiles >= 4 * groups && N >= 256)
+    return launch_gemm<GemmCfg<256, 2>, EpiStore, GroupedTiles, false>(A, W, M, N, K, 2 * static_cast<int64_t>(K), 2 * static_cast<int64_t>(K), sp, gp, 0, 0,
+                                                                       stream, Sched{0, 1, 0}, false, groups);
+  return launch_gemm<GemmCfg<128, 2>, EpiStore, GroupedTiles, false>(A, W, M, N, K, 2 * static_cast<int64_t>(K), 2 * static_cast<int64_t>(K), sp, gp, 0, 0, stream,
+                                                                     Sched{0, 1, 0}, false, groups);
 }

@@ -71,18 +71,29 @@ __global__ void __launch_bounds__(256) mix_norm_add_kernel(const T* __restrict__
   }
 }
 
-// ---- h = T(rms(x) * w) of fp32 rows
+// ---- h = T(rms(x) * w) of fp32 rows; center: of x minus its mean
 template <class T, int VEC>
-__global__ void __launch_bounds__(256) mix_rms_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, float eps) {
+__global__ void __launch_bounds__(256) mix_rms_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, float eps,
+                                                      int center) {
   __shared__ float red[8];
   const int64_t row = blockIdx.x;
   const float* xr = x + row * W;
-  float ss = 0.f;
+  float ss = 0.f, mean = 0.f;
+  if (center) {
+    float s = 0.f;
+    for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+      float v[VEC];
+      ld_vec<float, VEC>(xr + c, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s += v[i];
+    }
+    mean = block_sum<8>(s, red) / W;
+  }
   for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
     float v[VEC];
     ld_vec<float, VEC>(xr + c, v);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
+    for (int i = 0; i < VEC; ++i) ss += (v[i] - mean) * (v[i] - mean);
   }
   const float r = rsqrtf(block_sum<8>(ss, red) / W + eps);
   for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
@@ -90,7 +101,7 @@ __global__ void __launch_bounds__(256) mix_rms_kernel(const float* __restrict__ 
     ld_vec<float, VEC>(xr + c, v);
     ld_vec<float, VEC>(w + c, g);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[i] *= r * g[i];
+    for (int i = 0; i < VEC; ++i) v[i] = (v[i] - mean) * (r * g[i]);
     st_vec<T, VEC>(h + row * W + c, v);
   }
 }
@@ -517,17 +528,19 @@ __global__ void __launch_bounds__(256) mix_qk_prep_kernel(const T* __restrict__ 
     }
   }
 }
-// packed keys and values of flat cache rows; 16-byte units
+// packed keys and values of flat cache rows; ku / vu 16-byte units per head
 __global__ void __launch_bounds__(256) mix_gather_keys_kernel(const uint4* __restrict__ k_pool, const uint4* __restrict__ v_pool,
                                                               const int64_t* __restrict__ rows, uint4* __restrict__ k, uint4* __restrict__ v, int64_t n,
-                                                              int kheads, int units) {
-  const int64_t per = static_cast<int64_t>(kheads) * units;
+                                                              int kheads, int ku, int vu) {
+  const int64_t per = static_cast<int64_t>(kheads) * (ku + vu);
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x; i < n * per; i += static_cast<int64_t>(gridDim.x) * 256) {
-    const int64_t r = rows[i / per];
-    const int rest = static_cast<int>(i % per), g = rest / units, u = rest % units;
-    const int64_t src = ((r / 16 * kheads + g) * 16 + r % 16) * units + u;
-    k[i] = k_pool[src];
-    v[i] = v_pool[src];
+    const int64_t at = i / per, r = rows[at];
+    int rest = static_cast<int>(i % per);
+    const bool value = rest >= kheads * ku;
+    const int units = value ? vu : ku;
+    if (value) rest -= kheads * ku;
+    const int64_t src = ((r / 16 * kheads + rest / units) * 16 + r % 16) * units + rest % units, dst = at * kheads * units + rest;
+    if (value) v[dst] = v_pool[src]; else k[dst] = k_pool[src];
   }
 }
 
@@ -554,23 +567,9 @@ __global__ void mix_gelu_kernel(T* __restrict__ x, int64_t n) {
   }
 }
 
-static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
-
 }  // namespace prl
 
 using namespace prl;
-
-// dtype: 0 = bf16, 1 = fp32.  VEC = 8 when every row of every operand starts on a 16-byte boundary.
-#define MIX_DISPATCH(vec_, ...)                                                                      \
-  do {                                                                                               \
-    if (dtype == 0) {                                                                                \
-      using T = __nv_bfloat16;                                                                       \
-      if (vec_) { constexpr int VEC = 8; __VA_ARGS__; } else { constexpr int VEC = 1; __VA_ARGS__; } \
-    } else {                                                                                         \
-      using T = float;                                                                               \
-      if (vec_) { constexpr int VEC = 8; __VA_ARGS__; } else { constexpr int VEC = 1; __VA_ARGS__; } \
-    }                                                                                                \
-  } while (0)
 
 extern "C" int prl_mix_embed(const int64_t* ids, const void* emb, const float* w, float* x, void* h, int rows, int W, float eps, int dtype,
                              cudaStream_t st) {
@@ -588,10 +587,10 @@ extern "C" int prl_mix_norm_add(const void* y, int64_t ldy, float* x, const floa
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
-extern "C" int prl_mix_rms(const float* x, const float* w, void* h, int rows, int W, float eps, int dtype, cudaStream_t st) {
+extern "C" int prl_mix_rms(const float* x, const float* w, void* h, int rows, int W, float eps, int center, int dtype, cudaStream_t st) {
   if (rows <= 0) return 0;
   const bool vec = W % 8 == 0 && al16(x) && al16(w) && al16(h);
-  MIX_DISPATCH(vec, (mix_rms_kernel<T, VEC><<<rows, 256, 0, st>>>(x, w, static_cast<T*>(h), W, eps)));
+  MIX_DISPATCH(vec, (mix_rms_kernel<T, VEC><<<rows, 256, 0, st>>>(x, w, static_cast<T*>(h), W, eps, center)));
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
@@ -628,6 +627,20 @@ extern "C" int prl_mix_gated_norm(const void* y, int64_t ldy, const void* z, int
     return -223;
   }
 #undef MIX_GN
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+// the last taps - 1 inputs of every span become its slot's state
+extern "C" int prl_mix_conv_state(const void* x, int64_t ldx, void* state, const int32_t* cu, const int32_t* start, const int64_t* slot, int ch, int taps,
+                                  int spans, int dtype, cudaStream_t st) {
+  if (taps <= 1 || spans <= 0) return 0;
+  if (spans > 65535) return -220;
+  dim3 g2((ch + 127) / 128, spans);
+  if (dtype == 0)
+    mix_conv_state_kernel<__nv_bfloat16><<<g2, 128, 0, st>>>(static_cast<const __nv_bfloat16*>(x), ldx, static_cast<__nv_bfloat16*>(state), cu, start, slot, ch,
+                                                             taps);
+  else
+    mix_conv_state_kernel<float><<<g2, 128, 0, st>>>(static_cast<const float*>(x), ldx, static_cast<float*>(state), cu, start, slot, ch, taps);
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
@@ -677,17 +690,9 @@ extern "C" int prl_mix_conv(const void* x, int64_t ldx, const float* w, const fl
                                                                                   start, slot, seq_of, static_cast<T*>(out), ldo, ch, taps, total)));
     PRL_CUDA_CHECK(cudaGetLastError());
   }
-  if (taps > 1) {
-    dim3 g2((ch + 127) / 128, spans);
-    if (dtype == 0)
-      mix_conv_state_kernel<__nv_bfloat16><<<g2, 128, 0, st>>>(static_cast<const __nv_bfloat16*>(x), ldx, static_cast<__nv_bfloat16*>(state), cu, start,
-                                                               slot, ch, taps);
-    else
-      mix_conv_state_kernel<float><<<g2, 128, 0, st>>>(static_cast<const float*>(x), ldx, static_cast<float*>(state), cu, start, slot, ch, taps);
-    PRL_CUDA_CHECK(cudaGetLastError());
-  }
-  return 0;
+  return prl_mix_conv_state(x, ldx, state, cu, start, slot, ch, taps, spans, dtype, st);
 }
+
 extern "C" int prl_mix_latent_prep(const void* a, int64_t lda, int qr, int r, int rd, const float* wq, const float* wkv, const double* freq,
                                    const int64_t* pos, const int64_t* kvslot, void* cq, void* entry, void* pool, int rows, float eps, int dtype,
                                    cudaStream_t st) {
@@ -729,16 +734,18 @@ extern "C" int prl_mix_qk_prep(const void* p, int64_t ldp, int heads, int kheads
   return 0;
 }
 // row_bytes: bytes of one head's key, a multiple of 16
-extern "C" int prl_mix_gather_keys(const void* k_pool, const void* v_pool, const int64_t* rows, void* k, void* v, int64_t n, int kheads, int row_bytes,
-                                   cudaStream_t st) {
+extern "C" int prl_mix_gather_keys(const void* k_pool, const void* v_pool, const int64_t* rows, void* k, void* v, int64_t n, int kheads, int k_bytes,
+                                   int v_bytes, cudaStream_t st) {
   if (n <= 0) return 0;
-  if (row_bytes % 16 || !al16(k_pool) || !al16(v_pool) || !al16(k) || !al16(v)) return -225;
-  const int64_t blocks = (n * kheads * (row_bytes / 16) + 255) / 256;
+  if (k_bytes % 16 || v_bytes % 16 || !al16(k_pool) || !al16(v_pool) || !al16(k) || !al16(v)) return -225;
+  const int64_t blocks = (n * kheads * ((k_bytes + v_bytes) / 16) + 255) / 256;
   mix_gather_keys_kernel<<<static_cast<unsigned>(blocks < 148 * 32 ? blocks : 148 * 32), 256, 0, st>>>(
-      static_cast<const uint4*>(k_pool), static_cast<const uint4*>(v_pool), rows, static_cast<uint4*>(k), static_cast<uint4*>(v), n, kheads, row_bytes / 16);
+      static_cast<const uint4*>(k_pool), static_cast<const uint4*>(v_pool), rows, static_cast<uint4*>(k), static_cast<uint4*>(v), n, kheads, k_bytes / 16,
+      v_bytes / 16);
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
+
 extern "C" int prl_mix_clamped_glu(const void* gu, void* out, int64_t rows, int F, int blk, float limit, float alpha, int dtype, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (F <= 0 || blk <= 0 || F % blk) return -226;

@@ -86,6 +86,20 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return s;
 }
 
+inline bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+// dtype: 0 = bf16, 1 = fp32.  VEC = 8 when every row of every operand starts on a 16-byte boundary.
+#define MIX_DISPATCH(vec_, ...)                                                                      \
+  do {                                                                                               \
+    if (dtype == 0) {                                                                                \
+      using T = __nv_bfloat16;                                                                       \
+      if (vec_) { constexpr int VEC = 8; __VA_ARGS__; } else { constexpr int VEC = 1; __VA_ARGS__; } \
+    } else {                                                                                         \
+      using T = float;                                                                               \
+      if (vec_) { constexpr int VEC = 8; __VA_ARGS__; } else { constexpr int VEC = 1; __VA_ARGS__; } \
+    }                                                                                                \
+  } while (0)
+
 // The gated linear recurrences served by mix_scan.cu / mix_chunk.cu / mix_delta.cu:
 //   S_t = keep_t S_(t-1) + add_t k_t v_t^T,     y_t = S_t^T q_t
 //   kSsd    state-space duality: dt = softplus(g0 + b0), keep = exp(-exp(A_log) dt), add = dt;   y += D v

@@ -479,7 +479,7 @@ def _window(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b:
 def _diff(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch) -> torch.Tensor:
     nh, t, window = m["heads"], b.tokens, m["window"]
     kp, vp, eps = cache["k_pool"], cache["v_pool"], cfg.rms_norm_eps
-    mix = M.MapMix(w["lam"], float(m["diff"]), eps, m["vdim"])
+    mix = M.MapMix(w["lam"], float(m["diff"]), eps, m["vdim"], m["dim"])
     tl = b.t_long if packs(m, h.dtype, h.is_cuda) else 0            # tokens served by the packed kernel
     q, kv = M.map_prep(ops.linear(h, w["wqkv"]), w["b_qkv"], nh, m["dim"], m["vdim"], w["q_norm"], w["k_norm"], w["freq"], kp, vp, b, eps,
                        tl > 0 and b.gather is None)

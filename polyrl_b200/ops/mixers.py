@@ -160,7 +160,7 @@ def linear_silu_glu(x: torch.Tensor, wgu: torch.Tensor) -> torch.Tensor:
     """silu(gate) * up; ``wgu`` laid out as in ``linear_clamped_glu``.  Fused into the GEMM epilogue for bf16 rows."""
     f = wgu.shape[0] // 2
     if x.is_cuda and x.dtype == torch.bfloat16 and f % 128 == 0 and x.shape[1] % 8 == 0:
-        return _C().gemm_silu_glu(x, wgu)
+        return _C().gemm_swiglu(x, wgu, False)[0]
     return silu_glu(F.linear(x, wgu.to(x.dtype)), f)
 
 
@@ -281,12 +281,12 @@ def experts(h: torch.Tensor, router: torch.Tensor, wgu: torch.Tensor, wd: torch.
     logits = linear_f32(h, router)
     if h.is_cuda:
         C = _C()
-        pick, score, rank, plan = C.mix_route(logits, top)
-        rows, pos = C.mix_expert_rows(h, pick, score, rank, plan)
+        pick, score, rank, plan = C.mix_route(logits, top, _counter(h.device, e + 1))
+        rows, pos = C.mix_expert_rows(h, pick, score, rank, plan, e)
         if h.dtype == torch.bfloat16 and f % 128 == 0 and width % 8 == 0:
-            return Routed(C.gemm_experts(C.gemm_experts(rows, wgu, plan, True), wd, plan, False), pos)
-        gu = C.mix_expert_gemm(rows, wgu, plan)
-        return Routed(C.mix_expert_gemm(silu_glu(gu, f), wd, plan), pos)
+            return Routed(C.gemm_experts(C.gemm_experts(rows, wgu, plan, e, True), wd, plan, e, False), pos)
+        gu = C.mix_expert_gemm(rows, wgu, plan, e)
+        return Routed(C.mix_expert_gemm(silu_glu(gu, f), wd, plan, e), pos)
     score, pick = torch.topk(torch.sigmoid(logits), top, dim=-1)
     rows = h.new_empty(h.shape[0] * top, width)
     pos = torch.arange(rows.shape[0]).reshape(-1, top)
@@ -585,6 +585,7 @@ class MapMix:
     diff: float
     eps: float
     vdim: int
+    dim: int                    # of a query or key, without padding
 
     def __call__(self, a1: torch.Tensor, a2: torch.Tensor) -> torch.Tensor:
         return _rms((a1 - self.lam * a2)[..., :self.vdim], self.eps) * (1 - self.diff)
@@ -639,7 +640,7 @@ def map_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, t
 
             return _C().map_decode(q, k_pool, v_pool, table, kv_len, scale, _auto_splits(rows, g, min(max_len, window + 2 * PAGE)), window, mix.lam, mix.diff,
                                    mix.eps, mix.vdim)
-        return _C().mix_map_attention(q, k_pool, v_pool, table, seq_of, kv_len, scale, window, mix.lam, mix.diff, mix.eps, mix.vdim)
+        return _C().mix_map_attention(q, k_pool, v_pool, table, seq_of, kv_len, scale, window, mix.lam, mix.diff, mix.eps, mix.vdim, mix.dim)
     out = q.new_zeros(rows, h, mix.vdim)
     for i in range(rows):
         n = int(kv_len[i])
