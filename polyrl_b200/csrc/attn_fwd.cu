@@ -19,6 +19,8 @@
 // DK = 192 (latent attention expanded to heads: 128 + 64 rotary) keeps both K stages and drops to one V stage, which is
 // reloaded while the next scores and their softmax run.  An optional per-head sink adds exp(sink_h) to the softmax
 // denominator in the epilogue.
+// With two P stages (two maps per head) PV_j is read back after P_(j+1) has been written: the product runs while the softmax
+// warps work on the next scores.
 // Two maps per head (differential attention): the CTA runs the loop twice over the same values, keeps the first map's output in
 // TMEM (fp32) and writes  (a1 - lambda a2) / sqrt(mean^2 + eps) * keep.  Keys of width 32 lie pairwise in rows of 64 (both maps read
 // the same row, the queries are zero outside their half).
@@ -37,7 +39,9 @@ struct AfCfg {
   static constexpr int QKT = 128 * DK * 2;            // Q or K tile: DK / 64 chunks of 128 rows x 64 columns
   static constexpr int VT = 128 * DV * 2;             // V tile
   static constexpr int VST = DK * MAPS + DV <= 256 ? 2 : 1;       // V stages
-  static constexpr int SMEM = (MAPS + 2) * QKT /*Q, K x 2*/ + VST * VT /*V*/ + kAfTile /*P*/ + 1024 + 256;
+  static constexpr int BASE = (MAPS + 2) * QKT /*Q, K x 2*/ + VST * VT /*V*/ + 1024 + 256;
+  static constexpr int PST = MAPS == 2 && BASE + 2 * kAfTile <= 220 * 1024 ? 2 : 1;        // P stages
+  static constexpr int SMEM = BASE + PST * kAfTile;
 };
 
 struct AttnFwdParams {
@@ -66,22 +70,24 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
   using Cfg = AfCfg<DK, kAfD, MAPS>;
-  constexpr int QKT = Cfg::QKT, VST = Cfg::VST, VT = Cfg::VT, OW = kAfD / 2;
+  constexpr int QKT = Cfg::QKT, VST = Cfg::VST, VT = Cfg::VT, OW = kAfD / 2, PST = Cfg::PST;
   uint8_t* sK = smem + MAPS * QKT;                    // [2 stages]
   uint8_t* sV = smem + (MAPS + 2) * QKT;              // [VST stages]
   uint8_t* sP = sV + VST * VT;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + kAfTile);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + PST * kAfTile);
   uint64_t* q_full = bars;            // 1
   uint64_t* k_full = bars + 1;        // [2]
   uint64_t* v_full = bars + 3;        // [2]
   uint64_t* k_empty = bars + 5;       // [2]
   uint64_t* s_full = bars + 7;        // [2]
   uint64_t* s_empty = bars + 9;       // [2]  (128 arrivals)
-  uint64_t* p_full = bars + 11;       // 128 arrivals
+  uint64_t* p_full0 = bars + 11;      // 256 arrivals; P stage 1: bars + 16
   uint64_t* o_full = bars + 12;       // 1
   uint64_t* o_empty = bars + 13;      // 128 arrivals
   uint64_t* v_empty = bars + 14;      // [2]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
+  auto p_full = [&](int j) { return PST == 2 && (j & 1) ? bars + 16 : p_full0; };
+  auto p_phase = [&](int j) { return static_cast<uint32_t>(PST == 2 ? (j >> 1) & 1 : j & 1); };
   __shared__ int s_seq, s_q0;
   __shared__ float s_mx[2][2][128];             // [tile parity][warpgroup][row]: half-row maxima
   __shared__ float s_sum[MAPS][2][128];         // half-row sums
@@ -123,7 +129,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&k_empty[i], 1); mbar_init(&v_empty[i], 1);
       mbar_init(&s_full[i], 1); mbar_init(&s_empty[i], 256);
     }
-    mbar_init(p_full, 256); mbar_init(o_full, 1); mbar_init(o_empty, 256);
+    mbar_init(p_full0, 256); mbar_init(bars + 16, 256); mbar_init(o_full, 1); mbar_init(o_empty, 256);
     fence_barrier_init();
   }
   if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
@@ -176,14 +182,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       for (int j = 0; j < MAPS * nt; ++j) {
         const int s = j & 1;
         if (j + 1 < MAPS * nt) issue_s(j + 1);
-        mbar_wait(p_full, j & 1);
+        mbar_wait(p_full(j), p_phase(j));
         const int sv = j % VST;
         mbar_wait(&v_full[sv], (j / VST) & 1);
         mbar_wait(o_empty, (j & 1) ^ 1);
         tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk) {
-          const uint64_t da = umma_desc_sw128_kmajor(sP + (kk >> 2) * 16384) + 2 * (kk & 3);
+          const uint64_t da = umma_desc_sw128_kmajor(sP + (PST == 2 ? (j & 1) * kAfTile : 0) + (kk >> 2) * 16384) + 2 * (kk & 3);
           const uint64_t db = umma_desc_sw128_mnmajor(sV + sv * VT, 16384) + kk * 128;
           umma_bf16_ss(tO, da, db, idO, kk != 0);
         }
@@ -205,7 +211,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     float O[OW];
 #pragma unroll
     for (int i = 0; i < OW; ++i) O[i] = 0.f;
-    const uint32_t sP_u32 = smem_u32(sP) + g * 16384 + r * 128;
+    const uint32_t sP0_u32 = smem_u32(sP) + g * 16384 + r * 128;
     const bool rec = p.dbg != nullptr && blockIdx.x == gridDim.x / 2 && blockIdx.y == 0 && threadIdx.x == 64;
     long long* dbg = p.dbg;
     if (rec) dbg[0] = clock64();
@@ -218,7 +224,24 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         st_v4(dst + c, ov);
       }
     };
+    // own half of O = O * alpha + P V of key tile j
+    auto take = [&](int j, float alpha) {
+      mbar_wait(o_full, j & 1);
+      tc_fence_after();
+#pragma unroll
+      for (int c = 0; c < OW; c += 32) {
+        uint32_t v[32];
+        __syncwarp();
+        tmem_ld_32x32(tO + lane_base + g * OW + c, v);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) O[c + i] = O[c + i] * alpha + __uint_as_float(v[i]);
+      }
+      tc_fence_before();
+      mbar_arrive(o_empty);
+    };
     for (int map = 0; map < MAPS; ++map) {
+    float alpha_before = 0.f;
     for (int j = map * nt; j < (map + 1) * nt; ++j) {
       const int s = j & 1;
       mbar_wait(&s_full[s], (j >> 1) & 1);
@@ -255,6 +278,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
       const float alpha = (m_run == -INFINITY) ? 0.f : fast_exp2((m_run - m_use) * p.scale_log2);
       const float mb = m_use * p.scale_log2;
+      const uint32_t sP_u32 = sP0_u32 + (PST == 2 ? (j & 1) * kAfTile : 0);       // (PV_(j-2) has been taken: its P may be overwritten)
       // pass 2: probabilities -> bf16 P in shared memory (K-major, 128B swizzle), partial row sum
       float lsum = 0.f;
 #pragma unroll
@@ -291,27 +315,20 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (rec && j < 30) dbg[3 + 5 * j] = clock64();
       fence_proxy_async();
       tc_fence_before();
-      mbar_arrive(p_full);
+      mbar_arrive(p_full(j));
       mbar_arrive(&s_empty[s]);
       l_run = l_run * alpha + lsum;
       m_run = m_new;
-      // own half of O = O * alpha + P V
-      mbar_wait(o_full, j & 1);
-      tc_fence_after();
       if (rec && j < 30) dbg[4 + 5 * j] = clock64();
-#pragma unroll
-      for (int c = 0; c < OW; c += 32) {
-        uint32_t v[32];
-        __syncwarp();
-        tmem_ld_32x32(tO + lane_base + g * OW + c, v);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 32; ++i) O[c + i] = O[c + i] * alpha + __uint_as_float(v[i]);
+      if constexpr (PST == 2) {
+        if (j > map * nt) take(j - 1, alpha_before);
+        alpha_before = alpha;
+      } else {
+        take(j, alpha);
       }
-      tc_fence_before();
-      mbar_arrive(o_empty);
       if (rec && j < 30) dbg[5 + 5 * j] = clock64();
     }
+    if constexpr (PST == 2) take((map + 1) * nt - 1, alpha_before);
     // total row sum = the two groups' partial sums (same running max on both sides)
     s_sum[map][g][r] = l_run;
     asm volatile("bar.sync 1, 256;" ::: "memory");

@@ -8,21 +8,34 @@
 
 namespace prl {
 
-// NaN-free loads of `past` in groups: coefficients in shared memory, four results in flight
-template <class T, int VEC>
-__global__ void __launch_bounds__(256) mix_block_kernel(BlockParams p) {
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
+// NT threads per token; the results are read four layers at a time, their coefficients lie in shared memory
+template <class T, int VEC, int NT>
+__global__ void __launch_bounds__(NT, 1024 / NT) mix_block_kernel(BlockParams p) {
   extern __shared__ float sh[];                        // row [W], then a_prev [n + 1] and a_cur [n + 2]
-  __shared__ float red[8];
+  __shared__ float red[NT / 32];
   float* ap = sh + (p.W + 3) / 4 * 4;
   float* ac = ap + p.n + 1;
   const int64_t row = blockIdx.x;
   const int W = p.W;
   float* xr = p.past + row * W;
-  if (p.a_prev) for (int j = threadIdx.x; j <= p.n; j += 256) ap[j] = p.a_prev[j];
-  if (p.a_cur) for (int j = threadIdx.x; j <= p.n + 1; j += 256) ac[j] = p.a_cur[j];
+  if (p.a_prev) for (int j = threadIdx.x; j <= p.n; j += NT) ap[j] = p.a_prev[j];
+  if (p.a_cur) for (int j = threadIdx.x; j <= p.n + 1; j += NT) ac[j] = p.a_cur[j];
+  if (p.c1) {                                           // what the convolution reads after the norm
+    const T* st = static_cast<const T*>(p.state) + p.slot[row] * static_cast<int64_t>(p.taps - 1) * W;
+    for (int c = threadIdx.x * VEC; c < W; c += NT * VEC) {
+      prefetch_l2(p.w_next + c);
+      for (int j = 0; j < p.taps; ++j) {
+        if (j + 1 < p.taps) prefetch_l2(st + static_cast<int64_t>(j) * W + c);
+        prefetch_l2(p.c1 + static_cast<int64_t>(j) * W + c);
+        if (p.c2) prefetch_l2(p.c2 + static_cast<int64_t>(j) * W + c);
+      }
+    }
+  }
   __syncthreads();
   float s = 0.f;
-  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+  for (int c = threadIdx.x * VEC; c < W; c += NT * VEC) {
     float x[VEC], avg[VEC];
     if (p.ids) {
       ld_vec<T, VEC>(static_cast<const T*>(p.emb) + p.ids[row] * W + c, x);
@@ -93,18 +106,18 @@ __global__ void __launch_bounds__(256) mix_block_kernel(BlockParams p) {
   }
   if (!p.w_next) return;
   // a thread reads back only what it wrote to the row
-  const float mean = p.center ? block_sum<8>(s, red) / W : 0.f;
+  const float mean = p.center ? block_sum<NT / 32>(s, red) / W : 0.f;
   float ss = 0.f;
-  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+  for (int c = threadIdx.x * VEC; c < W; c += NT * VEC) {
     float x[VEC];
     ld_vec<float, VEC>(sh + c, x);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) ss += (x[i] - mean) * (x[i] - mean);
   }
-  const float r = rsqrtf(block_sum<8>(ss, red) / W + p.eps);
+  const float r = rsqrtf(block_sum<NT / 32>(ss, red) / W + p.eps);
   const bool fresh = p.c1 && p.start[row] == 0;
   T* st = p.c1 ? static_cast<T*>(p.state) + p.slot[row] * static_cast<int64_t>(p.taps - 1) * W : nullptr;
-  for (int c = threadIdx.x * VEC; c < W; c += 256 * VEC) {
+  for (int c = threadIdx.x * VEC; c < W; c += NT * VEC) {
     float x[VEC], g[VEC];
     ld_vec<float, VEC>(sh + c, x);
     ld_vec<float, VEC>(p.w_next + c, g);
@@ -248,7 +261,14 @@ __global__ void __launch_bounds__(256) mix_poly_norm_kernel(const T* __restrict_
   __shared__ float red[8][3];
   const int64_t row = blockIdx.x;
   const T* zr = z + row * ldz;
-  float hold[HOLD][VEC], s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  constexpr int U = sizeof(T) * VEC % 16 == 0 ? sizeof(T) * VEC / 16 : 0;      // held as loaded: 16-byte units, or one element
+  uint4 raw[HOLD][U ? U : 1];
+  T one[HOLD];
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  auto get = [&](int k, float (&v)[VEC]) {
+    if constexpr (U > 0) ld_vec<T, VEC>(reinterpret_cast<const T*>(&raw[k][0]), v);
+    else v[0] = to_f<T>(one[k]);
+  };
   const bool held = F <= 256 * VEC * HOLD;
   auto add = [&](const float (&v)[VEC]) {
 #pragma unroll
@@ -261,7 +281,22 @@ __global__ void __launch_bounds__(256) mix_poly_norm_kernel(const T* __restrict_
 #pragma unroll
     for (int k = 0; k < HOLD; ++k) {
       const int c = (k * 256 + threadIdx.x) * VEC;
-      if (c < F) { ld_vec<T, VEC>(zr + c, hold[k]); add(hold[k]); }
+      if (c < F) {
+        if constexpr (U > 0) {
+#pragma unroll
+          for (int u = 0; u < U; ++u) raw[k][u] = reinterpret_cast<const uint4*>(zr + c)[u];
+        } else {
+          one[k] = zr[c];
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < HOLD; ++k) {
+      if ((k * 256 + threadIdx.x) * VEC < F) {
+        float v[VEC];
+        get(k, v);
+        add(v);
+      }
     }
   } else {
     for (int c = threadIdx.x * VEC; c < F; c += 256 * VEC) {
@@ -286,7 +321,11 @@ __global__ void __launch_bounds__(256) mix_poly_norm_kernel(const T* __restrict_
 #pragma unroll
     for (int k = 0; k < HOLD; ++k) {
       const int c = (k * 256 + threadIdx.x) * VEC;
-      if (c < F) put(hold[k], c);
+      if (c < F) {
+        float v[VEC];
+        get(k, v);
+        put(v, c);
+      }
     }
   } else {
     for (int c = threadIdx.x * VEC; c < F; c += 256 * VEC) {
@@ -325,11 +364,20 @@ extern "C" int prl_mix_block(const BlockParams* bp, int dtype, cudaStream_t st) 
     vec = vec && al16(q);
   const int smem = ((p.W + 3) / 4 * 4 + 2 * p.n + 3) * 4;
   if (smem > 200 * 1024) return -261;
+  // few rows: one vector per thread where the width allows it (latency); many: small CTAs that overlap one another's barriers
+  const bool few = p.R <= 4 * 148;
+#define MIX_BLOCK(NT)                                                                                                            \
+  do {                                                                                                                           \
+    if (smem > 40 * 1024)                                                                                                        \
+      PRL_CUDA_CHECK(cudaFuncSetAttribute(mix_block_kernel<T, VEC, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));     \
+    mix_block_kernel<T, VEC, NT><<<p.R, NT, smem, st>>>(p);                                                                      \
+  } while (0)
   MIX_DISPATCH(vec, {
-    if (smem > 40 * 1024)
-      PRL_CUDA_CHECK(cudaFuncSetAttribute(mix_block_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    mix_block_kernel<T, VEC><<<p.R, 256, smem, st>>>(p);
+    if (p.W <= 128 * VEC || !few) MIX_BLOCK(128);
+    else if (p.W <= 256 * VEC) MIX_BLOCK(256);
+    else MIX_BLOCK(512);
   });
+#undef MIX_BLOCK
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

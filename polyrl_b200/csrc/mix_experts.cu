@@ -8,19 +8,17 @@
 namespace prl {
 
 constexpr int kMoeTile = 128;
-constexpr int kRouteTokens = 32;                        // tokens per CTA
-
-// one warp per token: the `top` largest logits (ties: the lower index), s = sigmoid; counts [E + 1] are zero between launches
+// a warp per token, `per` tokens per CTA: the `top` largest logits (ties: the lower index), s = sigmoid; counts [E + 1] are zero between launches
 template <int RN>
-__global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int top, int32_t* __restrict__ pick,
+__global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int top, int per, int32_t* __restrict__ pick,
                                                         float* __restrict__ score, int32_t* __restrict__ rank, int32_t* __restrict__ counts,
                                                         int32_t* __restrict__ plan) {
   extern __shared__ int hist[];                         // [E]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int e = threadIdx.x; e < E; e += 256) hist[e] = 0;
   __syncthreads();
-  for (int i = warp; i < kRouteTokens; i += 8) {
-    const int t = blockIdx.x * kRouteTokens + i;
+  for (int i = warp; i < per; i += 8) {
+    const int t = blockIdx.x * per + i;
     if (t >= T) break;
     float v[RN];
     uint32_t taken = 0;
@@ -59,8 +57,8 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
     if (hist[e]) hist[e] = atomicAdd(&counts[e], hist[e]);
   __syncthreads();
   if (lane == 0) {
-    for (int i = warp; i < kRouteTokens; i += 8) {
-      const int t = blockIdx.x * kRouteTokens + i;
+    for (int i = warp; i < per; i += 8) {
+      const int t = blockIdx.x * per + i;
       if (t >= T) break;
       for (int k = 0; k < top; ++k) {
         const int64_t at = static_cast<int64_t>(t) * top + k;
@@ -171,8 +169,8 @@ extern "C" int prl_mix_route(const float* logits, int64_t ld, int T, int E, int 
                              cudaStream_t st) {
   if (T <= 0) return 0;
   if (E < 1 || E > 1024 || top < 1 || top > E) return -270;
-  const int grid = (T + kRouteTokens - 1) / kRouteTokens;
-#define MIX_RT(RN) mix_route_kernel<RN><<<grid, 256, E * 4, st>>>(logits, ld, T, E, top, pick, score, rank, counts, plan)
+  const int per = T <= 8 * 148 ? 8 : 32, grid = (T + per - 1) / per;
+#define MIX_RT(RN) mix_route_kernel<RN><<<grid, 256, E * 4, st>>>(logits, ld, T, E, top, per, pick, score, rank, counts, plan)
   if (E <= 32) MIX_RT(1);
   else if (E <= 128) MIX_RT(4);
   else MIX_RT(32);

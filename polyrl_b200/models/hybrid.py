@@ -211,7 +211,7 @@ _DERIVED_ONLY = ("wq_up", "wk_up", "wv_up", "map_mix")              # stored ten
 
 def packs(m: dict, dtype: torch.dtype, is_cuda: bool) -> bool:
     """Long spans of this ``window`` or ``diff`` layer run on the packed tcgen05 attention."""
-    return is_cuda and dtype == torch.bfloat16 and max(m["dim"], m["vdim"]) <= 128
+    return is_cuda and dtype == torch.bfloat16 and max(m["dim"], m.get("vdim", 0)) <= 128
 
 
 def cache_width(m: dict, dtype: torch.dtype) -> int:
@@ -532,6 +532,38 @@ def _conv_of(cfg: ModelConfig, w: dict, cache: dict) -> M.InputConv | None:
     return M.InputConv(w["conv1"], w.get("conv2"), cache["input"]) if cfg.input_conv else None
 
 
+_SIDE: dict = {}
+
+
+def _side_stream(device: torch.device):
+    key = device.index
+    if key not in _SIDE:
+        _SIDE[key] = torch.cuda.Stream(device=device)
+    return _SIDE[key]
+
+
+def _sublayers(cfg: ModelConfig, i: int, w: dict, h: tuple, cache: dict, b: M.SpanBatch) -> tuple:
+    """(mixer rows, feed-forward rows, routed rows).  In single-token steps the two sublayers run on streams of their own: each is a chain of
+    kernels that leave most of the GPU idle.  What the side stream allocates is reused only by its own later work, which waits for the
+    kernel that consumed it; what it reads stays referenced until it has been waited for."""
+    lay = cfg.layers[i]
+
+    def mixer():
+        return ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h[0], cache, b), w["wo"])
+
+    if not lay["ff"]:
+        return mixer(), None, None
+    if not h[1].is_cuda or b.seq_of is not None:
+        return (mixer(), *_feed_forward(cfg, lay, w, h[1]))
+    main, side = torch.cuda.current_stream(h[1].device), _side_stream(h[1].device)
+    side.wait_stream(main)
+    with torch.cuda.stream(side):
+        y2, routed = _feed_forward(cfg, lay, w, h[1])
+    y1 = mixer()
+    main.wait_stream(side)
+    return y1, y2, routed
+
+
 def _forward_parallel(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids: torch.Tensor, caches: list[dict], b: M.SpanBatch,
                       final_norm: torch.Tensor | None) -> tuple[torch.Tensor, torch.Tensor]:
     n = len(layer_w)
@@ -539,9 +571,8 @@ def _forward_parallel(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids:
                             _conv_of(cfg, layer_w[0], caches[0]), b)
     x = None
     for i, w in enumerate(layer_w):
-        lay, last = cfg.layers[i], i + 1 == n
-        y1 = ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h[0], caches[i], b), w["wo"])
-        y2, routed = _feed_forward(cfg, lay, w, h[1]) if lay["ff"] else (None, None)
+        last = i + 1 == n
+        y1, y2, routed = _sublayers(cfg, i, w, h, caches[i], b)
         x, h = M.block_add(past, i, y1, y2, routed, w.get("ls1"), w.get("ls2"), layer_w[i - 1].get("depth") if i else None, w.get("depth"),
                            final_norm if last else layer_w[i + 1]["pre1"], cfg.rms_norm_eps, cfg.layer_norm,
                            None if last else _conv_of(cfg, layer_w[i + 1], caches[i + 1]), b, want_x=last)

@@ -55,9 +55,10 @@ _COUNTERS: dict = {}
 _RETIRED: list = []     # outgrown counters stay alive: captured graphs hold their address
 
 
-def _counter(device: torch.device, n: int) -> torch.Tensor:
-    """Zeroed arrival counters of the recurrence kernels (each launch leaves them zero again); the last element is an error flag."""
-    key = (device.type, device.index)
+def _counter(device: torch.device, n: int, use: str = "scan") -> torch.Tensor:
+    """Zeroed arrival counters of the recurrence and routing kernels (each launch leaves them zero again), one set per ``use``: the two may run
+    at the same time; the last element is an error flag."""
+    key = (device.type, device.index, use)
     if key not in _COUNTERS or _COUNTERS[key].numel() <= n:
         _RETIRED.append(_COUNTERS.get(key))
         _COUNTERS[key] = torch.zeros(max(n, 1 << 17) + 1, device=device, dtype=torch.int32)
@@ -66,7 +67,7 @@ def _counter(device: torch.device, n: int) -> torch.Tensor:
 
 def check_errors(device: torch.device) -> None:
     """Raise if a bounded wait inside a kernel ran out (reads one flag back: call it where the host synchronises anyway)."""
-    c = _COUNTERS.get((device.type, device.index))
+    c = _COUNTERS.get((device.type, device.index, "scan"))
     if c is not None and int(c[-1]):
         raise RuntimeError("a wait inside a chunked recurrence kernel timed out")
 
@@ -157,9 +158,11 @@ def linear_clamped_glu(x: torch.Tensor, wgu: torch.Tensor, limit: float, alpha: 
 
 
 def linear_silu_glu(x: torch.Tensor, wgu: torch.Tensor) -> torch.Tensor:
-    """silu(gate) * up; ``wgu`` laid out as in ``linear_clamped_glu``.  Fused into the GEMM epilogue for bf16 rows."""
+    """silu(gate) * up; ``wgu`` laid out as in ``linear_clamped_glu``.  Fused into the GEMM epilogue for bf16 rows — but for few rows of a narrow
+    layer, whose 256-row weight tiles would leave most SMs idle: library product, then the gate."""
     f = wgu.shape[0] // 2
-    if x.is_cuda and x.dtype == torch.bfloat16 and f % 128 == 0 and x.shape[1] % 8 == 0:
+    narrow = x.shape[0] <= 128 and wgu.shape[0] < 256 * 74
+    if not narrow and x.is_cuda and x.dtype == torch.bfloat16 and f % 128 == 0 and x.shape[1] % 8 == 0:
         return _C().gemm_swiglu(x, wgu, False)[0]
     return silu_glu(F.linear(x, wgu.to(x.dtype)), f)
 
@@ -281,7 +284,7 @@ def experts(h: torch.Tensor, router: torch.Tensor, wgu: torch.Tensor, wd: torch.
     logits = linear_f32(h, router)
     if h.is_cuda:
         C = _C()
-        pick, score, rank, plan = C.mix_route(logits, top, _counter(h.device, e + 1))
+        pick, score, rank, plan = C.mix_route(logits, top, _counter(h.device, e + 1, "route"))
         rows, pos = C.mix_expert_rows(h, pick, score, rank, plan, e)
         if h.dtype == torch.bfloat16 and f % 128 == 0 and width % 8 == 0:
             return Routed(C.gemm_experts(C.gemm_experts(rows, wgu, plan, e, True), wd, plan, e, False), pos)

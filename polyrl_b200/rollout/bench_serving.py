@@ -24,7 +24,7 @@ def _peaks() -> tuple[float, float, str]:
 
 def models(layers: int, design: str) -> dict:
     """The mixer stack and its closest stacks at the same width, feed-forward width and depth: llama with latent attention (MLA) beside
-    ludesun, ludesun beside lanilix, llama beside both."""
+    ludesun, ludesun beside lanilix, llama beside all; beside mabedra lanilix and a llama stack with the same experts in the same layers."""
     from ..models import ModelConfig, get_model_config
 
     def stack(name):
@@ -34,6 +34,11 @@ def models(layers: int, design: str) -> dict:
     hy = stack("ludesun-4b")
     base = dict(family="llama", vocab_size=hy.vocab_size, hidden_size=hy.hidden_size, intermediate_size=hy.intermediate_size, num_layers=layers, num_heads=32,
                 max_position_embeddings=16384, rope_theta=500000.0, rms_norm_eps=1e-5, eos_token_id=-1)
+    if design == "mabedra":
+        moe = dict(num_experts=16, num_experts_per_tok=2, moe_intermediate_size=2048, shared_expert_intermediate_size=4096, norm_topk_prob=False,
+                   dense_layers=tuple(range(0, layers, 4)))
+        return {"mabedra": stack("mabedra-7b"), "lanilix": stack("lanilix-4b"), "llama": ModelConfig(**base, num_kv_heads=8),
+                "llama with experts": ModelConfig(**base, num_kv_heads=8, **moe)}
     if design == "lanilix":
         return {"lanilix": stack("lanilix-4b"), "ludesun": hy, "llama": ModelConfig(**base, num_kv_heads=8)}
     return {"ludesun": hy,
@@ -67,6 +72,7 @@ def run_models(args) -> list[dict]:
     dev, rows = torch.device("cuda"), []
     prefills = [(16, 1024), (2, 8192)]
     decodes = [(64, 1024), (128, 2048)]
+    os.environ.setdefault("POLYRL_MOE_STATIC_DECODE", "1")        # llama-family experts: the decode form that can be captured
     for name, cfg in models(args.serving_layers, args.serving_design).items():
         w = TransformerWeights(cfg, device=dev, dtype=torch.bfloat16, init=True)
         n_params = cfg.num_params()
@@ -240,6 +246,106 @@ def run_kernels_lanilix(args) -> list[dict]:
     return K.rows
 
 
+def run_kernels_mabedra(args) -> list[dict]:
+    """Layer sizes of ``mabedra-7b``."""
+    from .. import ops
+    from ..ops import mixers as M
+    from ..ops.attention import attention_varlen
+
+    C, K = ops.ext(), _Kernels(args)
+    dev, rnd, rec = K.dev, K.rnd, K.rec
+    W, FF = 4096, 14336
+    f32 = dict(device=dev, dtype=torch.float32)
+    for tag, lens, start in _SHAPES:
+        b, blocks = K.batch(lens, start)
+        t, n, L, dec = sum(lens), len(lens), lens[0], lens[0] == 1
+        # ---- attention
+        H, G, D, V, rd = 32, 8, 64, 128, 64
+        kp, vp = rnd(blocks, G, 16, 2 * D), rnd(blocks, G, 16, V)
+        cols = 2 * (H + G) * D + G * V
+        p, bias, wn, freq = rnd(t, cols), torch.zeros(cols, **f32), torch.ones(D, **f32), M.rope_frequencies(rd, 5e5, dev)
+        rec("map rows: bias, norms, rotation, cache write", "query / key rows", tag, lambda: M.map_prep(p, bias, H, D, V, wn, wn, freq, kp, vp, b, 1e-6, not dec),
+            t * (cols * 2 + 2 * H * D * 2 + (1 if dec else 2) * G * (2 * D + V) * 2))
+        qk, wq, wk = rnd(t, (H + G) * 128), torch.ones(H * 128, **f32), torch.ones(G * 128, **f32)
+        rec("existing: query / key norm, rotation, cache write", "query / key rows", tag, lambda: M.qk_prep(qk, H, 128, wq, wk, freq, kp, vp, b, 1e-6, not dec),
+            t * ((H + G) * 128 * 2 + (H + (2 if dec else 4) * G) * 128 * 2))
+        del p, qk
+        mix = M.MapMix(torch.full((1,), 0.5, **f32), 0.5, 1e-6, V, D)
+        q2, q1 = rnd(t, 2 * H, D), rnd(t, H, 128)
+        k2, v, k1 = (None,) * 3 if dec else (rnd(t, G, 2 * D), rnd(t, G, V), rnd(t, G, 128))
+        for window in (4096, 512):
+            if dec:
+                rec(f"paged differential attention, window {window}", "paged decode", tag,
+                    lambda: M.map_attention(q2, kp, vp, b.table, None, b.kv_len, 0.125, window, mix, b.max_len), t * min(2048, window) * G * (2 * D + V) * 2)
+                rec(f"existing: paged windowed attention, window {window}", "paged decode", tag,
+                    lambda: M.window_attention(q1, kp, vp, b.table, None, b.kv_len, 0.088, window, 0, b.max_len), t * min(2048, window) * G * 256 * 2)
+            else:
+                pairs = sum(min(i + 1, window) for i in range(L))
+                rec(f"packed differential attention, window {window}", "packed attention", tag,
+                    lambda: M.map_attention_varlen(q2, k2, v, b.cu, b.cu, 0.125, window, mix), t * (2 * H * D + H * V + G * (2 * D + V)) * 2,
+                    n * pairs * H * 2 * (2 * D + 2 * V))
+                rec(f"existing: packed windowed attention, window {window}", "packed attention", tag,
+                    lambda: M.window_attention_varlen(q1, k1, v, b.cu, b.cu, 0.088, window, 0), t * (2 * H + 2 * G) * 128 * 2, n * pairs * H * 4 * 128)
+        if not dec:
+            rec("existing: attention_varlen (GQA 32/8)", "packed attention", tag, lambda: attention_varlen(q1, k1, v, b.cu, L, True, 0.088),
+                t * (2 * H + 2 * G) * 128 * 2, n * L * L / 2 * H * 4 * 128)
+        del kp, vp, q1, q2, k1, k2, v
+        # ---- rows
+        emb, ids, wn = rnd(128256, W), torch.randint(0, 128256, (t,), device=dev), torch.ones(W, **f32)
+        cw, cst = torch.randn(4, W, **f32), torch.zeros(n + 1, 3, W, device=dev, dtype=torch.bfloat16)
+        conv = M.InputConv(cw, cw.clone(), cst)
+        fused = conv if dec else None                           # single-token steps: the block kernels end in the convolutions
+        extra = n * W * (2 + 12) if dec else 0
+        rec("embedding + norm" + (" + convolutions" if dec else ""), "norm + residual add", tag, lambda: M.block_embed(ids, emb, 1, wn, 1e-6, True, fused, b), t * W * 8 + extra)
+        rec("existing: embedding + norm", "norm + residual add", tag, lambda: M.embed(ids, emb, wn, 1e-6), t * W * 8)
+        del emb
+        y1, y2, h = rnd(t, W), rnd(t, W), rnd(t, W)
+        if not dec:
+            rec("two input convolutions", "conv + silu", tag, lambda: M.input_conv(h, conv, b), t * W * 6 + n * 6 * W * 2)
+            rec("existing: conv + silu", "conv + silu", tag, lambda: M.conv_silu(h, cw, None, cst, b), t * W * 4 + n * 6 * W * 2)
+        past = torch.randn(17, t, W, **f32)
+        for i in (0, 5, 15):
+            a = torch.full((i + 2,), 0.1, **f32)
+            rec(f"block results, average over {i + 2}, next norm" + (" + convolutions" if dec else ""), "norm + residual add", tag,
+                lambda: M.block_add(past, i, y1, y2, None, wn, wn, a[1:] if i else None, a, wn, 1e-6, True, fused, b), t * W * (4 * (i + 2) + 6) + extra)
+        del past
+        x32 = torch.randn(t, W, **f32)
+        rec("existing: norm + residual add + next norm", "norm + residual add", tag, lambda: M.norm_add_(y1, x32, wn, 1e-6, wn), t * W * 12)
+        z, act = rnd(t, FF), torch.tensor([0.3, 0.3, 0.3, 0.1], **f32)
+        rec("polynomial activation", "gated norm", tag, lambda: M.poly_norm(z, act, 1e-6), t * FF * 4)
+        z2, gn = rnd(t, FF), torch.ones(FF, **f32)
+        rec("existing: gated norm (gate first)", "gated norm", tag, lambda: M.gated_norm(z, z2, gn, 1, 1e-6, M.SILU_FIRST), t * FF * 6)
+        del z, z2, x32, y2
+        # ---- experts
+        E, top, F = 16, 2, 2048
+        router = rnd(E, W, scale=W ** -0.5)
+        wgu, wd = rnd(E * 2 * F, W, scale=W ** -0.5), rnd(E * W, F, scale=F ** -0.5)
+        logits = M.linear_f32(h, router)
+        ctr = M._counter(dev, E + 1, "route")
+        pick, score, rank, plan = C.mix_route(logits, top, ctr)
+        xr, pos = C.mix_expert_rows(h, pick, score, rank, plan, E)
+        a = C.gemm_experts(xr, wgu, plan, E, True)
+        rec("routing", "norm + residual add", tag, lambda: C.mix_route(logits, top, ctr), t * (E * 4 + top * 12))
+        rec("rows in the experts' order", "norm + residual add", tag, lambda: C.mix_expert_rows(h, pick, score, rank, plan, E), t * W * 2 * (1 + top))
+        rec("experts: gate / up + silu glu", "gate / up + swiglu", tag, lambda: C.gemm_experts(xr, wgu, plan, E, True),
+            (E * 2 * F * W + t * top * (W + F)) * 2, 4.0 * t * top * W * F)
+        rec("experts: down", "down projection", tag, lambda: C.gemm_experts(a, wd, plan, E, False), (E * F * W + t * top * (W + F)) * 2, 2.0 * t * top * W * F)
+        routed = M.Routed(C.gemm_experts(a, wd, plan, E, False), pos)
+        past, a2 = torch.randn(7, t, W, **f32), torch.full((7,), 0.1, **f32)
+        ys = rnd(t, W)
+        rec("block results with routed rows, average over 7" + (" + convolutions" if dec else ""), "norm + residual add", tag,
+            lambda: M.block_add(past, 5, y1, ys, routed, wn, wn, a2[1:], a2, wn, 1e-6, True, fused, b), t * W * (28 + 6 + 2 * top) + extra)
+        del past, xr, a, routed
+        gu, dn, g = rnd(2 * top * F, W, scale=W ** -0.5), rnd(W, top * F, scale=W ** -0.5), rnd(t, top * F)
+        rec("existing: gate / up + swiglu, dense of the active width", "gate / up + swiglu", tag, lambda: ops.linear_swiglu(h, gu),
+            (t * W + 2 * top * F * W + t * top * F) * 2, 4.0 * t * top * W * F)
+        rec("existing: down projection, dense of the active width", "down projection", tag, lambda: ops.linear(g, dn), (t * W + top * F * W + t * top * F) * 2,
+            2.0 * t * top * W * F)
+        del gu, dn, g, wgu, wd, y1, h
+        torch.cuda.empty_cache()
+    return K.rows
+
+
 def run_kernels(args) -> list[dict]:
     from .. import ops
     from ..models import get_model_config, mla
@@ -338,7 +444,7 @@ def main(args) -> int:
         return 1
     args.steps_serving = max(5, args.steps)
     out = {"workload": "serving", "dtype": "bf16", "data": "random weights and tokens", "device": torch.cuda.get_device_name(), "peaks": _peaks()[2]}
-    kernels = {"ludesun": run_kernels, "lanilix": run_kernels_lanilix}[args.serving_design]
+    kernels = {"ludesun": run_kernels, "lanilix": run_kernels_lanilix, "mabedra": run_kernels_mabedra}[args.serving_design]
     out["kernels" if args.kernels else "models"] = kernels(args) if args.kernels else run_models(args)
     if os.environ.get("BENCH_SERVING_OUT"):
         Path(os.environ["BENCH_SERVING_OUT"]).write_text(json.dumps(out, indent=1))

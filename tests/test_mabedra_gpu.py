@@ -230,7 +230,7 @@ def test_routing_with_equal_and_infinite_logits():
 
     z = torch.zeros(40, 37, device=DEV)
     z[1], z[2, 30], z[3, 5], z[4] = float("-inf"), float("inf"), float("nan"), float("nan")
-    pick, score, rank, plan = M._C().mix_route(z, 3, M._counter(z.device, 38))
+    pick, score, rank, plan = M._C().mix_route(z, 3, M._counter(z.device, 38, "route"))
     pick = pick.cpu()
     for t in (0, 1, 3, 4):
         assert pick[t].tolist() == [0, 1, 2]
