@@ -96,8 +96,9 @@ struct AccReader {
   }
 };
 
-// Communication and grouping policy.  `m_blocks` and `b_row` let a grouped product (one weight per group of m-blocks) read its plan
-// from device memory: the number of m-blocks in use, and the first row of B for an m-block.  kCommWarps extra warps per CTA run `Comm::run` (peer-memory copies) while
+// Communication and grouping policy.  `m_blocks`, `b_row` and `rows` let a grouped product (one weight per group of m-blocks) read its
+// plan from device memory: the number of m-blocks in use, the first row of B for an m-block, the rows of the m-block in use.  A is loaded
+// in boxes of kABox rows; with kABox < 128 only the boxes that hold rows in use are (the others' results are never stored).  kCommWarps extra warps per CTA run `Comm::run` (peer-memory copies) while
 // the TMA producer consults `Comm::wait_n_block` before touching the rows of B of an n-block.
 struct NoComm {
   struct Params {};
@@ -108,6 +109,10 @@ struct NoComm {
   __device__ __forceinline__ static int m_blocks(const P&, int launched) { return launched; }
   template <class P>
   __device__ __forceinline__ static int b_row(const P&, int /*m_blk*/, int /*N*/) { return 0; }
+  static constexpr int kABox = kBlockM;
+  static constexpr bool kRagged = false;           // m-blocks may end early
+  template <class P>
+  __device__ __forceinline__ static int rows(const P&, int /*m_blk*/) { return kBlockM; }
 };
 using NoGate = NoComm;
 
@@ -165,14 +170,22 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
       for (int w = blockIdx.x; w < total_work; w += gridDim.x) {
         const WorkInfo wi = decode_work(w, num_m_blocks, num_n_blocks, n_splits, nb_per_split, sc);
         const int b0 = Gate::b_row(gp, wi.m_blk, N);
+        const int boxes = (Gate::rows(gp, wi.m_blk) + Gate::kABox - 1) / Gate::kABox;
         for (int nbs = wi.n_begin; nbs < wi.n_end; ++nbs) {
           const int nb = rot_n(nbs, num_n_blocks, sc);
           Gate::wait_n_block(gp, nb);
           for (int kb = 0; kb < num_kb; ++kb) {
             mbar_wait(&empty_bar[stage], phase ^ 1);
-            mbar_expect_tx(&full_bar[stage], Cfg::STAGE_BYTES);
-            tma_load_2d(&tmA, &full_bar[stage], smem_a + stage * Cfg::A_BYTES, kb * Cfg::BLOCK_K,
-                        wi.m_blk * kBlockM);
+            if constexpr (Gate::kABox == kBlockM) {
+              mbar_expect_tx(&full_bar[stage], Cfg::STAGE_BYTES);
+              tma_load_2d(&tmA, &full_bar[stage], smem_a + stage * Cfg::A_BYTES, kb * Cfg::BLOCK_K,
+                          wi.m_blk * kBlockM);
+            } else {
+              mbar_expect_tx(&full_bar[stage], Cfg::B_BYTES + boxes * Gate::kABox * 128);
+              for (int i = 0; i < boxes; ++i)
+                tma_load_2d(&tmA, &full_bar[stage], smem_a + stage * Cfg::A_BYTES + i * Gate::kABox * 128, kb * Cfg::BLOCK_K,
+                            wi.m_blk * kBlockM + i * Gate::kABox);
+            }
             tma_load_2d(&tmB, &full_bar[stage], smem_b + stage * Cfg::B_BYTES, kb * Cfg::BLOCK_K, b0 + nb * BN);
             if (++stage == kStages) { stage = 0; phase ^= 1; }
           }
@@ -224,18 +237,19 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
     for (int w = blockIdx.x; w < total_work; w += gridDim.x) {
       const WorkInfo wi = decode_work(w, num_m_blocks, num_n_blocks, n_splits, nb_per_split, sc);
       const int row = wi.m_blk * kBlockM + row_in_tile;
-      epi.begin(ep, row, M, wi);
+      const int end = Gate::kRagged ? wi.m_blk * kBlockM + Gate::rows(gp, wi.m_blk) : M;
+      epi.begin(ep, row, end, wi);
       for (int nb = wi.n_begin; nb < wi.n_end; ++nb, ++tile_iter) {
         const uint32_t as = tile_iter & 1;
         const uint32_t aphase = (tile_iter >> 1) & 1;
         mbar_wait(&tmem_full[as], aphase);
         tc_fence_after();
         AccReader acc{tmem_base + as * BN + (static_cast<uint32_t>(quad * 32) << 16)};
-        epi.template tile<BN>(ep, acc, row, M, rot_n(nb, num_n_blocks, sc) * BN, N);
+        epi.template tile<BN>(ep, acc, row, end, rot_n(nb, num_n_blocks, sc) * BN, N);
         tc_fence_before();
         mbar_arrive(&tmem_empty[as]);
       }
-      epi.end(ep, row, M, wi);
+      epi.end(ep, row, end, wi);
     }
   }
 
@@ -305,7 +319,7 @@ int launch_gemm(const void* A, const void* B, int M, int N, int K, int64_t lda_b
   constexpr int EB = IS_FP8 ? 1 : 2;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   CUtensorMap tmA, tmB;
-  if (make_tmap_kmajor(&tmA, A, M, K, lda_bytes, kBlockM, EB)) return -2;
+  if (make_tmap_kmajor(&tmA, A, M, K, lda_bytes, Gate::kABox, EB)) return -2;
   if (make_tmap_kmajor(&tmB, B, static_cast<uint64_t>(N) * groups, K, ldb_bytes, Cfg::BLOCK_N, EB)) return -3;      // N rows per group
   const int num_m_blocks = (M + kBlockM - 1) / kBlockM;
   const int num_n_blocks = (N + Cfg::BLOCK_N - 1) / Cfg::BLOCK_N;

@@ -166,17 +166,29 @@ struct EpiGelu {
   }
 };
 
-// one weight [N, K] per group of 128-row tiles: plan[0] = tiles in use, plan[1 + groups + i] = group of tile i (mix_experts.cu)
+// one weight [N, K] per group of 128-row tiles (mix_experts.cu): plan[0] = tiles in use, plan[1 + groups + i] = group of tile i in the low 16 bits,
+// its rows in use above.  BOX < 128: few rows per tile, only the boxes in use are read
+template <int BOX>
 struct GroupedTiles : NoComm {
   struct Params {
     const int32_t* plan;
     int groups;
   };
+  static constexpr int kABox = BOX;
+  static constexpr bool kRagged = true;
   __device__ __forceinline__ static void wait_n_block(const Params&, int) {}
   __device__ __forceinline__ static void run(const Params&, int) {}
   __device__ __forceinline__ static int m_blocks(const Params& p, int) { return p.plan[0]; }
-  __device__ __forceinline__ static int b_row(const Params& p, int m_blk, int N) { return p.plan[1 + p.groups + m_blk] * N; }
+  __device__ __forceinline__ static int b_row(const Params& p, int m_blk, int N) { return (p.plan[1 + p.groups + m_blk] & 0xffff) * N; }
+  __device__ __forceinline__ static int rows(const Params& p, int m_blk) { return p.plan[1 + p.groups + m_blk] >> 16; }
 };
+
+template <int BN, class Epi, int BOX>
+static int run_grouped(const void* A, const void* W, const typename Epi::Params& sp, const int32_t* plan, int M, int groups, int N, int K,
+                       cudaStream_t stream) {
+  const int64_t ld = 2 * static_cast<int64_t>(K);
+  return launch_gemm<GemmCfg<BN, 2>, Epi, GroupedTiles<BOX>, false>(A, W, M, N, K, ld, ld, sp, {plan, groups}, 0, 0, stream, Sched{0, 1, 0}, false, groups);
+}
 
 template <int BN, bool FP8>
 static int run_store(const void* A, const void* B, const StoreParams& sp, int M, int N, int K, int64_t lda, int64_t ldb,
@@ -275,18 +287,15 @@ extern "C" int prl_gemm_experts_bf16(const void* A, const void* W, void* D, cons
   if (tiles <= 0) return 0;
   if (N <= 0 || K <= 0 || K % 8 || groups < 1 || static_cast<int64_t>(groups) * N > 0x7fffffff) return -12;
   const int M = tiles * kBlockM;
-  const GroupedTiles::Params gp{plan, groups};
+  const bool few = tiles < 4 * groups;              // mostly tiles with a few rows: weights are streamed, the rows in use beside them
   if (glu) {
     if (N % 256) return -11;
     SwigluParams sp{static_cast<__nv_bfloat16*>(D), nullptr, N / 2, 0};
-    return launch_gemm<GemmCfg<256, 2>, EpiSwiglu, GroupedTiles, false>(A, W, M, N, K, 2 * static_cast<int64_t>(K), 2 * static_cast<int64_t>(K), sp, gp, 0, 0,
-                                                                        stream, Sched{0, 1, 0}, false, groups);
+    return few ? run_grouped<256, EpiSwiglu, 32>(A, W, sp, plan, M, groups, N, K, stream)
+               : run_grouped<256, EpiSwiglu, kBlockM>(A, W, sp, plan, M, groups, N, K, stream);
   }
   if (N % 8) return -13;
   StoreParams sp{static_cast<__nv_bfloat16*>(D), nullptr, N, nullptr, nullptr};
-  if (tiles >= 4 * groups && N >= 256)
-    return launch_gemm<GemmCfg<256, 2>, EpiStore, GroupedTiles, false>(A, W, M, N, K, 2 * static_cast<int64_t>(K), 2 * static_cast<int64_t>(K), sp, gp, 0, 0,
-                                                                       stream, Sched{0, 1, 0}, false, groups);
-  return launch_gemm<GemmCfg<128, 2>, EpiStore, GroupedTiles, false>(A, W, M, N, K, 2 * static_cast<int64_t>(K), 2 * static_cast<int64_t>(K), sp, gp, 0, 0, stream,
-                                                                     Sched{0, 1, 0}, false, groups);
+  return few || N < 256 ? run_grouped<128, EpiStore, 32>(A, W, sp, plan, M, groups, N, K, stream)
+                        : run_grouped<256, EpiStore, kBlockM>(A, W, sp, plan, M, groups, N, K, stream);
 }

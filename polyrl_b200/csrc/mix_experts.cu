@@ -1,7 +1,7 @@
 // polyrl_b200 — mixture of experts without host synchronisation: routing, rows in the experts' order, a plain grouped product.
 //
 // The plan of a step is device data: plan[0] = number of 128-row tiles, plan[1 + e] = first row of expert e (a multiple of 128),
-// plan[1 + E + i] = expert of tile i.  Grids are sized for the worst case and leave early, so a decode step can be captured.
+// plan[1 + E + i] = expert of tile i, and above its 16 bits the tile's rows in use.  Grids are sized for the worst case and leave early, so a decode step can be captured.
 // The order of an expert's rows depends on arrival; every row is computed by itself, so results do not.
 #include "mixers.cuh"
 
@@ -68,12 +68,11 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
   }
   if (!last_tile(&counts[E], gridDim.x)) return;
   // the last CTA to arrive has everybody's counts: first rows by a warp scan, then the experts of the tiles
-  __shared__ int s_tiles;
   if (warp == 0) {
     int base = 0;
     for (int e0 = 0; e0 < E; e0 += 32) {
       const int e = e0 + lane;
-      const int tiles = e < E ? (atomicAdd(&counts[e], 0) + kMoeTile - 1) / kMoeTile : 0;
+      const int rows = e < E ? atomicAdd(&counts[e], 0) : 0, tiles = (rows + kMoeTile - 1) / kMoeTile;
       int sum = tiles;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -82,18 +81,17 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
       }
       if (e < E) {
         plan[1 + e] = (base + sum - tiles) * kMoeTile;
-        hist[e] = base + sum - tiles;
+        hist[e] = rows;
         counts[e] = 0;
       }
       base += __shfl_sync(0xffffffffu, sum, 31);
     }
-    if (lane == 0) { s_tiles = base; plan[0] = base; }
+    if (lane == 0) plan[0] = base;
   }
   __syncthreads();
-  const int n = s_tiles;
   for (int e = threadIdx.x; e < E; e += 256) {
-    const int end = e + 1 < E ? hist[e + 1] : n;
-    for (int i = hist[e]; i < end; ++i) plan[1 + E + i] = e;
+    const int first = plan[1 + e] / kMoeTile;
+    for (int r = 0; r < hist[e]; r += kMoeTile) plan[1 + E + first + r / kMoeTile] = e | min(kMoeTile, hist[e] - r) << 16;
   }
 }
 
@@ -127,7 +125,7 @@ __global__ void __launch_bounds__(256) mix_expert_gemm_kernel(const T* __restric
   if (static_cast<int>(blockIdx.y) / 2 >= plan[0]) return;
   const int64_t r0 = static_cast<int64_t>(blockIdx.y) * 64;
   const int n0 = blockIdx.x * 64;
-  const int64_t w0 = static_cast<int64_t>(plan[1 + E + blockIdx.y / 2]) * N;
+  const int64_t w0 = static_cast<int64_t>(plan[1 + E + blockIdx.y / 2] & 0xffff) * N;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
