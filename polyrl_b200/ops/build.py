@@ -2,7 +2,7 @@
 
 Kernel ``.cu`` files are torch-free and compiled directly with ``nvcc -gencode arch=compute_100a,
 code=sm_100a -lineinfo``; only the ``bindings*.cpp`` files see torch headers.  The resulting ``.so`` files live in the
-package directory (git-ignored, but shipped to the GPU box by ``gpurun``), never in a JIT cache.
+package directory (git-ignored; they travel with the tree), never in a JIT cache.
 
 Usage:  python -m polyrl_b200.ops.build [--force] [--verbose]
 """
