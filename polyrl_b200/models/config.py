@@ -101,6 +101,10 @@ class ModelConfig:
     video_token_id: int = -1
     vision_start_token_id: int = -1
     vision_end_token_id: int = -1
+    # mixer stacks: residual streams with hyper-connections (0: one residual), norms whose weight is one number, a factor on the embedding
+    streams: int = 0
+    scalar_norm: bool = False
+    embed_scale: float = 1.0
     # mixer stacks (family "hybrid", models/hybrid.py): one dict per layer, {"kind", "sizes", "ff", "weights_of", ...}
     layers: tuple = ()
 
@@ -393,7 +397,7 @@ def _stack(hf: dict) -> ModelConfig:
 
 
 # designs whose config.json names an ``architecture`` instead of a ``model_type``
-ARCHITECTURES = {"Ludesun": _stack, "Lanilix": _stack, "Mabedra": _stack}
+ARCHITECTURES = {"Ludesun": _stack, "Lanilix": _stack, "Mabedra": _stack, "Dubazen": _stack}
 
 
 def _qwen_dense_layers(hf: dict) -> tuple:
@@ -639,6 +643,24 @@ PRESETS: dict[str, dict] = {
                            dict(kind="diff", weights_of=i, sizes=dict(heads=32, kv_heads=8, dim=64, vdim=128, scale=64 ** -0.5, diff=0.5, window=4096, rot_dim=64,
                                                                       rot_base=500000.0, rot_scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192.0)),
                                 **(dict(ff=14336, act="poly") if i % 4 == 0 else dict(ff=2048, act="moe", experts=16, top=2, shared=4096))) for i in range(16))),
+    # Dubazen stacks: residual streams, attention beside linear attention, gated linear attention and selective scans, all layers sparse
+    "tiny-dubazen": dict(family="hybrid", vocab_size=512, hidden_size=192, intermediate_size=64, num_layers=4, num_heads=1, num_kv_heads=1, rms_norm_eps=1e-5,
+                         eos_token_id=-1, bos_token_id=-1, hf_model_type="dubazen", streams=3, scalar_norm=True, embed_scale=8.0, layers=tuple(
+                             dict(weights_of=i, ff=64, act="moe", router="softmax", experts=8, top=2, shared=96, limit=4.0, shared_limit=5.0, alpha=1.702, kind=k,
+                                  sizes=s) for i, (k, s) in enumerate((
+                                      ("selective", dict(inner=256, state=12, dt_rank=10, conv=4)),
+                                      ("pair", dict(left=dict(kind="turn", heads=6, kv_heads=2, dim=40, vdim=32, scale=40 ** -0.5, rot_dim=20, rot_base=10000.0),
+                                                    right=dict(kind="decay", heads=3, dim=32, vdim=48, decay=[0.7, 0.95, 0.995]), left_scale=0.8, right_scale=1.1)),
+                                      ("gla", dict(heads=4, dim=32, vdim=40, tau=12.0, rank=12)),
+                                      ("selective", dict(inner=256, state=12, dt_rank=10, conv=4)))))),
+    "dubazen-7b": dict(family="hybrid", vocab_size=128256, hidden_size=4096, intermediate_size=2048, num_layers=16, num_heads=1, num_kv_heads=1, rms_norm_eps=1e-6,
+                       eos_token_id=-1, bos_token_id=-1, hf_model_type="dubazen", streams=4, scalar_norm=True, embed_scale=64.0, layers=tuple(
+                           dict(weights_of=i, ff=2048, act="moe", router="softmax", experts=16, top=2, shared=4096, limit=7.0, shared_limit=7.0, alpha=1.702, **(
+                               dict(kind="selective", sizes=dict(inner=8192, state=16, dt_rank=256, conv=4)) if i % 2 == 0 else
+                               dict(kind="pair", sizes=dict(left=dict(kind="turn", heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, rot_dim=64, rot_base=500000.0),
+                                                            right=dict(kind="decay", heads=32, dim=128, vdim=128, decay=[1 - 2.0 ** (-1 - 0.25 * j) for j in range(32)]),
+                                                            left_scale=1.0, right_scale=1.0)) if i % 4 == 1 else
+                               dict(kind="gla", sizes=dict(heads=16, dim=128, vdim=256, tau=16.0, rank=16)))) for i in range(16))),
     "tiny-gpt2": dict(family="gpt2", vocab_size=512, hidden_size=128, intermediate_size=512, num_layers=2,
                       num_heads=4, num_kv_heads=4, max_position_embeddings=256, rms_norm_eps=1e-5,
                       tie_word_embeddings=True, eos_token_id=1, bos_token_id=2, pad_token_id=0),
@@ -656,6 +678,10 @@ def get_model_config(name_or_path: str, **overrides) -> ModelConfig:
         p = p / "config.json"
     if p.exists():
         d = json.loads(p.read_text())
+        if d.get("architecture") in ARCHITECTURES:
+            from .stacks import sizes_from_tensors
+
+            d = sizes_from_tensors(d, p.parent)
         cfg = ModelConfig(**d) if "family" in d else ModelConfig.from_hf_config(d)
         for k, v in overrides.items():
             setattr(cfg, k, v)

@@ -74,6 +74,23 @@ class HFCheckpoint:
         return self._handles[fname].get_tensor(name)
 
 
+def tensor_shape(path: str | Path, name: str) -> tuple[int, ...] | None:
+    """Shape of a checkpoint tensor, or None when the directory has no such tensor (``*.safetensors``: nothing else is read)."""
+    try:
+        ck = HFCheckpoint(path)
+    except FileNotFoundError:
+        return None
+    if name not in ck.weight_map:
+        return None
+    fname = ck.weight_map[name]
+    if fname in ck._bin_cache:
+        return tuple(ck._bin_cache[fname][name].shape)
+    from safetensors import safe_open
+
+    with safe_open(str(ck.dir / fname), framework="pt") as h:
+        return tuple(h.get_slice(name).get_shape())
+
+
 def _layer_keys(cfg: ModelConfig, i: int) -> list[str]:
     if cfg.family == "gpt2":
         p = f"transformer.h.{i}."

@@ -10,6 +10,11 @@ the state slots), element-wise scales on their results (``layer_scale``).  With 
 x = sum_j depth[j] X_j over the embedding output X_0 and the results X_j of the layers so far; they are kept in fp32 for the step's
 tokens, and x itself is never stored: the kernel that adds a layer's results recomputes it from them.
 
+With ``ModelConfig.streams`` the residual is that many streams X_s (hyper-connections), all the embedding output at first, and every
+sublayer q has maps of its own:  u = sum_s in_q[s] X_s,  y = sublayer(norm_q(u)),  X_t <- sum_s mix_q[s, t] X_s + out_q[t] y.  Norms are on
+the inputs; the model's output is the sum of the streams.  ``scalar_norm``: the weight of such a norm is one number.  One kernel ends a
+sublayer and begins the next: it reads and writes the streams once.
+
 Mixers (``LAYER_KINDS``):
   ``ssd``     Mamba-2 state-space duality: causal convolution, scalar-decay recurrence, gate before a grouped norm
   ``mlstm``   xLSTM matrix memory with exponential gates
@@ -19,12 +24,14 @@ Mixers (``LAYER_KINDS``):
               and partly rotated in neighbouring pairs, the values are the keys as projected
   ``diff``    differential attention in a sliding window: two softmax maps per head over the same values, a1 - lambda a2, normed per head;
               projection biases, queries and keys normed per head and map, rotate-half positions with Llama 3.1 frequency scaling
-Feed-forwards (``act``): ``gelu``, ``clamped_glu``, ``poly`` (up, a N(z) + b N(z^2) + c N(z^3) + e with RMS norms N, down) or ``moe`` (silu-gated
-experts, the ``top`` largest sigmoid scores weigh the experts' inputs, plus a shared expert).  A layer may reuse the weights of an earlier one (``weights_of``) while keeping a
-cache or state of its own.
+  and those of ``mixer_kinds.py``
+Feed-forwards (``act``): ``gelu``, ``clamped_glu``, ``poly`` (up, a N(z) + b N(z^2) + c N(z^3) + e with RMS norms N, down) or ``moe`` (gated
+experts and a shared one; ``router``: ``sigmoid_in``, the ``top`` largest sigmoid scores weigh the experts' inputs, or ``softmax``, the ``top`` largest
+softmax scores over their sum weigh the outputs; with ``limit`` and ``alpha`` the experts are clamped, ``shared_limit`` being the shared one's).  A layer
+may reuse the weights of an earlier one (``weights_of``) while keeping a cache or state of its own.
 
 ``ModelConfig.layers`` holds one plain dict per layer: {"kind", "sizes", "ff" (0: no feed-forward), "weights_of" (own index when the
-layer owns its weights)} and what its feed-forward needs ("act", "limit", "alpha", "experts", "top", "shared").  ``stacks.py`` reads the designs' config.json and
+layer owns its weights)} and what its feed-forward needs ("act", "limit", "alpha", "experts", "top", "shared", "router", "shared_limit").  ``stacks.py`` reads the designs' config.json and
 checkpoint names; another design built from the same mixers needs only another reader and name map.
 
 Everything is one function of a packed step (ops/mixers.py ``SpanBatch``): prompts, portions of prompts and decoded tokens take the
@@ -39,10 +46,13 @@ from .. import ops
 from ..ops import mixers as M
 from ..ops import reference as ref
 from .config import ModelConfig
+from .mixer_kinds import KINDS
 
-LAYER_KINDS = ("ssd", "mlstm", "delta", "latent", "window", "diff")
+LAYER_KINDS = ("ssd", "mlstm", "delta", "latent", "window", "diff", *KINDS)
 MAPS = 2                            # softmax maps of a differential attention head
 MAX_EXPERTS = 1024
+MAX_STREAMS = 16
+ROUTERS = ("sigmoid_in", "softmax")
 
 
 def _pad8(n: int) -> int:
@@ -67,6 +77,10 @@ def validate(cfg: ModelConfig) -> None:
         raise ValueError("parallel blocks have one norm, on the input")
     if not cfg.parallel_block and (cfg.layer_norm or cfg.input_conv or cfg.layer_scale or cfg.depth_average):
         raise ValueError("layer norms, input convolutions, layer scales and depth averages need parallel blocks")
+    if cfg.streams and (not 1 <= cfg.streams <= MAX_STREAMS or cfg.parallel_block or cfg.sandwich_norm):
+        raise ValueError(f"residual streams: 1 to {MAX_STREAMS}, and norms on the sublayers' inputs only")
+    if cfg.scalar_norm and not cfg.streams:
+        raise ValueError("norms with one number as their weight need residual streams")
     for i, lay in enumerate(cfg.layers):
         kind, m = lay["kind"], lay["sizes"]
         if kind not in LAYER_KINDS:
@@ -76,6 +90,8 @@ def validate(cfg: ModelConfig) -> None:
         j = owner(cfg, i)
         if {k: v for k, v in cfg.layers[j].items() if k != "weights_of"} != {k: v for k, v in lay.items() if k != "weights_of"}:
             raise ValueError(f"layer {i} differs from layer {j} whose weights it uses")
+        if kind in KINDS and not KINDS[kind].fits(m):
+            raise ValueError(f"layer {i}: {kind} sizes")
         if kind == "ssd" and (m["heads"] % m["groups"] or (m["heads"] * m["vdim"]) % m["norm_groups"] or m["conv"] < 1 or m["state"] > 512):
             raise ValueError(f"layer {i}: ssd sizes")
         if kind == "mlstm" and (m["dim"] > 512 or m["gate_cap"] <= 0):
@@ -96,8 +112,9 @@ def validate(cfg: ModelConfig) -> None:
             raise ValueError(f"layer {i}: diff sizes")
         if lay["ff"] and lay.get("act", "gelu") not in ("gelu", "clamped_glu", "poly", "moe"):
             raise ValueError(f"layer {i}: unknown feed-forward {lay['act']!r}")
-        if lay["ff"] and lay.get("act") == "moe" and not (1 <= lay["top"] <= lay["experts"] <= MAX_EXPERTS and lay["shared"] >= 0 and cfg.parallel_block):
-            raise ValueError(f"layer {i}: experts (parallel blocks only)")
+        if lay["ff"] and lay.get("act") == "moe" and not (1 <= lay["top"] <= lay["experts"] <= MAX_EXPERTS and lay["shared"] >= 0
+                                                              and (cfg.parallel_block or cfg.streams) and lay.get("router", ROUTERS[0]) in ROUTERS):
+            raise ValueError(f"layer {i}: experts (parallel blocks and residual streams only)")
 
 
 # --------------------------------------------------------------------------------------------
@@ -105,16 +122,22 @@ def validate(cfg: ModelConfig) -> None:
 # --------------------------------------------------------------------------------------------
 def layer_param_specs(cfg: ModelConfig, i: int) -> list[tuple[str, tuple[int, ...]]]:
     lay, w = cfg.layers[i], cfg.hidden_size
-    m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
+    m, h, v = lay["sizes"], lay["sizes"].get("heads"), lay["sizes"].get("vdim")
     out: list[tuple[str, tuple[int, ...]]]
-    if cfg.parallel_block:
+    if cfg.streams:
+        out, n = [], cfg.streams
+        for q in ("1", "2") if lay["ff"] else ("1",):
+            out += [("pre" + q, () if cfg.scalar_norm else (w,)), (f"hc{q}.in", (n,)), (f"hc{q}.out", (n,)), (f"hc{q}.mix", (n, n))]
+    elif cfg.parallel_block:
         out = [("pre1", (w,))]
         for n in ("1", "2") if lay["ff"] else ("1",):
             out += ([("ls" + n, (w,))] if cfg.layer_scale else []) + ([("conv" + n, (w, cfg.input_conv))] if cfg.input_conv else [])
         out += [("depth", (i + 2,))] if cfg.depth_average else []
     else:
         out = ([("pre1", (w,))] if cfg.sandwich_norm else []) + [("norm1", (w,))]
-    if lay["kind"] == "ssd":            # one projection [gate | x | B | C]; the step sizes keep their own fp32-accumulated one
+    if lay["kind"] in KINDS:
+        out += KINDS[lay["kind"]].specs(m, w)
+    elif lay["kind"] == "ssd":          # one projection [gate | x | B | C]; the step sizes keep their own fp32-accumulated one
         ch = h * v + 2 * m["groups"] * m["state"]
         out += [("w_in", (h * v + ch, w)), ("w_dt", (h, w)), ("conv_w", (ch, m["conv"])), ("conv_b", (ch,)), ("dt_bias", (h,)), ("a_log", (h,)),
                 ("d_skip", (h,)), ("gn", (h * v,)), ("wo", (w, h * v))]
@@ -136,7 +159,7 @@ def layer_param_specs(cfg: ModelConfig, i: int) -> list[tuple[str, tuple[int, ..
                 ("sink", (h,)), ("wo", (w, h * v))]
     if lay["ff"]:
         f, act = lay["ff"], lay.get("act", "gelu")
-        if not cfg.parallel_block:
+        if not cfg.parallel_block and not cfg.streams:
             out += ([("pre2", (w,))] if cfg.sandwich_norm else []) + [("norm2", (w,))]
         # gate and up rows: interleaved in blocks of 128 (as the llama family's) where ff allows it, else one after the other
         if act == "moe":                # experts one after the other
@@ -157,7 +180,7 @@ def gate_up_stacks(lay: dict) -> list[tuple[str, int, int]]:
 
 
 def num_params(cfg: ModelConfig) -> int:
-    n = 2 * cfg.vocab_size * cfg.hidden_size + cfg.hidden_size
+    n = 2 * cfg.vocab_size * cfg.hidden_size + (1 if cfg.scalar_norm else cfg.hidden_size)
     for i in range(cfg.num_layers):
         if owner(cfg, i) == i:
             for _, shp in layer_param_specs(cfg, i):
@@ -173,9 +196,13 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
     base = name.split(".")[-1]
     if base in ("pre1", "norm1", "pre2", "norm2", "norm_w"):
         t.fill_(1.0 - cfg.norm_offset)
+    elif base in ("in", "out"):     # streams: read their mean, write to all of them
+        t.fill_(1.0 if base == "out" else 1.0 / cfg.streams)
+    elif base == "mix":
+        t.copy_(torch.eye(cfg.streams))
     elif base in ("gn", "q_ln", "kv_ln", "q_norm", "k_norm", "d_skip", "ls1", "ls2"):
         t.fill_(1.0)
-    elif base in ("conv_b", "sink", "b_qkv", "map_mix"):
+    elif base in ("conv_b", "sink", "b_qkv", "map_mix", "b_o"):
         t.zero_()
     elif base == "depth":           # the layer's own result
         t.zero_()
@@ -184,6 +211,10 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
         t.copy_(torch.tensor([1 / 3, 1 / 3, 1 / 3, 0.0]))
     elif base in ("conv1", "conv2"):
         t.normal_(0.0, 0.1 * t.shape[1] ** -0.5, generator=generator)
+    elif base == "b_a":             # slow decays
+        t.fill_(3.0)
+    elif base == "a_log" and t.dim() == 2:
+        t.copy_(torch.log(torch.arange(1, t.shape[1] + 1, device=t.device, dtype=torch.float32)).expand(t.shape))
     elif base == "a_log":
         t.copy_(torch.linspace(-2.0, 1.0, t.numel(), device=t.device))
     elif base == "dt_bias":
@@ -194,7 +225,7 @@ def init_param_(name: str, t: torch.Tensor, cfg: ModelConfig, generator=None) ->
     elif base == "conv_w":
         t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
     elif base in ("w_in", "w_dt", "w_if", "wa", "wq_up", "wk_up", "wv_up", "wo", "wup", "wdown", "w_ab", "wqk", "wgu", "wqkv", "router", "ewgu", "ewd",
-                  "swgu", "swd"):
+                  "swgu", "swd", "w_a", "w_x"):
         t.normal_(0.0, t.shape[1] ** -0.5, generator=generator)
     else:
         return False
@@ -248,13 +279,20 @@ def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: di
     """Weights of layer ``i`` in run-time form: vectors in fp32, matrices in ``dtype`` with the layouts the kernels want.  ``old`` (the
     previous result) is overwritten in place where shapes agree, so captured graphs stay valid across weight updates."""
     lay = cfg.layers[i]
-    m, h = lay["sizes"], lay["sizes"]["heads"]
-    device = w["wo"].device
+    m, h = lay["sizes"], lay["sizes"].get("heads")
+    own = {} if lay["kind"] not in KINDS else {n for n, _ in KINDS[lay["kind"]].specs(m, cfg.hidden_size)}
+    device = next(iter(w.values())).device
     is_cuda = device.type == "cuda"
     out: dict[str, torch.Tensor] = {}
+    if own:
+        out.update(KINDS[lay["kind"]].prepare(m, w, dtype, is_cuda))
     for k, t in w.items():
-        if k in _STREAM_NORMS:
-            out[k] = (t.float() + cfg.norm_offset).contiguous() if cfg.norm_offset else t.float().contiguous()
+        if k in own:
+            continue
+        if k.startswith("hc"):
+            out[k] = t.float().contiguous()
+        elif k in _STREAM_NORMS:
+            out[k] = (t.float() + cfg.norm_offset).reshape(-1).contiguous() if cfg.norm_offset else t.float().reshape(-1).contiguous()
         elif k == "gn" and t.numel() < h * m["vdim"]:             # one weight for all heads
             out[k] = t.float().repeat(h)
         elif k in _VECTORS:
@@ -297,7 +335,7 @@ def prepare_layer(cfg: ModelConfig, i: int, w: dict, dtype: torch.dtype, old: di
     if old is not None:
         for k, t in out.items():
             o = old.get(k)
-            derived = k not in w or t.data_ptr() != w[k].data_ptr()
+            derived = k not in w or t.data_ptr() != w[k].data_ptr() or t.shape != w[k].shape
             if derived and o is not None and o.shape == t.shape and o.dtype == t.dtype:
                 out[k] = o.copy_(t)
     return out
@@ -313,7 +351,7 @@ def prepare(cfg: ModelConfig, layer_w: list[dict], dtype: torch.dtype, old: list
 
 
 def prepare_head(cfg: ModelConfig, head_w: dict, dtype: torch.dtype, old: dict | None = None) -> dict:
-    norm = head_w["norm_w"].float().contiguous()
+    norm = head_w["norm_w"].float().expand(cfg.hidden_size).contiguous()
     if cfg.norm_offset:
         norm = norm + cfg.norm_offset
     if old is not None and norm.data_ptr() != head_w["norm_w"].data_ptr():
@@ -329,8 +367,11 @@ def cache_bytes(cfg: ModelConfig, dtype: torch.dtype) -> tuple[int, int]:
     es = torch.empty(0, dtype=dtype).element_size()
     tok = slot = 0
     for lay in cfg.layers:
-        m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
-        if lay["kind"] == "latent":
+        m, h, v = lay["sizes"], lay["sizes"].get("heads"), lay["sizes"].get("vdim")
+        if lay["kind"] in KINDS:
+            for s in KINDS[lay["kind"]].slabs(m, dtype).values():
+                tok, slot = (tok + s.bytes(es), slot) if s.paged else (tok, slot + s.bytes(es))
+        elif lay["kind"] == "latent":
             tok += (m["kv_rank"] + m["rot_dim"]) * es
         elif lay["kind"] == "window":
             tok += 2 * m["kv_heads"] * cache_width(m, dtype) * es
@@ -349,8 +390,9 @@ def cache_bytes(cfg: ModelConfig, dtype: torch.dtype) -> tuple[int, int]:
 
 def key_views(cfg: ModelConfig) -> list[tuple[int, int]]:
     """The distinct (window, kept first tokens) of the stack's attention layers; (0, 0) sees every key."""
-    return sorted({(lay["sizes"].get("window", 0), lay["sizes"].get("keep_first", 0)) for lay in cfg.layers
-                   if lay["kind"] in ("latent", "window", "diff")})
+    own = {v for lay in cfg.layers if lay["kind"] in KINDS for v in KINDS[lay["kind"]].key_views}
+    return sorted(own | {(lay["sizes"].get("window", 0), lay["sizes"].get("keep_first", 0)) for lay in cfg.layers
+                         if lay["kind"] in ("latent", "window", "diff")})
 
 
 def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device, dtype: torch.dtype) -> dict[str, torch.Tensor]:
@@ -363,7 +405,9 @@ def make_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device
 
 def _mixer_cache(cfg: ModelConfig, i: int, num_blocks: int, num_slots: int, device, dtype: torch.dtype) -> dict[str, torch.Tensor]:
     lay = cfg.layers[i]
-    m, h, v = lay["sizes"], lay["sizes"]["heads"], lay["sizes"]["vdim"]
+    m, h, v = lay["sizes"], lay["sizes"].get("heads"), lay["sizes"].get("vdim")
+    if lay["kind"] in KINDS:
+        return {n: s.make(num_blocks, num_slots, device, dtype) for n, s in KINDS[lay["kind"]].slabs(m, dtype).items()}
     if lay["kind"] == "latent":
         return {"pool": torch.zeros(num_blocks, 1, M.PAGE, m["kv_rank"] + m["rot_dim"], device=device, dtype=dtype)}
     if lay["kind"] == "window":
@@ -501,13 +545,21 @@ def _diff(cfg: ModelConfig, m: dict, w: dict, h: torch.Tensor, cache: dict, b: M
 _MIXERS = {"ssd": _ssd, "mlstm": _mlstm, "delta": _delta, "latent": _latent, "window": _window, "diff": _diff}
 
 
+def _mixer(cfg: ModelConfig, lay: dict, w: dict, h: torch.Tensor, cache: dict, b: M.SpanBatch, bias: bool = True) -> torch.Tensor:
+    """The mixer with its output product; ``bias=False``: an output bias (``b_o``) is left to the caller."""
+    kind = lay["kind"]
+    o = KINDS[kind].run(lay["sizes"], cfg.rms_norm_eps, w, h, cache, b) if kind in KINDS else _MIXERS[kind](cfg, lay["sizes"], w, h, cache, b)
+    y = ops.linear(o, w["wo"])
+    return y + w["b_o"].to(y.dtype) if bias and "b_o" in w else y
+
+
 def layer_step(cfg: ModelConfig, i: int, w: dict, x: torch.Tensor, h: torch.Tensor, cache: dict, b: M.SpanBatch,
                w_next: torch.Tensor | None = None) -> torch.Tensor:
     """Layer ``i`` on one packed step.  x: fp32 residual stream, updated in place; h: what its mixer reads, in the activation dtype (x
     itself, or its norm ``pre1``).  Returns x in that dtype — or the norm of x with the weight ``w_next``, which is the next layer's
     ``pre1`` or the model's final norm."""
     lay, eps = cfg.layers[i], cfg.rms_norm_eps
-    y = ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h, cache, b), w["wo"])
+    y = _mixer(cfg, lay, w, h, cache, b)
     if not lay["ff"]:
         return M.norm_add_(y, x, w["norm1"], eps, w_next)
     h = M.norm_add_(y, x, w["norm1"], eps, w.get("pre2"))
@@ -515,12 +567,20 @@ def layer_step(cfg: ModelConfig, i: int, w: dict, x: torch.Tensor, h: torch.Tens
     return M.norm_add_(ops.linear(a, w["wdown"]), x, w["norm2"], eps, w_next)
 
 
-def _feed_forward(cfg: ModelConfig, lay: dict, w: dict, h: torch.Tensor) -> tuple[torch.Tensor | None, M.Routed | None]:
-    """(rows, routed rows that are still to be gathered) of a parallel block's feed-forward."""
+def _feed_forward(cfg: ModelConfig, lay: dict, w: dict, h: torch.Tensor, beside: M.SpanBatch | None = None) -> tuple[torch.Tensor | None, M.Routed | None]:
+    """(rows, routed rows that are still to be gathered) of a feed-forward.  With ``beside`` the shared expert of a step of single tokens runs next to
+    the routed ones."""
     act = lay.get("act", "gelu")
     if act == "moe":
-        y = ops.linear(M.linear_silu_glu(h, w["swgu"]), w["swd"]) if "swgu" in w else None
-        return y, M.experts(h, w["router"], w["ewgu"], w["ewd"], lay["top"])
+        glu = (float(lay["limit"]), float(lay["alpha"])) if "limit" in lay else None
+        y = None
+        with M.beside(h, beside) as side:
+            if "swgu" in w:
+                with side():
+                    a = M.linear_silu_glu(h, w["swgu"]) if glu is None else M.linear_clamped_glu(h, w["swgu"], float(lay["shared_limit"]), glu[1])
+                    y = ops.linear(a, w["swd"])
+            routed = M.experts(h, w["router"], w["ewgu"], w["ewd"], lay["top"], glu, lay.get("router", ROUTERS[0]) == "softmax")
+        return y, routed
     if act == "poly":
         a = M.poly_norm(ops.linear(h, w["wup"]), w["act"], cfg.rms_norm_eps)
     else:
@@ -532,35 +592,20 @@ def _conv_of(cfg: ModelConfig, w: dict, cache: dict) -> M.InputConv | None:
     return M.InputConv(w["conv1"], w.get("conv2"), cache["input"]) if cfg.input_conv else None
 
 
-_SIDE: dict = {}
-
-
-def _side_stream(device: torch.device):
-    key = device.index
-    if key not in _SIDE:
-        _SIDE[key] = torch.cuda.Stream(device=device)
-    return _SIDE[key]
-
-
 def _sublayers(cfg: ModelConfig, i: int, w: dict, h: tuple, cache: dict, b: M.SpanBatch) -> tuple:
     """(mixer rows, feed-forward rows, routed rows).  In single-token steps the two sublayers run on streams of their own: each is a chain of
-    kernels that leave most of the GPU idle.  What the side stream allocates is reused only by its own later work, which waits for the
-    kernel that consumed it; what it reads stays referenced until it has been waited for."""
+    kernels that leave most of the GPU idle."""
     lay = cfg.layers[i]
 
     def mixer():
-        return ops.linear(_MIXERS[lay["kind"]](cfg, lay["sizes"], w, h[0], cache, b), w["wo"])
+        return _mixer(cfg, lay, w, h[0], cache, b)
 
     if not lay["ff"]:
         return mixer(), None, None
-    if not h[1].is_cuda or b.seq_of is not None:
-        return (mixer(), *_feed_forward(cfg, lay, w, h[1]))
-    main, side = torch.cuda.current_stream(h[1].device), _side_stream(h[1].device)
-    side.wait_stream(main)
-    with torch.cuda.stream(side):
-        y2, routed = _feed_forward(cfg, lay, w, h[1])
-    y1 = mixer()
-    main.wait_stream(side)
+    with M.beside(h[0], b) as side:
+        with side():
+            y2, routed = _feed_forward(cfg, lay, w, h[1])
+        y1 = mixer()
     return y1, y2, routed
 
 
@@ -579,12 +624,30 @@ def _forward_parallel(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids:
     return x, h[0]
 
 
+def _forward_streams(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids: torch.Tensor, caches: list[dict], b: M.SpanBatch,
+                     final_norm: torch.Tensor | None) -> tuple[torch.Tensor, torch.Tensor]:
+    eps = cfg.rms_norm_eps
+    subs = [(i, q) for i, lay in enumerate(cfg.layers) for q in ("1", "2") if q == "1" or lay["ff"]]
+    x, h = M.streams_embed(ids, embed_w["embed"], cfg.embed_scale, cfg.streams, layer_w[0]["hc1.in"], layer_w[0]["pre1"], eps)
+    for n, (i, q) in enumerate(subs):
+        lay, w = cfg.layers[i], layer_w[i]
+        y, routed = (_mixer(cfg, lay, w, h, caches[i], b, bias=False), None) if q == "1" else _feed_forward(cfg, lay, w, h, b)
+        bias = w.get("b_o") if q == "1" else None
+        hc = (w[f"hc{q}.mix"], w[f"hc{q}.out"])
+        if n + 1 == len(subs):
+            return M.streams_sum(x, y, bias, routed, *hc, final_norm, eps)
+        j, r = subs[n + 1]
+        x, h = M.streams_add(x, y, bias, routed, *hc, layer_w[j][f"hc{r}.in"], layer_w[j]["pre" + r], eps)
+
+
 def forward(cfg: ModelConfig, embed_w: dict, layer_w: list[dict], ids: torch.Tensor, caches: list[dict], b: M.SpanBatch,
             final_norm: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """The stack on one packed step: (fp32 residual stream after the last layer, the same in the activation dtype — normed with
     ``final_norm`` when that is given)."""
     if cfg.parallel_block:
         return _forward_parallel(cfg, embed_w, layer_w, ids, caches, b, final_norm)
+    if cfg.streams:
+        return _forward_streams(cfg, embed_w, layer_w, ids, caches, b, final_norm)
     x, h = M.embed(ids, embed_w["embed"], layer_w[0].get("pre1"), cfg.rms_norm_eps)
     for i, w in enumerate(layer_w):
         h = layer_step(cfg, i, w, x, h, caches[i], b, layer_w[i + 1].get("pre1") if i + 1 < len(layer_w) else final_norm)

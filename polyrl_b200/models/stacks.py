@@ -25,6 +25,15 @@ class Design:
     mlp_kinds: tuple = ("dense",)       # feed-forward kinds of config.json
     read_model: Callable = lambda hf: {}            # config.json -> further ModelConfig fields of the design
     write_model: Callable = lambda cfg: {}          # and back: further entries of config.json
+    complete: Callable = lambda e, i, shape: e      # (entry of layers, index, name -> shape or None): sizes that only a tensor's shape tells
+
+
+def sizes_from_tensors(hf: dict, folder) -> dict:
+    """config.json with the sizes filled in that stand in no other place than the shapes of the folder's tensors."""
+    from .hf_io import tensor_shape
+
+    design = DESIGNS[hf["architecture"].lower()]
+    return dict(hf, layers=[design.complete(e, i, lambda name: tensor_shape(folder, name)) for i, e in enumerate(hf["layers"])])
 
 
 def stack_config(design: Design, hf: dict) -> ModelConfig:
@@ -197,6 +206,18 @@ def _lanilix_parts(cfg: ModelConfig, i: int) -> list:
 
 
 # --------------------------------------------------------------------------------------------
+# experts
+# --------------------------------------------------------------------------------------------
+def _expert_parts(cfg: ModelConfig, lay: dict) -> list:
+    n, f = lay["experts"], lay["ff"]
+    out = [("ewgu", [f"mlp.e{j}.{k}" for j in range(n) for k in ("gate", "up")], [f] * (2 * n)),
+           ("ewd", [f"mlp.e{j}.down" for j in range(n)], [cfg.hidden_size] * n), _one("router", "mlp.router")]
+    if lay["shared"]:
+        out += [("swgu", ["mlp.shared.gate", "mlp.shared.up"], [lay["shared"]] * 2), _one("swd", "mlp.shared.down")]
+    return out
+
+
+# --------------------------------------------------------------------------------------------
 # Mabedra: differential attention in a sliding window; parallel blocks behind layer norms, with input convolutions, layer scales and
 # averages over depth; dense layers with a polynomial activation, sparse ones with a sigmoid router and a shared expert
 # --------------------------------------------------------------------------------------------
@@ -247,12 +268,81 @@ def _mabedra_parts(cfg: ModelConfig, i: int) -> list:
     out += [_one("ls2", "ls2"), _one("conv2", "canon2")]
     if lay["act"] == "poly":
         return out + [_one("wup", "mlp.up"), _one("wdown", "mlp.down"), _one("act", "mlp.act")]
-    n = lay["experts"]
-    out += [("ewgu", [f"mlp.e{j}.{k}" for j in range(n) for k in ("gate", "up")], [f] * (2 * n)),
-            ("ewd", [f"mlp.e{j}.down" for j in range(n)], [cfg.hidden_size] * n), _one("router", "mlp.router")]
-    if lay["shared"]:
-        out += [("swgu", ["mlp.shared.gate", "mlp.shared.up"], [lay["shared"]] * 2), _one("swd", "mlp.shared.down")]
+    return out + _expert_parts(cfg, lay)
+
+
+# --------------------------------------------------------------------------------------------
+# Dubazen: residual streams with hyper-connections; attention with rotated values beside linear attention with constant decays, gated linear
+# attention, selective scans; clamped experts behind a softmax router.  The rank of a gla layer's decay is told by its tensors only.
+# --------------------------------------------------------------------------------------------
+_DUBAZEN_SIZES = {"selective": ("inner", "state", "dt_rank", "conv"), "gla": ("heads", "dim", "vdim", "tau"), "turn": ("heads", "kv_heads", "dim", "vdim", "scale"),
+                  "decay": ("heads", "dim", "vdim")}
+_DUBAZEN_GLU_ALPHA = 1.702
+
+
+def _dubazen_complete(e: dict, i: int, shape: Callable) -> dict:
+    if e["type"] != "gla" or "rank" in e["mixer"]:
+        return e
+    found = shape(f"l{i}.mix.a1")
+    return e if found is None else dict(e, mixer=dict(e["mixer"], rank=found[0]))
+
+
+def _dubazen_read(e: dict, kind: str, i: int) -> dict:
+    m, mlp = e["mixer"], e.get("mlp")
+    if kind == "pair":
+        a, r = m["left"], m["right"]
+        sizes = {"left": {"kind": "turn", **{k: a[k] for k in _DUBAZEN_SIZES["turn"]}, "rot_dim": int(a["rot"]["dims"]), "rot_base": float(a["rot"]["base"])},
+                 "right": {"kind": "decay", **{k: r[k] for k in _DUBAZEN_SIZES["decay"]}, "decay": [float(x) for x in r["decay"]]},
+                 "left_scale": float(m["left_scale"]), "right_scale": float(m["right_scale"])}
+    else:
+        sizes = {k: m[k] for k in _DUBAZEN_SIZES[kind]}
+        if kind == "gla":
+            if "rank" not in m:
+                raise ValueError(f"Dubazen layer {i}: the rank of the decay is told by the model's tensors (or by mixer.rank)")
+            sizes["rank"] = int(m["rank"])
+    out = {"sizes": sizes}
+    if mlp:
+        shared = mlp.get("shared")
+        out.update(act="moe", router="softmax", ff=int(mlp["expert"]["ff"]), experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]),
+                   shared=int(shared["ff"]) if shared else 0, limit=float(mlp["expert"]["limit"]), shared_limit=float(shared["limit"]) if shared else 0.0,
+                   alpha=_DUBAZEN_GLU_ALPHA)
     return out
+
+
+def _dubazen_write(lay: dict) -> dict:
+    s, mlp = lay["sizes"], None
+    if lay["kind"] == "pair":
+        a, r = s["left"], s["right"]
+        mx = {"left": {**{k: a[k] for k in _DUBAZEN_SIZES["turn"]}, "rot": {"dims": a["rot_dim"], "base": a["rot_base"]}},
+              "right": {**{k: r[k] for k in _DUBAZEN_SIZES["decay"]}, "decay": list(r["decay"])}, "left_scale": s["left_scale"], "right_scale": s["right_scale"]}
+    else:
+        mx = {k: s[k] for k in _DUBAZEN_SIZES[lay["kind"]]}
+    if lay["ff"]:
+        mlp = {"kind": "moe", "expert": {"ff": lay["ff"], "limit": lay["limit"]}, "router": {"experts": lay["experts"], "top": lay["top"]}}
+        if lay["shared"]:
+            mlp["shared"] = {"ff": lay["shared"], "limit": lay["shared_limit"]}
+    return {"mixer": mx, "mlp": mlp}
+
+
+def _dubazen_parts(cfg: ModelConfig, i: int) -> list:
+    lay = cfg.layers[i]
+    m, kind = lay["sizes"], lay["kind"]
+    if kind == "pair":
+        a, r = m["left"], m["right"]
+        rows = [a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"]]
+        out = [("left.w_in", [f"mix.left.{n}" for n in "qkvg"], rows + [a["heads"] * a["vdim"]]), ("left.b_qkv", [f"mix.left.{n}.b" for n in "qkv"], rows),
+               _one("left.sink", "mix.left.sink"), _one("left.wo", "mix.left.o"), _one("left.b_o", "mix.left.o.b"),
+               ("right.w_in", [f"mix.right.{n}" for n in "qkvg"], [r["heads"] * r["dim"]] * 2 + [r["heads"] * r["vdim"]] * 2), _one("right.gn", "mix.right.norm"),
+               _one("right.wo", "mix.right.o")]
+    elif kind == "gla":
+        out = [("w_in", ["mix.q", "mix.k", "mix.v", "mix.g", "mix.a1"], [m["heads"] * m["dim"]] * 2 + [m["heads"] * m["vdim"]] * 2 + [m["rank"]]),
+               _one("w_a", "mix.a2"), _one("b_a", "mix.a2.b"), _one("gn", "mix.norm"), _one("wo", "mix.o")]
+    else:
+        out = [_one("w_in", "mix.in"), _one("conv_w", "mix.conv"), _one("conv_b", "mix.conv.b"), _one("w_x", "mix.x"), _one("w_dt", "mix.dt"),
+               _one("dt_bias", "mix.dt.b"), _one("a_log", "mix.A_log"), _one("d_skip", "mix.D"), _one("wo", "mix.o")]
+    for q in ("1", "2") if lay["ff"] else ("1",):
+        out += [_one("pre" + q, "norm" + q)] + [_one(f"hc{q}.{n}", f"hc{q}.{n}") for n in ("in", "out", "mix")]
+    return out + (_expert_parts(cfg, lay) if lay["ff"] else [])
 
 
 DESIGNS = {
@@ -263,4 +353,7 @@ DESIGNS = {
                       read_model=lambda hf: {"parallel_block": True, "layer_norm": True, "layer_scale": True, "depth_average": True,
                                              "input_conv": int(hf["canon"]["taps"])},
                       write_model=lambda cfg: {"canon": {"taps": cfg.input_conv}}),
+    "dubazen": Design("Dubazen", {"parallel": "pair", "gla": "gla", "mamba1": "selective"}, _dubazen_read, _dubazen_write, _dubazen_parts, mlp_kinds=("moe",),
+                      read_model=lambda hf: {"streams": int(hf["streams"]), "scalar_norm": True, "embed_scale": float(hf["embedding"]["scale"])},
+                      write_model=lambda cfg: {"streams": cfg.streams, "embedding": {"scale": cfg.embed_scale}}, complete=_dubazen_complete),
 }

@@ -83,7 +83,7 @@ def embed_param_specs(cfg: ModelConfig) -> ParamSpec:
 
 def head_param_specs(cfg: ModelConfig) -> ParamSpec:
     h = cfg.hidden_size
-    specs: ParamSpec = [("norm_w", (h,))]
+    specs: ParamSpec = [("norm_w", () if cfg.scalar_norm else (h,))]
     if cfg.family == "gpt2":
         specs.append(("norm_b", (h,)))
     if cfg.value_head:

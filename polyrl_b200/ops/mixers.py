@@ -8,6 +8,7 @@ Spans are ordered: the ``n_long`` spans of several tokens first, then the single
 from __future__ import annotations
 
 import math
+from contextlib import contextmanager, nullcontext
 from dataclasses import dataclass
 
 import torch
@@ -72,6 +73,27 @@ def check_errors(device: torch.device) -> None:
         raise RuntimeError("a wait inside a chunked recurrence kernel timed out")
 
 
+_SIDE: dict = {}
+
+
+@contextmanager
+def beside(like: torch.Tensor, b: SpanBatch | None):
+    """Two chains of small kernels next to each other in steps of single tokens:  ``with beside(x, b) as side: with side(): first()``; ``second()``.
+    Elsewhere they run one after the other.  What the side stream allocates is reused only by its own later work, which waits for the kernel
+    that consumed it; what it reads has to stay referenced until the outer block ends."""
+    if b is None or not like.is_cuda or b.seq_of is not None:
+        yield nullcontext
+        return
+    main = torch.cuda.current_stream(like.device)
+    depth = next((d for (i, d), s in _SIDE.items() if i == like.device.index and s == main), 0) + 1
+    if (like.device.index, depth) not in _SIDE:
+        _SIDE[like.device.index, depth] = torch.cuda.Stream(device=like.device)
+    other = _SIDE[like.device.index, depth]
+    other.wait_stream(main)
+    yield lambda: torch.cuda.stream(other)
+    main.wait_stream(other)
+
+
 # --------------------------------------------------------------------------------------------
 # rows
 # --------------------------------------------------------------------------------------------
@@ -114,15 +136,16 @@ def rms(x: torch.Tensor, w: torch.Tensor, eps: float, dtype: torch.dtype, center
 SIGMOID_LAST, SILU_FIRST, SILU_LAST = 0, 1, 2
 
 
-def gated_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate: int) -> torch.Tensor:
-    """Group RMS norm with a gate: rms(y) * w * sigmoid(z), rms(y * silu(z)) * w or rms(y) * w * silu(z)."""
+def gated_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate: int, out: torch.Tensor | None = None) -> torch.Tensor:
+    """Group RMS norm with a gate: rms(y) * w * sigmoid(z), rms(y * silu(z)) * w or rms(y) * w * silu(z), to ``out`` (rows of any pitch) when given."""
     if y.is_cuda:
-        return _C().mix_gated_norm(y, z, w, groups, eps, gate)
+        return _C().mix_gated_norm(y, z, w, groups, eps, gate, out)
     yf, zf = y.float(), z.float()
     if gate == SILU_FIRST:
         yf = yf * F.silu(zf)
     n = _rms(yf.reshape(y.shape[0], groups, -1), eps).reshape(y.shape) * w
-    return (n if gate == SILU_FIRST else n * (torch.sigmoid(zf) if gate == SIGMOID_LAST else F.silu(zf))).to(y.dtype)
+    n = (n if gate == SILU_FIRST else n * (torch.sigmoid(zf) if gate == SIGMOID_LAST else F.silu(zf))).to(y.dtype)
+    return n if out is None else out.copy_(n)
 
 
 def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -141,6 +164,17 @@ def linear_gelu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         _C().mix_gelu_(y)
         return y
     return F.gelu(F.linear(x, w.to(x.dtype)), approximate="tanh")
+
+
+def linear_silu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """silu(x @ w.T); fused into the GEMM epilogue for bf16 rows."""
+    if x.is_cuda:
+        if x.dtype == torch.bfloat16 and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0:
+            return _C().gemm_silu(x, w)
+        y = F.linear(x, w)
+        _C().mix_silu_(y)
+        return y
+    return F.silu(F.linear(x, w.to(x.dtype)))
 
 
 def linear_clamped_glu(x: torch.Tensor, wgu: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
@@ -196,12 +230,14 @@ class InputConv:
 
 @dataclass
 class Routed:
-    """Rows of ``experts`` in the experts' order; row ``pos[t, j]`` belongs to token t."""
+    """Rows of ``experts`` in the experts' order; row ``pos[t, j]`` belongs to token t, with ``weight[t, j]`` if there are weights."""
     rows: torch.Tensor
     pos: torch.Tensor
+    weight: torch.Tensor | None = None
 
     def sum(self) -> torch.Tensor:
-        return self.rows.float()[self.pos.long()].sum(1)
+        r = self.rows.float()[self.pos.long()]
+        return r.sum(1) if self.weight is None else (r * self.weight[..., None]).sum(1)
 
 
 def input_conv(h: torch.Tensor, conv: InputConv | None, b: SpanBatch) -> tuple[torch.Tensor, torch.Tensor | None]:
@@ -276,30 +312,80 @@ def block_add(past: torch.Tensor, i: int, y1: torch.Tensor, y2: torch.Tensor | N
 TILE = 128              # rows of the expert kernels' tiles: every expert's rows start on one
 
 
-def experts(h: torch.Tensor, router: torch.Tensor, wgu: torch.Tensor, wd: torch.Tensor, top: int) -> Routed:
-    """Silu-gated experts on weighted inputs: token t goes to the ``top`` experts with the largest s = sigmoid(router h), each reads s h.
-    wgu [E * 2 F, W] holds every expert's gate and up rows as in ``linear_silu_glu``, wd [E * W, F].  No host synchronisation."""
+def experts(h: torch.Tensor, router: torch.Tensor, wgu: torch.Tensor, wd: torch.Tensor, top: int, clamp: tuple[float, float] | None = None,
+            softmax: bool = False) -> Routed:
+    """Gated experts.  Token t goes to the ``top`` experts with the largest scores: s = sigmoid(router h), and each reads s h — or, with ``softmax``,
+    s = softmax(router h) over all experts, each reads h and its result counts with s over the sum of the chosen ones (+ 1e-20).  The gate is
+    silu(gate) * up, with ``clamp`` = (limit, alpha) that of ``linear_clamped_glu``.  wgu [E * 2 F, W] holds every expert's gate and up rows as in
+    ``linear_silu_glu``, wd [E * W, F].  No host synchronisation."""
     e, width = router.shape[0], h.shape[1]
     f = wgu.shape[0] // (2 * e)
     logits = linear_f32(h, router)
     if h.is_cuda:
         C = _C()
-        pick, score, rank, plan = C.mix_route(logits, top, _counter(h.device, e + 1, "route"))
-        rows, pos = C.mix_expert_rows(h, pick, score, rank, plan, e)
+        pick, score, rank, plan = C.mix_route(logits, top, _counter(h.device, e + 1, "route"), softmax)
+        rows, pos = C.mix_expert_rows(h, pick, None if softmax else score, rank, plan, e)
+        limit, alpha = clamp or (0.0, 0.0)
         if h.dtype == torch.bfloat16 and f % 128 == 0 and width % 8 == 0:
-            return Routed(C.gemm_experts(C.gemm_experts(rows, wgu, plan, e, True), wd, plan, e, False), pos)
-        gu = C.mix_expert_gemm(rows, wgu, plan, e)
-        return Routed(C.mix_expert_gemm(silu_glu(gu, f), wd, plan, e), pos)
-    score, pick = torch.topk(torch.sigmoid(logits), top, dim=-1)
+            out = C.gemm_experts(C.gemm_experts(rows, wgu, plan, e, 1 if clamp is None else 2, limit, alpha), wd, plan, e, 0)
+        else:
+            gu = C.mix_expert_gemm(rows, wgu, plan, e)
+            blk = 128 if f % 128 == 0 else f
+            out = C.mix_expert_gemm(silu_glu(gu, f) if clamp is None else C.mix_clamped_glu(gu, blk, limit, alpha), wd, plan, e)
+        return Routed(out, pos, score if softmax else None)
+    score, pick = torch.topk(torch.softmax(logits, -1) if softmax else torch.sigmoid(logits), top, dim=-1)
+    if softmax:
+        score = score / (score.sum(-1, keepdim=True) + 1e-20)
     rows = h.new_empty(h.shape[0] * top, width)
     pos = torch.arange(rows.shape[0]).reshape(-1, top)
-    x = (h.float()[:, None] * score[..., None]).to(h.dtype)
+    x = h[:, None].expand(-1, top, -1) if softmax else (h.float()[:, None] * score[..., None]).to(h.dtype)
     for j in range(e):
         t, k = (pick == j).nonzero(as_tuple=True)
         if t.numel():
-            a = silu_glu(F.linear(x[t, k], wgu[j * 2 * f:(j + 1) * 2 * f]), f)
+            up = wgu[j * 2 * f:(j + 1) * 2 * f]
+            a = silu_glu(F.linear(x[t, k], up), f) if clamp is None else linear_clamped_glu(x[t, k], up, *clamp)
             rows[pos[t, k]] = F.linear(a, wd[j * width:(j + 1) * width])
-    return Routed(rows, pos)
+    return Routed(rows, pos, score if softmax else None)
+
+
+# --------------------------------------------------------------------------------------------
+# residual streams
+# --------------------------------------------------------------------------------------------
+def streams_embed(ids: torch.Tensor, w: torch.Tensor, scale: float, streams: int, win: torch.Tensor, w_norm: torch.Tensor, eps: float) -> tuple:
+    """(streams in fp32 — one row per token while all of them are equal: [T, 1, W] — and what the first sublayer reads, the norm of sum_s win[s] x)."""
+    if w.is_cuda:
+        return tuple(_C().mix_streams_embed(ids, w, scale, streams, win, w_norm, eps))
+    x = F.embedding(ids, w).float() * scale
+    return x[:, None], (_rms(x * win.sum(), eps) * w_norm).to(w.dtype)
+
+
+def _streams_after(x, y, bias, routed, mix, out):
+    t = (0 if y is None else y.float()) + (0 if bias is None else bias) + (0 if routed is None else routed.sum())
+    return torch.einsum("sr,tsw->trw", mix, x.expand(-1, mix.shape[0], -1)) + out[:, None] * t[:, None]
+
+
+def streams_add(x: torch.Tensor, y: torch.Tensor | None, bias: torch.Tensor | None, routed: Routed | None, mix: torch.Tensor, out: torch.Tensor,
+                win: torch.Tensor, w_norm: torch.Tensor, eps: float) -> tuple[torch.Tensor, torch.Tensor]:
+    """End of a sublayer and beginning of the next:  X_t = sum_s mix[s, t] x_s + out[t] (y + bias + weighted routed rows)  in fp32 [T, streams, W] (in
+    place where x has that shape), and norm(sum_t win[t] X_t) * w_norm in y's dtype."""
+    if x.is_cuda:
+        return tuple(_C().mix_streams_add(x, y, bias, *_routed(routed), mix, out, win, w_norm, eps, False))
+    x = _streams_after(x, y, bias, routed, mix, out)
+    return x, (_rms(torch.einsum("s,tsw->tw", win, x), eps) * w_norm).to((y if y is not None else routed.rows).dtype)
+
+
+def streams_sum(x: torch.Tensor, y: torch.Tensor | None, bias: torch.Tensor | None, routed: Routed | None, mix: torch.Tensor, out: torch.Tensor,
+                w_norm: torch.Tensor | None, eps: float) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """End of the last sublayer: (sum of the streams in fp32, its norm when there is a weight)."""
+    if x.is_cuda:
+        x, h = _C().mix_streams_add(x, y, bias, *_routed(routed), mix, out, None, w_norm, eps, True)
+        return x, (h if w_norm is not None else None)
+    x = _streams_after(x, y, bias, routed, mix, out).sum(1)
+    return x, (None if w_norm is None else (_rms(x, eps) * w_norm).to((y if y is not None else routed.rows).dtype))
+
+
+def _routed(r: Routed | None) -> tuple:
+    return (None, None, None) if r is None else (r.rows, r.pos, r.weight)
 
 
 # --------------------------------------------------------------------------------------------
@@ -325,19 +411,20 @@ def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, state
 # --------------------------------------------------------------------------------------------
 # gated linear recurrences
 # --------------------------------------------------------------------------------------------
-SSD, MLSTM, DELTA = 0, 1, 2
+SSD, MLSTM, DELTA, DECAY, GLA = range(5)
 
 
 @dataclass
 class Gates:
-    """Raw gate projections (fp32 [T, H]) and per-head constants of a recurrence."""
-    g0: torch.Tensor
+    """Raw gate projections (fp32 [T, H], ``GLA``: [T, H * N]) and per-head constants of a recurrence."""
+    g0: torch.Tensor | None = None
     g1: torch.Tensor | None = None
     b0: torch.Tensor | None = None
     b1: torch.Tensor | None = None
     a_log: torch.Tensor | None = None
     d_skip: torch.Tensor | None = None
-    cap: float = 1.0
+    cap: float = 1.0                    # GLA: tau
+    raw: bool = False                   # DECAY: q, k and v are still to be silu-activated (single tokens only)
 
 
 CHUNK_MIN = 8           # spans shorter than this go through the token-by-token kernel
@@ -349,7 +436,8 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
 
     ``SSD``: add = softplus(g0 + b0), keep = exp(-exp(a_log) add), y += d_skip v.  ``MLSTM``: capped log gates with a running
     maximum and a normaliser.  ``DELTA``: the gated delta rule on unit vectors k' = k / |k|, q' = q / |q| (1e-6 under the root): keep =
-    exp(-exp(a_log) softplus(g0 + b0)) and the write is k' u^T with u = sigmoid(g1) (v - keep S^T k').  q / k [T, groups * N] (consecutive heads share a group), v [T, H * V], cache["S"] [slots, H, N, V]
+    exp(-exp(a_log) softplus(g0 + b0)) and the write is k' u^T with u = sigmoid(g1) (v - keep S^T k').  ``DECAY``: add = 1, keep = exp(a_log).
+    ``GLA``: add = 1 and a keep for every state row, sigmoid(g0 + b0)^(1 / cap).  q / k [T, groups * N] (consecutive heads share a group), v [T, H * V], cache["S"] [slots, H, N, V]
     (+ "n" [slots, H, N], "m" [slots, H])."""
     if not v.is_cuda:
         return _scan_cpu(mode, q, k, v, gates, qscale, cache, b)
@@ -358,7 +446,7 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
     out = torch.empty(v.shape, device=v.device, dtype=v.dtype)
 
     def run(lo: int, hi: int, form: int) -> None:       # 0: token by token, 1: one token per span, 2 / 3: chunked
-        _C().mix_scan_(mode, q, k, v, gates.g0, gates.g1, gates.b0, gates.b1, gates.a_log, gates.d_skip, qscale, gates.cap, S, cache.get("n"),
+        _C().mix_scan_(mode, q, k, v, gates.g0, gates.g1, gates.b0, gates.b1, gates.a_log, gates.d_skip, qscale, gates.cap, gates.raw, S, cache.get("n"),
                        cache.get("m"), b.cu[lo:hi + 1], b.start[lo:hi], b.slot[lo:hi], ctr, form, out)
 
     chunk = v.dtype == torch.bfloat16 and b.max_long >= CHUNK_MIN
@@ -366,7 +454,7 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
         _C().mix_delta_chunk_(q, k, v, gates.g0, gates.g1, gates.b0, gates.a_log, qscale, S, b.cu[:b.n_long + 1], b.start[:b.n_long],
                               b.slot[:b.n_long], ctr, out)
     elif b.n_long:
-        chunk = chunk and mode != DELTA and _C().mix_chunk_supported(N)
+        chunk = chunk and mode not in (DELTA, GLA) and _C().mix_chunk_supported(N)
         run(0, b.n_long, (3 if b.max_long >= TC_MIN else 2) if chunk else 0)
     if b.n_long < b.spans:
         run(b.n_long, b.spans, 1)
@@ -390,9 +478,15 @@ def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
             kt = k[t].float().reshape(-1, N).repeat_interleave(rep, 0)
             if mode == DELTA:
                 qt, kt = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6) for x in (qt, kt))
-            qt = qt * qscale
             vt = v[t].float().reshape(H, V)
-            if mode in (SSD, DELTA):
+            if g.raw:
+                qt, kt, vt = (F.silu(x).to(v.dtype).float() for x in (qt, kt, vt))
+            qt = qt * qscale
+            if mode == DECAY:
+                keep, add = torch.exp(g.a_log), torch.ones(H)
+            elif mode == GLA:
+                keep, add = torch.exp(F.logsigmoid(g.g0[t] + g.b0) / g.cap).reshape(H, N), torch.ones(H)
+            elif mode in (SSD, DELTA):
                 add = F.softplus(g.g0[t] + g.b0, threshold=1e9)
                 keep = torch.exp(-torch.exp(g.a_log) * add)
             else:
@@ -406,7 +500,7 @@ def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
                 u = torch.sigmoid(g.g1[t])[:, None] * (vt - torch.einsum("hnv,hn->hv", S, kt))
                 S = S + kt[:, :, None] * u[:, None, :]
             else:
-                S = keep[:, None, None] * S + (add[:, None] * kt)[:, :, None] * vt[:, None, :]
+                S = keep.reshape(H, -1, 1) * S + (add[:, None] * kt)[:, :, None] * vt[:, None, :]
             y = torch.einsum("hnv,hn->hv", S, qt)
             if mode == SSD:
                 y = y + g.d_skip[:, None] * vt
@@ -416,6 +510,25 @@ def _scan_cpu(mode, q, k, v, g: Gates, qscale, cache, b: SpanBatch):
         S_pool[sl] = S
         if mode == MLSTM:
             cache["n"][sl], cache["m"][sl] = n, m
+    return out
+
+
+def selective_scan(x: torch.Tensor, dt: torch.Tensor, bm: torch.Tensor, cm: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor, a_neg: torch.Tensor,
+                   d_skip: torch.Tensor, state: torch.Tensor, b: SpanBatch) -> torch.Tensor:
+    """Per channel c and state n, with d = softplus(dt + dt_bias):  S[c, n] = exp(d_c a_neg[c, n]) S[c, n] + d_c x_c B_n,
+    y_c = sum_n S[c, n] C_n + d_skip_c x_c; returns y silu(z).  x, z [T, C], dt fp32 [T, C], bm, cm [T, N], state [slots, C, N]."""
+    if x.is_cuda:
+        return _C().mix_selective(x, dt, bm, cm, z, dt_bias, a_neg, d_skip, state, b.cu, b.start, b.slot, b.n_long)
+    out = torch.empty_like(x)
+    cu = b.cu.tolist()
+    for s in range(b.spans):
+        sl = int(b.slot[s])
+        S = state[sl].clone() if int(b.start[s]) else torch.zeros_like(state[0])
+        for t in range(cu[s], cu[s + 1]):
+            xt, d = x[t].float(), F.softplus(dt[t] + dt_bias, threshold=1e9)
+            S = torch.exp(d[:, None] * a_neg) * S + (d * xt)[:, None] * bm[t].float()
+            out[t] = ((S @ cm[t].float() + d_skip * xt) * F.silu(z[t].float())).to(x.dtype)
+        state[sl] = S
     return out
 
 
@@ -499,10 +612,14 @@ def latent_attention(q_lat: torch.Tensor, q: torch.Tensor, d: int, pool: torch.T
     return out
 
 
+def sink_varlen_ok(kw: int, vw: int) -> bool:
+    """Widths that the packed kernel takes."""
+    return (kw, vw) in ((64, 64), (64, 128), (128, 64), (128, 128), (192, 128))
+
+
 def sink_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.Tensor, cu_k: torch.Tensor, scale: float,
                           sink: torch.Tensor | None) -> torch.Tensor:
-    """Causal (bottom-right aligned) attention of packed spans on expanded keys, with a sink: the tcgen05 kernel, query / key width
-    128 or 192, value width 128, bf16."""
+    """Causal (bottom-right aligned) attention of packed spans, with a sink: the tcgen05 kernel, widths of ``sink_varlen_ok``, bf16."""
     return _C().attn_fwd(q, k, v, cu_q, cu_k, scale, True, False, None, sink)[0]
 
 
@@ -576,6 +693,67 @@ def window_attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, c
                             keep_first: int) -> torch.Tensor:
     """Packed spans, bottom-right aligned: the tcgen05 kernel, width 64 or 128, bf16."""
     return _C().attn_fwd(q, k, v, cu_q, cu_k, scale, True, False, None, None, window, keep_first)[0]
+
+
+# --------------------------------------------------------------------------------------------
+# attention with rotated values and a sink
+# --------------------------------------------------------------------------------------------
+def turn_prep(p: torch.Tensor, bias: torch.Tensor, heads: int, dim: int, vdim: int, freq: torch.Tensor, vfreq: torch.Tensor, k_pool: torch.Tensor,
+              v_pool: torch.Tensor, b: SpanBatch, eps: float, want_kv: bool) -> tuple[torch.Tensor, tuple | None]:
+    """Rows [queries: heads x dim | keys: groups x dim | values: groups x vdim] as projected, without their ``bias`` -> queries [T, heads, key width],
+    rotated (entries i and i + freq.numel()) and divided by their root mean square; the keys treated alike go to ``k_pool`` ([pages, groups, PAGE, key
+    width]), the values, rotated over all of ``vdim``, to ``v_pool``.  Packed keys and values are returned too when asked for."""
+    g, kw, vw = k_pool.shape[1], k_pool.shape[3], v_pool.shape[3]
+    if p.is_cuda:
+        q, k, v = _C().mix_turn_prep(p, bias, heads, dim, vdim, freq, vfreq, b.pos, b.kv_slot, k_pool, v_pool, eps, want_kv)
+        return q, ((k, v) if want_kv else None)
+    t, nq = p.shape[0], heads * dim
+    x = p.float() + bias
+
+    def turned(y, f):
+        n = 2 * f.numel()
+        return torch.cat([_rotate(y[..., :n], f, b.pos), y[..., n:]], -1)
+
+    q, k = (_rms(turned(y.reshape(t, -1, dim), freq), eps).to(p.dtype) for y in (x[:, :nq], x[:, nq:nq + g * dim]))
+    v = turned(x[:, nq + g * dim:].reshape(t, g, vdim), vfreq).to(p.dtype)
+    q, k, v = F.pad(q, (0, kw - dim)), F.pad(k, (0, kw - dim)), F.pad(v, (0, vw - vdim))
+    page, off = b.kv_slot // PAGE, b.kv_slot % PAGE
+    k_pool[page, :, off], v_pool[page, :, off] = k, v
+    return q, ((k, v) if want_kv else None)
+
+
+def turn_back(o: torch.Tensor, gate: torch.Tensor, vfreq: torch.Tensor, pos: torch.Tensor, scale: float, out: torch.Tensor) -> torch.Tensor:
+    """o [T, heads, value width]: entries (m, m + vdim / 2) of every head turned by -pos * vfreq[m], times scale * sigmoid(gate) -> out [T, heads * vdim]."""
+    if o.is_cuda:
+        _C().mix_turn_back(o, gate, vfreq, pos, scale, out)
+        return out
+    x = _rotate(o[..., :2 * vfreq.numel()].float(), -vfreq, pos).reshape(o.shape[0], -1)
+    return out.copy_((x * torch.sigmoid(gate.float()) * scale).to(o.dtype))
+
+
+def sink_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, table: torch.Tensor, seq_of: torch.Tensor | None, kv_len: torch.Tensor,
+                   scale: float, sink: torch.Tensor, max_len: int) -> torch.Tensor:
+    """Paged form, one query row [heads, key width] per entry of ``kv_len`` (its own token is its last key) -> [rows, heads, value width]; ``sink``
+    [heads] adds exp(sink) to the denominator."""
+    rows, h, kw = q.shape
+    g, vw = k_pool.shape[1], v_pool.shape[3]
+    if q.is_cuda:
+        if q.dtype == torch.bfloat16 and sink_varlen_ok(kw, vw) and h // g <= 16 and seq_of is None:
+            from .functional import _auto_splits
+
+            return _C().sink_decode(q, k_pool, v_pool, table, kv_len, scale, _auto_splits(rows, g, max_len), sink)
+        return _C().mix_sink_attention(q, k_pool, v_pool, table, seq_of, kv_len, scale, sink)
+    out = q.new_zeros(rows, h, vw)
+    for i in range(rows):
+        n = int(kv_len[i])
+        if n == 0:
+            continue
+        pages = table[int(seq_of[i]) if seq_of is not None else i, : (n + PAGE - 1) // PAGE].long()
+        j = torch.arange(n)
+        k, v = (x[pages[j // PAGE], :, j % PAGE].float().repeat_interleave(h // g, 1) for x in (k_pool, v_pool))
+        s = torch.cat([torch.einsum("hd,jhd->hj", q[i].float(), k) * scale, sink[:, None]], -1)
+        out[i] = torch.einsum("hj,jhd->hd", torch.softmax(s, -1)[:, :n], v).to(q.dtype)
+    return out
 
 
 # --------------------------------------------------------------------------------------------
