@@ -445,10 +445,10 @@ static int run_attn_fwd(const void* q, const void* k, const void* v, const AttnF
 }
 
 // q:[Tq, nq*dk] (pitch ldq), k:[Tk, nkv*dk], v:[Tk, nkv*dv] (pitches ldk/ldv), o:[Tq, nq*dv] (pitch ldo); pitches in ELEMENTS;
-// dk = 64 (dv = 64), 128 or 192 (dv = 128).  window > 0 (causal only): query i sees keys j <= i with i - j < window or j < keep_first.  cu_q / cu_k: int32 [B+1] device arrays.  max_tiles: upper bound on sum_b ceil(lq_b / 128) (e.g. Tq/128 + B).
+// dk, dv = 64 or 128; dk = 192 (dv = 128).  window > 0 (causal only): query i sees keys j <= i with i - j < window or j < keep_first.  cu_q / cu_k: int32 [B+1] device arrays.  max_tiles: upper bound on sum_b ceil(lq_b / 128) (e.g. Tq/128 + B).
 // sink: fp32 [nq] or null.
 extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o, float* lse, const int32_t* cu_q,
-                            const int32_t* cu_k, int B, int Tq, int Tk, int nq, int nkv, int dk, int64_t ldq, int64_t ldk, int64_t ldv,
+                            const int32_t* cu_k, int B, int Tq, int Tk, int nq, int nkv, int dk, int dv, int64_t ldq, int64_t ldk, int64_t ldv,
                             int64_t ldo, float sm_scale, int causal, int max_tiles, const float* sink, int window, int keep_first, long long* dbg,
                             cudaStream_t stream) {
   if (Tq <= 0 || B <= 0) return 0;
@@ -466,9 +466,11 @@ extern "C" int prl_attn_fwd(const void* q, const void* k, const void* v, void* o
   p.keep_first = window > 0 ? keep_first : 0;
   p.sink = sink;
   p.dbg = dbg;
-  if (dk == 64) return run_attn_fwd<64, 64, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
-  if (dk == 128) return run_attn_fwd<128, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
-  if (dk == 192) return run_attn_fwd<192, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 64 && dv == 64) return run_attn_fwd<64, 64, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 64 && dv == 128) return run_attn_fwd<64, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 128 && dv == 64) return run_attn_fwd<128, 64, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 128 && dv == 128) return run_attn_fwd<128, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
+  if (dk == 192 && dv == 128) return run_attn_fwd<192, 128, 1>(q, k, v, p, Tk, ldq, ldk, ldv, max_tiles, stream);
   return -114;
 }
 

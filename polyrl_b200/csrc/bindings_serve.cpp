@@ -9,16 +9,17 @@ extern "C" {
 int prl_gemm_bf16(const void*, const void*, void*, const void*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
 int prl_sample(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int64_t*, float*, cudaStream_t);
 int prl_sample_topk_topp(const void*, int, int64_t, int, int, const float*, const uint64_t*, int, int, float, int64_t*, float*, cudaStream_t);
-int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int32_t*, const int32_t*, int, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, float, int, int, const float*, int, int, long long*, cudaStream_t);
+int prl_attn_fwd(const void*, const void*, const void*, void*, float*, const int32_t*, const int32_t*, int, int, int, int, int, int, int, int64_t, int64_t, int64_t, int64_t, float, int, int, const float*, int, int, long long*, cudaStream_t);
 int prl_paged_decode_workspace_floats(int, int, int, int);
 int prl_paged_decode(const void*, int64_t, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, float, int, int, int, float*, void*, int64_t, cudaStream_t);
 int prl_gemm_clamped_glu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, float, float, cudaStream_t);
 int prl_gemm_swiglu_bf16(const void*, const void*, void*, void*, int, int, int, int64_t, int64_t, int64_t, int64_t, cudaStream_t);
-int prl_gemm_experts_bf16(const void*, const void*, void*, const int32_t*, int, int, int, int, int, cudaStream_t);
+int prl_gemm_experts_bf16(const void*, const void*, void*, const int32_t*, int, int, int, int, int, float, float, cudaStream_t);
+int prl_sink_decode(const void*, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, int, float, int, const float*, float*, void*, cudaStream_t);
 int prl_map_attn_fwd(const void*, const void*, const void*, void*, const int32_t*, const int32_t*, int, int, int, int, int, int, int, int, int, float, int, const float*, float, float, int, cudaStream_t);
 int prl_map_decode_ok(int, int, int);
 int prl_map_decode(const void*, const void*, const void*, const int32_t*, int64_t, const int32_t*, int, int, int, int, int, int, float, int, int, const float*, float, float, float*, void*, cudaStream_t);
-int prl_gemm_gelu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, cudaStream_t);
+int prl_gemm_gelu_bf16(const void*, const void*, void*, int, int, int, int64_t, int64_t, int64_t, int, cudaStream_t);
 int prl_mix_embed(const int64_t*, const void*, const float*, float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_norm_add(const void*, int64_t, float*, const float*, const float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_rms(const float*, const float*, void*, int, int, float, int, int, cudaStream_t);
@@ -26,7 +27,9 @@ int prl_mix_gated_norm(const void*, int64_t, const void*, int64_t, const float*,
 int prl_mix_conv(const void*, int64_t, const float*, const float*, void*, const int32_t*, const int32_t*, const int64_t*, const int32_t*, void*, int64_t, int, int, int, int, int, cudaStream_t);
 int prl_mix_latent_prep(const void*, int64_t, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, int, float, int, cudaStream_t);
 int prl_mix_rope(void*, int64_t, int, int, int, int, const double*, const int64_t*, int, int, cudaStream_t);
-int prl_mix_gelu(void*, int64_t, int, cudaStream_t);
+int prl_mix_gelu(void*, int64_t, int, int, cudaStream_t);
+int prl_mix_turn_rows(const void*, int64_t, const float*, const double*, const double*, const int64_t*, const int64_t*, void*, void*, void*, void*, void*, int, int, int, int, int, int, int, int, float, int, cudaStream_t);
+int prl_mix_turn_back(const void*, const void*, int64_t, const double*, const int64_t*, float, void*, int64_t, int, int, int, int, int, cudaStream_t);
 int prl_mix_qk_prep(const void*, int64_t, int, int, int, int, int, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, void*, void*, int, float, int, cudaStream_t);
 int prl_mix_gather_keys(const void*, const void*, const int64_t*, void*, void*, int64_t, int, int, int, cudaStream_t);
 int prl_mix_map_rows(const void*, int64_t, const float*, const float*, const float*, const double*, const int64_t*, const int64_t*, void*, void*, void*, void*, void*, int, int, int, int, int, int, int, int, int, float, int, cudaStream_t);
@@ -34,7 +37,7 @@ int prl_mix_input_conv(const void*, int64_t, const float*, const float*, void*, 
 int prl_mix_poly_norm(const void*, int64_t, const float*, void*, int, int, float, int, cudaStream_t);
 int prl_mix_silu_glu(const void*, void*, int64_t, int, int, int, cudaStream_t);
 int prl_mix_route_tiles(int64_t, int64_t);
-int prl_mix_route(const float*, int64_t, int, int, int, int32_t*, float*, int32_t*, int32_t*, int32_t*, cudaStream_t);
+int prl_mix_route(const float*, int64_t, int, int, int, int32_t*, float*, int32_t*, int32_t*, int32_t*, int, cudaStream_t);
 int prl_mix_expert_rows(const void*, int64_t, const int32_t*, const float*, const int32_t*, const int32_t*, void*, int32_t*, int, int, int, int, cudaStream_t);
 int prl_mix_expert_gemm(const void*, const void*, const int32_t*, void*, int, int, int, int, int, cudaStream_t);
 int prl_mix_clamped_glu(const void*, void*, int64_t, int, int, float, float, int, cudaStream_t);
@@ -54,6 +57,9 @@ int prl_mix_chunk_tc(const prl::ScanParams*, int, int32_t*, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
 int prl_mix_window(const prl::WindowParams*, int, cudaStream_t);
 int prl_mix_block(const prl::BlockParams*, int, cudaStream_t);
+int prl_mix_sink(const prl::SinkParams*, int, cudaStream_t);
+int prl_mix_selective(const prl::SelectiveParams*, int, int, cudaStream_t);
+int prl_mix_streams(const prl::StreamsParams*, int, cudaStream_t);
 int prl_mix_map_attention(const prl::MapParams*, int, cudaStream_t);
 int prl_mix_delta(const prl::ScanParams*, int64_t, int64_t, void*, float*, int32_t*, cudaStream_t);
 }
@@ -121,8 +127,8 @@ std::vector<at::Tensor> attn_fwd(const at::Tensor& q, const at::Tensor& k, const
                                  const at::Tensor& cu_k, double sm_scale, bool causal, bool want_lse,
                                  const c10::optional<at::Tensor>& dbg, const c10::optional<at::Tensor>& sink, int64_t window, int64_t keep_first) {
   CHECK_BF16(q); CHECK_BF16(k); CHECK_BF16(v);
-  const int64_t dk = q.size(-1), dv = dk == 64 ? 64 : 128;
-  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && (dk == 64 || dk == 128 || dk == 192) && k.size(2) == dk && v.size(2) == dv &&
+  const int64_t dk = q.size(-1), dv = v.size(-1);
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && (dk == 64 || dk == 128 || dk == 192) && k.size(2) == dk && (dv == 128 || (dv == 64 && dk != 192)) &&
               v.size(1) == k.size(1) && v.size(0) == k.size(0), "attn_fwd: query / key width 64, 128 or 192, value width 64 or 128");
   TORCH_CHECK(window >= 0 && window <= 0x7fffffff && keep_first >= 0 && keep_first <= 0x7fffff00 && (window == 0 || causal), "attn_fwd: window");
   TORCH_CHECK(q.stride(2) == 1 && q.stride(1) == dk && k.stride(2) == 1 && k.stride(1) == dk && v.stride(2) == 1 && v.stride(1) == dv,
@@ -138,7 +144,7 @@ std::vector<at::Tensor> attn_fwd(const at::Tensor& q, const at::Tensor& k, const
   at::Tensor o = at::empty({Tq, nq, dv}, q.options());
   at::Tensor lse = want_lse ? at::empty({nq, Tq}, q.options().dtype(at::kFloat)) : at::Tensor();
   check(prl_attn_fwd(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), want_lse ? lse.data_ptr<float>() : nullptr,
-                     cu_q.data_ptr<int>(), cu_k.data_ptr<int>(), B, Tq, Tk, nq, nkv, static_cast<int>(dk), q.stride(0), k.stride(0), v.stride(0),
+                     cu_q.data_ptr<int>(), cu_k.data_ptr<int>(), B, Tq, Tk, nq, nkv, static_cast<int>(dk), static_cast<int>(dv), q.stride(0), k.stride(0), v.stride(0),
                      static_cast<int64_t>(nq) * dv, static_cast<float>(sm_scale), causal ? 1 : 0, Tq / 128 + B,
                      sink.has_value() ? sink->data_ptr<float>() : nullptr, static_cast<int>(window), static_cast<int>(keep_first),
                      dbg.has_value() ? reinterpret_cast<long long*>(dbg->data_ptr<int64_t>()) : nullptr, cur_stream()),
@@ -229,12 +235,14 @@ at::Tensor mix_rms(const at::Tensor& x, const at::Tensor& w, double eps, bool bf
   return h;
 }
 
-at::Tensor mix_gated_norm(const at::Tensor& y, const at::Tensor& z, const at::Tensor& w, int64_t groups, double eps, int64_t gate) {
+at::Tensor mix_gated_norm(const at::Tensor& y, const at::Tensor& z, const at::Tensor& w, int64_t groups, double eps, int64_t gate,
+                          const c10::optional<at::Tensor>& to) {
   const int dt = dt_of(y, "mix_gated_norm");
   rows2(y, "mix_gated_norm y"); rows2(z, "mix_gated_norm z");
   TORCH_CHECK(z.scalar_type() == y.scalar_type() && z.sizes() == y.sizes() && groups > 0 && y.size(1) % groups == 0);
   c10::cuda::CUDAGuard g(y.device());
-  at::Tensor out = at::empty(y.sizes(), y.options());
+  at::Tensor out = to.has_value() ? *to : at::empty(y.sizes(), y.options());
+  TORCH_CHECK(out.is_cuda() && out.scalar_type() == y.scalar_type() && out.sizes() == y.sizes() && out.stride(1) == 1, "mix_gated_norm: out");
   check(prl_mix_gated_norm(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), vecf(w, y.size(1), "mix_gated_norm w"), out.data_ptr(), out.stride(0),
                            y.size(0), groups, y.size(1) / groups, static_cast<float>(eps), static_cast<int>(gate), dt, cur_stream()), "mix_gated_norm");
   return out;
@@ -259,33 +267,39 @@ at::Tensor mix_conv(const at::Tensor& x, const at::Tensor& w, const c10::optiona
 }
 
 // gated linear recurrences over packed spans (mix_scan_): form 0 = token by token, 1 = every span is one token, 2 = chunked (bf16), 3 = chunked on
-// tcgen05 where the layout allows, else 2; the last counter element is the error flag; mode 0 = state-space duality, 1 = matrix memory, 2 = gated delta rule (csrc/mixers.cuh)
-prl::ScanParams scan_params(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
+// tcgen05 where the layout allows, else 2; the last counter element is the error flag; mode 0 = state-space duality, 1 = matrix memory, 2 = gated delta rule, 3 = constant decay, 4 = decay per state row
+// (csrc/mixers.cuh)
+prl::ScanParams scan_params(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const c10::optional<at::Tensor>& g0, const c10::optional<at::Tensor>& g1,
                             const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log, double qscale,
                             const at::Tensor& S, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, const at::Tensor& counter,
                             const at::Tensor& out) {
-  rows2(q, "mix_scan q"); rows2(k, "mix_scan k"); rows2(v, "mix_scan v"); rows2(g0, "mix_scan g0");
-  CHECK_F32(S); CHECK_F32(g0);
-  TORCH_CHECK(mode >= 0 && mode <= 2);
+  rows2(q, "mix_scan q"); rows2(k, "mix_scan k"); rows2(v, "mix_scan v");
+  CHECK_F32(S);
+  TORCH_CHECK(mode >= 0 && mode <= 4);
   TORCH_CHECK(S.dim() == 4 && S.is_contiguous());
   const int64_t H = S.size(1), N = S.size(2), V = S.size(3), T = v.size(0), spans = start.numel();
   TORCH_CHECK(q.scalar_type() == v.scalar_type() && k.scalar_type() == v.scalar_type() && q.size(0) == T && k.size(0) == T && v.size(1) == H * V &&
               q.sizes() == k.sizes() && q.size(1) % N == 0 && q.size(1) > 0 && H % (q.size(1) / N) == 0, "mix_scan: shapes");
-  TORCH_CHECK(g0.size(0) == T && g0.size(1) == H);
   TORCH_CHECK(N <= 512, "mix_scan: state rows per head <= 512");
   prl::ScanParams p{};
   p.q = q.data_ptr(); p.k = k.data_ptr(); p.v = v.data_ptr();
   p.ldq = q.stride(0); p.ldk = k.stride(0); p.ldv = v.stride(0);
   p.rep = H / (q.size(1) / N);
-  p.g0 = g0.data_ptr<float>(); p.ldg = g0.stride(0);
-  p.b0 = vecf(b0, H, "b0"); p.b1 = vecf(b1, H, "b1"); p.a_log = vecf(a_log, H, "a_log");
-  if (mode != 0) {
+  const int64_t gates = mode == 4 ? H * N : H;
+  if (mode != 3) {
+    TORCH_CHECK(g0.has_value());
+    rows2(*g0, "mix_scan g0"); CHECK_F32(*g0);
+    TORCH_CHECK(g0->size(0) == T && g0->size(1) == gates, "mix_scan: gates");
+    p.g0 = g0->data_ptr<float>(); p.ldg = g0->stride(0);
+  }
+  p.b0 = vecf(b0, gates, "b0"); p.b1 = vecf(b1, H, "b1"); p.a_log = vecf(a_log, H, "a_log");
+  if (mode == 1 || mode == 2) {
     TORCH_CHECK(g1.has_value());
     CHECK_F32(*g1);
-    TORCH_CHECK(g1->dim() == 2 && g1->size(0) == T && g1->size(1) == H && g1->stride(1) == 1 && g1->stride(0) == g0.stride(0));
+    TORCH_CHECK(g1->dim() == 2 && g1->size(0) == T && g1->size(1) == H && g1->stride(1) == 1 && g1->stride(0) == g0->stride(0));
     p.g1 = g1->data_ptr<float>();
   }
-  TORCH_CHECK(mode == 1 || a_log.has_value());
+  TORCH_CHECK(mode == 1 || mode == 4 || a_log.has_value());
   p.qscale = static_cast<float>(qscale);
   TORCH_CHECK(out.is_cuda() && out.scalar_type() == v.scalar_type() && out.is_contiguous() && out.dim() == 2 && out.size(0) == T && out.size(1) == H * V);
   p.out = out.data_ptr(); p.ldo = H * V;
@@ -297,15 +311,17 @@ prl::ScanParams scan_params(int64_t mode, const at::Tensor& q, const at::Tensor&
   return p;
 }
 
-void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& g1,
+void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const c10::optional<at::Tensor>& g0, const c10::optional<at::Tensor>& g1,
                      const c10::optional<at::Tensor>& b0, const c10::optional<at::Tensor>& b1, const c10::optional<at::Tensor>& a_log,
-                     const c10::optional<at::Tensor>& d_skip, double qscale, double cap, at::Tensor S, const c10::optional<at::Tensor>& nst,
+                     const c10::optional<at::Tensor>& d_skip, double qscale, double cap, bool raw, at::Tensor S, const c10::optional<at::Tensor>& nst,
                      const c10::optional<at::Tensor>& mst, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, at::Tensor counter,
                      int64_t form, at::Tensor out) {
   const int dt = dt_of(v, "mix_scan");
   prl::ScanParams p = scan_params(mode, q, k, v, g0, g1, b0, b1, a_log, qscale, S, cu, start, slot, counter, out);
   p.d_skip = vecf(d_skip, p.H, "d_skip");
   p.cap = static_cast<float>(cap);
+  p.raw = raw;
+  TORCH_CHECK(mode != 4 || cap > 0);
   if (mode == 1) {
     TORCH_CHECK(nst.has_value() && mst.has_value());
     CHECK_F32(*nst); CHECK_F32(*mst);
@@ -313,7 +329,7 @@ void mix_scan_(int64_t mode, const at::Tensor& q, const at::Tensor& k, const at:
     p.nst = nst->data_ptr<float>(); p.mst = mst->data_ptr<float>();
   }
   c10::cuda::CUDAGuard g(v.device());
-  TORCH_CHECK(form < 2 || mode < 2, "mix_scan: the delta rule has its own chunked kernel");
+  TORCH_CHECK(form < 2 || mode < 2 || mode == 3, "mix_scan: no chunked form here");
   if (form == 3 && dt == 0 && prl_mix_chunk_tc_ok(&p)) {
     check(prl_mix_chunk_tc(&p, static_cast<int>(mode), p.counter + counter.numel() - 1, cur_stream()), "mix_chunk_tc");
   } else if (form >= 2) {
@@ -474,21 +490,21 @@ at::Tensor mix_clamped_glu(const at::Tensor& gu, int64_t blk, double limit, doub
   return out;
 }
 
-at::Tensor gemm_gelu(const at::Tensor& a, const at::Tensor& w) {
+at::Tensor gemm_act(const at::Tensor& a, const at::Tensor& w, bool silu) {
   CHECK_BF16(a); CHECK_BF16(w); CHECK_LASTDIM(a); CHECK_LASTDIM(w);
   TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && a.size(1) == w.size(1) && w.size(0) % 8 == 0 && a.size(1) % 8 == 0 && a.stride(0) % 8 == 0 &&
               w.stride(0) % 8 == 0);
   c10::cuda::CUDAGuard g(a.device());
   at::Tensor h = at::empty({a.size(0), w.size(0)}, a.options());
-  check(prl_gemm_gelu_bf16(a.data_ptr(), w.data_ptr(), h.data_ptr(), a.size(0), w.size(0), a.size(1), a.stride(0), w.stride(0), h.stride(0), cur_stream()),
-        "gemm_gelu");
+  check(prl_gemm_gelu_bf16(a.data_ptr(), w.data_ptr(), h.data_ptr(), a.size(0), w.size(0), a.size(1), a.stride(0), w.stride(0), h.stride(0), silu, cur_stream()),
+        "gemm_act");
   return h;
 }
-void mix_gelu_(at::Tensor x) {
-  const int dt = dt_of(x, "mix_gelu");
+void mix_act_(at::Tensor x, bool silu) {
+  const int dt = dt_of(x, "mix_act");
   TORCH_CHECK(x.is_contiguous());
   c10::cuda::CUDAGuard g(x.device());
-  check(prl_mix_gelu(x.data_ptr(), x.numel(), dt, cur_stream()), "mix_gelu");
+  check(prl_mix_gelu(x.data_ptr(), x.numel(), silu, dt, cur_stream()), "mix_act");
 }
 
 std::vector<at::Tensor> gemm_swiglu(const at::Tensor& a, const at::Tensor& wgu, bool save_gu) {
@@ -622,9 +638,182 @@ std::vector<at::Tensor> mix_input_conv(const at::Tensor& h, const at::Tensor& w1
   return {o1, o2};
 }
 
+// ---------------------------------------------------------------------------------------------- residual streams
+const float* norm_weight(prl::StreamsParams& p, const c10::optional<at::Tensor>& w) {
+  if (!w.has_value()) return nullptr;
+  p.w_scalar = w->numel() == 1 && p.W != 1;
+  return vecf(w, p.w_scalar ? 1 : p.W, "streams: norm weight");
+}
+// -> (streams [T, 1, W], h)
+std::vector<at::Tensor> mix_streams_embed(const at::Tensor& ids, const at::Tensor& emb, double scale, int64_t streams, const at::Tensor& win, const at::Tensor& w_norm,
+                                          double eps) {
+  const int dt = dt_of(emb, "mix_streams_embed");
+  TORCH_CHECK(emb.is_contiguous() && emb.dim() == 2);
+  c10::cuda::CUDAGuard g(emb.device());
+  prl::StreamsParams p{};
+  p.R = ids.numel(); p.W = emb.size(1); p.S = streams;
+  p.ids = veci<int64_t>(ids, p.R, "ids");
+  p.emb = emb.data_ptr(); p.scale = static_cast<float>(scale); p.eps = static_cast<float>(eps);
+  at::Tensor x = at::empty({p.R, 1, p.W}, emb.options().dtype(at::kFloat)), h = at::empty({p.R, p.W}, emb.options());
+  p.x_out = x.data_ptr<float>(); p.row_out = p.W;
+  p.win = vecf(win, streams, "win");
+  p.w_next = norm_weight(p, w_norm);
+  p.h = h.data_ptr();
+  check(prl_mix_streams(&p, dt, cur_stream()), "mix_streams_embed");
+  return {x, h};
+}
+// x [T, 1 or streams, W] -> (streams after the sublayer, h), or with `last` (their sum [T, W], h)
+std::vector<at::Tensor> mix_streams_add(at::Tensor x, const c10::optional<at::Tensor>& y, const c10::optional<at::Tensor>& bias, const c10::optional<at::Tensor>& rows,
+                                        const c10::optional<at::Tensor>& pos, const c10::optional<at::Tensor>& weight, const at::Tensor& mix, const at::Tensor& out,
+                                        const c10::optional<at::Tensor>& win, const c10::optional<at::Tensor>& w_next, double eps, bool last) {
+  CHECK_F32(x);
+  TORCH_CHECK(x.dim() == 3 && x.is_contiguous() && (y.has_value() || rows.has_value()), "mix_streams_add: x [T, streams, W] and something to add");
+  const at::Tensor& like = y.has_value() ? *y : *rows;
+  const int dt = dt_of(like, "mix_streams_add");
+  prl::StreamsParams p{};
+  p.R = x.size(0); p.W = x.size(2); p.S = out.numel();
+  TORCH_CHECK((x.size(1) == 1 || x.size(1) == p.S) && (last || win.has_value()), "mix_streams_add: streams");
+  c10::cuda::CUDAGuard g(x.device());
+  p.x_in = x.data_ptr<float>(); p.row_in = x.stride(0); p.stream_in = x.size(1) == 1 ? 0 : p.W;
+  if (y.has_value()) {
+    rows2(*y, "mix_streams_add y");
+    TORCH_CHECK(y->size(0) == p.R && y->size(1) == p.W);
+    p.y = y->data_ptr(); p.ldy = y->stride(0);
+  }
+  p.bias = vecf(bias, p.W, "bias");
+  if (rows.has_value()) {
+    TORCH_CHECK(pos.has_value() && rows->scalar_type() == like.scalar_type() && rows->is_contiguous() && rows->dim() == 2 && rows->size(1) == p.W &&
+                pos->dim() == 2 && pos->size(0) == p.R);
+    p.rows = rows->data_ptr(); p.top = pos->size(1);
+    p.pos = veci<int32_t>(*pos, static_cast<int64_t>(p.R) * p.top, "pos");
+    p.weight = vecf(weight, static_cast<int64_t>(p.R) * p.top, "weight");
+  }
+  p.mix = vecf(mix, static_cast<int64_t>(p.S) * p.S, "mix"); p.out = vecf(out, p.S, "out"); p.win = vecf(win, p.S, "win");
+  p.eps = static_cast<float>(eps);
+  p.w_next = norm_weight(p, w_next);
+  at::Tensor z, h;
+  if (last) {
+    z = at::empty({p.R, p.W}, x.options());
+    p.sum = z.data_ptr<float>();
+  } else {
+    z = p.stream_in || p.S == 1 ? x : at::empty({p.R, p.S, p.W}, x.options());
+    p.x_out = z.data_ptr<float>(); p.row_out = z.stride(0);
+  }
+  if (p.w_next) { h = at::empty({p.R, p.W}, like.options()); p.h = h.data_ptr(); }
+  check(prl_mix_streams(&p, dt, cur_stream()), "mix_streams_add");
+  return {z, h};
+}
+
+// ---------------------------------------------------------------------------------------------- selective scan
+// the first n_long spans token by token in one CTA per span and channels, the rest as single tokens
+at::Tensor mix_selective(const at::Tensor& x, const at::Tensor& dt, const at::Tensor& b, const at::Tensor& c, const at::Tensor& z, const at::Tensor& dt_bias,
+                         const at::Tensor& a_neg, const at::Tensor& d_skip, at::Tensor S, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot,
+                         int64_t n_long) {
+  const int d = dt_of(x, "mix_selective");
+  for (const at::Tensor& t : {x, b, c, z, dt}) rows2(t, "mix_selective");
+  CHECK_F32(dt); CHECK_F32(S);
+  const int64_t T = x.size(0), C = x.size(1), N = b.size(1), spans = start.numel();
+  for (const at::Tensor& t : {b, c, z}) TORCH_CHECK(t.is_cuda() && t.scalar_type() == x.scalar_type() && t.size(0) == T, "mix_selective: rows");
+  TORCH_CHECK(z.size(1) == C && c.size(1) == N && dt.size(0) == T && dt.size(1) == C && S.dim() == 3 && S.is_contiguous() && S.size(1) == C && S.size(2) == N &&
+              n_long >= 0 && n_long <= spans, "mix_selective: shapes");
+  prl::SelectiveParams p{};
+  p.x = x.data_ptr(); p.z = z.data_ptr(); p.b = b.data_ptr(); p.c = c.data_ptr();
+  p.ldx = x.stride(0); p.ldz = z.stride(0); p.ldb = b.stride(0); p.ldc = c.stride(0);
+  p.dt = dt.data_ptr<float>(); p.ldd = dt.stride(0);
+  p.dt_bias = vecf(dt_bias, C, "dt_bias"); p.d_skip = vecf(d_skip, C, "d_skip"); p.a_neg = vecf(a_neg, C * N, "a_neg");
+  c10::cuda::CUDAGuard g(x.device());
+  at::Tensor out = at::empty({T, C}, x.options());
+  p.out = out.data_ptr(); p.ldo = C;
+  p.S = S.data_ptr<float>();
+  p.cu = veci<int32_t>(cu, spans + 1, "cu"); p.start = veci<int32_t>(start, spans, "start"); p.slot = veci<int64_t>(slot, spans, "slot");
+  p.C = C; p.N = N;
+  p.spans = n_long;
+  check(prl_mix_selective(&p, d, 0, cur_stream()), "mix_selective");
+  p.cu += n_long; p.start += n_long; p.slot += n_long;
+  p.spans = spans - n_long;
+  check(prl_mix_selective(&p, d, 1, cur_stream()), "mix_selective step");
+  return out;
+}
+
+// ---------------------------------------------------------------------------------------------- attention with rotated values and a sink
+// rows [queries H x D | keys G x D | values G x V] -> q [T, H, kw], pools, and packed keys / values when asked for
+std::vector<at::Tensor> mix_turn_prep(const at::Tensor& p, const at::Tensor& bias, int64_t heads, int64_t dim, int64_t vdim, const at::Tensor& freq,
+                                      const at::Tensor& vfreq, const at::Tensor& pos, const at::Tensor& kvslot, at::Tensor k_pool, at::Tensor v_pool, double eps,
+                                      bool want_kv) {
+  const int dt = dt_of(p, "mix_turn_prep");
+  rows2(p, "mix_turn_prep p");
+  for (const at::Tensor& t : {k_pool, v_pool})
+    TORCH_CHECK(t.is_cuda() && t.dim() == 4 && t.size(2) == 16 && t.is_contiguous() && t.scalar_type() == p.scalar_type() && t.size(0) == k_pool.size(0) &&
+                t.size(1) == k_pool.size(1), "mix_turn_prep: pools");
+  for (const at::Tensor& t : {freq, vfreq}) TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kDouble && t.is_contiguous());
+  const int64_t T = p.size(0), G = k_pool.size(1), kw = k_pool.size(3), vw = v_pool.size(3), rd = 2 * freq.numel(), cols = (heads + G) * dim + G * vdim;
+  TORCH_CHECK(p.size(1) >= cols && G >= 1 && heads % G == 0 && 2 * vfreq.numel() == vdim, "mix_turn_prep: sizes");
+  c10::cuda::CUDAGuard g(p.device());
+  at::Tensor q = at::empty({T, heads, kw}, p.options()), k = at::empty({want_kv ? T : 0, G, kw}, p.options()), v = at::empty({want_kv ? T : 0, G, vw}, p.options());
+  check(prl_mix_turn_rows(p.data_ptr(), p.stride(0), vecf(bias, cols, "bias"), freq.data_ptr<double>(), vfreq.data_ptr<double>(), veci<int64_t>(pos, T, "pos"),
+                          veci<int64_t>(kvslot, T, "kvslot"), q.data_ptr(), want_kv ? k.data_ptr() : nullptr, want_kv ? v.data_ptr() : nullptr, k_pool.data_ptr(),
+                          v_pool.data_ptr(), T, heads, G, dim, vdim, rd, kw, vw, static_cast<float>(eps), dt, cur_stream()), "mix_turn_prep");
+  return {q, k, v};
+}
+// o [T, H, vw] turned back, times scale * sigmoid(gate) -> out [T, H * vdim]
+void mix_turn_back(const at::Tensor& o, const at::Tensor& gate, const at::Tensor& vfreq, const at::Tensor& pos, double scale, at::Tensor out) {
+  const int dt = dt_of(o, "mix_turn_back");
+  rows2(gate, "mix_turn_back gate"); rows2(out, "mix_turn_back out");
+  const int64_t T = o.size(0), H = o.size(1), V = 2 * vfreq.numel();
+  TORCH_CHECK(o.dim() == 3 && o.is_contiguous() && o.size(2) >= V && gate.scalar_type() == o.scalar_type() && out.scalar_type() == o.scalar_type() && out.is_cuda() &&
+              gate.size(0) == T && gate.size(1) == H * V && out.size(0) == T && out.size(1) == H * V, "mix_turn_back: shapes");
+  TORCH_CHECK(vfreq.is_cuda() && vfreq.scalar_type() == at::kDouble && vfreq.is_contiguous());
+  c10::cuda::CUDAGuard g(o.device());
+  check(prl_mix_turn_back(o.data_ptr(), gate.data_ptr(), gate.stride(0), vfreq.data_ptr<double>(), veci<int64_t>(pos, T, "pos"), static_cast<float>(scale),
+                          out.data_ptr(), out.stride(0), T, H, V, o.size(2), dt, cur_stream()), "mix_turn_back");
+}
+void sink_pools(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table, const char* what) {
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && k_pool.dim() == 4 && k_pool.size(3) == q.size(2), what, ": q [rows, heads, key width]");
+  for (const at::Tensor& t : {k_pool, v_pool})
+    TORCH_CHECK(t.is_cuda() && t.dim() == 4 && t.size(2) == 16 && t.is_contiguous() && t.scalar_type() == q.scalar_type() && t.size(0) == k_pool.size(0) &&
+                t.size(1) == k_pool.size(1), what, ": pools");
+  TORCH_CHECK(k_pool.size(1) >= 1 && q.size(1) % k_pool.size(1) == 0, what, ": heads");
+  TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.dim() == 2 && table.stride(1) == 1, what, ": table");
+}
+// paged, any widths: q [R, H, D] -> [R, H, V]
+at::Tensor mix_sink_attention(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table, const c10::optional<at::Tensor>& seq_of,
+                              const at::Tensor& kv_len, double scale, const c10::optional<at::Tensor>& sink) {
+  const int dt = dt_of(q, "mix_sink_attention");
+  sink_pools(q, k_pool, v_pool, table, "mix_sink_attention");
+  const int64_t R = q.size(0);
+  TORCH_CHECK(seq_of.has_value() || table.size(0) >= R);
+  prl::SinkParams p{};
+  p.q = q.data_ptr(); p.k_pool = k_pool.data_ptr(); p.v_pool = v_pool.data_ptr();
+  p.table = table.data_ptr<int32_t>(); p.ld_table = table.stride(0);
+  p.seq_of = seq_of.has_value() ? veci<int32_t>(*seq_of, R, "seq_of") : nullptr;
+  p.kv_len = veci<int32_t>(kv_len, R, "kv_len");
+  p.R = R; p.H = q.size(1); p.G = k_pool.size(1); p.D = q.size(2); p.V = v_pool.size(3);
+  p.sink = vecf(sink, p.H, "sink");
+  p.scale = static_cast<float>(scale);
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty({R, p.H, p.V}, q.options());
+  p.out = out.data_ptr();
+  check(prl_mix_sink(&p, dt, cur_stream()), "mix_sink_attention");
+  return out;
+}
+// single tokens on the tensor cores (bf16): widths and heads of prl_sink_decode
+at::Tensor sink_decode(const at::Tensor& q, const at::Tensor& k_pool, const at::Tensor& v_pool, const at::Tensor& table, const at::Tensor& kv_len, double scale,
+                       int64_t splits, const at::Tensor& sink) {
+  CHECK_BF16(q);
+  sink_pools(q, k_pool, v_pool, table, "sink_decode");
+  const int64_t R = q.size(0), H = q.size(1), G = k_pool.size(1), kw = q.size(2), vw = v_pool.size(3);
+  TORCH_CHECK(table.size(0) >= R && splits >= 1, "sink_decode: sizes");
+  c10::cuda::CUDAGuard g(q.device());
+  at::Tensor out = at::empty({R, H, vw}, q.options());
+  at::Tensor work = at::empty({prl_paged_decode_workspace_floats(R, H, vw, splits)}, q.options().dtype(at::kFloat));
+  check(prl_sink_decode(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), table.data_ptr<int32_t>(), table.stride(0), veci<int32_t>(kv_len, R, "kv_len"), R, H, G,
+                        kw, vw, static_cast<float>(scale), splits, vecf(sink, H, "sink"), work.data_ptr<float>(), out.data_ptr(), cur_stream()), "sink_decode");
+  return out;
+}
+
 // ---------------------------------------------------------------------------------------------- experts
 // logits [T, E] -> (experts [T, top], scores, ranks, plan); counter: >= E + 1 zeros, left zero
-std::vector<at::Tensor> mix_route(const at::Tensor& logits, int64_t top, at::Tensor counter) {
+std::vector<at::Tensor> mix_route(const at::Tensor& logits, int64_t top, at::Tensor counter, bool softmax) {
   CHECK_F32(logits);
   rows2(logits, "mix_route logits");
   const int64_t T = logits.size(0), E = logits.size(1);
@@ -635,11 +824,11 @@ std::vector<at::Tensor> mix_route(const at::Tensor& logits, int64_t top, at::Ten
   at::Tensor pick = at::empty({T, top}, i32), score = at::empty({T, top}, logits.options()), rank = at::empty({T, top}, i32);
   at::Tensor plan = at::empty({1 + E + prl_mix_route_tiles(T * top, E)}, i32);
   check(prl_mix_route(logits.data_ptr<float>(), logits.stride(0), T, E, top, pick.data_ptr<int32_t>(), score.data_ptr<float>(), rank.data_ptr<int32_t>(),
-                      counter.data_ptr<int32_t>(), plan.data_ptr<int32_t>(), cur_stream()), "mix_route");
+                      counter.data_ptr<int32_t>(), plan.data_ptr<int32_t>(), softmax, cur_stream()), "mix_route");
   return {pick, score, rank, plan};
 }
 // -> (rows in the experts' order [tiles * 128, W], place of every (token, choice))
-std::vector<at::Tensor> mix_expert_rows(const at::Tensor& h, const at::Tensor& pick, const at::Tensor& score, const at::Tensor& rank, const at::Tensor& plan,
+std::vector<at::Tensor> mix_expert_rows(const at::Tensor& h, const at::Tensor& pick, const c10::optional<at::Tensor>& score, const at::Tensor& rank, const at::Tensor& plan,
                                         int64_t experts) {
   const int dt = dt_of(h, "mix_expert_rows");
   rows2(h, "mix_expert_rows h");
@@ -663,8 +852,8 @@ at::Tensor mix_expert_gemm(const at::Tensor& x, const at::Tensor& w, const at::T
                             cur_stream()), "mix_expert_gemm");
   return out;
 }
-// the same on tcgen05 (bf16); glu: w holds gate and up rows in blocks of 128, the result is silu(gate) * up
-at::Tensor gemm_experts(const at::Tensor& x, const at::Tensor& w, const at::Tensor& plan, int64_t experts, bool glu) {
+// the same on tcgen05 (bf16); glu: w holds gate and up rows in blocks of 128, the result is silu(gate) * up (1) or the clamped gate (2)
+at::Tensor gemm_experts(const at::Tensor& x, const at::Tensor& w, const at::Tensor& plan, int64_t experts, int64_t glu, double limit, double alpha) {
   CHECK_BF16(x); CHECK_BF16(w);
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w.dim() == 2 && w.is_contiguous() && w.size(1) == x.size(1) && x.size(0) % 128 == 0 && experts >= 1 &&
               w.size(0) % experts == 0 && x.size(1) % 8 == 0, "gemm_experts: shapes");
@@ -672,7 +861,7 @@ at::Tensor gemm_experts(const at::Tensor& x, const at::Tensor& w, const at::Tens
   c10::cuda::CUDAGuard g(x.device());
   at::Tensor out = at::empty({x.size(0), glu ? N / 2 : N}, x.options());
   check(prl_gemm_experts_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), veci<int32_t>(plan, 1 + experts + tiles, "plan"), tiles, experts, N, x.size(1), glu,
-                              cur_stream()), "gemm_experts");
+                              static_cast<float>(limit), static_cast<float>(alpha), cur_stream()), "gemm_experts");
   return out;
 }
 
@@ -832,18 +1021,28 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mix_window_attention", &mix_window_attention);
   m.def("gemm_clamped_glu", &gemm_clamped_glu);
   m.def("mix_clamped_glu", &mix_clamped_glu);
-  m.def("gemm_gelu", &gemm_gelu);
-  m.def("mix_gelu_", &mix_gelu_);
+  m.def("gemm_gelu", [](const at::Tensor& a, const at::Tensor& w) { return gemm_act(a, w, false); });
+  m.def("gemm_silu", [](const at::Tensor& a, const at::Tensor& w) { return gemm_act(a, w, true); });
+  m.def("mix_gelu_", [](at::Tensor x) { mix_act_(x, false); });
+  m.def("mix_silu_", [](at::Tensor x) { mix_act_(x, true); });
+  m.def("mix_streams_embed", &mix_streams_embed);
+  m.def("mix_streams_add", &mix_streams_add);
+  m.def("mix_selective", &mix_selective);
+  m.def("mix_turn_prep", &mix_turn_prep);
+  m.def("mix_turn_back", &mix_turn_back);
+  m.def("mix_sink_attention", &mix_sink_attention);
+  m.def("sink_decode", &sink_decode);
   m.def("gemm_swiglu", &gemm_swiglu);
   m.def("mix_silu_glu", &mix_silu_glu);
   m.def("mix_poly_norm", &mix_poly_norm);
   m.def("mix_block_embed", &mix_block_embed);
   m.def("mix_block_add", &mix_block_add);
   m.def("mix_input_conv", &mix_input_conv);
-  m.def("mix_route", &mix_route);
+  m.def("mix_route", &mix_route, py::arg("logits"), py::arg("top"), py::arg("counter"), py::arg("softmax") = false);
   m.def("mix_expert_rows", &mix_expert_rows);
   m.def("mix_expert_gemm", &mix_expert_gemm);
-  m.def("gemm_experts", &gemm_experts);
+  m.def("gemm_experts", &gemm_experts, py::arg("x"), py::arg("w"), py::arg("plan"), py::arg("experts"), py::arg("glu"), py::arg("limit") = 0.0,
+        py::arg("alpha") = 0.0);
   m.def("mix_map_prep", &mix_map_prep);
   m.def("mix_map_attention", &mix_map_attention);
   m.def("map_attn_fwd", &map_attn_fwd);

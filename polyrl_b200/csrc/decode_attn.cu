@@ -42,8 +42,8 @@ __global__ void __launch_bounds__(kAttnWarps * 32, MINB)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [num_seqs, nq * DK / QM] (row pitch ldq)
                     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                     const int32_t* __restrict__ block_table, int64_t ld_bt, const int32_t* __restrict__ seq_lens,
-                    int nq, int nkv, int splits, float scale_log2, int window, int keep_first, float* __restrict__ o_part,
-                    float* __restrict__ ml_part, __nv_bfloat16* __restrict__ out_direct, int64_t ldo) {
+                    int nq, int nkv, int splits, float scale_log2, int window, int keep_first, const float* __restrict__ sink,
+                    float* __restrict__ o_part, float* __restrict__ ml_part, __nv_bfloat16* __restrict__ out_direct, int64_t ldo) {
   static_assert(DK % 64 == 0 && DV % 64 == 0, "row widths must be multiples of 64");
   constexpr int KC = DK / 32;    // 32-wide d chunks for QK (two MMAs each)
   constexpr int DB = DV / 64;    // 64-wide d blocks for PV (eight n-tiles each)
@@ -226,6 +226,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
       ll += sm_l[w][g] * f;
     }
     const int head = kvh * G + g;
+    if (out_direct && sink && ll > 0.f) ll += exp2f(sink[head] * 1.4426950408889634f - mm);
     if (out_direct) {        // single split: normalise and write the final bf16 output here (no merge kernel)
       out_direct[static_cast<int64_t>(seq) * ldo + head * DV + dcol] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
       continue;
@@ -239,7 +240,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int64_t ldq,     // [nu
 // merge splits -> bf16 output [num_seqs, nq*D]
 template <int D>
 __global__ void decode_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part, int splits,
-                                    __nv_bfloat16* __restrict__ out, int64_t ldo, int nq) {
+                                    const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int64_t ldo, int nq) {
   const int seq = blockIdx.x / nq, head = blockIdx.x % nq;
   const int64_t base = (static_cast<int64_t>(seq) * nq + head) * splits;
   float mm = -INFINITY;
@@ -249,6 +250,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ o_part, const floa
     const float m = ml_part[(base + s) * 2];
     ll += (m == -INFINITY) ? 0.f : ml_part[(base + s) * 2 + 1] * exp2f(m - mm);
   }
+  if (sink && ll > 0.f) ll += exp2f(sink[head] * 1.4426950408889634f - mm);
   const float inv = ll > 0.f ? 1.f / ll : 0.f;
   for (int dcol = threadIdx.x; dcol < D; dcol += blockDim.x) {
     float acc = 0.f;
@@ -324,20 +326,49 @@ extern "C" int prl_paged_decode(const void* q, int64_t ldq, const void* k_cache,
     auto kern = minb >= 4 ? paged_decode_kernel<128, 128, 1, 4> : paged_decode_kernel<128, 128, 1, 3>;
     kern<<<grid, kAttnWarps * 32, 0, s>>>(
         static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(k_cache),
-        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, o_part,
+        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, nullptr, o_part,
         ml_part, splits == 1 ? static_cast<__nv_bfloat16*>(out) : nullptr, ldo);
     if (splits > 1)
-      decode_merge_kernel<128><<<num_seqs * nq, 128, 0, s>>>(o_part, ml_part, splits, static_cast<__nv_bfloat16*>(out), ldo, nq);
+      decode_merge_kernel<128><<<num_seqs * nq, 128, 0, s>>>(o_part, ml_part, splits, nullptr, static_cast<__nv_bfloat16*>(out), ldo, nq);
   } else if (d == 64) {
     paged_decode_kernel<64, 64, 1, 3><<<grid, kAttnWarps * 32, 0, s>>>(
         static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(k_cache),
-        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, o_part,
+        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, keep_first, nullptr, o_part,
         ml_part, splits == 1 ? static_cast<__nv_bfloat16*>(out) : nullptr, ldo);
     if (splits > 1)
-      decode_merge_kernel<64><<<num_seqs * nq, 64, 0, s>>>(o_part, ml_part, splits, static_cast<__nv_bfloat16*>(out), ldo, nq);
+      decode_merge_kernel<64><<<num_seqs * nq, 64, 0, s>>>(o_part, ml_part, splits, nullptr, static_cast<__nv_bfloat16*>(out), ldo, nq);
   } else {
     return -31;
   }
+  PRL_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// widths kw, vw of cached keys and values: 64 or 128 (kw = 192: vw = 128), up to 16 query heads per key head; sink [nq]: exp(sink) is added to the
+// denominator.  q:[num_seqs, nq * kw] contiguous, out [num_seqs, nq * vw]
+extern "C" int prl_sink_decode(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_table, int64_t ld_bt, const int32_t* seq_lens,
+                               int num_seqs, int nq, int nkv, int kw, int vw, float sm_scale, int splits, const float* sink, float* workspace, void* out,
+                               cudaStream_t s) {
+  if (num_seqs <= 0) return 0;
+  if (nkv < 1 || nq % nkv != 0 || nq / nkv > 16) return -30;
+  if (splits < 1) splits = 1;
+  float* ml_part = workspace + static_cast<int64_t>(num_seqs) * nq * splits * vw;
+  __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
+#define PRL_SINK_DECODE(DK, DV)                                                                                                                       \
+  do {                                                                                                                                                \
+    paged_decode_kernel<DK, DV, 1, DK == 192 ? 2 : 3><<<num_seqs * nkv * splits, kAttnWarps * 32, 0, s>>>(                                              \
+        static_cast<const __nv_bfloat16*>(q), static_cast<int64_t>(nq) * DK, static_cast<const __nv_bfloat16*>(k_cache),                               \
+        static_cast<const __nv_bfloat16*>(v_cache), block_table, ld_bt, seq_lens, nq, nkv, splits, sm_scale * 1.4426950408889634f, 0x7fffffff, 0, sink, \
+        workspace, ml_part, splits == 1 ? o : nullptr, static_cast<int64_t>(nq) * DV);                                                                  \
+    if (splits > 1) decode_merge_kernel<DV><<<num_seqs * nq, DV, 0, s>>>(workspace, ml_part, splits, sink, o, static_cast<int64_t>(nq) * DV, nq);       \
+  } while (0)
+  if (kw == 64 && vw == 64) PRL_SINK_DECODE(64, 64);
+  else if (kw == 64 && vw == 128) PRL_SINK_DECODE(64, 128);
+  else if (kw == 128 && vw == 64) PRL_SINK_DECODE(128, 64);
+  else if (kw == 128 && vw == 128) PRL_SINK_DECODE(128, 128);
+  else if (kw == 192 && vw == 128) PRL_SINK_DECODE(192, 128);
+  else return -31;
+#undef PRL_SINK_DECODE
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
@@ -359,7 +390,7 @@ extern "C" int prl_map_decode(const void* q, const void* k_cache, const void* v_
 #define PRL_MAP_DECODE(DK, DV, QM)                                                                                                                       \
   paged_decode_kernel<DK, DV, QM, 3><<<grid, kAttnWarps * 32, 0, s>>>(                                                                                    \
       static_cast<const __nv_bfloat16*>(q), nq * 64, static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache), block_table, \
-      ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, 0, workspace, ml_part, nullptr, 0)
+      ld_bt, seq_lens, nq, nkv, splits, scale_log2, window, 0, nullptr, workspace, ml_part, nullptr, 0)
   if (kw == 32 && vw == 64) PRL_MAP_DECODE(64, 64, 1);
   else if (kw == 32) PRL_MAP_DECODE(64, 128, 1);
   else if (vw == 64) PRL_MAP_DECODE(128, 64, 2);

@@ -61,16 +61,21 @@ struct TmaStoreParams {
 };
 struct EpiTmaStore {
   using Params = TmaStoreParams;
-  static constexpr bool kGelu = false;
+  static constexpr int kAct = 0;
 };
 // same with gelu (tanh form) on the accumulators, in the exactly equivalent shape z * sigmoid(2 u)
 struct EpiTmaStoreGelu {
   using Params = TmaStoreParams;
-  static constexpr bool kGelu = true;
+  static constexpr int kAct = 1;
+};
+struct EpiTmaStoreSilu {
+  using Params = TmaStoreParams;
+  static constexpr int kAct = 2;
 };
 __device__ __forceinline__ float gelu_fast(float z) {
   return __fdividef(z, 1.0f + __expf(fminf(-1.5957691216057308f * (z + 0.044715f * z * z * z), 80.f)));
 }
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(fminf(-z, 80.f))); }
 
 template <class Cfg, class Epi>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kNumThreads, 1)
@@ -245,9 +250,10 @@ gemm2_sm100_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
                 }
               }
             }
-            if constexpr (Epi::kGelu) {
+            if constexpr (Epi::kAct != 0) {
 #pragma unroll
-              for (int j = 0; j < 64; ++j) r[j] = __float_as_uint(gelu_fast(__uint_as_float(r[j])));
+              for (int j = 0; j < 64; ++j)
+                r[j] = __float_as_uint(Epi::kAct == 1 ? gelu_fast(__uint_as_float(r[j])) : silu_fast(__uint_as_float(r[j])));
             }
             // row `lane` of the 32 x 64 box: 8 x 16 B chunks, chunk j lands at (j ^ (lane & 7)) (128B swizzle)
             const uint32_t row_base = smem_u32(buf) + lane * 128;

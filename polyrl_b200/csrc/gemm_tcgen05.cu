@@ -140,12 +140,13 @@ struct EpiClampedGlu {
   }
 };
 
-// H[M, N] = gelu(acc)
+// H[M, N] = gelu(acc) or silu(acc)
 struct GeluParams {
   __nv_bfloat16* H;
   int64_t ldh;
 };
-struct EpiGelu {
+template <bool SILU>
+struct EpiAct {
   using Params = GeluParams;
   __device__ __forceinline__ void begin(const Params&, int, int, const WorkInfo&) {}
   __device__ __forceinline__ void end(const Params&, int, int, const WorkInfo&) {}
@@ -159,7 +160,7 @@ struct EpiGelu {
       if (row >= M || valid <= 0) continue;
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        v[i] = gelu_fast(v[i]);
+        v[i] = SILU ? silu_fast(v[i]) : gelu_fast(v[i]);
       }
       store_row_chunk(p.H + static_cast<int64_t>(row) * p.ldh + n0 + c, v, valid);
     }
@@ -268,28 +269,38 @@ extern "C" int prl_gemm_clamped_glu_bf16(const void* A, const void* Wgu, void* H
   return launch_gemm<Cfg, EpiClampedGlu, NoGate, false>(A, Wgu, M, N2, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);
 }
 
-// H = gelu_tanh(A·W^T)
-extern "C" int prl_gemm_gelu_bf16(const void* A, const void* W, void* H, int M, int N, int K, int64_t lda, int64_t ldw, int64_t ldh,
-                                  cudaStream_t stream) {
+// H = gelu_tanh(A·W^T), or silu of it
+template <bool SILU>
+static int run_act(const void* A, const void* W, void* H, int M, int N, int K, int64_t lda, int64_t ldw, int64_t ldh, cudaStream_t stream) {
+  using EpiTma = std::conditional_t<SILU, EpiTmaStoreSilu, EpiTmaStoreGelu>;
   GeluParams sp{static_cast<__nv_bfloat16*>(H), ldh};
   if (M > kBlockM && N > 128) {
     using Cfg2 = Gemm2Cfg<256, false, false, true>;
-    return launch_gemm2<Cfg2, EpiTmaStoreGelu>(A, W, H, M, N, K, lda * 2, ldw * 2, ldh * 2, TmaStoreParams{nullptr, 0}, 0, stream);
+    return launch_gemm2<Cfg2, EpiTma>(A, W, H, M, N, K, lda * 2, ldw * 2, ldh * 2, TmaStoreParams{nullptr, 0}, 0, stream);
   }
   using Cfg = GemmCfg<64, 2>;
-  return launch_gemm<Cfg, EpiGelu, NoGate, false>(A, W, M, N, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);
+  return launch_gemm<Cfg, EpiAct<SILU>, NoGate, false>(A, W, M, N, K, lda * 2, ldw * 2, sp, NoGate::Params{}, 0, 0, stream);
+}
+extern "C" int prl_gemm_gelu_bf16(const void* A, const void* W, void* H, int M, int N, int K, int64_t lda, int64_t ldw, int64_t ldh, int silu,
+                                  cudaStream_t stream) {
+  return silu ? run_act<true>(A, W, H, M, N, K, lda, ldw, ldh, stream) : run_act<false>(A, W, H, M, N, K, lda, ldw, ldh, stream);
 }
 
 // rows of D = A · (weight of the rows' group)^T for 128-row tiles sorted by group.  A:[tiles * 128, K], W:[groups * N, K], contiguous.  glu: W holds gate
-// and up rows in blocks of 128, D:[., N / 2] = silu(gate) * up
-extern "C" int prl_gemm_experts_bf16(const void* A, const void* W, void* D, const int32_t* plan, int tiles, int groups, int N, int K, int glu,
-                                     cudaStream_t stream) {
+// and up rows in blocks of 128, D:[., N / 2] = silu(gate) * up (glu = 1) or the clamped gate with limit and alpha (glu = 2)
+extern "C" int prl_gemm_experts_bf16(const void* A, const void* W, void* D, const int32_t* plan, int tiles, int groups, int N, int K, int glu, float limit,
+                                     float alpha, cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (N <= 0 || K <= 0 || K % 8 || groups < 1 || static_cast<int64_t>(groups) * N > 0x7fffffff) return -12;
   const int M = tiles * kBlockM;
   const bool few = tiles < 4 * groups;              // mostly tiles with a few rows: weights are streamed, the rows in use beside them
   if (glu) {
     if (N % 256) return -11;
+    if (glu == 2) {
+      ClampedGluParams cp{static_cast<__nv_bfloat16*>(D), N / 2, limit, alpha};
+      return few ? run_grouped<256, EpiClampedGlu, 32>(A, W, cp, plan, M, groups, N, K, stream)
+                 : run_grouped<256, EpiClampedGlu, kBlockM>(A, W, cp, plan, M, groups, N, K, stream);
+    }
     SwigluParams sp{static_cast<__nv_bfloat16*>(D), nullptr, N / 2, 0};
     return few ? run_grouped<256, EpiSwiglu, 32>(A, W, sp, plan, M, groups, N, K, stream)
                : run_grouped<256, EpiSwiglu, kBlockM>(A, W, sp, plan, M, groups, N, K, stream);

@@ -1,7 +1,7 @@
 // polyrl_b200 — gated linear recurrences over prompt portions, chunk-parallel on the tensor cores (bf16 activations).
 //
 // Same recurrences as mix_scan.cu, 64 tokens at a time.  With La the running sum of log keep inside the chunk,
-//     kSsd    weight(t, s) = exp(La_t - La_s) dt_s,       carry-in factor exp(La_t)
+//     kSsd    weight(t, s) = exp(La_t - La_s) dt_s,       carry-in factor exp(La_t);  kDecay the same with dt = 1
 //     kMlstm  F = running sum of f,  g_s = i_s - F_s,  M_t = max(m_0, max_{s <= t} g_s),  m_t = F_t + M_t:
 //             weight(t, s) = exp(g_s - M_t),               carry-in factor exp(m_0 - M_t)
 // so that  y_t = sum_{s <= t} weight(t, s) (q_t . k_s) v_s + carry_t S_0^T q_t  and the state after the chunk is
@@ -144,10 +144,13 @@ mix_chunk_kernel(ScanParams p, int vec) {
       for (int e = 0; e < 2; ++e) {
         const int t = lane + 32 * e;
         la[e] = 0.f;
-        ad[e] = MODE == kSsd ? 0.f : -INFINITY;
+        ad[e] = MODE == kMlstm ? -INFINITY : 0.f;
         if (t < nv) {
           const int64_t r = static_cast<int64_t>(t0 + c0 + t) * p.ldg + h;
-          if (MODE == kSsd) {
+          if (MODE == kDecay) {
+            ad[e] = 1.f;
+            la[e] = p.a_log[h];
+          } else if (MODE == kSsd) {
             ad[e] = softplus_f(p.g0[r] + b0);
             la[e] = a_neg * ad[e];
           } else {
@@ -163,7 +166,7 @@ mix_chunk_kernel(ScanParams p, int vec) {
       }
       la[1] += __shfl_sync(0xffffffffu, la[0], 31);
       const float la_end = __shfl_sync(0xffffffffu, la[1], 31);
-      if (MODE == kSsd) {
+      if (MODE != kMlstm) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int t = lane + 32 * e;
@@ -427,5 +430,6 @@ extern "C" int prl_mix_chunk_supported(int N) { return N <= 256; }
 extern "C" int prl_mix_chunk(const ScanParams* p, int mode, cudaStream_t st) {
   if (p->spans <= 0) return 0;
   if (p->spans > 65535 || p->H > 65535 || p->N > 256) return -210;
-  return mode == kSsd ? pick_chunk<kSsd>(*p, st) : pick_chunk<kMlstm>(*p, st);
+  if (mode != kSsd && mode != kMlstm && mode != kDecay) return -211;
+  return mode == kSsd ? pick_chunk<kSsd>(*p, st) : mode == kDecay ? pick_chunk<kDecay>(*p, st) : pick_chunk<kMlstm>(*p, st);
 }

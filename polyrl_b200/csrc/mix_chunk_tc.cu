@@ -62,21 +62,24 @@ __device__ __forceinline__ void tc_raw(TcRaw& g, const ScanParams& p, int64_t t0
   for (int e = 0; e < 4; ++e) {
     const int t = 4 * lane + e;
     const bool ok = t < nv;
-    g.a[e] = ok ? p.g0[(t0 + t) * p.ldg + h] : 0.f;
+    g.a[e] = ok && MODE != kDecay ? p.g0[(t0 + t) * p.ldg + h] : 0.f;
     g.b[e] = (ok && MODE == kMlstm) ? p.g1[(t0 + t) * p.ldg + h] : 0.f;
   }
 }
 // one warp: weights of the chunk.  weight(t, s) = 2^(row_t + col_s) mul_s (qscale folded into row), carry: carried-in factor with
 // qscale, wgt: weight of a token in the chunk's final state
 template <int MODE>
-__device__ __forceinline__ void tc_gates(TcGates& sm, float& m_run, const TcRaw& g, const ScanParams& p, int nv, float b0, float b1, float a_neg, int lane) {
+__device__ __forceinline__ void tc_gates(TcGates& sm, float& m_run, const TcRaw& g, const ScanParams& p, int nv, int h, float b0, float b1, float a_neg, int lane) {
   constexpr float kL2e = 1.4426950408889634f;
   const float lq = log2f(p.qscale);
   float la[4], ad[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     const bool ok = 4 * lane + e < nv;
-    if (MODE == kSsd) {
+    if (MODE == kDecay) {
+      ad[e] = ok ? 1.f : 0.f;
+      la[e] = ok ? p.a_log[h] : 0.f;
+    } else if (MODE == kSsd) {
       ad[e] = ok ? softplus_f(g.a[e] + b0) : 0.f;
       la[e] = a_neg * ad[e];
     } else {
@@ -95,7 +98,7 @@ __device__ __forceinline__ void tc_gates(TcGates& sm, float& m_run, const TcRaw&
   const float end = __shfl_sync(0xffffffffu, run, 31);
 #pragma unroll
   for (int e = 0; e < 4; ++e) la[e] += lane ? before : 0.f;
-  if (MODE == kSsd) {
+  if (MODE != kMlstm) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int t = 4 * lane + e;
@@ -219,7 +222,7 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
   if (w == 4) {          // rows 0..31, columns 64..127 of the scores: the warp whose share lies above the diagonal runs the gates, a chunk ahead
     if (MODE == kMlstm && lane == 0) sm.m = fresh ? 0.f : p.mst[slot * p.H + h];
     __syncwarp();
-    tc_gates<MODE>(sm.gate[0], sm.m, raw, p, min(kTcC, len), b0, b1, a_neg, lane);
+    tc_gates<MODE>(sm.gate[0], sm.m, raw, p, min(kTcC, len), h, b0, b1, a_neg, lane);
     if (len > kTcC) tc_raw<MODE>(raw, p, t0 + kTcC, min(kTcC, len - kTcC), h, lane);
   }
   tc_fence_before();
@@ -282,7 +285,7 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
     tc_fence_after();
     if (w == 4 && more) {
       const int c1 = c0 + kTcC;
-      tc_gates<MODE>(sm.gate[(ci + 1) & 1], sm.m, raw, p, min(kTcC, len - c1), b0, b1, a_neg, lane);
+      tc_gates<MODE>(sm.gate[(ci + 1) & 1], sm.m, raw, p, min(kTcC, len - c1), h, b0, b1, a_neg, lane);
       if (len > c1 + kTcC) tc_raw<MODE>(raw, p, t0 + c1 + kTcC, min(kTcC, len - c1 - kTcC), h, lane);
     }
     // ---- weighted scores of row r, columns [64 g, +64)
@@ -435,7 +438,7 @@ mix_chunk_tc_kernel(ScanParams p, int32_t* err) {
               const float2 x = unpack_bf16(q[e]);
               y0 += skip * x.x;
               y1 += skip * x.y;
-            } else {
+            } else if (MODE == kMlstm) {
               y0 *= inv;
               y1 *= inv;
             }
@@ -521,6 +524,8 @@ extern "C" int prl_mix_chunk_tc_ok(const ScanParams* p) {
 extern "C" int prl_mix_chunk_tc(const ScanParams* p, int mode, int32_t* err, cudaStream_t st) {
   if (p->spans <= 0) return 0;
   if (p->spans > 65535 || p->H > 65535 || !prl_mix_chunk_tc_ok(p)) return -240;
+  if (mode != kSsd && mode != kMlstm && mode != kDecay) return -241;
+  if (mode == kDecay) return p->N <= 128 ? run_tc<kDecay, 2>(*p, err, st) : run_tc<kDecay, 4>(*p, err, st);
   if (p->N <= 128) return mode == kSsd ? run_tc<kSsd, 2>(*p, err, st) : run_tc<kMlstm, 2>(*p, err, st);
   return mode == kSsd ? run_tc<kSsd, 4>(*p, err, st) : run_tc<kMlstm, 4>(*p, err, st);
 }

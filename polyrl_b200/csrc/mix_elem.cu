@@ -556,13 +556,14 @@ __global__ void mix_clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__
   }
 }
 
-template <class T, int VEC>
-__global__ void mix_gelu_kernel(T* __restrict__ x, int64_t n) {
+// x = gelu(x) or silu(x) in place
+template <class T, int VEC, bool SILU>
+__global__ void mix_act_kernel(T* __restrict__ x, int64_t n) {
   for (int64_t i = (static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x) * VEC; i < n; i += static_cast<int64_t>(gridDim.x) * blockDim.x * VEC) {
     float v[VEC];
     ld_vec<T, VEC>(x + i, v);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) v[j] = gelu_tanh_f(v[j]);
+    for (int j = 0; j < VEC; ++j) v[j] = SILU ? silu_f(v[j]) : gelu_tanh_f(v[j]);
     st_vec<T, VEC>(x + i, v);
   }
 }
@@ -758,12 +759,13 @@ extern "C" int prl_mix_clamped_glu(const void* gu, void* out, int64_t rows, int 
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
-extern "C" int prl_mix_gelu(void* x, int64_t n, int dtype, cudaStream_t st) {
+extern "C" int prl_mix_gelu(void* x, int64_t n, int silu, int dtype, cudaStream_t st) {
   if (n <= 0) return 0;
   const bool vec = n % 8 == 0 && al16(x);
   const int64_t blocks = (n / (vec ? 8 : 1) + 255) / 256;
   const unsigned grid = static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16);
-  MIX_DISPATCH(vec, (mix_gelu_kernel<T, VEC><<<grid > 0 ? grid : 1, 256, 0, st>>>(static_cast<T*>(x), n)));
+  if (silu) MIX_DISPATCH(vec, (mix_act_kernel<T, VEC, true><<<grid > 0 ? grid : 1, 256, 0, st>>>(static_cast<T*>(x), n)));
+  else MIX_DISPATCH(vec, (mix_act_kernel<T, VEC, false><<<grid > 0 ? grid : 1, 256, 0, st>>>(static_cast<T*>(x), n)));
   PRL_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

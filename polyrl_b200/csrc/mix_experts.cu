@@ -8,8 +8,9 @@
 namespace prl {
 
 constexpr int kMoeTile = 128;
-// a warp per token, `per` tokens per CTA: the `top` largest logits (ties: the lower index), s = sigmoid; counts [E + 1] are zero between launches
-template <int RN>
+// a warp per token, `per` tokens per CTA: the `top` largest logits (ties: the lower index); s = sigmoid, or the softmax over all experts divided by
+// the sum of the chosen ones (+ 1e-20); counts [E + 1] are zero between launches
+template <int RN, bool SOFTMAX>
 __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int top, int per, int32_t* __restrict__ pick,
                                                         float* __restrict__ score, int32_t* __restrict__ rank, int32_t* __restrict__ counts,
                                                         int32_t* __restrict__ plan) {
@@ -20,7 +21,7 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
   for (int i = warp; i < per; i += 8) {
     const int t = blockIdx.x * per + i;
     if (t >= T) break;
-    float v[RN];
+    float v[RN], top_v = 0.f, all = 0.f, chosen = 0.f;
     uint32_t taken = 0;
 #pragma unroll
     for (int r = 0; r < RN; ++r) {
@@ -28,6 +29,17 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
       v[r] = e < E ? logits[t * ld + e] : 0.f;
       if (!(v[r] == v[r])) v[r] = -INFINITY;
       if (e >= E) taken |= 1u << r;
+    }
+    if (SOFTMAX) {
+      top_v = -INFINITY;
+#pragma unroll
+      for (int r = 0; r < RN; ++r)
+        if (r * 32 + lane < E) top_v = fmaxf(top_v, v[r]);
+      top_v = warp_max(top_v);
+#pragma unroll
+      for (int r = 0; r < RN; ++r)
+        if (r * 32 + lane < E) all += expf(v[r] - top_v);
+      all = warp_sum(all);
     }
     for (int k = 0; k < top; ++k) {
       float bv = -INFINITY;
@@ -44,13 +56,17 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
         if (ov > bv || (ov == bv && oe < be)) { bv = ov; be = oe; }
       }
       if ((be & 31) == lane) taken |= 1u << (be >> 5);
+      const float s = SOFTMAX ? expf(bv - top_v) / all : sigmoid_f(bv);
+      chosen += s;
       if (lane == 0) {
         const int64_t at = static_cast<int64_t>(t) * top + k;
         pick[at] = be;
-        score[at] = sigmoid_f(bv);
+        score[at] = s;
         rank[at] = atomicAdd(&hist[be], 1);
       }
     }
+    if (SOFTMAX && lane == 0)
+      for (int k = 0; k < top; ++k) score[static_cast<int64_t>(t) * top + k] /= chosen + 1e-20f;
   }
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += 256)
@@ -95,7 +111,7 @@ __global__ void __launch_bounds__(256) mix_route_kernel(const float* __restrict_
   }
 }
 
-// rows[first row of the expert + rank] = score * h[t]
+// rows[first row of the expert + rank] = h[t], times its score where there are scores
 template <class T, int VEC>
 __global__ void __launch_bounds__(128) mix_expert_rows_kernel(const T* __restrict__ h, int64_t ldh, const int32_t* __restrict__ pick,
                                                               const float* __restrict__ score, const int32_t* __restrict__ rank,
@@ -108,7 +124,7 @@ __global__ void __launch_bounds__(128) mix_expert_rows_kernel(const T* __restric
     float v[VEC];
     ld_vec<T, VEC>(h + t * ldh + c, v);
     for (int k = 0; k < top; ++k) {
-      const float s = score[t * top + k];
+      const float s = score ? score[t * top + k] : 1.f;
       float y[VEC];
 #pragma unroll
       for (int i = 0; i < VEC; ++i) y[i] = v[i] * s;
@@ -164,11 +180,15 @@ extern "C" int prl_mix_route_tiles(int64_t rows, int64_t experts) {         // u
 }
 
 extern "C" int prl_mix_route(const float* logits, int64_t ld, int T, int E, int top, int32_t* pick, float* score, int32_t* rank, int32_t* counts, int32_t* plan,
-                             cudaStream_t st) {
+                             int softmax, cudaStream_t st) {
   if (T <= 0) return 0;
   if (E < 1 || E > 1024 || top < 1 || top > E) return -270;
   const int per = T <= 8 * 148 ? 8 : 32, grid = (T + per - 1) / per;
-#define MIX_RT(RN) mix_route_kernel<RN><<<grid, 256, E * 4, st>>>(logits, ld, T, E, top, per, pick, score, rank, counts, plan)
+#define MIX_RT(RN)                                                                                                                        \
+  do {                                                                                                                                    \
+    if (softmax) mix_route_kernel<RN, true><<<grid, 256, E * 4, st>>>(logits, ld, T, E, top, per, pick, score, rank, counts, plan);        \
+    else mix_route_kernel<RN, false><<<grid, 256, E * 4, st>>>(logits, ld, T, E, top, per, pick, score, rank, counts, plan);               \
+  } while (0)
   if (E <= 32) MIX_RT(1);
   else if (E <= 128) MIX_RT(4);
   else MIX_RT(32);

@@ -6,6 +6,8 @@
 //   kDelta (gated delta rule)                k' = k / |k|, q' = scale q / |q|,  S = keep S + k' u^T,  u = beta (v - keep S^T k'),  y = S^T q'
 //                                            with keep = exp(-exp(A_log) softplus(a + bias)), beta = sigmoid(b).  With S the state before the
 //                                            token, y = keep S^T q' + (k' . q') u, so one pass over S gives both products.
+//   kDecay (constant decay)                  S = e^a S + k v^T,  y = S^T q, a per head; single tokens may come ahead of their silu
+//   kGla   (decay per state row)             S = diag(keep) S + k v^T,  y = S^T q with keep = sigmoid(g + bias)^(1 / tau)
 //
 // mix_step_kernel (mix_delta_step_kernel for kDelta) serves spans of one token (decode): every state byte is read and written once, streaming.
 // mix_scan_kernel: one CTA = one (span, head, 32 value columns): lane = value column, warp w owns the state rows w, w + 8, ... in registers
@@ -17,11 +19,16 @@ namespace prl {
 constexpr int kScanWarps = 8;
 constexpr int kScanVT = 32;
 
+__device__ __forceinline__ float gla_keep(const ScanParams& p, int64_t t, int h, int n) {
+  const int64_t c = static_cast<int64_t>(h) * p.N + n;
+  return decay_f(logsigmoid_f(p.g0[t * p.ldg + c] + (p.b0 ? p.b0[c] : 0.f)) / p.cap);
+}
+
 template <class T, int MODE, int RN>
 __global__ void __launch_bounds__(kScanWarps * 32)
 mix_scan_kernel(ScanParams p) {
   constexpr int NMAX = RN * kScanWarps;
-  __shared__ float s_q[2][NMAX], s_k[2][NMAX], s_n[NMAX];
+  __shared__ float s_q[2][NMAX], s_k[2][NMAX], s_n[NMAX], s_w[MODE == kGla ? 2 : 1][MODE == kGla ? NMAX : 1];
   constexpr int ND = MODE == kDelta ? 3 : 1;
   __shared__ float s_red[2][kScanWarps][33], s_dot[2][ND][kScanWarps], s_red2[MODE == kDelta ? 2 : 1][kScanWarps][33];
   const int vt = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
@@ -50,8 +57,9 @@ mix_scan_kernel(ScanParams p) {
     if (!fresh) m = p.mst[hb];
     for (int n = tid; n < NMAX; n += kScanWarps * 32) s_n[n] = (!fresh && n < p.N) ? p.nst[hb * p.N + n] : 0.f;
   }
-  const float b0 = p.b0 ? p.b0[h] : 0.f, b1 = p.b1 ? p.b1[h] : 0.f;
-  const float a_neg = MODE != kMlstm ? -expf(p.a_log[h]) : 0.f;
+  const float b0 = MODE != kGla && p.b0 ? p.b0[h] : 0.f, b1 = p.b1 ? p.b1[h] : 0.f;
+  const float a_neg = MODE == kSsd || MODE == kDelta ? -expf(p.a_log[h]) : 0.f;
+  const float fixed = MODE == kDecay ? decay_f(p.a_log[h]) : 1.f;
   const float skip = (MODE == kSsd && p.d_skip) ? p.d_skip[h] : 0.f;
 
   for (int t = t0; t < t1; ++t) {
@@ -97,10 +105,14 @@ mix_scan_kernel(ScanParams p) {
     for (int n = tid; n < NMAX; n += kScanWarps * 32) {
       s_q[b][n] = n < p.N ? to_f<T>(q[static_cast<int64_t>(t) * p.ldq + n]) * p.qscale : 0.f;
       s_k[b][n] = n < p.N ? to_f<T>(k[static_cast<int64_t>(t) * p.ldk + n]) : 0.f;
+      if constexpr (MODE == kGla) s_w[b][n] = n < p.N ? gla_keep(p, t, h, n) : 1.f;
     }
     const float vv = col_ok ? to_f<T>(v[static_cast<int64_t>(t) * p.ldv + col]) : 0.f;
     float keep, add, floor_ = 0.f;
-    if constexpr (MODE == kSsd) {
+    if constexpr (MODE == kDecay || MODE == kGla) {
+      keep = fixed;
+      add = 1.f;
+    } else if constexpr (MODE == kSsd) {
       add = softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0);
       keep = expf(a_neg * add);
     } else {
@@ -118,7 +130,7 @@ mix_scan_kernel(ScanParams p) {
 #pragma unroll
     for (int i = 0; i < RN; ++i) {
       const int n = i * kScanWarps + w;
-      S[i] = keep * S[i] + av * s_k[b][n];
+      S[i] = (MODE == kGla ? s_w[b][n] : keep) * S[i] + av * s_k[b][n];
       acc += s_q[b][n] * S[i];
     }
     s_red[b][w][lane] = acc;
@@ -139,7 +151,7 @@ mix_scan_kernel(ScanParams p) {
       for (int i = 0; i < kScanWarps; ++i) y += s_red[b][i][lane];
       if constexpr (MODE == kSsd) {
         y += skip * vv;
-      } else {
+      } else if constexpr (MODE == kMlstm) {
         float d = 0.f;
 #pragma unroll
         for (int i = 0; i < kScanWarps; ++i) d += s_dot[b][0][i];
@@ -180,7 +192,7 @@ template <class T, int MODE, int CPL>
 __global__ void __launch_bounds__(kScanWarps * 32)
 mix_step_kernel(ScanParams p) {
   constexpr int U = 8;                                   // state rows in flight per warp
-  __shared__ float s_q[512], s_k[512], s_n[512];
+  __shared__ float s_q[512], s_k[512], s_n[512], s_w[MODE == kGla ? 512 : 1];
   __shared__ float s_red[kScanWarps][32 * CPL + 1], s_dot[kScanWarps];
   const int vt = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
   const int w = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
@@ -206,11 +218,15 @@ mix_step_kernel(ScanParams p) {
   const T* k = static_cast<const T*>(p.k) + static_cast<int64_t>(t) * p.ldk + static_cast<int64_t>(h / p.rep) * p.N;
   const T* v = static_cast<const T*>(p.v) + static_cast<int64_t>(t) * p.ldv + static_cast<int64_t>(h) * p.V;
   float vv[CPL];
+  auto act = [&](float x) { return MODE == kDecay && p.raw ? to_f<T>(from_f<T>(silu_f(x))) : x; };         // (rounded like an activated row)
 #pragma unroll
-  for (int c = 0; c < CPL; ++c) vv[c] = ok ? to_f<T>(v[col + c]) : 0.f;
+  for (int c = 0; c < CPL; ++c) vv[c] = ok ? act(to_f<T>(v[col + c])) : 0.f;
   float keep, add, floor_ = 0.f, m2 = 0.f;
-  const float b0 = p.b0 ? p.b0[h] : 0.f;
-  if constexpr (MODE == kSsd) {
+  const float b0 = MODE != kGla && p.b0 ? p.b0[h] : 0.f;
+  if constexpr (MODE == kDecay || MODE == kGla) {
+    keep = MODE == kDecay ? decay_f(p.a_log[h]) : 1.f;
+    add = 1.f;
+  } else if constexpr (MODE == kSsd) {
     add = softplus_f(p.g0[static_cast<int64_t>(t) * p.ldg + h] + b0);
     keep = expf(-expf(p.a_log[h]) * add);
   } else {
@@ -224,9 +240,10 @@ mix_step_kernel(ScanParams p) {
   }
   float dot = 0.f;
   for (int n = tid; n < p.N; n += kScanWarps * 32) {
-    const float qn = to_f<T>(q[n]) * p.qscale, kn = to_f<T>(k[n]);
+    const float qn = act(to_f<T>(q[n])) * p.qscale, kn = act(to_f<T>(k[n]));
     s_q[n] = qn;
     s_k[n] = kn;
+    if constexpr (MODE == kGla) s_w[n] = gla_keep(p, t, h, n);
     if constexpr (MODE == kMlstm) {
       const float nn = keep * (fresh ? 0.f : p.nst[hb * p.N + n]) + add * kn;
       s_n[n] = nn;
@@ -250,7 +267,7 @@ mix_step_kernel(ScanParams p) {
         const float ak = add * s_k[n], qn = s_q[n];
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
-          st[u][c] = keep * st[u][c] + ak * vv[c];
+          st[u][c] = (MODE == kGla ? s_w[n] : keep) * st[u][c] + ak * vv[c];
           acc[c] += qn * st[u][c];
         }
         if (ok) st_cols<CPL>(Sg + static_cast<int64_t>(n) * p.V, st[u]);
@@ -268,7 +285,7 @@ mix_step_kernel(ScanParams p) {
       for (int i = 0; i < kScanWarps; ++i) y += s_red[i][c];
       if constexpr (MODE == kSsd) {
         if (p.d_skip) y += p.d_skip[h] * to_f<T>(v[gc]);
-      } else {
+      } else if constexpr (MODE == kMlstm) {
         float d = 0.f;
 #pragma unroll
         for (int i = 0; i < kScanWarps; ++i) d += s_dot[i];
@@ -416,12 +433,14 @@ using namespace prl;
 template <class T>
 static int run_scan(const ScanParams& p, int mode, int single, cudaStream_t st) {
   if (mode == kDelta) return single ? launch_delta_step<T>(p, st) : launch_scan<T, kDelta>(p, st);
+  if (mode == kDecay) return single ? launch_step<T, kDecay>(p, st) : launch_scan<T, kDecay>(p, st);
+  if (mode == kGla) return single ? launch_step<T, kGla>(p, st) : launch_scan<T, kGla>(p, st);
   if (single) return mode == kSsd ? launch_step<T, kSsd>(p, st) : launch_step<T, kMlstm>(p, st);
   return mode == kSsd ? launch_scan<T, kSsd>(p, st) : launch_scan<T, kMlstm>(p, st);
 }
-// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm / kDelta; single: every span is one token
+// dtype: 0 = bf16, 1 = fp32 activations; mode: kSsd / kMlstm / kDelta / kDecay / kGla; single: every span is one token
 extern "C" int prl_mix_scan(const ScanParams* p, int mode, int dtype, int single, cudaStream_t st) {
   if (p->spans <= 0) return 0;
-  if (p->spans > 65535 || p->H > 65535) return -202;
+  if (p->spans > 65535 || p->H > 65535 || (p->raw && !(mode == kDecay && single))) return -202;
   return dtype == 0 ? run_scan<__nv_bfloat16>(*p, mode, single, st) : run_scan<float>(*p, mode, single, st);
 }

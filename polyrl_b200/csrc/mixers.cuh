@@ -105,7 +105,9 @@ inline bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) =
 //   kSsd    state-space duality: dt = softplus(g0 + b0), keep = exp(-exp(A_log) dt), add = dt;   y += D v
 //   kMlstm  matrix memory with a running maximum m and normaliser n (csrc/mix_scan.cu)
 //   kDelta  gated delta rule: unit k and q, the write corrects what the decayed state already answers for k (csrc/mix_scan.cu)
-enum : int { kSsd = 0, kMlstm = 1, kDelta = 2 };
+//   kDecay  constant decay per head: keep = exp(a_log), add = 1
+//   kGla    a decay for every state row: keep_n = sigmoid(g0_n + b0_n)^(1 / cap), add = 1
+enum : int { kSsd = 0, kMlstm = 1, kDelta = 2, kDecay = 3, kGla = 4 };
 constexpr float kUnitEps = 1e-6f;        // under the root of a unit vector's norm
 
 // n and m are read by every value tile of a head and may be overwritten only after the last tile has read them: the last
