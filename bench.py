@@ -55,7 +55,7 @@ def parse():
     ap.add_argument("--workload", default="ppo", choices=["ppo", "serving"],
                     help="ppo: the flagship step (default); serving: prefill / decode throughput of a mixer stack beside the closest "
                          "models of equal size (random weights, one GPU)")
-    ap.add_argument("--serving-design", default="ludesun", choices=["ludesun", "lanilix", "mabedra"], help="mixer stack of --workload serving")
+    ap.add_argument("--serving-design", default="ludesun", choices=["ludesun", "lanilix", "mabedra", "dubazen"], help="mixer stack of --workload serving")
     ap.add_argument("--serving-layers", type=int, default=16)
     ap.add_argument("--kernels", action="store_true", help="with --workload serving: time the single kernels against their rooflines instead")
     ap.add_argument("--comm", default=os.environ.get("BENCH_COMM", "p2p"), choices=["p2p", "nccl"])

@@ -57,6 +57,11 @@ int prl_mix_chunk_tc(const prl::ScanParams*, int, int32_t*, cudaStream_t);
 int prl_mix_latent(const prl::LatentParams*, int, int, cudaStream_t);
 int prl_mix_window(const prl::WindowParams*, int, cudaStream_t);
 int prl_mix_block(const prl::BlockParams*, int, cudaStream_t);
+int prl_mix_gla_ok(const prl::ScanParams*);
+int64_t prl_mix_gla_chunks(int64_t, int64_t);
+int64_t prl_mix_gla_work_bytes(int);
+int64_t prl_mix_gla_keep_floats(int);
+int prl_mix_gla(const prl::ScanParams*, int64_t, int64_t, void*, float*, int32_t*, cudaStream_t);
 int prl_mix_sink(const prl::SinkParams*, int, cudaStream_t);
 int prl_mix_selective(const prl::SelectiveParams*, int, int, cudaStream_t);
 int prl_mix_streams(const prl::StreamsParams*, int, cudaStream_t);
@@ -354,6 +359,22 @@ void mix_delta_chunk_(const at::Tensor& q, const at::Tensor& k, const at::Tensor
   at::Tensor work = at::empty({chunks * p.H * prl_mix_delta_work_bytes()}, v.options().dtype(at::kByte));
   at::Tensor gates = at::empty({chunks * p.H * prl_mix_delta_gate_floats()}, v.options().dtype(at::kFloat));
   check(prl_mix_delta(&p, v.size(0), chunks, work.data_ptr(), gates.data_ptr<float>(), p.counter + counter.numel() - 1, cur_stream()), "mix_delta_chunk");
+}
+
+// gated linear attention in chunks of 64 tokens (bf16); false: the layout is left to mix_scan_.  The last counter element is the error flag
+bool mix_gla_chunk_(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g0, const c10::optional<at::Tensor>& b0, double qscale, double tau,
+                    at::Tensor S, const at::Tensor& cu, const at::Tensor& start, const at::Tensor& slot, at::Tensor counter, at::Tensor out) {
+  if (dt_of(v, "mix_gla_chunk") != 0) return false;
+  prl::ScanParams p = scan_params(4, q, k, v, g0, c10::nullopt, b0, c10::nullopt, c10::nullopt, qscale, S, cu, start, slot, counter, out);
+  TORCH_CHECK(tau > 0);
+  p.cap = static_cast<float>(tau);
+  if (!prl_mix_gla_ok(&p)) return false;
+  c10::cuda::CUDAGuard g(v.device());
+  const int64_t chunks = prl_mix_gla_chunks(v.size(0), p.spans);
+  at::Tensor work = at::empty({chunks * p.H * prl_mix_gla_work_bytes(p.N)}, v.options().dtype(at::kByte));
+  at::Tensor keep = at::empty({chunks * p.H * prl_mix_gla_keep_floats(p.N)}, v.options().dtype(at::kFloat));
+  check(prl_mix_gla(&p, v.size(0), chunks, work.data_ptr(), keep.data_ptr<float>(), p.counter + counter.numel() - 1, cur_stream()), "mix_gla_chunk");
+  return true;
 }
 
 // a [T, qr + r + rd] -> (normed query latent [T, qr], packed cache rows [T, r + rd] or empty); cache rows also go to pool[kvslot]
@@ -1016,6 +1037,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mix_latent", &mix_latent);
   m.def("mix_delta_chunk_ok", &mix_delta_chunk_ok);
   m.def("mix_delta_chunk_", &mix_delta_chunk_);
+  m.def("mix_gla_chunk_", &mix_gla_chunk_);
   m.def("mix_qk_prep", &mix_qk_prep);
   m.def("mix_gather_keys", &mix_gather_keys);
   m.def("mix_window_attention", &mix_window_attention);

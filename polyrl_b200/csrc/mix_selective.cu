@@ -19,18 +19,6 @@ __device__ __forceinline__ float sel_decay(float x) {
   if constexpr (sizeof(T) == 2) return fast_exp2(x);         // x is scaled by log2 e already
   else return decay_f(x);
 }
-// softplus by log(1 + e) = 2 artanh(e / (2 + e)), e = exp(-|z|) <= 1: seven terms of the series, below 2e-8 relative
-__device__ __forceinline__ float softplus_series(float z) {
-  const float e = __expf(-fabsf(z)), s = __fdividef(e, 2.f + e), q = s * s;
-  float a = 1.f / 13.f;
-  a = a * q + 1.f / 11.f;
-  a = a * q + 1.f / 9.f;
-  a = a * q + 1.f / 7.f;
-  a = a * q + 1.f / 5.f;
-  a = a * q + 1.f / 3.f;
-  a = a * q + 1.f;
-  return fmaxf(z, 0.f) + 2.f * s * a;
-}
 template <class T>
 __device__ __forceinline__ float sel_softplus(float z) {
   if constexpr (sizeof(T) == 2) return softplus_series(z);

@@ -65,6 +65,18 @@ template <class T>
 __device__ __forceinline__ float silu_t(float z) { return z * sigmoid_t<T>(z); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float logsigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// softplus by log(1 + e) = 2 artanh(e / (2 + e)), e = exp(-|z|) <= 1: seven terms of the series, below 2e-8 relative
+__device__ __forceinline__ float softplus_series(float z) {
+  const float e = __expf(-fabsf(z)), s = __fdividef(e, 2.f + e), q = s * s;
+  float a = 1.f / 13.f;
+  a = a * q + 1.f / 11.f;
+  a = a * q + 1.f / 9.f;
+  a = a * q + 1.f / 7.f;
+  a = a * q + 1.f / 5.f;
+  a = a * q + 1.f / 3.f;
+  a = a * q + 1.f;
+  return fmaxf(z, 0.f) + 2.f * s * a;
+}
 // exp of x <= 0, to the last bit near 1: a slow decay is the distance from 1, and its rounding adds up over a sequence
 __device__ __forceinline__ float decay_f(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
 __device__ __forceinline__ float softcap_f(float z, float cap) { return cap * tanhf(z / cap); }

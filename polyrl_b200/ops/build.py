@@ -26,7 +26,7 @@ BUILD = CSRC / "build"
 MODULES: dict[str, dict] = {
     "_serve": {"bindings": "bindings_serve.cpp",
                "cu": ["gemm_tcgen05.cu", "gemm2.cu", "attn_fwd.cu", "decode_attn.cu", "sampling.cu", "mix_elem.cu", "mix_scan.cu", "mix_chunk.cu", "mix_chunk_tc.cu", "mix_delta.cu", "mix_latent.cu",
-                      "mix_window.cu", "mix_maps.cu", "mix_block.cu", "mix_experts.cu", "mix_streams.cu", "mix_selective.cu"]},
+                      "mix_window.cu", "mix_maps.cu", "mix_block.cu", "mix_experts.cu", "mix_streams.cu", "mix_selective.cu", "mix_gla.cu"]},
     "_C": {"bindings": "bindings.cpp",
            "cu": ["gemm_tcgen05.cu", "gemm2.cu", "skinny_gemm.cu", "decode_gemm.cu", "vmm.cu", "linear_ce.cu", "ag_gemm.cu", "elementwise.cu",
                   "optim.cu", "attn_bwd.cu", "attn_fwd.cu", "p2p.cu", "nvls.cu"]},

@@ -453,6 +453,9 @@ def scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: Ga
     if b.n_long and mode == DELTA and chunk and _C().mix_delta_chunk_ok(q, k, v, S):
         _C().mix_delta_chunk_(q, k, v, gates.g0, gates.g1, gates.b0, gates.a_log, qscale, S, b.cu[:b.n_long + 1], b.start[:b.n_long],
                               b.slot[:b.n_long], ctr, out)
+    elif b.n_long and mode == GLA and chunk and _C().mix_gla_chunk_(q, k, v, gates.g0, gates.b0, qscale, gates.cap, S, b.cu[:b.n_long + 1], b.start[:b.n_long],
+                                                                    b.slot[:b.n_long], ctr, out):
+        pass
     elif b.n_long:
         chunk = chunk and mode not in (DELTA, GLA) and _C().mix_chunk_supported(N)
         run(0, b.n_long, (3 if b.max_long >= TC_MIN else 2) if chunk else 0)

@@ -24,7 +24,7 @@ def _peaks() -> tuple[float, float, str]:
 
 def models(layers: int, design: str) -> dict:
     """The mixer stack and its closest stacks at the same width, feed-forward width and depth: llama with latent attention (MLA) beside
-    ludesun, ludesun beside lanilix, llama beside all; beside mabedra lanilix and a llama stack with the same experts in the same layers."""
+    ludesun, ludesun beside lanilix, llama beside all; beside mabedra lanilix and a llama stack with the same experts in the same layers; beside dubazen mabedra and the latter with experts in every layer."""
     from ..models import ModelConfig, get_model_config
 
     def stack(name):
@@ -34,9 +34,12 @@ def models(layers: int, design: str) -> dict:
     hy = stack("ludesun-4b")
     base = dict(family="llama", vocab_size=hy.vocab_size, hidden_size=hy.hidden_size, intermediate_size=hy.intermediate_size, num_layers=layers, num_heads=32,
                 max_position_embeddings=16384, rope_theta=500000.0, rms_norm_eps=1e-5, eos_token_id=-1)
+    if design in ("mabedra", "dubazen"):
+        moe = dict(num_experts=16, num_experts_per_tok=2, moe_intermediate_size=2048, shared_expert_intermediate_size=4096, norm_topk_prob=design == "dubazen",
+                   dense_layers=tuple(range(0, layers, 4)) if design == "mabedra" else ())
+    if design == "dubazen":
+        return {"dubazen": stack("dubazen-7b"), "mabedra": stack("mabedra-7b"), "llama with experts": ModelConfig(**base, num_kv_heads=8, **moe)}
     if design == "mabedra":
-        moe = dict(num_experts=16, num_experts_per_tok=2, moe_intermediate_size=2048, shared_expert_intermediate_size=4096, norm_topk_prob=False,
-                   dense_layers=tuple(range(0, layers, 4)))
         return {"mabedra": stack("mabedra-7b"), "lanilix": stack("lanilix-4b"), "llama": ModelConfig(**base, num_kv_heads=8),
                 "llama with experts": ModelConfig(**base, num_kv_heads=8, **moe)}
     if design == "lanilix":
@@ -346,6 +349,121 @@ def run_kernels_mabedra(args) -> list[dict]:
     return K.rows
 
 
+def run_kernels_dubazen(args) -> list[dict]:
+    """Layer sizes of ``dubazen-7b``."""
+    from .. import ops
+    from ..ops import mixers as M
+    from ..ops.attention import attention_varlen
+
+    C, K = ops.ext(), _Kernels(args)
+    dev, rnd, rec = K.dev, K.rnd, K.rec
+    W = 4096
+    f32 = dict(device=dev, dtype=torch.float32)
+    for tag, lens, start in _SHAPES:
+        b, blocks = K.batch(lens, start)
+        t, n, L, dec = sum(lens), len(lens), lens[0], lens[0] == 1
+        rw = (2 if dec else 1) * n
+        # ---- recurrences
+        I, N = 8192, 16
+        p, x, dt, bc = rnd(t, 2 * I), rnd(t, I), rnd(t, I, dtype=torch.float32), rnd(t, 256 + 2 * N)
+        vec, a_neg, state = torch.full((I,), -2.0, **f32), -torch.arange(1, N + 1, **f32).expand(I, N).contiguous(), torch.zeros(n + 1, I, N, **f32)
+        rec("selective scan", "recurrence ssd", tag, lambda: M.selective_scan(x, dt, bc[:, 256:256 + N], bc[:, 256 + N:], p[:, I:], vec, a_neg, vec, state, b),
+            t * (I * 10 + 4 * N) + rw * I * N * 4)
+        cw, cb, cst = torch.randn(4, I, device=dev), torch.randn(I, device=dev), torch.zeros(n + 1, 3, I, device=dev, dtype=torch.bfloat16)
+        rec("existing: conv + silu", "conv + silu", tag, lambda: M.conv_silu(p[:, :I], cw, cb, cst, b), t * I * 4 + n * 6 * I * 2)
+        del p, x, dt, bc, state
+        H, N, V = 16, 128, 256
+        cache, q, k, v, z = {"S": torch.zeros(n + 1, H, N, V, **f32)}, rnd(t, H * N), rnd(t, H * N), rnd(t, H * V), rnd(t, H * N, dtype=torch.float32)
+        gates = M.Gates(z, b0=torch.full((H * N,), 3.0, **f32), cap=16.0)
+        # per token and head: two products with the state, half a chunk of 64 earlier tokens for each of Q K' and P V
+        rec("recurrence gla", "recurrence delta", tag, lambda: M.scan(M.GLA, q, k, v, gates, N ** -0.5, cache, b), t * H * (2 * N * 2 + 2 * V * 2 + N * 4) + rw * H * N * V * 4,
+            0 if dec else t * H * (4 * N * V + 64 * (N + V)))
+        o, g, gn = rnd(t, H * V), rnd(t, H * V), torch.ones(H * V, device=dev)
+        rec("existing: gated norm per head", "gated norm", tag, lambda: M.gated_norm(o, g, gn, H, 1e-6, M.SILU_LAST), t * H * V * 6)
+        del z
+        H, N, V = 32, 128, 128
+        q, k, v, cache = rnd(t, H * N), rnd(t, H * N), rnd(t, H * V), {"S": torch.zeros(n + 1, H, N, V, **f32)}
+        light = M.Gates(a_log=torch.linspace(-1, -0.001, H, **f32), raw=dec)
+        rec("recurrence with constant decay" + (" + silu" if dec else ""), "recurrence ssd", tag, lambda: M.scan(M.DECAY, q, k, v, light, 1.0, cache, b),
+            t * H * (2 * N + 2 * V) * 2 + rw * H * N * V * 4, 0 if dec else t * H * (64 * (N + V) + 4 * N * V))
+        gates = M.Gates(rnd(t, H, dtype=torch.float32), rnd(t, H, dtype=torch.float32), torch.full((H,), -2.0, **f32), None, torch.linspace(-4, 1, H, **f32))
+        rec("existing: recurrence delta", "recurrence delta", tag, lambda: M.scan(M.DELTA, q, k, v, gates, N ** -0.5, cache, b),
+            t * (2 * H * N * 2 + 2 * H * V * 2 + 2 * H * 4) + rw * H * N * V * 4, 0 if dec else t * H * (6 * N * V + 64 * (2 * N + 2 * V)))
+        H2, V2, N2, G2 = 128, 64, 128, 8
+        cache2 = {"S": torch.zeros(n + 1, H2, N2, V2, **f32)}
+        q2, k2, v2 = rnd(t, G2 * N2), rnd(t, G2 * N2, scale=N2 ** -0.5), rnd(t, H2 * V2)
+        gates2 = M.Gates(rnd(t, H2, dtype=torch.float32), None, torch.full((H2,), -2.0, **f32), None, torch.linspace(-2, 1, H2, **f32), torch.ones(H2, **f32))
+        rec("existing: recurrence ssd", "recurrence ssd", tag, lambda: M.scan(M.SSD, q2, k2, v2, gates2, 1.0, cache2, b),
+            t * (2 * G2 * N2 * 2 + 2 * H2 * V2 * 2 + H2 * 4) + rw * H2 * N2 * V2 * 4, 0 if dec else t * H2 * (64 * (N2 + V2) + 4 * N2 * V2))
+        if not dec:
+            hb, wq = rnd(t, W), rnd(H * (2 * N + V), W, scale=W ** -0.5)
+            rec("projection + silu", "gate / up + swiglu", tag, lambda: M.linear_silu(hb, wq), (t * W + wq.numel() + t * wq.shape[0]) * 2, 2.0 * t * wq.numel())
+            rec("existing: projection + gelu", "gate / up + swiglu", tag, lambda: M.linear_gelu(hb, wq), (t * W + wq.numel() + t * wq.shape[0]) * 2, 2.0 * t * wq.numel())
+            del hb, wq
+        del cache, cache2, q, k, v, q2, k2, v2, o
+        # ---- attention
+        H, G, D, rd = 32, 8, 128, 64
+        cols = (H + 2 * G) * D
+        p, bias, freq, vfreq = rnd(t, cols), torch.zeros(cols, **f32), M.rope_frequencies(rd, 5e5, dev), M.rope_frequencies(D, 5e5, dev)
+        kp, vp, sink = rnd(blocks, G, 16, D), rnd(blocks, G, 16, D), torch.zeros(H, **f32)
+        rec("attention rows: bias, rotation, norms, rotated values, cache write", "query / key rows", tag, lambda: M.turn_prep(p, bias, H, D, D, freq, vfreq, kp, vp, b, 1e-6, not dec),
+            t * (cols * 2 + H * D * 2 + (1 if dec else 2) * G * 2 * D * 2))
+        wq, wk = torch.ones(H * D, **f32), torch.ones(G * D, **f32)
+        rec("existing: query / key norm, rotation, cache write", "query / key rows", tag, lambda: M.qk_prep(p, H, D, wq, wk, freq, kp, vp, b, 1e-6, not dec),
+            t * ((H + G) * D * 2 + (H + (2 if dec else 4) * G) * D * 2))
+        q, o, gate = rnd(t, H, D), rnd(t, H, D), rnd(t, H * D)
+        out = torch.empty_like(gate)
+        rec("outputs turned back + gate", "gated norm", tag, lambda: M.turn_back(o, gate, vfreq, b.pos, 1.0, out), t * H * D * 6)
+        if dec:
+            rec("paged attention + sink", "paged decode", tag, lambda: M.sink_attention(q, kp, vp, b.table, None, b.kv_len, 0.088, sink, 2048), t * 2048 * G * D * 4)
+            rec("existing: paged decode (GQA 32/8)", "paged decode", tag,
+                lambda: ops.paged_decode_attention(q.view(t, H * D), kp, vp, b.table, b.kv_len, H, G, D, 0.088, max_len=2048), t * 2048 * G * D * 4)
+        else:
+            k, v = rnd(t, G, D), rnd(t, G, D)
+            rec("packed attention + sink", "packed attention", tag, lambda: M.sink_attention_varlen(q, k, v, b.cu, b.cu, 0.088, sink), t * (2 * H + 2 * G) * D * 2,
+                n * L * L / 2 * H * 4 * D)
+            rec("existing: attention_varlen (GQA 32/8)", "packed attention", tag, lambda: attention_varlen(q, k, v, b.cu, L, True, 0.088), t * (2 * H + 2 * G) * D * 2,
+                n * L * L / 2 * H * 4 * D)
+            del k, v
+        del p, kp, vp, q, o, gate, out
+        # ---- residual streams
+        S = 4
+        emb, ids, one, wn = rnd(128256, W), torch.randint(0, 128256, (t,), device=dev), torch.ones(1, **f32), torch.ones(W, **f32)
+        win, mix, ov = torch.full((S,), 0.25, **f32), torch.eye(S, **f32), torch.ones(S, **f32)
+        rec("embedding + norm, streams", "norm + residual add", tag, lambda: M.streams_embed(ids, emb, 64.0, S, win, one, 1e-6), t * W * 8)
+        rec("existing: embedding + norm", "norm + residual add", tag, lambda: M.embed(ids, emb, wn, 1e-6), t * W * 8)
+        del emb
+        xs, y = torch.randn(t, S, W, **f32), rnd(t, W)
+        rec("four streams: mix, add, next norm", "norm + residual add", tag, lambda: M.streams_add(xs, y, wn, None, mix, ov, win, one, 1e-6), t * W * (8 * S + 4))
+        x1 = xs[:, :1].contiguous()
+        rec("four streams, first sublayer", "norm + residual add", tag, lambda: M.streams_add(x1, y, wn, None, mix, ov, win, one, 1e-6), t * W * (4 + 4 * S + 4))
+        rec("four streams, sum and norm", "norm + residual add", tag, lambda: M.streams_sum(xs, y, wn, None, mix, ov, wn, 1e-6), t * W * (4 * S + 8))
+        x32 = torch.randn(t, W, **f32)
+        rec("existing: norm + residual add + next norm", "norm + residual add", tag, lambda: M.norm_add_(y, x32, wn, 1e-6, wn), t * W * 12)
+        del x32, x1
+        # ---- experts
+        E, top, F = 16, 2, 2048
+        h, router = rnd(t, W), rnd(E, W, scale=W ** -0.5)
+        wgu, wd = rnd(E * 2 * F, W, scale=W ** -0.5), rnd(E * W, F, scale=F ** -0.5)
+        logits, ctr = M.linear_f32(h, router), M._counter(dev, E + 1, "route")
+        pick, score, rank, plan = C.mix_route(logits, top, ctr, True)
+        xr, pos = C.mix_expert_rows(h, pick, None, rank, plan, E)
+        a = C.gemm_experts(xr, wgu, plan, E, 2, 7.0, 1.702)
+        rec("routing, softmax", "routing", tag, lambda: C.mix_route(logits, top, ctr, True), t * (E * 4 + top * 12))
+        rec("existing: routing, sigmoid", "routing", tag, lambda: C.mix_route(logits, top, ctr), t * (E * 4 + top * 12))
+        rec("rows in the experts' order", "rows in the experts' order", tag, lambda: C.mix_expert_rows(h, pick, None, rank, plan, E), t * W * 2 * (1 + top))
+        rec("experts: gate / up + clamped glu", "experts: gate / up", tag, lambda: C.gemm_experts(xr, wgu, plan, E, 2, 7.0, 1.702), (E * 2 * F * W + t * top * (W + F)) * 2,
+            4.0 * t * top * W * F)
+        rec("existing: experts: gate / up + silu glu", "experts: gate / up", tag, lambda: C.gemm_experts(xr, wgu, plan, E, 1), (E * 2 * F * W + t * top * (W + F)) * 2,
+            4.0 * t * top * W * F)
+        rec("existing: experts: down", "experts: down", tag, lambda: C.gemm_experts(a, wd, plan, E, 0), (E * F * W + t * top * (W + F)) * 2, 2.0 * t * top * W * F)
+        routed = M.Routed(C.gemm_experts(a, wd, plan, E, 0), pos, score)
+        rec("four streams with routed rows", "norm + residual add", tag, lambda: M.streams_add(xs, y, None, routed, mix, ov, win, one, 1e-6), t * W * (8 * S + 4 + 2 * top))
+        del xs, y, xr, a, routed, wgu, wd, h
+        torch.cuda.empty_cache()
+    return K.rows
+
+
 def run_kernels(args) -> list[dict]:
     from .. import ops
     from ..models import get_model_config, mla
@@ -444,7 +562,7 @@ def main(args) -> int:
         return 1
     args.steps_serving = max(5, args.steps)
     out = {"workload": "serving", "dtype": "bf16", "data": "random weights and tokens", "device": torch.cuda.get_device_name(), "peaks": _peaks()[2]}
-    kernels = {"ludesun": run_kernels, "lanilix": run_kernels_lanilix, "mabedra": run_kernels_mabedra}[args.serving_design]
+    kernels = {"ludesun": run_kernels, "lanilix": run_kernels_lanilix, "mabedra": run_kernels_mabedra, "dubazen": run_kernels_dubazen}[args.serving_design]
     out["kernels" if args.kernels else "models"] = kernels(args) if args.kernels else run_models(args)
     if os.environ.get("BENCH_SERVING_OUT"):
         Path(os.environ["BENCH_SERVING_OUT"]).write_text(json.dumps(out, indent=1))
