@@ -179,7 +179,7 @@ def test_step_sizes_of_every_magnitude():
 
 # ---------------------------------------------------------------------------------------------- attention with rotated values
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("H,G,d,e,rot", [(1, 1, 1, 2, 0), (6, 2, 10, 14, 6), (4, 4, 24, 40, 24), (8, 2, 64, 128, 32), (8, 1, 128, 48, 32), (4, 2, 72, 48, 0), (20, 1, 16, 32, 8),
+@pytest.mark.parametrize("H,G,d,e,rot", [(1, 1, 1, 2, 0), (6, 2, 10, 14, 6), (4, 4, 24, 40, 24), (8, 2, 64, 128, 32), (6, 1, 128, 80, 48), (4, 2, 72, 48, 0), (20, 1, 16, 32, 8),
                                          (3, 3, 136, 16, 16), (6, 3, 128, 128, 128), (4, 2, 192, 96, 64), (2, 1, 200, 64, 16), (2, 2, 48, 200, 48), (2, 1, 160, 16, 160)])
 def test_attention(dtype, H, G, d, e, rot):
     """Biases, rotations, norms, sink, gate, cache writes and every attention kernel: a prompt, a portion beside single tokens, single tokens."""
