@@ -615,35 +615,14 @@ mix_delta_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (w == 8) { tc_fence_after(); tmem_dealloc(sm.tmem, 512); }
 }
 
-using DeltaEncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
-                                   const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-// rows [tokens, heads * width] of pitch ld -> boxes of 64 tokens x 1 head x box columns, zeros beyond the head's width
-static int delta_tmap(CUtensorMap* m, const void* ptr, int64_t tokens, int heads, int width, int64_t ld, int box, bool swizzle) {
-  ensure_thread_ctx();
-  static DeltaEncodeFn fn = nullptr;
-  if (!fn) {
-    void* q = nullptr;
-    cudaDriverEntryPointQueryResult qr;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &q, cudaEnableDefault, &qr) != cudaSuccess || !q) return -1;
-    fn = reinterpret_cast<DeltaEncodeFn>(q);
-  }
-  const cuuint64_t dim[3] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(tokens)};
-  const cuuint64_t stride[2] = {static_cast<cuuint64_t>(width) * 2, static_cast<cuuint64_t>(ld) * 2};
-  const cuuint32_t bx[3] = {static_cast<cuuint32_t>(box), 1, kDc}, one[3] = {1, 1, 1};
-  const CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dim, stride, bx, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        swizzle ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? 0 : -static_cast<int>(r);
-}
-
 template <int NB>
 static int run_delta(const ScanParams& p, int64_t tokens, int total_chunks, uint8_t* work, float* gates, int32_t* err, cudaStream_t st) {
   constexpr int smem1 = 4 * kDcTile + 2 * kDc * kDpLd * 4 + 1024, smem2 = DeltaTc<NB>::OFF_F + static_cast<int>(sizeof(DeltaShared)) + 1024;
   static_assert(smem2 <= 232448, "shared memory");
   CUtensorMap tmQ, tmK, tmV, tmO;
   const int G = p.H / p.rep;
-  if (delta_tmap(&tmQ, p.q, tokens, G, p.N, p.ldq, 64, true) || delta_tmap(&tmK, p.k, tokens, G, p.N, p.ldk, 64, true) ||
-      delta_tmap(&tmV, p.v, tokens, p.H, p.V, p.ldv, 128, false) || delta_tmap(&tmO, p.out, tokens, p.H, p.V, p.ldo, 128, false))
+  if (tc_tokens_tmap(&tmQ, p.q, tokens, G, p.N, p.ldq, kDc, 64, true) || tc_tokens_tmap(&tmK, p.k, tokens, G, p.N, p.ldk, kDc, 64, true) ||
+      tc_tokens_tmap(&tmV, p.v, tokens, p.H, p.V, p.ldv, kDc, 128, false) || tc_tokens_tmap(&tmO, p.out, tokens, p.H, p.V, p.ldo, kDc, 128, false))
     return -261;
   static bool attr = false;
   if (!attr) {

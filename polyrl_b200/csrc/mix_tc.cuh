@@ -1,4 +1,4 @@
-// polyrl_b200 — pieces of the tcgen05 recurrence kernels: bounded barrier waits, 128B-swizzled bf16 tiles, hi + lo bf16 pairs.
+// polyrl_b200 — pieces of the tcgen05 recurrence kernels: bounded barrier waits, 128B-swizzled bf16 tiles, hi + lo bf16 pairs, tensor maps.
 #pragma once
 #include "mixers.cuh"
 
@@ -38,6 +38,27 @@ __device__ __forceinline__ void tc_split(float a, float b, uint32_t& hi, uint32_
   hi = pack_bf16(a, b);
   const float2 h = unpack_bf16(hi);
   lo = pack_bf16(a - h.x, b - h.y);
+}
+
+using TcEncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// rows [tokens, heads * width] of pitch ld -> boxes of `rows` tokens x 1 head x box columns, zeros beyond the head's width
+inline int tc_tokens_tmap(CUtensorMap* m, const void* ptr, int64_t tokens, int heads, int width, int64_t ld, int rows, int box, bool swizzle) {
+  ensure_thread_ctx();
+  static TcEncodeFn fn = nullptr;
+  if (!fn) {
+    void* q = nullptr;
+    cudaDriverEntryPointQueryResult qr;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &q, cudaEnableDefault, &qr) != cudaSuccess || !q) return -1;
+    fn = reinterpret_cast<TcEncodeFn>(q);
+  }
+  const cuuint64_t dim[3] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(tokens)};
+  const cuuint64_t stride[2] = {static_cast<cuuint64_t>(width) * 2, static_cast<cuuint64_t>(ld) * 2};
+  const cuuint32_t bx[3] = {static_cast<cuuint32_t>(box), 1, static_cast<cuuint32_t>(rows)}, one[3] = {1, 1, 1};
+  const CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dim, stride, bx, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        swizzle ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -static_cast<int>(r);
 }
 
 }  // namespace prl

@@ -2,7 +2,7 @@
 
 Families: ``llama`` (Llama-2/3, Qwen2/2.5/3 — RMSNorm, RoPE, SwiGLU, GQA, optional qkv bias / qk-norm) and
 ``gpt2`` (LayerNorm, learned positions, GELU MLP, biases); ``hybrid`` (stacks whose layers each pick a sequence mixer,
-models/hybrid.py: Ludesun).  Shapes for the presets follow the public
+models/hybrid.py; the designs are in models/stacks.py).  Shapes for the presets follow the public
 HF configs (the reference loads the same families through HF AutoModel:
 3rdparty/verl/verl/workers/fsdp_workers.py:269-577).
 """
